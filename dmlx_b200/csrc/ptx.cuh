@@ -96,6 +96,13 @@ __device__ __forceinline__ void fence_proxy_async_smem() {
   asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
 }
 
+// Returns once every lane's shared-memory loads that `mix` was formed from have delivered their values: the warp-wide
+// reduction needs them.  To be called before one lane releases a slot that the async proxy will refill; the arrival alone
+// does not wait for loads other lanes still have in flight.
+__device__ __forceinline__ void warp_loads_landed(uint32_t mix) {
+  if (__reduce_xor_sync(0xffffffffu, mix) == 0x9E3779B9u) __nanosleep(20);  // (the branch only ties the result down)
+}
+
 // ---- tcgen05: tensor memory + MMA --------------------------------------------------------------
 __device__ __forceinline__ void tmem_alloc(uint32_t* dst_smem, uint32_t ncols) {
   asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(dst_smem)),

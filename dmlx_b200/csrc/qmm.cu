@@ -875,13 +875,13 @@ __global__ void __launch_bounds__(kTc2Threads, 1) qmm_tc2_kernel(const __grid_co
       if (!ok) break;
       if (!kDense) {
         uint4 raw = make_uint4(0u, 0u, 0u, 0u);
-        __nv_bfloat162 s2, b2;
+        __nv_bfloat162 s2 = __float2bfloat162_rn(0.f), b2 = s2;
         if (tile < n_tiles) {
           const unsigned char* blk = raw_blk(sr, tile);
           raw = reinterpret_cast<const uint4*>(blk + plane * kPlaneBytes)[r];
           row_params<MODE>(blk, r, plane, s2, b2);
         }
-        __syncwarp();
+        ptx::warp_loads_landed(raw.x ^ raw.y ^ raw.z ^ raw.w ^ *reinterpret_cast<const uint32_t*>(&s2) ^ *reinterpret_cast<const uint32_t*>(&b2));
         if (lane == 0) ptx::mbar_arrive(&raw_free[sr]);  // this warp's share of the blocks is in registers
         ok = ptx::mbar_wait(&mma_done[s], ph ^ 1u);     // the stage's MMA tiles may be overwritten
         if (!ok) break;
