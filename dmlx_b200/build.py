@@ -8,6 +8,7 @@ library in dmlx_b200/; both are ignored by git but travel with the working tree.
 """
 from __future__ import annotations
 
+import fcntl
 import os
 import subprocess
 import sys
@@ -51,7 +52,14 @@ def _compile(src: str, verbose: bool) -> str:
 
 
 def build(force: bool = False, verbose: bool = False) -> str:
+    """Compiles what is out of date; processes that start at the same time build once (a lock in the object folder)."""
     os.makedirs(OBJ_DIR, exist_ok=True)
+    with open(os.path.join(OBJ_DIR, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build(force, verbose)
+
+
+def _build(force: bool, verbose: bool) -> str:
     dep_t = _deps_mtime()
     todo, objs = [], []
     for src in sources():
@@ -64,10 +72,12 @@ def build(force: bool = False, verbose: bool = False) -> str:
         with ThreadPoolExecutor(max_workers=min(8, len(todo))) as ex:
             list(ex.map(lambda s: _compile(s, verbose), todo))
     if todo or not os.path.exists(LIB):
-        cmd = ["nvcc", "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", LIB, *objs]
+        tmp = LIB + ".tmp"
+        cmd = ["nvcc", "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", tmp, *objs]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+        os.replace(tmp, LIB)
     return LIB
 
 
