@@ -256,6 +256,51 @@ _sig("b200_ep_abort", i32, vp)
 _sig("b200_ep_watch", i32, P(EpWatchOps), i32, i32)
 
 
+class KvLayer(C.Structure):
+    _fields_ = [(n, i32) for n in ("n_kv_heads", "key_dim", "value_dim")]
+
+
+class ModelInfo(C.Structure):
+    _fields_ = [(n, i32) for n in ("vocab", "max_rows", "max_reqs", "max_seqs", "logits_f32")]
+
+
+class DecoderLayer(C.Structure):
+    _fields_ = [(n, i32) for n in ("n_heads", "n_kv_heads", "key_dim", "value_dim", "window", "ffn", "flags")] + [("scale", f32)]
+
+
+class DecoderConfig(C.Structure):
+    _fields_ = [(n, i32) for n in ("n_layers", "hidden", "vocab", "loop_start", "loop_stop", "loop_times", "dtype", "max_rows", "max_reqs",
+                                   "max_seqs")] + [("norm_eps", f32), ("embed_scale", f32)]
+
+
+_sig("b200_kv_create_layers", i32, P(KvConfig), P(KvLayer), P(vp))
+_sig("b200_argmax_f32", i32, vp, i32, i32, vp, vp)
+_sig("b200_qmm_f32", i32, vp, vp, i32, vp, i32, i32, i32, vp)
+_sig("b200_llama_model", vp, vp)
+_sig("b200_model_get_info", None, vp, P(ModelInfo))
+_sig("b200_model_step", i32, vp, vp, vp, i32, vp, i32, vp, P(i32), vp)
+_sig("b200_model_forward", i32, vp, vp, vp, i32, i32, vp, vp)
+_sig("b200_model_device_buffers", None, vp, P(vp), P(vp), P(vp))
+_sig("b200_model_set_samplers", i32, vp, P(SampleParams), i32)
+_sig("b200_model_last_logprobs", i32, vp, P(f32), i32)
+_sig("b200_model_launch_count", C.c_int64, vp)
+_sig("b200_model_enable_graphs", None, vp, i32)
+_sig("b200_model_profile_enable", None, vp, i32)
+_sig("b200_model_profile_collect", i32, vp, P(C.c_double), P(C.c_int64))
+_sig("b200_model_want_logits", i32, vp, P(i32), i32)
+_sig("b200_model_logits", i32, vp, i32, i32, P(f32))
+_sig("b200_decoder_create", i32, P(DecoderConfig), P(DecoderLayer), P(vp))
+_sig("b200_decoder_destroy", None, vp)
+_sig("b200_decoder_set_tensor", i32, vp, i32, i32, vp, u64)
+_sig("b200_decoder_finalize", i32, vp)
+_sig("b200_decoder_random_init", i32, vp, u32)
+_sig("b200_decoder_cache_layers", i32, vp, P(KvLayer), i32)
+_sig("b200_decoder_record_layers", i32, vp, i32)
+_sig("b200_decoder_recorded_layers", i32, vp, i32, P(f32))
+_sig("b200_decoder_set_attn_mma", None, vp, i32)
+_sig("b200_decoder_model", vp, vp)
+_sig("b200_engine_create_model", vp, vp, vp, u64)
+
 _sig("b200_request_prompt", u64, vp, P(u32), u64)
 _sig("b200_engine_create", vp, vp, vp, u64)
 _sig("b200_engine_destroy", None, vp)

@@ -1,0 +1,695 @@
+// Paged attention for layers with a sliding window, a distance bias and a learned sink, keys and values of different
+// widths, and any GQA group; decode rows and prefill chunks through one path.
+//
+// Rows are grouped: consecutive rows of one sequence (a prefill chunk) share a pass over the pages, a decoded token is a
+// group of its own.  The 16 rows of an MMA tile carry (token of the group) x (query head of the kv head's GQA group), so
+// a group holds floor(16 / G) tokens; groups with more than 16 query heads per kv head are cut into head blocks of 16.
+// A group's key range is [first row's window start, last row's position]; it is cut into chunks of pages, and a work item
+// is (chunk, kv head, head block), walked by a persistent grid whose warps are independent workers (each with its own
+// ring of TMA-staged pages, as in paged_attn.cu).  A group of one chunk is normalised and written by the kernel itself; the
+// partial (max, sum, out) of longer ones go through scratch to a combine pass.  The sink joins the denominator exactly
+// once, where a row is normalised.
+//
+// Scores, biases and softmax are f32.  The weights enter the P V product as two bf16 terms (the rounded weight and what
+// the rounding left over), so they carry 16 bits of mantissa instead of 8.
+//
+// attn_simt_kernel is the same contract on CUDA cores for any width and for f32 pools.
+#include <cuda_bf16.h>
+
+#include <algorithm>
+#include <cmath>
+
+#include "common.h"
+#include "kv_pool.cuh"
+#include "ptx.cuh"
+#include "tma.cuh"
+
+namespace {
+
+constexpr int kStages = 3;
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr float kNone = -1e30f;  // running maximum before any key
+
+struct WinArgs {
+  KvDev d;
+  KvLayerDev L;
+  const __nv_bfloat16* q;
+  int q_stride;
+  const int* row_seq;
+  const int* row_ctx;
+  int total_rows, n_q_heads, window;
+  int G, head_block, n_blocks;  // query heads per kv head; heads of one MMA tile; tiles per kv head
+  const int *group_first, *chunk_start, *part_base, *row_group, *hdr;
+  float* part_o;   // [slot][q head][L.vd]
+  float* part_ml;  // [slot][q head][2]
+  float scale_log2;
+  const float *slopes, *sinks;
+  __nv_bfloat16* out;
+  int out_stride;
+};
+
+// ---- plan ------------------------------------------------------------------------------------------------
+template <bool MAX>
+__device__ int scan_incl(int v, int* warp_buf) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  int inc = v;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int t = __shfl_up_sync(0xffffffffu, inc, o);
+    if (lane >= o) inc = MAX ? max(inc, t) : inc + t;
+  }
+  if (lane == 31) warp_buf[warp] = inc;
+  __syncthreads();
+  if (warp == 0) {
+    int w = lane < (int)(blockDim.x >> 5) ? warp_buf[lane] : (MAX ? -1 : 0);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int t = __shfl_up_sync(0xffffffffu, w, o);
+      if (lane >= o) w = MAX ? max(w, t) : w + t;
+    }
+    const int ex = __shfl_up_sync(0xffffffffu, w, 1);
+    warp_buf[lane] = lane == 0 ? (MAX ? -1 : 0) : ex;
+  }
+  __syncthreads();
+  const int r = MAX ? max(warp_buf[warp], inc) : warp_buf[warp] + inc;
+  __syncthreads();
+  return r;
+}
+
+__device__ __forceinline__ int first_key(int ctx, int window) { return window > 0 ? max(0, ctx - window) : 0; }
+
+// Pages of a group's key range.
+__device__ __forceinline__ int group_pages(int ctx_first, int ctx_last, int window, int page_size) {
+  return (max(ctx_last, 1) - 1) / page_size - first_key(ctx_first, window) / page_size + 1;
+}
+
+// Groups of rows and their chunks.  The chunk length (pages) follows the batch: long chunks cost fewer partial sums,
+// short ones give a small batch enough work items for the grid; prefill batches of many groups take one chunk per group.
+// It doubles until the partial slots fit the scratch (with one chunk per group there are none), so a step always fits.
+__global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict__ row_seq, const int* __restrict__ row_ctx, int total_rows,
+                                                           int page_size, int window, int q_tokens, int single_chunk, int items_per_chunk,
+                                                           int n_workers, int forced_ppc, int max_slots, int* __restrict__ group_first,
+                                                           int* __restrict__ chunk_start, int* __restrict__ part_base,
+                                                           int* __restrict__ row_group, int* __restrict__ hdr) {
+  __shared__ int warp_buf[32];
+  __shared__ int carry_start, carry_groups, carry_chunks, carry_slots;
+  const int tid = threadIdx.x;
+  if (tid == 0) { carry_start = -1; carry_groups = 0; }
+  __syncthreads();
+  for (int base = 0; base < total_rows; base += blockDim.x) {
+    const int i = base + tid;
+    const bool valid = i < total_rows;
+    const bool joinable = valid && i > 0 && row_seq[i] == row_seq[i - 1] && row_ctx[i] == row_ctx[i - 1] + 1;
+    const int run_start = max(scan_incl<true>(valid && !joinable ? i : -1, warp_buf), carry_start);
+    const int head = valid && ((i - run_start) % q_tokens == 0) ? 1 : 0;
+    const int heads_incl = scan_incl<false>(head, warp_buf);
+    const int gid = carry_groups + heads_incl - 1;
+    if (valid) {
+      row_group[i] = gid;
+      if (head) group_first[gid] = i;
+    }
+    __syncthreads();
+    if (tid == blockDim.x - 1) { carry_start = run_start; carry_groups += heads_incl; }
+    __syncthreads();
+  }
+  const int n_groups = carry_groups;
+  if (tid == 0) group_first[n_groups] = total_rows;
+  __syncthreads();
+  int ppc = 0x3fffffff;
+  if (forced_ppc > 0) {
+    ppc = forced_ppc;
+  } else if (!single_chunk) {
+    int pages = 0;
+    for (int g = tid; g < n_groups; g += blockDim.x)
+      pages += group_pages(row_ctx[group_first[g]], row_ctx[group_first[g + 1] - 1], window, page_size);
+    // a sum of at most 2^20 rows x 2^15 pages would overflow; saturate per thread
+    pages = min(max(pages, 0), 0x7fffffff / 1024);
+    const int total = scan_incl<false>(pages, warp_buf);
+    if (tid == blockDim.x - 1) carry_chunks = total;
+    __syncthreads();
+    const int all = carry_chunks, mean = all / max(n_groups, 1);
+    const long long spread = (long long)all * items_per_chunk / (2 * n_workers);
+    ppc = (int)min((long long)(mean < 96 ? 8 : (mean < 192 ? 16 : 32)), max(spread, 4ll));
+    __syncthreads();
+  }
+  for (int round = 0; round < 32; ++round) {
+    if (tid == 0) { carry_chunks = 0; carry_slots = 0; }
+    __syncthreads();
+    for (int base = 0; base < n_groups; base += blockDim.x) {
+      const int g = base + tid;
+      int chunks = 0, slots = 0;
+      if (g < n_groups) {
+        const int first = group_first[g], next = group_first[g + 1];
+        const int pages = group_pages(row_ctx[first], row_ctx[next - 1], window, page_size);
+        chunks = pages / ppc + (pages % ppc ? 1 : 0);
+        slots = chunks > 1 ? chunks * (next - first) : 0;
+      }
+      const int c_incl = scan_incl<false>(chunks, warp_buf);
+      const int s_incl = scan_incl<false>(slots, warp_buf);
+      if (g < n_groups) {
+        chunk_start[g] = carry_chunks + c_incl - chunks;
+        part_base[g] = slots > 0 ? carry_slots + s_incl - slots : -1;
+      }
+      __syncthreads();
+      if (tid == blockDim.x - 1) { carry_chunks += c_incl; carry_slots += s_incl; }
+      __syncthreads();
+    }
+    if (carry_slots <= max_slots) break;
+    __syncthreads();
+    ppc = ppc > (1 << 28) ? ppc : ppc * 2;
+  }
+  if (tid == 0) {
+    chunk_start[n_groups] = carry_chunks;
+    hdr[0] = n_groups;
+    hdr[1] = ppc;
+  }
+}
+
+// ---- tensor-core kernel ------------------------------------------------------------------------------------
+struct WinItem {
+  int head, block, seq, first_row, n_rows, ctx0, page_begin, page_end, slot0;  // slot0 < 0: the group has one chunk
+};
+
+__device__ __forceinline__ WinItem decode_item(const WinArgs& a, int item, int n_groups, int ppc) {
+  WinItem it;
+  const int per_chunk = a.L.heads * a.n_blocks;
+  const int chunk = item / per_chunk, rest = item - chunk * per_chunk;
+  it.head = rest / a.n_blocks;
+  it.block = rest - it.head * a.n_blocks;
+  int lo = 0, hi = n_groups - 1;  // last group with chunk_start[group] <= chunk
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (a.chunk_start[mid] <= chunk) lo = mid; else hi = mid - 1;
+  }
+  it.first_row = a.group_first[lo];
+  it.n_rows = a.group_first[lo + 1] - it.first_row;
+  it.seq = a.row_seq[it.first_row];
+  it.ctx0 = a.row_ctx[it.first_row];
+  const int c = chunk - a.chunk_start[lo];
+  const int p0 = first_key(it.ctx0, a.window) / a.d.page_size;
+  const int p_end = (it.ctx0 + it.n_rows - 1 - 1) / a.d.page_size + 1;
+  it.page_begin = p0 + (c == 0 ? 0 : c * ppc);
+  it.page_end = ppc < p_end - it.page_begin ? it.page_begin + ppc : p_end;
+  it.slot0 = a.part_base[lo] < 0 ? -1 : a.part_base[lo] + c * it.n_rows;
+  return it;
+}
+
+__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4_trans(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+// (p0, p1) as two bf16 pairs: the rounded values and the remainders.
+__device__ __forceinline__ void split_bf16(float p0, float p1, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
+  const float2 f = __bfloat1622float2(h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(p0 - f.x, p1 - f.y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+// KB, VB: 64-column boxes a key / value row may take (1, 2 or 4); the steps beyond the layer's own widths are skipped.
+template <int KB, int VB, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32, 1)
+    window_attn_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap, WinArgs a) {
+  constexpr int KS = KB * 4;  // 16-column steps of Q K^T
+  constexpr int NO = VB * 8;  // 8-column tiles of the output
+  const int n_kb = (a.L.kd + 63) / 64, n_vb = (a.L.vd + 63) / 64, n_ks = a.L.kd / 16, n_vs = a.L.vd / 16;
+  const int k_tile = n_kb * 4096, stage_bytes = (n_kb + n_vb) * 4096;
+
+  extern __shared__ unsigned char smem_dyn[];
+  unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~(uintptr_t)1023);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int g = lane >> 2, t = lane & 3;
+  unsigned char* my_tiles = smem + (size_t)warp * kStages * stage_bytes;
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + (size_t)WARPS * kStages * stage_bytes) + warp * kStages;
+  const int H = a.L.heads;
+  const int n_groups = a.hdr[0], ppc = a.hdr[1];
+  const int n_items = a.chunk_start[n_groups] * H * a.n_blocks;
+  const int worker = blockIdx.x * WARPS + warp, n_workers = gridDim.x * WARPS;
+
+  if (lane == 0) {
+    for (int s = 0; s < kStages; ++s) ptx::mbar_init(&full_bar[s], 1);
+    ptx::mbar_fence_init();
+  }
+  __syncwarp();
+
+  // producer cursor (all lanes track it, lane 0 issues); the lanes hold the page ids of a window of 32 pages of the
+  // item's chunk, refilled every 32 pages
+  int p_item = worker, p_page = 0, p_end = 0, p_begin = 0, p_head = 0, p_pid = 0, p_seq = 0;
+  uint32_t prod_n = 0;
+  auto producer_enter_item = [&]() {
+    if (p_item < n_items) {
+      const WinItem it = decode_item(a, p_item, n_groups, ppc);
+      p_begin = it.page_begin; p_page = it.page_begin; p_end = it.page_end; p_head = it.head; p_seq = it.seq;
+      const int pg = it.page_begin + lane;
+      if (pg < it.page_end) p_pid = a.d.block_table[(size_t)it.seq * a.d.max_pages_per_seq + pg];
+    }
+  };
+  auto produce_one = [&]() {
+    if (p_item >= n_items) return;
+    const int rel = p_page - p_begin;
+    if (rel > 0 && (rel & 31) == 0) {
+      const int pg = p_page + lane;
+      if (pg < p_end) p_pid = a.d.block_table[(size_t)p_seq * a.d.max_pages_per_seq + pg];
+    }
+    const int pid = __shfl_sync(0xffffffffu, p_pid, rel & 31);
+    const uint32_t s = prod_n % kStages;
+    if (lane == 0) {
+      ptx::fence_proxy_async_smem();
+      unsigned char* kd = my_tiles + (size_t)s * stage_bytes;
+      const int row0 = (pid * H + p_head) * 32;
+      ptx::mbar_expect_tx(&full_bar[s], stage_bytes);
+      for (int b = 0; b < n_kb; ++b) ptx::tma_load_2d(kd + b * 4096, &kmap, b * 64, row0, &full_bar[s]);
+      for (int b = 0; b < n_vb; ++b) ptx::tma_load_2d(kd + k_tile + b * 4096, &vmap, b * 64, row0, &full_bar[s]);
+    }
+    prod_n += 1;
+    p_page += 1;
+    if (p_page >= p_end) {
+      p_item += n_workers;
+      producer_enter_item();
+    }
+  };
+  producer_enter_item();
+  for (int i = 0; i < kStages; ++i) produce_one();
+
+  bool alive = true;
+  uint32_t cons_n = 0;
+  const int ld_r = lane & 7, ld_m = lane >> 3;
+  // MMA rows g and g+8 of this lane: (token of the group, query head within the block)
+  const int hb = a.head_block;
+  const int tokA = g / hb, headA = g - tokA * hb, tokB = (g + 8) / hb, headB = (g + 8) - tokB * hb;
+  for (int item = worker; item < n_items && alive; item += n_workers) {
+    const WinItem it = decode_item(a, item, n_groups, ppc);
+    const int h0 = it.head * a.G + it.block * hb;  // first query head of the block
+    const int heads_here = min(hb, a.G - it.block * hb);
+    const bool onA = tokA < it.n_rows && headA < heads_here, onB = tokB < it.n_rows && headB < heads_here;
+    const int ctxA = onA ? it.ctx0 + tokA : 0, ctxB = onB ? it.ctx0 + tokB : 0;
+    const int loA = first_key(ctxA, a.window), loB = first_key(ctxB, a.window);
+    const int qhA = h0 + (onA ? headA : 0), qhB = h0 + (onB ? headB : 0);
+    const float slA = a.slopes ? a.slopes[qhA] : 0.f, slB = a.slopes ? a.slopes[qhB] : 0.f;
+    uint32_t qa0[KS], qa1[KS], qa2[KS], qa3[KS];
+    {
+      const uint32_t* qA = reinterpret_cast<const uint32_t*>(a.q + (size_t)(it.first_row + (onA ? tokA : 0)) * a.q_stride + (size_t)qhA * a.L.kd);
+      const uint32_t* qB = reinterpret_cast<const uint32_t*>(a.q + (size_t)(it.first_row + (onB ? tokB : 0)) * a.q_stride + (size_t)qhB * a.L.kd);
+#pragma unroll
+      for (int ks = 0; ks < KS; ++ks) {
+        const bool in = ks < n_ks;
+        qa0[ks] = onA && in ? qA[ks * 8 + t] : 0u;
+        qa2[ks] = onA && in ? qA[ks * 8 + 4 + t] : 0u;
+        qa1[ks] = onB && in ? qB[ks * 8 + t] : 0u;
+        qa3[ks] = onB && in ? qB[ks * 8 + 4 + t] : 0u;
+      }
+    }
+    float o[NO][4];
+#pragma unroll
+    for (int j = 0; j < NO; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
+    float mA = kNone, lA = 0.f, mB = kNone, lB = 0.f;
+
+    for (int pg = it.page_begin; pg < it.page_end; ++pg) {
+      const uint32_t s = cons_n % kStages;
+      alive = ptx::mbar_wait(&full_bar[s], (cons_n / kStages) & 1u);
+      if (!alive) break;
+      const uint32_t kbase = ptx::smem_u32(my_tiles + (size_t)s * stage_bytes), vbase = kbase + k_tile;
+      float sc[4][4];
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) { sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f; }
+#pragma unroll
+      for (int kk = 0; kk < KS / 2; ++kk) {
+        if (2 * kk < n_ks) {
+#pragma unroll
+          for (int nt = 0; nt < 4; ++nt) {
+            const int row = nt * 8 + ld_r, cc = 4 * kk + ld_m;
+            uint32_t b[4];
+            ldsm4(kbase + (cc >> 3) * 4096 + row * 128 + (((cc & 7) ^ (row & 7)) << 4), b);
+            mma16816(sc[nt], qa0[2 * kk], qa1[2 * kk], qa2[2 * kk], qa3[2 * kk], b[0], b[1]);
+            mma16816(sc[nt], qa0[2 * kk + 1], qa1[2 * kk + 1], qa2[2 * kk + 1], qa3[2 * kk + 1], b[2], b[3]);
+          }
+        }
+      }
+      // ---- online softmax on rows g (A) and g+8 (B), each with its own window and bias ----
+      const int tok0 = pg * 32;
+      float mxA = kNone, mxB = kNone;
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int tok = tok0 + nt * 8 + 2 * t + e;
+          const float sa = sc[nt][e] * a.scale_log2 - slA * (float)(ctxA - 1 - tok);
+          const float sb = sc[nt][2 + e] * a.scale_log2 - slB * (float)(ctxB - 1 - tok);
+          sc[nt][e] = tok < ctxA && tok >= loA ? sa : kNone;
+          sc[nt][2 + e] = tok < ctxB && tok >= loB ? sb : kNone;
+          mxA = fmaxf(mxA, sc[nt][e]);
+          mxB = fmaxf(mxB, sc[nt][2 + e]);
+        }
+      }
+      mxA = fmaxf(mxA, __shfl_xor_sync(0xffffffffu, mxA, 1));
+      mxA = fmaxf(mxA, __shfl_xor_sync(0xffffffffu, mxA, 2));
+      mxB = fmaxf(mxB, __shfl_xor_sync(0xffffffffu, mxB, 1));
+      mxB = fmaxf(mxB, __shfl_xor_sync(0xffffffffu, mxB, 2));
+      const float mA_new = fmaxf(mA, mxA), mB_new = fmaxf(mB, mxB);
+      const float corrA = exp2f(mA - mA_new), corrB = exp2f(mB - mB_new);
+      float psA = 0.f, psB = 0.f;
+      uint32_t ph[2][4], pl[2][4];
+#pragma unroll
+      for (int kt = 0; kt < 2; ++kt) {
+        float pA[4], pB[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float sa = sc[2 * kt + (e >> 1)][e & 1], sb = sc[2 * kt + (e >> 1)][2 + (e & 1)];
+          pA[e] = sa > kNone ? exp2f(sa - mA_new) : 0.f;
+          pB[e] = sb > kNone ? exp2f(sb - mB_new) : 0.f;
+          psA += pA[e];
+          psB += pB[e];
+        }
+        split_bf16(pA[0], pA[1], ph[kt][0], pl[kt][0]);
+        split_bf16(pB[0], pB[1], ph[kt][1], pl[kt][1]);
+        split_bf16(pA[2], pA[3], ph[kt][2], pl[kt][2]);
+        split_bf16(pB[2], pB[3], ph[kt][3], pl[kt][3]);
+      }
+      lA = lA * corrA + psA; mA = mA_new;
+      lB = lB * corrB + psB; mB = mB_new;
+      if (__any_sync(0xffffffffu, corrA != 1.f || corrB != 1.f)) {
+#pragma unroll
+        for (int j = 0; j < NO; ++j) { o[j][0] *= corrA; o[j][1] *= corrA; o[j][2] *= corrB; o[j][3] *= corrB; }
+      }
+#pragma unroll
+      for (int jj = 0; jj < NO / 2; ++jj) {
+        if (jj < n_vs) {
+#pragma unroll
+          for (int kt = 0; kt < 2; ++kt) {
+            const int row = kt * 16 + (ld_m & 1) * 8 + ld_r, cc = 2 * jj + (ld_m >> 1);
+            uint32_t b[4];
+            ldsm4_trans(vbase + (cc >> 3) * 4096 + row * 128 + (((cc & 7) ^ (row & 7)) << 4), b);
+            mma16816(o[2 * jj], ph[kt][0], ph[kt][1], ph[kt][2], ph[kt][3], b[0], b[1]);
+            mma16816(o[2 * jj + 1], ph[kt][0], ph[kt][1], ph[kt][2], ph[kt][3], b[2], b[3]);
+            mma16816(o[2 * jj], pl[kt][0], pl[kt][1], pl[kt][2], pl[kt][3], b[0], b[1]);
+            mma16816(o[2 * jj + 1], pl[kt][0], pl[kt][1], pl[kt][2], pl[kt][3], b[2], b[3]);
+          }
+        }
+      }
+      __syncwarp();
+      cons_n += 1;
+      produce_one();  // refill the slot just drained
+    }
+    if (!alive) break;
+    lA += __shfl_xor_sync(0xffffffffu, lA, 1);
+    lA += __shfl_xor_sync(0xffffffffu, lA, 2);
+    lB += __shfl_xor_sync(0xffffffffu, lB, 1);
+    lB += __shfl_xor_sync(0xffffffffu, lB, 2);
+    auto store = [&](bool on, int tok, int qh, float m, float l, int e0) {
+      if (!on) return;
+      if (it.slot0 < 0) {
+        float f = 1.f;
+        if (a.sinks) {
+          const float sk = a.sinks[qh], mm = fmaxf(m, sk);
+          f = exp2f(m - mm);
+          l = l * f + exp2f(sk - mm);
+        }
+        const float inv = l > 0.f ? f / l : 0.f;
+        __nv_bfloat16* dst = a.out + (size_t)(it.first_row + tok) * a.out_stride + (size_t)qh * a.L.value_dim;
+#pragma unroll
+        for (int j = 0; j < NO; ++j) {
+          const int c = j * 8 + 2 * t;
+          if ((a.L.value_dim & 1) == 0) {
+            if (c < a.L.value_dim) *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(o[j][e0] * inv, o[j][e0 + 1] * inv);
+          } else {
+            if (c < a.L.value_dim) dst[c] = __float2bfloat16(o[j][e0] * inv);
+            if (c + 1 < a.L.value_dim) dst[c + 1] = __float2bfloat16(o[j][e0 + 1] * inv);
+          }
+        }
+      } else {
+        const size_t pidx = (size_t)(it.slot0 + tok) * a.n_q_heads + qh;
+#pragma unroll
+        for (int j = 0; j < NO; ++j)
+          if (j * 8 < a.L.vd) *reinterpret_cast<float2*>(a.part_o + pidx * a.L.vd + j * 8 + 2 * t) = make_float2(o[j][e0], o[j][e0 + 1]);
+        if (t == 0) { a.part_ml[pidx * 2] = m; a.part_ml[pidx * 2 + 1] = l; }
+      }
+    };
+    store(onA, tokA, qhA, mA, lA, 0);
+    store(onB, tokB, qhB, mB, lB, 2);
+  }
+  if (!alive && lane == 0) atomicExch(a.d.state + ST_ATTN_ERR, B200_ERR_DEVICE_FLAGGED);
+}
+
+// One warp per (row, query head) of the groups that were cut into several chunks.
+__global__ void __launch_bounds__(256) window_combine_kernel(WinArgs a) {
+  const int lane = threadIdx.x & 31;
+  const long long w = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (w >= (long long)a.total_rows * a.n_q_heads || a.d.state[ST_ATTN_ERR] != 0) return;
+  const int row = (int)(w / a.n_q_heads), qh = (int)(w - (long long)row * a.n_q_heads);
+  const int grp = a.row_group[row];
+  if (a.part_base[grp] < 0) return;
+  const int first = a.group_first[grp], size = a.group_first[grp + 1] - first, n_chunks = a.chunk_start[grp + 1] - a.chunk_start[grp];
+  const size_t slot0 = (size_t)a.part_base[grp] + (row - first);
+  float mm = a.sinks ? a.sinks[qh] : kNone;
+  for (int c = lane; c < n_chunks; c += 32) mm = fmaxf(mm, a.part_ml[((slot0 + (size_t)c * size) * a.n_q_heads + qh) * 2]);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, o));
+  float l = 0.f;
+  for (int c = lane; c < n_chunks; c += 32) {
+    const size_t pidx = (slot0 + (size_t)c * size) * a.n_q_heads + qh;
+    l += a.part_ml[pidx * 2 + 1] * exp2f(a.part_ml[pidx * 2] - mm);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+  if (a.sinks) l += exp2f(a.sinks[qh] - mm);
+  const float inv = l > 0.f ? 1.0f / l : 0.f;
+  __nv_bfloat16* dst = a.out + (size_t)row * a.out_stride + (size_t)qh * a.L.value_dim;
+  for (int v0 = 0; v0 < a.L.vd; v0 += 128) {  // four columns per lane
+    const int v = v0 + 4 * lane;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    if (v < a.L.vd) {
+#pragma unroll 4
+      for (int c = 0; c < n_chunks; ++c) {
+        const size_t pidx = (slot0 + (size_t)c * size) * a.n_q_heads + qh;
+        const float wgt = exp2f(a.part_ml[pidx * 2] - mm);
+        const float4 p = *reinterpret_cast<const float4*>(a.part_o + pidx * a.L.vd + v);
+        acc[0] += p.x * wgt; acc[1] += p.y * wgt; acc[2] += p.z * wgt; acc[3] += p.w * wgt;
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (v + e < a.L.value_dim) dst[v + e] = __float2bfloat16(acc[e] * inv);
+    }
+  }
+}
+
+// ---- CUDA-core kernel: any width, bf16 or f32 pools -----------------------------------------------------------
+__device__ __forceinline__ float to_f(float x) { return x; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 x) { return __bfloat162float(x); }
+__device__ __forceinline__ void put(float* p, float x) { *p = x; }
+__device__ __forceinline__ void put(__nv_bfloat16* p, float x) { *p = __float2bfloat16(x); }
+
+struct SimtArgs {
+  KvDev d;
+  KvLayerDev L;
+  const void* q;
+  int q_stride;
+  const int* row_seq;
+  const int* row_ctx;
+  int total_rows, n_q_heads, window;
+  float scale;
+  const float *slopes_log2, *sinks_log2;
+  void* out;
+  int out_stride;
+};
+
+// One warp per (row, query head): 32 keys at a time (one per lane) for the scores, value columns over the lanes for the
+// weighted sum; query and output row in shared memory.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_simt_kernel(SimtArgs a) {
+  extern __shared__ float sh[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, kd = a.L.key_dim, vd = a.L.value_dim;
+  float* q = sh + warp * (kd + vd);
+  float* o = q + kd;
+  const long long w = (long long)blockIdx.x * 4 + warp;
+  if (w >= (long long)a.total_rows * a.n_q_heads) return;
+  const int row = (int)(w / a.n_q_heads), qh = (int)(w - (long long)row * a.n_q_heads), head = qh / (a.n_q_heads / a.L.heads);
+  const T* qg = (const T*)a.q + (size_t)row * a.q_stride + (size_t)qh * a.L.kd;
+  for (int c = lane; c < kd; c += 32) q[c] = to_f(qg[c]);
+  for (int c = lane; c < vd; c += 32) o[c] = 0.f;
+  __syncwarp();
+  const int seq = a.row_seq[row], ctx = a.row_ctx[row], lo = first_key(ctx, a.window);
+  if (seq < 0 || seq >= a.d.max_seqs || (ctx + 31) / 32 > a.d.seq_pages[seq]) return;  // reservation failed: the step is flagged
+  const int* table = a.d.block_table + (size_t)seq * a.d.max_pages_per_seq;
+  const T* kp = (const T*)((const char*)a.d.k_pool + a.L.k_off);
+  const T* vp = (const T*)((const char*)a.d.v_pool + a.L.v_off);
+  const float slope = a.slopes_log2 ? a.slopes_log2[qh] : 0.f, scale = a.scale * kLog2e;
+  float m = kNone, l = 0.f;
+  for (int pg = lo / 32; pg * 32 < ctx; ++pg) {
+    const int tok = pg * 32 + lane;
+    const size_t tile = ((size_t)table[pg] * a.L.heads + head) * 32;
+    const bool on = tok >= lo && tok < ctx;
+    float s = kNone;
+    if (on) {
+      const T* kr = kp + (tile + lane) * a.L.kd;
+      float acc = 0.f;
+      for (int c = 0; c < kd; ++c) acc = fmaf(q[c], to_f(kr[c]), acc);
+      s = acc * scale - slope * (float)(ctx - 1 - tok);
+    }
+    float mx = s;
+#pragma unroll
+    for (int b = 16; b > 0; b >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, b));
+    const float m_new = fmaxf(m, mx), corr = exp2f(m - m_new), p = on ? exp2f(s - m_new) : 0.f;
+    float ps = p;
+#pragma unroll
+    for (int b = 16; b > 0; b >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, b);
+    l = l * corr + ps;
+    m = m_new;
+    const int k0 = max(lo - pg * 32, 0), k1 = min(ctx - pg * 32, 32);
+    for (int c0 = 0; c0 < vd; c0 += 32) {
+      const int c = c0 + lane;
+      float acc = c < vd ? o[c] * corr : 0.f;
+      for (int k = k0; k < k1; ++k) {
+        const float pk = __shfl_sync(0xffffffffu, p, k);
+        if (c < vd) acc = fmaf(pk, to_f(vp[(tile + k) * a.L.vd + c]), acc);
+      }
+      if (c < vd) o[c] = acc;
+    }
+    __syncwarp();
+  }
+  float f = 1.f;
+  if (a.sinks_log2) {
+    const float sk = a.sinks_log2[qh], mm = fmaxf(m, sk);
+    f = exp2f(m - mm);
+    l = l * f + exp2f(sk - mm);
+  }
+  T* out = (T*)a.out + (size_t)row * a.out_stride + (size_t)qh * vd;
+  for (int c = lane; c < vd; c += 32) put(out + c, l > 0.f ? o[c] * f / l : 0.f);
+}
+
+int g_sms = 0;
+b200_status sm_count() {
+  if (g_sms == 0) {
+    int dev = 0;
+    B200_CUDA_TRY(cudaGetDevice(&dev));
+    B200_CUDA_TRY(cudaDeviceGetAttribute(&g_sms, cudaDevAttrMultiProcessorCount, dev));
+  }
+  return B200_OK;
+}
+
+int head_block_of(int gqa) { return std::min(gqa, 16); }
+int q_tokens_of(int gqa) { return gqa >= 16 ? 1 : 16 / gqa; }
+
+WindowPlan* find_plan(b200_kv* kv, int window, int q_tokens) {
+  for (WindowPlan* p : kv->plans)
+    if (p->window == window && p->q_tokens == q_tokens) return p;
+  return nullptr;
+}
+
+template <int KB, int VB>
+b200_status launch_mma(const b200_kv* kv, const WinArgs& a, int layer, cudaStream_t s) {
+  constexpr int WARPS = KB + VB <= 4 ? 4 : 2;
+  const int boxes = (a.L.kd + 63) / 64 + (a.L.vd + 63) / 64;
+  const size_t smem = (size_t)WARPS * kStages * boxes * 4096 + 1024 + sizeof(uint64_t) * WARPS * kStages;
+  static bool configured = false;
+  if (!configured) {
+    const int most = WARPS * kStages * (KB + VB) * 4096 + 1024 + (int)sizeof(uint64_t) * WARPS * kStages;
+    B200_CUDA_TRY((cudaFuncSetAttribute(window_attn_mma_kernel<KB, VB, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, most)));
+    configured = true;
+  }
+  const int per_sm = smem <= 74 * 1024 ? 3 : (smem <= 112 * 1024 ? 2 : 1);
+  window_attn_mma_kernel<KB, VB, WARPS><<<g_sms * per_sm, WARPS * 32, smem, s>>>(kv->lay_kmap[layer], kv->lay_vmap[layer], a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+template <int KB>
+b200_status launch_mma_v(const b200_kv* kv, const WinArgs& a, int layer, cudaStream_t s) {
+  if (a.L.vd <= 64) return launch_mma<KB, 1>(kv, a, layer, s);
+  if (a.L.vd <= 128) return launch_mma<KB, 2>(kv, a, layer, s);
+  return launch_mma<KB, 4>(kv, a, layer, s);
+}
+
+}  // namespace
+
+extern int b200_attn_pages_per_chunk;
+
+b200_status b200_window_attn_plan(b200_kv* kv, int32_t window, int32_t gqa, const int32_t* d_row_seq, const int32_t* d_row_ctx,
+                                  int32_t total_rows, int32_t prefill, void* stream) {
+  if (total_rows <= 0) return B200_OK;
+  if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
+  b200_status st = sm_count();
+  if (st != B200_OK) return st;
+  const int qt = q_tokens_of(gqa), R = kv->cfg.max_rows + 2;
+  WindowPlan* p = find_plan(kv, window, qt);
+  if (!p) {
+    p = new WindowPlan();
+    p->window = window;
+    p->q_tokens = qt;
+    if (cudaMalloc((void**)&p->buf, sizeof(int) * ((size_t)4 * R + 2)) != cudaSuccess) {
+      delete p;
+      b200_set_error("attention plan: out of device memory");
+      return B200_ERR_CUDA;
+    }
+    kv->plans.push_back(p);
+  }
+  const int forced = b200_attn_pages_per_chunk <= 0 ? 0 : std::min(std::max(b200_attn_pages_per_chunk, 1), 1 << 20);
+  const int per_chunk = kv->cfg.n_kv_heads * ((gqa + 15) / 16);
+  window_plan_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(d_row_seq, d_row_ctx, total_rows, kv->cfg.page_size, window, qt,
+                                                          prefill && total_rows >= 1024 ? 1 : 0, per_chunk, g_sms * 4, forced, kv->max_chunks,
+                                                          p->buf, p->buf + R, p->buf + 2 * R, p->buf + 3 * R, p->buf + 4 * R);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
+                                 bool mma, void* stream) {
+  if (c.layer < 0 || c.layer >= kv->cfg.n_layers || !kv->layered) { b200_set_error("window attention: layer %d of no layered pool", c.layer); return B200_ERR_INVALID_ARGUMENT; }
+  const KvLayerDev& L = kv->lay[c.layer];
+  if (c.n_q_heads <= 0 || c.n_q_heads % L.heads != 0) { b200_set_error("window attention: %d query heads over %d kv heads", c.n_q_heads, L.heads); return B200_ERR_INVALID_ARGUMENT; }
+  if (total_rows <= 0) return B200_OK;
+  if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
+  b200_status st = sm_count();
+  if (st != B200_OK) return st;
+  cudaStream_t s = (cudaStream_t)stream;
+  const int G = c.n_q_heads / L.heads;
+  if (!b200_window_attn_takes_mma(kv, c.layer) || !mma) {
+    SimtArgs a;
+    a.d = kv->dev; a.L = L; a.q = c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx; a.total_rows = total_rows;
+    a.n_q_heads = c.n_q_heads; a.window = c.window; a.scale = c.scale; a.slopes_log2 = c.slopes_log2; a.sinks_log2 = c.sinks_log2;
+    a.out = c.out; a.out_stride = c.out_stride;
+    const size_t smem = sizeof(float) * 4 * (L.key_dim + L.value_dim);
+    if (smem > 200 * 1024) { b200_set_error("window attention: head widths %d / %d are too large", L.key_dim, L.value_dim); return B200_ERR_UNSUPPORTED; }
+    const unsigned grid = (unsigned)(((long long)total_rows * c.n_q_heads + 3) / 4);
+    auto* kernel = kv->dev.elem_bytes == 4 ? attn_simt_kernel<float> : attn_simt_kernel<__nv_bfloat16>;
+    if (smem > 48 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    kernel<<<grid, 128, smem, s>>>(a);
+    B200_LAUNCH_CHECK();
+    return B200_OK;
+  }
+  const WindowPlan* p = find_plan(kv, c.window, q_tokens_of(G));
+  if (!p) { b200_set_error("window attention: no plan for window %d and group %d", c.window, G); return B200_ERR_INVALID_ARGUMENT; }
+  const int R = kv->cfg.max_rows + 2;
+  WinArgs a;
+  a.d = kv->dev; a.L = L; a.q = (const __nv_bfloat16*)c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx;
+  a.total_rows = total_rows; a.n_q_heads = c.n_q_heads; a.window = c.window;
+  a.G = G; a.head_block = head_block_of(G); a.n_blocks = (G + 15) / 16;
+  a.group_first = p->buf; a.chunk_start = p->buf + R; a.part_base = p->buf + 2 * R; a.row_group = p->buf + 3 * R; a.hdr = p->buf + 4 * R;
+  a.part_o = kv->d_part_o; a.part_ml = kv->d_part_ml;
+  a.scale_log2 = c.scale * kLog2e;
+  a.slopes = c.slopes_log2; a.sinks = c.sinks_log2;
+  a.out = (__nv_bfloat16*)c.out; a.out_stride = c.out_stride;
+  if (L.kd <= 64) st = launch_mma_v<1>(kv, a, c.layer, s);
+  else if (L.kd <= 128) st = launch_mma_v<2>(kv, a, c.layer, s);
+  else st = launch_mma_v<4>(kv, a, c.layer, s);
+  if (st != B200_OK) return st;
+  // a window that spans no more pages than the shortest chunk the plan may choose never leaves partial sums
+  const int shortest = b200_attn_pages_per_chunk > 0 ? b200_attn_pages_per_chunk : 4;
+  const int most_pages = c.window > 0 ? (c.window + q_tokens_of(G) - 2) / 32 + 2 : kv->cfg.max_pages_per_seq;
+  if (std::min(most_pages, kv->cfg.max_pages_per_seq) <= shortest) return B200_OK;
+  window_combine_kernel<<<(unsigned)(((long long)total_rows * c.n_q_heads + 7) / 8), 256, 0, s>>>(a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+bool b200_window_attn_takes_mma(const b200_kv* kv, int32_t layer) {
+  return kv->layered && kv->dev.elem_bytes == 2 && kv->lay[layer].kd <= 256 && kv->lay[layer].vd <= 256;
+}

@@ -1,0 +1,812 @@
+// Configurable decoder stack over a packed ragged batch (model_step.cu packs it and reserves its pages).  Each layer says
+// which mechanisms it has (b200_decoder_layer); the stack may run a range of layers several times with the same weights, each
+// pass opening with x = W_in [x ; x0].
+//
+// A layer is six launches: q/k/v matmul; decoder_qkv_kernel (split-K finish, biases, per-head norms, q to the attention's
+// operand, k and v straight into their pages); attention (attn_window.cu); o matmul; decoder_rows_kernel (split-K
+// finish, post-norm, f32 residual add, and the norm or the [x ; x0] rows the next matmul reads); then the feed-forward's
+// two matmuls around the SwiGLU epilogue and decoder_rows_kernel again.
+//
+// The residual, every norm, the biases and the logits are f32; matrix operands are bf16, or f32 with B200_DT_F32 (the same
+// kernels instantiated for float, matmuls through b200_qmm_f32, attention on CUDA cores).
+//
+// Matrices are padded with zero rows and columns to multiples of 64, so any width runs; the columns an activation row has
+// behind its own width meet zero weights.
+#include <cuda_bf16.h>
+
+#include <algorithm>
+#include <cmath>
+#include <cstring>
+#include <map>
+#include <vector>
+
+#include "common.h"
+#include "kv_pool.cuh"
+#include "model_step.cuh"
+#include "qmm.cuh"
+
+namespace {
+
+constexpr double kLog2e = 1.4426950408889634;
+
+int pad64(int n) { return (n + 63) / 64 * 64; }
+
+// Result of a matmul, row by row: f32 split-K partial tiles (ws) or rows the matmul wrote itself (y).
+struct MatSrc {
+  const float* ws = nullptr;
+  int splits = 0, tn = 0, tts = 0;
+  const void* y = nullptr;
+  int y_stride = 0;
+};
+
+__device__ __forceinline__ float ld(const float* p) { return *p; }
+__device__ __forceinline__ float ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+template <int VEC>
+struct Vec { float v[VEC]; };
+
+template <int VEC>
+__device__ __forceinline__ Vec<VEC> load_vec(const float* p) {
+  Vec<VEC> r;
+  if constexpr (VEC == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    r.v[0] = f.x; r.v[1] = f.y; r.v[2] = f.z; r.v[3] = f.w;
+  } else {
+    r.v[0] = *p;
+  }
+  return r;
+}
+template <int VEC>
+__device__ __forceinline__ Vec<VEC> load_vec(const __nv_bfloat16* p) {
+  Vec<VEC> r;
+  if constexpr (VEC == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    r.v[0] = __uint_as_float(u.x << 16); r.v[1] = __uint_as_float(u.x & 0xFFFF0000u);
+    r.v[2] = __uint_as_float(u.y << 16); r.v[3] = __uint_as_float(u.y & 0xFFFF0000u);
+  } else {
+    r.v[0] = __bfloat162float(*p);
+  }
+  return r;
+}
+template <int VEC>
+__device__ __forceinline__ void store_vec(float* p, const Vec<VEC>& x) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(x.v[0], x.v[1], x.v[2], x.v[3]);
+  else *p = x.v[0];
+}
+template <int VEC>
+__device__ __forceinline__ void store_vec(__nv_bfloat16* p, const Vec<VEC>& x) {
+  if constexpr (VEC == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(x.v[0], x.v[1]), b = __floats2bfloat162_rn(x.v[2], x.v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  } else {
+    *p = __float2bfloat16(x.v[0]);
+  }
+}
+
+// Columns c .. c + VEC - 1 of one row; the splits are summed in split order.
+template <typename T, int VEC>
+__device__ __forceinline__ Vec<VEC> mat_value(const MatSrc& s, int row, int c) {
+  if (!s.ws) return load_vec<VEC>((const T*)s.y + (size_t)row * s.y_stride + c);
+  const int nt = c >> 7, r = c & 127, tt = row / s.tn, tr = row - tt * s.tn;
+  const float* p = s.ws + (((size_t)(nt * s.tts + tt) * s.splits) * s.tn + tr) * 128 + r;
+  Vec<VEC> acc = load_vec<VEC>(p);
+  for (int i = 1; i < s.splits; ++i) {
+    const Vec<VEC> b = load_vec<VEC>(p + (size_t)i * s.tn * 128);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) acc.v[e] += b.v[e];
+  }
+  return acc;
+}
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+
+__device__ float block_sum(float v, float* part) {
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = threadIdx.x < (blockDim.x >> 5) ? part[threadIdx.x] : 0.f;
+  if (threadIdx.x < 32) {
+    t = warp_sum(t);
+    if (threadIdx.x == 0) part[0] = t;
+  }
+  __syncthreads();
+  return part[0];
+}
+
+// ---- between the matmuls ------------------------------------------------------------------------------------
+struct RowArgs {
+  int hidden;
+  float eps;
+  const uint32_t* tokens = nullptr;  // set: the row is the embedding of its token (x and x0 are written)
+  const __nv_bfloat16* embed = nullptr;
+  int vocab = 0;
+  float embed_scale = 1.f;
+  MatSrc src;
+  const float* post_w = nullptr;  // post-norm of the sublayer's output
+  int replace = 0;                // x = src instead of x += src
+  float* x = nullptr;
+  float* x0 = nullptr;            // embedding output (null without a loop)
+  const float* norm_w = nullptr;  // h = norm(x) * norm_w for the next matmul
+  void* h = nullptr;
+  int h_stride = 0;
+  void* cat = nullptr;            // [x ; x0] for the loop's input matmul
+  int cat_stride = 0;
+};
+
+// One CTA per row: sublayer output -> residual stream -> what the next matmul reads.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
+  extern __shared__ float row_sh[];
+  __shared__ float part[32];
+  const int row = blockIdx.x, n = a.hidden / VEC;
+  float* xr = a.x + (size_t)row * a.hidden;
+  float ss = 0.f;
+  if (a.tokens) {
+    const uint32_t tok = min(a.tokens[row], (uint32_t)(a.vocab - 1));
+    const __nv_bfloat16* e = a.embed + (size_t)tok * a.hidden;
+    float* x0r = a.x0 ? a.x0 + (size_t)row * a.hidden : nullptr;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      Vec<VEC> v = load_vec<VEC>(e + i * VEC);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) { v.v[k] *= a.embed_scale; ss += v.v[k] * v.v[k]; }
+      store_vec<VEC>(row_sh + i * VEC, v);
+      store_vec<VEC>(xr + i * VEC, v);
+      if (x0r) store_vec<VEC>(x0r + i * VEC, v);
+    }
+  } else {
+    float ys = 0.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      const Vec<VEC> v = mat_value<T, VEC>(a.src, row, i * VEC);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) ys += v.v[k] * v.v[k];
+      store_vec<VEC>(row_sh + i * VEC, v);
+    }
+    const float r = a.post_w ? 1.0f / sqrtf(block_sum(ys, part) / (float)a.hidden + a.eps) : 1.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {  // a thread meets the columns it wrote itself
+      Vec<VEC> v = load_vec<VEC>(row_sh + i * VEC);
+      if (a.post_w) {
+        const Vec<VEC> w = load_vec<VEC>(a.post_w + i * VEC);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) v.v[k] *= r * w.v[k];
+      }
+      if (!a.replace) {
+        const Vec<VEC> x = load_vec<VEC>(xr + i * VEC);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) v.v[k] += x.v[k];
+      }
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) ss += v.v[k] * v.v[k];
+      store_vec<VEC>(row_sh + i * VEC, v);
+      store_vec<VEC>(xr + i * VEC, v);
+    }
+  }
+  if (a.norm_w) {
+    const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)a.hidden + a.eps);
+    T* hr = (T*)a.h + (size_t)row * a.h_stride;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      Vec<VEC> v = load_vec<VEC>(row_sh + i * VEC);
+      const Vec<VEC> w = load_vec<VEC>(a.norm_w + i * VEC);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) v.v[k] *= r * w.v[k];
+      store_vec<VEC>(hr + i * VEC, v);
+    }
+  }
+  if (a.cat) {
+    T* cr = (T*)a.cat + (size_t)row * a.cat_stride;
+    const float* x0r = a.x0 + (size_t)row * a.hidden;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      store_vec<VEC>(cr + i * VEC, load_vec<VEC>(row_sh + i * VEC));
+      // the embedding row itself was written by this thread above
+      store_vec<VEC>(cr + a.hidden + i * VEC, load_vec<VEC>(x0r + i * VEC));
+    }
+  }
+}
+
+// Rows idx[r] of x, normalised, as the head's operand.
+template <typename T>
+__global__ void __launch_bounds__(256) decoder_final_kernel(const float* __restrict__ x, const int* __restrict__ idx, const float* __restrict__ w,
+                                                            T* __restrict__ out, int hidden, int out_stride, float eps) {
+  __shared__ float part[32];
+  const float* xr = x + (size_t)max(idx[blockIdx.x], 0) * hidden;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) ss += xr[c] * xr[c];
+  const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)hidden + eps);
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) st(out + (size_t)blockIdx.x * out_stride + c, xr[c] * r * w[c]);
+}
+
+__global__ void __launch_bounds__(256) decoder_logits_kernel(MatSrc src, float* __restrict__ logits, int vocab) {
+  const int c = blockIdx.x * 256 + threadIdx.x;
+  if (c < vocab) logits[(size_t)blockIdx.y * vocab + c] = mat_value<float, 1>(src, blockIdx.y, c).v[0];
+}
+
+// ---- between the q/k/v projection and attention ---------------------------------------------------------------
+struct QkvArgs {
+  KvDev d;
+  KvLayerDev L;
+  MatSrc src;
+  const float* bias;  // [q | k | v] columns, null without biases
+  int hq, qk_norm;
+  float eps;
+  void* q;
+  int q_stride;
+  const int *pos, *row_seq;
+};
+
+// One warp per (row, head); q heads, then k heads, then v heads.  Grid y covers the heads, eight at a time.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) decoder_qkv_kernel(QkvArgs a) {
+  constexpr int KEEP = VEC == 4 ? 2 : 4;  // passes of 32 x VEC columns kept in registers; wider heads are read again
+  const int row = blockIdx.x, lane = threadIdx.x & 31, H = a.L.heads;
+  const int u = blockIdx.y * 8 + (threadIdx.x >> 5);
+  if (u >= a.hq + 2 * H) return;
+  const bool is_q = u < a.hq, is_v = u >= a.hq + H;
+  const int head = is_q ? u : (is_v ? u - a.hq - H : u - a.hq);
+  const int dim = is_v ? a.L.value_dim : a.L.key_dim, width = is_v ? a.L.vd : a.L.kd;
+  const int n0 = is_v ? (a.hq + H) * a.L.key_dim + head * dim : u * dim;
+  T* dst = nullptr;
+  if (is_q) {
+    dst = (T*)a.q + (size_t)row * a.q_stride + (size_t)head * a.L.kd;
+  } else {
+    const int pos = a.pos[row], seq = a.row_seq[row];
+    const int page_idx = pos / a.d.page_size, slot = pos - page_idx * a.d.page_size;
+    // a step whose reservation failed has no page for this row: nothing is written (the error word is set)
+    if (seq < 0 || seq >= a.d.max_seqs || page_idx >= a.d.seq_pages[seq]) return;
+    const int page = a.d.block_table[(size_t)seq * a.d.max_pages_per_seq + page_idx];
+    char* pool = is_v ? (char*)a.d.v_pool + a.L.v_off : (char*)a.d.k_pool + a.L.k_off;
+    dst = (T*)pool + (((size_t)page * H + head) * a.d.page_size + slot) * (size_t)width;
+  }
+  auto value = [&](int c) {
+    Vec<VEC> v = mat_value<T, VEC>(a.src, row, n0 + c);
+    if (a.bias) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v.v[e] += a.bias[n0 + c + e];
+    }
+    return v;
+  };
+  Vec<VEC> keep[KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int c = (i * 32 + lane) * VEC;
+    if (c < dim) {
+      keep[i] = value(c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += keep[i].v[e] * keep[i].v[e];
+    }
+  }
+  for (int c = (KEEP * 32 + lane) * VEC; c < dim; c += 32 * VEC) {
+    const Vec<VEC> v = value(c);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss += v.v[e] * v.v[e];
+  }
+  float r = 1.f;
+  if (a.qk_norm && !is_v) r = 1.0f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int c = (i * 32 + lane) * VEC;
+    if (c < dim) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) keep[i].v[e] *= r;
+      store_vec<VEC>(dst + c, keep[i]);
+    }
+  }
+  for (int c = (KEEP * 32 + lane) * VEC; c < dim; c += 32 * VEC) {
+    Vec<VEC> v = value(c);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v.v[e] *= r;
+    store_vec<VEC>(dst + c, v);
+  }
+  for (int c = dim + lane; c < width; c += 32) st(dst + c, 0.f);
+}
+
+struct HostTensor { std::vector<uint16_t> bits; };
+
+float bf16_to_f(uint16_t b) {
+  const uint32_t u = (uint32_t)b << 16;
+  float f;
+  std::memcpy(&f, &u, 4);
+  return f;
+}
+
+const char* kTensorNames[] = {"q", "k", "v", "o", "gate", "up", "down", "head", "loop input", "embedding", "q bias", "k bias", "v bias",
+                              "sink", "norm 1", "norm 2", "post-norm 1", "post-norm 2", "final norm"};
+
+}  // namespace
+
+struct b200_decoder : b200_model {
+  b200_decoder_config cfg{};
+  struct Layer {
+    b200_decoder_layer s{};
+    b200_qweight *wqkv = nullptr, *wo = nullptr, *wgu = nullptr, *wdown = nullptr;
+    float *bias = nullptr, *sinks = nullptr, *slopes = nullptr, *norm1 = nullptr, *norm2 = nullptr, *post1 = nullptr, *post2 = nullptr;
+    int qkv_n() const { return s.n_heads * s.key_dim + s.n_kv_heads * (s.key_dim + s.value_dim); }
+    int attn_n() const { return s.n_heads * s.value_dim; }
+  };
+  std::vector<Layer> layers;
+  struct Run { int layer; bool opens; };  // opens: the first layer of a pass of the loop
+  std::vector<Run> runs;
+  std::map<std::pair<int, int>, HostTensor> staged;
+  __nv_bfloat16* embed = nullptr;
+  float* final_norm = nullptr;
+  b200_qweight *head = nullptr, *loop_in = nullptr;
+  // activations: residual and embedding output in f32, operands in the model's type
+  float *x = nullptr, *x0 = nullptr, *rec = nullptr;
+  void *h = nullptr, *cat = nullptr, *y = nullptr, *q = nullptr, *attn = nullptr, *act = nullptr, *last = nullptr;
+  int hp = 0, catp = 0;  // padded widths of h and [x ; x0]
+  bool attn_mma = true, recording = false;
+
+  size_t elem() const { return cfg.dtype == B200_DT_F32 ? 4 : 2; }
+  bool f32() const { return cfg.dtype == B200_DT_F32; }
+  ~b200_decoder() override;
+  b200_status check_pool(const b200_kv* kv) const override;
+  b200_status run_layers(b200_kv* kv, int n_req, int T, int n_logits, void* stream) override;
+  b200_status reserve_logit_rows(int rows) override;
+  b200_status matmul(const b200_qweight* w, const void* in, int rows, int defer, MatSrc* src, void* stream);
+  b200_status rows_step(RowArgs a, int rows, int next, cudaStream_t s);
+  b200_status attention(b200_kv* kv, int run, int rows, void* stream);
+};
+
+b200_decoder::~b200_decoder() {
+  void* dev[] = {embed, final_norm, x, x0, rec, h, cat, y, q, attn, act, last};
+  for (void* p : dev) if (p) cudaFree(p);
+  for (Layer& l : layers) {
+    void* lp[] = {l.bias, l.sinks, l.slopes, l.norm1, l.norm2, l.post1, l.post2};
+    for (void* p : lp) if (p) cudaFree(p);
+    for (b200_qweight* w : {l.wqkv, l.wo, l.wgu, l.wdown}) b200_qweight_destroy(w);
+  }
+  b200_qweight_destroy(head);
+  b200_qweight_destroy(loop_in);
+}
+
+b200_status b200_decoder::check_pool(const b200_kv* kv) const {
+  bool ok = kv->layered && kv->cfg.n_layers == (int)runs.size() && kv->dev.elem_bytes == (int)elem();
+  for (size_t r = 0; ok && r < runs.size(); ++r) {
+    const b200_decoder_layer& s = layers[runs[r].layer].s;
+    const KvLayerDev& L = kv->lay[r];
+    ok = L.heads == s.n_kv_heads && L.key_dim == s.key_dim && L.value_dim == s.value_dim && s.n_heads <= kv->cfg.n_q_heads;
+  }
+  if (!ok) { b200_set_error("decoder: the page pool was built for a different model shape"); return B200_ERR_INVALID_ARGUMENT; }
+  return B200_OK;
+}
+
+b200_status b200_decoder::reserve_logit_rows(int rows) {
+  void* p = nullptr;
+  if (cudaMalloc(&p, (size_t)rows * hp * elem()) != cudaSuccess) { b200_set_error("decoder: no memory for %d logit rows", rows); return B200_ERR_CUDA; }
+  B200_CUDA_TRY(cudaMemset(p, 0, (size_t)rows * hp * elem()));
+  cudaFree(last);
+  last = p;
+  return B200_OK;
+}
+
+// y = in W^T.  src describes where the result is: rows of `y`, or the f32 partial sums of a split K (defer = 1: if K was
+// split; 2: always f32).
+b200_status b200_decoder::matmul(const b200_qweight* w, const void* in, int rows, int defer, MatSrc* src, void* stream) {
+  *src = MatSrc{};
+  src->y = y;
+  src->y_stride = w->n;
+  if (f32()) return b200_qmm_f32(w, (const float*)in, rows, (float*)y, w->n, w->n, B200_EPI_NONE, stream);
+  b200_qmm_partials p;
+  b200_status st = b200_qmm_deferred(w, in, rows, y, defer, stream, &p);
+  if (st == B200_OK && p.pending) { src->ws = p.d_ws; src->splits = p.splits; src->tn = p.tn; src->tts = p.tts; }
+  return st;
+}
+
+// decoder_rows_kernel with what run `next` reads (its first norm, or [x ; x0] when it opens a pass; nothing past the end).
+// next < 0: a.norm_w is already set.
+b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t s) {
+  a.hidden = cfg.hidden;
+  a.eps = cfg.norm_eps;
+  a.x = x;
+  a.x0 = x0;
+  a.h = h;
+  a.h_stride = hp;
+  if (next >= 0 && next < (int)runs.size()) {
+    if (runs[next].opens) { a.cat = cat; a.cat_stride = catp; }
+    else a.norm_w = layers[runs[next].layer].norm1;
+  }
+  const int vec = cfg.hidden % 4 == 0 ? 4 : 1;
+  const int threads = std::min(512, (cfg.hidden / vec + 31) / 32 * 32);
+  const size_t smem = sizeof(float) * cfg.hidden;
+  auto* kernel = f32() ? (vec == 4 ? decoder_rows_kernel<float, 4> : decoder_rows_kernel<float, 1>)
+                       : (vec == 4 ? decoder_rows_kernel<__nv_bfloat16, 4> : decoder_rows_kernel<__nv_bfloat16, 1>);
+  if (smem > 47 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  kernel<<<rows, threads, smem, s>>>(a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+b200_status b200_decoder::attention(b200_kv* kv, int run, int rows, void* stream) {
+  const Layer& l = layers[runs[run].layer];
+  WindowAttnCall c;
+  c.layer = run;
+  c.n_q_heads = l.s.n_heads;
+  c.window = l.s.window;
+  c.q = q;
+  c.q_stride = l.s.n_heads * kv->lay[run].kd;
+  c.scale = l.s.scale;
+  c.slopes_log2 = l.slopes;
+  c.sinks_log2 = l.sinks;
+  c.out = attn;
+  c.out_stride = pad64(l.attn_n());
+  return b200_window_attn_run(kv, c, d_row_seq, d_row_ctx, rows, attn_mma, stream);
+}
+
+b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits, void* stream) {
+  b200_decoder* m = this;
+  cudaStream_t cs = (cudaStream_t)stream;
+  b200_status st = B200_OK;
+  MatSrc src;
+  // one plan per (window, GQA group) of the stack, shared by its layers
+  std::vector<std::pair<int, int>> planned;
+  for (size_t r = 0; r < runs.size(); ++r) {
+    const b200_decoder_layer& s = layers[runs[r].layer].s;
+    const std::pair<int, int> key{s.window, s.n_heads / s.n_kv_heads};
+    if (!attn_mma || !b200_window_attn_takes_mma(kv, (int)r) || std::find(planned.begin(), planned.end(), key) != planned.end()) continue;
+    planned.push_back(key);
+    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, key.first, key.second, d_row_seq, d_row_ctx, T, T > n_req ? 1 : 0, stream));
+  }
+  {
+    RowArgs a{};
+    a.tokens = d_tokens;
+    a.embed = embed;
+    a.vocab = cfg.vocab;
+    a.embed_scale = cfg.embed_scale;
+    MODEL_STEP(rows_step(a, T, 0, cs));
+  }
+  for (size_t r = 0; r < runs.size(); ++r) {
+    const Layer& l = layers[runs[r].layer];
+    const b200_decoder_layer& s = l.s;
+    if (runs[r].opens) {  // x = W_in [x ; x0]; the residual is f32, so the product stays f32
+      MODEL_STEP_CAT(1, matmul(loop_in, cat, T, 2, &src, stream));
+      RowArgs a{};
+      a.src = src;
+      a.replace = 1;
+      a.norm_w = l.norm1;
+      MODEL_STEP(rows_step(a, T, -1, cs));
+    }
+    MODEL_STEP_CAT(1, matmul(l.wqkv, h, T, 1, &src, stream));
+    {
+      QkvArgs a;
+      a.d = kv->dev; a.L = kv->lay[r]; a.src = src; a.bias = l.bias; a.hq = s.n_heads; a.qk_norm = s.flags & B200_DEC_QK_NORM ? 1 : 0;
+      a.eps = cfg.norm_eps; a.q = q; a.q_stride = s.n_heads * kv->lay[r].kd; a.pos = d_pos; a.row_seq = d_row_seq;
+      const bool v4 = s.key_dim % 4 == 0 && s.value_dim % 4 == 0;
+      auto* kernel = f32() ? (v4 ? decoder_qkv_kernel<float, 4> : decoder_qkv_kernel<float, 1>)
+                           : (v4 ? decoder_qkv_kernel<__nv_bfloat16, 4> : decoder_qkv_kernel<__nv_bfloat16, 1>);
+      auto launch = [&]() -> b200_status {
+        kernel<<<dim3(T, (s.n_heads + 2 * s.n_kv_heads + 7) / 8), 256, 0, cs>>>(a);
+        B200_LAUNCH_CHECK();
+        return B200_OK;
+      };
+      MODEL_STEP_CAT(2, launch());
+    }
+    MODEL_STEP_CAT(0, attention(kv, (int)r, T, stream));
+    MODEL_STEP_CAT(1, matmul(l.wo, attn, T, 1, &src, stream));
+    {
+      RowArgs a{};
+      a.src = src;
+      a.post_w = l.post1;
+      if (s.ffn > 0) a.norm_w = l.norm2;
+      MODEL_STEP(rows_step(a, T, s.ffn > 0 ? -1 : (int)r + 1, cs));
+    }
+    if (s.ffn > 0) {
+      if (f32()) MODEL_STEP_CAT(1, b200_qmm_f32(l.wgu, (const float*)h, T, (float*)act, pad64(s.ffn), pad64(s.ffn), B200_EPI_SWIGLU, stream));
+      else MODEL_STEP_CAT(1, b200_qmm(l.wgu, h, T, act, B200_EPI_SWIGLU, nullptr, 0.f, B200_QMM_AUTO, stream));
+      MODEL_STEP_CAT(1, matmul(l.wdown, act, T, 1, &src, stream));
+      RowArgs a{};
+      a.src = src;
+      a.post_w = l.post2;
+      MODEL_STEP(rows_step(a, T, (int)r + 1, cs));
+    }
+    if (recording)
+      B200_CUDA_TRY(cudaMemcpyAsync(rec + r * (size_t)max_rows * cfg.hidden, x, sizeof(float) * (size_t)T * cfg.hidden, cudaMemcpyDeviceToDevice, cs));
+  }
+  auto head_rows = [&]() -> b200_status {
+    if (f32()) decoder_final_kernel<float><<<n_logits, 256, 0, cs>>>(x, d_logit_row, final_norm, (float*)last, cfg.hidden, hp, cfg.norm_eps);
+    else decoder_final_kernel<__nv_bfloat16><<<n_logits, 256, 0, cs>>>(x, d_logit_row, final_norm, (__nv_bfloat16*)last, cfg.hidden, hp, cfg.norm_eps);
+    B200_LAUNCH_CHECK();
+    return B200_OK;
+  };
+  MODEL_STEP(head_rows());
+  if (f32()) {
+    MODEL_STEP_CAT(1, b200_qmm_f32(head, (const float*)last, n_logits, (float*)logits, cfg.vocab, cfg.vocab, B200_EPI_NONE, stream));
+    return B200_OK;
+  }
+  MODEL_STEP_CAT(1, matmul(head, last, n_logits, 2, &src, stream));
+  auto finish = [&]() -> b200_status {
+    decoder_logits_kernel<<<dim3((cfg.vocab + 255) / 256, n_logits), 256, 0, cs>>>(src, (float*)logits, cfg.vocab);
+    B200_LAUNCH_CHECK();
+    return B200_OK;
+  };
+  MODEL_STEP(finish());
+  return B200_OK;
+}
+
+// ---- construction and weights -----------------------------------------------------------------------------------
+namespace {
+
+// Elements of one tensor of the configuration; 0 when the layer does not have it.
+uint64_t tensor_elems(const b200_decoder* m, int layer, int which) {
+  const b200_decoder_config& c = m->cfg;
+  const uint64_t D = c.hidden;
+  switch (which) {
+    case B200_DEC_W_HEAD: case B200_DEC_W_EMBED: return (uint64_t)c.vocab * D;
+    case B200_DEC_W_LOOP_IN: return c.loop_times > 0 ? 2 * D * D : 0;
+    case B200_DEC_FINAL_NORM: return D;
+    default: break;
+  }
+  const b200_decoder_layer& s = m->layers[layer].s;
+  const uint64_t qn = (uint64_t)s.n_heads * s.key_dim, kn = (uint64_t)s.n_kv_heads * s.key_dim, vn = (uint64_t)s.n_kv_heads * s.value_dim;
+  const bool bias = s.flags & B200_DEC_QKV_BIAS, post = s.flags & B200_DEC_POST_NORM;
+  switch (which) {
+    case B200_DEC_W_Q: return qn * D;
+    case B200_DEC_W_K: return kn * D;
+    case B200_DEC_W_V: return vn * D;
+    case B200_DEC_W_O: return D * s.n_heads * s.value_dim;
+    case B200_DEC_W_GATE: case B200_DEC_W_UP: case B200_DEC_W_DOWN: return D * s.ffn;
+    case B200_DEC_B_Q: return bias ? qn : 0;
+    case B200_DEC_B_K: return bias ? kn : 0;
+    case B200_DEC_B_V: return bias ? vn : 0;
+    case B200_DEC_W_SINK: return s.flags & B200_DEC_SINK ? s.n_heads : 0;
+    case B200_DEC_NORM1: return D;
+    case B200_DEC_NORM2: return s.ffn > 0 ? D : 0;
+    case B200_DEC_POSTNORM1: return post ? D : 0;
+    case B200_DEC_POSTNORM2: return post && s.ffn > 0 ? D : 0;
+    default: return 0;
+  }
+}
+
+bool global_tensor(int which) {
+  return which == B200_DEC_W_HEAD || which == B200_DEC_W_EMBED || which == B200_DEC_W_LOOP_IN || which == B200_DEC_FINAL_NORM;
+}
+
+b200_status take(b200_decoder* m, int layer, int which, std::vector<uint16_t>* out) {
+  auto it = m->staged.find({global_tensor(which) ? -1 : layer, which});
+  if (it == m->staged.end()) { b200_set_error("decoder: the %s tensor of layer %d was never set", kTensorNames[which], layer); return B200_ERR_INVALID_ARGUMENT; }
+  *out = std::move(it->second.bits);
+  m->staged.erase(it);
+  return B200_OK;
+}
+
+b200_status upload_f32(const std::vector<float>& v, float** out) {
+  B200_CUDA_TRY(cudaMalloc((void**)out, sizeof(float) * std::max<size_t>(v.size(), 1)));
+  B200_CUDA_TRY(cudaMemcpy(*out, v.data(), sizeof(float) * v.size(), cudaMemcpyHostToDevice));
+  return B200_OK;
+}
+
+b200_status take_vector(b200_decoder* m, int layer, int which, float** out, double factor = 1.0) {
+  std::vector<uint16_t> bits;
+  b200_status st = take(m, layer, which, &bits);
+  if (st != B200_OK) return st;
+  std::vector<float> v(bits.size());
+  for (size_t i = 0; i < bits.size(); ++i) v[i] = factor == 1.0 ? bf16_to_f(bits[i]) : (float)(bf16_to_f(bits[i]) * factor);
+  return upload_f32(v, out);
+}
+
+// Rows of several [n_i, k] matrices, one behind the other or interleaved, as one weight padded to multiples of 64.
+b200_status make_weight(const std::vector<const std::vector<uint16_t>*>& parts, int k, bool interleave, b200_qweight** out) {
+  size_t n = 0;
+  for (auto* p : parts) n += p->size() / k;
+  const int np = interleave ? 2 * pad64((int)n / 2) : pad64((int)n), kp = pad64(k);
+  std::vector<uint16_t> w((size_t)np * kp, 0);
+  size_t row = 0;
+  auto put = [&](const std::vector<uint16_t>* p, size_t r) { std::memcpy(&w[row++ * kp], &(*p)[r * k], sizeof(uint16_t) * k); };
+  if (interleave) {
+    for (size_t r = 0; r < parts[0]->size() / k; ++r) for (auto* p : parts) put(p, r);
+  } else {
+    for (auto* p : parts) for (size_t r = 0; r < p->size() / k; ++r) put(p, r);
+  }
+  return b200_qweight_create(B200_Q_BF16, 1, np, kp, w.data(), nullptr, nullptr, out);
+}
+
+b200_status take_weight(b200_decoder* m, int layer, std::vector<int> which, int k, bool interleave, b200_qweight** out) {
+  std::vector<std::vector<uint16_t>> host(which.size());
+  std::vector<const std::vector<uint16_t>*> parts;
+  for (size_t i = 0; i < which.size(); ++i) {
+    b200_status st = take(m, layer, which[i], &host[i]);
+    if (st != B200_OK) return st;
+    parts.push_back(&host[i]);
+  }
+  return make_weight(parts, k, interleave, out);
+}
+
+b200_status make_slopes(b200_decoder::Layer& l) {
+  if (!(l.s.flags & B200_DEC_DISTANCE_BIAS)) return B200_OK;
+  std::vector<float> v(l.s.n_heads);
+  for (int h = 0; h < l.s.n_heads; ++h) v[h] = (float)(std::exp2(-8.0 * (h + 1) / l.s.n_heads) * kLog2e);
+  return upload_f32(v, &l.slopes);
+}
+
+}  // namespace
+
+extern "C" {
+
+b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder_layer* layers, b200_decoder** out) {
+  *out = nullptr;
+  b200_status st = b200_require_device();
+  if (st != B200_OK) return st;
+  const bool loop = c->loop_times > 0;
+  if (c->n_layers <= 0 || c->hidden <= 0 || c->vocab <= 0 || c->max_rows <= 0 || c->max_reqs <= 0 || c->max_seqs <= 0 ||
+      (c->dtype != B200_DT_BF16 && c->dtype != B200_DT_F32) ||
+      (loop && (c->loop_start < 0 || c->loop_stop > c->n_layers || c->loop_start >= c->loop_stop))) {
+    b200_set_error("decoder: invalid configuration");
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  if (c->hidden > 48 * 1024) { b200_set_error("decoder: width %d is larger than a row buffer", c->hidden); return B200_ERR_UNSUPPORTED; }
+  auto* m = new b200_decoder();
+  m->cfg = *c;
+  m->layers.resize(c->n_layers);
+  size_t qw = 0, yw = pad64(c->hidden), aw = 0, fw = 0;
+  for (int i = 0; i < c->n_layers; ++i) {
+    const b200_decoder_layer& s = layers[i];
+    if (s.n_heads <= 0 || s.n_kv_heads <= 0 || s.n_heads % s.n_kv_heads != 0 || s.key_dim <= 0 || s.value_dim <= 0 || s.ffn < 0 || s.window < 0) {
+      b200_set_error("decoder: layer %d has an invalid shape", i);
+      delete m;
+      return B200_ERR_INVALID_ARGUMENT;
+    }
+    m->layers[i].s = s;
+    qw = std::max(qw, (size_t)s.n_heads * ((s.key_dim + 15) / 16 * 16));
+    yw = std::max(yw, (size_t)pad64(m->layers[i].qkv_n()));
+    aw = std::max(aw, (size_t)pad64(m->layers[i].attn_n()));
+    fw = std::max(fw, (size_t)pad64(s.ffn));
+  }
+  const int lo = loop ? c->loop_start : 0, hi = loop ? c->loop_stop : 0;
+  for (int i = 0; i < lo; ++i) m->runs.push_back({i, false});
+  for (int p = 0; p < c->loop_times && loop; ++p) for (int i = lo; i < hi; ++i) m->runs.push_back({i, i == lo});
+  for (int i = hi; i < c->n_layers; ++i) m->runs.push_back({i, false});
+  m->hp = pad64(c->hidden);
+  m->catp = pad64(2 * c->hidden);
+  st = m->alloc_step(c->vocab, c->max_rows, c->max_reqs, c->max_seqs, true);
+  const size_t R = c->max_rows, e = m->elem();
+  auto alloc = [&](void** p, size_t bytes) {
+    if (st != B200_OK || bytes == 0) return;
+    if (cudaMalloc(p, bytes) != cudaSuccess || cudaMemset(*p, 0, bytes) != cudaSuccess) {  // zero: padding columns stay finite
+      b200_set_error("decoder: cudaMalloc(%zu) failed", bytes);
+      st = B200_ERR_CUDA;
+    }
+  };
+  alloc((void**)&m->embed, (size_t)c->vocab * c->hidden * 2);
+  alloc((void**)&m->x, R * c->hidden * 4);
+  if (loop) {
+    alloc((void**)&m->x0, R * c->hidden * 4);
+    alloc(&m->cat, R * m->catp * e);
+  }
+  alloc(&m->h, R * m->hp * e);
+  alloc(&m->y, std::max(R * yw, (size_t)c->max_reqs * 64) * e);
+  alloc(&m->q, R * qw * e);
+  alloc(&m->attn, R * aw * e);
+  alloc(&m->act, R * fw * e);
+  alloc(&m->last, (size_t)c->max_reqs * m->hp * e);
+  if (st != B200_OK) { delete m; return st; }
+  *out = m;
+  return B200_OK;
+}
+
+void b200_decoder_destroy(b200_decoder* m) { delete m; }
+b200_model* b200_decoder_model(b200_decoder* m) { return m; }
+
+b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t which, const void* h_bf16, uint64_t n) {
+  if (which < 0 || which > B200_DEC_FINAL_NORM || (!global_tensor(which) && (layer < 0 || layer >= m->cfg.n_layers))) {
+    b200_set_error("decoder: no tensor %d in layer %d", which, layer);
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  const uint64_t want = tensor_elems(m, layer, which);
+  if (want != n) {
+    b200_set_error("decoder: the %s tensor of layer %d has %llu elements, the configuration asks for %llu", kTensorNames[which], layer,
+                   (unsigned long long)n, (unsigned long long)want);
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  m->staged[{global_tensor(which) ? -1 : layer, which}].bits.assign((const uint16_t*)h_bf16, (const uint16_t*)h_bf16 + n);
+  return B200_OK;
+}
+
+b200_status b200_decoder_finalize(b200_decoder* m) {
+  const b200_decoder_config& c = m->cfg;
+  b200_status st;
+  for (int i = 0; i < c.n_layers; ++i) {
+    b200_decoder::Layer& l = m->layers[i];
+    const b200_decoder_layer& s = l.s;
+    if ((st = take_weight(m, i, {B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V}, c.hidden, false, &l.wqkv)) != B200_OK) return st;
+    if ((st = take_weight(m, i, {B200_DEC_W_O}, l.attn_n(), false, &l.wo)) != B200_OK) return st;
+    if ((st = take_vector(m, i, B200_DEC_NORM1, &l.norm1)) != B200_OK) return st;
+    if (s.flags & B200_DEC_POST_NORM) if ((st = take_vector(m, i, B200_DEC_POSTNORM1, &l.post1)) != B200_OK) return st;
+    if (s.ffn > 0) {
+      if ((st = take_weight(m, i, {B200_DEC_W_GATE, B200_DEC_W_UP}, c.hidden, true, &l.wgu)) != B200_OK) return st;
+      if ((st = take_weight(m, i, {B200_DEC_W_DOWN}, s.ffn, false, &l.wdown)) != B200_OK) return st;
+      if ((st = take_vector(m, i, B200_DEC_NORM2, &l.norm2)) != B200_OK) return st;
+      if (s.flags & B200_DEC_POST_NORM) if ((st = take_vector(m, i, B200_DEC_POSTNORM2, &l.post2)) != B200_OK) return st;
+    }
+    if (s.flags & B200_DEC_QKV_BIAS) {
+      std::vector<float> all;
+      for (int w : {B200_DEC_B_Q, B200_DEC_B_K, B200_DEC_B_V}) {
+        std::vector<uint16_t> bits;
+        if ((st = take(m, i, w, &bits)) != B200_OK) return st;
+        for (uint16_t b : bits) all.push_back(bf16_to_f(b));
+      }
+      if ((st = upload_f32(all, &l.bias)) != B200_OK) return st;
+    }
+    if (s.flags & B200_DEC_SINK) if ((st = take_vector(m, i, B200_DEC_W_SINK, &l.sinks, kLog2e)) != B200_OK) return st;
+    if ((st = make_slopes(l)) != B200_OK) return st;
+  }
+  if (c.loop_times > 0) if ((st = take_weight(m, -1, {B200_DEC_W_LOOP_IN}, 2 * c.hidden, false, &m->loop_in)) != B200_OK) return st;
+  if ((st = take_weight(m, -1, {B200_DEC_W_HEAD}, c.hidden, false, &m->head)) != B200_OK) return st;
+  if ((st = take_vector(m, -1, B200_DEC_FINAL_NORM, &m->final_norm)) != B200_OK) return st;
+  std::vector<uint16_t> table;
+  if ((st = take(m, -1, B200_DEC_W_EMBED, &table)) != B200_OK) return st;
+  B200_CUDA_TRY(cudaMemcpy(m->embed, table.data(), table.size() * 2, cudaMemcpyHostToDevice));
+  m->ready = true;
+  return B200_OK;
+}
+
+b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
+  const b200_decoder_config& c = m->cfg;
+  b200_status st;
+  const std::vector<float> ones(c.hidden, 1.f);
+  auto weight = [&](int n, int k, uint32_t salt, b200_qweight** out) -> b200_status {
+    if (n % 128 || k % 64) { b200_set_error("random_init: a %d x %d projection (multiples of 128 and 64 only)", n, k); return B200_ERR_INVALID_ARGUMENT; }
+    return b200_qweight_random(B200_Q_BF16, 1, n, k, seed + salt, out);
+  };
+  for (int i = 0; i < c.n_layers; ++i) {
+    b200_decoder::Layer& l = m->layers[i];
+    const b200_decoder_layer& s = l.s;
+    if ((st = weight(l.qkv_n(), c.hidden, 16 * i + 1, &l.wqkv)) != B200_OK) return st;
+    if ((st = weight(c.hidden, l.attn_n(), 16 * i + 2, &l.wo)) != B200_OK) return st;
+    if ((st = upload_f32(ones, &l.norm1)) != B200_OK) return st;
+    if (s.flags & B200_DEC_POST_NORM) if ((st = upload_f32(ones, &l.post1)) != B200_OK) return st;
+    if (s.ffn > 0) {
+      if ((st = weight(2 * s.ffn, c.hidden, 16 * i + 3, &l.wgu)) != B200_OK) return st;
+      if ((st = weight(c.hidden, s.ffn, 16 * i + 4, &l.wdown)) != B200_OK) return st;
+      if ((st = upload_f32(ones, &l.norm2)) != B200_OK) return st;
+      if (s.flags & B200_DEC_POST_NORM) if ((st = upload_f32(ones, &l.post2)) != B200_OK) return st;
+    }
+    if (s.flags & B200_DEC_QKV_BIAS) if ((st = upload_f32(std::vector<float>(l.qkv_n(), 0.01f), &l.bias)) != B200_OK) return st;
+    if (s.flags & B200_DEC_SINK) if ((st = upload_f32(std::vector<float>(s.n_heads, 0.5f), &l.sinks)) != B200_OK) return st;
+    if ((st = make_slopes(l)) != B200_OK) return st;
+  }
+  if (c.loop_times > 0) if ((st = weight(c.hidden, 2 * c.hidden, 11, &m->loop_in)) != B200_OK) return st;
+  if ((st = weight(c.vocab, c.hidden, 7, &m->head)) != B200_OK) return st;
+  if ((st = upload_f32(ones, &m->final_norm)) != B200_OK) return st;
+  std::vector<uint16_t> emb((size_t)c.vocab * c.hidden);
+  uint32_t s = seed * 2654435761u + 12345u;
+  for (auto& e : emb) { s = s * 1664525u + 1013904223u; e = (uint16_t)(((s >> 16) & 0x807F) | 0x3C80); }
+  B200_CUDA_TRY(cudaMemcpy(m->embed, emb.data(), emb.size() * 2, cudaMemcpyHostToDevice));
+  m->ready = true;
+  return B200_OK;
+}
+
+int32_t b200_decoder_cache_layers(const b200_decoder* m, b200_kv_layer* out, int32_t cap) {
+  for (size_t r = 0; r < m->runs.size() && (int)r < cap; ++r) {
+    const b200_decoder_layer& s = m->layers[m->runs[r].layer].s;
+    out[r] = b200_kv_layer{s.n_kv_heads, s.key_dim, s.value_dim};
+  }
+  return (int32_t)m->runs.size();
+}
+
+b200_status b200_decoder_record_layers(b200_decoder* m, int32_t on) {
+  if (on && !m->rec) B200_CUDA_TRY(cudaMalloc((void**)&m->rec, sizeof(float) * m->runs.size() * (size_t)m->max_rows * m->cfg.hidden));
+  m->recording = on != 0;
+  m->drop_graphs();
+  return B200_OK;
+}
+
+b200_status b200_decoder_recorded_layers(b200_decoder* m, int32_t rows, float* h_out) {
+  if (!m->rec || rows < 0 || rows > m->max_rows) { b200_set_error("recorded_layers: nothing recorded, or %d rows", rows); return B200_ERR_INVALID_ARGUMENT; }
+  B200_CUDA_TRY(cudaDeviceSynchronize());
+  for (size_t r = 0; r < m->runs.size(); ++r)
+    B200_CUDA_TRY(cudaMemcpy(h_out + r * (size_t)rows * m->cfg.hidden, m->rec + r * (size_t)m->max_rows * m->cfg.hidden,
+                             sizeof(float) * (size_t)rows * m->cfg.hidden, cudaMemcpyDeviceToHost));
+  return B200_OK;
+}
+
+void b200_decoder_set_attn_mma(b200_decoder* m, int32_t on) {
+  m->attn_mma = on != 0;
+  m->drop_graphs();
+}
+
+}  // extern "C"

@@ -86,16 +86,17 @@ __global__ void embed_kernel(const __nv_bfloat16* __restrict__ table, const uint
 }
 
 // First strict maximum of each row (ties keep the smaller index).
-__global__ void argmax_kernel(const __nv_bfloat16* __restrict__ logits, int vocab, uint32_t* __restrict__ out) {
+template <typename T>
+__global__ void argmax_kernel(const T* __restrict__ logits, int vocab, uint32_t* __restrict__ out) {
   __shared__ float s_val[32];
   __shared__ int s_idx[32];
   const int row = blockIdx.x;
-  const __nv_bfloat16* lr = logits + (size_t)row * vocab;
+  const T* lr = logits + (size_t)row * vocab;
   float best = -INFINITY;
   int bi = 0x7fffffff;
   // 16-byte loads where the row allows it (row start and length multiples of 8 elements); a thread
   // meets its elements in increasing index order, so a strict > keeps the first maximum it saw.
-  const bool vec = (vocab % 8 == 0) && ((reinterpret_cast<uintptr_t>(lr) & 15) == 0);
+  const bool vec = sizeof(T) == 2 && (vocab % 8 == 0) && ((reinterpret_cast<uintptr_t>(lr) & 15) == 0);
   if (vec) {
     const uint4* lv = reinterpret_cast<const uint4*>(lr);
     for (int c = threadIdx.x; c < vocab / 8; c += blockDim.x) {
@@ -110,7 +111,7 @@ __global__ void argmax_kernel(const __nv_bfloat16* __restrict__ logits, int voca
     }
   } else {
     for (int i = threadIdx.x; i < vocab; i += blockDim.x) {
-      float v = __bfloat162float(lr[i]);
+      float v = (float)lr[i];
       if (v > best || (v == best && i < bi)) { best = v; bi = i; }
     }
   }
@@ -221,6 +222,15 @@ b200_status b200_argmax(const void* d_logits, int32_t rows, int32_t vocab, uint3
   if (st != B200_OK) return st;
   if (rows <= 0) return B200_OK;
   argmax_kernel<<<rows, 1024, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)d_logits, vocab, d_out);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+b200_status b200_argmax_f32(const float* d_logits, int32_t rows, int32_t vocab, uint32_t* d_out, void* stream) {
+  b200_status st = b200_require_device();
+  if (st != B200_OK) return st;
+  if (rows <= 0) return B200_OK;
+  argmax_kernel<<<rows, 1024, 0, (cudaStream_t)stream>>>(d_logits, vocab, d_out);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

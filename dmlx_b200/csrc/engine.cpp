@@ -1,6 +1,6 @@
 // Engine step: the caller the reference's framework is missing (its scheduler and batch builder are
 // "not wired up" to a forward pass, docs/en/technical/continuous-batching-design.md:187).  One call
-// runs schedule() -> ragged batch descriptors -> b200_llama_step -> postprocess(), i.e. the
+// runs schedule() -> ragged batch descriptors -> b200_model_step -> postprocess(), i.e. the
 // Engine_Step loop described at src/scheduler.zig:7-10, with the device page pool behind the
 // scheduler's BlockManager (admission takes one page, completion releases the sequence).
 //
@@ -16,7 +16,7 @@
 #include "common.h"
 
 struct b200_engine {
-  b200_llama* model = nullptr;
+  b200_model* model = nullptr;
   b200_kv* kv = nullptr;
   b200_sched_bm* bm = nullptr;
   b200_scheduler* sched = nullptr;
@@ -111,6 +111,10 @@ b200_status try_share_prefix(b200_engine* e, b200_request* r, b200_engine::Live*
 extern "C" {
 
 b200_engine* b200_engine_create(b200_llama* model, b200_kv* kv, uint64_t max_prefill_tokens) {
+  return b200_engine_create_model(b200_llama_model(model), kv, max_prefill_tokens);
+}
+
+b200_engine* b200_engine_create_model(b200_model* model, b200_kv* kv, uint64_t max_prefill_tokens) {
   auto* e = new b200_engine();
   e->model = model;
   e->kv = kv;
@@ -332,11 +336,11 @@ b200_status b200_engine_step(b200_engine* e, b200_token_output* out, uint64_t ca
       any = true;
     }
     if (any) {
-      st = b200_llama_set_samplers(e->model, e->samp_rows.data(), (int32_t)e->samp_rows.size());
+      st = b200_model_set_samplers(e->model, e->samp_rows.data(), (int32_t)e->samp_rows.size());
       if (st != B200_OK) return st;
     }
   }
-  st = b200_llama_step(e->model, e->kv, e->descs.data(), (int32_t)e->descs.size(), e->flat.data(), (int32_t)e->flat.size(),
+  st = b200_model_step(e->model, e->kv, e->descs.data(), (int32_t)e->descs.size(), e->flat.data(), (int32_t)e->flat.size(),
                        e->next.data(), &e->last_free_pages, stream);
   // A flagged step has changed neither the pool (the reservation is all or nothing) nor any sequence's
   // next input token: the scheduler state is left as it was and the caller may step again.

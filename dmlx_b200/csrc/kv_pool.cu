@@ -5,6 +5,8 @@
 //                    -> one (page, kv_head) tile is 32*head_dim contiguous elements (8 KiB for
 //                       bf16 at head_dim 128), the unit the attention kernel stages with one bulk
 //                       copy.
+//                    Pools made by b200_kv_create_layers keep the same order with heads and widths of each layer
+//                    (keys and values may differ) and hold bf16 or f32; KvLayerDev says where a layer starts.
 //   k_scale,v_scale: [layer][page][kv_head] f32 (FP8 pools only)
 //   free_stack     : [n_pages] i32, entries [0, free_top) are free; free_stack[free_top-1] pops next
 //   ref_count, tokens_used : [n_pages] i32
@@ -252,14 +254,15 @@ __global__ void __launch_bounds__(kReserveThreads) reserve_kernel(KvDev d, const
 // Copies every queued CoW page (all layers, K and V, scales for FP8 pools).
 __global__ void cow_copy_kernel(KvDev d) {
   const int n_cow = d.state[ST_N_COW];
-  const size_t page_bytes = (size_t)d.n_kv_heads * d.page_size * d.head_dim * d.elem_bytes;
+  const int layer = blockIdx.y >> 1, is_v = blockIdx.y & 1;
+  const KvLayerDev L = d.layer[layer];
+  const size_t page_bytes = (size_t)L.heads * d.page_size * (is_v ? L.vd : L.kd) * d.elem_bytes;  // multiple of 16
   const size_t vecs = page_bytes / 16;
+  char* base = is_v ? (char*)d.v_pool + L.v_off : (char*)d.k_pool + L.k_off;
   for (int c = blockIdx.x; c < n_cow; c += gridDim.x) {
     int2 pr = d.cow_list[c];
-    int layer = blockIdx.y >> 1, is_v = blockIdx.y & 1;
-    char* pool = (char*)(is_v ? d.v_pool : d.k_pool);
-    const uint4* src = (const uint4*)(pool + ((size_t)layer * d.n_pages + pr.x) * page_bytes);
-    uint4* dst = (uint4*)(pool + ((size_t)layer * d.n_pages + pr.y) * page_bytes);
+    const uint4* src = (const uint4*)(base + (size_t)pr.x * page_bytes);
+    uint4* dst = (uint4*)(base + (size_t)pr.y * page_bytes);
     for (size_t i = threadIdx.x; i < vecs; i += blockDim.x) dst[i] = src[i];
     if (d.elem_bytes == 1 && threadIdx.x < d.n_kv_heads) {
       float* sc = is_v ? d.v_scale : d.k_scale;
@@ -402,22 +405,26 @@ __global__ void append_fp8_kernel(KvDev d, int layer, const __nv_bfloat16* __res
   }
 }
 
-// Test helper: contiguous [len, H, D] bf16 view of one sequence of one layer.
-__global__ void gather_kernel(KvDev d, int layer, int seq, __nv_bfloat16* k_out, __nv_bfloat16* v_out, int cap_rows) {
+// Test helper: contiguous [len, H, key_dim] and [len, H, value_dim] views of one sequence of one layer (bf16, or f32 for
+// an f32 pool).
+__global__ void gather_kernel(KvDev d, int layer, int seq, void* k_out, void* v_out, int cap_rows) {
   const int len = min(d.seq_len[seq], cap_rows);
-  const int D = d.head_dim, H = d.n_kv_heads;
-  const size_t total = (size_t)len * H * D;
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-    int c = i % D, h = (i / D) % H, t = i / ((size_t)D * H);
-    int page = d.block_table[(size_t)seq * d.max_pages_per_seq + t / d.page_size];
-    size_t tile_idx = ((size_t)layer * d.n_pages + page) * H + h;
-    size_t off = tile_idx * (size_t)d.page_size * D + (size_t)(t % d.page_size) * D + c;
-    if (d.elem_bytes == 2) {
-      k_out[i] = ((const __nv_bfloat16*)d.k_pool)[off];
-      v_out[i] = ((const __nv_bfloat16*)d.v_pool)[off];
-    } else {
-      k_out[i] = __float2bfloat16(from_e4m3(((const unsigned char*)d.k_pool)[off]) * d.k_scale[tile_idx]);
-      v_out[i] = __float2bfloat16(from_e4m3(((const unsigned char*)d.v_pool)[off]) * d.v_scale[tile_idx]);
+  const KvLayerDev L = d.layer[layer];
+  for (int is_v = 0; is_v < 2; ++is_v) {
+    const int D = is_v ? L.value_dim : L.key_dim, W = is_v ? L.vd : L.kd;
+    const char* pool = is_v ? (const char*)d.v_pool + L.v_off : (const char*)d.k_pool + L.k_off;
+    const float* scales = is_v ? d.v_scale : d.k_scale;
+    void* out = is_v ? v_out : k_out;
+    const size_t total = (size_t)len * L.heads * D;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+      const int c = i % D, h = (i / D) % L.heads, t = i / ((size_t)D * L.heads);
+      const int page = d.block_table[(size_t)seq * d.max_pages_per_seq + t / d.page_size];
+      const size_t off = (((size_t)page * L.heads + h) * d.page_size + t % d.page_size) * (size_t)W + c;
+      if (d.elem_bytes == 4) ((float*)out)[i] = ((const float*)pool)[off];
+      else if (d.elem_bytes == 2) ((__nv_bfloat16*)out)[i] = ((const __nv_bfloat16*)pool)[off];
+      else
+        ((__nv_bfloat16*)out)[i] = __float2bfloat16(from_e4m3(((const unsigned char*)pool)[off]) *
+                                                    scales[((size_t)layer * d.n_pages + page) * L.heads + h]);
     }
   }
 }
@@ -529,18 +536,50 @@ static b200_status run_admin(b200_kv* kv, int op, int a0, int a1, int a2, const 
 
 extern "C" {
 
+static b200_status kv_create(const b200_kv_config* c, const b200_kv_layer* layers, b200_kv** out);
+
 b200_status b200_kv_create(const b200_kv_config* c, b200_kv** out) {
   *out = nullptr;
+  if (c->kv_dtype != B200_KV_BF16 && c->kv_dtype != B200_KV_FP8_E4M3) {
+    b200_set_error("kv_dtype %d: pools of one shape hold bf16 (0) or FP8-E4M3 (1) pages", c->kv_dtype);
+    b200_status st = b200_require_device();
+    return st != B200_OK ? st : B200_ERR_INVALID_QUANT_BITS;
+  }
+  return kv_create(c, nullptr, out);
+}
+
+b200_status b200_kv_create_layers(const b200_kv_config* c, const b200_kv_layer* layers, b200_kv** out) {
+  *out = nullptr;
+  if (!layers) { b200_set_error("kv_create_layers: no layer shapes"); return B200_ERR_INVALID_ARGUMENT; }
+  if (c->kv_dtype != B200_KV_BF16 && c->kv_dtype != B200_KV_F32) {
+    b200_set_error("kv_dtype %d: layered pools hold bf16 (0) or f32 (2) pages", c->kv_dtype);
+    b200_status st = b200_require_device();
+    return st != B200_OK ? st : B200_ERR_INVALID_QUANT_BITS;
+  }
+  return kv_create(c, layers, out);
+}
+
+static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* layers, b200_kv** out) {
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
-  if (c->page_size != 32) { b200_set_error("page_size must be 32"); return B200_ERR_INVALID_ARGUMENT; }
-  if (c->kv_dtype != B200_KV_BF16 && c->kv_dtype != B200_KV_FP8_E4M3) {
-    b200_set_error("kv_dtype %d: only bf16 (0) and FP8-E4M3 (1) pages exist", c->kv_dtype);
-    return B200_ERR_INVALID_QUANT_BITS;
+  b200_kv_config cfg = *c_in;
+  if (layers && cfg.n_layers > 0) {  // the uniform fields hold the widest layer (never used to address a layered pool)
+    cfg.n_kv_heads = 1;
+    cfg.head_dim = 0;
+    for (int l = 0; l < cfg.n_layers; ++l) {
+      if (layers[l].n_kv_heads <= 0 || layers[l].key_dim <= 0 || layers[l].value_dim <= 0) {
+        b200_set_error("kv_create_layers: layer %d has no shape", l);
+        return B200_ERR_INVALID_ARGUMENT;
+      }
+      cfg.n_kv_heads = std::max(cfg.n_kv_heads, layers[l].n_kv_heads);
+      cfg.head_dim = std::max(cfg.head_dim, std::max(layers[l].key_dim, layers[l].value_dim));
+    }
   }
-  if (c->head_dim != 64 && c->head_dim != 128) { b200_set_error("head_dim must be 64 or 128"); return B200_ERR_INVALID_ARGUMENT; }
+  const b200_kv_config* c = &cfg;
+  if (c->page_size != 32) { b200_set_error("page_size must be 32"); return B200_ERR_INVALID_ARGUMENT; }
+  if (!layers && c->head_dim != 64 && c->head_dim != 128) { b200_set_error("head_dim must be 64 or 128"); return B200_ERR_INVALID_ARGUMENT; }
   if (c->n_layers <= 0 || c->n_kv_heads <= 0 || c->n_pages <= 0 || c->max_seqs <= 0 || c->max_pages_per_seq <= 0 ||
-      c->max_rows <= 0 || c->n_q_heads <= 0 || c->n_q_heads % c->n_kv_heads != 0) {
+      c->max_rows <= 0 || c->n_q_heads <= 0 || (!layers && c->n_q_heads % c->n_kv_heads != 0)) {
     b200_set_error("invalid pool configuration");
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -549,9 +588,26 @@ b200_status b200_kv_create(const b200_kv_config* c, b200_kv** out) {
   KvDev& d = kv->dev;
   d.n_layers = c->n_layers; d.n_kv_heads = c->n_kv_heads; d.head_dim = c->head_dim; d.page_size = c->page_size;
   d.n_pages = c->n_pages; d.max_seqs = c->max_seqs; d.max_pages_per_seq = c->max_pages_per_seq;
-  d.elem_bytes = c->kv_dtype == B200_KV_BF16 ? 2 : 1;
+  d.elem_bytes = c->kv_dtype == B200_KV_BF16 ? 2 : (c->kv_dtype == B200_KV_F32 ? 4 : 1);
   d.max_touch = std::max(c->max_rows, c->n_pages + c->max_seqs);  // a bulk fill may touch every page
-  size_t pool_bytes = (size_t)c->n_layers * c->n_pages * c->n_kv_heads * c->page_size * c->head_dim * d.elem_bytes;
+  // Layers lie one behind the other.  A layered pool stores rows of a multiple of 16 elements (zero behind the model's
+  // width), so a token row is a whole number of 32-byte sectors and a TMA-addressable stride.
+  kv->layered = layers != nullptr;
+  kv->lay.resize(c->n_layers);
+  size_t k_bytes = 0, v_bytes = 0;
+  for (int l = 0; l < c->n_layers; ++l) {
+    KvLayerDev& L = kv->lay[l];
+    L.heads = layers ? layers[l].n_kv_heads : c->n_kv_heads;
+    L.key_dim = layers ? layers[l].key_dim : c->head_dim;
+    L.value_dim = layers ? layers[l].value_dim : c->head_dim;
+    L.kd = layers ? (L.key_dim + 15) / 16 * 16 : L.key_dim;
+    L.vd = layers ? (L.value_dim + 15) / 16 * 16 : L.value_dim;
+    L.k_off = k_bytes;
+    L.v_off = v_bytes;
+    k_bytes += (size_t)c->n_pages * L.heads * c->page_size * L.kd * d.elem_bytes;
+    v_bytes += (size_t)c->n_pages * L.heads * c->page_size * L.vd * d.elem_bytes;
+    kv->max_vd = std::max(kv->max_vd, L.vd);
+  }
   size_t n_tiles = (size_t)c->n_layers * c->n_pages * c->n_kv_heads;
 #define KV_ALLOC(ptr, bytes)                                            \
   do {                                                                  \
@@ -562,8 +618,10 @@ b200_status b200_kv_create(const b200_kv_config* c, b200_kv** out) {
       return B200_ERR_CUDA;                                             \
     }                                                                   \
   } while (0)
-  KV_ALLOC(d.k_pool, pool_bytes);
-  KV_ALLOC(d.v_pool, pool_bytes);
+  KV_ALLOC(d.k_pool, k_bytes);
+  KV_ALLOC(d.v_pool, v_bytes);
+  KV_ALLOC(d.layer, sizeof(KvLayerDev) * c->n_layers);
+  cudaMemcpy(const_cast<KvLayerDev*>(d.layer), kv->lay.data(), sizeof(KvLayerDev) * c->n_layers, cudaMemcpyHostToDevice);
   if (d.elem_bytes == 1) {
     KV_ALLOC(d.k_scale, n_tiles * sizeof(float));
     KV_ALLOC(d.v_scale, n_tiles * sizeof(float));
@@ -584,15 +642,28 @@ b200_status b200_kv_create(const b200_kv_config* c, b200_kv** out) {
   kv->max_chunks = c->attn_scratch_chunks > 0 ? c->attn_scratch_chunks : c->n_pages / 4 + c->max_rows + 8;
   KV_ALLOC(kv->d_chunk_start, sizeof(int) * (c->max_rows + 2));
   KV_ALLOC(kv->d_groups, sizeof(int) * 3 * (c->max_rows + 2));
-  KV_ALLOC(kv->d_part_o, sizeof(float) * (size_t)kv->max_chunks * c->n_q_heads * c->head_dim);
+  KV_ALLOC(kv->d_part_o, sizeof(float) * (size_t)kv->max_chunks * c->n_q_heads * kv->max_vd);
   KV_ALLOC(kv->d_part_ml, sizeof(float) * (size_t)kv->max_chunks * c->n_q_heads * 2);
 #undef KV_ALLOC
   cudaMemset(d.block_table, 0, sizeof(int) * (size_t)c->max_seqs * c->max_pages_per_seq);
   // Pages start zeroed so that slots never written hold finite values: attention multiplies
   // masked slots by a zero weight instead of branching around them.
-  cudaMemset(d.k_pool, 0, pool_bytes);
-  cudaMemset(d.v_pool, 0, pool_bytes);
-  if (d.elem_bytes == 2) {
+  cudaMemset(d.k_pool, 0, k_bytes);
+  cudaMemset(d.v_pool, 0, v_bytes);
+  if (layers && d.elem_bytes == 2) {
+    kv->lay_kmap.resize(c->n_layers);
+    kv->lay_vmap.resize(c->n_layers);
+    const uint32_t box[2] = {64, 32};
+    for (int l = 0; l < c->n_layers && st == B200_OK; ++l) {
+      const KvLayerDev& L = kv->lay[l];
+      const uint64_t rows = (uint64_t)c->n_pages * L.heads * c->page_size;
+      const uint64_t kdims[2] = {(uint64_t)L.kd, rows}, vdims[2] = {(uint64_t)L.vd, rows};
+      const uint64_t kst[1] = {(uint64_t)L.kd * 2}, vst[1] = {(uint64_t)L.vd * 2};
+      st = b200_make_tensor_map(&kv->lay_kmap[l], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (char*)d.k_pool + L.k_off, kdims, kst, box);
+      if (st == B200_OK) st = b200_make_tensor_map(&kv->lay_vmap[l], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (char*)d.v_pool + L.v_off, vdims, vst, box);
+    }
+    if (st != B200_OK) { b200_kv_destroy(kv); return st; }
+  } else if (!layers && d.elem_bytes == 2) {
     const uint64_t rows_per_layer = (uint64_t)c->n_pages * c->n_kv_heads * c->page_size;
     const uint64_t dims[3] = {(uint64_t)c->head_dim, rows_per_layer, (uint64_t)c->n_layers};
     const uint64_t strides[2] = {(uint64_t)c->head_dim * 2, rows_per_layer * c->head_dim * 2};
@@ -600,7 +671,7 @@ b200_status b200_kv_create(const b200_kv_config* c, b200_kv** out) {
     st = b200_make_tensor_map(&kv->kmap, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, d.k_pool, dims, strides, box);
     if (st == B200_OK) st = b200_make_tensor_map(&kv->vmap, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, d.v_pool, dims, strides, box);
     if (st != B200_OK) { b200_kv_destroy(kv); return st; }
-  } else if (c->head_dim == 128) {
+  } else if (!layers && c->head_dim == 128) {
     // FP8 pools: a token row of one head is 128 bytes, a page tile one 128 x 32 box
     const uint64_t rows_per_layer = (uint64_t)c->n_pages * c->n_kv_heads * c->page_size;
     const uint64_t dims[3] = {128, rows_per_layer, (uint64_t)c->n_layers};
@@ -621,8 +692,12 @@ void b200_kv_destroy(b200_kv* kv) {
   KvDev& d = kv->dev;
   void* ptrs[] = {d.k_pool, d.v_pool, d.k_scale, d.v_scale, d.free_stack, d.ref_count, d.tokens_used, d.block_table,
                   d.seq_pages, d.seq_len, d.state, d.touch_list, d.cow_list, kv->d_admin_in, kv->d_admin_out,
-                  kv->d_chunk_start, kv->d_part_o, kv->d_part_ml, kv->d_groups};
+                  kv->d_chunk_start, kv->d_part_o, kv->d_part_ml, kv->d_groups, const_cast<KvLayerDev*>(d.layer)};
   for (void* p : ptrs) if (p) cudaFree(p);
+  for (WindowPlan* p : kv->plans) {
+    if (p->buf) cudaFree(p->buf);
+    delete p;
+  }
   delete kv;
 }
 
@@ -710,6 +785,7 @@ b200_status b200_kv_append(b200_kv* kv, int32_t layer, const void* d_k_rows, con
 b200_status b200_kv_append_strided(b200_kv* kv, int32_t layer, const void* d_k_rows, const void* d_v_rows,
                                    int32_t k_stride, int32_t v_stride, int32_t total_rows, void* stream) {
   if (layer < 0 || layer >= kv->cfg.n_layers) { b200_set_error("append: layer %d out of range", layer); return B200_ERR_INVALID_ARGUMENT; }
+  if (kv->layered) { b200_set_error("append: layered pools are written by the decoder step"); return B200_ERR_UNSUPPORTED; }
   if (total_rows <= 0) return B200_OK;
   cudaStream_t s = (cudaStream_t)stream;
   int gx = std::min(total_rows, 2048);
@@ -798,7 +874,7 @@ extern "C" b200_status b200_kv_rope_append_partials(b200_kv* kv, int32_t layer, 
                                                     const int32_t* d_positions, const int32_t* d_row_seq, int32_t total_rows,
                                                     int32_t n_q_heads, float theta, void* stream) {
   const b200_kv_config& c = kv->cfg;
-  if (c.kv_dtype != B200_KV_BF16 || c.head_dim != 128) { b200_set_error("rope+append from partial sums: bf16 pools with head_dim 128 only"); return B200_ERR_UNSUPPORTED; }
+  if (kv->layered || c.kv_dtype != B200_KV_BF16 || c.head_dim != 128) { b200_set_error("rope+append from partial sums: bf16 pools with head_dim 128 only"); return B200_ERR_UNSUPPORTED; }
   if (!parts || !parts->pending || !parts->d_ws || parts->rows != total_rows || parts->n != (n_q_heads + 2 * c.n_kv_heads) * 128 ||
       parts->nt * 128 != parts->n || parts->tn <= 0 || parts->tts != (total_rows + parts->tn - 1) / parts->tn || parts->splits <= 0) {
     b200_set_error("rope+append from partial sums: the partial sums do not describe a q/k/v projection of %d rows", total_rows);
@@ -817,6 +893,7 @@ b200_status b200_kv_rope_append_strided(b200_kv* kv, int32_t layer, void* d_q, c
                                         int32_t q_stride, int32_t k_stride, int32_t v_stride, const int32_t* d_positions,
                                         const int32_t* d_row_seq, int32_t total_rows, int32_t n_q_heads, float theta, void* stream) {
   const b200_kv_config& c = kv->cfg;
+  if (kv->layered) { b200_set_error("append: layered pools are written by the decoder step"); return B200_ERR_UNSUPPORTED; }
   if (c.kv_dtype != B200_KV_BF16 || (c.head_dim != 64 && c.head_dim != 128)) {
     b200_status st = b200_rope(d_q, const_cast<void*>(d_k_rows), d_positions, total_rows, n_q_heads, c.n_kv_heads, c.head_dim, q_stride,
                                k_stride, theta, stream);
@@ -882,8 +959,7 @@ b200_status b200_kv_gather(b200_kv* kv, int32_t layer, int32_t seq, void* d_k_ou
     b200_set_error("gather: layer/slot out of range");
     return B200_ERR_INVALID_BATCH_INDEX;
   }
-  gather_kernel<<<296, 256, 0, (cudaStream_t)stream>>>(kv->dev, layer, seq, (__nv_bfloat16*)d_k_out,
-                                                       (__nv_bfloat16*)d_v_out, cap_rows);
+  gather_kernel<<<296, 256, 0, (cudaStream_t)stream>>>(kv->dev, layer, seq, d_k_out, d_v_out, cap_rows);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -896,10 +972,10 @@ b200_status b200_kv_page_load(b200_kv* kv, int32_t layer, int32_t page, const vo
   }
   const KvDev& d = kv->dev;
   if (d.elem_bytes == 1 && (!h_k_scales || !h_v_scales)) { b200_set_error("page_load: FP8 pages need their scales"); return B200_ERR_INVALID_ARGUMENT; }
-  size_t page_bytes = (size_t)d.n_kv_heads * d.page_size * d.head_dim * d.elem_bytes;
-  size_t off = ((size_t)layer * d.n_pages + page) * page_bytes;
-  B200_CUDA_TRY(cudaMemcpy((char*)d.k_pool + off, h_k, page_bytes, cudaMemcpyHostToDevice));
-  B200_CUDA_TRY(cudaMemcpy((char*)d.v_pool + off, h_v, page_bytes, cudaMemcpyHostToDevice));
+  const KvLayerDev& L = kv->lay[layer];
+  const size_t k_bytes = (size_t)L.heads * d.page_size * L.kd * d.elem_bytes, v_bytes = (size_t)L.heads * d.page_size * L.vd * d.elem_bytes;
+  B200_CUDA_TRY(cudaMemcpy((char*)d.k_pool + L.k_off + (size_t)page * k_bytes, h_k, k_bytes, cudaMemcpyHostToDevice));
+  B200_CUDA_TRY(cudaMemcpy((char*)d.v_pool + L.v_off + (size_t)page * v_bytes, h_v, v_bytes, cudaMemcpyHostToDevice));
   if (d.elem_bytes == 1) {
     size_t so = ((size_t)layer * d.n_pages + page) * d.n_kv_heads;
     B200_CUDA_TRY(cudaMemcpy(d.k_scale + so, h_k_scales, sizeof(float) * d.n_kv_heads, cudaMemcpyHostToDevice));
@@ -915,13 +991,14 @@ __global__ void __launch_bounds__(256) copy_pages_kernel(KvDev src, KvDev dst, c
                                                          const int* __restrict__ dst_table) {
   const int layer = blockIdx.y, sp = src_table[blockIdx.x], dp = dst_table[blockIdx.x];
   if (sp < 0 || sp >= src.n_pages || dp < 0 || dp >= dst.n_pages) return;
-  const size_t page_bytes = (size_t)src.n_kv_heads * src.page_size * src.head_dim * src.elem_bytes;  // multiple of 16
-  const size_t so = ((size_t)layer * src.n_pages + sp) * page_bytes, dof = ((size_t)layer * dst.n_pages + dp) * page_bytes;
-  const uint4* sk = reinterpret_cast<const uint4*>((const char*)src.k_pool + so);
-  const uint4* sv = reinterpret_cast<const uint4*>((const char*)src.v_pool + so);
-  uint4* dk = reinterpret_cast<uint4*>((char*)dst.k_pool + dof);
-  uint4* dv = reinterpret_cast<uint4*>((char*)dst.v_pool + dof);
-  for (size_t i = threadIdx.x; i < page_bytes / 16; i += blockDim.x) { dk[i] = sk[i]; dv[i] = sv[i]; }
+  const KvLayerDev L = src.layer[layer], M = dst.layer[layer];  // the same shapes; the pools may differ in page count
+  const size_t k_bytes = (size_t)L.heads * src.page_size * L.kd * src.elem_bytes, v_bytes = (size_t)L.heads * src.page_size * L.vd * src.elem_bytes;
+  const uint4* sk = reinterpret_cast<const uint4*>((const char*)src.k_pool + L.k_off + (size_t)sp * k_bytes);
+  const uint4* sv = reinterpret_cast<const uint4*>((const char*)src.v_pool + L.v_off + (size_t)sp * v_bytes);
+  uint4* dk = reinterpret_cast<uint4*>((char*)dst.k_pool + M.k_off + (size_t)dp * k_bytes);
+  uint4* dv = reinterpret_cast<uint4*>((char*)dst.v_pool + M.v_off + (size_t)dp * v_bytes);
+  for (size_t i = threadIdx.x; i < k_bytes / 16; i += blockDim.x) dk[i] = sk[i];
+  for (size_t i = threadIdx.x; i < v_bytes / 16; i += blockDim.x) dv[i] = sv[i];
   if (src.elem_bytes == 1 && threadIdx.x < src.n_kv_heads) {
     const size_t ss = ((size_t)layer * src.n_pages + sp) * src.n_kv_heads + threadIdx.x;
     const size_t ds = ((size_t)layer * dst.n_pages + dp) * dst.n_kv_heads + threadIdx.x;
@@ -936,6 +1013,12 @@ b200_status b200_kv_extend(b200_kv* kv, int32_t dst_seq, b200_kv* src, int32_t s
       a.kv_dtype != b.kv_dtype) {
     b200_set_error("extend: the two pools differ in shape or element type");
     return B200_ERR_INVALID_ARGUMENT;
+  }
+  for (int l = 0; l < a.n_layers; ++l) {
+    if (kv->lay[l].heads != src->lay[l].heads || kv->lay[l].kd != src->lay[l].kd || kv->lay[l].vd != src->lay[l].vd) {
+      b200_set_error("extend: the two pools differ in the shape of layer %d", l);
+      return B200_ERR_INVALID_ARGUMENT;
+    }
   }
   if (dst_seq < 0 || dst_seq >= a.max_seqs || src_seq < 0 || src_seq >= b.max_seqs) {
     b200_set_error("extend: slot out of range");
@@ -976,10 +1059,10 @@ b200_status b200_kv_page_raw(b200_kv* kv, int32_t layer, int32_t page, void* h_k
     return B200_ERR_INVALID_BLOCK_ID;
   }
   const KvDev& d = kv->dev;
-  size_t page_bytes = (size_t)d.n_kv_heads * d.page_size * d.head_dim * d.elem_bytes;
-  size_t off = ((size_t)layer * d.n_pages + page) * page_bytes;
-  B200_CUDA_TRY(cudaMemcpy(h_k, (char*)d.k_pool + off, page_bytes, cudaMemcpyDeviceToHost));
-  B200_CUDA_TRY(cudaMemcpy(h_v, (char*)d.v_pool + off, page_bytes, cudaMemcpyDeviceToHost));
+  const KvLayerDev& L = kv->lay[layer];
+  const size_t k_bytes = (size_t)L.heads * d.page_size * L.kd * d.elem_bytes, v_bytes = (size_t)L.heads * d.page_size * L.vd * d.elem_bytes;
+  B200_CUDA_TRY(cudaMemcpy(h_k, (char*)d.k_pool + L.k_off + (size_t)page * k_bytes, k_bytes, cudaMemcpyDeviceToHost));
+  B200_CUDA_TRY(cudaMemcpy(h_v, (char*)d.v_pool + L.v_off + (size_t)page * v_bytes, v_bytes, cudaMemcpyDeviceToHost));
   if (d.elem_bytes == 1 && h_k_scales && h_v_scales) {
     size_t so = ((size_t)layer * d.n_pages + page) * d.n_kv_heads;
     B200_CUDA_TRY(cudaMemcpy(h_k_scales, d.k_scale + so, sizeof(float) * d.n_kv_heads, cudaMemcpyDeviceToHost));

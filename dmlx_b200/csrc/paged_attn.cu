@@ -1606,6 +1606,7 @@ b200_status b200_paged_attn_decode_strided(b200_kv* kv, int32_t layer, const voi
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
   const b200_kv_config& c = kv->cfg;
+  if (kv->layered) { b200_set_error("attention: layered pools are read by the decoder step's attention"); return B200_ERR_UNSUPPORTED; }
   if (layer < 0 || layer >= c.n_layers) { b200_set_error("attention: layer %d out of range", layer); return B200_ERR_INVALID_ARGUMENT; }
   const bool fp8 = c.kv_dtype == B200_KV_FP8_E4M3;
   // MMA rows 0..7 carry the group's heads; the FP8 tensor-core kernel is built for head_dim 128
@@ -1657,7 +1658,7 @@ b200_status b200_paged_attn_prefill_strided(b200_kv* kv, int32_t layer, const vo
   // Grouping needs the GQA group to divide the 16 MMA rows, and head_dim 128 for FP8 pools; anything
   // else takes the per-row kernels (same results).
   const bool fp8 = c.kv_dtype == B200_KV_FP8_E4M3;
-  if ((fp8 && c.head_dim != 128) || !(G == 1 || G == 2 || G == 4 || G == 8) || b200_attn_path == 1)
+  if (kv->layered || (fp8 && c.head_dim != 128) || !(G == 1 || G == 2 || G == 4 || G == 8) || b200_attn_path == 1)
     return b200_paged_attn_decode_strided(kv, layer, d_q, q_stride, d_row_seq, d_row_ctx, total_rows, d_out, stream, reuse_plan);
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;

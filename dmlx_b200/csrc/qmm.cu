@@ -429,7 +429,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
       const int n = nt * kTileN + warp * 32 + lane;
       // One K split and a small token tile: apply the epilogue here and skip the finish kernel.  With
       // large token tiles the strided 64-byte row stores cost more than the extra pass.
-      const bool direct = gridDim.y == 1 && tn <= 64;
+      const bool direct = gridDim.y == 1 && tn <= 64 && !a.keep_f32;
       const size_t n_pad = a.items ? (size_t)a.nt * kTileN : (size_t)kTileN;  // stride between token rows
       float* wsp = a.items ? a.ws + ((size_t)split * a.rows + t0) * n_pad + n
                            : a.ws + (((size_t)(nt * gridDim.z + blockIdx.z) * gridDim.y + split) * tn) * kTileN + warp * 32 + lane;
@@ -728,7 +728,7 @@ __global__ void __launch_bounds__(kTcaThreads, 2) qmm_tca_kernel(const __grid_co
     if (ok && warp < 4) {
       ptx::tc_fence_after_sync();
       const int n = nt * kTileN + warp * 32 + lane;
-      const bool direct = gridDim.y == 1 && (tn <= 64 || a.direct_large);
+      const bool direct = gridDim.y == 1 && (tn <= 64 || a.direct_large) && !a.keep_f32;
       const size_t n_pad = a.items ? (size_t)a.nt * kTileN : (size_t)kTileN;
       float* wsp = a.items ? a.ws + ((size_t)split * a.rows + t0) * n_pad + n
                            : a.ws + (((size_t)(nt * gridDim.z + blockIdx.z) * gridDim.y + split) * tn) * kTileN + warp * 32 + lane;
@@ -960,7 +960,7 @@ __global__ void __launch_bounds__(kTc2Threads, 1) qmm_tc2_kernel(const __grid_co
       ptx::tc_fence_after_sync();
       const int lq = warp & 3;
       const int nt = nt0 + etile, n = nt * kTileN + lq * 32 + lane;
-      const bool direct = gridDim.y == 1;
+      const bool direct = gridDim.y == 1 && !a.keep_f32;
       float* wsp = a.ws + (((size_t)(nt * gridDim.z + tt) * gridDim.y + split) * tn) * kTileN + lq * 32 + lane;
       const int ch = ((tn / 2 + 31) / 32) * 32;
       const int c_end = min(rows_here, (half + 1) * ch);
@@ -2361,7 +2361,7 @@ static b200_status launch_tc(QmmArgs& a, int rows, cudaStream_t s) {
   a.x_row0 = 0;
   qmm_tc_kernel<MODE><<<dim3(a.nt, splits, a.items ? a.max_items : tts), kTcThreads, smem, s>>>(xmap, a);
   B200_LAUNCH_CHECK();
-  return (splits == 1 && tn <= 64) ? B200_OK : launch_finish(a, splits, s);  // a single small split writes its output itself
+  return (splits == 1 && tn <= 64 && !a.keep_f32) ? B200_OK : launch_finish(a, splits, s);  // a single small split writes its output itself
 }
 
 // Quantised weights, up to 128 rows per token tile (dense) or grouped work items: dequantised weights
@@ -2410,7 +2410,7 @@ static b200_status launch_tca(QmmArgs& a, int rows, cudaStream_t s) {
   // ... and so does a single K split of up to 128-row tiles (gate/up at 128 rows 44.9 -> 42.9 us, lm_head 159 -> 147 us;
   // with 256-row tiles at one CTA per SM the longer epilogue costs more than the finish pass: 290 -> 302 us)
   a.direct_large = (!a.items && splits == 1 && (tts >= 4 || tn <= 128)) ? 1 : 0;
-  const bool direct = splits == 1 && (tn <= 64 || a.direct_large);
+  const bool direct = splits == 1 && (tn <= 64 || a.direct_large) && !a.keep_f32;
   st = ensure_state(direct ? 0 : (size_t)splits * (a.items ? (size_t)rows : (size_t)tts * tn) * a.nt * kTileN * sizeof(float));
   if (st != B200_OK) return st;
   a.ws = g_ws; a.err = g_err;
@@ -2603,7 +2603,7 @@ static b200_status launch_tc2(QmmArgs& a, int rows, cudaStream_t s) {
   const int splits0 = pick_splits(pairs * tts, a.kc, g_sms, 1, 2 + tn / 32);
   a.chunks_per_split = (a.kc + splits0 - 1) / splits0;
   const int splits = (a.kc + a.chunks_per_split - 1) / a.chunks_per_split;
-  st = ensure_state(splits > 1 ? (size_t)splits * (size_t)tts * tn * a.nt * kTileN * sizeof(float) : 0);
+  st = ensure_state(splits > 1 || a.keep_f32 ? (size_t)splits * (size_t)tts * tn * a.nt * kTileN * sizeof(float) : 0);
   if (st != B200_OK) return st;
   a.ws = g_ws; a.err = g_err;
   CUtensorMap xmap;
@@ -2612,7 +2612,7 @@ static b200_status launch_tc2(QmmArgs& a, int rows, cudaStream_t s) {
   a.x_row0 = 0;
   qmm_tc2_kernel<MODE><<<dim3(pairs, splits, tts), kTc2Threads, smem, s>>>(xmap, a);
   B200_LAUNCH_CHECK();
-  return splits == 1 ? B200_OK : launch_finish(a, splits, s);
+  return splits == 1 && !a.keep_f32 ? B200_OK : launch_finish(a, splits, s);
 }
 
 template <int MODE, int NT8>
@@ -2734,13 +2734,17 @@ extern "C" b200_status b200_qmm(const b200_qweight* w, const void* d_x, int32_t 
 
 // Set by b200_qmm_deferred around its call of qmm_entry (one calling thread per process uses the matmul entry points).
 static b200_qmm_partials* g_defer_target = nullptr;
+static bool g_defer_always = false;  // defer = 2: also when K is not split
 
 extern "C" b200_status b200_qmm_deferred(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t defer, void* stream,
                                          b200_qmm_partials* out) {
   std::memset(out, 0, sizeof(*out));
+  if (defer == 2 && w->mode == B200_Q_MXFP4_G32) { b200_set_error("qmm_deferred: f32 sums of MXFP4 weights are not kept"); return B200_ERR_UNSUPPORTED; }
   g_defer_target = defer ? out : nullptr;
+  g_defer_always = defer == 2;
   const b200_status st = qmm_entry(w, d_x, rows, d_y, B200_EPI_NONE, nullptr, 0.f, B200_QMM_AUTO, stream, nullptr, 0.f, nullptr, nullptr);
   g_defer_target = nullptr;
+  g_defer_always = false;
   return st;
 }
 
@@ -2812,6 +2816,7 @@ static b200_status qmm_entry(const b200_qweight* w, const void* d_x, int32_t row
   a.rows = rows; a.n = w->n; a.k = w->k; a.nt = w->nt; a.kc = w->kc; a.epilogue = epilogue; a.swiglu_limit = swiglu_limit;
   a.norm_w = (const __nv_bfloat16*)d_norm_w; a.norm_out = (__nv_bfloat16*)d_norm_out; a.norm_eps = norm_eps;
   a.defer = g_defer_target;
+  a.keep_f32 = g_defer_always ? 1 : 0;
   cudaStream_t s = (cudaStream_t)stream;
   auto dispatch = [&]() -> b200_status {
     if (path == B200_QMM_MXFP4_BLOCK_SCALED) return launch_mx(w, a, rows, s);
@@ -2840,6 +2845,95 @@ static b200_status qmm_entry(const b200_qweight* w, const void* d_x, int32_t row
   st = dispatch();
   if (did_norm) *did_norm = a.did_norm;
   return st;
+}
+
+// ---- 32-bit matmul ---------------------------------------------------------------------------------------
+// f32 activations times dense bf16 weights (widened exactly), f32 accumulation on the CUDA cores.  CTA tile: 64 rows x one
+// weight tile of 128, 32 columns of K at a time in shared memory; a thread owns 8 rows x 4 outputs.
+namespace {
+constexpr int kF32Rows = 64, kF32K = 32;
+
+__global__ void __launch_bounds__(256) qmm_f32_kernel(const unsigned char* __restrict__ blocks, const float* __restrict__ x, int rows, int k, int kc,
+                                                      float* __restrict__ y, int y_stride, int n_valid, int swiglu) {
+  __shared__ float xs[kF32K][kF32Rows + 4];
+  __shared__ float ws[kF32K][kTileN + 4];
+  const int nt = blockIdx.x, r0 = blockIdx.y * kF32Rows, tid = threadIdx.x;
+  const int tr = (tid / 32) * 8, tc = (tid % 32) * 4;
+  float acc[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f; }
+  for (int c = 0; c < kc; ++c) {
+    const unsigned char* blk = blocks + ((size_t)nt * kc + c) * (kTileN * 128);
+    for (int half = 0; half < 2; ++half) {
+      for (int i = tid; i < kTileN * 4; i += 256) {  // 16-byte chunks: row r, chunk position swizzled within its 128 bytes
+        const int r = i >> 2, cc = half * 4 + (i & 3);
+        const uint4 v = *reinterpret_cast<const uint4*>(blk + r * 128 + ((cc ^ (r & 7)) << 4));
+        const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          ws[(i & 3) * 8 + 2 * e][r] = ptx::bf16_lo(w[e]);
+          ws[(i & 3) * 8 + 2 * e + 1][r] = ptx::bf16_hi(w[e]);
+        }
+      }
+      for (int i = tid; i < kF32Rows * (kF32K / 4); i += 256) {
+        const int r = i / (kF32K / 4), q = i % (kF32K / 4);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r0 + r < rows) v = *reinterpret_cast<const float4*>(x + (size_t)(r0 + r) * k + c * kChunkK + half * kF32K + q * 4);
+        xs[q * 4][r] = v.x; xs[q * 4 + 1][r] = v.y; xs[q * 4 + 2][r] = v.z; xs[q * 4 + 3][r] = v.w;
+      }
+      __syncthreads();
+#pragma unroll 8
+      for (int kk = 0; kk < kF32K; ++kk) {
+        const float4 w = *reinterpret_cast<const float4*>(&ws[kk][tc]);
+        const float4 xa = *reinterpret_cast<const float4*>(&xs[kk][tr]), xb = *reinterpret_cast<const float4*>(&xs[kk][tr + 4]);
+        const float xv[8] = {xa.x, xa.y, xa.z, xa.w, xb.x, xb.y, xb.z, xb.w};
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          acc[i][0] = fmaf(xv[i], w.x, acc[i][0]);
+          acc[i][1] = fmaf(xv[i], w.y, acc[i][1]);
+          acc[i][2] = fmaf(xv[i], w.z, acc[i][2]);
+          acc[i][3] = fmaf(xv[i], w.w, acc[i][3]);
+        }
+      }
+      __syncthreads();
+    }
+  }
+  const int n = nt * kTileN + tc;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int row = r0 + tr + i;
+    if (row >= rows) continue;
+    if (swiglu) {  // columns alternate gate, up
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int col = n / 2 + e;
+        const float gt = acc[i][2 * e], up = acc[i][2 * e + 1];
+        if (col < n_valid) y[(size_t)row * y_stride + col] = gt / (1.0f + expf(-gt)) * up;
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (n + e < n_valid) y[(size_t)row * y_stride + n + e] = acc[i][e];
+    }
+  }
+}
+}  // namespace
+
+extern "C" b200_status b200_qmm_f32(const b200_qweight* w, const float* d_x, int32_t rows, float* d_y, int32_t y_stride, int32_t n_valid,
+                                    int32_t epilogue, void* stream) {
+  b200_status st = b200_require_device();
+  if (st != B200_OK) return st;
+  if (w->mode != B200_Q_BF16 || w->n_experts != 1) { b200_set_error("qmm_f32: dense bf16 weights only"); return B200_ERR_UNSUPPORTED; }
+  const bool swiglu = epilogue == B200_EPI_SWIGLU;
+  if ((epilogue != B200_EPI_NONE && !swiglu) || n_valid < 0 || n_valid > (swiglu ? w->n / 2 : w->n) || y_stride < n_valid) {
+    b200_set_error("qmm_f32: bad epilogue, n_valid or stride");
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  if (rows <= 0) return B200_OK;
+  qmm_f32_kernel<<<dim3(w->nt, (rows + kF32Rows - 1) / kF32Rows), 256, 0, (cudaStream_t)stream>>>(w->d_blocks, d_x, rows, w->k, w->kc, d_y, y_stride,
+                                                                                                n_valid, swiglu ? 1 : 0);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
 }
 
 // Grouped matmul over an expert-sorted batch: work item i = {expert, first row, rows}; every
@@ -3040,7 +3134,7 @@ b200_status launch_tc_static(QmmArgs& a, int rows, int dev, cudaStream_t s) {
   a.x_row0 = 0;
   qmm_tc_kernel<MODE><<<dim3(a.nt, splits, tts), kTcThreads, smem, s>>>(xmap, a);
   B200_LAUNCH_CHECK();
-  return (splits == 1 && tn <= 64) ? B200_OK : launch_finish(a, splits, s);
+  return (splits == 1 && tn <= 64 && !a.keep_f32) ? B200_OK : launch_finish(a, splits, s);
 }
 }  // namespace
 

@@ -51,6 +51,7 @@ struct QmmArgs {
   int mx_expert_rows;           // rows of the code matrix per expert (nt * 128)
   int kc128;                    // K / 128
   int did_norm;                 // host only: the finish pass also wrote norm_out
+  int keep_f32;                 // the caller wants the f32 sums: no kernel writes bf16 output itself
   b200_qmm_partials* defer = nullptr;  // when set, a dense launch with epilogue NONE leaves its finish pass to the caller
 
   __device__ __forceinline__ int row_base_out(int token) const { return token; }

@@ -13,7 +13,7 @@ import torch
 from . import _lib
 from ._lib import KvConfig, PackDesc, lib
 
-KV_BF16, KV_FP8_E4M3 = 0, 1
+KV_BF16, KV_FP8_E4M3, KV_F32 = 0, 1, 2
 Q_AFFINE4_G64, Q_MXFP4_G32 = 0, 1
 EPI_NONE, EPI_RESIDUAL, EPI_SWIGLU = 0, 1, 2
 QMM_AUTO, QMM_SIMT, QMM_TCGEN05, QMM_MMA, QMM_TCGEN05_X2, QMM_TCGEN05_TMEM_A, QMM_MXFP4_BLOCK_SCALED, QMM_MMA_I8 = 0, 1, 2, 3, 4, 5, 6, 7
@@ -81,7 +81,7 @@ class PagedKVCache:
         self.cfg = cfg
 
     def close(self):
-        if getattr(self, "_h", None):
+        if getattr(self, "_h", None) and lib is not None:
             lib.b200_kv_destroy(self._h)
             self._h = None
 
@@ -181,26 +181,33 @@ class PagedKVCache:
         _lib.check(lib.b200_kv_error_word(self._h, C.byref(out)))
         return out.value
 
+    def layer_shape(self, layer: int):
+        """(kv heads, key width, value width) of one layer."""
+        return self.cfg.n_kv_heads, self.cfg.head_dim, self.cfg.head_dim
+
+    def page_shapes(self, layer: int):
+        """Shapes of one page of a layer as stored: keys, values."""
+        h, kd, vd = self.layer_shape(layer)
+        return (h, self.cfg.page_size, kd), (h, self.cfg.page_size, vd)
+
     def gather(self, layer: int, seq: int):
         n = self.seq_len(seq)
-        shape = (max(n, 1), self.cfg.n_kv_heads, self.cfg.head_dim)
-        k = torch.empty(shape, dtype=torch.bfloat16, device="cuda")
-        v = torch.empty_like(k)
+        h, kd, vd = self.layer_shape(layer)
+        dtype = torch.float32 if self.cfg.kv_dtype == KV_F32 else torch.bfloat16
+        k = torch.empty((max(n, 1), h, kd), dtype=dtype, device="cuda")
+        v = torch.empty((max(n, 1), h, vd), dtype=dtype, device="cuda")
         _lib.check(lib.b200_kv_gather(self._h, layer, seq, _ptr(k), _ptr(v), n, _stream()))
         return k[:n], v[:n]
 
     def page_raw(self, layer: int, page: int):
         c = self.cfg
-        eb = 2 if c.kv_dtype == KV_BF16 else 1
-        nbytes = c.n_kv_heads * c.page_size * c.head_dim * eb
-        k, v = np.zeros(nbytes, np.uint8), np.zeros(nbytes, np.uint8)
+        dt = {KV_BF16: np.uint16, KV_FP8_E4M3: np.uint8, KV_F32: np.float32}[c.kv_dtype]
+        ksh, vsh = self.page_shapes(layer)
+        k, v = np.zeros(ksh, dt), np.zeros(vsh, dt)
         ks, vs = np.zeros(c.n_kv_heads, np.float32), np.zeros(c.n_kv_heads, np.float32)
         _lib.check(lib.b200_kv_page_raw(self._h, layer, page, k.ctypes.data, v.ctypes.data,
                                         ks.ctypes.data_as(C.POINTER(C.c_float)), vs.ctypes.data_as(C.POINTER(C.c_float))))
-        shape = (c.n_kv_heads, c.page_size, c.head_dim)
-        if eb == 2:
-            return k.view(np.uint16).reshape(shape), v.view(np.uint16).reshape(shape), ks, vs
-        return k.reshape(shape), v.reshape(shape), ks, vs
+        return k, v, ks, vs
 
     def page_load(self, layer: int, page: int, k: np.ndarray, v: np.ndarray, k_scales=None, v_scales=None):
         """Inverse of page_raw: host page bytes (and, for FP8 pools, per-head scales) into the pool."""
@@ -212,6 +219,28 @@ class PagedKVCache:
 
     def set_len(self, seq: int, n_tokens: int):
         _lib.check(lib.b200_kv_set_len(self._h, seq, n_tokens))
+
+
+class LayeredKVCache(PagedKVCache):
+    """A page pool whose layers have shapes of their own: `layers` is [(kv heads, key width, value width)], bf16 or f32 pages.
+    Rows are written and read by the decoder step; everything the allocator does works as on any pool."""
+
+    def __init__(self, layers: Sequence[Sequence[int]], n_pages: int, max_seqs: int, max_pages_per_seq: int, n_q_heads: int,
+                 max_rows: int = 4096, kv_dtype: int = KV_BF16, attn_scratch_chunks: int = 0):
+        cfg = KvConfig(len(layers), 0, 0, 32, n_pages, max_seqs, max_pages_per_seq, kv_dtype, max_rows, n_q_heads, attn_scratch_chunks)
+        arr = (_lib.KvLayer * max(len(layers), 1))(*[_lib.KvLayer(*l) for l in layers])
+        h = C.c_void_p()
+        _lib.check(lib.b200_kv_create_layers(C.byref(cfg), arr, C.byref(h)))
+        cfg.n_kv_heads = max(l[0] for l in layers)
+        self._h, self.cfg, self.layers = h.value, cfg, [tuple(l) for l in layers]
+
+    def layer_shape(self, layer: int):
+        return self.layers[layer]
+
+    def page_shapes(self, layer: int):  # stored rows are a multiple of 16 elements wide
+        h, kd, vd = self.layers[layer]
+        up = lambda n: (n + 15) // 16 * 16
+        return (h, 32, up(kd)), (h, 32, up(vd))
 
 
 def set_attn_pages_per_chunk(n: int):
@@ -264,9 +293,18 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Ten
     return out
 
 
+def qmm_f32(w: "QWeight", x: torch.Tensor, epilogue: int = EPI_NONE, n_valid: Optional[int] = None) -> torch.Tensor:
+    """b200_qmm_f32: f32 activations and result, dense bf16 weights."""
+    n_out = (w.n // 2 if epilogue == EPI_SWIGLU else w.n) if n_valid is None else n_valid
+    out = torch.empty((x.shape[0], n_out), dtype=torch.float32, device=x.device)
+    _lib.check(lib.b200_qmm_f32(w._h, _ptr(x), x.shape[0], _ptr(out), n_out, n_out, epilogue, _stream()))
+    return out
+
+
 def argmax(logits: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     out = out if out is not None else torch.empty(logits.shape[0], dtype=torch.int32, device=logits.device)
-    _lib.check(lib.b200_argmax(_ptr(logits), logits.shape[0], logits.shape[1], _ptr(out), _stream()))
+    fn = lib.b200_argmax_f32 if logits.dtype == torch.float32 else lib.b200_argmax
+    _lib.check(fn(_ptr(logits), logits.shape[0], logits.shape[1], _ptr(out), _stream()))
     return out
 
 
@@ -378,7 +416,73 @@ Q_BF16 = 2
 W_Q, W_K, W_V, W_O, W_GATE, W_UP, W_DOWN, W_LM_HEAD = range(8)
 
 
-class LlamaModel:
+class Model:
+    """Any model behind the common step interface (b200_model_*): one packed ragged batch in, one token per request out,
+    and on request the logits of any packed rows."""
+
+    _m = None  # b200_model handle
+
+    def info(self) -> "_lib.ModelInfo":
+        out = _lib.ModelInfo()
+        lib.b200_model_get_info(self._m, C.byref(out))
+        return out
+
+    def step(self, kv: PagedKVCache, descs: Sequence[Sequence[int]], prefill_tokens: Sequence[int] = (),
+             want_rows: Sequence[int] = ()):
+        """b200_model_step with host buffers.  Returns (next token per request, free pages); the logits of `want_rows`
+        (packed row indices) are then rows len(descs).. of logits()."""
+        n = len(descs)
+        d = (PackDesc * max(n, 1))()
+        for i, (slot, count, base, src) in enumerate(descs):
+            d[i].seq_slot, d[i].count, d[i].base_pos, d[i].src_offset = slot, count, base, src
+        pt = (C.c_uint32 * max(len(prefill_tokens), 1))(*[int(t) for t in prefill_tokens])
+        out = (C.c_uint32 * max(n, 1))()
+        free = C.c_int32()
+        if len(want_rows):
+            _lib.check(lib.b200_model_want_logits(self._m, (C.c_int32 * len(want_rows))(*want_rows), len(want_rows)))
+        _lib.check(lib.b200_model_step(self._m, kv._h, d, n, pt, len(prefill_tokens), out, C.byref(free), _stream()))
+        return np.array([out[i] for i in range(n)], np.uint32), free.value
+
+    def logits(self, first: int, n: int) -> np.ndarray:
+        """f32 logits of the last step: rows 0.. are the requests' last rows, then the wanted rows."""
+        out = np.zeros((n, self.info().vocab), np.float32)
+        _lib.check(lib.b200_model_logits(self._m, first, n, out.ctypes.data_as(C.POINTER(C.c_float))))
+        return out
+
+    def forward_device(self, kv: PagedKVCache, d_desc: torch.Tensor, total_rows: int,
+                       d_prefill: Optional[torch.Tensor] = None):
+        """b200_model_forward on device-resident descriptors (asynchronous)."""
+        _lib.check(lib.b200_model_forward(self._m, kv._h, _ptr(d_desc), d_desc.shape[0], total_rows, _ptr(d_prefill),
+                                          _stream()))
+
+    def set_samplers(self, rows):
+        """Sampler rows (temperature, top_k, top_p, uniform) for the requests of the next step()."""
+        arr = sample_params_array(rows)
+        _lib.check(lib.b200_model_set_samplers(self._m, arr.ctypes.data_as(C.POINTER(_lib.SampleParams)), len(rows)))
+
+    def last_logprobs(self, n_req: int) -> np.ndarray:
+        out = np.zeros(n_req, np.float32)
+        _lib.check(lib.b200_model_last_logprobs(self._m, out.ctypes.data_as(C.POINTER(C.c_float)), n_req))
+        return out
+
+    def launch_count(self) -> int:
+        return int(lib.b200_model_launch_count(self._m))
+
+    def enable_graphs(self, on: bool = True):
+        lib.b200_model_enable_graphs(self._m, int(on))
+
+    def profile_enable(self, on: bool = True):
+        lib.b200_model_profile_enable(self._m, int(on))
+
+    def profile_collect(self):
+        """{category: (milliseconds, calls)} for attention / matmul / rope+append / other."""
+        ms, calls = (C.c_double * 4)(), (C.c_int64 * 4)()
+        _lib.check(lib.b200_model_profile_collect(self._m, ms, calls))
+        names = ("attention", "matmul", "rope_append", "other")
+        return {n: (ms[i], calls[i]) for i, n in enumerate(names)}
+
+
+class LlamaModel(Model):
     """The LLaMA layer stack behind b200_llama_step (ModelVTable.forward + greedy sampling,
     src/generation.zig:47-53,104-145)."""
 
@@ -389,9 +493,10 @@ class LlamaModel:
         h = C.c_void_p()
         _lib.check(lib.b200_llama_create(C.byref(self.cfg), C.byref(h)))
         self._h = h.value
+        self._m = lib.b200_llama_model(self._h)
 
     def close(self):
-        if getattr(self, "_h", None):
+        if getattr(self, "_h", None) and lib is not None:
             lib.b200_llama_destroy(self._h)
             self._h = None
 
@@ -421,57 +526,77 @@ class LlamaModel:
     def random_init(self, mode: int, seed: int = 1):
         _lib.check(lib.b200_llama_random_init(self._h, mode, seed))
 
-    def step(self, kv: PagedKVCache, descs: Sequence[Sequence[int]], prefill_tokens: Sequence[int] = ()):
-        """b200_llama_step with host buffers.  Returns (next token per request, free pages)."""
-        n = len(descs)
-        d = (PackDesc * max(n, 1))()
-        for i, (slot, count, base, src) in enumerate(descs):
-            d[i].seq_slot, d[i].count, d[i].base_pos, d[i].src_offset = slot, count, base, src
-        pt = (C.c_uint32 * max(len(prefill_tokens), 1))(*[int(t) for t in prefill_tokens])
-        out = (C.c_uint32 * max(n, 1))()
-        free = C.c_int32()
-        _lib.check(lib.b200_llama_step(self._h, kv._h, d, n, pt, len(prefill_tokens), out, C.byref(free), _stream()))
-        return np.array([out[i] for i in range(n)], np.uint32), free.value
-
-    def forward_device(self, kv: PagedKVCache, d_desc: torch.Tensor, total_rows: int,
-                       d_prefill: Optional[torch.Tensor] = None):
-        """b200_llama_forward on device-resident descriptors (asynchronous)."""
-        _lib.check(lib.b200_llama_forward(self._h, kv._h, _ptr(d_desc), d_desc.shape[0], total_rows, _ptr(d_prefill),
-                                          _stream()))
-
-    def set_samplers(self, rows):
-        """Sampler rows (temperature, top_k, top_p, uniform) for the requests of the next step()."""
-        arr = sample_params_array(rows)
-        _lib.check(lib.b200_llama_set_samplers(self._h, arr.ctypes.data_as(C.POINTER(_lib.SampleParams)), len(rows)))
-
-    def last_logprobs(self, n_req: int) -> np.ndarray:
-        out = np.zeros(n_req, np.float32)
-        _lib.check(lib.b200_llama_last_logprobs(self._h, out.ctypes.data_as(C.POINTER(C.c_float)), n_req))
-        return out
-
     def last_logits(self, n_req: int) -> np.ndarray:
         out = np.zeros((n_req, self.cfg.vocab), np.uint16)
         _lib.check(lib.b200_llama_last_logits(self._h, out.ctypes.data, n_req))
         return (out.astype(np.uint32) << 16).view(np.float32)
 
-    def launch_count(self) -> int:
-        return int(lib.b200_llama_launch_count(self._h))
-
-    def enable_graphs(self, on: bool = True):
-        lib.b200_llama_enable_graphs(self._h, int(on))
-
     def set_fused_qkv_rope(self, on: bool = True):
         lib.b200_llama_set_fused_qkv_rope(self._h, int(on))
 
-    def profile_enable(self, on: bool = True):
-        lib.b200_llama_profile_enable(self._h, int(on))
 
-    def profile_collect(self):
-        """{category: (milliseconds, calls)} for attention / matmul / rope+append / other."""
-        ms, calls = (C.c_double * 4)(), (C.c_int64 * 4)()
-        _lib.check(lib.b200_llama_profile_collect(self._h, ms, calls))
-        names = ("attention", "matmul", "rope_append", "other")
-        return {n: (ms[i], calls[i]) for i, n in enumerate(names)}
+DT_BF16, DT_F32 = 0, 1
+DEC_QKV_BIAS, DEC_QK_NORM, DEC_DISTANCE_BIAS, DEC_SINK, DEC_POST_NORM = 1, 2, 4, 8, 16
+DEC_TENSORS = ("q", "k", "v", "o", "gate", "up", "down", "head", "loop_in", "embed", "q_bias", "k_bias", "v_bias", "sink", "norm1", "norm2",
+               "postnorm1", "postnorm2", "final_norm")
+
+
+class DecoderModel(Model):
+    """The configurable decoder stack (b200_decoder_*).  `layers` is a list of dicts with the fields of
+    b200_decoder_layer; `loop` is (start, stop, times) or None."""
+
+    def __init__(self, hidden: int, vocab: int, layers: Sequence[dict], norm_eps: float, embed_scale: float = 1.0, loop=None,
+                 dtype: int = DT_BF16, max_rows: int = 2048, max_reqs: int = 64, max_seqs: int = 64):
+        start, stop, times = loop if loop else (0, 0, 0)
+        self.cfg = _lib.DecoderConfig(len(layers), hidden, vocab, start, stop, times, dtype, max_rows, max_reqs, max_seqs, norm_eps,
+                                      embed_scale)
+        arr = (_lib.DecoderLayer * max(len(layers), 1))(*[_lib.DecoderLayer(**l) for l in layers])
+        h = C.c_void_p()
+        _lib.check(lib.b200_decoder_create(C.byref(self.cfg), arr, C.byref(h)))
+        self._h = h.value
+        self._m = lib.b200_decoder_model(self._h)
+        self.layers = [dict(l) for l in layers]
+
+    def close(self):
+        if getattr(self, "_h", None) and lib is not None:  # (interpreter shutdown clears module globals)
+            lib.b200_decoder_destroy(self._h)
+            self._h = self._m = None
+
+    def __del__(self):
+        self.close()
+
+    def set_tensor(self, layer: int, which: str, bf16_bits: np.ndarray):
+        t = np.ascontiguousarray(bf16_bits, np.uint16)
+        _lib.check(lib.b200_decoder_set_tensor(self._h, layer, DEC_TENSORS.index(which), t.ctypes.data, t.size))
+
+    def finalize(self):
+        _lib.check(lib.b200_decoder_finalize(self._h))
+
+    def random_init(self, seed: int = 1):
+        _lib.check(lib.b200_decoder_random_init(self._h, seed))
+
+    def cache_layers(self):
+        """[(kv heads, key width, value width)] of the cache layers, one per layer run."""
+        n = lib.b200_decoder_cache_layers(self._h, None, 0)
+        arr = (_lib.KvLayer * n)()
+        lib.b200_decoder_cache_layers(self._h, arr, n)
+        return [(l.n_kv_heads, l.key_dim, l.value_dim) for l in arr]
+
+    def make_cache(self, n_pages: int, max_seqs: int, max_pages_per_seq: int, max_rows: Optional[int] = None) -> LayeredKVCache:
+        return LayeredKVCache(self.cache_layers(), n_pages, max_seqs, max_pages_per_seq, max(l["n_heads"] for l in self.layers),
+                              max_rows or self.cfg.max_rows, KV_F32 if self.cfg.dtype == DT_F32 else KV_BF16)
+
+    def record_layers(self, on: bool = True):
+        _lib.check(lib.b200_decoder_record_layers(self._h, int(on)))
+
+    def recorded_layers(self, rows: int) -> np.ndarray:
+        """Residual stream after every layer run of the last step: [layer runs, rows, hidden]."""
+        out = np.zeros((len(self.cache_layers()), rows, self.cfg.hidden), np.float32)
+        _lib.check(lib.b200_decoder_recorded_layers(self._h, rows, out.ctypes.data_as(C.POINTER(C.c_float))))
+        return out
+
+    def set_attn_mma(self, on: bool = True):
+        lib.b200_decoder_set_attn_mma(self._h, int(on))
 
 
 # ---------------------------------------------------------------------------------------------
@@ -588,8 +713,8 @@ def moe_combine(y_sorted: torch.Tensor, inv_order: torch.Tensor, n_tokens: int, 
 class Engine:
     """b200_engine_*: scheduler + device page pool + model step in one loop."""
 
-    def __init__(self, model: LlamaModel, kv: PagedKVCache, max_prefill_tokens: int = 512):
-        self._h = lib.b200_engine_create(model._h, kv._h, max_prefill_tokens)
+    def __init__(self, model: Model, kv: PagedKVCache, max_prefill_tokens: int = 512):
+        self._h = lib.b200_engine_create_model(model._m, kv._h, max_prefill_tokens)
         if not self._h:
             raise _lib.B200Error(_lib.ERR_CUDA)
         self._keep = (model, kv)

@@ -12,54 +12,16 @@ two never read each other's files by name; the container format and tensor names
 
 Saving copies pages device -> host -> file; restoring allocates pages for an empty sequence slot,
 loads them and sets the slot's length, after which the slot decodes as if it had prefilled those
-tokens itself.  The safetensors container is written and parsed here (8-byte little-endian header
-length, JSON header, raw little-endian data): no third-party package is needed.
+tokens itself.
 """
 from __future__ import annotations
 
-import json
 import os
-import struct
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import numpy as np
 
-_DTYPES = {"BF16": np.uint16, "U8": np.uint8, "F32": np.float32}
-
-
-def write_safetensors(path: str, tensors: Dict[str, Tuple[str, np.ndarray]], metadata: Dict[str, str]) -> None:
-    """tensors: name -> (safetensors dtype tag, array whose bytes are stored as they are)."""
-    header: Dict[str, object] = {"__metadata__": {k: str(v) for k, v in metadata.items()}}
-    blobs: List[bytes] = []
-    off = 0
-    for name in sorted(tensors):
-        tag, arr = tensors[name]
-        raw = np.ascontiguousarray(arr).tobytes()
-        header[name] = {"dtype": tag, "shape": list(arr.shape), "data_offsets": [off, off + len(raw)]}
-        blobs.append(raw)
-        off += len(raw)
-    hj = json.dumps(header, separators=(",", ":")).encode()
-    hj += b" " * ((8 - len(hj) % 8) % 8)
-    tmp = path + ".tmp"
-    with open(tmp, "wb") as f:
-        f.write(struct.pack("<Q", len(hj)))
-        f.write(hj)
-        for b in blobs:
-            f.write(b)
-    os.replace(tmp, path)  # a reader never sees a half-written block
-
-
-def read_safetensors(path: str) -> Tuple[Dict[str, np.ndarray], Dict[str, str]]:
-    with open(path, "rb") as f:
-        (n,) = struct.unpack("<Q", f.read(8))
-        header = json.loads(f.read(n))
-        data = f.read()
-    meta = header.pop("__metadata__", {})
-    out = {}
-    for name, info in header.items():
-        a, b = info["data_offsets"]
-        out[name] = np.frombuffer(data[a:b], dtype=_DTYPES[info["dtype"]]).reshape(info["shape"])
-    return out, meta
+from .safetensors_io import read_safetensors, write_safetensors
 
 
 def chain_hashes(token_ids: Sequence[int], block_size: int = 32) -> List[int]:
@@ -89,14 +51,14 @@ class PrefixDiskStore:
     # -- one block ---------------------------------------------------------------------------
     def save_block(self, kv, page: int, block_hash: int) -> None:
         c = kv.cfg
-        fp8 = c.kv_dtype != 0
+        fp8 = c.kv_dtype == 1
         tensors, meta = {}, {"layer_count": c.n_layers, "block_size": self.block_size, "block_hash": block_hash}
-        shape = (1, c.n_kv_heads, c.page_size, c.head_dim)
         for l in range(c.n_layers):
             k, v, ks, vs = kv.page_raw(l, page)
-            tag = "U8" if fp8 else "BF16"
-            tensors[f"layer_{l}_keys"] = (tag, k.reshape(shape))
-            tensors[f"layer_{l}_values"] = (tag, v.reshape(shape))
+            tag = {np.dtype(np.uint8): "U8", np.dtype(np.uint16): "BF16", np.dtype(np.float32): "F32"}[k.dtype]
+            shape = (1, *k.shape)
+            tensors[f"layer_{l}_keys"] = (tag, k[None])
+            tensors[f"layer_{l}_values"] = (tag, v[None])
             if fp8:
                 tensors[f"layer_{l}_key_scales"] = ("F32", ks)
                 tensors[f"layer_{l}_value_scales"] = ("F32", vs)
@@ -136,17 +98,17 @@ class PrefixDiskStore:
             n -= 1
         if n == 0:
             return 0
-        fp8 = c.kv_dtype != 0
-        want_shape, want_dtype = (1, c.n_kv_heads, c.page_size, c.head_dim), (np.uint8 if fp8 else np.uint16)
+        fp8 = c.kv_dtype == 1
+        want_dtype = {0: np.uint16, 1: np.uint8, 2: np.float32}[c.kv_dtype]
         blocks = []
         for b in range(n):  # every block is checked before the pool is touched
             tensors, meta = self.load_block(hashes[b])
             if int(meta["layer_count"]) != c.n_layers:
                 raise ValueError("stored block has a different layer count")
             for l in range(c.n_layers):
-                for name in (f"layer_{l}_keys", f"layer_{l}_values"):
+                for name, want_shape in zip((f"layer_{l}_keys", f"layer_{l}_values"), kv.page_shapes(l)):
                     t = tensors[name]
-                    if tuple(t.shape) != want_shape or t.dtype != want_dtype:
+                    if tuple(t.shape) != (1, *want_shape) or t.dtype != want_dtype:
                         raise ValueError("stored block does not match the pool's page shape or element type")
                 if fp8 and (f"layer_{l}_key_scales" not in tensors or f"layer_{l}_value_scales" not in tensors):
                     raise ValueError("stored FP8 block has no scales")

@@ -218,7 +218,7 @@ b200_status b200_pack_batch(const b200_pack_desc* d_desc, int32_t n_req,
 /* Stands in for PagedKVCache (src/kvcache/paged.zig:305-1139) behind the KVCacheStrategy vtable
  * (src/kvcache/interface.zig:31-77), with the page allocator of paged.BlockManager (:44-206)
  * whose free stack, ref-counts and page tables live in device memory. */
-enum { B200_KV_BF16 = 0, B200_KV_FP8_E4M3 = 1 };
+enum { B200_KV_BF16 = 0, B200_KV_FP8_E4M3 = 1, B200_KV_F32 = 2 /* layered pools only */ };
 typedef struct b200_kv_config {
   int32_t n_layers;
   int32_t n_kv_heads;        /* LayerConfig.num_kv_heads  src/kvcache/interface.zig:162-169 */
@@ -236,6 +236,13 @@ typedef struct b200_kv_config {
                                 * slots than the pool holds is flagged B200_ERR_CAPACITY and changes nothing. */
 } b200_kv_config;
 b200_status b200_kv_create(const b200_kv_config* cfg, b200_kv** out);            /* :342-411 init, :1141-1186 factories */
+/* A pool whose layers have shapes of their own (no reference counterpart: LayerConfig is one shape for all layers):
+ * heads, and widths of keys and values, per layer; n_kv_heads and head_dim of the configuration are ignored.  bf16
+ * or f32 pages.  Page tables, reference counts, copy-on-write, fork, rollback, extend and page_raw / page_load work as on
+ * any pool (page bytes per layer: [n_kv_heads][32][width rounded up to 16]); rows are written and read by
+ * b200_decoder_*. */
+typedef struct b200_kv_layer { int32_t n_kv_heads, key_dim, value_dim; } b200_kv_layer;
+b200_status b200_kv_create_layers(const b200_kv_config* cfg, const b200_kv_layer* layers, b200_kv** out);
 void b200_kv_destroy(b200_kv* kv);                                               /* :1111-1138 deinit */
 /* Pool size and number of sequence slots of a pool. */
 b200_status b200_kv_dims(const b200_kv* kv, int32_t* n_pages, int32_t* max_seqs);
@@ -302,7 +309,8 @@ b200_status b200_kv_ref_counts(b200_kv* kv, int32_t* out, int32_t cap);
 /* Reads and clears the device error word: 0, or a b200_status set by a kernel. */
 b200_status b200_kv_error_word(b200_kv* kv, int32_t* out);
 /* Tests only: the contiguous [len, n_kv_heads, head_dim] bf16 view updateAndFetch would return
- * (:705-802); FP8 pages are dequantised. */
+ * (:705-802); FP8 pages are dequantised.  Layered pools: [len, heads, key_dim] and [len, heads, value_dim] in the
+ * pool's element type. */
 b200_status b200_kv_gather(b200_kv* kv, int32_t layer, int32_t seq, void* d_k_out, void* d_v_out,
                            int32_t cap_rows, void* stream);
 /* Raw E4M3 codes and scales of one page (FP8 pools; bit-exact checks). */
@@ -352,6 +360,9 @@ b200_status b200_embed_gather(const void* d_table, const uint32_t* d_ids, void* 
 /* Greedy: first strict maximum per row of bf16 logits [rows, vocab] (src/sampling.zig:22-39). */
 b200_status b200_argmax(const void* d_logits, int32_t rows, int32_t vocab, uint32_t* d_out,
                         void* stream);
+/* The same on f32 logits. */
+b200_status b200_argmax_f32(const float* d_logits, int32_t rows, int32_t vocab, uint32_t* d_out,
+                            void* stream);
 
 /* ---- sampling beyond greedy (src/sampling.zig:42-242, 277-322) ------------------------------- */
 /* One row of SamplerConfig (:277-285) plus the uniform variate in [0,1) that sampleFromProbs (:258-268)
@@ -436,9 +447,16 @@ b200_status b200_qmm(const b200_qweight* w, const void* d_x, int32_t rows, void*
 /* b200_qmm with epilogue NONE whose split-K finish pass may be left to the caller's next kernel (no reference
  * counterpart).  defer = 0: exactly b200_qmm.  defer != 0: when the chosen kernel splits K, the finish pass is not
  * launched, out->pending = 1 and out describes the partial sums (d_y is NOT written); when it does not split K,
- * d_y is written and out->pending = 0. */
+ * d_y is written and out->pending = 0.  defer = 2: the f32 sums are left in the scratch even when K is not split
+ * (pending = 1 always), for results that must not be rounded to bf16. */
 b200_status b200_qmm_deferred(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t defer,
                               void* stream, b200_qmm_partials* out);
+
+/* y = x W^T in 32-bit throughout (no reference counterpart): f32 activations [rows, K], dense bf16 weights
+ * (B200_Q_BF16) widened exactly, f32 accumulation on the CUDA cores, f32 result with `y_stride` elements between rows;
+ * columns from n_valid on are not written (n_valid <= N).  SWIGLU halves the columns as in b200_qmm. */
+b200_status b200_qmm_f32(const b200_qweight* w, const float* d_x, int32_t rows, float* d_y, int32_t y_stride,
+                         int32_t n_valid, int32_t epilogue, void* stream);
 
 /* y = residual + x W^T and normed = rmsnorm(y) * norm_weight in one call: the pair that closes the
  * attention and the FFN half of a block (src/models/llama.zig:466-477: residual add, then the next
@@ -532,6 +550,92 @@ void b200_llama_set_fused_qkv_rope(b200_llama* m, int32_t on);
 void b200_llama_profile_enable(b200_llama* m, int32_t on);
 b200_status b200_llama_profile_collect(b200_llama* m, double* ms, int64_t* calls);
 
+/* ---- any model behind one step interface -------------------------------------------------------- */
+/* What ModelVTable is to the reference (src/generation.zig:47-53): the engine, the samplers and the trace replay drive a
+ * model through this handle.  A model's own handle converts without copying; the view lives as long as the model. */
+typedef struct b200_model b200_model;
+b200_model* b200_llama_model(b200_llama* m);
+typedef struct b200_model_info {
+  int32_t vocab, max_rows, max_reqs, max_seqs;
+  int32_t logits_f32;  /* element type of the logits on the device: 1 = f32, 0 = bf16 */
+} b200_model_info;
+void b200_model_get_info(const b200_model* m, b200_model_info* out);
+/* The b200_llama_* calls of the same names, for any model. */
+b200_status b200_model_step(b200_model* m, b200_kv* kv, const b200_pack_desc* h_desc, int32_t n_req,
+                            const uint32_t* h_prefill_tokens, int32_t n_prefill_tokens, uint32_t* h_next_tokens,
+                            int32_t* out_free_pages, void* stream);
+b200_status b200_model_forward(b200_model* m, b200_kv* kv, const b200_pack_desc* d_desc, int32_t n_req, int32_t total_rows,
+                               const uint32_t* d_prefill_tokens, void* stream);
+void b200_model_device_buffers(b200_model* m, b200_pack_desc** d_desc, uint32_t** d_prefill, uint32_t** d_next);
+b200_status b200_model_set_samplers(b200_model* m, const b200_sample_params* h_rows, int32_t n_req);
+b200_status b200_model_last_logprobs(b200_model* m, float* h_out, int32_t n_req);
+int64_t b200_model_launch_count(const b200_model* m);
+void b200_model_enable_graphs(b200_model* m, int32_t on);
+void b200_model_profile_enable(b200_model* m, int32_t on);
+b200_status b200_model_profile_collect(b200_model* m, double* ms, int64_t* calls);
+/* Logits of more rows than the sampled ones: packed row indices (batch order) whose logits the NEXT step computes
+ * beside each request's last row (one use).  b200_model_logits then returns f32 rows: 0..n_req-1 are the requests'
+ * last rows, n_req.. the wanted ones in the order given. */
+b200_status b200_model_want_logits(b200_model* m, const int32_t* h_rows, int32_t n);
+b200_status b200_model_logits(b200_model* m, int32_t first, int32_t n, float* h_out);
+
+/* ---- configurable decoder stack ------------------------------------------------------------------- */
+/* A decoder-only stack whose layers are described one by one (no reference counterpart; the reference has one file per
+ * model family).  Every mechanism is a parameter of its layer, and a layer that does not set it does not have it:
+ *   x = embed[token] * embed_scale, kept in f32 between the layers;
+ *   x += postnorm1(attention(norm1(x))); x += postnorm2(W_down(silu(W_gate h) * W_up h)), h = norm2(x);
+ *   layers loop_start .. loop_stop-1 run loop_times times with the same weights, every pass with cache layers of its own,
+ *   and each pass opens with x = W_in [x ; x0], x0 the embedding output;
+ *   logits = head(final_norm(x)), f32.
+ * Norms, scores, softmax and the residual are f32; matrix operands are bf16, or f32 throughout with
+ * dtype = B200_DT_F32. */
+enum { B200_DT_BF16 = 0, B200_DT_F32 = 1 };
+enum {
+  B200_DEC_QKV_BIAS = 1,       /* biases on the q, k and v projections */
+  B200_DEC_QK_NORM = 2,        /* q and k divided by their root mean square per head (no weight) */
+  B200_DEC_DISTANCE_BIAS = 4,  /* score -= 2^(-8 (h + 1) / n_heads) * (i - j) */
+  B200_DEC_SINK = 8,           /* learned sink per query head in the softmax's denominator */
+  B200_DEC_POST_NORM = 16      /* RMSNorm on each sublayer's output before the residual add */
+};
+typedef struct b200_decoder_layer {
+  int32_t n_heads, n_kv_heads, key_dim, value_dim;
+  int32_t window; /* position i sees j with 0 <= i - j < window; 0 = the whole context */
+  int32_t ffn;    /* 0 = the layer has no feed-forward */
+  int32_t flags;  /* B200_DEC_* */
+  float scale;    /* score = (q . k) * scale */
+} b200_decoder_layer;
+typedef struct b200_decoder_config {
+  int32_t n_layers, hidden, vocab;
+  int32_t loop_start, loop_stop, loop_times; /* loop_times = 0: no loop */
+  int32_t dtype;                             /* B200_DT_* */
+  int32_t max_rows, max_reqs, max_seqs;
+  float norm_eps, embed_scale;
+} b200_decoder_config;
+typedef struct b200_decoder b200_decoder;
+enum { B200_DEC_W_Q = 0, B200_DEC_W_K = 1, B200_DEC_W_V = 2, B200_DEC_W_O = 3, B200_DEC_W_GATE = 4, B200_DEC_W_UP = 5,
+       B200_DEC_W_DOWN = 6, B200_DEC_W_HEAD = 7, B200_DEC_W_LOOP_IN = 8, B200_DEC_W_EMBED = 9, B200_DEC_B_Q = 10,
+       B200_DEC_B_K = 11, B200_DEC_B_V = 12, B200_DEC_W_SINK = 13, B200_DEC_NORM1 = 14, B200_DEC_NORM2 = 15,
+       B200_DEC_POSTNORM1 = 16, B200_DEC_POSTNORM2 = 17, B200_DEC_FINAL_NORM = 18 };
+b200_status b200_decoder_create(const b200_decoder_config* cfg, const b200_decoder_layer* layers, b200_decoder** out);
+void b200_decoder_destroy(b200_decoder* m);
+/* One tensor, bf16 on the host, matrices [out, in]; n_elems is checked against the shape the configuration gives.
+ * `layer` is ignored for embed, head, loop_in and final_norm. */
+b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t which, const void* h_bf16, uint64_t n_elems);
+/* Fuses q/k/v and gate/up; fails, naming it, if a tensor the configuration needs was not set. */
+b200_status b200_decoder_finalize(b200_decoder* m);
+/* Synthetic weights generated on the device (benchmarks).  Matrix sizes must be multiples of 128. */
+b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed);
+/* Cache layers the stack needs (a looped layer counts once per pass) and their shapes, for b200_kv_create_layers. */
+int32_t b200_decoder_cache_layers(const b200_decoder* m, b200_kv_layer* out, int32_t cap);
+/* Residual stream after each layer run, recorded for the NEXT steps when on: [layer runs, rows of the step, hidden] f32
+ * (checks of a model against an oracle). */
+b200_status b200_decoder_record_layers(b200_decoder* m, int32_t on);
+b200_status b200_decoder_recorded_layers(b200_decoder* m, int32_t rows, float* h_out);
+/* 1 (default): attention on the tensor cores where the layer's shape allows it (bf16, widths up to 256); 0: the
+ * CUDA-core kernel, which serves every shape and f32 (tests compare the two). */
+void b200_decoder_set_attn_mma(b200_decoder* m, int32_t on);
+b200_model* b200_decoder_model(b200_decoder* m);
+
 /* ---- engine step: schedule -> pack -> model step -> postprocess ------------------------------- */
 /* The Engine_Step loop of src/scheduler.zig:7-10 wired to a forward pass (the reference leaves
  * it unwired, docs/en/technical/continuous-batching-design.md:187; its production loop is
@@ -539,6 +643,7 @@ b200_status b200_llama_profile_collect(b200_llama* m, double* ms, int64_t* calls
  * Prefill is chunked by max_prefill_tokens (src/scheduler.zig:183-186). */
 typedef struct b200_engine b200_engine;
 b200_engine* b200_engine_create(b200_llama* model, b200_kv* kv, uint64_t max_prefill_tokens);
+b200_engine* b200_engine_create_model(b200_model* model, b200_kv* kv, uint64_t max_prefill_tokens); /* any model */
 void b200_engine_destroy(b200_engine* e);
 b200_status b200_engine_submit(b200_engine* e, uint64_t id, const uint32_t* prompt, uint64_t n_prompt,
                                uint64_t max_tokens, const uint32_t* stop_tokens, uint64_t n_stop);
