@@ -306,6 +306,15 @@ __global__ void __launch_bounds__(256) decoder_qkv_kernel(QkvArgs a) {
   for (int c = dim + lane; c < width; c += 32) st(dst + c, 0.f);
 }
 
+b200_status launch_qkv(const QkvArgs& a, int rows, cudaStream_t s) {
+  const bool v4 = a.L.key_dim % 4 == 0 && a.L.value_dim % 4 == 0 && a.src.y_stride % 4 == 0;
+  auto* kernel = a.d.elem_bytes == 4 ? (v4 ? decoder_qkv_kernel<float, 4> : decoder_qkv_kernel<float, 1>)
+                                     : (v4 ? decoder_qkv_kernel<__nv_bfloat16, 4> : decoder_qkv_kernel<__nv_bfloat16, 1>);
+  kernel<<<dim3(rows, (a.hq + 2 * a.L.heads + 7) / 8), 256, 0, s>>>(a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
 struct HostTensor { std::vector<uint16_t> bits; };
 
 float bf16_to_f(uint16_t b) {
@@ -476,15 +485,7 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
       QkvArgs a;
       a.d = kv->dev; a.L = kv->lay[r]; a.src = src; a.bias = l.bias; a.hq = s.n_heads; a.qk_norm = s.flags & B200_DEC_QK_NORM ? 1 : 0;
       a.eps = cfg.norm_eps; a.q = q; a.q_stride = s.n_heads * kv->lay[r].kd; a.pos = d_pos; a.row_seq = d_row_seq;
-      const bool v4 = s.key_dim % 4 == 0 && s.value_dim % 4 == 0;
-      auto* kernel = f32() ? (v4 ? decoder_qkv_kernel<float, 4> : decoder_qkv_kernel<float, 1>)
-                           : (v4 ? decoder_qkv_kernel<__nv_bfloat16, 4> : decoder_qkv_kernel<__nv_bfloat16, 1>);
-      auto launch = [&]() -> b200_status {
-        kernel<<<dim3(T, (s.n_heads + 2 * s.n_kv_heads + 7) / 8), 256, 0, cs>>>(a);
-        B200_LAUNCH_CHECK();
-        return B200_OK;
-      };
-      MODEL_STEP_CAT(2, launch());
+      MODEL_STEP_CAT(2, launch_qkv(a, T, cs));
     }
     MODEL_STEP_CAT(0, attention(kv, (int)r, T, stream));
     MODEL_STEP_CAT(1, matmul(l.wo, attn, T, 1, &src, stream));
@@ -807,6 +808,42 @@ b200_status b200_decoder_recorded_layers(b200_decoder* m, int32_t rows, float* h
 void b200_decoder_set_attn_mma(b200_decoder* m, int32_t on) {
   m->attn_mma = on != 0;
   m->drop_graphs();
+}
+
+b200_status b200_decoder_qkv(b200_kv* kv, int32_t layer, const void* d_qkv, int32_t stride, const float* d_bias, int32_t n_q_heads,
+                             int32_t qk_norm, float eps, void* d_q, const int32_t* d_positions, const int32_t* d_row_seq,
+                             int32_t total_rows, void* stream) {
+  if (!kv->layered || layer < 0 || layer >= kv->cfg.n_layers || n_q_heads <= 0 || n_q_heads % kv->lay[layer].heads != 0) {
+    b200_set_error("decoder_qkv: layer %d with %d query heads", layer, n_q_heads);
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  if (total_rows <= 0) return B200_OK;
+  QkvArgs a;
+  a.d = kv->dev; a.L = kv->lay[layer]; a.bias = d_bias; a.hq = n_q_heads; a.qk_norm = qk_norm; a.eps = eps; a.q = d_q;
+  a.src.y = d_qkv;
+  a.src.y_stride = stride;
+  a.q_stride = n_q_heads * a.L.kd;
+  a.pos = d_positions; a.row_seq = d_row_seq;
+  return launch_qkv(a, total_rows, (cudaStream_t)stream);
+}
+
+b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, int32_t n_q_heads, int32_t window, float scale,
+                                   const float* d_slopes_log2, const float* d_sinks_log2, const int32_t* d_row_seq,
+                                   const int32_t* d_row_ctx, int32_t total_rows, int32_t prefill, int32_t mma, void* d_out,
+                                   int32_t out_stride, void* stream) {
+  if (!kv->layered || layer < 0 || layer >= kv->cfg.n_layers || n_q_heads <= 0 || n_q_heads > kv->cfg.n_q_heads ||
+      n_q_heads % kv->lay[layer].heads != 0 || window < 0) {
+    b200_set_error("decoder_attention: layer %d with %d query heads, window %d", layer, n_q_heads, window);
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  b200_status st = B200_OK;
+  if (mma && b200_window_attn_takes_mma(kv, layer))
+    st = b200_window_attn_plan(kv, window, n_q_heads / kv->lay[layer].heads, d_row_seq, d_row_ctx, total_rows, prefill, stream);
+  if (st != B200_OK) return st;
+  WindowAttnCall c;
+  c.layer = layer; c.n_q_heads = n_q_heads; c.window = window; c.q = d_q; c.q_stride = n_q_heads * kv->lay[layer].kd; c.scale = scale;
+  c.slopes_log2 = d_slopes_log2; c.sinks_log2 = d_sinks_log2; c.out = d_out; c.out_stride = out_stride;
+  return b200_window_attn_run(kv, c, d_row_seq, d_row_ctx, total_rows, mma != 0, stream);
 }
 
 }  // extern "C"

@@ -242,6 +242,33 @@ class LayeredKVCache(PagedKVCache):
         up = lambda n: (n + 15) // 16 * 16
         return (h, 32, up(kd)), (h, 32, up(vd))
 
+    def _element(self):
+        return torch.float32 if self.cfg.kv_dtype == KV_F32 else torch.bfloat16
+
+    def qkv(self, layer: int, rows: torch.Tensor, n_q_heads: int, positions: torch.Tensor, row_seq: torch.Tensor,
+            bias: Optional[torch.Tensor] = None, qk_norm: bool = True, eps: float = 1e-5) -> torch.Tensor:
+        """b200_decoder_qkv: biases and per-head norms of projection rows [q | k | v]; k and v go into the pages reserved for
+        the step.  Returns q [T, heads, stored key width]."""
+        assert rows.dtype == self._element()
+        kd = self.page_shapes(layer)[0][2]
+        q = torch.empty((rows.shape[0], n_q_heads, kd), dtype=rows.dtype, device=rows.device)
+        _lib.check(lib.b200_decoder_qkv(self._h, layer, _ptr(rows), rows.shape[1], _ptr(bias), n_q_heads, int(qk_norm), eps, _ptr(q),
+                                        _ptr(positions), _ptr(row_seq), rows.shape[0], _stream()))
+        return q
+
+    def window_attention(self, layer: int, q: torch.Tensor, row_seq: torch.Tensor, row_ctx: torch.Tensor, scale: float, window: int = 0,
+                         slopes: Optional[np.ndarray] = None, sinks: Optional[np.ndarray] = None, prefill: bool = False,
+                         mma: bool = True) -> torch.Tensor:
+        """b200_decoder_attention on q as qkv() returns it -> [T, heads, value width]."""
+        t, hq, _ = q.shape
+        vd = self.layers[layer][2]
+        log2 = lambda a: None if a is None else torch.tensor(np.asarray(a, np.float64) * 1.4426950408889634, dtype=torch.float32, device=q.device)
+        sl, sk = log2(slopes), log2(sinks)
+        out = torch.empty((t, hq, vd), dtype=q.dtype, device=q.device)
+        _lib.check(lib.b200_decoder_attention(self._h, layer, _ptr(q), hq, window, scale, _ptr(sl), _ptr(sk), _ptr(row_seq), _ptr(row_ctx), t,
+                                              int(prefill), int(mma), _ptr(out), hq * vd, _stream()))
+        return out
+
 
 def set_attn_pages_per_chunk(n: int):
     lib.b200_set_attn_pages_per_chunk(n)

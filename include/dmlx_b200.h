@@ -635,6 +635,20 @@ b200_status b200_decoder_recorded_layers(b200_decoder* m, int32_t rows, float* h
  * CUDA-core kernel, which serves every shape and f32 (tests compare the two). */
 void b200_decoder_set_attn_mma(b200_decoder* m, int32_t on);
 b200_model* b200_decoder_model(b200_decoder* m);
+/* The two steps of a decoder layer that touch the pages, for hosts that drive the layers themselves (pages reserved with
+ * b200_kv_reserve; element type = the pool's).
+ * qkv: rows of [q heads x key_dim | kv heads x key_dim | kv heads x value_dim], `stride` elements apart; adds d_bias (f32, may
+ * be null), divides every q and k head by its root mean square when qk_norm, writes q as [q heads][key_dim rounded up to 16]
+ * and k, v into their pages.
+ * attention: d_q as written by qkv; out rows [q heads x value_dim], out_stride apart.  d_slopes_log2 / d_sinks_log2: f32 per
+ * query head, multiplied by log2(e), may be null.  `mma` as in b200_decoder_set_attn_mma. */
+b200_status b200_decoder_qkv(b200_kv* kv, int32_t layer, const void* d_qkv, int32_t stride, const float* d_bias, int32_t n_q_heads,
+                             int32_t qk_norm, float eps, void* d_q, const int32_t* d_positions, const int32_t* d_row_seq,
+                             int32_t total_rows, void* stream);
+b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, int32_t n_q_heads, int32_t window, float scale,
+                                   const float* d_slopes_log2, const float* d_sinks_log2, const int32_t* d_row_seq,
+                                   const int32_t* d_row_ctx, int32_t total_rows, int32_t prefill, int32_t mma, void* d_out,
+                                   int32_t out_stride, void* stream);
 
 /* ---- engine step: schedule -> pack -> model step -> postprocess ------------------------------- */
 /* The Engine_Step loop of src/scheduler.zig:7-10 wired to a forward pass (the reference leaves

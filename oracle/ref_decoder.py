@@ -71,15 +71,20 @@ def attend(q, k, v, scale, window=0, slopes=None, sink=None):
 
 
 # ---- layers ------------------------------------------------------------------------------------------
-def attention_mixer(h, w, name, mixer, eps, rnd=ident):
+ALL = frozenset({"bias", "qk_norm", "distance", "sink", "post_norm"})
+
+
+def attention_mixer(h, w, name, mixer, eps, rnd=ident, has=ALL):
     hq, g, d, e = mixer["heads"], mixer["kv_heads"], mixer["dim"], mixer["vdim"]
     t = h.shape[0]
-    proj = lambda n: linear(h, w[f"{name}.mix.{n}"], w[f"{name}.mix.{n}.b"])
-    q = root_mean_square_norm(proj("q").reshape(t, hq, d), eps)
-    k = root_mean_square_norm(proj("k").reshape(t, g, d), eps)
+    proj = lambda n: linear(h, w[f"{name}.mix.{n}"], w[f"{name}.mix.{n}.b"] if "bias" in has else None)
+    unit = (lambda a: root_mean_square_norm(a, eps)) if "qk_norm" in has else ident
+    q = unit(proj("q").reshape(t, hq, d))
+    k = unit(proj("k").reshape(t, g, d))
     v = proj("v").reshape(t, g, e)
     window = (mixer.get("mask") or {}).get("size", 0)
-    y = attend(rnd(q), rnd(k), rnd(v), mixer["scale"], window, distance_slopes(hq), w[f"{name}.mix.sink"])
+    y = attend(rnd(q), rnd(k), rnd(v), mixer["scale"], window, distance_slopes(hq) if "distance" in has else None,
+               w[f"{name}.mix.sink"] if "sink" in has else None)
     return rnd(linear(rnd(y.reshape(t, hq * e)), w[f"{name}.mix.o"]))
 
 
@@ -88,13 +93,14 @@ def gated_mlp(h, w, name, rnd=ident):
     return rnd(linear(rnd(a), w[f"{name}.mlp.down"]))
 
 
-def layer(x, w, i, spec, eps, rnd=ident):
+def layer(x, w, i, spec, eps, rnd=ident, has=ALL):
     n = f"l{i}"
-    y = attention_mixer(rnd(root_mean_square_norm(x, eps, w[n + ".norm1"])), w, n, spec["mixer"], eps, rnd)
-    x = x + root_mean_square_norm(y, eps, w[n + ".norm1b"])
+    post = (lambda y, p: root_mean_square_norm(y, eps, w[f"{n}.{p}"])) if "post_norm" in has else (lambda y, p: y)
+    y = attention_mixer(rnd(root_mean_square_norm(x, eps, w[n + ".norm1"])), w, n, spec["mixer"], eps, rnd, has)
+    x = x + post(y, "norm1b")
     if spec.get("mlp"):
         y = gated_mlp(rnd(root_mean_square_norm(x, eps, w[n + ".norm2"])), w, n, rnd)
-        x = x + root_mean_square_norm(y, eps, w[n + ".norm2b"])
+        x = x + post(y, "norm2b")
     return x
 
 
@@ -108,7 +114,7 @@ def layer_runs(cfg):
     return [(i, False) for i in range(a)] + one * loop["times"] + [(i, False) for i in range(b, n)]
 
 
-def forward(tokens, w, cfg, rnd=ident, dtype=np.float64, want_layers=False):
+def forward(tokens, w, cfg, rnd=ident, dtype=np.float64, want_layers=False, has=ALL):
     """Logits [T, vocab] of one sequence (and the residual after every layer run)."""
     eps = cfg["norm"]["eps"]
     x0 = x = w["embed"][np.asarray(tokens)].astype(dtype) * dtype(cfg["embedding"]["scale"])
@@ -116,7 +122,7 @@ def forward(tokens, w, cfg, rnd=ident, dtype=np.float64, want_layers=False):
     for i, opens in layer_runs(cfg):
         if opens:
             x = linear(np.concatenate([rnd(x), rnd(x0)], -1), w["loop.in"])
-        x = layer(x, w, i, cfg["layers"][i], eps, rnd)
+        x = layer(x, w, i, cfg["layers"][i], eps, rnd, has)
         trail.append(x)
     logits = linear(rnd(root_mean_square_norm(x, eps, w["final.norm"])), w["head"])
     return (logits, np.stack(trail)) if want_layers else logits
@@ -144,3 +150,39 @@ def tensor_shapes(cfg):
             out[f"{n}.{p}"] = (d,)
     out["final.norm"], out["head"] = (d,), (cfg["vocab"], d)
     return out
+
+
+def random_weights(cfg, seed, spread=1.0):
+    """Weights as bf16 can hold them: projections keep unit variance (times `spread`), norms scatter around 1, biases and
+    sinks are large enough to be missed."""
+    from .ref_math import bf16_round
+
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg).items():
+        if ".norm" in name or name == "final.norm":
+            a = 1.0 + 0.3 * rng.normal(size=shape)
+        elif name.endswith(".b"):
+            a = 0.5 * rng.normal(size=shape)
+        elif name.endswith(".sink"):
+            a = 1.0 + rng.normal(size=shape)
+        elif name == "embed":
+            a = rng.normal(size=shape) / cfg["embedding"]["scale"]
+        else:
+            a = spread * rng.normal(size=shape) / np.sqrt(shape[1])
+        out[name] = bf16_round(a.astype(np.float32)).astype(np.float64)
+    return out
+
+
+def write_model(folder, cfg, weights):
+    """A model folder (config.json, model.safetensors) with these weights in bf16."""
+    import json
+    import os
+
+    from dmlx_b200.safetensors_io import write_safetensors
+
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    bits = lambda a: (a.astype(np.float32).view(np.uint32) >> 16).astype(np.uint16)
+    write_safetensors(os.path.join(folder, "model.safetensors"), {n: ("BF16", bits(a)) for n, a in weights.items()}, {})
