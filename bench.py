@@ -14,6 +14,8 @@ Prints ONE JSON line (rank 0).  Workloads (synthetic seeded inputs):
       sequences, contexts log-uniform 128..32768, 32 query / 8 KV heads, head_dim 128, 32-token
       pages scattered by a random permutation over a pool of 1.25x the pages in use.
       One step = one decode of all 64 sequences through one attention layer.
+  tafuvik : the looped decoder stack (one GPU) beside the LLaMA stack at equal size, both bf16 — decode steps of 64
+      requests and prefill steps of 4096 rows at a few layer shapes, with each kernel category against its roofline.
 Multi-GPU (torchrun, one rank per GPU): independent replicas of the workload, no collective in the
 step (requests never interact); `value` = tokens of all ranks / max-over-ranks time.
 """
@@ -1088,6 +1090,147 @@ def run_reference(args, rank: int):
     }))
 
 
+# Layer shapes of the looped decoder and of the LLaMA stack beside it (head widths the latter has): six layer runs each.
+DECODER_SIZES = {
+    "d4096_h32x8_k128v128": dict(hidden=4096, heads=32, kv_heads=8, key_dim=128, value_dim=128, ffn=14336, llama_dim=128),
+    "d2048_h16x4_k96v64": dict(hidden=2048, heads=16, kv_heads=4, key_dim=96, value_dim=64, ffn=8192, llama_dim=128),
+    "d2048_h32x8_k64v64": dict(hidden=2048, heads=32, kv_heads=8, key_dim=64, value_dim=64, ffn=8192, llama_dim=64),
+}
+DECODER_VOCAB, DECODER_REQS, DECODER_ROWS = 32768, 64, 4096
+
+
+def _decoder_work(z, runs, window, ctxs, prefill, llama):
+    """Algorithmic work of one step by category: (bytes, flops) of attention, matmuls, cache append, the rest."""
+    kd, vd = (z["llama_dim"],) * 2 if llama else (z["key_dim"], z["value_dim"])
+    hq, g, d, f = z["heads"], z["kv_heads"], z["hidden"], z["ffn"]
+    rows = DECODER_ROWS if prefill else len(ctxs)
+    heads_out = len(ctxs)
+    if prefill:
+        per = rows // len(ctxs)
+        keys = len(ctxs) * float(np.minimum(np.arange(per) + 1, window or per).sum())
+        read = float(rows)  # every cached token once
+    else:
+        keys = read = float(np.minimum(ctxs, window or 1 << 30).sum())
+    attn_b = runs * (read * g * (kd + vd) * 2 + rows * hq * (kd + vd) * 2)
+    attn_f = runs * keys * hq * (kd + vd) * 2
+    weights = runs * (d * (hq * kd + g * (kd + vd)) + d * hq * vd + 3 * d * f) + d * DECODER_VOCAB
+    flops = 2.0 * rows * (weights - d * DECODER_VOCAB) + 2.0 * heads_out * d * DECODER_VOCAB
+    qkv = hq * kd + g * (kd + vd)
+    return {"attention": (attn_b, attn_f), "matmul": (weights * 2.0, flops), "rope_append": (runs * rows * qkv * 4.0, 0.0),
+            "other": (runs * rows * d * (28.0 if not llama else 8.0), 0.0)}
+
+
+def run_tafuvik(args, local: int):
+    import torch
+
+    from dmlx_b200 import device as dev
+
+    torch.cuda.set_device(local)
+    torch.cuda.set_stream(torch.cuda.Stream())
+    hbm, kind = load_peaks()
+    p = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    tflops = float(json.load(open(p))["bf16_tflops"]) if os.path.exists(p) else 1590.0
+    K, W = min(args.steps, 50), max(args.warmup, 3)
+    rng = np.random.default_rng(77)
+    ctxs = np.clip(np.rint(rng.lognormal(np.log(2600), 0.6, DECODER_REQS)), 256, 12000).astype(np.int64)
+    sampler = ClockSampler(local)
+    sampler.start()
+    out, launches = {}, 0
+    flags = dev.DEC_QKV_BIAS | dev.DEC_QK_NORM | dev.DEC_DISTANCE_BIAS | dev.DEC_SINK | dev.DEC_POST_NORM
+    for name, z in DECODER_SIZES.items():
+        for which in ("llama", "tafuvik_whole_context", "tafuvik_window_1024"):
+            llama, window = which == "llama", 1024 if which.endswith("1024") else 0
+            pages = int((-(-(ctxs + 4 * (K + W) + 64) // PAGE)).sum()) + 16
+            most = int(-(-(ctxs.max() + 4 * (K + W) + 64) // PAGE))
+            if llama:
+                model = dev.LlamaModel(6, z["hidden"], z["heads"], z["kv_heads"], z["llama_dim"], z["ffn"], DECODER_VOCAB, DECODER_ROWS,
+                                       DECODER_REQS, DECODER_REQS)
+                model.random_init(dev.Q_BF16, 3)
+                kv = dev.PagedKVCache(6, z["kv_heads"], z["llama_dim"], pages, DECODER_REQS, most, z["heads"], max_rows=DECODER_ROWS)
+            else:
+                layer = dict(n_heads=z["heads"], n_kv_heads=z["kv_heads"], key_dim=z["key_dim"], value_dim=z["value_dim"], window=window,
+                             ffn=z["ffn"], flags=flags, scale=z["key_dim"] ** -0.5)
+                model = dev.DecoderModel(z["hidden"], DECODER_VOCAB, [layer] * 4, 1e-5, 1.0, (1, 3, 2), dev.DT_BF16, DECODER_ROWS, DECODER_REQS,
+                                         DECODER_REQS)
+                model.random_init(3)
+                kv = model.make_cache(pages, DECODER_REQS, most)
+            kv.set_free_order(np.random.default_rng(5).permutation(pages).tolist())
+            for mode in ("decode", "prefill"):
+                kv.reset()
+                kv.set_free_order(np.random.default_rng(5).permutation(pages).tolist())
+                lens = ctxs.copy()
+                steps = K if mode == "decode" else max(K // 5, 4)
+                tokens = torch.randint(0, DECODER_VOCAB, (DECODER_ROWS,), dtype=torch.int32, device="cuda")
+                if mode == "decode":
+                    kv.reserve(dev.pack_desc_array([(i, int(n), 0, -1) for i, n in enumerate(ctxs)]).cuda())
+                cur = torch.zeros((DECODER_REQS if mode == "decode" else 2, 4), dtype=torch.int32, device="cuda")
+
+                def one(_=None):
+                    if mode == "decode":
+                        cur.copy_(torch.tensor([(i, 1, int(n), -1) for i, n in enumerate(lens)], dtype=torch.int32).pin_memory(), non_blocking=True)
+                        model.forward_device(kv, cur, DECODER_REQS)
+                        lens[:] += 1
+                    else:
+                        half = DECODER_ROWS // 2
+                        cur.copy_(torch.tensor([(0, half, 0, 0), (1, half, 0, half)], dtype=torch.int32).pin_memory(), non_blocking=True)
+                        model.forward_device(kv, cur, DECODER_ROWS, tokens)
+
+                def between():
+                    if mode == "prefill":  # pages back for the next prompt (on another stream: after the step has finished)
+                        torch.cuda.synchronize()
+                        kv.release([0, 1])
+
+                for _ in range(W):
+                    one()
+                    between()
+                torch.cuda.synchronize()
+                before = model.launch_count()
+                evs = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(steps if mode == "prefill" else 1)]
+                if mode == "prefill":
+                    for a, b in evs:
+                        a.record()
+                        one()
+                        b.record()
+                        between()
+                else:
+                    evs[0][0].record()
+                    for _ in range(steps):
+                        one()
+                    evs[0][1].record()
+                torch.cuda.synchronize()
+                ms = sum(a.elapsed_time(b) for a, b in evs) / steps
+                launches += model.launch_count() - before
+                model.profile_enable(True)
+                for _ in range(4):
+                    one()
+                    between()
+                prof = model.profile_collect()
+                model.profile_enable(False)
+                assert kv.error_word() == 0 and dev.qmm_error_word() == 0
+                rows = DECODER_REQS if mode == "decode" else DECODER_ROWS
+                work = _decoder_work(z, 6, window, ctxs if mode == "decode" else ctxs[:2], mode == "prefill", llama)
+                entry = {"ms_per_step": ms, "tokens_per_s": rows / ms * 1e3}
+                for cat, (nbytes, flops) in work.items():
+                    t = prof[cat][0] / 4
+                    ideal = max(nbytes / hbm / 1e6, flops / tflops / 1e9)
+                    entry[cat] = {"ms": t, "of_roofline": ideal / t if t > 0 else None}
+                out.setdefault(name, {}).setdefault(mode, {})[which] = entry
+            kv.close()
+            model.close()
+    clocks = sampler.stop()
+    head = out["d4096_h32x8_k128v128"]["decode"]["tafuvik_window_1024"]
+    print(json.dumps({
+        "metric": "decode tokens/sec (looped decoder stack, 6 layer runs)", "value": head["tokens_per_s"], "unit": "decode tokens/s", "n_gpus": 1,
+        "steps": K, "warmup": W, "ms_per_step": head["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "tafuvik", "layer_runs": 6, "vocab": DECODER_VOCAB, "decode_requests": DECODER_REQS,
+                   "cached_tokens": int(ctxs.sum()), "prefill": f"2 prompts of {DECODER_ROWS // 2} tokens in one step", "parallelism": "dp1",
+                   "l2": "weights and caches larger than L2"},
+        "note": "of_roofline: the larger of bytes / measured copy bandwidth and FLOPs / measured burst bf16 rate, over the category's time "
+                "(eager launches with an event pair each, so small kernels carry their launch gap)",
+        "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind}, "sizes": out, "e2e": None, "gpu_launches": launches, "clocks": clocks}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1139,6 +1282,10 @@ def main():
     if args.mx_persistent >= 0:
         from dmlx_b200 import _lib
         _lib.lib.b200_set_qmm_mx_persistent(args.mx_persistent)
+    if args.workload == "tafuvik":
+        if rank == 0:
+            run_tafuvik(args, local)
+        return
     if args.workload == "llama8b_int4_arrivals":
         run_arrivals(args, rank, world, local)
         return

@@ -300,7 +300,7 @@ _sig("b200_decoder_recorded_layers", i32, vp, i32, P(f32))
 _sig("b200_decoder_set_attn_mma", None, vp, i32)
 _sig("b200_decoder_model", vp, vp)
 _sig("b200_decoder_qkv", i32, vp, i32, vp, i32, vp, i32, i32, f32, vp, vp, vp, i32, vp)
-_sig("b200_decoder_attention", i32, vp, i32, vp, i32, i32, f32, vp, vp, vp, vp, i32, i32, i32, vp, i32, vp)
+_sig("b200_decoder_attention", i32, vp, i32, vp, i32, i32, f32, vp, vp, vp, vp, i32, i32, vp, i32, vp)
 _sig("b200_engine_create_model", vp, vp, vp, u64)
 
 _sig("b200_request_prompt", u64, vp, P(u32), u64)

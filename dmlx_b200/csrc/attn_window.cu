@@ -18,6 +18,7 @@
 
 #include <algorithm>
 #include <cmath>
+#include <type_traits>
 
 #include "common.h"
 #include "kv_pool.cuh"
@@ -83,11 +84,12 @@ __device__ __forceinline__ int group_pages(int ctx_first, int ctx_last, int wind
   return (max(ctx_last, 1) - 1) / page_size - first_key(ctx_first, window) / page_size + 1;
 }
 
-// Groups of rows and their chunks.  The chunk length (pages) follows the batch: long chunks cost fewer partial sums,
-// short ones give a small batch enough work items for the grid; prefill batches of many groups take one chunk per group.
-// It doubles until the partial slots fit the scratch (with one chunk per group there are none), so a step always fits.
+// Groups of rows and their chunks.  A group's pages are cut evenly into ceil(pages / ppc) chunks.  ppc is the candidate with
+// the smallest estimated time, in pages of one worker's stream: the average load or the longest item, half an item for
+// the uneven end of the walk, a page and a bit per item for its start and end, and, where groups are cut, the partial sums
+// and the combine pass.  It doubles until the partial slots fit the scratch (uncut groups need none), so a step always fits.
 __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict__ row_seq, const int* __restrict__ row_ctx, int total_rows,
-                                                           int page_size, int window, int q_tokens, int single_chunk, int items_per_chunk,
+                                                           int page_size, int window, int q_tokens, int items_per_chunk,
                                                            int n_workers, int forced_ppc, int max_slots, int* __restrict__ group_first,
                                                            int* __restrict__ chunk_start, int* __restrict__ part_base,
                                                            int* __restrict__ row_group, int* __restrict__ hdr) {
@@ -118,18 +120,50 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
   int ppc = 0x3fffffff;
   if (forced_ppc > 0) {
     ppc = forced_ppc;
-  } else if (!single_chunk) {
-    int pages = 0;
-    for (int g = tid; g < n_groups; g += blockDim.x)
-      pages += group_pages(row_ctx[group_first[g]], row_ctx[group_first[g + 1] - 1], window, page_size);
-    // a sum of at most 2^20 rows x 2^15 pages would overflow; saturate per thread
-    pages = min(max(pages, 0), 0x7fffffff / 1024);
-    const int total = scan_incl<false>(pages, warp_buf);
-    if (tid == blockDim.x - 1) carry_chunks = total;
+  } else {
+    constexpr int kCand = 6;  // 4, 8, 16, 32, 64 pages, uncut
+    long long chunks[kCand] = {}, slots[kCand] = {}, pages_sum = 0;
+    int longest = 0;
+    for (int g = tid; g < n_groups; g += blockDim.x) {
+      const int first = group_first[g], next = group_first[g + 1];
+      const int pages = group_pages(row_ctx[first], row_ctx[next - 1], window, page_size);
+      pages_sum += pages;
+      longest = max(longest, pages);
+#pragma unroll
+      for (int k = 0; k < kCand; ++k) {
+        const int c = k == kCand - 1 ? 1 : (pages + (4 << k) - 1) >> (k + 2);
+        chunks[k] += c;
+        slots[k] += c > 1 ? c * (next - first) : 0;
+      }
+    }
+    __shared__ long long s_red[32][2 * kCand + 2];
+#pragma unroll
+    for (int k = 0; k < 2 * kCand + 2; ++k) {
+      long long v = k < kCand ? chunks[k < kCand ? k : 0] : (k < 2 * kCand ? slots[k < 2 * kCand ? (k >= kCand ? k - kCand : 0) : 0] : (k == 2 * kCand ? pages_sum : longest));
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const long long w = __shfl_xor_sync(0xffffffffu, v, o);
+        v = k == 2 * kCand + 1 ? (v > w ? v : w) : v + w;
+      }
+      if ((tid & 31) == 0) s_red[tid >> 5][k] = v;
+    }
     __syncthreads();
-    const int all = carry_chunks, mean = all / max(n_groups, 1);
-    const long long spread = (long long)all * items_per_chunk / (2 * n_workers);
-    ppc = (int)min((long long)(mean < 96 ? 8 : (mean < 192 ? 16 : 32)), max(spread, 4ll));
+    if (tid == 0) {
+      long long tot[2 * kCand + 2] = {};
+      for (int w = 0; w < (int)(blockDim.x >> 5); ++w)
+        for (int k = 0; k < 2 * kCand + 2; ++k) tot[k] = k == 2 * kCand + 1 ? (tot[k] > s_red[w][k] ? tot[k] : s_red[w][k]) : tot[k] + s_red[w][k];
+      const float per = (float)items_per_chunk / (float)n_workers, load = (float)tot[2 * kCand] * per;
+      float best = 3.4e38f;
+      for (int k = 0; k < kCand; ++k) {
+        const float length = fminf(k == kCand - 1 ? 1e9f : (float)(4 << k), (float)tot[2 * kCand + 1]);
+        const float items = (float)tot[k] * per;
+        float t = fmaxf(load, length) + (items > 1.f ? 0.5f * length : 0.f) + 1.25f * items;
+        if (tot[kCand + k] > 0) t += 3.f + 0.25f * (float)tot[kCand + k] * per;
+        if (t < best) { best = t; carry_chunks = k; }
+      }
+    }
+    __syncthreads();
+    ppc = carry_chunks == kCand - 1 ? 0x3fffffff : 4 << carry_chunks;
     __syncthreads();
   }
   for (int round = 0; round < 32; ++round) {
@@ -170,7 +204,7 @@ struct WinItem {
   int head, block, seq, first_row, n_rows, ctx0, page_begin, page_end, slot0;  // slot0 < 0: the group has one chunk
 };
 
-__device__ __forceinline__ WinItem decode_item(const WinArgs& a, int item, int n_groups, int ppc) {
+__device__ __forceinline__ WinItem decode_item(const WinArgs& a, int item, int n_groups) {
   WinItem it;
   const int per_chunk = a.L.heads * a.n_blocks;
   const int chunk = item / per_chunk, rest = item - chunk * per_chunk;
@@ -185,11 +219,12 @@ __device__ __forceinline__ WinItem decode_item(const WinArgs& a, int item, int n
   it.n_rows = a.group_first[lo + 1] - it.first_row;
   it.seq = a.row_seq[it.first_row];
   it.ctx0 = a.row_ctx[it.first_row];
-  const int c = chunk - a.chunk_start[lo];
+  const int c = chunk - a.chunk_start[lo], n_chunks = a.chunk_start[lo + 1] - a.chunk_start[lo];
   const int p0 = first_key(it.ctx0, a.window) / a.d.page_size;
-  const int p_end = (it.ctx0 + it.n_rows - 1 - 1) / a.d.page_size + 1;
-  it.page_begin = p0 + (c == 0 ? 0 : c * ppc);
-  it.page_end = ppc < p_end - it.page_begin ? it.page_begin + ppc : p_end;
+  const int pages = (it.ctx0 + it.n_rows - 2) / a.d.page_size + 1 - p0;
+  const int each = pages / n_chunks, more = pages - each * n_chunks;  // the first `more` chunks hold one page more
+  it.page_begin = p0 + c * each + min(c, more);
+  it.page_end = it.page_begin + each + (c < more ? 1 : 0);
   it.slot0 = a.part_base[lo] < 0 ? -1 : a.part_base[lo] + c * it.n_rows;
   return it;
 }
@@ -205,6 +240,11 @@ __device__ __forceinline__ void ldsm4_trans(uint32_t addr, uint32_t (&r)[4]) {
 __device__ __forceinline__ void mma16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 // (p0, p1) as two bf16 pairs: the rounded values and the remainders.
 __device__ __forceinline__ void split_bf16(float p0, float p1, uint32_t& hi, uint32_t& lo) {
@@ -231,7 +271,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
   unsigned char* my_tiles = smem + (size_t)warp * kStages * stage_bytes;
   uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + (size_t)WARPS * kStages * stage_bytes) + warp * kStages;
   const int H = a.L.heads;
-  const int n_groups = a.hdr[0], ppc = a.hdr[1];
+  const int n_groups = a.hdr[0];
   const int n_items = a.chunk_start[n_groups] * H * a.n_blocks;
   const int worker = blockIdx.x * WARPS + warp, n_workers = gridDim.x * WARPS;
 
@@ -247,7 +287,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
   uint32_t prod_n = 0;
   auto producer_enter_item = [&]() {
     if (p_item < n_items) {
-      const WinItem it = decode_item(a, p_item, n_groups, ppc);
+      const WinItem it = decode_item(a, p_item, n_groups);
       p_begin = it.page_begin; p_page = it.page_begin; p_end = it.page_end; p_head = it.head; p_seq = it.seq;
       const int pg = it.page_begin + lane;
       if (pg < it.page_end) p_pid = a.d.block_table[(size_t)it.seq * a.d.max_pages_per_seq + pg];
@@ -287,13 +327,15 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
   const int hb = a.head_block;
   const int tokA = g / hb, headA = g - tokA * hb, tokB = (g + 8) / hb, headB = (g + 8) - tokB * hb;
   for (int item = worker; item < n_items && alive; item += n_workers) {
-    const WinItem it = decode_item(a, item, n_groups, ppc);
+    const WinItem it = decode_item(a, item, n_groups);
     const int h0 = it.head * a.G + it.block * hb;  // first query head of the block
     const int heads_here = min(hb, a.G - it.block * hb);
     const bool onA = tokA < it.n_rows && headA < heads_here, onB = tokB < it.n_rows && headB < heads_here;
     const int ctxA = onA ? it.ctx0 + tokA : 0, ctxB = onB ? it.ctx0 + tokB : 0;
     const int loA = first_key(ctxA, a.window), loB = first_key(ctxB, a.window);
     const int qhA = h0 + (onA ? headA : 0), qhB = h0 + (onB ? headB : 0);
+    const int lo_last = first_key(it.ctx0 + it.n_rows - 1, a.window);  // the latest window start of the group
+    const bool any_b = it.n_rows * hb > 8;                            // rows 8..15 of the tile carry something
     const float slA = a.slopes ? a.slopes[qhA] : 0.f, slB = a.slopes ? a.slopes[qhB] : 0.f;
     uint32_t qa0[KS], qa1[KS], qa2[KS], qa3[KS];
     {
@@ -334,48 +376,60 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
           }
         }
       }
-      // ---- online softmax on rows g (A) and g+8 (B), each with its own window and bias ----
+      // ---- online softmax on rows g (A) and, where the tile has any, g+8 (B), each with its own window and bias ----
       const int tok0 = pg * 32;
-      float mxA = kNone, mxB = kNone;
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt) {
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int tok = tok0 + nt * 8 + 2 * t + e;
-          const float sa = sc[nt][e] * a.scale_log2 - slA * (float)(ctxA - 1 - tok);
-          const float sb = sc[nt][2 + e] * a.scale_log2 - slB * (float)(ctxB - 1 - tok);
-          sc[nt][e] = tok < ctxA && tok >= loA ? sa : kNone;
-          sc[nt][2 + e] = tok < ctxB && tok >= loB ? sb : kNone;
-          mxA = fmaxf(mxA, sc[nt][e]);
-          mxB = fmaxf(mxB, sc[nt][2 + e]);
-        }
-      }
-      mxA = fmaxf(mxA, __shfl_xor_sync(0xffffffffu, mxA, 1));
-      mxA = fmaxf(mxA, __shfl_xor_sync(0xffffffffu, mxA, 2));
-      mxB = fmaxf(mxB, __shfl_xor_sync(0xffffffffu, mxB, 1));
-      mxB = fmaxf(mxB, __shfl_xor_sync(0xffffffffu, mxB, 2));
-      const float mA_new = fmaxf(mA, mxA), mB_new = fmaxf(mB, mxB);
-      const float corrA = exp2f(mA - mA_new), corrB = exp2f(mB - mB_new);
-      float psA = 0.f, psB = 0.f;
       uint32_t ph[2][4], pl[2][4];
+      // a page every row of the group sees whole needs no masks
+      const bool edge = tok0 + 32 > it.ctx0 || tok0 < lo_last;
+      auto row_softmax = [&](auto edge_tag, auto half_tag, float& m, float& l, int ctx, int lo, float slope) -> float {
+        constexpr bool EDGE = decltype(edge_tag)::value;
+        constexpr int E0 = decltype(half_tag)::value;  // 0: row g, 1: row g + 8
+        float mx = kNone;
+        const float b0 = slope * (float)(tok0 + 2 * t - (ctx - 1));  // exact integers; the bias of the lane's first key
 #pragma unroll
-      for (int kt = 0; kt < 2; ++kt) {
-        float pA[4], pB[4];
+        for (int nt = 0; nt < 4; ++nt) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float sa = sc[2 * kt + (e >> 1)][e & 1], sb = sc[2 * kt + (e >> 1)][2 + (e & 1)];
-          pA[e] = sa > kNone ? exp2f(sa - mA_new) : 0.f;
-          pB[e] = sb > kNone ? exp2f(sb - mB_new) : 0.f;
-          psA += pA[e];
-          psB += pB[e];
+          for (int e = 0; e < 2; ++e) {
+            float v = sc[nt][2 * E0 + e] * a.scale_log2 + fmaf(slope, (float)(nt * 8 + e), b0);
+            if (EDGE) {
+              const int tok = tok0 + nt * 8 + 2 * t + e;
+              v = tok < ctx && tok >= lo ? v : kNone;
+            }
+            sc[nt][2 * E0 + e] = v;
+            mx = fmaxf(mx, v);
+          }
         }
-        split_bf16(pA[0], pA[1], ph[kt][0], pl[kt][0]);
-        split_bf16(pB[0], pB[1], ph[kt][1], pl[kt][1]);
-        split_bf16(pA[2], pA[3], ph[kt][2], pl[kt][2]);
-        split_bf16(pB[2], pB[3], ph[kt][3], pl[kt][3]);
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float m_new = fmaxf(m, mx), corr = ex2(m - m_new);
+        float ps = 0.f;
+#pragma unroll
+        for (int kt = 0; kt < 2; ++kt) {
+          float p[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float v = sc[2 * kt + (e >> 1)][2 * E0 + (e & 1)];
+            p[e] = ex2(v - m_new);
+            if (EDGE) p[e] = v > kNone ? p[e] : 0.f;
+            ps += p[e];
+          }
+          split_bf16(p[0], p[1], ph[kt][E0], pl[kt][E0]);
+          split_bf16(p[2], p[3], ph[kt][2 + E0], pl[kt][2 + E0]);
+        }
+        l = l * corr + ps;
+        m = m_new;
+        return corr;
+      };
+      using T0 = std::integral_constant<int, 0>;
+      using T1 = std::integral_constant<int, 1>;
+      float corrA, corrB = 1.f;
+      corrA = edge ? row_softmax(std::true_type{}, T0{}, mA, lA, ctxA, loA, slA) : row_softmax(std::false_type{}, T0{}, mA, lA, ctxA, loA, slA);
+      if (any_b) {
+        corrB = edge ? row_softmax(std::true_type{}, T1{}, mB, lB, ctxB, loB, slB) : row_softmax(std::false_type{}, T1{}, mB, lB, ctxB, loB, slB);
+      } else {
+#pragma unroll
+        for (int kt = 0; kt < 2; ++kt) { ph[kt][1] = ph[kt][3] = pl[kt][1] = pl[kt][3] = 0u; }
       }
-      lA = lA * corrA + psA; mA = mA_new;
-      lB = lB * corrB + psB; mB = mB_new;
       if (__any_sync(0xffffffffu, corrA != 1.f || corrB != 1.f)) {
 #pragma unroll
         for (int j = 0; j < NO; ++j) { o[j][0] *= corrA; o[j][1] *= corrA; o[j][2] *= corrB; o[j][3] *= corrB; }
@@ -613,7 +667,7 @@ b200_status launch_mma_v(const b200_kv* kv, const WinArgs& a, int layer, cudaStr
 extern int b200_attn_pages_per_chunk;
 
 b200_status b200_window_attn_plan(b200_kv* kv, int32_t window, int32_t gqa, const int32_t* d_row_seq, const int32_t* d_row_ctx,
-                                  int32_t total_rows, int32_t prefill, void* stream) {
+                                  int32_t total_rows, void* stream) {
   if (total_rows <= 0) return B200_OK;
   if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
   b200_status st = sm_count();
@@ -634,7 +688,7 @@ b200_status b200_window_attn_plan(b200_kv* kv, int32_t window, int32_t gqa, cons
   const int forced = b200_attn_pages_per_chunk <= 0 ? 0 : std::min(std::max(b200_attn_pages_per_chunk, 1), 1 << 20);
   const int per_chunk = kv->cfg.n_kv_heads * ((gqa + 15) / 16);
   window_plan_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(d_row_seq, d_row_ctx, total_rows, kv->cfg.page_size, window, qt,
-                                                          prefill && total_rows >= 1024 ? 1 : 0, per_chunk, g_sms * 4, forced, kv->max_chunks,
+                                                          per_chunk, g_sms * 4, forced, kv->max_chunks,
                                                           p->buf, p->buf + R, p->buf + 2 * R, p->buf + 3 * R, p->buf + 4 * R);
   B200_LAUNCH_CHECK();
   return B200_OK;

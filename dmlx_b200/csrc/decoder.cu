@@ -459,7 +459,7 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
     const std::pair<int, int> key{s.window, s.n_heads / s.n_kv_heads};
     if (!attn_mma || !b200_window_attn_takes_mma(kv, (int)r) || std::find(planned.begin(), planned.end(), key) != planned.end()) continue;
     planned.push_back(key);
-    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, key.first, key.second, d_row_seq, d_row_ctx, T, T > n_req ? 1 : 0, stream));
+    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, key.first, key.second, d_row_seq, d_row_ctx, T, stream));
   }
   {
     RowArgs a{};
@@ -829,7 +829,7 @@ b200_status b200_decoder_qkv(b200_kv* kv, int32_t layer, const void* d_qkv, int3
 
 b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, int32_t n_q_heads, int32_t window, float scale,
                                    const float* d_slopes_log2, const float* d_sinks_log2, const int32_t* d_row_seq,
-                                   const int32_t* d_row_ctx, int32_t total_rows, int32_t prefill, int32_t mma, void* d_out,
+                                   const int32_t* d_row_ctx, int32_t total_rows, int32_t mma, void* d_out,
                                    int32_t out_stride, void* stream) {
   if (!kv->layered || layer < 0 || layer >= kv->cfg.n_layers || n_q_heads <= 0 || n_q_heads > kv->cfg.n_q_heads ||
       n_q_heads % kv->lay[layer].heads != 0 || window < 0) {
@@ -838,7 +838,7 @@ b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, 
   }
   b200_status st = B200_OK;
   if (mma && b200_window_attn_takes_mma(kv, layer))
-    st = b200_window_attn_plan(kv, window, n_q_heads / kv->lay[layer].heads, d_row_seq, d_row_ctx, total_rows, prefill, stream);
+    st = b200_window_attn_plan(kv, window, n_q_heads / kv->lay[layer].heads, d_row_seq, d_row_ctx, total_rows, stream);
   if (st != B200_OK) return st;
   WindowAttnCall c;
   c.layer = layer; c.n_q_heads = n_q_heads; c.window = window; c.q = d_q; c.q_stride = n_q_heads * kv->lay[layer].kd; c.scale = scale;

@@ -257,7 +257,7 @@ class LayeredKVCache(PagedKVCache):
         return q
 
     def window_attention(self, layer: int, q: torch.Tensor, row_seq: torch.Tensor, row_ctx: torch.Tensor, scale: float, window: int = 0,
-                         slopes: Optional[np.ndarray] = None, sinks: Optional[np.ndarray] = None, prefill: bool = False,
+                         slopes: Optional[np.ndarray] = None, sinks: Optional[np.ndarray] = None,
                          mma: bool = True) -> torch.Tensor:
         """b200_decoder_attention on q as qkv() returns it -> [T, heads, value width]."""
         t, hq, _ = q.shape
@@ -266,7 +266,7 @@ class LayeredKVCache(PagedKVCache):
         sl, sk = log2(slopes), log2(sinks)
         out = torch.empty((t, hq, vd), dtype=q.dtype, device=q.device)
         _lib.check(lib.b200_decoder_attention(self._h, layer, _ptr(q), hq, window, scale, _ptr(sl), _ptr(sk), _ptr(row_seq), _ptr(row_ctx), t,
-                                              int(prefill), int(mma), _ptr(out), hq * vd, _stream()))
+                                              int(mma), _ptr(out), hq * vd, _stream()))
         return out
 
 

@@ -647,7 +647,7 @@ b200_status b200_decoder_qkv(b200_kv* kv, int32_t layer, const void* d_qkv, int3
                              int32_t total_rows, void* stream);
 b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, int32_t n_q_heads, int32_t window, float scale,
                                    const float* d_slopes_log2, const float* d_sinks_log2, const int32_t* d_row_seq,
-                                   const int32_t* d_row_ctx, int32_t total_rows, int32_t prefill, int32_t mma, void* d_out,
+                                   const int32_t* d_row_ctx, int32_t total_rows, int32_t mma, void* d_out,
                                    int32_t out_stride, void* stream);
 
 /* ---- engine step: schedule -> pack -> model step -> postprocess ------------------------------- */

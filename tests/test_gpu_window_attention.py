@@ -83,12 +83,12 @@ def test_prompts_and_decoding_of_unequal_requests(shape, f32):
     first = {}
     for window in WINDOWS:
         for mma in ((False,) if f32 else (True, False)):
-            first[window, mma] = p.kv.window_attention(0, qd, seq, ctx, scale, window, slopes, sinks, True, mma).double().cpu().numpy()
+            first[window, mma] = p.kv.window_attention(0, qd, seq, ctx, scale, window, slopes, sinks, mma).double().cpu().numpy()
     qd2, seq2, ctx2 = p.append([(i, lens[i], more[i]) for i in range(4)], q2, k2, v2)
     for (window, mma), got in first.items():
         parts = [R.attend(*cases[0][4][i], scale, window, slopes, sinks) for i in range(4)]
         _check(got, np.concatenate(parts), f32, ("prompt", window, mma))
-        got2 = p.kv.window_attention(0, qd2, seq2, ctx2, scale, window, slopes, sinks, True, mma).double().cpu().numpy()
+        got2 = p.kv.window_attention(0, qd2, seq2, ctx2, scale, window, slopes, sinks, mma).double().cpu().numpy()
         parts = []
         for i in range(4):
             kk = np.concatenate([k[off[i]:off[i + 1]], k2[off2[i]:off2[i + 1]]])
@@ -122,11 +122,11 @@ def test_window_edges_show_a_key_one_token_off(shape, window):
             want = R.attend(q, k, v, 0.3, window)
             assert (np.abs(want[at]).max() > 1.0) == inside
             for mma in (True, False):
-                whole = p.kv.window_attention(0, qd, seq, ctx, 0.3, window, None, None, True, mma).double().cpu().numpy()
+                whole = p.kv.window_attention(0, qd, seq, ctx, 0.3, window, None, None, mma).double().cpu().numpy()
                 rows = slice(max(at - 3, 0), at + 1)
                 _check(whole[rows], want[rows], False, ("prompt", at, inside, mma))
                 one = p.kv.window_attention(0, qd[at:at + 1].contiguous(), seq[at:at + 1].contiguous(), ctx[at:at + 1].contiguous(), 0.3, window,
-                                            None, None, False, mma).double().cpu().numpy()
+                                            None, None, mma).double().cpu().numpy()
                 _check(one, want[at:at + 1], False, ("decode", at, inside, mma))
 
 
@@ -145,11 +145,10 @@ def test_sink_counts_once_whatever_the_number_of_chunks(mma):
     try:
         for chunk in (1, 3, 8, 64, 0):
             dev.set_attn_pages_per_chunk(chunk)
-            got = p.kv.window_attention(0, qd[rows].contiguous(), seq[rows].contiguous(), ctx[rows].contiguous(), 1.0, 0, None, sinks, False,
-                                        mma).double().cpu().numpy()
+            got = p.kv.window_attention(0, qd[rows].contiguous(), seq[rows].contiguous(), ctx[rows].contiguous(), 1.0, 0, None, sinks, mma).double().cpu().numpy()
             want = np.array([[(r + 1) / (r + 1 + np.exp(s)) for s in sinks] for r in rows])
             np.testing.assert_allclose(got, np.broadcast_to(want[..., None], got.shape), rtol=5e-3)
-            full = p.kv.window_attention(0, qd, seq, ctx, 1.0, 0, None, sinks, True, mma).double().cpu().numpy()
+            full = p.kv.window_attention(0, qd, seq, ctx, 1.0, 0, None, sinks, mma).double().cpu().numpy()
             np.testing.assert_allclose(full[rows], np.broadcast_to(want[..., None], got.shape), rtol=5e-3)
     finally:
         dev.set_attn_pages_per_chunk(0)
@@ -163,7 +162,7 @@ def test_distance_bias_is_relative_and_joins_before_the_sink():
     slopes, sinks = R.distance_slopes(4), np.full(4, 1.5)
     p = Pool(shape, [n], True)
     qd, seq, ctx = p.append([(0, 0, n)], q, k, v)
-    got = p.kv.window_attention(0, qd, seq, ctx, 0.2, 0, slopes, sinks, True).double().cpu().numpy()
+    got = p.kv.window_attention(0, qd, seq, ctx, 0.2, 0, slopes, sinks).double().cpu().numpy()
     _check(got, R.attend(q, k, v, 0.2, 0, slopes, sinks), True, "relative")
     assert np.abs(got - R.attend(q, k, v, 0.2, 0, slopes, None)).max() > 1e-2
     assert np.abs(got - R.attend(q, k, v, 0.2, 0, None, sinks)).max() > 1e-2
@@ -192,8 +191,8 @@ def test_far_key_among_thousands_long_context_and_full_scratch():
     want = R.attend(q[-40:], k, v, 0.125, 0)
     tail = slice(960, 1000)
     assert want[-1, 0].mean() > 3.0
-    for rows, prefill in ((tail, True), (slice(999, 1000), False)):
-        got = kv.window_attention(0, qd[rows].contiguous(), seq[rows].contiguous(), ctx[rows].contiguous(), 0.125, 0, prefill=prefill).double().cpu().numpy()
+    for rows in (tail, slice(999, 1000)):
+        got = kv.window_attention(0, qd[rows].contiguous(), seq[rows].contiguous(), ctx[rows].contiguous(), 0.125, 0).double().cpu().numpy()
         _check(got, want[-len(got):], False, rows)
     assert kv.error_word() == 0
 
