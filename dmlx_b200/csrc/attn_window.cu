@@ -27,7 +27,6 @@
 
 namespace {
 
-constexpr int kStages = 3;
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kNone = -1e30f;  // running maximum before any key
 
@@ -47,6 +46,7 @@ struct WinArgs {
   const float *slopes, *sinks;
   __nv_bfloat16* out;
   int out_stride;
+  int stages;      // ring slots (pages) per warp
 };
 
 // ---- plan ------------------------------------------------------------------------------------------------
@@ -256,24 +256,26 @@ __device__ __forceinline__ void split_bf16(float p0, float p1, uint32_t& hi, uin
 }
 
 // KB, VB: 64-column boxes a key / value row may take (1, 2 or 4); the steps beyond the layer's own widths are skipped.
-template <int KB, int VB, int WARPS>
-__global__ void __launch_bounds__(WARPS * 32, 1)
+// A block is as many independent warps as its shared memory and registers feed.
+constexpr int most_warps(int kb, int vb) { return kb + vb == 2 ? 12 : (kb + vb == 3 ? 9 : 8); }
+template <int KB, int VB>
+__global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
     window_attn_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap, WinArgs a) {
   constexpr int KS = KB * 4;  // 16-column steps of Q K^T
   constexpr int NO = VB * 8;  // 8-column tiles of the output
   const int n_kb = (a.L.kd + 63) / 64, n_vb = (a.L.vd + 63) / 64, n_ks = a.L.kd / 16, n_vs = a.L.vd / 16;
-  const int k_tile = n_kb * 4096, stage_bytes = (n_kb + n_vb) * 4096;
+  const int warps = blockDim.x >> 5, kStages = a.stages, k_tile = n_kb * 4096, stage_bytes = (n_kb + n_vb) * 4096;
 
   extern __shared__ unsigned char smem_dyn[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~(uintptr_t)1023);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, t = lane & 3;
   unsigned char* my_tiles = smem + (size_t)warp * kStages * stage_bytes;
-  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + (size_t)WARPS * kStages * stage_bytes) + warp * kStages;
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + (size_t)warps * kStages * stage_bytes) + warp * kStages;
   const int H = a.L.heads;
   const int n_groups = a.hdr[0];
   const int n_items = a.chunk_start[n_groups] * H * a.n_blocks;
-  const int worker = blockIdx.x * WARPS + warp, n_workers = gridDim.x * WARPS;
+  const int worker = blockIdx.x * warps + warp, n_workers = gridDim.x * warps;
 
   if (lane == 0) {
     for (int s = 0; s < kStages; ++s) ptx::mbar_init(&full_bar[s], 1);
@@ -284,7 +286,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
   // producer cursor (all lanes track it, lane 0 issues); the lanes hold the page ids of a window of 32 pages of the
   // item's chunk, refilled every 32 pages
   int p_item = worker, p_page = 0, p_end = 0, p_begin = 0, p_head = 0, p_pid = 0, p_seq = 0;
-  uint32_t prod_n = 0;
+  int prod_s = 0;  // slot of the next page
   auto producer_enter_item = [&]() {
     if (p_item < n_items) {
       const WinItem it = decode_item(a, p_item, n_groups);
@@ -301,7 +303,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
       if (pg < p_end) p_pid = a.d.block_table[(size_t)p_seq * a.d.max_pages_per_seq + pg];
     }
     const int pid = __shfl_sync(0xffffffffu, p_pid, rel & 31);
-    const uint32_t s = prod_n % kStages;
+    const int s = prod_s;
     if (lane == 0) {
       ptx::fence_proxy_async_smem();
       unsigned char* kd = my_tiles + (size_t)s * stage_bytes;
@@ -310,7 +312,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
       for (int b = 0; b < n_kb; ++b) ptx::tma_load_2d(kd + b * 4096, &kmap, b * 64, row0, &full_bar[s]);
       for (int b = 0; b < n_vb; ++b) ptx::tma_load_2d(kd + k_tile + b * 4096, &vmap, b * 64, row0, &full_bar[s]);
     }
-    prod_n += 1;
+    if (++prod_s == kStages) prod_s = 0;
     p_page += 1;
     if (p_page >= p_end) {
       p_item += n_workers;
@@ -321,7 +323,8 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
   for (int i = 0; i < kStages; ++i) produce_one();
 
   bool alive = true;
-  uint32_t cons_n = 0;
+  int cons_s = 0;
+  uint32_t cons_ph = 0;
   const int ld_r = lane & 7, ld_m = lane >> 3;
   // MMA rows g and g+8 of this lane: (token of the group, query head within the block)
   const int hb = a.head_block;
@@ -356,8 +359,8 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
     float mA = kNone, lA = 0.f, mB = kNone, lB = 0.f;
 
     for (int pg = it.page_begin; pg < it.page_end; ++pg) {
-      const uint32_t s = cons_n % kStages;
-      alive = ptx::mbar_wait(&full_bar[s], (cons_n / kStages) & 1u);
+      const int s = cons_s;
+      alive = ptx::mbar_wait(&full_bar[s], cons_ph);
       if (!alive) break;
       const uint32_t kbase = ptx::smem_u32(my_tiles + (size_t)s * stage_bytes), vbase = kbase + k_tile;
       float sc[4][4];
@@ -450,7 +453,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1)
         }
       }
       __syncwarp();
-      cons_n += 1;
+      if (++cons_s == kStages) { cons_s = 0; cons_ph ^= 1u; }
       produce_one();  // refill the slot just drained
     }
     if (!alive) break;
@@ -638,25 +641,41 @@ WindowPlan* find_plan(b200_kv* kv, int window, int q_tokens) {
   return nullptr;
 }
 
+// Warps of a block and ring slots per warp, by the 4 KiB boxes of a staged page (keys + values).  The warps are
+// bound by dependent issue, so more of them with two slots each beat fewer with three (decode of 64 contexts of 2600
+// tokens on average at 8 x 128 / 128: 138-181 us with 7 x 2 against 164-201 us with 4 x 3; 4 x 96 / 64: 72 us with
+// 8 x 2 against 106 us).
+struct Shape { int warps, stages; };
+Shape shape_of(int boxes) {
+  switch (boxes) {
+    case 2: return {12, 2};
+    case 3: return {8, 2};
+    case 4: return {7, 2};
+    case 5: return {5, 2};
+    case 6: return {4, 2};
+    default: return {3, 2};
+  }
+}
+
 template <int KB, int VB>
-b200_status launch_mma(const b200_kv* kv, const WinArgs& a, int layer, cudaStream_t s) {
-  constexpr int WARPS = KB + VB <= 4 ? 4 : 2;
+b200_status launch_mma(const b200_kv* kv, WinArgs& a, int layer, cudaStream_t s) {
   const int boxes = (a.L.kd + 63) / 64 + (a.L.vd + 63) / 64;
-  const size_t smem = (size_t)WARPS * kStages * boxes * 4096 + 1024 + sizeof(uint64_t) * WARPS * kStages;
+  const Shape sh = shape_of(boxes);
+  static_assert(most_warps(1, 1) >= 12 && most_warps(2, 1) >= 8 && most_warps(1, 2) >= 8, "a block's shape exceeds its launch bound");
+  a.stages = sh.stages;
+  const size_t smem = (size_t)sh.warps * sh.stages * (boxes * 4096 + sizeof(uint64_t)) + 1024;
   static bool configured = false;
   if (!configured) {
-    const int most = WARPS * kStages * (KB + VB) * 4096 + 1024 + (int)sizeof(uint64_t) * WARPS * kStages;
-    B200_CUDA_TRY((cudaFuncSetAttribute(window_attn_mma_kernel<KB, VB, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, most)));
+    B200_CUDA_TRY((cudaFuncSetAttribute(window_attn_mma_kernel<KB, VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024)));
     configured = true;
   }
-  const int per_sm = smem <= 74 * 1024 ? 3 : (smem <= 112 * 1024 ? 2 : 1);
-  window_attn_mma_kernel<KB, VB, WARPS><<<g_sms * per_sm, WARPS * 32, smem, s>>>(kv->lay_kmap[layer], kv->lay_vmap[layer], a);
+  window_attn_mma_kernel<KB, VB><<<g_sms, sh.warps * 32, smem, s>>>(kv->lay_kmap[layer], kv->lay_vmap[layer], a);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
 
 template <int KB>
-b200_status launch_mma_v(const b200_kv* kv, const WinArgs& a, int layer, cudaStream_t s) {
+b200_status launch_mma_v(const b200_kv* kv, WinArgs& a, int layer, cudaStream_t s) {
   if (a.L.vd <= 64) return launch_mma<KB, 1>(kv, a, layer, s);
   if (a.L.vd <= 128) return launch_mma<KB, 2>(kv, a, layer, s);
   return launch_mma<KB, 4>(kv, a, layer, s);
@@ -666,7 +685,7 @@ b200_status launch_mma_v(const b200_kv* kv, const WinArgs& a, int layer, cudaStr
 
 extern int b200_attn_pages_per_chunk;
 
-b200_status b200_window_attn_plan(b200_kv* kv, int32_t window, int32_t gqa, const int32_t* d_row_seq, const int32_t* d_row_ctx,
+b200_status b200_window_attn_plan(b200_kv* kv, int32_t layer, int32_t window, int32_t gqa, const int32_t* d_row_seq, const int32_t* d_row_ctx,
                                   int32_t total_rows, void* stream) {
   if (total_rows <= 0) return B200_OK;
   if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
@@ -686,9 +705,10 @@ b200_status b200_window_attn_plan(b200_kv* kv, int32_t window, int32_t gqa, cons
     kv->plans.push_back(p);
   }
   const int forced = b200_attn_pages_per_chunk <= 0 ? 0 : std::min(std::max(b200_attn_pages_per_chunk, 1), 1 << 20);
-  const int per_chunk = kv->cfg.n_kv_heads * ((gqa + 15) / 16);
+  const KvLayerDev& L = kv->lay[layer];
+  const int per_chunk = L.heads * ((gqa + 15) / 16), warps = shape_of((L.kd + 63) / 64 + (L.vd + 63) / 64).warps;
   window_plan_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(d_row_seq, d_row_ctx, total_rows, kv->cfg.page_size, window, qt,
-                                                          per_chunk, g_sms * 4, forced, kv->max_chunks,
+                                                          per_chunk, g_sms * warps, forced, kv->max_chunks,
                                                           p->buf, p->buf + R, p->buf + 2 * R, p->buf + 3 * R, p->buf + 4 * R);
   B200_LAUNCH_CHECK();
   return B200_OK;

@@ -140,73 +140,104 @@ struct RowArgs {
   int cat_stride = 0;
 };
 
-// One CTA per row: sublayer output -> residual stream -> what the next matmul reads.
-template <typename T, int VEC>
+// One CTA per row: sublayer output -> residual stream -> what the next matmul reads.  NQ > 0: a thread keeps its NQ
+// groups of VEC columns in registers and asks for the residual before the first reduction; NQ = 0: any width, the row
+// waits in shared memory.
+template <typename T, int VEC, int NQ>
 __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
   extern __shared__ float row_sh[];
   __shared__ float part[32];
   const int row = blockIdx.x, n = a.hidden / VEC;
   float* xr = a.x + (size_t)row * a.hidden;
+  float* x0r = a.x0 ? a.x0 + (size_t)row * a.hidden : nullptr;
+  Vec<VEC> keep[NQ > 0 ? NQ : 1];
+  // visits the thread's groups; get/put move a group between them and registers or shared memory
+  auto each = [&](auto f) {
+    if constexpr (NQ > 0) {
+#pragma unroll
+      for (int k = 0; k < NQ; ++k) {
+        const int i = threadIdx.x + k * blockDim.x;
+        if (i < n) f(i, k);
+      }
+    } else {
+      for (int i = threadIdx.x; i < n; i += blockDim.x) f(i, 0);
+    }
+  };
+  auto get = [&](int i, int k) -> Vec<VEC> {
+    if constexpr (NQ > 0) return keep[k];
+    else return load_vec<VEC>(row_sh + i * VEC);
+  };
+  auto put = [&](int i, int k, const Vec<VEC>& v) {
+    if constexpr (NQ > 0) keep[k] = v;
+    else store_vec<VEC>(row_sh + i * VEC, v);
+  };
   float ss = 0.f;
   if (a.tokens) {
     const uint32_t tok = min(a.tokens[row], (uint32_t)(a.vocab - 1));
     const __nv_bfloat16* e = a.embed + (size_t)tok * a.hidden;
-    float* x0r = a.x0 ? a.x0 + (size_t)row * a.hidden : nullptr;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    each([&](int i, int k) {
       Vec<VEC> v = load_vec<VEC>(e + i * VEC);
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) { v.v[k] *= a.embed_scale; ss += v.v[k] * v.v[k]; }
-      store_vec<VEC>(row_sh + i * VEC, v);
+      for (int j = 0; j < VEC; ++j) { v.v[j] *= a.embed_scale; ss += v.v[j] * v.v[j]; }
+      put(i, k, v);
       store_vec<VEC>(xr + i * VEC, v);
       if (x0r) store_vec<VEC>(x0r + i * VEC, v);
-    }
+    });
   } else {
     float ys = 0.f;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    Vec<VEC> res[NQ > 0 ? NQ : 1];
+    each([&](int i, int k) {
+      if constexpr (NQ > 0) { if (!a.replace) res[k] = load_vec<VEC>(xr + i * VEC); }
       const Vec<VEC> v = mat_value<T, VEC>(a.src, row, i * VEC);
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) ys += v.v[k] * v.v[k];
-      store_vec<VEC>(row_sh + i * VEC, v);
-    }
+      for (int j = 0; j < VEC; ++j) ys += v.v[j] * v.v[j];
+      put(i, k, v);
+    });
     const float r = a.post_w ? 1.0f / sqrtf(block_sum(ys, part) / (float)a.hidden + a.eps) : 1.f;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {  // a thread meets the columns it wrote itself
-      Vec<VEC> v = load_vec<VEC>(row_sh + i * VEC);
+    each([&](int i, int k) {
+      Vec<VEC> v = get(i, k);
       if (a.post_w) {
         const Vec<VEC> w = load_vec<VEC>(a.post_w + i * VEC);
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) v.v[k] *= r * w.v[k];
+        for (int j = 0; j < VEC; ++j) v.v[j] *= r * w.v[j];
       }
       if (!a.replace) {
-        const Vec<VEC> x = load_vec<VEC>(xr + i * VEC);
+        Vec<VEC> x;
+        if constexpr (NQ > 0) x = res[k];
+        else x = load_vec<VEC>(xr + i * VEC);
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) v.v[k] += x.v[k];
+        for (int j = 0; j < VEC; ++j) v.v[j] += x.v[j];
       }
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) ss += v.v[k] * v.v[k];
-      store_vec<VEC>(row_sh + i * VEC, v);
+      for (int j = 0; j < VEC; ++j) ss += v.v[j] * v.v[j];
+      put(i, k, v);
       store_vec<VEC>(xr + i * VEC, v);
-    }
+    });
   }
   if (a.norm_w) {
     const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)a.hidden + a.eps);
     T* hr = (T*)a.h + (size_t)row * a.h_stride;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-      Vec<VEC> v = load_vec<VEC>(row_sh + i * VEC);
+    each([&](int i, int k) {
+      Vec<VEC> v = get(i, k);
       const Vec<VEC> w = load_vec<VEC>(a.norm_w + i * VEC);
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) v.v[k] *= r * w.v[k];
+      for (int j = 0; j < VEC; ++j) v.v[j] *= r * w.v[j];
       store_vec<VEC>(hr + i * VEC, v);
-    }
+    });
   }
   if (a.cat) {
     T* cr = (T*)a.cat + (size_t)row * a.cat_stride;
-    const float* x0r = a.x0 + (size_t)row * a.hidden;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-      store_vec<VEC>(cr + i * VEC, load_vec<VEC>(row_sh + i * VEC));
-      // the embedding row itself was written by this thread above
-      store_vec<VEC>(cr + a.hidden + i * VEC, load_vec<VEC>(x0r + i * VEC));
-    }
+    each([&](int i, int k) {
+      store_vec<VEC>(cr + i * VEC, get(i, k));
+      store_vec<VEC>(cr + a.hidden + i * VEC, load_vec<VEC>(x0r + i * VEC));  // (an embedding row was written by this thread)
+    });
   }
+}
+
+template <typename T>
+void (*rows_kernel(int vec, int nq))(RowArgs) {
+  if (vec == 1) return decoder_rows_kernel<T, 1, 0>;
+  return nq <= 1 ? decoder_rows_kernel<T, 4, 1> : (nq <= 2 ? decoder_rows_kernel<T, 4, 2> : (nq <= 4 ? decoder_rows_kernel<T, 4, 4> : decoder_rows_kernel<T, 4, 0>));
 }
 
 // Rows idx[r] of x, normalised, as the head's operand.
@@ -421,10 +452,9 @@ b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t 
     else a.norm_w = layers[runs[next].layer].norm1;
   }
   const int vec = cfg.hidden % 4 == 0 ? 4 : 1;
-  const int threads = std::min(512, (cfg.hidden / vec + 31) / 32 * 32);
-  const size_t smem = sizeof(float) * cfg.hidden;
-  auto* kernel = f32() ? (vec == 4 ? decoder_rows_kernel<float, 4> : decoder_rows_kernel<float, 1>)
-                       : (vec == 4 ? decoder_rows_kernel<__nv_bfloat16, 4> : decoder_rows_kernel<__nv_bfloat16, 1>);
+  const int threads = std::min(512, (cfg.hidden / vec + 31) / 32 * 32), nq = (cfg.hidden / vec + threads - 1) / threads;
+  const size_t smem = vec == 4 && nq <= 4 ? 0 : sizeof(float) * cfg.hidden;
+  auto* kernel = f32() ? rows_kernel<float>(vec, nq) : rows_kernel<__nv_bfloat16>(vec, nq);
   if (smem > 47 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   kernel<<<rows, threads, smem, s>>>(a);
   B200_LAUNCH_CHECK();
@@ -459,7 +489,7 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
     const std::pair<int, int> key{s.window, s.n_heads / s.n_kv_heads};
     if (!attn_mma || !b200_window_attn_takes_mma(kv, (int)r) || std::find(planned.begin(), planned.end(), key) != planned.end()) continue;
     planned.push_back(key);
-    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, key.first, key.second, d_row_seq, d_row_ctx, T, stream));
+    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, (int)r, key.first, key.second, d_row_seq, d_row_ctx, T, stream));
   }
   {
     RowArgs a{};
@@ -838,7 +868,7 @@ b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, 
   }
   b200_status st = B200_OK;
   if (mma && b200_window_attn_takes_mma(kv, layer))
-    st = b200_window_attn_plan(kv, window, n_q_heads / kv->lay[layer].heads, d_row_seq, d_row_ctx, total_rows, stream);
+    st = b200_window_attn_plan(kv, layer, window, n_q_heads / kv->lay[layer].heads, d_row_seq, d_row_ctx, total_rows, stream);
   if (st != B200_OK) return st;
   WindowAttnCall c;
   c.layer = layer; c.n_q_heads = n_q_heads; c.window = window; c.q = d_q; c.q_stride = n_q_heads * kv->lay[layer].kd; c.scale = scale;

@@ -91,8 +91,9 @@ struct WindowAttnCall {
   void* out = nullptr;
   int out_stride = 0;
 };
-// Builds (once per step) the plan that calls of this window and GQA group size share.
-b200_status b200_window_attn_plan(b200_kv* kv, int32_t window, int32_t gqa_group, const int32_t* d_row_seq, const int32_t* d_row_ctx,
+// Builds (once per step) the plan that calls of this window and GQA group size share; `layer` is one of the layers it is
+// for (its shape says how many workers the grid has).
+b200_status b200_window_attn_plan(b200_kv* kv, int32_t layer, int32_t window, int32_t gqa_group, const int32_t* d_row_seq, const int32_t* d_row_ctx,
                                   int32_t total_rows, void* stream);
 // mma = false forces the CUDA-core kernel (which needs no plan).
 b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
