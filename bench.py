@@ -1132,14 +1132,15 @@ def run_tafuvik(args, local: int):
     tflops = float(json.load(open(p))["bf16_tflops"]) if os.path.exists(p) else 1590.0
     K, W = min(args.steps, 50), max(args.warmup, 3)
     rng = np.random.default_rng(77)
-    ctxs = np.clip(np.rint(rng.lognormal(np.log(2600), 0.6, DECODER_REQS)), 256, 12000).astype(np.int64)
+    all_ctxs = np.clip(np.rint(rng.lognormal(np.log(2600), 0.6, DECODER_REQS)), 256, 12000).astype(np.int64)
     sampler = ClockSampler(local)
     sampler.start()
     out, launches = {}, 0
     flags = dev.DEC_QKV_BIAS | dev.DEC_QK_NORM | dev.DEC_DISTANCE_BIAS | dev.DEC_SINK | dev.DEC_POST_NORM
     for name, z in DECODER_SIZES.items():
-        for which in ("llama", "tafuvik_whole_context", "tafuvik_window_1024"):
-            llama, window = which == "llama", 1024 if which.endswith("1024") else 0
+        for which in ("llama", "llama_contexts_of_1024", "tafuvik_whole_context", "tafuvik_window_1024"):
+            llama, window = which.startswith("llama"), 1024 if which == "tafuvik_window_1024" else 0
+            ctxs = np.minimum(all_ctxs, 1024) if which == "llama_contexts_of_1024" else all_ctxs  # as many keys as the window leaves
             pages = int((-(-(ctxs + 4 * (K + W) + 64) // PAGE)).sum()) + 16
             most = int(-(-(ctxs.max() + 4 * (K + W) + 64) // PAGE))
             if llama:
@@ -1155,7 +1156,7 @@ def run_tafuvik(args, local: int):
                 model.random_init(3)
                 kv = model.make_cache(pages, DECODER_REQS, most)
             kv.set_free_order(np.random.default_rng(5).permutation(pages).tolist())
-            for mode in ("decode", "prefill"):
+            for mode in ("decode",) if which == "llama_contexts_of_1024" else ("decode", "prefill"):
                 kv.reset()
                 kv.set_free_order(np.random.default_rng(5).permutation(pages).tolist())
                 lens = ctxs.copy()
@@ -1224,7 +1225,7 @@ def run_tafuvik(args, local: int):
         "steps": K, "warmup": W, "ms_per_step": head["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic",
         "config": {"workload": "tafuvik", "layer_runs": 6, "vocab": DECODER_VOCAB, "decode_requests": DECODER_REQS,
-                   "cached_tokens": int(ctxs.sum()), "prefill": f"2 prompts of {DECODER_ROWS // 2} tokens in one step", "parallelism": "dp1",
+                   "cached_tokens": int(all_ctxs.sum()), "prefill": f"2 prompts of {DECODER_ROWS // 2} tokens in one step", "parallelism": "dp1",
                    "l2": "weights and caches larger than L2"},
         "note": "of_roofline: the larger of bytes / measured copy bandwidth and FLOPs / measured burst bf16 rate, over the category's time "
                 "(eager launches with an event pair each, so small kernels carry their launch gap)",

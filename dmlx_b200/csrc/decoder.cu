@@ -452,7 +452,7 @@ b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t 
     else a.norm_w = layers[runs[next].layer].norm1;
   }
   const int vec = cfg.hidden % 4 == 0 ? 4 : 1;
-  const int threads = std::min(512, (cfg.hidden / vec + 31) / 32 * 32), nq = (cfg.hidden / vec + threads - 1) / threads;
+  const int threads = std::min(rows >= 512 ? 256 : 512, (cfg.hidden / vec + 31) / 32 * 32), nq = (cfg.hidden / vec + threads - 1) / threads;
   const size_t smem = vec == 4 && nq <= 4 ? 0 : sizeof(float) * cfg.hidden;
   auto* kernel = f32() ? rows_kernel<float>(vec, nq) : rows_kernel<__nv_bfloat16>(vec, nq);
   if (smem > 47 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
