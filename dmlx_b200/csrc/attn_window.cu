@@ -13,7 +13,7 @@
 // Scores, biases and softmax are f32.  The weights enter the P V product as two bf16 terms (the rounded weight and what
 // the rounding left over), so they carry 16 bits of mantissa instead of 8.
 //
-// attn_simt_kernel is the same contract on CUDA cores for any width and for f32 pools.
+// attn_simt_kernel does the same on CUDA cores for any width and for f32 pools.
 #include <cuda_bf16.h>
 
 #include <algorithm>

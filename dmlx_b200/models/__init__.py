@@ -1,8 +1,8 @@
 """Models by configuration: a folder with config.json and model.safetensors becomes a model on the device.
 
-Each architecture registers a loader under the names its config.json may carry (the role of the reference's
-model registry, src/model_registry.zig): `load_model(path)` reads the configuration, picks the loader and
-returns a `LoadedModel`, which the engine, the command line and the trace replay all drive the same way.
+Each architecture registers a loader under the names its config.json may carry: `load_model(path)` reads the
+configuration, picks the loader and returns a `LoadedModel`, which the engine, the command line and the trace replay
+all drive the same way.
 """
 from __future__ import annotations
 
