@@ -24,101 +24,13 @@
 #include "kv_pool.cuh"
 #include "model_step.cuh"
 #include "qmm.cuh"
+#include "rows.cuh"
 
 namespace {
 
 constexpr double kLog2e = 1.4426950408889634;
 
 int pad64(int n) { return (n + 63) / 64 * 64; }
-
-// Result of a matmul, row by row: f32 split-K partial tiles (ws) or rows the matmul wrote itself (y).
-struct MatSrc {
-  const float* ws = nullptr;
-  int splits = 0, tn = 0, tts = 0;
-  const void* y = nullptr;
-  int y_stride = 0;
-};
-
-__device__ __forceinline__ float ld(const float* p) { return *p; }
-__device__ __forceinline__ float ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
-__device__ __forceinline__ void st(float* p, float v) { *p = v; }
-__device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
-
-template <int VEC>
-struct Vec { float v[VEC]; };
-
-template <int VEC>
-__device__ __forceinline__ Vec<VEC> load_vec(const float* p) {
-  Vec<VEC> r;
-  if constexpr (VEC == 4) {
-    const float4 f = *reinterpret_cast<const float4*>(p);
-    r.v[0] = f.x; r.v[1] = f.y; r.v[2] = f.z; r.v[3] = f.w;
-  } else {
-    r.v[0] = *p;
-  }
-  return r;
-}
-template <int VEC>
-__device__ __forceinline__ Vec<VEC> load_vec(const __nv_bfloat16* p) {
-  Vec<VEC> r;
-  if constexpr (VEC == 4) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    r.v[0] = __uint_as_float(u.x << 16); r.v[1] = __uint_as_float(u.x & 0xFFFF0000u);
-    r.v[2] = __uint_as_float(u.y << 16); r.v[3] = __uint_as_float(u.y & 0xFFFF0000u);
-  } else {
-    r.v[0] = __bfloat162float(*p);
-  }
-  return r;
-}
-template <int VEC>
-__device__ __forceinline__ void store_vec(float* p, const Vec<VEC>& x) {
-  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(x.v[0], x.v[1], x.v[2], x.v[3]);
-  else *p = x.v[0];
-}
-template <int VEC>
-__device__ __forceinline__ void store_vec(__nv_bfloat16* p, const Vec<VEC>& x) {
-  if constexpr (VEC == 4) {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(x.v[0], x.v[1]), b = __floats2bfloat162_rn(x.v[2], x.v[3]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
-  } else {
-    *p = __float2bfloat16(x.v[0]);
-  }
-}
-
-// Columns c .. c + VEC - 1 of one row; the splits are summed in split order.
-template <typename T, int VEC>
-__device__ __forceinline__ Vec<VEC> mat_value(const MatSrc& s, int row, int c) {
-  if (!s.ws) return load_vec<VEC>((const T*)s.y + (size_t)row * s.y_stride + c);
-  const int nt = c >> 7, r = c & 127, tt = row / s.tn, tr = row - tt * s.tn;
-  const float* p = s.ws + (((size_t)(nt * s.tts + tt) * s.splits) * s.tn + tr) * 128 + r;
-  Vec<VEC> acc = load_vec<VEC>(p);
-  for (int i = 1; i < s.splits; ++i) {
-    const Vec<VEC> b = load_vec<VEC>(p + (size_t)i * s.tn * 128);
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) acc.v[e] += b.v[e];
-  }
-  return acc;
-}
-
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-
-__device__ float block_sum(float v, float* part) {
-  v = warp_sum(v);
-  __syncthreads();
-  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float t = threadIdx.x < (blockDim.x >> 5) ? part[threadIdx.x] : 0.f;
-  if (threadIdx.x < 32) {
-    t = warp_sum(t);
-    if (threadIdx.x == 0) part[0] = t;
-  }
-  __syncthreads();
-  return part[0];
-}
 
 // ---- between the matmuls ------------------------------------------------------------------------------------
 struct RowArgs {

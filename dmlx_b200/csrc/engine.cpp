@@ -81,6 +81,7 @@ uint64_t pages_needed(uint64_t len, uint64_t count) {
 // token is always left to compute (its logits give the first output token).
 b200_status try_share_prefix(b200_engine* e, b200_request* r, b200_engine::Live* self, bool* shared) {
   *shared = false;
+  if (b200_kv_state_bytes(e->kv) > 0) return B200_OK;  // a recurrent state belongs to a whole sequence, not to its pages
   const int32_t slot = b200_request_kv_slot(r);
   std::vector<uint32_t> prompt(b200_request_prompt_len(r));
   b200_request_prompt(r, prompt.data(), prompt.size());

@@ -1,0 +1,39 @@
+// Gated linear attention over the recurrent state of a layered pool (gla.cu).
+#pragma once
+#include "kv_pool.cuh"
+#include "rows.cuh"
+
+// One layer over the rows of a step.  `src` holds the projection of every row: columns [q | k | v | g | a1] of widths
+// heads * dk, heads * dk, heads * dv, heads * dv, rank.  Per head and key channel alpha = sigmoid(W_a2 a1 + b)^(1 / tau);
+// S <- diag(alpha) S + k v^T, o = S^T (q * q_scale); the output row is rms_norm(o) * norm * silu(g), [heads][dv].
+struct GlaCall {
+  int layer = 0, heads = 0, dk = 0, dv = 0, rank = 0;
+  MatSrc src;
+  const float *a2 = nullptr, *a2_bias = nullptr;  // [heads * dk][rank], [heads * dk]
+  const float* norm = nullptr;                    // [dv]
+  float q_scale = 1.f, inv_tau = 1.f, eps = 0.f;
+  void* out = nullptr;
+  int out_stride = 0;
+};
+
+// Buffers of the chunk-wise path, shared by the layers of a model: made for a number of rows and requests.
+struct GlaScratch {
+  int max_rows = 0, max_reqs = 0, max_chunks = 0;
+  size_t chunk_bytes = 0, v_bytes = 0, o_elems = 0;  // per (chunk, head); per row
+  unsigned char *chunks = nullptr, *values = nullptr;
+  float* o = nullptr;
+  int4* plan = nullptr;      // [max_chunks] {first row, rows, request, -}
+  int* first_chunk = nullptr;  // [max_reqs + 1]
+  bool alloc();              // false: out of memory
+  void need(int heads, int dk, int dv);  // before alloc: a layer of this shape will use it
+  void free();
+};
+
+// A step's rows are cut once for all layers.  Portions of more than `step_tokens` tokens go chunk by chunk on the tensor
+// cores (bf16), shorter ones token by token.
+b200_status b200_gla_plan(GlaScratch& g, const int32_t* d_cu, int n_req, int total_rows, void* stream);
+b200_status b200_gla_run(b200_kv* kv, const GlaScratch& g, const GlaCall& c, const int32_t* d_cu, const int32_t* d_row_seq,
+                         const int32_t* d_pos, int n_req, int total_rows, bool chunked, void* stream);
+// Whether a layer's shape fits the chunk-wise kernels.
+bool b200_gla_takes_chunks(int dk, int dv, int elem_bytes);
+constexpr int kGlaStepTokens = 4;

@@ -10,6 +10,7 @@
 //   k_scale,v_scale: [layer][page][kv_head] f32 (FP8 pools only)
 //   free_stack     : [n_pages] i32, entries [0, free_top) are free; free_stack[free_top-1] pops next
 //   ref_count, tokens_used : [n_pages] i32
+//   rec_pool       : [layer][slot][state_elems] f32, recurrent state of layers that have one (layered pools)
 //   block_table    : [max_seqs][max_pages_per_seq] i32 ; seq_pages, seq_len : [max_seqs] i32
 //   state          : {free_top, error word, n_touch, n_cow}
 // The allocator reproduces the sequential semantics of the reference's LIFO block manager
@@ -411,10 +412,12 @@ __global__ void gather_kernel(KvDev d, int layer, int seq, void* k_out, void* v_
   const int len = min(d.seq_len[seq], cap_rows);
   const KvLayerDev L = d.layer[layer];
   for (int is_v = 0; is_v < 2; ++is_v) {
-    const int D = is_v ? L.value_dim : L.key_dim, W = is_v ? L.vd : L.kd;
+    const int D = is_v ? L.value_dim : L.key_dim;
+    int W = is_v ? L.vd : L.kd;
     const char* pool = is_v ? (const char*)d.v_pool + L.v_off : (const char*)d.k_pool + L.k_off;
     const float* scales = is_v ? d.v_scale : d.k_scale;
     void* out = is_v ? v_out : k_out;
+    if (is_v && L.values_in_keys) { W = L.kd; pool = (const char*)d.k_pool + L.k_off; }
     const size_t total = (size_t)len * L.heads * D;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
       const int c = i % D, h = (i / D) % L.heads, t = i / ((size_t)D * L.heads);
@@ -534,7 +537,20 @@ static b200_status run_admin(b200_kv* kv, int op, int a0, int a1, int a2, const 
   return out[0];
 }
 
+// Recurrent state of one slot to another slot (the same pool or one of the same shape).
+static b200_status copy_state(b200_kv* dst_kv, int dst, const b200_kv* src_kv, int src) {
+  for (size_t l = 0; l < dst_kv->lay.size(); ++l) {
+    const KvLayerDev &D = dst_kv->lay[l], &S = src_kv->lay[l];
+    if (D.rec_elems > 0)
+      B200_CUDA_TRY(cudaMemcpy(dst_kv->dev.rec_pool + D.rec_off + (size_t)dst * D.rec_elems, src_kv->dev.rec_pool + S.rec_off + (size_t)src * S.rec_elems,
+                               sizeof(float) * D.rec_elems, cudaMemcpyDeviceToDevice));
+  }
+  return B200_OK;
+}
+
 extern "C" {
+
+uint64_t b200_kv_state_bytes(const b200_kv* kv) { return kv->rec_slot_bytes; }
 
 static b200_status kv_create(const b200_kv_config* c, const b200_kv_layer* layers, b200_kv** out);
 
@@ -567,7 +583,10 @@ static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* la
     cfg.n_kv_heads = 1;
     cfg.head_dim = 0;
     for (int l = 0; l < cfg.n_layers; ++l) {
-      if (layers[l].n_kv_heads <= 0 || layers[l].key_dim <= 0 || layers[l].value_dim <= 0) {
+      const b200_kv_layer& y = layers[l];
+      const bool pages = y.n_kv_heads > 0 && y.key_dim > 0 && y.value_dim > 0 && (!y.values_in_keys || y.value_dim <= y.key_dim);
+      const bool none = y.n_kv_heads == 0 && y.key_dim == 0 && y.value_dim == 0 && y.state_elems > 0;
+      if ((!pages && !none) || y.state_elems < 0) {
         b200_set_error("kv_create_layers: layer %d has no shape", l);
         return B200_ERR_INVALID_ARGUMENT;
       }
@@ -594,19 +613,24 @@ static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* la
   // width), so a token row is a whole number of 32-byte sectors and a TMA-addressable stride.
   kv->layered = layers != nullptr;
   kv->lay.resize(c->n_layers);
-  size_t k_bytes = 0, v_bytes = 0;
+  size_t k_bytes = 0, v_bytes = 0, rec_elems = 0;
   for (int l = 0; l < c->n_layers; ++l) {
     KvLayerDev& L = kv->lay[l];
     L.heads = layers ? layers[l].n_kv_heads : c->n_kv_heads;
     L.key_dim = layers ? layers[l].key_dim : c->head_dim;
     L.value_dim = layers ? layers[l].value_dim : c->head_dim;
     L.kd = layers ? (L.key_dim + 15) / 16 * 16 : L.key_dim;
-    L.vd = layers ? (L.value_dim + 15) / 16 * 16 : L.value_dim;
+    L.values_in_keys = layers ? layers[l].values_in_keys : 0;
+    L.vd = layers ? (L.values_in_keys ? 0 : (L.value_dim + 15) / 16 * 16) : L.value_dim;
+    L.rec_elems = layers ? layers[l].state_elems : 0;
+    L.rec_off = rec_elems = (rec_elems + 31) / 32 * 32;
+    rec_elems += (size_t)c->max_seqs * L.rec_elems;
+    kv->rec_slot_bytes += sizeof(float) * (uint64_t)L.rec_elems;
     L.k_off = k_bytes;
     L.v_off = v_bytes;
     k_bytes += (size_t)c->n_pages * L.heads * c->page_size * L.kd * d.elem_bytes;
     v_bytes += (size_t)c->n_pages * L.heads * c->page_size * L.vd * d.elem_bytes;
-    kv->max_vd = std::max(kv->max_vd, L.vd);
+    kv->max_vd = std::max(kv->max_vd, L.values_in_keys ? (L.value_dim + 15) / 16 * 16 : L.vd);
   }
   size_t n_tiles = (size_t)c->n_layers * c->n_pages * c->n_kv_heads;
 #define KV_ALLOC(ptr, bytes)                                            \
@@ -618,8 +642,9 @@ static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* la
       return B200_ERR_CUDA;                                             \
     }                                                                   \
   } while (0)
-  KV_ALLOC(d.k_pool, k_bytes);
-  KV_ALLOC(d.v_pool, v_bytes);
+  KV_ALLOC(d.k_pool, std::max<size_t>(k_bytes, 16));
+  KV_ALLOC(d.v_pool, std::max<size_t>(v_bytes, 16));
+  if (rec_elems > 0) KV_ALLOC(d.rec_pool, sizeof(float) * rec_elems);
   KV_ALLOC(d.layer, sizeof(KvLayerDev) * c->n_layers);
   cudaMemcpy(const_cast<KvLayerDev*>(d.layer), kv->lay.data(), sizeof(KvLayerDev) * c->n_layers, cudaMemcpyHostToDevice);
   if (d.elem_bytes == 1) {
@@ -642,7 +667,7 @@ static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* la
   kv->max_chunks = c->attn_scratch_chunks > 0 ? c->attn_scratch_chunks : c->n_pages / 4 + c->max_rows + 8;
   KV_ALLOC(kv->d_chunk_start, sizeof(int) * (c->max_rows + 2));
   KV_ALLOC(kv->d_groups, sizeof(int) * 3 * (c->max_rows + 2));
-  KV_ALLOC(kv->d_part_o, sizeof(float) * (size_t)kv->max_chunks * c->n_q_heads * kv->max_vd);
+  KV_ALLOC(kv->d_part_o, sizeof(float) * (size_t)kv->max_chunks * c->n_q_heads * std::max(kv->max_vd, 1));
   KV_ALLOC(kv->d_part_ml, sizeof(float) * (size_t)kv->max_chunks * c->n_q_heads * 2);
 #undef KV_ALLOC
   cudaMemset(d.block_table, 0, sizeof(int) * (size_t)c->max_seqs * c->max_pages_per_seq);
@@ -650,17 +675,19 @@ static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* la
   // masked slots by a zero weight instead of branching around them.
   cudaMemset(d.k_pool, 0, k_bytes);
   cudaMemset(d.v_pool, 0, v_bytes);
+  if (rec_elems > 0) cudaMemset(d.rec_pool, 0, sizeof(float) * rec_elems);
   if (layers && d.elem_bytes == 2) {
     kv->lay_kmap.resize(c->n_layers);
     kv->lay_vmap.resize(c->n_layers);
     const uint32_t box[2] = {64, 32};
     for (int l = 0; l < c->n_layers && st == B200_OK; ++l) {
       const KvLayerDev& L = kv->lay[l];
+      if (L.heads == 0) continue;
       const uint64_t rows = (uint64_t)c->n_pages * L.heads * c->page_size;
       const uint64_t kdims[2] = {(uint64_t)L.kd, rows}, vdims[2] = {(uint64_t)L.vd, rows};
       const uint64_t kst[1] = {(uint64_t)L.kd * 2}, vst[1] = {(uint64_t)L.vd * 2};
       st = b200_make_tensor_map(&kv->lay_kmap[l], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (char*)d.k_pool + L.k_off, kdims, kst, box);
-      if (st == B200_OK) st = b200_make_tensor_map(&kv->lay_vmap[l], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (char*)d.v_pool + L.v_off, vdims, vst, box);
+      if (st == B200_OK && L.vd > 0) st = b200_make_tensor_map(&kv->lay_vmap[l], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (char*)d.v_pool + L.v_off, vdims, vst, box);
     }
     if (st != B200_OK) { b200_kv_destroy(kv); return st; }
   } else if (!layers && d.elem_bytes == 2) {
@@ -690,7 +717,7 @@ static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* la
 void b200_kv_destroy(b200_kv* kv) {
   if (!kv) return;
   KvDev& d = kv->dev;
-  void* ptrs[] = {d.k_pool, d.v_pool, d.k_scale, d.v_scale, d.free_stack, d.ref_count, d.tokens_used, d.block_table,
+  void* ptrs[] = {d.k_pool, d.v_pool, d.rec_pool, d.k_scale, d.v_scale, d.free_stack, d.ref_count, d.tokens_used, d.block_table,
                   d.seq_pages, d.seq_len, d.state, d.touch_list, d.cow_list, kv->d_admin_in, kv->d_admin_out,
                   kv->d_chunk_start, kv->d_part_o, kv->d_part_ml, kv->d_groups, const_cast<KvLayerDev*>(d.layer)};
   for (void* p : ptrs) if (p) cudaFree(p);
@@ -737,12 +764,27 @@ b200_status b200_kv_release(b200_kv* kv, const int32_t* seqs, int32_t n) {
   return run_admin(kv, OP_RELEASE, n, 0, 0, seqs, n, nullptr, 0);
 }
 b200_status b200_kv_fork(b200_kv* kv, int32_t src, int32_t dst, int32_t n_tokens) {
+  if (kv->rec_slot_bytes > 0 && n_tokens > 0) {
+    int32_t len = 0;
+    b200_status st = b200_kv_seq_len(kv, src, &len);
+    if (st != B200_OK) return st;
+    if (n_tokens != len) { b200_set_error("fork: recurrent state exists for all %d tokens of the sequence, not for the first %d", len, n_tokens); return B200_ERR_UNSUPPORTED; }
+    st = run_admin(kv, OP_FORK, src, dst, n_tokens, nullptr, 0, nullptr, 0);
+    return st == B200_OK ? copy_state(kv, dst, kv, src) : st;
+  }
   return run_admin(kv, OP_FORK, src, dst, n_tokens, nullptr, 0, nullptr, 0);
 }
 b200_status b200_kv_set_len(b200_kv* kv, int32_t seq, int32_t n_tokens) {
+  if (kv->rec_slot_bytes > 0) { b200_set_error("set_len: the recurrent state of restored tokens is not in the pages"); return B200_ERR_UNSUPPORTED; }
   return run_admin(kv, OP_SET_LEN, seq, n_tokens, 0, nullptr, 0, nullptr, 0);
 }
 b200_status b200_kv_rollback(b200_kv* kv, int32_t seq, int32_t to_len) {
+  if (kv->rec_slot_bytes > 0 && to_len > 0) {
+    int32_t len = 0;
+    b200_status st = b200_kv_seq_len(kv, seq, &len);
+    if (st != B200_OK) return st;
+    if (to_len < len) { b200_set_error("rollback: recurrent state cannot go back from %d to %d tokens", len, to_len); return B200_ERR_UNSUPPORTED; }
+  }
   return run_admin(kv, OP_ROLLBACK, seq, to_len, 0, nullptr, 0, nullptr, 0);
 }
 b200_status b200_kv_filter(b200_kv* kv, const int32_t* keep, int32_t n_keep) {
@@ -1015,7 +1057,8 @@ b200_status b200_kv_extend(b200_kv* kv, int32_t dst_seq, b200_kv* src, int32_t s
     return B200_ERR_INVALID_ARGUMENT;
   }
   for (int l = 0; l < a.n_layers; ++l) {
-    if (kv->lay[l].heads != src->lay[l].heads || kv->lay[l].kd != src->lay[l].kd || kv->lay[l].vd != src->lay[l].vd) {
+    if (kv->lay[l].heads != src->lay[l].heads || kv->lay[l].kd != src->lay[l].kd || kv->lay[l].vd != src->lay[l].vd ||
+        kv->lay[l].values_in_keys != src->lay[l].values_in_keys || kv->lay[l].rec_elems != src->lay[l].rec_elems) {
       b200_set_error("extend: the two pools differ in the shape of layer %d", l);
       return B200_ERR_INVALID_ARGUMENT;
     }
@@ -1049,7 +1092,8 @@ b200_status b200_kv_extend(b200_kv* kv, int32_t dst_seq, b200_kv* src, int32_t s
   if (e == cudaSuccess) e = cudaDeviceSynchronize();
   cudaFree(d_ids);
   if (e != cudaSuccess) { b200_set_error("extend: %s", cudaGetErrorString(e)); return B200_ERR_CUDA; }
-  return b200_kv_set_len(kv, dst_seq, src_len);
+  if ((st = copy_state(kv, dst_seq, src, src_seq)) != B200_OK) return st;
+  return run_admin(kv, OP_SET_LEN, dst_seq, src_len, 0, nullptr, 0, nullptr, 0);
 }
 
 b200_status b200_kv_page_raw(b200_kv* kv, int32_t layer, int32_t page, void* h_k, void* h_v, float* h_k_scales,

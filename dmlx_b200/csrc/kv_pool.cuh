@@ -16,12 +16,16 @@ enum { ST_FREE_TOP = 0, ST_ERR = 1, ST_N_TOUCH = 2, ST_N_COW = 3, ST_ATTN_ERR = 
 struct KvLayerDev {
   size_t k_off = 0, v_off = 0;  // bytes from the start of k_pool / v_pool
   int heads = 0, kd = 0, vd = 0, key_dim = 0, value_dim = 0;
+  int values_in_keys = 0;  // the values are the first value_dim columns of the key rows (vd = 0)
+  int rec_elems = 0;       // f32 elements of recurrent state per sequence slot ...
+  size_t rec_off = 0;      // ... and where the layer's [max_seqs][rec_elems] start in rec_pool, in elements
 };
 
 // Plain-old-data view of the pool, passed to kernels by value.
 struct KvDev {
   void* k_pool = nullptr;
   void* v_pool = nullptr;
+  float* rec_pool = nullptr;  // recurrent state, [layer][slot][elements]
   float* k_scale = nullptr;
   float* v_scale = nullptr;
   int* free_stack = nullptr;
@@ -53,6 +57,7 @@ struct b200_kv {
   std::vector<CUtensorMap> lay_kmap, lay_vmap;  // per-layer 2-D maps (layered bf16 pools): [page*kv_head*32 rows][width]
   std::vector<WindowPlan*> plans;
   bool layered = false;
+  uint64_t rec_slot_bytes = 0;        // recurrent state of one slot, all layers
   int max_vd = 0;                     // widest stored value row (sizes the split-K scratch)
   int* d_admin_in = nullptr;
   int* d_admin_out = nullptr;

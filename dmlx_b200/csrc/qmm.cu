@@ -105,9 +105,9 @@ __device__ __forceinline__ void finish_store(const QmmArgs& a, int token, int n,
       u0 = fminf(fmaxf(u0, -L), L); u1 = fminf(fmaxf(u1, -L), L);
     }
     const float y0 = g0 / (1.0f + __expf(-g0)) * u0 * rs, y1 = g1 / (1.0f + __expf(-g1)) * u1 * rs;
-    *reinterpret_cast<__nv_bfloat162*>(a.y + (size_t)a.row_base_out(token) * (a.n / 2) + n / 2) = __floats2bfloat162_rn(y0, y1);
+    *reinterpret_cast<__nv_bfloat162*>(a.y + (size_t)a.row_base_out(token) * a.out_stride(a.n / 2) + n / 2) = __floats2bfloat162_rn(y0, y1);
   } else {
-    const size_t o = (size_t)a.row_base_out(token) * a.n + n;
+    const size_t o = (size_t)a.row_base_out(token) * a.out_stride(a.n) + n;
     if (a.epilogue == B200_EPI_RESIDUAL) {
       const uint2 rv = *reinterpret_cast<const uint2*>(a.residual + o);
       acc.x += ptx::bf16_lo(rv.x); acc.y += ptx::bf16_hi(rv.x); acc.z += ptx::bf16_lo(rv.y); acc.w += ptx::bf16_hi(rv.y);
@@ -325,8 +325,17 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
   const int nt = blockIdx.x, split = blockIdx.y;
   // Dense: blockIdx.z is a token tile.  Grouped: blockIdx.z is a work item {expert, first row,
   // rows} of the expert-sorted batch; unused items leave before touching any barrier.
-  int t0 = blockIdx.z * tn, rows_here = min(tn, a.rows - t0);
+  // Block-diagonal: blockIdx.z is (matrix, token tile).
+  int t0 = blockIdx.z * tn, x_col = 0, y_col = 0;
   const unsigned char* blocks = a.blocks;
+  if (a.groups > 0) {
+    const int tts = gridDim.z / a.groups, e = blockIdx.z / tts;
+    t0 = ((int)blockIdx.z - e * tts) * tn;
+    blocks += (size_t)e * a.expert_stride;
+    x_col = e * a.x_group;
+    y_col = e * a.y_group;
+  }
+  int rows_here = min(tn, a.rows - t0);
   if (a.items) {
     if ((int)blockIdx.z >= *a.n_items) return;
     const int4 it = a.items[blockIdx.z];
@@ -375,7 +384,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
         // dense bf16 blocks are stored in the swizzled K-major layout and land in the MMA tile directly
         ptx::bulk_g2s(MODE == B200_Q_BF16 ? a_tile(s) : raw_blk(s), blocks + ((size_t)nt * a.kc + kc0 + i) * BB, BB,
                       &loaded[s]);
-        ptx::tma_load_2d(x_tile(s), &xmap, (kc0 + i) * kChunkK, a.x_row0 + t0, &loaded[s]);
+        ptx::tma_load_2d(x_tile(s), &xmap, x_col + (kc0 + i) * kChunkK, a.x_row0 + t0, &loaded[s]);
       }
     }
   } else if (warp == 9) {
@@ -429,7 +438,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
       const int n = nt * kTileN + warp * 32 + lane;
       // One K split and a small token tile: apply the epilogue here and skip the finish kernel.  With
       // large token tiles the strided 64-byte row stores cost more than the extra pass.
-      const bool direct = gridDim.y == 1 && tn <= 64 && !a.keep_f32;
+      // (Dense weights in groups: their tiles are never split, and the pass would move the whole output twice more.)
+      const bool direct = gridDim.y == 1 && !a.keep_f32 && (tn <= 64 || (MODE == B200_Q_BF16 && (a.items || a.groups > 0)));
       const size_t n_pad = a.items ? (size_t)a.nt * kTileN : (size_t)kTileN;  // stride between token rows
       float* wsp = a.items ? a.ws + ((size_t)split * a.rows + t0) * n_pad + n
                            : a.ws + (((size_t)(nt * gridDim.z + blockIdx.z) * gridDim.y + split) * tn) * kTileN + warp * 32 + lane;
@@ -451,7 +461,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
               float g = mine, u = other;
               if (a.swiglu_limit > 0.f) { g = fminf(g, a.swiglu_limit); u = fminf(fmaxf(u, -a.swiglu_limit), a.swiglu_limit); }
               const int token = t0 + c0 + j;
-              a.y[(size_t)token * (a.n / 2) + n / 2] = __float2bfloat16(g / (1.0f + __expf(-g)) * u * a.row_scale(token));
+              a.y[(size_t)token * a.out_stride(a.n / 2) + n / 2] = __float2bfloat16(g / (1.0f + __expf(-g)) * u * a.row_scale(token));
             }
           }
         } else {
@@ -459,7 +469,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
           for (int j = 0; j < 32; ++j) {
             if (c0 + j < rows_here && n < a.n) {
               const int token = t0 + c0 + j;
-              const size_t o = (size_t)token * a.n + n;
+              const size_t o = (size_t)token * a.out_stride(a.n) + y_col + n;
               float acc = __uint_as_float(v[j]);
               if (a.epilogue == B200_EPI_RESIDUAL) acc += __bfloat162float(a.residual[o]);
               a.y[o] = __float2bfloat16(acc * a.row_scale(token));
@@ -497,7 +507,7 @@ __device__ __forceinline__ void tile_epilogue_store(const QmmArgs& a, const uint
         float g = odd ? got : a0, u = odd ? a1 : got;
         if (L > 0.f) { g = fminf(g, L); u = fminf(fmaxf(u, -L), L); }
         const int token = t0 + tok;
-        a.y[(size_t)token * (a.n / 2) + n / 2] = __float2bfloat16(g / (1.0f + __expf(-g)) * u * a.row_scale(token));
+        a.y[(size_t)token * a.out_stride(a.n / 2) + n / 2] = __float2bfloat16(g / (1.0f + __expf(-g)) * u * a.row_scale(token));
       }
     }
   } else {
@@ -505,7 +515,7 @@ __device__ __forceinline__ void tile_epilogue_store(const QmmArgs& a, const uint
     for (int j = 0; j < 32; ++j) {
       if (c0 + j < rows_here && n < a.n) {
         const int token = t0 + c0 + j;
-        const size_t o = (size_t)token * a.n + n;
+        const size_t o = (size_t)token * a.out_stride(a.n) + n;
         float acc = __uint_as_float(v[j]);
         if (a.epilogue == B200_EPI_RESIDUAL) acc += __bfloat162float(a.residual[o]);
         a.y[o] = __float2bfloat16(acc * a.row_scale(token));
@@ -953,7 +963,7 @@ __global__ void __launch_bounds__(kTc2Threads, 1) qmm_tc2_kernel(const __grid_co
           const int tok = idx >> 4, c16 = idx & 15, tile = c16 >> 3;
           const int col = (nt0 + tile) * 64 + (c16 & 7) * 8;
           if (tile < n_tiles && col < n_out)
-            *reinterpret_cast<uint4*>(a.y + (size_t)(t0 + tok) * n_out + col) = *reinterpret_cast<const uint4*>(stage_h + (size_t)idx * 8);
+            *reinterpret_cast<uint4*>(a.y + (size_t)(t0 + tok) * a.out_stride(n_out) + col) = *reinterpret_cast<const uint4*>(stage_h + (size_t)idx * 8);
         }
       }
     } else if (ok && etile < n_tiles) {
@@ -2315,13 +2325,14 @@ static b200_status launch_simt(QmmArgs& a, int rows, cudaStream_t s) {
 }
 
 template <int MODE>
-static b200_status launch_tc(QmmArgs& a, int rows, cudaStream_t s) {
+static b200_status launch_tc(QmmArgs& a, int rows, cudaStream_t s, int x_stride = 0) {
   // grouped launches fix the token tile (an expert's rows are cut into tiles of a.tn); dense ones
   // take the whole batch up to 256 rows per tile
   const int tn = a.items ? a.tn : std::min(256, ((rows + 15) / 16) * 16);
   a.tn = tn;
   const int tts = (rows + tn - 1) / tn;
   const int tiles = a.items ? a.nt * a.max_items : a.nt * tts;
+  const bool grouped_bf16 = MODE == B200_Q_BF16 && (a.items || a.groups > 0);
   b200_status st = ensure_state(0);
   if (st != B200_OK) return st;
   constexpr int kRaw = MODE == B200_Q_BF16 ? 0 : ((block_bytes(MODE) + 127) / 128) * 128;
@@ -2349,18 +2360,19 @@ static b200_status launch_tc(QmmArgs& a, int rows, cudaStream_t s) {
     return B200_ERR_CAPACITY;
   }
   // A CTA pays its first load (about 2.3 us measured), set-up and epilogue once: about 12 chunks' worth.
-  const int splits0 = a.items ? 1 : pick_splits(tiles, a.kc, g_sms, ctas_per_sm, 12);
+  const int splits0 = a.items || a.groups > 0 ? 1 : pick_splits(tiles, a.kc, g_sms, ctas_per_sm, 12);
   a.chunks_per_split = (a.kc + splits0 - 1) / splits0;
   const int splits = (a.kc + a.chunks_per_split - 1) / a.chunks_per_split;
-  st = ensure_state((size_t)splits * (a.items ? (size_t)rows : (size_t)tts * tn) * a.nt * kTileN * sizeof(float));
+  st = ensure_state(grouped_bf16 ? 0 : (size_t)splits * (a.items ? (size_t)rows : (size_t)tts * tn) * a.nt * kTileN * sizeof(float));
   if (st != B200_OK) return st;
   a.ws = g_ws; a.err = g_err;
   CUtensorMap xmap;
-  st = make_x_map(&xmap, a.x, rows, a.k, tn);
+  st = make_x_map(&xmap, a.x, rows, x_stride > 0 ? x_stride : a.k, tn);
   if (st != B200_OK) return st;
   a.x_row0 = 0;
-  qmm_tc_kernel<MODE><<<dim3(a.nt, splits, a.items ? a.max_items : tts), kTcThreads, smem, s>>>(xmap, a);
+  qmm_tc_kernel<MODE><<<dim3(a.nt, splits, a.items ? a.max_items : tts * std::max(a.groups, 1)), kTcThreads, smem, s>>>(xmap, a);
   B200_LAUNCH_CHECK();
+  if (grouped_bf16) return B200_OK;
   return (splits == 1 && tn <= 64 && !a.keep_f32) ? B200_OK : launch_finish(a, splits, s);  // a single small split writes its output itself
 }
 
@@ -2734,6 +2746,7 @@ extern "C" b200_status b200_qmm(const b200_qweight* w, const void* d_x, int32_t 
 
 // Set by b200_qmm_deferred around its call of qmm_entry (one calling thread per process uses the matmul entry points).
 static b200_qmm_partials* g_defer_target = nullptr;
+static int g_y_stride = 0;         // set by b200_qmm_to around its call
 static bool g_defer_always = false;  // defer = 2: also when K is not split
 
 extern "C" b200_status b200_qmm_deferred(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t defer, void* stream,
@@ -2745,6 +2758,14 @@ extern "C" b200_status b200_qmm_deferred(const b200_qweight* w, const void* d_x,
   const b200_status st = qmm_entry(w, d_x, rows, d_y, B200_EPI_NONE, nullptr, 0.f, B200_QMM_AUTO, stream, nullptr, 0.f, nullptr, nullptr);
   g_defer_target = nullptr;
   g_defer_always = false;
+  return st;
+}
+
+b200_status b200_qmm_to(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t y_stride, int32_t epilogue, void* stream) {
+  if (w->mode != B200_Q_BF16 || epilogue == B200_EPI_RESIDUAL || y_stride % 8 != 0) { b200_set_error("qmm_to: dense bf16 weights, no residual, output rows of 16-byte multiples"); return B200_ERR_INVALID_ARGUMENT; }
+  g_y_stride = y_stride;
+  const b200_status st = qmm_entry(w, d_x, rows, d_y, epilogue, nullptr, 0.f, B200_QMM_AUTO, stream, nullptr, 0.f, nullptr, nullptr);
+  g_y_stride = 0;
   return st;
 }
 
@@ -2816,6 +2837,7 @@ static b200_status qmm_entry(const b200_qweight* w, const void* d_x, int32_t row
   a.rows = rows; a.n = w->n; a.k = w->k; a.nt = w->nt; a.kc = w->kc; a.epilogue = epilogue; a.swiglu_limit = swiglu_limit;
   a.norm_w = (const __nv_bfloat16*)d_norm_w; a.norm_out = (__nv_bfloat16*)d_norm_out; a.norm_eps = norm_eps;
   a.defer = g_defer_target;
+  a.y_stride = g_y_stride;
   a.keep_f32 = g_defer_always ? 1 : 0;
   cudaStream_t s = (cudaStream_t)stream;
   auto dispatch = [&]() -> b200_status {
@@ -2853,11 +2875,33 @@ static b200_status qmm_entry(const b200_qweight* w, const void* d_x, int32_t row
 namespace {
 constexpr int kF32Rows = 64, kF32K = 32;
 
-__global__ void __launch_bounds__(256) qmm_f32_kernel(const unsigned char* __restrict__ blocks, const float* __restrict__ x, int rows, int k, int kc,
-                                                      float* __restrict__ y, int y_stride, int n_valid, int swiglu) {
+struct F32Args {
+  const unsigned char* blocks;
+  const float* x;
+  float* y;
+  int rows, kc, x_stride, y_stride, n_valid, swiglu;
+  size_t expert_stride;        // bytes between the matrices of a stack
+  int x_group, y_group;        // block-diagonal: columns of x and y per matrix (grid z)
+  const int4* items;           // grouped: {matrix, first sorted row, rows} (grid y)
+  const int *n_items, *order;  // order: sorted row -> assignment, of which order_div share a row of x
+  int order_div;
+};
+
+__global__ void __launch_bounds__(256) qmm_f32_kernel(F32Args a) {
   __shared__ float xs[kF32K][kF32Rows + 4];
   __shared__ float ws[kF32K][kTileN + 4];
-  const int nt = blockIdx.x, r0 = blockIdx.y * kF32Rows, tid = threadIdx.x;
+  const int nt = blockIdx.x, tid = threadIdx.x, kc = a.kc, n_valid = a.n_valid, y_stride = a.y_stride, swiglu = a.swiglu;
+  int r0 = blockIdx.y * kF32Rows, rows = a.rows;
+  const unsigned char* blocks = a.blocks + (size_t)blockIdx.z * a.expert_stride;
+  const float* x = a.x + (size_t)blockIdx.z * a.x_group;
+  float* y = a.y + (size_t)blockIdx.z * a.y_group;
+  if (a.items) {
+    if ((int)blockIdx.y >= *a.n_items) return;
+    const int4 it = a.items[blockIdx.y];
+    blocks += (size_t)it.x * a.expert_stride;
+    r0 = it.y;
+    rows = it.y + it.z;
+  }
   const int tr = (tid / 32) * 8, tc = (tid % 32) * 4;
   float acc[8][4];
 #pragma unroll
@@ -2878,7 +2922,10 @@ __global__ void __launch_bounds__(256) qmm_f32_kernel(const unsigned char* __res
       for (int i = tid; i < kF32Rows * (kF32K / 4); i += 256) {
         const int r = i / (kF32K / 4), q = i % (kF32K / 4);
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r0 + r < rows) v = *reinterpret_cast<const float4*>(x + (size_t)(r0 + r) * k + c * kChunkK + half * kF32K + q * 4);
+        if (r0 + r < rows) {
+          const int src = a.order ? a.order[r0 + r] / a.order_div : r0 + r;
+          v = *reinterpret_cast<const float4*>(x + (size_t)src * a.x_stride + c * kChunkK + half * kF32K + q * 4);
+        }
         xs[q * 4][r] = v.x; xs[q * 4 + 1][r] = v.y; xs[q * 4 + 2][r] = v.z; xs[q * 4 + 3][r] = v.w;
       }
       __syncthreads();
@@ -2930,10 +2977,56 @@ extern "C" b200_status b200_qmm_f32(const b200_qweight* w, const float* d_x, int
     return B200_ERR_INVALID_ARGUMENT;
   }
   if (rows <= 0) return B200_OK;
-  qmm_f32_kernel<<<dim3(w->nt, (rows + kF32Rows - 1) / kF32Rows), 256, 0, (cudaStream_t)stream>>>(w->d_blocks, d_x, rows, w->k, w->kc, d_y, y_stride,
-                                                                                                n_valid, swiglu ? 1 : 0);
+  F32Args a{};
+  a.blocks = w->d_blocks; a.x = d_x; a.y = d_y; a.rows = rows; a.kc = w->kc; a.x_stride = w->k; a.y_stride = y_stride; a.n_valid = n_valid;
+  a.swiglu = swiglu ? 1 : 0;
+  qmm_f32_kernel<<<dim3(w->nt, (rows + kF32Rows - 1) / kF32Rows), 256, 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
+}
+
+b200_status b200_qmm_f32_blocks(const b200_qweight* w, const float* d_x, int32_t x_stride, int32_t x_group, int32_t rows, float* d_y,
+                                int32_t y_stride, int32_t y_group, void* stream) {
+  b200_status st = b200_require_device();
+  if (st != B200_OK) return st;
+  if (w->mode != B200_Q_BF16 || x_group < w->k || x_stride % 4 != 0 || x_group % 4 != 0) { b200_set_error("qmm_f32_blocks: dense bf16 blocks, strides of 16 bytes"); return B200_ERR_INVALID_ARGUMENT; }
+  if (rows <= 0) return B200_OK;
+  F32Args a{};
+  a.blocks = w->d_blocks; a.x = d_x; a.y = d_y; a.rows = rows; a.kc = w->kc; a.x_stride = x_stride; a.y_stride = y_stride; a.n_valid = w->n;
+  a.expert_stride = (size_t)w->nt * w->kc * w->block_bytes; a.x_group = x_group; a.y_group = y_group;
+  qmm_f32_kernel<<<dim3(w->nt, (rows + kF32Rows - 1) / kF32Rows, w->n_experts), 256, 0, (cudaStream_t)stream>>>(a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+b200_status b200_qmm_f32_grouped(const b200_qweight* w, const float* d_x, const int* d_order, int32_t order_div, float* d_y, int32_t y_stride,
+                                 int32_t epilogue, const int4* d_items, const int* d_n_items, int32_t max_items, void* stream) {
+  b200_status st = b200_require_device();
+  if (st != B200_OK) return st;
+  const bool swiglu = epilogue == B200_EPI_SWIGLU;
+  if (w->mode != B200_Q_BF16 || (epilogue != B200_EPI_NONE && !swiglu)) { b200_set_error("qmm_f32_grouped: dense bf16 weights, no or the SwiGLU epilogue"); return B200_ERR_UNSUPPORTED; }
+  if (max_items <= 0) return B200_OK;
+  F32Args a{};
+  a.blocks = w->d_blocks; a.x = d_x; a.y = d_y; a.kc = w->kc; a.x_stride = w->k; a.y_stride = y_stride; a.n_valid = swiglu ? w->n / 2 : w->n;
+  a.swiglu = swiglu ? 1 : 0; a.expert_stride = (size_t)w->nt * w->kc * w->block_bytes;
+  a.items = d_items; a.n_items = d_n_items; a.order = d_order; a.order_div = order_div > 0 ? order_div : 1;
+  qmm_f32_kernel<<<dim3(w->nt, max_items), 256, 0, (cudaStream_t)stream>>>(a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+b200_status b200_qmm_blocks(const b200_qweight* w, const void* d_x, int32_t x_stride, int32_t x_group, int32_t rows, void* d_y, int32_t y_stride,
+                            int32_t y_group, void* stream) {
+  b200_status st = b200_require_device();
+  if (st != B200_OK) return st;
+  if (w->mode != B200_Q_BF16 || x_group < w->k || x_stride % 8 != 0 || x_group % 8 != 0) { b200_set_error("qmm_blocks: dense bf16 blocks, strides of 16 bytes"); return B200_ERR_INVALID_ARGUMENT; }
+  if (rows <= 0) return B200_OK;
+  QmmArgs a{};
+  a.blocks = w->d_blocks; a.x = (const __nv_bfloat16*)d_x; a.y = (__nv_bfloat16*)d_y;
+  a.rows = rows; a.n = w->n; a.k = w->k; a.nt = w->nt; a.kc = w->kc; a.epilogue = B200_EPI_NONE;
+  a.expert_stride = (size_t)w->nt * w->kc * w->block_bytes;
+  a.groups = w->n_experts; a.x_group = x_group; a.y_group = y_group; a.y_stride = y_stride;
+  return launch_tc<B200_Q_BF16>(a, rows, (cudaStream_t)stream, x_stride);
 }
 
 // Grouped matmul over an expert-sorted batch: work item i = {expert, first row, rows}; every

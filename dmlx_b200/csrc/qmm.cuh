@@ -51,9 +51,13 @@ struct QmmArgs {
   int mx_expert_rows;           // rows of the code matrix per expert (nt * 128)
   int kc128;                    // K / 128
   int did_norm;                 // host only: the finish pass also wrote norm_out
+  int y_stride;                 // elements between output rows (0: exactly the outputs of a row)
+  // block-diagonal launches: matrix e of a stack multiplies columns e * x_group .. of every row and writes columns e * y_group ..
+  int groups, x_group, y_group;
   int keep_f32;                 // the caller wants the f32 sums: no kernel writes bf16 output itself
   b200_qmm_partials* defer = nullptr;  // when set, a dense launch with epilogue NONE leaves its finish pass to the caller
 
+  __device__ __forceinline__ size_t out_stride(int per_row) const { return y_stride > 0 ? y_stride : per_row; }
   __device__ __forceinline__ int row_base_out(int token) const { return token; }
   __device__ __forceinline__ float row_scale(int token) const { return row_scales ? row_scales[token] : 1.0f; }
 };
@@ -61,6 +65,18 @@ struct QmmArgs {
 b200_status b200_qmm_grouped(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t epilogue,
                              const float* d_row_scales, float swiglu_limit, const int4* d_items, const int* d_n_items,
                              int32_t max_items, int32_t tile_rows, void* stream);
+// Dense bf16 weights, rows of the output y_stride elements apart.
+b200_status b200_qmm_to(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t y_stride, int32_t epilogue, void* stream);
+// Block-diagonal matmul: the n_experts matrices [n, k] of w are the blocks (one per attention head, say).
+// y[r][e * y_group + i] = sum_j w_e[i][j] x[r][e * x_group + j]; rows of x are x_stride apart, those of y y_stride.  bf16, f32 accumulation.
+b200_status b200_qmm_blocks(const b200_qweight* w, const void* d_x, int32_t x_stride, int32_t x_group, int32_t rows, void* d_y, int32_t y_stride,
+                            int32_t y_group, void* stream);
+// The f32 forms (f32 activations, dense bf16 weights widened exactly, CUDA cores).  Grouped: rows of x are taken through
+// order (x row order[p] / order_div for sorted row p; null: sorted row p itself), items of at most 64 rows.
+b200_status b200_qmm_f32_blocks(const b200_qweight* w, const float* d_x, int32_t x_stride, int32_t x_group, int32_t rows, float* d_y,
+                                int32_t y_stride, int32_t y_group, void* stream);
+b200_status b200_qmm_f32_grouped(const b200_qweight* w, const float* d_x, const int* d_order, int32_t order_div, float* d_y, int32_t y_stride,
+                                 int32_t epilogue, const int4* d_items, const int* d_n_items, int32_t max_items, void* stream);
 // 1 if b200_qmm_grouped_from_tokens can serve this weight and tile size (block-scaled MXFP4 path).
 int b200_qmm_grouped_takes_tokens(const b200_qweight* w, int32_t tile_rows);
 // The same matmul with the expert-sorted activation rows read from the unsorted token matrix:

@@ -241,7 +241,15 @@ b200_status b200_kv_create(const b200_kv_config* cfg, b200_kv** out);           
  * or f32 pages.  Page tables, reference counts, copy-on-write, fork, rollback, extend and page_raw / page_load work as on
  * any pool (page bytes per layer: [n_kv_heads][32][width rounded up to 16]); rows are written and read by
  * b200_decoder_*. */
-typedef struct b200_kv_layer { int32_t n_kv_heads, key_dim, value_dim; } b200_kv_layer;
+typedef struct b200_kv_layer {
+  int32_t n_kv_heads, key_dim, value_dim; /* all 0: the layer has no pages */
+  int32_t values_in_keys;                 /* 1: the values are the first value_dim columns of the key rows, stored once */
+  int32_t state_elems;                    /* f32 elements of recurrent state per sequence slot (0: none) */
+} b200_kv_layer;
+/* Bytes of recurrent state per sequence slot over all layers.  State belongs to a slot's whole length: a sequence at
+ * position 0 starts from zero whatever the slot held before; fork and extend copy it and take the whole sequence only,
+ * rollback goes to 0 only, and set_len is refused (UNSUPPORTED), since pages alone do not restore a state. */
+uint64_t b200_kv_state_bytes(const b200_kv* kv);
 b200_status b200_kv_create_layers(const b200_kv_config* cfg, const b200_kv_layer* layers, b200_kv** out);
 void b200_kv_destroy(b200_kv* kv);                                               /* :1111-1138 deinit */
 /* Pool size and number of sequence slots of a pool. */
