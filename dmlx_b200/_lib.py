@@ -257,7 +257,7 @@ _sig("b200_ep_watch", i32, P(EpWatchOps), i32, i32)
 
 
 class KvLayer(C.Structure):
-    _fields_ = [(n, i32) for n in ("n_kv_heads", "key_dim", "value_dim")]
+    _fields_ = [(n, i32) for n in ("n_kv_heads", "key_dim", "value_dim", "values_in_keys", "state_elems")]
 
 
 class ModelInfo(C.Structure):
@@ -265,12 +265,14 @@ class ModelInfo(C.Structure):
 
 
 class DecoderLayer(C.Structure):
-    _fields_ = [(n, i32) for n in ("n_heads", "n_kv_heads", "key_dim", "value_dim", "window", "ffn", "flags")] + [("scale", f32)]
+    _fields_ = [(n, i32) for n in ("n_heads", "n_kv_heads", "key_dim", "value_dim", "window", "ffn", "flags")] + [("scale", f32)] + [
+        (n, i32) for n in ("mixer", "kv_rank", "rot_dim")] + [("rot_base", f32), ("decay_rank", i32), ("decay_tau", f32)] + [
+        (n, i32) for n in ("n_experts", "top_k", "expert_ffn")]
 
 
 class DecoderConfig(C.Structure):
     _fields_ = [(n, i32) for n in ("n_layers", "hidden", "vocab", "loop_start", "loop_stop", "loop_times", "dtype", "max_rows", "max_reqs",
-                                   "max_seqs")] + [("norm_eps", f32), ("embed_scale", f32)]
+                                   "max_seqs")] + [("norm_eps", f32), ("embed_scale", f32), ("logit_scale", f32), ("flags", i32)]
 
 
 _sig("b200_kv_create_layers", i32, P(KvConfig), P(KvLayer), P(vp))
@@ -292,7 +294,9 @@ _sig("b200_model_logits", i32, vp, i32, i32, P(f32))
 _sig("b200_decoder_create", i32, P(DecoderConfig), P(DecoderLayer), P(vp))
 _sig("b200_decoder_destroy", None, vp)
 _sig("b200_decoder_set_tensor", i32, vp, i32, i32, vp, u64)
+_sig("b200_decoder_set_table", i32, vp, i32, P(i32), u64)
 _sig("b200_decoder_finalize", i32, vp)
+_sig("b200_kv_state_bytes", u64, vp)
 _sig("b200_decoder_random_init", i32, vp, u32)
 _sig("b200_decoder_cache_layers", i32, vp, P(KvLayer), i32)
 _sig("b200_decoder_record_layers", i32, vp, i32)

@@ -1,0 +1,22 @@
+// Latent attention over one layer of a layered pool whose values lie inside its key rows (attn_latent.cu).
+#pragma once
+#include "kv_pool.cuh"
+#include "rows.cuh"
+
+// Cosine and sine of every row's rotation, [rows][dims / 2]; made once per step for the layers that share base and width.
+b200_status b200_rotation_table(const double* d_freq, int dims, const int32_t* d_pos, int rows, float2* d_out, void* stream);
+
+// From the projection rows [heads x (dim + rot) | rank + rot] to what attention reads: the unrotated query parts ([heads][plain_stride],
+// zero behind dim), the rotated ones (written at column `rank` of every head of q), and the normed latent with the rotated key
+// part in its page.
+struct LatentPrep {
+  int layer = 0, heads = 0, dim = 0, rot = 0, rank = 0;
+  MatSrc src;
+  const float* norm = nullptr;  // [rank]
+  float eps = 0.f;
+  const float2* rotation = nullptr;
+  void* q_plain = nullptr;      // [rows][heads][plain_stride]
+  int plain_stride = 0;
+  void* q = nullptr;            // [rows][heads][stored key width]
+};
+b200_status b200_latent_prep(b200_kv* kv, const LatentPrep& p, const int32_t* d_pos, const int32_t* d_row_seq, int rows, void* stream);

@@ -555,7 +555,7 @@ struct SimtArgs {
   float scale;
   const float *slopes_log2, *sinks_log2;
   void* out;
-  int out_stride;
+  int out_stride, out_head_stride;
 };
 
 // One warp per (row, query head): 32 keys at a time (one per lane) for the scores, value columns over the lanes for the
@@ -577,7 +577,8 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(SimtArgs a) {
   if (seq < 0 || seq >= a.d.max_seqs || (ctx + 31) / 32 > a.d.seq_pages[seq]) return;  // reservation failed: the step is flagged
   const int* table = a.d.block_table + (size_t)seq * a.d.max_pages_per_seq;
   const T* kp = (const T*)((const char*)a.d.k_pool + a.L.k_off);
-  const T* vp = (const T*)((const char*)a.d.v_pool + a.L.v_off);
+  const T* vp = a.L.values_in_keys ? kp : (const T*)((const char*)a.d.v_pool + a.L.v_off);
+  const int v_row = a.L.values_in_keys ? a.L.kd : a.L.vd;
   const float slope = a.slopes_log2 ? a.slopes_log2[qh] : 0.f, scale = a.scale * kLog2e;
   float m = kNone, l = 0.f;
   for (int pg = lo / 32; pg * 32 < ctx; ++pg) {
@@ -606,7 +607,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(SimtArgs a) {
       float acc = c < vd ? o[c] * corr : 0.f;
       for (int k = k0; k < k1; ++k) {
         const float pk = __shfl_sync(0xffffffffu, p, k);
-        if (c < vd) acc = fmaf(pk, to_f(vp[(tile + k) * a.L.vd + c]), acc);
+        if (c < vd) acc = fmaf(pk, to_f(vp[(tile + k) * v_row + c]), acc);
       }
       if (c < vd) o[c] = acc;
     }
@@ -618,7 +619,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(SimtArgs a) {
     f = exp2f(m - mm);
     l = l * f + exp2f(sk - mm);
   }
-  T* out = (T*)a.out + (size_t)row * a.out_stride + (size_t)qh * vd;
+  T* out = (T*)a.out + (size_t)row * a.out_stride + (size_t)qh * a.out_head_stride;
   for (int c = lane; c < vd; c += 32) put(out + c, l > 0.f ? o[c] * f / l : 0.f);
 }
 
@@ -718,7 +719,7 @@ b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
                                  bool mma, void* stream) {
   if (c.layer < 0 || c.layer >= kv->cfg.n_layers || !kv->layered) { b200_set_error("window attention: layer %d of no layered pool", c.layer); return B200_ERR_INVALID_ARGUMENT; }
   const KvLayerDev& L = kv->lay[c.layer];
-  if (c.n_q_heads <= 0 || c.n_q_heads % L.heads != 0) { b200_set_error("window attention: %d query heads over %d kv heads", c.n_q_heads, L.heads); return B200_ERR_INVALID_ARGUMENT; }
+  if (L.heads <= 0 || c.n_q_heads <= 0 || c.n_q_heads % L.heads != 0) { b200_set_error("window attention: %d query heads over %d kv heads", c.n_q_heads, L.heads); return B200_ERR_INVALID_ARGUMENT; }
   if (total_rows <= 0) return B200_OK;
   if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
   b200_status st = sm_count();
@@ -729,7 +730,7 @@ b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
     SimtArgs a;
     a.d = kv->dev; a.L = L; a.q = c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx; a.total_rows = total_rows;
     a.n_q_heads = c.n_q_heads; a.window = c.window; a.scale = c.scale; a.slopes_log2 = c.slopes_log2; a.sinks_log2 = c.sinks_log2;
-    a.out = c.out; a.out_stride = c.out_stride;
+    a.out = c.out; a.out_stride = c.out_stride; a.out_head_stride = c.out_head_stride > 0 ? c.out_head_stride : L.value_dim;
     const size_t smem = sizeof(float) * 4 * (L.key_dim + L.value_dim);
     if (smem > 200 * 1024) { b200_set_error("window attention: head widths %d / %d are too large", L.key_dim, L.value_dim); return B200_ERR_UNSUPPORTED; }
     const unsigned grid = (unsigned)(((long long)total_rows * c.n_q_heads + 3) / 4);
@@ -765,5 +766,5 @@ b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
 }
 
 bool b200_window_attn_takes_mma(const b200_kv* kv, int32_t layer) {
-  return kv->layered && kv->dev.elem_bytes == 2 && kv->lay[layer].kd <= 256 && kv->lay[layer].vd <= 256;
+  return kv->layered && kv->dev.elem_bytes == 2 && !kv->lay[layer].values_in_keys && kv->lay[layer].kd <= 256 && kv->lay[layer].vd <= 256;
 }

@@ -2,10 +2,16 @@
 // which mechanisms it has (b200_decoder_layer); the stack may run a range of layers several times with the same weights, each
 // pass opening with x = W_in [x ; x0].
 //
-// A layer is six launches: q/k/v matmul; decoder_qkv_kernel (split-K finish, biases, per-head norms, q to the attention's
-// operand, k and v straight into their pages); attention (attn_window.cu); o matmul; decoder_rows_kernel (split-K
+// An attention layer is six launches: q/k/v matmul; decoder_qkv_kernel (split-K finish, biases, per-head norms, q to the
+// attention's operand, k and v straight into their pages); attention (attn_window.cu); o matmul; decoder_rows_kernel (split-K
 // finish, post-norm, f32 residual add, and the norm or the [x ; x0] rows the next matmul reads); then the feed-forward's
 // two matmuls around the SwiGLU epilogue and decoder_rows_kernel again.
+//
+// Latent attention: projection; latent_prep_kernel (attn_latent.cu); W_uk per head onto the queries; attention over the latents;
+// W_uv per head.  Gated linear attention: projection; the kernels of gla.cu.  Where mixer and feed-forward run in parallel, the
+// mixer's W_o and the dense feed-forward's W_down are one matmul over the concatenation [mixer output | SwiGLU output], and a
+// single decoder_rows_kernel adds it, gathers the experts' rows, averages over depth and norms for the next layer.  Experts by
+// token id are planned for all layers at the start of the step (moe.cu).
 //
 // The residual, every norm, the biases and the logits are f32; matrix operands are bf16, or f32 with B200_DT_F32 (the same
 // kernels instantiated for float, matmuls through b200_qmm_f32, attention on CUDA cores).
@@ -20,9 +26,12 @@
 #include <map>
 #include <vector>
 
+#include "attn_latent.cuh"
 #include "common.h"
+#include "gla.cuh"
 #include "kv_pool.cuh"
 #include "model_step.cuh"
+#include "moe.cuh"
 #include "qmm.cuh"
 #include "rows.cuh"
 
@@ -50,6 +59,16 @@ struct RowArgs {
   int h_stride = 0;
   void* cat = nullptr;            // [x ; x0] for the loop's input matmul
   int cat_stride = 0;
+  // experts: src also gets moe_w times the sum of the row's moe_k rows of moe_y
+  const void* moe_y = nullptr;
+  const int* moe_rows = nullptr;  // [row * moe_k + j] -> row of moe_y
+  int moe_k = 0, moe_stride = 0;
+  float moe_w = 0.f;
+  // depth average: the result is kept as hist[n_hist], and x becomes sum_j depth[j] hist[j]
+  const float* depth = nullptr;   // null for the embedding, which is kept as it is
+  float* hist = nullptr;
+  size_t hist_stride = 0;
+  int n_hist = 0;
 };
 
 // One CTA per row: sublayer output -> residual stream -> what the next matmul reads.  NQ > 0: a thread keeps its NQ
@@ -94,13 +113,25 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
       put(i, k, v);
       store_vec<VEC>(xr + i * VEC, v);
       if (x0r) store_vec<VEC>(x0r + i * VEC, v);
+      if (a.hist) store_vec<VEC>(a.hist + (size_t)row * a.hidden + i * VEC, v);
     });
   } else {
     float ys = 0.f;
     Vec<VEC> res[NQ > 0 ? NQ : 1];
     each([&](int i, int k) {
       if constexpr (NQ > 0) { if (!a.replace) res[k] = load_vec<VEC>(xr + i * VEC); }
-      const Vec<VEC> v = mat_value<T, VEC>(a.src, row, i * VEC);
+      Vec<VEC> v;
+      if (a.src.ws || a.src.y) {
+        v = mat_value<T, VEC>(a.src, row, i * VEC);
+      } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v.v[j] = 0.f;
+      }
+      for (int m = 0; m < a.moe_k; ++m) {
+        const Vec<VEC> e = load_vec<VEC>((const T*)a.moe_y + (size_t)a.moe_rows[row * a.moe_k + m] * a.moe_stride + i * VEC);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(a.moe_w, e.v[j], v.v[j]);
+      }
 #pragma unroll
       for (int j = 0; j < VEC; ++j) ys += v.v[j] * v.v[j];
       put(i, k, v);
@@ -119,6 +150,20 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
         else x = load_vec<VEC>(xr + i * VEC);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) v.v[j] += x.v[j];
+      }
+      if (a.depth) {
+        float* hr = a.hist + (size_t)row * a.hidden + i * VEC;
+        store_vec<VEC>(hr + a.n_hist * a.hist_stride, v);
+        const float own = a.depth[a.n_hist];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v.v[j] *= own;
+#pragma unroll 4
+        for (int d = 0; d < a.n_hist; ++d) {
+          const Vec<VEC> x = load_vec<VEC>(hr + d * a.hist_stride);
+          const float w = a.depth[d];
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(w, x.v[j], v.v[j]);
+        }
       }
 #pragma unroll
       for (int j = 0; j < VEC; ++j) ss += v.v[j] * v.v[j];
@@ -268,7 +313,9 @@ float bf16_to_f(uint16_t b) {
 }
 
 const char* kTensorNames[] = {"q", "k", "v", "o", "gate", "up", "down", "head", "loop input", "embedding", "q bias", "k bias", "v bias",
-                              "sink", "norm 1", "norm 2", "post-norm 1", "post-norm 2", "final norm"};
+                              "sink", "norm 1", "norm 2", "post-norm 1", "post-norm 2", "final norm", "latent", "latent norm", "key expansion",
+                              "value expansion", "output gate", "decay 1", "decay 2", "decay bias", "head norm", "expert gate", "expert up",
+                              "expert down", "depth weights"};
 
 }  // namespace
 
@@ -276,11 +323,47 @@ struct b200_decoder : b200_model {
   b200_decoder_config cfg{};
   struct Layer {
     b200_decoder_layer s{};
-    b200_qweight *wqkv = nullptr, *wo = nullptr, *wgu = nullptr, *wdown = nullptr;
+    // wqkv: all projections the mixer takes from h.  wo: W_o, in parallel layers [W_o | W_down] over concatenated columns.
+    b200_qweight *wqkv = nullptr, *wo = nullptr, *wgu = nullptr, *wdown = nullptr, *wuk = nullptr, *wuv = nullptr, *we_gu = nullptr, *we_down = nullptr;
     float *bias = nullptr, *sinks = nullptr, *slopes = nullptr, *norm1 = nullptr, *norm2 = nullptr, *post1 = nullptr, *post2 = nullptr;
-    int qkv_n() const { return s.n_heads * s.key_dim + s.n_kv_heads * (s.key_dim + s.value_dim); }
+    float *dkv_norm = nullptr, *a2 = nullptr, *a2_bias = nullptr, *head_norm = nullptr, *depth = nullptr;
+    int* table = nullptr;
+    std::vector<int> h_table;
+    int moe = -1;       // place among the layers with experts
+    int rotation = -1;  // its rotation table
+    int qkv_n() const {
+      if (s.mixer == B200_MIX_LATENT) return s.n_heads * (s.key_dim + s.rot_dim) + s.kv_rank + s.rot_dim;
+      if (s.mixer == B200_MIX_GLA) return 2 * s.n_heads * (s.key_dim + s.value_dim) + s.decay_rank;
+      return s.n_heads * s.key_dim + s.n_kv_heads * (s.key_dim + s.value_dim);
+    }
     int attn_n() const { return s.n_heads * s.value_dim; }
+    bool parallel() const { return (s.flags & B200_DEC_PARALLEL) != 0; }
+    int out_k() const { return pad64(attn_n()) + (parallel() && s.ffn > 0 ? pad64(s.ffn) : 0); }  // columns wo reads
+    int plain_stride() const { return pad64(s.key_dim); }
+    int latent_width() const { return (s.kv_rank + s.rot_dim + 15) / 16 * 16; }
+    std::vector<int> projections() const {
+      if (s.mixer == B200_MIX_LATENT) return {B200_DEC_W_Q, B200_DEC_W_DKV};
+      if (s.mixer == B200_MIX_GLA) return {B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V, B200_DEC_W_OUT_GATE, B200_DEC_W_A1};
+      return {B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V};
+    }
+    b200_kv_layer cache() const {
+      if (s.mixer == B200_MIX_LATENT) return b200_kv_layer{1, s.kv_rank + s.rot_dim, s.kv_rank, 1, 0};
+      if (s.mixer == B200_MIX_GLA) return b200_kv_layer{0, 0, 0, 0, s.n_heads * s.key_dim * s.value_dim};
+      return b200_kv_layer{s.n_kv_heads, s.key_dim, s.value_dim, 0, 0};
+    }
   };
+  // Rotations of a step, one table per (base, width) in the stack.
+  struct Rotation { float base; int dims; double* freq; float2* rows; };
+  std::vector<Rotation> rotations;
+  // Experts by token id: plan buffers of every layer that has them (d_moe: the same on the device), and the rows they work on.
+  std::vector<MoeTableLayer> moe;
+  MoeTableLayer* d_moe = nullptr;
+  std::vector<int> moe_layers;
+  void *moe_x = nullptr, *moe_act = nullptr, *moe_y = nullptr;
+  GlaScratch gla;
+  bool has_gla = false;
+  void *q_plain = nullptr, *lat_out = nullptr;
+  float* hist = nullptr;  // [layers + 1][max_rows][hidden]: embedding output and results of the layers
   std::vector<Layer> layers;
   struct Run { int layer; bool opens; };  // opens: the first layer of a pass of the loop
   std::vector<Run> runs;
@@ -303,16 +386,29 @@ struct b200_decoder : b200_model {
   b200_status matmul(const b200_qweight* w, const void* in, int rows, int defer, MatSrc* src, void* stream);
   b200_status rows_step(RowArgs a, int rows, int next, cudaStream_t s);
   b200_status attention(b200_kv* kv, int run, int rows, void* stream);
+  b200_status mixer(b200_kv* kv, int run, int n_req, int T, void* stream);
+  b200_status experts(const Layer& l, int T, int tile_rows, void* stream);
+  b200_status begin_step(b200_kv* kv, int n_req, int T, int tile_rows, void* stream);
+  int moe_tile_rows(int T) const;
 };
 
 b200_decoder::~b200_decoder() {
-  void* dev[] = {embed, final_norm, x, x0, rec, h, cat, y, q, attn, act, last};
+  void* dev[] = {embed, final_norm, x, x0, rec, h, cat, y, q, attn, act, last, q_plain, lat_out, hist, moe_x, moe_act, moe_y, d_moe};
   for (void* p : dev) if (p) cudaFree(p);
   for (Layer& l : layers) {
-    void* lp[] = {l.bias, l.sinks, l.slopes, l.norm1, l.norm2, l.post1, l.post2};
+    void* lp[] = {l.bias, l.sinks, l.slopes, l.norm1, l.norm2, l.post1, l.post2, l.dkv_norm, l.a2, l.a2_bias, l.head_norm, l.depth, l.table};
     for (void* p : lp) if (p) cudaFree(p);
-    for (b200_qweight* w : {l.wqkv, l.wo, l.wgu, l.wdown}) b200_qweight_destroy(w);
+    for (b200_qweight* w : {l.wqkv, l.wo, l.wgu, l.wdown, l.wuk, l.wuv, l.we_gu, l.we_down}) b200_qweight_destroy(w);
   }
+  for (MoeTableLayer& t : moe) {
+    void* tp[] = {t.indices, t.offsets, t.order, t.inv_order, t.n_items, t.items};
+    for (void* p : tp) if (p) cudaFree(p);
+  }
+  for (Rotation& t : rotations) {
+    if (t.freq) cudaFree(t.freq);
+    if (t.rows) cudaFree(t.rows);
+  }
+  gla.free();
   b200_qweight_destroy(head);
   b200_qweight_destroy(loop_in);
 }
@@ -320,9 +416,10 @@ b200_decoder::~b200_decoder() {
 b200_status b200_decoder::check_pool(const b200_kv* kv) const {
   bool ok = kv->layered && kv->cfg.n_layers == (int)runs.size() && kv->dev.elem_bytes == (int)elem();
   for (size_t r = 0; ok && r < runs.size(); ++r) {
-    const b200_decoder_layer& s = layers[runs[r].layer].s;
+    const b200_kv_layer want = layers[runs[r].layer].cache();
     const KvLayerDev& L = kv->lay[r];
-    ok = L.heads == s.n_kv_heads && L.key_dim == s.key_dim && L.value_dim == s.value_dim && s.n_heads <= kv->cfg.n_q_heads;
+    ok = L.heads == want.n_kv_heads && L.key_dim == want.key_dim && L.value_dim == want.value_dim && L.values_in_keys == want.values_in_keys &&
+         L.rec_elems == want.state_elems && layers[runs[r].layer].s.n_heads <= kv->cfg.n_q_heads;
   }
   if (!ok) { b200_set_error("decoder: the page pool was built for a different model shape"); return B200_ERR_INVALID_ARGUMENT; }
   return B200_OK;
@@ -359,6 +456,7 @@ b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t 
   a.x0 = x0;
   a.h = h;
   a.h_stride = hp;
+  if (hist) { a.hist = hist; a.hist_stride = (size_t)max_rows * cfg.hidden; }
   if (next >= 0 && next < (int)runs.size()) {
     if (runs[next].opens) { a.cat = cat; a.cat_stride = catp; }
     else a.norm_w = layers[runs[next].layer].norm1;
@@ -385,8 +483,107 @@ b200_status b200_decoder::attention(b200_kv* kv, int run, int rows, void* stream
   c.slopes_log2 = l.slopes;
   c.sinks_log2 = l.sinks;
   c.out = attn;
-  c.out_stride = pad64(l.attn_n());
+  c.out_stride = l.out_k();
+  if (l.s.mixer == B200_MIX_LATENT) {
+    c.out = lat_out;
+    c.out_head_stride = pad64(l.s.kv_rank);
+    c.out_stride = l.s.n_heads * c.out_head_stride;
+  }
   return b200_window_attn_run(kv, c, d_row_seq, d_row_ctx, rows, attn_mma, stream);
+}
+
+// Token tile of the experts' matmuls: the rows an expert gets on average, rounded up.
+int b200_decoder::moe_tile_rows(int T) const {
+  if (f32()) return 64;
+  int rows = 0;
+  for (int i : moe_layers) rows = std::max(rows, (T * layers[i].s.top_k + layers[i].s.n_experts - 1) / layers[i].s.n_experts);
+  return std::min(128, std::max(16, (rows + 15) / 16 * 16));
+}
+
+// What the layers of a step share: attention plans, chunks of the recurrent layers, rotations, experts.
+b200_status b200_decoder::begin_step(b200_kv* kv, int n_req, int T, int tile_rows, void* stream) {
+  b200_decoder* m = this;
+  cudaStream_t cs = (cudaStream_t)stream;
+  b200_status st = B200_OK;
+  // one plan per (window, GQA group) of the stack, shared by its layers
+  std::vector<std::pair<int, int>> planned;
+  for (size_t r = 0; r < runs.size(); ++r) {
+    const b200_decoder_layer& s = layers[runs[r].layer].s;
+    if (s.mixer != B200_MIX_ATTENTION) continue;
+    const std::pair<int, int> key{s.window, s.n_heads / s.n_kv_heads};
+    if (!attn_mma || !b200_window_attn_takes_mma(kv, (int)r) || std::find(planned.begin(), planned.end(), key) != planned.end()) continue;
+    planned.push_back(key);
+    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, (int)r, key.first, key.second, d_row_seq, d_row_ctx, T, stream));
+  }
+  if (has_gla && T > n_req) MODEL_STEP_CAT(0, b200_gla_plan(gla, d_cu, n_req, T, stream));
+  for (const Rotation& t : rotations) MODEL_STEP(b200_rotation_table(t.freq, t.dims, d_pos, T, t.rows, stream));
+  if (!moe_layers.empty()) {
+    int most = 0;
+    for (const MoeTableLayer& t : moe) most = std::max(most, t.n_experts);
+    MODEL_STEP(b200_moe_table_plan(d_moe, (int)moe.size(), most, d_tokens, T, cfg.vocab, tile_rows, stream));
+  }
+  return B200_OK;
+}
+
+// Mixer of one layer run: h -> the rows W_o reads.
+b200_status b200_decoder::mixer(b200_kv* kv, int run, int n_req, int T, void* stream) {
+  b200_decoder* m = this;
+  cudaStream_t cs = (cudaStream_t)stream;
+  const Layer& l = layers[runs[run].layer];
+  const b200_decoder_layer& s = l.s;
+  b200_status st = B200_OK;
+  MatSrc src;
+  MODEL_STEP_CAT(1, matmul(l.wqkv, h, T, 1, &src, stream));
+  if (s.mixer == B200_MIX_GLA) {
+    GlaCall c;
+    c.layer = run; c.heads = s.n_heads; c.dk = s.key_dim; c.dv = s.value_dim; c.rank = s.decay_rank; c.src = src;
+    c.a2 = l.a2; c.a2_bias = l.a2_bias; c.norm = l.head_norm; c.eps = cfg.norm_eps;
+    c.q_scale = (float)(1.0 / std::sqrt((double)s.key_dim));
+    c.inv_tau = 1.0f / s.decay_tau;
+    c.out = attn; c.out_stride = l.out_k();
+    MODEL_STEP_CAT(0, b200_gla_run(kv, gla, c, d_cu, d_row_seq, d_pos, n_req, T, attn_mma, stream));
+    return B200_OK;
+  }
+  if (s.mixer == B200_MIX_LATENT) {
+    LatentPrep p;
+    p.layer = run; p.heads = s.n_heads; p.dim = s.key_dim; p.rot = s.rot_dim; p.rank = s.kv_rank; p.src = src; p.norm = l.dkv_norm;
+    p.eps = cfg.norm_eps; p.rotation = l.rotation >= 0 ? rotations[l.rotation].rows : nullptr;
+    p.q_plain = q_plain; p.plain_stride = l.plain_stride(); p.q = q;
+    MODEL_STEP_CAT(2, b200_latent_prep(kv, p, d_pos, d_row_seq, T, stream));
+    const int H = s.n_heads, kd = kv->lay[run].kd, lat = pad64(s.kv_rank);
+    auto blocks = [&](const b200_qweight* w, const void* in, int in_group, void* out, int out_stride, int out_group) {
+      return f32() ? b200_qmm_f32_blocks(w, (const float*)in, H * in_group, in_group, T, (float*)out, out_stride, out_group, stream)
+                   : b200_qmm_blocks(w, in, H * in_group, in_group, T, out, out_stride, out_group, stream);
+    };
+    MODEL_STEP_CAT(1, blocks(l.wuk, q_plain, l.plain_stride(), q, H * kd, kd));
+    MODEL_STEP_CAT(0, attention(kv, run, T, stream));
+    MODEL_STEP_CAT(1, blocks(l.wuv, lat_out, lat, attn, l.out_k(), s.value_dim));
+    return B200_OK;
+  }
+  QkvArgs a;
+  a.d = kv->dev; a.L = kv->lay[run]; a.src = src; a.bias = l.bias; a.hq = s.n_heads; a.qk_norm = s.flags & B200_DEC_QK_NORM ? 1 : 0;
+  a.eps = cfg.norm_eps; a.q = q; a.q_stride = s.n_heads * kv->lay[run].kd; a.pos = d_pos; a.row_seq = d_row_seq;
+  MODEL_STEP_CAT(2, launch_qkv(a, T, cs));
+  MODEL_STEP_CAT(0, attention(kv, run, T, stream));
+  return B200_OK;
+}
+
+// The experts of one layer: h -> moe_y, one row per assignment in the experts' order.
+b200_status b200_decoder::experts(const Layer& l, int T, int tile_rows, void* stream) {
+  b200_decoder* m = this;
+  cudaStream_t cs = (cudaStream_t)stream;
+  b200_status st = B200_OK;
+  const MoeTableLayer& t = moe[l.moe];
+  const int A = T * t.top, act_w = pad64(l.s.expert_ffn), items = std::min(A, t.n_experts + A / tile_rows);
+  if (f32()) {
+    MODEL_STEP_CAT(1, b200_qmm_f32_grouped(l.we_gu, (const float*)h, t.order, t.top, (float*)moe_act, act_w, B200_EPI_SWIGLU, t.items, t.n_items, items, stream));
+    MODEL_STEP_CAT(1, b200_qmm_f32_grouped(l.we_down, (const float*)moe_act, nullptr, 1, (float*)moe_y, hp, B200_EPI_NONE, t.items, t.n_items, items, stream));
+    return B200_OK;
+  }
+  MODEL_STEP(b200_moe_gather_order(h, t.order, t.top, A, hp, moe_x, stream));
+  MODEL_STEP_CAT(1, b200_qmm_grouped(l.we_gu, moe_x, A, moe_act, B200_EPI_SWIGLU, nullptr, 0.f, t.items, t.n_items, items, tile_rows, stream));
+  MODEL_STEP_CAT(1, b200_qmm_grouped(l.we_down, moe_act, A, moe_y, B200_EPI_NONE, nullptr, 0.f, t.items, t.n_items, items, tile_rows, stream));
+  return B200_OK;
 }
 
 b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits, void* stream) {
@@ -394,15 +591,8 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
   cudaStream_t cs = (cudaStream_t)stream;
   b200_status st = B200_OK;
   MatSrc src;
-  // one plan per (window, GQA group) of the stack, shared by its layers
-  std::vector<std::pair<int, int>> planned;
-  for (size_t r = 0; r < runs.size(); ++r) {
-    const b200_decoder_layer& s = layers[runs[r].layer].s;
-    const std::pair<int, int> key{s.window, s.n_heads / s.n_kv_heads};
-    if (!attn_mma || !b200_window_attn_takes_mma(kv, (int)r) || std::find(planned.begin(), planned.end(), key) != planned.end()) continue;
-    planned.push_back(key);
-    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, (int)r, key.first, key.second, d_row_seq, d_row_ctx, T, stream));
-  }
+  const int tile_rows = moe_tile_rows(T);
+  if ((st = begin_step(kv, n_req, T, tile_rows, stream)) != B200_OK) return st;
   {
     RowArgs a{};
     a.tokens = d_tokens;
@@ -422,30 +612,46 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
       a.norm_w = l.norm1;
       MODEL_STEP(rows_step(a, T, -1, cs));
     }
-    MODEL_STEP_CAT(1, matmul(l.wqkv, h, T, 1, &src, stream));
-    {
-      QkvArgs a;
-      a.d = kv->dev; a.L = kv->lay[r]; a.src = src; a.bias = l.bias; a.hq = s.n_heads; a.qk_norm = s.flags & B200_DEC_QK_NORM ? 1 : 0;
-      a.eps = cfg.norm_eps; a.q = q; a.q_stride = s.n_heads * kv->lay[r].kd; a.pos = d_pos; a.row_seq = d_row_seq;
-      MODEL_STEP_CAT(2, launch_qkv(a, T, cs));
-    }
-    MODEL_STEP_CAT(0, attention(kv, (int)r, T, stream));
-    MODEL_STEP_CAT(1, matmul(l.wo, attn, T, 1, &src, stream));
-    {
+    // SwiGLU of the dense feed-forward, experts: both from h
+    auto feed_forward = [&](void* out, int out_stride) -> b200_status {
+      if (s.n_experts > 0 && (st = experts(l, T, tile_rows, stream)) != B200_OK) return st;
+      if (s.ffn == 0) return B200_OK;
+      if (f32()) MODEL_STEP_CAT(1, b200_qmm_f32(l.wgu, (const float*)h, T, (float*)out, out_stride, pad64(s.ffn), B200_EPI_SWIGLU, stream));
+      else MODEL_STEP_CAT(1, b200_qmm_to(l.wgu, h, T, out, out_stride, B200_EPI_SWIGLU, stream));
+      return B200_OK;
+    };
+    auto last_rows = [&](const float* post) -> b200_status {  // the layer's last sublayer joins the residual
       RowArgs a{};
       a.src = src;
-      a.post_w = l.post1;
-      if (s.ffn > 0) a.norm_w = l.norm2;
-      MODEL_STEP(rows_step(a, T, s.ffn > 0 ? -1 : (int)r + 1, cs));
-    }
-    if (s.ffn > 0) {
-      if (f32()) MODEL_STEP_CAT(1, b200_qmm_f32(l.wgu, (const float*)h, T, (float*)act, pad64(s.ffn), pad64(s.ffn), B200_EPI_SWIGLU, stream));
-      else MODEL_STEP_CAT(1, b200_qmm(l.wgu, h, T, act, B200_EPI_SWIGLU, nullptr, 0.f, B200_QMM_AUTO, stream));
-      MODEL_STEP_CAT(1, matmul(l.wdown, act, T, 1, &src, stream));
-      RowArgs a{};
-      a.src = src;
-      a.post_w = l.post2;
-      MODEL_STEP(rows_step(a, T, (int)r + 1, cs));
+      a.post_w = post;
+      if (s.n_experts > 0) {
+        a.moe_y = moe_y; a.moe_rows = moe[l.moe].inv_order; a.moe_k = s.top_k; a.moe_stride = hp; a.moe_w = 1.0f / (float)s.top_k;
+      }
+      if (l.depth) { a.depth = l.depth; a.n_hist = (int)r + 1; }
+      return rows_step(a, T, (int)r + 1, cs);
+    };
+    if (l.parallel()) {
+      if ((st = feed_forward((char*)attn + pad64(l.attn_n()) * elem(), l.out_k())) != B200_OK) return st;
+      if ((st = mixer(kv, (int)r, n_req, T, stream)) != B200_OK) return st;
+      MODEL_STEP_CAT(1, matmul(l.wo, attn, T, 1, &src, stream));
+      MODEL_STEP(last_rows(nullptr));
+    } else {
+      const bool ff = s.ffn > 0 || s.n_experts > 0;
+      if ((st = mixer(kv, (int)r, n_req, T, stream)) != B200_OK) return st;
+      MODEL_STEP_CAT(1, matmul(l.wo, attn, T, 1, &src, stream));
+      if (!ff) {
+        MODEL_STEP(last_rows(l.post1));
+      } else {
+        RowArgs a{};
+        a.src = src;
+        a.post_w = l.post1;
+        a.norm_w = l.norm2;
+        MODEL_STEP(rows_step(a, T, -1, cs));
+        if ((st = feed_forward(act, pad64(s.ffn))) != B200_OK) return st;
+        src = MatSrc{};
+        if (s.ffn > 0) MODEL_STEP_CAT(1, matmul(l.wdown, act, T, 1, &src, stream));
+        MODEL_STEP(last_rows(l.post2));
+      }
     }
     if (recording)
       B200_CUDA_TRY(cudaMemcpyAsync(rec + r * (size_t)max_rows * cfg.hidden, x, sizeof(float) * (size_t)T * cfg.hidden, cudaMemcpyDeviceToDevice, cs));
@@ -481,26 +687,41 @@ uint64_t tensor_elems(const b200_decoder* m, int layer, int which) {
   switch (which) {
     case B200_DEC_W_HEAD: case B200_DEC_W_EMBED: return (uint64_t)c.vocab * D;
     case B200_DEC_W_LOOP_IN: return c.loop_times > 0 ? 2 * D * D : 0;
-    case B200_DEC_FINAL_NORM: return D;
+    case B200_DEC_FINAL_NORM: return c.flags & B200_DEC_SCALAR_NORM ? 1 : D;
     default: break;
   }
   const b200_decoder_layer& s = m->layers[layer].s;
-  const uint64_t qn = (uint64_t)s.n_heads * s.key_dim, kn = (uint64_t)s.n_kv_heads * s.key_dim, vn = (uint64_t)s.n_kv_heads * s.value_dim;
-  const bool bias = s.flags & B200_DEC_QKV_BIAS, post = s.flags & B200_DEC_POST_NORM;
+  const uint64_t H = s.n_heads, norm = c.flags & B200_DEC_SCALAR_NORM ? 1 : D, ef = (uint64_t)s.n_experts * s.expert_ffn;
+  const bool latent = s.mixer == B200_MIX_LATENT, gla = s.mixer == B200_MIX_GLA, soft = s.mixer == B200_MIX_ATTENTION;
+  const uint64_t qn = H * (s.key_dim + (latent ? s.rot_dim : 0)), kn = (gla ? H : s.n_kv_heads) * (uint64_t)s.key_dim,
+                 vn = (gla ? H : s.n_kv_heads) * (uint64_t)s.value_dim;
+  const bool bias = soft && s.flags & B200_DEC_QKV_BIAS, post = s.flags & B200_DEC_POST_NORM;
+  const bool ff = s.ffn > 0 || s.n_experts > 0, second = ff && !(s.flags & B200_DEC_PARALLEL);
   switch (which) {
     case B200_DEC_W_Q: return qn * D;
-    case B200_DEC_W_K: return kn * D;
-    case B200_DEC_W_V: return vn * D;
-    case B200_DEC_W_O: return D * s.n_heads * s.value_dim;
+    case B200_DEC_W_K: return latent ? 0 : kn * D;
+    case B200_DEC_W_V: return latent ? 0 : vn * D;
+    case B200_DEC_W_O: return D * H * s.value_dim;
     case B200_DEC_W_GATE: case B200_DEC_W_UP: case B200_DEC_W_DOWN: return D * s.ffn;
     case B200_DEC_B_Q: return bias ? qn : 0;
     case B200_DEC_B_K: return bias ? kn : 0;
     case B200_DEC_B_V: return bias ? vn : 0;
-    case B200_DEC_W_SINK: return s.flags & B200_DEC_SINK ? s.n_heads : 0;
-    case B200_DEC_NORM1: return D;
-    case B200_DEC_NORM2: return s.ffn > 0 ? D : 0;
-    case B200_DEC_POSTNORM1: return post ? D : 0;
-    case B200_DEC_POSTNORM2: return post && s.ffn > 0 ? D : 0;
+    case B200_DEC_W_SINK: return s.flags & B200_DEC_SINK ? H : 0;
+    case B200_DEC_NORM1: return norm;
+    case B200_DEC_NORM2: return second ? norm : 0;
+    case B200_DEC_POSTNORM1: return post ? norm : 0;
+    case B200_DEC_POSTNORM2: return post && second ? norm : 0;
+    case B200_DEC_W_DKV: return latent ? (uint64_t)(s.kv_rank + s.rot_dim) * D : 0;
+    case B200_DEC_DKV_NORM: return latent ? s.kv_rank : 0;
+    case B200_DEC_W_UK: return latent ? H * s.key_dim * s.kv_rank : 0;
+    case B200_DEC_W_UV: return latent ? H * s.value_dim * s.kv_rank : 0;
+    case B200_DEC_W_OUT_GATE: return gla ? vn * D : 0;
+    case B200_DEC_W_A1: return gla ? s.decay_rank * D : 0;
+    case B200_DEC_W_A2: return gla ? kn * s.decay_rank : 0;
+    case B200_DEC_B_A2: return gla ? kn : 0;
+    case B200_DEC_HEAD_NORM: return gla ? s.value_dim : 0;
+    case B200_DEC_W_EXPERT_GATE: case B200_DEC_W_EXPERT_UP: case B200_DEC_W_EXPERT_DOWN: return ef * D;
+    case B200_DEC_DEPTH: return c.flags & B200_DEC_DEPTH_AVERAGE ? layer + 2 : 0;
     default: return 0;
   }
 }
@@ -530,6 +751,85 @@ b200_status take_vector(b200_decoder* m, int layer, int which, float** out, doub
   std::vector<float> v(bits.size());
   for (size_t i = 0; i < bits.size(); ++i) v[i] = factor == 1.0 ? bf16_to_f(bits[i]) : (float)(bf16_to_f(bits[i]) * factor);
   return upload_f32(v, out);
+}
+
+// A norm's weight over the whole width, also where the checkpoint holds one number.
+b200_status take_norm(b200_decoder* m, int layer, int which, float** out, double factor = 1.0) {
+  std::vector<uint16_t> bits;
+  b200_status st = take(m, layer, which, &bits);
+  if (st != B200_OK) return st;
+  std::vector<float> v(m->cfg.hidden);
+  for (size_t i = 0; i < v.size(); ++i) v[i] = (float)(bf16_to_f(bits[bits.size() == 1 ? 0 : i]) * factor);
+  return upload_f32(v, out);
+}
+
+// Matrices [n, k_i] beside one another as one weight, each padded to a multiple of 64 columns.
+b200_status take_beside(b200_decoder* m, int layer, std::vector<std::pair<int, int>> which_k, int n, b200_qweight** out) {
+  int kp = 0;
+  for (auto& wk : which_k) kp += pad64(wk.second);
+  const int np = pad64(n);
+  std::vector<uint16_t> w((size_t)np * kp, 0);
+  int col = 0;
+  for (auto& wk : which_k) {
+    std::vector<uint16_t> part;
+    b200_status st = take(m, layer, wk.first, &part);
+    if (st != B200_OK) return st;
+    for (int r = 0; r < n; ++r) std::memcpy(&w[(size_t)r * kp + col], &part[(size_t)r * wk.second], sizeof(uint16_t) * wk.second);
+    col += pad64(wk.second);
+  }
+  return b200_qweight_create(B200_Q_BF16, 1, np, kp, w.data(), nullptr, nullptr, out);
+}
+
+// A stack of `count` matrices [n, k] held as [count][n][k] (transposed: [count][k][n]); n rows each, columns padded to 64.
+b200_status take_stack(b200_decoder* m, int layer, int which, int count, int n, int k, bool transposed, b200_qweight** out) {
+  std::vector<uint16_t> part;
+  b200_status st = take(m, layer, which, &part);
+  if (st != B200_OK) return st;
+  const int kp = pad64(k);
+  std::vector<uint16_t> w((size_t)count * n * kp, 0);
+  for (int e = 0; e < count; ++e)
+    for (int r = 0; r < n; ++r)
+      for (int c = 0; c < k; ++c)
+        w[((size_t)e * n + r) * kp + c] = part[transposed ? ((size_t)e * k + c) * n + r : ((size_t)e * n + r) * k + c];
+  return b200_qweight_create(B200_Q_BF16, count, n, kp, w.data(), nullptr, nullptr, out);
+}
+
+// Experts: gate and up rows interleaved, [2 pad(ff), pad(hidden)]; down [pad(hidden), pad(ff)].
+b200_status take_experts(b200_decoder* m, int layer, b200_decoder::Layer& l) {
+  const int E = l.s.n_experts, f = l.s.expert_ffn, D = m->cfg.hidden, fp = pad64(f), dp = pad64(D);
+  std::vector<uint16_t> gate, up, down;
+  b200_status st;
+  if ((st = take(m, layer, B200_DEC_W_EXPERT_GATE, &gate)) != B200_OK || (st = take(m, layer, B200_DEC_W_EXPERT_UP, &up)) != B200_OK ||
+      (st = take(m, layer, B200_DEC_W_EXPERT_DOWN, &down)) != B200_OK)
+    return st;
+  std::vector<uint16_t> w((size_t)E * 2 * fp * dp, 0);
+  for (int e = 0; e < E; ++e)
+    for (int r = 0; r < f; ++r) {
+      uint16_t* dst = &w[((size_t)e * 2 * fp + 2 * r) * dp];
+      std::memcpy(dst, &gate[((size_t)e * f + r) * D], sizeof(uint16_t) * D);
+      std::memcpy(dst + dp, &up[((size_t)e * f + r) * D], sizeof(uint16_t) * D);
+    }
+  if ((st = b200_qweight_create(B200_Q_BF16, E, 2 * fp, dp, w.data(), nullptr, nullptr, &l.we_gu)) != B200_OK) return st;
+  w.assign((size_t)E * dp * fp, 0);
+  for (int e = 0; e < E; ++e)
+    for (int r = 0; r < D; ++r) std::memcpy(&w[((size_t)e * dp + r) * fp], &down[((size_t)e * D + r) * f], sizeof(uint16_t) * f);
+  return b200_qweight_create(B200_Q_BF16, E, dp, fp, w.data(), nullptr, nullptr, &l.we_down);
+}
+
+b200_status upload_table(b200_decoder* m, int layer, b200_decoder::Layer& l) {
+  if (l.h_table.empty()) { b200_set_error("decoder: the expert table of layer %d was never set", layer); return B200_ERR_INVALID_ARGUMENT; }
+  B200_CUDA_TRY(cudaMalloc((void**)&l.table, sizeof(int) * l.h_table.size()));
+  B200_CUDA_TRY(cudaMemcpy(l.table, l.h_table.data(), sizeof(int) * l.h_table.size(), cudaMemcpyHostToDevice));
+  m->moe[l.moe].table = l.table;
+  return B200_OK;
+}
+
+// After the last table is in place: the plan structures the kernels read.
+b200_status upload_moe(b200_decoder* m) {
+  if (m->moe.empty()) return B200_OK;
+  if (!m->d_moe) B200_CUDA_TRY(cudaMalloc((void**)&m->d_moe, sizeof(MoeTableLayer) * m->moe.size()));
+  B200_CUDA_TRY(cudaMemcpy(m->d_moe, m->moe.data(), sizeof(MoeTableLayer) * m->moe.size(), cudaMemcpyHostToDevice));
+  return B200_OK;
 }
 
 // Rows of several [n_i, k] matrices, one behind the other or interleaved, as one weight padded to multiples of 64.
@@ -577,6 +877,7 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
   const bool loop = c->loop_times > 0;
   if (c->n_layers <= 0 || c->hidden <= 0 || c->vocab <= 0 || c->max_rows <= 0 || c->max_reqs <= 0 || c->max_seqs <= 0 ||
       (c->dtype != B200_DT_BF16 && c->dtype != B200_DT_F32) ||
+      (loop && (c->flags & B200_DEC_DEPTH_AVERAGE)) ||
       (loop && (c->loop_start < 0 || c->loop_stop > c->n_layers || c->loop_start >= c->loop_stop))) {
     b200_set_error("decoder: invalid configuration");
     return B200_ERR_INVALID_ARGUMENT;
@@ -585,19 +886,47 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
   auto* m = new b200_decoder();
   m->cfg = *c;
   m->layers.resize(c->n_layers);
-  size_t qw = 0, yw = pad64(c->hidden), aw = 0, fw = 0;
+  size_t qw = 0, yw = pad64(c->hidden), aw = 0, fw = 0, plain_w = 0, lat_w = 0, assign = 0, moe_aw = 0;
   for (int i = 0; i < c->n_layers; ++i) {
     const b200_decoder_layer& s = layers[i];
-    if (s.n_heads <= 0 || s.n_kv_heads <= 0 || s.n_heads % s.n_kv_heads != 0 || s.key_dim <= 0 || s.value_dim <= 0 || s.ffn < 0 || s.window < 0) {
+    bool good = s.n_heads > 0 && s.key_dim > 0 && s.value_dim > 0 && s.ffn >= 0 && s.window >= 0 && s.n_experts >= 0;
+    if (s.mixer == B200_MIX_ATTENTION) good = good && s.n_kv_heads > 0 && s.n_heads % s.n_kv_heads == 0;
+    else if (s.mixer == B200_MIX_LATENT) good = good && s.kv_rank > 0 && s.rot_dim >= 0 && s.rot_dim % 2 == 0 && (s.rot_dim == 0 || s.rot_base > 0.f) && s.window == 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS));
+    else if (s.mixer == B200_MIX_GLA) good = good && s.decay_rank > 0 && s.decay_tau > 0.f && s.window == 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS | B200_DEC_SINK));
+    else good = false;
+    if (s.n_experts > 0) good = good && s.top_k > 0 && s.top_k <= s.n_experts && s.n_experts <= b200_moe_max_experts() && s.expert_ffn > 0;
+    if (s.flags & B200_DEC_PARALLEL) good = good && !(s.flags & B200_DEC_POST_NORM);
+    if (!good) {
       b200_set_error("decoder: layer %d has an invalid shape", i);
       delete m;
       return B200_ERR_INVALID_ARGUMENT;
     }
-    m->layers[i].s = s;
-    qw = std::max(qw, (size_t)s.n_heads * ((s.key_dim + 15) / 16 * 16));
-    yw = std::max(yw, (size_t)pad64(m->layers[i].qkv_n()));
-    aw = std::max(aw, (size_t)pad64(m->layers[i].attn_n()));
+    b200_decoder::Layer& l = m->layers[i];
+    l.s = s;
+    qw = std::max(qw, (size_t)s.n_heads * (s.mixer == B200_MIX_LATENT ? l.latent_width() : (s.key_dim + 15) / 16 * 16));
+    yw = std::max(yw, (size_t)pad64(l.qkv_n()));
+    aw = std::max(aw, (size_t)l.out_k());
     fw = std::max(fw, (size_t)pad64(s.ffn));
+    if (s.mixer == B200_MIX_LATENT) {
+      plain_w = std::max(plain_w, (size_t)s.n_heads * l.plain_stride());
+      lat_w = std::max(lat_w, (size_t)s.n_heads * pad64(s.kv_rank));
+      for (size_t t = 0; t < m->rotations.size() && l.rotation < 0; ++t)
+        if (m->rotations[t].base == s.rot_base && m->rotations[t].dims == s.rot_dim) l.rotation = (int)t;
+      if (l.rotation < 0 && s.rot_dim > 0) {
+        l.rotation = (int)m->rotations.size();
+        m->rotations.push_back({s.rot_base, s.rot_dim, nullptr, nullptr});
+      }
+    }
+    if (s.mixer == B200_MIX_GLA) {
+      m->has_gla = true;
+      if (b200_gla_takes_chunks(s.key_dim, s.value_dim, (int)m->elem())) m->gla.need(s.n_heads, s.key_dim, s.value_dim);
+    }
+    if (s.n_experts > 0) {
+      l.moe = (int)m->moe_layers.size();
+      m->moe_layers.push_back(i);
+      assign = std::max(assign, (size_t)s.top_k);
+      moe_aw = std::max(moe_aw, (size_t)s.top_k * pad64(s.expert_ffn));
+    }
   }
   const int lo = loop ? c->loop_start : 0, hi = loop ? c->loop_stop : 0;
   for (int i = 0; i < lo; ++i) m->runs.push_back({i, false});
@@ -626,6 +955,40 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
   alloc(&m->attn, R * aw * e);
   alloc(&m->act, R * fw * e);
   alloc(&m->last, (size_t)c->max_reqs * m->hp * e);
+  alloc(&m->q_plain, R * plain_w * e);
+  alloc(&m->lat_out, R * lat_w * e);
+  if (c->flags & B200_DEC_DEPTH_AVERAGE) alloc((void**)&m->hist, (size_t)(c->n_layers + 1) * R * c->hidden * 4);
+  for (b200_decoder::Rotation& t : m->rotations) {
+    std::vector<double> f(t.dims / 2);
+    for (int i = 0; i < t.dims / 2; ++i) f[i] = std::pow((double)t.base, -2.0 * i / t.dims);
+    alloc((void**)&t.freq, sizeof(double) * f.size());
+    alloc((void**)&t.rows, sizeof(float2) * R * f.size());
+    if (st == B200_OK) cudaMemcpy(t.freq, f.data(), sizeof(double) * f.size(), cudaMemcpyHostToDevice);
+  }
+  if (!m->moe_layers.empty()) {
+    if (!m->f32()) alloc(&m->moe_x, R * assign * m->hp * e);
+    alloc(&m->moe_act, R * moe_aw * e);
+    alloc(&m->moe_y, R * assign * m->hp * e);
+    for (int i : m->moe_layers) {
+      const b200_decoder_layer& s = m->layers[i].s;
+      const size_t A = R * s.top_k;
+      MoeTableLayer t;
+      t.n_experts = s.n_experts;
+      t.top = s.top_k;
+      alloc((void**)&t.indices, 4 * A + 16);
+      alloc((void**)&t.offsets, 4 * (s.n_experts + 1));
+      alloc((void**)&t.order, 4 * A);
+      alloc((void**)&t.inv_order, 4 * A);
+      alloc((void**)&t.n_items, 4);
+      alloc((void**)&t.items, sizeof(int4) * (s.n_experts + A / 16 + 1));
+      m->moe.push_back(t);
+    }
+  }
+  if (m->has_gla && st == B200_OK) {
+    m->gla.max_rows = c->max_rows;
+    m->gla.max_reqs = c->max_reqs;
+    if (!m->gla.alloc()) { b200_set_error("decoder: no memory for the chunks of %d rows", c->max_rows); st = B200_ERR_CUDA; }
+  }
   if (st != B200_OK) { delete m; return st; }
   *out = m;
   return B200_OK;
@@ -635,7 +998,7 @@ void b200_decoder_destroy(b200_decoder* m) { delete m; }
 b200_model* b200_decoder_model(b200_decoder* m) { return m; }
 
 b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t which, const void* h_bf16, uint64_t n) {
-  if (which < 0 || which > B200_DEC_FINAL_NORM || (!global_tensor(which) && (layer < 0 || layer >= m->cfg.n_layers))) {
+  if (which < 0 || which > B200_DEC_DEPTH || (!global_tensor(which) && (layer < 0 || layer >= m->cfg.n_layers))) {
     b200_set_error("decoder: no tensor %d in layer %d", which, layer);
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -649,21 +1012,54 @@ b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t whic
   return B200_OK;
 }
 
+b200_status b200_decoder_set_table(b200_decoder* m, int32_t layer, const int32_t* h_table, uint64_t n) {
+  if (layer < 0 || layer >= m->cfg.n_layers || m->layers[layer].s.n_experts <= 0 || n != (uint64_t)m->cfg.vocab * m->layers[layer].s.top_k) {
+    b200_set_error("decoder: an expert table of %llu numbers for layer %d", (unsigned long long)n, layer);
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  for (uint64_t i = 0; i < n; ++i)
+    if (h_table[i] < 0 || h_table[i] >= m->layers[layer].s.n_experts) {
+      b200_set_error("decoder: the expert table of layer %d names expert %d of %d", layer, h_table[i], m->layers[layer].s.n_experts);
+      return B200_ERR_INVALID_ARGUMENT;
+    }
+  m->layers[layer].h_table.assign(h_table, h_table + n);
+  return B200_OK;
+}
+
 b200_status b200_decoder_finalize(b200_decoder* m) {
   const b200_decoder_config& c = m->cfg;
   b200_status st;
   for (int i = 0; i < c.n_layers; ++i) {
     b200_decoder::Layer& l = m->layers[i];
     const b200_decoder_layer& s = l.s;
-    if ((st = take_weight(m, i, {B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V}, c.hidden, false, &l.wqkv)) != B200_OK) return st;
-    if ((st = take_weight(m, i, {B200_DEC_W_O}, l.attn_n(), false, &l.wo)) != B200_OK) return st;
-    if ((st = take_vector(m, i, B200_DEC_NORM1, &l.norm1)) != B200_OK) return st;
-    if (s.flags & B200_DEC_POST_NORM) if ((st = take_vector(m, i, B200_DEC_POSTNORM1, &l.post1)) != B200_OK) return st;
+    if ((st = take_weight(m, i, l.projections(), c.hidden, false, &l.wqkv)) != B200_OK) return st;
+    if (l.parallel() && s.ffn > 0) st = take_beside(m, i, {{B200_DEC_W_O, l.attn_n()}, {B200_DEC_W_DOWN, s.ffn}}, c.hidden, &l.wo);
+    else st = take_weight(m, i, {B200_DEC_W_O}, l.attn_n(), false, &l.wo);
+    if (st != B200_OK) return st;
+    if ((st = take_norm(m, i, B200_DEC_NORM1, &l.norm1)) != B200_OK) return st;
+    if (s.flags & B200_DEC_POST_NORM) if ((st = take_norm(m, i, B200_DEC_POSTNORM1, &l.post1)) != B200_OK) return st;
     if (s.ffn > 0) {
       if ((st = take_weight(m, i, {B200_DEC_W_GATE, B200_DEC_W_UP}, c.hidden, true, &l.wgu)) != B200_OK) return st;
-      if ((st = take_weight(m, i, {B200_DEC_W_DOWN}, s.ffn, false, &l.wdown)) != B200_OK) return st;
-      if ((st = take_vector(m, i, B200_DEC_NORM2, &l.norm2)) != B200_OK) return st;
-      if (s.flags & B200_DEC_POST_NORM) if ((st = take_vector(m, i, B200_DEC_POSTNORM2, &l.post2)) != B200_OK) return st;
+      if (!l.parallel()) if ((st = take_weight(m, i, {B200_DEC_W_DOWN}, s.ffn, false, &l.wdown)) != B200_OK) return st;
+    }
+    if (s.n_experts > 0) {
+      if ((st = take_experts(m, i, l)) != B200_OK) return st;
+      if ((st = upload_table(m, i, l)) != B200_OK) return st;
+    }
+    if ((s.ffn > 0 || s.n_experts > 0) && !l.parallel()) {
+      if ((st = take_norm(m, i, B200_DEC_NORM2, &l.norm2)) != B200_OK) return st;
+      if (s.flags & B200_DEC_POST_NORM) if ((st = take_norm(m, i, B200_DEC_POSTNORM2, &l.post2)) != B200_OK) return st;
+    }
+    if (c.flags & B200_DEC_DEPTH_AVERAGE) if ((st = take_vector(m, i, B200_DEC_DEPTH, &l.depth)) != B200_OK) return st;
+    if (s.mixer == B200_MIX_LATENT) {
+      if ((st = take_vector(m, i, B200_DEC_DKV_NORM, &l.dkv_norm)) != B200_OK) return st;
+      if ((st = take_stack(m, i, B200_DEC_W_UK, s.n_heads, s.kv_rank, s.key_dim, true, &l.wuk)) != B200_OK) return st;
+      if ((st = take_stack(m, i, B200_DEC_W_UV, s.n_heads, s.value_dim, s.kv_rank, false, &l.wuv)) != B200_OK) return st;
+    }
+    if (s.mixer == B200_MIX_GLA) {
+      if ((st = take_vector(m, i, B200_DEC_W_A2, &l.a2)) != B200_OK) return st;
+      if ((st = take_vector(m, i, B200_DEC_B_A2, &l.a2_bias)) != B200_OK) return st;
+      if ((st = take_vector(m, i, B200_DEC_HEAD_NORM, &l.head_norm)) != B200_OK) return st;
     }
     if (s.flags & B200_DEC_QKV_BIAS) {
       std::vector<float> all;
@@ -679,7 +1075,9 @@ b200_status b200_decoder_finalize(b200_decoder* m) {
   }
   if (c.loop_times > 0) if ((st = take_weight(m, -1, {B200_DEC_W_LOOP_IN}, 2 * c.hidden, false, &m->loop_in)) != B200_OK) return st;
   if ((st = take_weight(m, -1, {B200_DEC_W_HEAD}, c.hidden, false, &m->head)) != B200_OK) return st;
-  if ((st = take_vector(m, -1, B200_DEC_FINAL_NORM, &m->final_norm)) != B200_OK) return st;
+  // (the logits' scale rides on the final norm's weight)
+  if ((st = take_norm(m, -1, B200_DEC_FINAL_NORM, &m->final_norm, c.logit_scale)) != B200_OK) return st;
+  if ((st = upload_moe(m)) != B200_OK) return st;
   std::vector<uint16_t> table;
   if ((st = take(m, -1, B200_DEC_W_EMBED, &table)) != B200_OK) return st;
   B200_CUDA_TRY(cudaMemcpy(m->embed, table.data(), table.size() * 2, cudaMemcpyHostToDevice));
@@ -691,27 +1089,57 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
   const b200_decoder_config& c = m->cfg;
   b200_status st;
   const std::vector<float> ones(c.hidden, 1.f);
-  auto weight = [&](int n, int k, uint32_t salt, b200_qweight** out) -> b200_status {
-    if (n % 128 || k % 64) { b200_set_error("random_init: a %d x %d projection (multiples of 128 and 64 only)", n, k); return B200_ERR_INVALID_ARGUMENT; }
-    return b200_qweight_random(B200_Q_BF16, 1, n, k, seed + salt, out);
+  auto stack = [&](int count, int n, int k, uint32_t salt, b200_qweight** out) -> b200_status {
+    if (n % 64 || k % 64) { b200_set_error("random_init: a %d x %d projection (multiples of 64 only)", n, k); return B200_ERR_INVALID_ARGUMENT; }
+    return b200_qweight_random(B200_Q_BF16, count, n, k, seed + salt, out);
   };
+  auto weight = [&](int n, int k, uint32_t salt, b200_qweight** out) -> b200_status { return stack(1, n, k, salt, out); };
   for (int i = 0; i < c.n_layers; ++i) {
     b200_decoder::Layer& l = m->layers[i];
     const b200_decoder_layer& s = l.s;
-    if ((st = weight(l.qkv_n(), c.hidden, 16 * i + 1, &l.wqkv)) != B200_OK) return st;
-    if ((st = weight(c.hidden, l.attn_n(), 16 * i + 2, &l.wo)) != B200_OK) return st;
+    if ((st = weight(pad64(l.qkv_n()), c.hidden, 16 * i + 1, &l.wqkv)) != B200_OK) return st;
+    if ((st = weight(c.hidden, l.out_k(), 16 * i + 2, &l.wo)) != B200_OK) return st;
     if ((st = upload_f32(ones, &l.norm1)) != B200_OK) return st;
     if (s.flags & B200_DEC_POST_NORM) if ((st = upload_f32(ones, &l.post1)) != B200_OK) return st;
     if (s.ffn > 0) {
       if ((st = weight(2 * s.ffn, c.hidden, 16 * i + 3, &l.wgu)) != B200_OK) return st;
-      if ((st = weight(c.hidden, s.ffn, 16 * i + 4, &l.wdown)) != B200_OK) return st;
+      if (!l.parallel()) if ((st = weight(c.hidden, s.ffn, 16 * i + 4, &l.wdown)) != B200_OK) return st;
+    }
+    if ((s.ffn > 0 || s.n_experts > 0) && !l.parallel()) {
       if ((st = upload_f32(ones, &l.norm2)) != B200_OK) return st;
       if (s.flags & B200_DEC_POST_NORM) if ((st = upload_f32(ones, &l.post2)) != B200_OK) return st;
+    }
+    if (s.n_experts > 0) {
+      if ((st = stack(s.n_experts, 2 * s.expert_ffn, c.hidden, 16 * i + 5, &l.we_gu)) != B200_OK) return st;
+      if ((st = stack(s.n_experts, c.hidden, s.expert_ffn, 16 * i + 6, &l.we_down)) != B200_OK) return st;
+      l.h_table.resize((size_t)c.vocab * s.top_k);
+      uint32_t x = seed * 747796405u + i;
+      for (int v = 0; v < c.vocab; ++v) {  // experts an odd step apart from a random one: all different
+        x = x * 1664525u + 1013904223u;
+        for (int j = 0; j < s.top_k; ++j) l.h_table[(size_t)v * s.top_k + j] = (int)(((x >> 8) + (uint32_t)j) % (uint32_t)s.n_experts);
+      }
+      if ((st = upload_table(m, i, l)) != B200_OK) return st;
+    }
+    if (c.flags & B200_DEC_DEPTH_AVERAGE) {
+      std::vector<float> d(i + 2, 0.1f);
+      d[i + 1] = 0.8f;
+      if ((st = upload_f32(d, &l.depth)) != B200_OK) return st;
+    }
+    if (s.mixer == B200_MIX_LATENT) {
+      if ((st = upload_f32(std::vector<float>(s.kv_rank, 1.f), &l.dkv_norm)) != B200_OK) return st;
+      if ((st = stack(s.n_heads, s.kv_rank, l.plain_stride(), 16 * i + 7, &l.wuk)) != B200_OK) return st;
+      if ((st = stack(s.n_heads, s.value_dim, pad64(s.kv_rank), 16 * i + 8, &l.wuv)) != B200_OK) return st;
+    }
+    if (s.mixer == B200_MIX_GLA) {
+      if ((st = upload_f32(std::vector<float>((size_t)s.n_heads * s.key_dim * s.decay_rank, 0.02f), &l.a2)) != B200_OK) return st;
+      if ((st = upload_f32(std::vector<float>((size_t)s.n_heads * s.key_dim, 2.f), &l.a2_bias)) != B200_OK) return st;
+      if ((st = upload_f32(std::vector<float>(s.value_dim, 1.f), &l.head_norm)) != B200_OK) return st;
     }
     if (s.flags & B200_DEC_QKV_BIAS) if ((st = upload_f32(std::vector<float>(l.qkv_n(), 0.01f), &l.bias)) != B200_OK) return st;
     if (s.flags & B200_DEC_SINK) if ((st = upload_f32(std::vector<float>(s.n_heads, 0.5f), &l.sinks)) != B200_OK) return st;
     if ((st = make_slopes(l)) != B200_OK) return st;
   }
+  if ((st = upload_moe(m)) != B200_OK) return st;
   if (c.loop_times > 0) if ((st = weight(c.hidden, 2 * c.hidden, 11, &m->loop_in)) != B200_OK) return st;
   if ((st = weight(c.vocab, c.hidden, 7, &m->head)) != B200_OK) return st;
   if ((st = upload_f32(ones, &m->final_norm)) != B200_OK) return st;
@@ -725,8 +1153,7 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
 
 int32_t b200_decoder_cache_layers(const b200_decoder* m, b200_kv_layer* out, int32_t cap) {
   for (size_t r = 0; r < m->runs.size() && (int)r < cap; ++r) {
-    const b200_decoder_layer& s = m->layers[m->runs[r].layer].s;
-    out[r] = b200_kv_layer{s.n_kv_heads, s.key_dim, s.value_dim};
+    out[r] = m->layers[m->runs[r].layer].cache();
   }
   return (int32_t)m->runs.size();
 }
@@ -755,7 +1182,7 @@ void b200_decoder_set_attn_mma(b200_decoder* m, int32_t on) {
 b200_status b200_decoder_qkv(b200_kv* kv, int32_t layer, const void* d_qkv, int32_t stride, const float* d_bias, int32_t n_q_heads,
                              int32_t qk_norm, float eps, void* d_q, const int32_t* d_positions, const int32_t* d_row_seq,
                              int32_t total_rows, void* stream) {
-  if (!kv->layered || layer < 0 || layer >= kv->cfg.n_layers || n_q_heads <= 0 || n_q_heads % kv->lay[layer].heads != 0) {
+  if (!kv->layered || layer < 0 || layer >= kv->cfg.n_layers || n_q_heads <= 0 || kv->lay[layer].heads <= 0 || n_q_heads % kv->lay[layer].heads != 0) {
     b200_set_error("decoder_qkv: layer %d with %d query heads", layer, n_q_heads);
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -773,7 +1200,7 @@ b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, 
                                    const float* d_slopes_log2, const float* d_sinks_log2, const int32_t* d_row_seq,
                                    const int32_t* d_row_ctx, int32_t total_rows, int32_t mma, void* d_out,
                                    int32_t out_stride, void* stream) {
-  if (!kv->layered || layer < 0 || layer >= kv->cfg.n_layers || n_q_heads <= 0 || n_q_heads > kv->cfg.n_q_heads ||
+  if (!kv->layered || layer < 0 || layer >= kv->cfg.n_layers || n_q_heads <= 0 || n_q_heads > kv->cfg.n_q_heads || kv->lay[layer].heads <= 0 ||
       n_q_heads % kv->lay[layer].heads != 0 || window < 0) {
     b200_set_error("decoder_attention: layer %d with %d query heads, window %d", layer, n_q_heads, window);
     return B200_ERR_INVALID_ARGUMENT;

@@ -95,6 +95,7 @@ struct WindowAttnCall {
   const float* sinks_log2 = nullptr;
   void* out = nullptr;
   int out_stride = 0;
+  int out_head_stride = 0;  // elements between heads of an output row (0: value_dim)
 };
 // Builds (once per step) the plan that calls of this window and GQA group size share; `layer` is one of the layers it is
 // for (its shape says how many workers the grid has).

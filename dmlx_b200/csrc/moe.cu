@@ -17,6 +17,7 @@
 #include <vector>
 
 #include "common.h"
+#include "moe.cuh"
 #include "qmm.cuh"
 
 b200_status b200_gather_rows(const void* d_src, const int32_t* d_idx, void* d_dst, int32_t rows, int32_t hidden, void* stream);
@@ -136,9 +137,8 @@ __global__ void offsets_items_kernel(const int* __restrict__ counts, int n_exper
 // One CTA per expert: collects, in flat order, the assignments routed to it (stable).  A thread looks
 // at 8 consecutive assignments per pass (two 16-byte loads), so a pass of the CTA covers 8192 of them
 // with one block scan.
-__global__ void __launch_bounds__(1024) place_kernel(const uint32_t* __restrict__ indices, int n_assign,
-                                                     const int* __restrict__ offsets, int* __restrict__ order,
-                                                     int* __restrict__ inv_order) {
+__device__ __forceinline__ void place_assignments(const uint32_t* __restrict__ indices, int n_assign, const int* __restrict__ offsets,
+                                                  int* __restrict__ order, int* __restrict__ inv_order) {
   __shared__ int warp_sums[32];
   __shared__ int s_base;
   const int e = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -192,6 +192,63 @@ __global__ void __launch_bounds__(1024) place_kernel(const uint32_t* __restrict_
     if (tid == 0) s_base += total;
     __syncthreads();
   }
+}
+
+__global__ void __launch_bounds__(1024) place_kernel(const uint32_t* __restrict__ indices, int n_assign,
+                                                     const int* __restrict__ offsets, int* __restrict__ order,
+                                                     int* __restrict__ inv_order) {
+  place_assignments(indices, n_assign, offsets, order, inv_order);
+}
+
+// ---- experts by token id ----------------------------------------------------------------------------------------------
+// Without a router the experts of a step's tokens are known before the first layer runs: one CTA per layer looks them up, counts
+// them and lays out the work items; one CTA per (expert, layer) then places the assignments.
+__global__ void __launch_bounds__(1024) table_route_kernel(const MoeTableLayer* __restrict__ layers, const uint32_t* __restrict__ tokens, int n_tokens,
+                                                           int vocab, int tile_rows) {
+  __shared__ int s_count[kMaxExperts], s_off[kMaxExperts + 1], s_item[kMaxExperts + 1];
+  const MoeTableLayer L = layers[blockIdx.x];
+  const int tid = threadIdx.x, n = n_tokens * L.top;
+  for (int e = tid; e < L.n_experts; e += blockDim.x) s_count[e] = 0;
+  __syncthreads();
+  for (int a = tid; a < n; a += blockDim.x) {
+    const int t = a / L.top;
+    const uint32_t tok = min(tokens[t], (uint32_t)(vocab - 1));
+    const int e = L.table[(size_t)tok * L.top + (a - t * L.top)];  // (entries are checked when the table is set)
+    L.indices[a] = (uint32_t)e;
+    atomicAdd(&s_count[e], 1);
+  }
+  __syncthreads();
+  if (tid == 0) {
+    int o = 0, it = 0;
+    for (int e = 0; e < L.n_experts; ++e) {
+      s_off[e] = o;
+      s_item[e] = it;
+      o += s_count[e];
+      it += (s_count[e] + tile_rows - 1) / tile_rows;
+    }
+    s_off[L.n_experts] = o;
+    *L.n_items = it;
+  }
+  __syncthreads();
+  for (int e = tid; e <= L.n_experts; e += blockDim.x) L.offsets[e] = s_off[e];
+  for (int e = tid; e < L.n_experts; e += blockDim.x) {
+    const int cnt = s_count[e];
+    for (int t = 0, i = s_item[e]; t < cnt; t += tile_rows, ++i) L.items[i] = make_int4(e, s_off[e] + t, min(tile_rows, cnt - t), 0);
+  }
+}
+
+__global__ void __launch_bounds__(1024) table_place_kernel(const MoeTableLayer* __restrict__ layers, int n_tokens) {
+  const MoeTableLayer L = layers[blockIdx.y];
+  if ((int)blockIdx.x >= L.n_experts) return;
+  place_assignments(L.indices, n_tokens * L.top, L.offsets, L.order, L.inv_order);
+}
+
+// Rows of x in the experts' order, 16 bytes at a time.
+__global__ void __launch_bounds__(128) gather_rows_by_order_kernel(const uint4* __restrict__ x, const int* __restrict__ order, int top, int vecs,
+                                                                   uint4* __restrict__ out) {
+  const uint4* src = x + (size_t)(order[blockIdx.x] / top) * vecs;
+  uint4* dst = out + (size_t)blockIdx.x * vecs;
+  for (int i = threadIdx.x; i < vecs; i += blockDim.x) dst[i] = src[i];
 }
 
 // row_scales[p] = weights[order[p]] alone (the rows themselves are read in place by the matmul).
@@ -314,6 +371,27 @@ __global__ void combine_kernel(const __nv_bfloat16* __restrict__ y_sorted, const
 }
 
 }  // namespace
+
+int b200_moe_max_experts() { return kMaxExperts; }
+int b200_moe_max_top() { return kMaxTopK; }
+
+b200_status b200_moe_table_plan(const MoeTableLayer* d_layers, int n_layers, int most_experts, const uint32_t* d_tokens, int n_tokens, int vocab,
+                                int tile_rows, void* stream) {
+  if (n_layers <= 0 || n_tokens <= 0) return B200_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  table_route_kernel<<<n_layers, 1024, 0, s>>>(d_layers, d_tokens, n_tokens, vocab, tile_rows);
+  B200_LAUNCH_CHECK();
+  table_place_kernel<<<dim3(most_experts, n_layers), 1024, 0, s>>>(d_layers, n_tokens);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+b200_status b200_moe_gather_order(const void* d_x, const int* d_order, int top, int n_assign, int width, void* d_out, void* stream) {
+  if (n_assign <= 0) return B200_OK;
+  gather_rows_by_order_kernel<<<n_assign, 128, 0, (cudaStream_t)stream>>>((const uint4*)d_x, d_order, top, width / 8, (uint4*)d_out);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
 
 extern "C" {
 

@@ -96,6 +96,10 @@ class PagedKVCache:
         arr = (C.c_int32 * len(ids))(*ids)
         _lib.check(lib.b200_kv_set_free_order(self._h, arr, len(ids)))
 
+    def state_bytes(self) -> int:
+        """Recurrent state per sequence slot (0: everything a sequence holds is in its pages)."""
+        return int(lib.b200_kv_state_bytes(self._h))
+
     def free_count(self) -> int:
         out = C.c_int32()
         _lib.check(lib.b200_kv_free_count(self._h, C.byref(out)))
@@ -222,8 +226,8 @@ class PagedKVCache:
 
 
 class LayeredKVCache(PagedKVCache):
-    """A page pool whose layers have shapes of their own: `layers` is [(kv heads, key width, value width)], bf16 or f32 pages.
-    Rows are written and read by the decoder step; everything the allocator does works as on any pool."""
+    """A page pool whose layers have shapes of their own: `layers` is [(kv heads, key width, value width)] with, where they are
+    set, values_in_keys and state_elems behind (b200_kv_layer); bf16 or f32 pages.  Rows are written and read by the decoder step; everything the allocator does works as on any pool."""
 
     def __init__(self, layers: Sequence[Sequence[int]], n_pages: int, max_seqs: int, max_pages_per_seq: int, n_q_heads: int,
                  max_rows: int = 4096, kv_dtype: int = KV_BF16, attn_scratch_chunks: int = 0):
@@ -232,15 +236,15 @@ class LayeredKVCache(PagedKVCache):
         h = C.c_void_p()
         _lib.check(lib.b200_kv_create_layers(C.byref(cfg), arr, C.byref(h)))
         cfg.n_kv_heads = max(l[0] for l in layers)
-        self._h, self.cfg, self.layers = h.value, cfg, [tuple(l) for l in layers]
+        self._h, self.cfg, self.layers = h.value, cfg, [tuple(l) + (0,) * (5 - len(l)) for l in layers]
 
     def layer_shape(self, layer: int):
-        return self.layers[layer]
+        return self.layers[layer][:3]
 
     def page_shapes(self, layer: int):  # stored rows are a multiple of 16 elements wide
-        h, kd, vd = self.layers[layer]
+        h, kd, vd, in_keys, _ = self.layers[layer]
         up = lambda n: (n + 15) // 16 * 16
-        return (h, 32, up(kd)), (h, 32, up(vd))
+        return (h, 32, up(kd)), (h, 32, 0 if in_keys else up(vd))
 
     def _element(self):
         return torch.float32 if self.cfg.kv_dtype == KV_F32 else torch.bfloat16
@@ -563,9 +567,12 @@ class LlamaModel(Model):
 
 
 DT_BF16, DT_F32 = 0, 1
-DEC_QKV_BIAS, DEC_QK_NORM, DEC_DISTANCE_BIAS, DEC_SINK, DEC_POST_NORM = 1, 2, 4, 8, 16
+DEC_QKV_BIAS, DEC_QK_NORM, DEC_DISTANCE_BIAS, DEC_SINK, DEC_POST_NORM, DEC_PARALLEL = 1, 2, 4, 8, 16, 32
+DEC_SCALAR_NORM, DEC_DEPTH_AVERAGE = 1, 2  # of the whole stack
+MIX_ATTENTION, MIX_LATENT, MIX_GLA = 0, 1, 2
 DEC_TENSORS = ("q", "k", "v", "o", "gate", "up", "down", "head", "loop_in", "embed", "q_bias", "k_bias", "v_bias", "sink", "norm1", "norm2",
-               "postnorm1", "postnorm2", "final_norm")
+               "postnorm1", "postnorm2", "final_norm", "dkv", "dkv_norm", "uk", "uv", "out_gate", "a1", "a2", "a2_bias", "head_norm",
+               "expert_gate", "expert_up", "expert_down", "depth")
 
 
 class DecoderModel(Model):
@@ -573,10 +580,10 @@ class DecoderModel(Model):
     b200_decoder_layer; `loop` is (start, stop, times) or None."""
 
     def __init__(self, hidden: int, vocab: int, layers: Sequence[dict], norm_eps: float, embed_scale: float = 1.0, loop=None,
-                 dtype: int = DT_BF16, max_rows: int = 2048, max_reqs: int = 64, max_seqs: int = 64):
+                 dtype: int = DT_BF16, max_rows: int = 2048, max_reqs: int = 64, max_seqs: int = 64, logit_scale: float = 1.0, flags: int = 0):
         start, stop, times = loop if loop else (0, 0, 0)
         self.cfg = _lib.DecoderConfig(len(layers), hidden, vocab, start, stop, times, dtype, max_rows, max_reqs, max_seqs, norm_eps,
-                                      embed_scale)
+                                      embed_scale, logit_scale, flags)
         arr = (_lib.DecoderLayer * max(len(layers), 1))(*[_lib.DecoderLayer(**l) for l in layers])
         h = C.c_void_p()
         _lib.check(lib.b200_decoder_create(C.byref(self.cfg), arr, C.byref(h)))
@@ -596,6 +603,11 @@ class DecoderModel(Model):
         t = np.ascontiguousarray(bf16_bits, np.uint16)
         _lib.check(lib.b200_decoder_set_tensor(self._h, layer, DEC_TENSORS.index(which), t.ctypes.data, t.size))
 
+    def set_table(self, layer: int, table: np.ndarray):
+        """Experts of every token id: int [vocab, top]."""
+        t = np.ascontiguousarray(table, np.int32)
+        _lib.check(lib.b200_decoder_set_table(self._h, layer, t.ctypes.data_as(C.POINTER(C.c_int32)), t.size))
+
     def finalize(self):
         _lib.check(lib.b200_decoder_finalize(self._h))
 
@@ -603,11 +615,11 @@ class DecoderModel(Model):
         _lib.check(lib.b200_decoder_random_init(self._h, seed))
 
     def cache_layers(self):
-        """[(kv heads, key width, value width)] of the cache layers, one per layer run."""
+        """[(kv heads, key width, value width, values in keys, state elements)] of the cache layers, one per layer run."""
         n = lib.b200_decoder_cache_layers(self._h, None, 0)
         arr = (_lib.KvLayer * n)()
         lib.b200_decoder_cache_layers(self._h, arr, n)
-        return [(l.n_kv_heads, l.key_dim, l.value_dim) for l in arr]
+        return [(l.n_kv_heads, l.key_dim, l.value_dim, l.values_in_keys, l.state_elems) for l in arr]
 
     def make_cache(self, n_pages: int, max_seqs: int, max_pages_per_seq: int, max_rows: Optional[int] = None) -> LayeredKVCache:
         return LayeredKVCache(self.cache_layers(), n_pages, max_seqs, max_pages_per_seq, max(l["n_heads"] for l in self.layers),

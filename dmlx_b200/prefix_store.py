@@ -77,6 +77,8 @@ class PrefixDiskStore:
     def save_prefix(self, kv, seq: int, token_ids: Sequence[int]) -> int:
         """Store every full block of `seq` (holding the K/V of token_ids) that is not on disk yet.
         Returns the number of blocks written."""
+        if kv.state_bytes():
+            raise ValueError("a model with recurrent state has no prefix pages: its state belongs to a whole sequence")
         table = kv.block_table(seq)
         n_full = min(kv.seq_len(seq), len(token_ids)) // self.block_size
         written = 0
@@ -89,6 +91,8 @@ class PrefixDiskStore:
     def restore_prefix(self, kv, seq: int, token_ids: Sequence[int]) -> int:
         """Fill the empty slot `seq` with the longest run of leading blocks of token_ids found on disk
         (at least one prompt token is always left to compute).  Returns the tokens restored."""
+        if kv.state_bytes():
+            return 0
         c = kv.cfg
         hashes = chain_hashes(token_ids, self.block_size)
         n = 0

@@ -591,10 +591,16 @@ b200_status b200_model_logits(b200_model* m, int32_t first, int32_t n, float* h_
 /* A decoder-only stack whose layers are described one by one (no reference counterpart; the reference has one file per
  * model family).  Every mechanism is a parameter of its layer, and a layer that does not set it does not have it:
  *   x = embed[token] * embed_scale, kept in f32 between the layers;
- *   x += postnorm1(attention(norm1(x))); x += postnorm2(W_down(silu(W_gate h) * W_up h)), h = norm2(x);
+ *   x += postnorm1(mixer(norm1(x))); x += postnorm2(ff(h)), h = norm2(x);
+ *   with B200_DEC_PARALLEL instead x += mixer(h) + ff(h), h = norm1(x);
+ *   mixer: grouped-query attention, latent attention or gated linear attention (B200_MIX_*);
+ *   ff(h) = W_down(silu(W_gate h) * W_up h) of width ffn, plus 1 / top_k times the same of each expert the token's id has in
+ *   the layer's table;
+ *   with B200_DEC_DEPTH_AVERAGE what follows layer i is sum_j depth[j] X_j over the embedding output X_0 and the results X_1 ..
+ *   X_(i+1) of the layers so far;
  *   layers loop_start .. loop_stop-1 run loop_times times with the same weights, every pass with cache layers of its own,
  *   and each pass opens with x = W_in [x ; x0], x0 the embedding output;
- *   logits = head(final_norm(x)), f32.
+ *   logits = head(final_norm(x)) * logit_scale, f32.
  * Norms, scores, softmax and the residual are f32; matrix operands are bf16, or f32 throughout with
  * dtype = B200_DT_F32. */
 enum { B200_DT_BF16 = 0, B200_DT_F32 = 1 };
@@ -603,32 +609,57 @@ enum {
   B200_DEC_QK_NORM = 2,        /* q and k divided by their root mean square per head (no weight) */
   B200_DEC_DISTANCE_BIAS = 4,  /* score -= 2^(-8 (h + 1) / n_heads) * (i - j) */
   B200_DEC_SINK = 8,           /* learned sink per query head in the softmax's denominator */
-  B200_DEC_POST_NORM = 16      /* RMSNorm on each sublayer's output before the residual add */
+  B200_DEC_POST_NORM = 16,     /* RMSNorm on each sublayer's output before the residual add */
+  B200_DEC_PARALLEL = 32,      /* mixer and feed-forward read the same norm and are added together */
+  /* of the whole stack (b200_decoder_config.flags) */
+  B200_DEC_SCALAR_NORM = 1,    /* a norm's weight is one number for all coordinates */
+  B200_DEC_DEPTH_AVERAGE = 2   /* weighted average over depth after every layer */
 };
+/* B200_MIX_ATTENTION: softmax attention, keys and values per kv head.
+ * B200_MIX_LATENT: keys and values of all heads come from one latent of kv_rank numbers per token, c = norm(W_dkv h); per head
+ *   the key is W_uk c (key_dim wide) beside rot_dim rotated numbers shared by all heads, the value W_uv c (value_dim).  Cached are
+ *   c and the rotated part.  Rotation: pairs (2i, 2i+1), angle position * rot_base^(-2i / rot_dim).
+ * B200_MIX_GLA: state S [key_dim][value_dim] per head, S <- diag(alpha) S + k v^T, o = S^T q key_dim^(-1/2), alpha =
+ *   sigmoid(W_a2 W_a1 h + b)^(1 / decay_tau) with decay_rank rows in W_a1; rms_norm(o) * w * silu(W_g h). */
+enum { B200_MIX_ATTENTION = 0, B200_MIX_LATENT = 1, B200_MIX_GLA = 2 };
 typedef struct b200_decoder_layer {
   int32_t n_heads, n_kv_heads, key_dim, value_dim;
   int32_t window; /* position i sees j with 0 <= i - j < window; 0 = the whole context */
-  int32_t ffn;    /* 0 = the layer has no feed-forward */
+  int32_t ffn;    /* width of the dense feed-forward (beside experts: of the shared expert); 0 = none */
   int32_t flags;  /* B200_DEC_* */
   float scale;    /* score = (q . k) * scale */
+  int32_t mixer;  /* B200_MIX_* */
+  int32_t kv_rank, rot_dim;                 /* latent attention */
+  float rot_base;
+  int32_t decay_rank;                       /* gated linear attention */
+  float decay_tau;
+  int32_t n_experts, top_k, expert_ffn;     /* experts by token id (b200_decoder_set_table); n_experts 0 = none */
 } b200_decoder_layer;
 typedef struct b200_decoder_config {
   int32_t n_layers, hidden, vocab;
   int32_t loop_start, loop_stop, loop_times; /* loop_times = 0: no loop */
   int32_t dtype;                             /* B200_DT_* */
   int32_t max_rows, max_reqs, max_seqs;
-  float norm_eps, embed_scale;
+  float norm_eps, embed_scale, logit_scale;
+  int32_t flags; /* B200_DEC_SCALAR_NORM, B200_DEC_DEPTH_AVERAGE */
 } b200_decoder_config;
 typedef struct b200_decoder b200_decoder;
 enum { B200_DEC_W_Q = 0, B200_DEC_W_K = 1, B200_DEC_W_V = 2, B200_DEC_W_O = 3, B200_DEC_W_GATE = 4, B200_DEC_W_UP = 5,
        B200_DEC_W_DOWN = 6, B200_DEC_W_HEAD = 7, B200_DEC_W_LOOP_IN = 8, B200_DEC_W_EMBED = 9, B200_DEC_B_Q = 10,
        B200_DEC_B_K = 11, B200_DEC_B_V = 12, B200_DEC_W_SINK = 13, B200_DEC_NORM1 = 14, B200_DEC_NORM2 = 15,
-       B200_DEC_POSTNORM1 = 16, B200_DEC_POSTNORM2 = 17, B200_DEC_FINAL_NORM = 18 };
+       B200_DEC_POSTNORM1 = 16, B200_DEC_POSTNORM2 = 17, B200_DEC_FINAL_NORM = 18,
+       B200_DEC_W_DKV = 19, B200_DEC_DKV_NORM = 20, B200_DEC_W_UK = 21, B200_DEC_W_UV = 22,
+       B200_DEC_W_OUT_GATE = 23, B200_DEC_W_A1 = 24, B200_DEC_W_A2 = 25, B200_DEC_B_A2 = 26, B200_DEC_HEAD_NORM = 27,
+       /* experts stacked: [n_experts][expert_ffn][hidden], down [n_experts][hidden][expert_ffn] */
+       B200_DEC_W_EXPERT_GATE = 28, B200_DEC_W_EXPERT_UP = 29, B200_DEC_W_EXPERT_DOWN = 30,
+       B200_DEC_DEPTH = 31 /* [layer + 2] */ };
 b200_status b200_decoder_create(const b200_decoder_config* cfg, const b200_decoder_layer* layers, b200_decoder** out);
 void b200_decoder_destroy(b200_decoder* m);
 /* One tensor, bf16 on the host, matrices [out, in]; n_elems is checked against the shape the configuration gives.
  * `layer` is ignored for embed, head, loop_in and final_norm. */
 b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t which, const void* h_bf16, uint64_t n_elems);
+/* Experts of every token id in one layer: [vocab][top_k] expert numbers, all different within a row. */
+b200_status b200_decoder_set_table(b200_decoder* m, int32_t layer, const int32_t* h_table, uint64_t n_elems);
 /* Fuses q/k/v and gate/up; fails, naming it, if a tensor the configuration needs was not set. */
 b200_status b200_decoder_finalize(b200_decoder* m);
 /* Synthetic weights generated on the device (benchmarks).  Matrix sizes must be multiples of 128. */
@@ -639,7 +670,8 @@ int32_t b200_decoder_cache_layers(const b200_decoder* m, b200_kv_layer* out, int
  * (checks of a model against an oracle). */
 b200_status b200_decoder_record_layers(b200_decoder* m, int32_t on);
 b200_status b200_decoder_recorded_layers(b200_decoder* m, int32_t rows, float* h_out);
-/* 1 (default): attention on the tensor cores where the layer's shape allows it (bf16, widths up to 256); 0: the
+/* 1 (default): attention (and gated linear attention of longer portions) on the tensor cores where the layer's shape allows it
+ * (bf16); 0: the
  * CUDA-core kernel, which serves every shape and f32 (tests compare the two). */
 void b200_decoder_set_attn_mma(b200_decoder* m, int32_t on);
 b200_model* b200_decoder_model(b200_decoder* m);
