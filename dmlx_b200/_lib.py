@@ -275,6 +275,11 @@ class DecoderConfig(C.Structure):
                                    "max_seqs")] + [("norm_eps", f32), ("embed_scale", f32), ("logit_scale", f32), ("flags", i32)]
 
 
+class GlaShape(C.Structure):
+    _fields_ = [(n, i32) for n in ("heads", "key_dim", "value_dim", "decay_rank")] + [(n, f32) for n in ("q_scale", "inv_tau", "eps")]
+
+
+_sig("b200_decoder_gla", i32, vp, i32, P(GlaShape), vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, vp, i32, vp)
 _sig("b200_kv_create_layers", i32, P(KvConfig), P(KvLayer), P(vp))
 _sig("b200_argmax_f32", i32, vp, i32, i32, vp, vp)
 _sig("b200_qmm_f32", i32, vp, vp, i32, vp, i32, i32, i32, vp)

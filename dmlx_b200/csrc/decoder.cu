@@ -1215,4 +1215,27 @@ b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, 
   return b200_window_attn_run(kv, c, d_row_seq, d_row_ctx, total_rows, mma != 0, stream);
 }
 
+b200_status b200_decoder_gla(b200_kv* kv, int32_t layer, const b200_gla_shape* z, const void* d_rows, int32_t stride, const float* d_a2,
+                             const float* d_a2_bias, const float* d_norm, const int32_t* d_cu, const int32_t* d_row_seq,
+                             const int32_t* d_positions, int32_t n_req, int32_t total_rows, int32_t chunked, void* d_out, int32_t out_stride,
+                             void* stream) {
+  if (n_req <= 0 || total_rows <= 0) return B200_OK;
+  GlaScratch g;
+  g.max_rows = total_rows;
+  g.max_reqs = n_req;
+  if (b200_gla_takes_chunks(z->key_dim, z->value_dim, kv->dev.elem_bytes)) g.need(z->heads, z->key_dim, z->value_dim);
+  if (!g.alloc()) { g.free(); b200_set_error("decoder_gla: no memory for %d rows", total_rows); return B200_ERR_CUDA; }
+  GlaCall c;
+  c.layer = layer; c.heads = z->heads; c.dk = z->key_dim; c.dv = z->value_dim; c.rank = z->decay_rank;
+  c.src.y = d_rows; c.src.y_stride = stride;
+  c.a2 = d_a2; c.a2_bias = d_a2_bias; c.norm = d_norm; c.q_scale = z->q_scale; c.inv_tau = z->inv_tau; c.eps = z->eps;
+  c.out = d_out; c.out_stride = out_stride;
+  b200_status st = b200_gla_plan(g, d_cu, n_req, total_rows, stream);
+  if (st == B200_OK) st = b200_gla_run(kv, g, c, d_cu, d_row_seq, d_positions, n_req, total_rows, chunked != 0, stream);
+  const cudaError_t e = cudaStreamSynchronize((cudaStream_t)stream);
+  g.free();
+  if (st == B200_OK && e != cudaSuccess) { b200_set_error("decoder_gla: %s", cudaGetErrorString(e)); return B200_ERR_CUDA; }
+  return st;
+}
+
 }  // extern "C"

@@ -260,6 +260,17 @@ class LayeredKVCache(PagedKVCache):
                                         _ptr(positions), _ptr(row_seq), rows.shape[0], _stream()))
         return q
 
+    def gla(self, layer: int, rows: torch.Tensor, a2: torch.Tensor, a2_bias: torch.Tensor, norm: torch.Tensor, heads: int, tau: float, eps: float,
+            cu: torch.Tensor, row_seq: torch.Tensor, positions: torch.Tensor, chunked: bool = True) -> torch.Tensor:
+        """b200_decoder_gla on projection rows [q | k | v | g | a1] -> [T, heads, value width]; the layer's state moves on."""
+        rank, vd = a2.shape[1], norm.shape[0]
+        kd = a2.shape[0] // heads
+        shape = _lib.GlaShape(heads, kd, vd, rank, kd ** -0.5, 1.0 / tau, eps)
+        out = torch.zeros((rows.shape[0], heads, vd), dtype=rows.dtype, device=rows.device)
+        _lib.check(lib.b200_decoder_gla(self._h, layer, C.byref(shape), _ptr(rows), rows.shape[1], _ptr(a2), _ptr(a2_bias), _ptr(norm), _ptr(cu),
+                                        _ptr(row_seq), _ptr(positions), cu.shape[0] - 1, rows.shape[0], int(chunked), _ptr(out), heads * vd, _stream()))
+        return out
+
     def window_attention(self, layer: int, q: torch.Tensor, row_seq: torch.Tensor, row_ctx: torch.Tensor, scale: float, window: int = 0,
                          slopes: Optional[np.ndarray] = None, sinks: Optional[np.ndarray] = None,
                          mma: bool = True) -> torch.Tensor:

@@ -689,6 +689,17 @@ b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, 
                                    const float* d_slopes_log2, const float* d_sinks_log2, const int32_t* d_row_seq,
                                    const int32_t* d_row_ctx, int32_t total_rows, int32_t mma, void* d_out,
                                    int32_t out_stride, void* stream);
+/* Gated linear attention of one layer over the rows of a batch, for hosts that drive the layers themselves: d_rows [rows][q | k | v |
+ * g | a1] in the pool's element type, `stride` elements apart; d_cu [n_req + 1] the requests' first rows, d_row_seq and d_positions
+ * per row (a request whose first row stands at position 0 starts from a zero state).  chunked = 0: token by token. */
+typedef struct b200_gla_shape {
+  int32_t heads, key_dim, value_dim, decay_rank;
+  float q_scale, inv_tau, eps;
+} b200_gla_shape;
+b200_status b200_decoder_gla(b200_kv* kv, int32_t layer, const b200_gla_shape* shape, const void* d_rows, int32_t stride, const float* d_a2,
+                             const float* d_a2_bias, const float* d_norm, const int32_t* d_cu, const int32_t* d_row_seq,
+                             const int32_t* d_positions, int32_t n_req, int32_t total_rows, int32_t chunked, void* d_out, int32_t out_stride,
+                             void* stream);
 
 /* ---- engine step: schedule -> pack -> model step -> postprocess ------------------------------- */
 /* The Engine_Step loop of src/scheduler.zig:7-10 wired to a forward pass (the reference leaves

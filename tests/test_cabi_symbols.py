@@ -59,7 +59,7 @@ def test_struct_layouts_match_the_header(tmp_path):
         "b200_pack_desc": _lib.PackDesc, "b200_token_output": _lib.TokenOutput, "b200_sample_params": _lib.SampleParams,
         "b200_kv_config": _lib.KvConfig, "b200_llama_config": _lib.LlamaConfig, "b200_qmm_partials": _lib.QmmPartials,
         "b200_kv_layer": _lib.KvLayer, "b200_model_info": _lib.ModelInfo, "b200_decoder_layer": _lib.DecoderLayer,
-        "b200_decoder_config": _lib.DecoderConfig, "b200_moe_config": _lib.MoeConfig, "b200_ep_watch_ops": _lib.EpWatchOps,
+        "b200_decoder_config": _lib.DecoderConfig, "b200_gla_shape": _lib.GlaShape, "b200_moe_config": _lib.MoeConfig, "b200_ep_watch_ops": _lib.EpWatchOps,
     }
     lines = ['#include <stdio.h>', '#include <stddef.h>', '#include "dmlx_b200.h"', 'int main(void) {']
     for cname, cls in pairs.items():
