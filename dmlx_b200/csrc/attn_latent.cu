@@ -104,3 +104,346 @@ b200_status b200_latent_prep(b200_kv* kv, const LatentPrep& p, const int32_t* d_
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
+
+template <int NR>
+__global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __grid_constant__ CUtensorMap kmap, LatentArgs la) {
+  const WinArgs& a = la.w;
+  extern __shared__ unsigned char latent_dyn[];
+  unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(latent_dyn) + 1023) & ~(uintptr_t)1023);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, stages = a.stages, n_kb = la.n_kb, n_mc = la.n_mc;
+  const int stage_bytes = n_kb * kBoxBytes;
+  unsigned char* qbuf = smem + (size_t)stages * stage_bytes;  // [box][NR rows][128 B]
+  unsigned char* pbuf = qbuf + (size_t)n_kb * NR * 128;       // [key][NR values | NR remainders]
+  LatentShared<NR>& sh = *reinterpret_cast<LatentShared<NR>*>(pbuf + kPBytes);
+  const int n_groups = a.hdr[0], n_items = a.chunk_start[n_groups] * a.n_blocks;
+  if (tid == 0) {
+    for (int s = 0; s < stages; ++s) { ptx::mbar_init(&sh.k_full[s], 1); ptx::mbar_init(&sh.k_free[s], 1); }
+    ptx::mbar_init(&sh.s_full[0], 1);
+    ptx::mbar_init(&sh.s_full[1], 1);
+    ptx::mbar_init(&sh.p_ready, 128);
+    ptx::mbar_init(&sh.pv_done, 1);
+    ptx::mbar_init(&sh.q_full, 128);
+    ptx::mbar_fence_init();
+  }
+  if (warp == 1) {
+    ptx::tmem_alloc(&sh.tmem, la.tmem_cols);
+    ptx::tmem_relinquish();
+  }
+  ptx::tc_fence_before_sync();
+  __syncthreads();
+  ptx::tc_fence_after_sync();
+  const uint32_t tmem = sh.tmem, tmem_o = tmem + 2 * NR;  // S twice, then O: n_mc x [NR of the values | NR of the remainders]
+  bool ok = true;
+
+  if (warp == 0) {
+    if (lane == 0) {  // ---- loads ----
+      int s = 0;
+      uint32_t ph = 0, issued = 0;
+      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x) {
+        const WinItem it = decode_item(a, item, n_groups);
+        const int* table = a.d.block_table + (size_t)it.seq * a.d.max_pages_per_seq;
+        for (int pg = it.page_begin; pg < it.page_end; pg += kTilePages) {
+          const int pages = min(kTilePages, it.page_end - pg);
+          ok = wait(&sh.k_free[s], ph ^ 1u);
+          if (!ok) break;
+          ptx::mbar_expect_tx(&sh.k_full[s], pages * n_kb * 4096);
+          for (int p = 0; p < pages; ++p) {
+            const int row0 = table[pg + p] * 32;
+            for (int b = 0; b < n_kb; ++b)
+              ptx::tma_load_2d(smem + (size_t)s * stage_bytes + b * kBoxBytes + p * 4096, &kmap, b * 64, row0, &sh.k_full[s]);
+          }
+          ++issued;
+          if (++s == stages) { s = 0; ph ^= 1u; }
+        }
+      }
+      if (!ok) {  // leave no copy in flight behind
+        for (uint32_t i = issued > (uint32_t)stages ? issued - stages : 0; i < issued; ++i) wait(&sh.k_full[i % stages], (i / stages) & 1u);
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {  // ---- matrix products ----
+      const uint32_t id_s = ptx::umma_idesc_bf16(128, NR), id_o = ptx::umma_idesc_bf16(128, 2 * NR) | ptx::kUmmaAMn | ptx::kUmmaBMn;
+      const int n_ks = a.L.kd / 16;
+      const uint32_t q0 = ptx::smem_u32(qbuf), p0 = ptx::smem_u32(pbuf), t0 = ptx::smem_u32(smem);
+      int sc = 0, sp = 0;  // stage of the next tile to score, of the next to sum
+      uint32_t phc = 0, n_scored = 0, n_summed = 0, n_item = 0;
+      auto score = [&]() {  // the next tile's S^T
+        ok = wait(&sh.k_full[sc], phc);
+        if (!ok) return;
+        ptx::tc_fence_after_sync();
+        const uint32_t kt = t0 + sc * stage_bytes, dst = tmem + (n_scored & 1u) * NR;
+        for (int ks = 0; ks < n_ks; ++ks) {
+          const uint64_t da = ptx::umma_desc_k_sw128(kt + (ks >> 2) * kBoxBytes) + 2 * (ks & 3);
+          const uint64_t db = ptx::umma_desc_k_sw128(q0 + (ks >> 2) * NR * 128) + 2 * (ks & 3);
+          ptx::umma_bf16(dst, da, db, id_s, ks > 0 ? 1u : 0u);
+        }
+        ptx::umma_commit(&sh.s_full[n_scored & 1u]);
+        ++n_scored;
+        if (++sc == stages) { sc = 0; phc ^= 1u; }
+      };
+      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
+        const WinItem it = decode_item(a, item, n_groups);
+        const int tiles = (it.page_end - it.page_begin + kTilePages - 1) / kTilePages;
+        ok = wait(&sh.q_full, n_item & 1u);
+        if (!ok) break;
+        score();
+        for (int j = 0; j < tiles && ok; ++j) {
+          if (stages > 1 && j + 1 < tiles) score();  // ahead of this tile's softmax
+          if (!ok) break;
+          ok = wait(&sh.p_ready, n_summed & 1u);
+          if (!ok) break;
+          ptx::tc_fence_after_sync();
+          const int pages = min(kTilePages, it.page_end - it.page_begin - j * kTilePages);
+          const uint32_t kt = t0 + sp * stage_bytes;
+          for (int mc = 0; mc < n_mc; ++mc) {
+            for (int ks = 0; ks < 2 * pages; ++ks) {
+              const uint64_t da = ptx::umma_desc_mn_sw128(kt + 2 * mc * kBoxBytes + ks * 2048, kBoxBytes);
+              const uint64_t db = ptx::umma_desc_mn_sw128(p0 + ks * 2048, kPBytes);
+              ptx::umma_bf16(tmem_o + mc * 2 * NR, da, db, id_o, (j > 0 || ks > 0) ? 1u : 0u);
+            }
+          }
+          ptx::umma_commit(&sh.k_free[sp]);
+          ptx::umma_commit(&sh.pv_done);
+          ++n_summed;
+          if (++sp == stages) sp = 0;
+          if (stages == 1 && j + 1 < tiles) score();
+        }
+      }
+    }
+  } else if (warp >= 4) {
+    // ---- softmax: thread = key of the tile = tensor-memory lane ----
+    const int key = tid - 128, quarter = warp - 4;
+    const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
+    uint32_t n_tile = 0, n_pv = 0;  // tiles scored / summed so far (phases of the barriers)
+    bool dead = false;              // some thread's wait ran out: decided together, so that all leave
+    for (int item = blockIdx.x; item < n_items && !dead; item += gridDim.x) {
+      const WinItem it = decode_item(a, item, n_groups);
+      const int hb = a.head_block, h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0);
+      const int vecs = a.L.kd / 8;
+      for (int i = key; i < NR * vecs; i += 128) {
+        const int r = i / vecs, c = i - r * vecs, tok = r / hb, head = r - tok * hb;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (tok < it.n_rows && head < heads_here)
+          v = *reinterpret_cast<const uint4*>(a.q + (size_t)(it.first_row + tok) * a.q_stride + (size_t)(h0 + head) * a.L.kd + c * 8);
+        *reinterpret_cast<uint4*>(qbuf + (c >> 3) * NR * 128 + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+      }
+      if (key < NR) {
+        const int tok = key / hb, head = key - tok * hb;
+        sh.ctx[key] = tok < it.n_rows && head < heads_here ? it.ctx0 + tok : 0;
+        sh.m[key] = kAttnNone;
+      }
+      ptx::fence_proxy_async_smem();
+      ptx::mbar_arrive(&sh.q_full);
+      float l[NR];
+#pragma unroll
+      for (int r = 0; r < NR; ++r) l[r] = 0.f;
+      for (int pg = it.page_begin; pg < it.page_end; pg += kTilePages) {
+        const int pages = min(kTilePages, it.page_end - pg), tok0 = pg * 32;
+        ok = wait(&sh.s_full[n_tile & 1u], (n_tile >> 1) & 1u) && ok;
+        ptx::tc_fence_after_sync();
+        __syncwarp();
+        float v[NR];
+        load_rows<NR>(tmem + lanes + (n_tile & 1u) * NR, v);
+        ++n_tile;
+        const bool edge = tok0 + kTileKeys > it.ctx0 || pages < kTilePages;
+        softmax_sync_and(true);  // sh.ctx, sh.m of a new item are in place; the previous tile's sh.m has been read
+        {
+          float w[NR];
+          const bool in_tile = key < pages * 32;
+#pragma unroll
+          for (int r = 0; r < NR; ++r) {
+            v[r] *= a.scale_log2;
+            if (edge) v[r] = in_tile && tok0 + key < sh.ctx[r] ? v[r] : kAttnNone;
+            w[r] = v[r];
+          }
+          const float mx = transpose_reduce<NR, true>(w, lane);
+          if (NR == 32) sh.red[quarter][lane] = mx;
+          else if ((lane & 1) == 0) sh.red[quarter][lane >> 1] = mx;
+        }
+        if (!softmax_sync_and(ok)) { dead = true; break; }
+        bool moved = false;
+        if (key < NR) {
+          const float m_old = sh.m[key], mx = fmaxf(fmaxf(sh.red[0][key], sh.red[1][key]), fmaxf(sh.red[2][key], sh.red[3][key]));
+          moved = mx > m_old + kGrow;
+          sh.corr[key] = moved ? ex2(m_old - mx) : 1.f;
+          if (moved) sh.m[key] = mx;
+        }
+        const bool first = pg == it.page_begin;
+        const bool rescale = softmax_sync_or(moved) && !first;
+        if (!first) {  // P and O are the previous tile's until its product is done
+          ok = wait(&sh.pv_done, n_pv & 1u) && ok;
+          ++n_pv;
+          ptx::tc_fence_after_sync();
+          __syncwarp();
+        }
+        if (rescale) {
+          float corr[NR];
+#pragma unroll
+          for (int r = 0; r < NR; ++r) { corr[r] = sh.corr[r]; l[r] *= corr[r]; }
+          for (int c = 0; c < n_mc * 2; ++c) {
+#pragma unroll
+            for (int h = 0; h < NR / 16; ++h) {
+              uint32_t o[16];
+              ptx::tmem_ld16(tmem_o + lanes + c * NR + h * 16, o);
+              ptx::tmem_ld_wait();
+#pragma unroll
+              for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * corr[h * 16 + e]);
+              ptx::tmem_st16(tmem_o + lanes + c * NR + h * 16, o);
+            }
+          }
+          ptx::tmem_st_wait();
+        }
+#pragma unroll
+        for (int r = 0; r < NR; r += 8) {
+          uint32_t hi[4], lo[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            float p[2];
+#pragma unroll
+            for (int f = 0; f < 2; ++f) {
+              const float x = v[r + 2 * e + f];
+              p[f] = x > kAttnNone ? ex2(x - sh.m[r + 2 * e + f]) : 0.f;
+              l[r + 2 * e + f] += p[f];
+            }
+            const __nv_bfloat162 h2 = __floats2bfloat162_rn(p[0], p[1]);
+            const float2 back = __bfloat1622float2(h2);
+            const __nv_bfloat162 l2 = __floats2bfloat162_rn(p[0] - back.x, p[1] - back.y);
+            hi[e] = *reinterpret_cast<const uint32_t*>(&h2);
+            lo[e] = *reinterpret_cast<const uint32_t*>(&l2);
+          }
+          const int c = r / 8;
+          *reinterpret_cast<uint4*>(pbuf + key * 128 + ((c ^ (key & 7)) << 4)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4*>(pbuf + key * 128 + (((c + NR / 8) ^ (key & 7)) << 4)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        }
+        ptx::fence_proxy_async_smem();
+        ptx::tc_fence_before_sync();
+        ptx::mbar_arrive(&sh.p_ready);
+      }
+      if (dead) break;
+      {
+        const float sum = transpose_reduce<NR, false>(l, lane);
+        if (NR == 32) sh.red[quarter][lane] = sum;
+        else if ((lane & 1) == 0) sh.red[quarter][lane >> 1] = sum;
+      }
+      ok = wait(&sh.pv_done, n_pv & 1u) && ok;
+      ++n_pv;
+      if (!softmax_sync_and(ok)) { dead = true; break; }
+      ptx::tc_fence_after_sync();
+      if (key < NR && sh.ctx[key] > 0) {
+        float sum = sh.red[0][key] + sh.red[1][key] + sh.red[2][key] + sh.red[3][key], f = 1.f;
+        const float m = sh.m[key];
+        const int tok = key / hb, head = key - tok * hb;
+        if (it.slot0 < 0) {
+          if (a.sinks) {
+            const float sk = a.sinks[h0 + head], mm = fmaxf(m, sk);
+            f = exp2f(m - mm);
+            sum = sum * f + exp2f(sk - mm);
+          }
+          sh.l[key] = sum > 0.f ? f / sum : 0.f;
+        } else {
+          const size_t pidx = (size_t)(it.slot0 + tok) * a.n_q_heads + h0 + head;
+          a.part_ml[pidx * 2] = m;
+          a.part_ml[pidx * 2 + 1] = sum;
+        }
+      }
+      softmax_sync_and(true);
+      for (int mc = 0; mc < n_mc; ++mc) {
+        float o[NR];
+        {
+          float lo[NR];
+          load_rows<NR>(tmem_o + lanes + mc * 2 * NR, o);
+          load_rows<NR>(tmem_o + lanes + mc * 2 * NR + NR, lo);
+#pragma unroll
+          for (int r = 0; r < NR; ++r) o[r] += lo[r];
+        }
+        const int dim = mc * 128 + key;
+#pragma unroll
+        for (int r = 0; r < NR; ++r) {
+          const int tok = r / hb, head = r - tok * hb;
+          if (sh.ctx[r] > 0 && dim < a.L.vd) {
+            if (it.slot0 >= 0) a.part_o[((size_t)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd + dim] = o[r];
+            else if (dim < a.L.value_dim)
+              a.out[(size_t)(it.first_row + tok) * a.out_stride + (size_t)(h0 + head) * a.out_head + dim] = __float2bfloat16(o[r] * sh.l[r]);
+          }
+        }
+        __syncwarp();
+      }
+      ptx::tc_fence_before_sync();
+      softmax_sync_and(true);  // sh.ctx and sh.l have been read
+    }
+    ok = ok && !dead;
+  }
+  if (!ok) atomicExch(a.d.state + ST_ATTN_ERR, B200_ERR_DEVICE_FLAGGED);
+  ptx::tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 1) ptx::tmem_dealloc(tmem, la.tmem_cols);
+}
+
+int g_sms = 0;
+constexpr int kSmemLimit = 227 * 1024;
+
+template <int NR>
+size_t smem_of(int n_kb, int stages) {
+  return (size_t)stages * n_kb * kBoxBytes + (size_t)n_kb * NR * 128 + kPBytes + sizeof(LatentShared<NR>) + 1024;
+}
+
+// Rows of a tile: 16 where a decode step would leave more of them empty.
+int rows_of(int heads, int total_rows) { return heads <= 16 && total_rows <= 256 ? 16 : 32; }
+
+template <int NR>
+b200_status launch(const b200_kv* kv, LatentArgs& la, int layer, cudaStream_t s) {
+  int stages = 4;
+  while (stages > 1 && smem_of<NR>(la.n_kb, stages) > kSmemLimit) --stages;
+  la.w.stages = stages;
+  la.tmem_cols = 32;
+  while (la.tmem_cols < (uint32_t)(2 * NR + la.n_mc * 2 * NR)) la.tmem_cols <<= 1;
+  static bool configured = false;
+  if (!configured) {
+    B200_CUDA_TRY(cudaFuncSetAttribute(latent_attn_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit));
+    configured = true;
+  }
+  latent_attn_kernel<NR><<<g_sms, kLatentThreads, smem_of<NR>(la.n_kb, stages), s>>>(kv->lay_kmap[layer], la);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+}  // namespace
+
+bool b200_latent_attn_takes_mma(const b200_kv* kv, int32_t layer) {
+  const KvLayerDev& L = kv->lay[layer];
+  return kv->layered && L.values_in_keys && L.heads == 1 && kv->dev.elem_bytes == 2 && smem_of<32>((L.kd + 63) / 64, 1) <= kSmemLimit &&
+         64 + (L.value_dim + 127) / 128 * 64 <= 512;
+}
+
+b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t heads, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
+                                  void* stream) {
+  if (g_sms == 0) {
+    int dev = 0;
+    B200_CUDA_TRY(cudaGetDevice(&dev));
+    B200_CUDA_TRY(cudaDeviceGetAttribute(&g_sms, cudaDevAttrMultiProcessorCount, dev));
+  }
+  const int rows = rows_of(heads, total_rows);
+  return b200_attn_make_plan(kv, 0, std::max(1, rows / heads), (heads + rows - 1) / rows, g_sms, d_row_seq, d_row_ctx, total_rows, stream);
+}
+
+b200_status b200_latent_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
+                                 void* stream) {
+  const KvLayerDev& L = kv->lay[c.layer];
+  if (c.window != 0 || c.slopes_log2) { b200_set_error("latent attention has no window and no distance bias"); return B200_ERR_UNSUPPORTED; }
+  LatentArgs la;
+  WinArgs& a = la.w;
+  const int rows = rows_of(c.n_q_heads, total_rows), hb = std::min(c.n_q_heads, rows);
+  if (!b200_attn_use_plan(kv, 0, std::max(1, rows / c.n_q_heads), &a)) return B200_ERR_INVALID_ARGUMENT;
+  a.d = kv->dev; a.L = L; a.L.vd = (L.value_dim + 15) / 16 * 16;
+  a.q = (const __nv_bfloat16*)c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx;
+  a.total_rows = total_rows; a.n_q_heads = c.n_q_heads; a.window = 0;
+  a.G = c.n_q_heads; a.head_block = hb; a.n_blocks = (c.n_q_heads + hb - 1) / hb;
+  a.scale_log2 = c.scale * kAttnLog2e;
+  a.slopes = nullptr; a.sinks = c.sinks_log2;
+  a.out = (__nv_bfloat16*)c.out; a.out_stride = c.out_stride; a.out_head = c.out_head_stride > 0 ? c.out_head_stride : L.value_dim;
+  la.n_kb = (L.kd + 63) / 64;
+  la.n_mc = (L.value_dim + 127) / 128;
+  b200_status st = rows == 16 ? launch<16>(kv, la, c.layer, (cudaStream_t)stream) : launch<32>(kv, la, c.layer, (cudaStream_t)stream);
+  if (st != B200_OK) return st;
+  return b200_attn_combine(kv, a, stream);
+}

@@ -20,3 +20,10 @@ struct LatentPrep {
   void* q = nullptr;            // [rows][heads][stored key width]
 };
 b200_status b200_latent_prep(b200_kv* kv, const LatentPrep& p, const int32_t* d_pos, const int32_t* d_row_seq, int rows, void* stream);
+
+// The tensor-core kernel (b200_window_attn_plan / _run come here for layers whose values lie in their keys).
+bool b200_latent_attn_takes_mma(const b200_kv* kv, int32_t layer);
+b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t n_q_heads, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
+                                  void* stream);
+b200_status b200_latent_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
+                                 void* stream);

@@ -20,6 +20,8 @@
 #include <cmath>
 #include <type_traits>
 
+#include "attn_latent.cuh"
+#include "attn_plan.cuh"
 #include "common.h"
 #include "kv_pool.cuh"
 #include "ptx.cuh"
@@ -27,27 +29,7 @@
 
 namespace {
 
-constexpr float kLog2e = 1.4426950408889634f;
-constexpr float kNone = -1e30f;  // running maximum before any key
-
-struct WinArgs {
-  KvDev d;
-  KvLayerDev L;
-  const __nv_bfloat16* q;
-  int q_stride;
-  const int* row_seq;
-  const int* row_ctx;
-  int total_rows, n_q_heads, window;
-  int G, head_block, n_blocks;  // query heads per kv head; heads of one MMA tile; tiles per kv head
-  const int *group_first, *chunk_start, *part_base, *row_group, *hdr;
-  float* part_o;   // [slot][q head][L.vd]
-  float* part_ml;  // [slot][q head][2]
-  float scale_log2;
-  const float *slopes, *sinks;
-  __nv_bfloat16* out;
-  int out_stride;
-  int stages;      // ring slots (pages) per warp
-};
+constexpr float kLog2e = kAttnLog2e, kNone = kAttnNone;
 
 // ---- plan ------------------------------------------------------------------------------------------------
 template <bool MAX>
@@ -76,8 +58,6 @@ __device__ int scan_incl(int v, int* warp_buf) {
   __syncthreads();
   return r;
 }
-
-__device__ __forceinline__ int first_key(int ctx, int window) { return window > 0 ? max(0, ctx - window) : 0; }
 
 // Pages of a group's key range.
 __device__ __forceinline__ int group_pages(int ctx_first, int ctx_last, int window, int page_size) {
@@ -200,35 +180,6 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
 }
 
 // ---- tensor-core kernel ------------------------------------------------------------------------------------
-struct WinItem {
-  int head, block, seq, first_row, n_rows, ctx0, page_begin, page_end, slot0;  // slot0 < 0: the group has one chunk
-};
-
-__device__ __forceinline__ WinItem decode_item(const WinArgs& a, int item, int n_groups) {
-  WinItem it;
-  const int per_chunk = a.L.heads * a.n_blocks;
-  const int chunk = item / per_chunk, rest = item - chunk * per_chunk;
-  it.head = rest / a.n_blocks;
-  it.block = rest - it.head * a.n_blocks;
-  int lo = 0, hi = n_groups - 1;  // last group with chunk_start[group] <= chunk
-  while (lo < hi) {
-    const int mid = (lo + hi + 1) >> 1;
-    if (a.chunk_start[mid] <= chunk) lo = mid; else hi = mid - 1;
-  }
-  it.first_row = a.group_first[lo];
-  it.n_rows = a.group_first[lo + 1] - it.first_row;
-  it.seq = a.row_seq[it.first_row];
-  it.ctx0 = a.row_ctx[it.first_row];
-  const int c = chunk - a.chunk_start[lo], n_chunks = a.chunk_start[lo + 1] - a.chunk_start[lo];
-  const int p0 = first_key(it.ctx0, a.window) / a.d.page_size;
-  const int pages = (it.ctx0 + it.n_rows - 2) / a.d.page_size + 1 - p0;
-  const int each = pages / n_chunks, more = pages - each * n_chunks;  // the first `more` chunks hold one page more
-  it.page_begin = p0 + c * each + min(c, more);
-  it.page_end = it.page_begin + each + (c < more ? 1 : 0);
-  it.slot0 = a.part_base[lo] < 0 ? -1 : a.part_base[lo] + c * it.n_rows;
-  return it;
-}
-
 __device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -471,7 +422,7 @@ __global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
           l = l * f + exp2f(sk - mm);
         }
         const float inv = l > 0.f ? f / l : 0.f;
-        __nv_bfloat16* dst = a.out + (size_t)(it.first_row + tok) * a.out_stride + (size_t)qh * a.L.value_dim;
+        __nv_bfloat16* dst = a.out + (size_t)(it.first_row + tok) * a.out_stride + (size_t)qh * a.out_head;
 #pragma unroll
         for (int j = 0; j < NO; ++j) {
           const int c = j * 8 + 2 * t;
@@ -519,7 +470,7 @@ __global__ void __launch_bounds__(256) window_combine_kernel(WinArgs a) {
   for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
   if (a.sinks) l += exp2f(a.sinks[qh] - mm);
   const float inv = l > 0.f ? 1.0f / l : 0.f;
-  __nv_bfloat16* dst = a.out + (size_t)row * a.out_stride + (size_t)qh * a.L.value_dim;
+  __nv_bfloat16* dst = a.out + (size_t)row * a.out_stride + (size_t)qh * a.out_head;
   for (int v0 = 0; v0 < a.L.vd; v0 += 128) {  // four columns per lane
     const int v = v0 + 4 * lane;
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -686,13 +637,11 @@ b200_status launch_mma_v(const b200_kv* kv, WinArgs& a, int layer, cudaStream_t 
 
 extern int b200_attn_pages_per_chunk;
 
-b200_status b200_window_attn_plan(b200_kv* kv, int32_t layer, int32_t window, int32_t gqa, const int32_t* d_row_seq, const int32_t* d_row_ctx,
-                                  int32_t total_rows, void* stream) {
+b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t items_per_chunk, int32_t n_workers, const int32_t* d_row_seq,
+                                const int32_t* d_row_ctx, int32_t total_rows, void* stream) {
   if (total_rows <= 0) return B200_OK;
   if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
-  b200_status st = sm_count();
-  if (st != B200_OK) return st;
-  const int qt = q_tokens_of(gqa), R = kv->cfg.max_rows + 2;
+  const int R = kv->cfg.max_rows + 2;
   WindowPlan* p = find_plan(kv, window, qt);
   if (!p) {
     p = new WindowPlan();
@@ -706,13 +655,37 @@ b200_status b200_window_attn_plan(b200_kv* kv, int32_t layer, int32_t window, in
     kv->plans.push_back(p);
   }
   const int forced = b200_attn_pages_per_chunk <= 0 ? 0 : std::min(std::max(b200_attn_pages_per_chunk, 1), 1 << 20);
-  const KvLayerDev& L = kv->lay[layer];
-  const int per_chunk = L.heads * ((gqa + 15) / 16), warps = shape_of((L.kd + 63) / 64 + (L.vd + 63) / 64).warps;
   window_plan_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(d_row_seq, d_row_ctx, total_rows, kv->cfg.page_size, window, qt,
-                                                          per_chunk, g_sms * warps, forced, kv->max_chunks,
+                                                          items_per_chunk, n_workers, forced, kv->max_chunks,
                                                           p->buf, p->buf + R, p->buf + 2 * R, p->buf + 3 * R, p->buf + 4 * R);
   B200_LAUNCH_CHECK();
   return B200_OK;
+}
+
+bool b200_attn_use_plan(b200_kv* kv, int32_t window, int32_t q_tokens, WinArgs* a) {
+  const WindowPlan* p = find_plan(kv, window, q_tokens);
+  if (!p) { b200_set_error("attention: no plan for window %d and groups of %d", window, q_tokens); return false; }
+  const int R = kv->cfg.max_rows + 2;
+  a->group_first = p->buf; a->chunk_start = p->buf + R; a->part_base = p->buf + 2 * R; a->row_group = p->buf + 3 * R; a->hdr = p->buf + 4 * R;
+  a->part_o = kv->d_part_o; a->part_ml = kv->d_part_ml;
+  return true;
+}
+
+b200_status b200_attn_combine(b200_kv* kv, const WinArgs& a, void* stream) {
+  window_combine_kernel<<<(unsigned)(((long long)a.total_rows * a.n_q_heads + 7) / 8), 256, 0, (cudaStream_t)stream>>>(a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+b200_status b200_window_attn_plan(b200_kv* kv, int32_t layer, int32_t window, int32_t gqa, const int32_t* d_row_seq, const int32_t* d_row_ctx,
+                                  int32_t total_rows, void* stream) {
+  if (total_rows <= 0) return B200_OK;
+  b200_status st = sm_count();
+  if (st != B200_OK) return st;
+  const KvLayerDev& L = kv->lay[layer];
+  if (L.values_in_keys) return b200_latent_attn_plan(kv, layer, gqa, d_row_seq, d_row_ctx, total_rows, stream);
+  const int per_chunk = L.heads * ((gqa + 15) / 16), warps = shape_of((L.kd + 63) / 64 + (L.vd + 63) / 64).warps;
+  return b200_attn_make_plan(kv, window, q_tokens_of(gqa), per_chunk, g_sms * warps, d_row_seq, d_row_ctx, total_rows, stream);
 }
 
 b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
@@ -740,18 +713,15 @@ b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
     B200_LAUNCH_CHECK();
     return B200_OK;
   }
-  const WindowPlan* p = find_plan(kv, c.window, q_tokens_of(G));
-  if (!p) { b200_set_error("window attention: no plan for window %d and group %d", c.window, G); return B200_ERR_INVALID_ARGUMENT; }
-  const int R = kv->cfg.max_rows + 2;
+  if (L.values_in_keys) return b200_latent_attn_run(kv, c, d_row_seq, d_row_ctx, total_rows, stream);
   WinArgs a;
+  if (!b200_attn_use_plan(kv, c.window, q_tokens_of(G), &a)) return B200_ERR_INVALID_ARGUMENT;
   a.d = kv->dev; a.L = L; a.q = (const __nv_bfloat16*)c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx;
   a.total_rows = total_rows; a.n_q_heads = c.n_q_heads; a.window = c.window;
   a.G = G; a.head_block = head_block_of(G); a.n_blocks = (G + 15) / 16;
-  a.group_first = p->buf; a.chunk_start = p->buf + R; a.part_base = p->buf + 2 * R; a.row_group = p->buf + 3 * R; a.hdr = p->buf + 4 * R;
-  a.part_o = kv->d_part_o; a.part_ml = kv->d_part_ml;
   a.scale_log2 = c.scale * kLog2e;
   a.slopes = c.slopes_log2; a.sinks = c.sinks_log2;
-  a.out = (__nv_bfloat16*)c.out; a.out_stride = c.out_stride;
+  a.out = (__nv_bfloat16*)c.out; a.out_stride = c.out_stride; a.out_head = c.out_head_stride > 0 ? c.out_head_stride : L.value_dim;
   if (L.kd <= 64) st = launch_mma_v<1>(kv, a, c.layer, s);
   else if (L.kd <= 128) st = launch_mma_v<2>(kv, a, c.layer, s);
   else st = launch_mma_v<4>(kv, a, c.layer, s);
@@ -760,11 +730,10 @@ b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
   const int shortest = b200_attn_pages_per_chunk > 0 ? b200_attn_pages_per_chunk : 4;
   const int most_pages = c.window > 0 ? (c.window + q_tokens_of(G) - 2) / 32 + 2 : kv->cfg.max_pages_per_seq;
   if (std::min(most_pages, kv->cfg.max_pages_per_seq) <= shortest) return B200_OK;
-  window_combine_kernel<<<(unsigned)(((long long)total_rows * c.n_q_heads + 7) / 8), 256, 0, s>>>(a);
-  B200_LAUNCH_CHECK();
-  return B200_OK;
+  return b200_attn_combine(kv, a, stream);
 }
 
 bool b200_window_attn_takes_mma(const b200_kv* kv, int32_t layer) {
-  return kv->layered && kv->dev.elem_bytes == 2 && !kv->lay[layer].values_in_keys && kv->lay[layer].kd <= 256 && kv->lay[layer].vd <= 256;
+  if (kv->layered && kv->lay[layer].values_in_keys) return b200_latent_attn_takes_mma(kv, layer);
+  return kv->layered && kv->dev.elem_bytes == 2 && kv->lay[layer].kd <= 256 && kv->lay[layer].vd <= 256;
 }

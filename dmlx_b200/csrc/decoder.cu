@@ -509,8 +509,8 @@ b200_status b200_decoder::begin_step(b200_kv* kv, int n_req, int T, int tile_row
   std::vector<std::pair<int, int>> planned;
   for (size_t r = 0; r < runs.size(); ++r) {
     const b200_decoder_layer& s = layers[runs[r].layer].s;
-    if (s.mixer != B200_MIX_ATTENTION) continue;
-    const std::pair<int, int> key{s.window, s.n_heads / s.n_kv_heads};
+    if (s.mixer == B200_MIX_GLA) continue;
+    const std::pair<int, int> key{s.window, s.mixer == B200_MIX_LATENT ? s.n_heads : s.n_heads / s.n_kv_heads};
     if (!attn_mma || !b200_window_attn_takes_mma(kv, (int)r) || std::find(planned.begin(), planned.end(), key) != planned.end()) continue;
     planned.push_back(key);
     MODEL_STEP_CAT(0, b200_window_attn_plan(kv, (int)r, key.first, key.second, d_row_seq, d_row_ctx, T, stream));

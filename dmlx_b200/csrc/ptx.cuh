@@ -224,6 +224,19 @@ __device__ __forceinline__ uint64_t umma_desc_k_sw128(uint32_t smem_addr) {
   d |= (uint64_t)2 << 61;                       // layout: SWIZZLE_128B
   return d;
 }
+// The same for an operand whose M (or N) elements are contiguous: rows of 64 of them (128 bytes, 128B swizzle), one row per K element,
+// 8-row groups 1024 bytes apart, the next 64 M elements `block_bytes` further on.
+__device__ __forceinline__ uint64_t umma_desc_mn_sw128(uint32_t smem_addr, uint32_t block_bytes) {
+  uint64_t d = 0;
+  d |= (uint64_t)((smem_addr & 0x3FFFF) >> 4);
+  d |= (uint64_t)(block_bytes >> 4) << 16;      // leading byte offset: between blocks of 64 M elements
+  d |= (uint64_t)(1024 >> 4) << 32;             // stride byte offset: between groups of 8 K elements
+  d |= (uint64_t)1 << 46;
+  d |= (uint64_t)2 << 61;
+  return d;
+}
+constexpr uint32_t kUmmaAMn = 1u << 15, kUmmaBMn = 1u << 16;  // instruction descriptor: A / B operand with M / N contiguous
+
 // Shared-memory descriptor of an unswizzled K-major operand one 16-byte column wide: 8-row core
 // matrices of 128 contiguous bytes, 128 bytes apart.
 __device__ __forceinline__ uint64_t umma_desc_k_noswizzle_16B(uint32_t smem_addr) {

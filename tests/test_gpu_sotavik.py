@@ -25,6 +25,7 @@ def _load(tmp_path, cfg, seed, dtype, max_rows=512, slots=4, change=None, rank=7
     w = R.random_weights(cfg, seed, rank)
     if change:
         change(w)
+        w = {n: a if n.endswith(".table") else _bf16(a) for n, a in w.items()}
     R.write_model(str(tmp_path), cfg, w)
     return load_model(str(tmp_path), dtype, Limits(max_rows, slots, slots)), w
 
