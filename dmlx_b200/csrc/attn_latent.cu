@@ -1,12 +1,23 @@
 // Latent attention: all heads attend to one row per token, [latent c | rotated key part], and their values are W_uv c.  W_uk is
 // taken to the query side (q_head <- W_uk^T q_head) and W_uv behind the weighted sum, so the pages are read once for all heads
 // and hold kv_rank + rot_dim numbers per token.
+//
+// latent_attn_kernel (tcgen05, bf16): a tile is 128 keys (four pages, one TMA box per 64 columns of a page) against up to 32 rows, a
+// row being (token of the group, head).  The operands are swapped, so the keys fill the M = 128 side whatever the number of rows:
+//   S^T [keys][rows] = K Q^T,          A = the tile as it lies (K-major), B = the rows' queries;
+//   O^T [latent][rows] += C^T P,       A = the same tile read the other way (its latent columns are the M side), B = P.
+// The softmax warps hold one key per thread; maxima over the keys go through a shuffle transpose.  P is written as two bf16 terms
+// (value and remainder) side by side, which the second product accumulates in separate columns, so weights keep 16 bits and the
+// tile is read once for both.  The running maximum a row is scaled by moves only when it has grown by 2^8.
 #include <cuda_bf16.h>
 
 #include <algorithm>
 
 #include "attn_latent.cuh"
+#include "attn_plan.cuh"
 #include "common.h"
+#include "ptx.cuh"
+#include "tma.cuh"
 
 namespace {
 
@@ -104,6 +115,81 @@ b200_status b200_latent_prep(b200_kv* kv, const LatentPrep& p, const int32_t* d_
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
+
+// ---- tensor-core kernel ----------------------------------------------------------------------------------------------
+namespace {
+
+constexpr int kTileKeys = 128, kTilePages = 4, kBoxBytes = kTileKeys * 128;  // bytes of a tile's 64-column box
+constexpr int kPBytes = kTileKeys * 128;
+constexpr int kLatentThreads = 256;    // warp 0 loads, warp 1 issues the MMAs, warps 4-7 softmax
+constexpr float kGrow = 8.f;           // log2 units a row's maximum may grow before its sums are rescaled
+constexpr uint32_t kPolls = 1u << 18;  // a wait inside a CTA is microseconds
+
+__device__ __forceinline__ bool wait(uint64_t* bar, uint32_t parity) { return ptx::mbar_wait_limit(bar, parity, kPolls); }
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// Barriers of the 128 softmax threads: true where every one (some one) of them passed true.
+__device__ __forceinline__ bool softmax_sync_and(bool x) {
+  uint32_t r;
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %1, 0;\n\tbar.red.and.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}" : "=r"(r) : "r"((uint32_t)x) : "memory");
+  return r != 0;
+}
+__device__ __forceinline__ bool softmax_sync_or(bool x) {
+  uint32_t r;
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %1, 0;\n\tbar.red.or.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}" : "=r"(r) : "r"((uint32_t)x) : "memory");
+  return r != 0;
+}
+
+// Reduces NR values over the warp's lanes: every step hands half of the columns to the partner lane.  Lane l ends up with
+// column l (NR = 32) or l / 2 (NR = 16).
+template <int NR, bool MAX>
+__device__ __forceinline__ float transpose_reduce(float (&w)[NR], int lane) {
+  int o = 16;
+#pragma unroll
+  for (int n = NR / 2; n >= 1; n >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < n; ++i) {
+      const float send = up ? w[i] : w[i + n], keep = up ? w[i + n] : w[i];
+      const float got = __shfl_xor_sync(0xffffffffu, send, o);
+      w[i] = MAX ? fmaxf(keep, got) : keep + got;
+    }
+    o >>= 1;
+  }
+  if (NR == 16) {
+    const float got = __shfl_xor_sync(0xffffffffu, w[0], 1);
+    w[0] = MAX ? fmaxf(w[0], got) : w[0] + got;
+  }
+  return w[0];
+}
+
+template <int NR>
+__device__ __forceinline__ void load_rows(uint32_t taddr, float (&v)[NR]) {
+  uint32_t u[NR / 16][16];
+#pragma unroll
+  for (int c = 0; c < NR / 16; ++c) ptx::tmem_ld16(taddr + c * 16, u[c]);
+  ptx::tmem_ld_wait();
+#pragma unroll
+  for (int c = 0; c < NR; ++c) v[c] = __uint_as_float(u[c / 16][c % 16]);
+}
+
+struct LatentArgs {
+  WinArgs w;
+  int n_kb, n_mc;     // 64-column boxes of a key row; blocks of 128 latent columns
+  uint32_t tmem_cols;
+};
+
+// Shared memory behind the tiles, the queries and P.
+template <int NR>
+struct LatentShared {
+  uint64_t k_full[4], k_free[4], s_full[2], p_ready, pv_done, q_full;
+  uint32_t tmem;
+  float red[4][NR], m[NR], corr[NR], l[NR];
+  int ctx[NR];
+};
 
 template <int NR>
 __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __grid_constant__ CUtensorMap kmap, LatentArgs la) {
