@@ -16,6 +16,7 @@ Prints ONE JSON line (rank 0).  Workloads (synthetic seeded inputs):
       One step = one decode of all 64 sequences through one attention layer.
   tafuvik : the looped decoder stack (one GPU) beside the LLaMA stack at equal size, both bf16 — decode steps of 64
       requests and prefill steps of 4096 rows at a few layer shapes, with each kernel category against its roofline.
+  sotavik : the Sotavik stack (latent attention, gated linear attention, experts by token id; one GPU) the same way.
 Multi-GPU (torchrun, one rank per GPU): independent replicas of the workload, no collective in the
 step (requests never interact); `value` = tokens of all ranks / max-over-ranks time.
 """
@@ -1120,6 +1121,174 @@ def _decoder_work(z, runs, window, ctxs, prefill, llama):
             "other": (runs * rows * d * (28.0 if not llama else 8.0), 0.0)}
 
 
+def _time_stack(model, kv, ctxs, pages, mode, K, W):
+    """One model on one pool: decode steps of DECODER_REQS requests on the contexts given, or two prompts in one step.  Returns
+    (ms per step, {category: ms per step}, kernels launched in the timed steps)."""
+    import torch
+
+    from dmlx_b200 import device as dev
+
+    kv.reset()
+    kv.set_free_order(np.random.default_rng(5).permutation(pages).tolist())
+    lens = ctxs.copy()
+    steps = K if mode == "decode" else max(K // 5, 4)
+    tokens = torch.randint(0, DECODER_VOCAB, (DECODER_ROWS,), dtype=torch.int32, device="cuda")
+    if mode == "decode":
+        kv.reserve(dev.pack_desc_array([(i, int(n), 0, -1) for i, n in enumerate(ctxs)]).cuda())
+    cur = torch.zeros((DECODER_REQS if mode == "decode" else 2, 4), dtype=torch.int32, device="cuda")
+
+    def one(_=None):
+        if mode == "decode":
+            cur.copy_(torch.tensor([(i, 1, int(n), -1) for i, n in enumerate(lens)], dtype=torch.int32).pin_memory(), non_blocking=True)
+            model.forward_device(kv, cur, DECODER_REQS)
+            lens[:] += 1
+        else:
+            half = DECODER_ROWS // 2
+            cur.copy_(torch.tensor([(0, half, 0, 0), (1, half, 0, half)], dtype=torch.int32).pin_memory(), non_blocking=True)
+            model.forward_device(kv, cur, DECODER_ROWS, tokens)
+
+    def between():
+        if mode == "prefill":  # pages back for the next prompt (on another stream: after the step has finished)
+            torch.cuda.synchronize()
+            kv.release([0, 1])
+
+    for _ in range(W):
+        one()
+        between()
+    torch.cuda.synchronize()
+    before = model.launch_count()
+    evs = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(steps if mode == "prefill" else 1)]
+    if mode == "prefill":
+        for a, b in evs:
+            a.record()
+            one()
+            b.record()
+            between()
+    else:
+        evs[0][0].record()
+        for _ in range(steps):
+            one()
+        evs[0][1].record()
+    torch.cuda.synchronize()
+    ms = sum(a.elapsed_time(b) for a, b in evs) / steps
+    launches = model.launch_count() - before
+    model.profile_enable(True)
+    for _ in range(4):
+        one()
+        between()
+    prof = {c: t / 4 for c, (t, _) in model.profile_collect().items()}
+    model.profile_enable(False)
+    assert kv.error_word() == 0 and dev.qmm_error_word() == 0
+    return ms, prof, launches
+
+
+# Layer shapes of the Sotavik bench beside LLaMA of equal width: as many query heads, an equal active feed-forward width.
+SOTAVIK_SIZES = {
+    "d4096": dict(hidden=4096, heads=32, kv_heads=8, head_dim=128, ffn=14336, latent=dict(heads=32, dim=128, rot=64, vdim=128, rank=512),
+                  gla=dict(heads=16, dim=128, vdim=256, decay_rank=16), experts=32, top=4, expert_ffn=2048, shared=6144),
+    "d2048": dict(hidden=2048, heads=16, kv_heads=4, head_dim=128, ffn=8192, latent=dict(heads=16, dim=96, rot=32, vdim=64, rank=256),
+                  gla=dict(heads=8, dim=128, vdim=256, decay_rank=16), experts=32, top=4, expert_ffn=1024, shared=4096),
+}
+SOTAVIK_STACKS = {"sotavik_latent": "LLLLLL", "sotavik_gla": "GGGGGG", "sotavik_mixed": "GLLGLG"}
+
+
+def _sotavik_layers(z, order):
+    from dmlx_b200 import device as dev
+
+    ff = dict(ffn=z["shared"], n_experts=z["experts"], top_k=z["top"], expert_ffn=z["expert_ffn"])
+    l, g = z["latent"], z["gla"]
+    make = {"L": dict(mixer=dev.MIX_LATENT, n_heads=l["heads"], n_kv_heads=1, key_dim=l["dim"], value_dim=l["vdim"], kv_rank=l["rank"], rot_dim=l["rot"],
+                      rot_base=1e4, scale=(l["dim"] + l["rot"]) ** -0.5, flags=dev.DEC_SINK | dev.DEC_PARALLEL, **ff),
+            "G": dict(mixer=dev.MIX_GLA, n_heads=g["heads"], n_kv_heads=g["heads"], key_dim=g["dim"], value_dim=g["vdim"], decay_rank=g["decay_rank"],
+                      decay_tau=16.0, flags=dev.DEC_PARALLEL, **ff)}
+    return [make[c] for c in order]
+
+
+def _sotavik_work(z, order, ctxs, prefill):
+    """As _decoder_work.  Attention FLOPs are those of the definition (keys of every head), not of the latent form the kernel runs."""
+    d, l, g = z["hidden"], z["latent"], z["gla"]
+    rows = DECODER_ROWS if prefill else len(ctxs)
+    if prefill:
+        per = rows // len(ctxs)
+        keys, read = len(ctxs) * per * (per + 1) / 2.0, float(rows)
+    else:
+        keys = read = float(ctxs.sum())
+    nl, ng, n = order.count("L"), order.count("G"), len(order)
+    lat, hq, hk, hv = l["rank"] + l["rot"], l["heads"] * (l["dim"] + l["rot"]), g["heads"] * g["dim"], g["heads"] * g["vdim"]
+    seqs = len(ctxs)
+    attn_b = nl * (read * lat + rows * l["heads"] * (lat + l["rank"])) * 2.0
+    attn_f = nl * 2.0 * keys * l["heads"] * (l["dim"] + l["rot"] + l["vdim"])
+    attn_b += ng * (seqs * hk * g["vdim"] * (4.0 if prefill else 8.0) + rows * (2 * hk + 3 * hv) * 2.0)
+    attn_f += ng * 4.0 * rows * hk * g["vdim"]
+    dense = nl * (d * (hq + lat) + l["heads"] * (l["dim"] + l["vdim"]) * l["rank"] + d * l["heads"] * l["vdim"])
+    dense += ng * (d * (2 * hk + 2 * hv + g["decay_rank"]) + d * hv) + n * 3 * d * z["shared"]
+    used = min(z["experts"], rows * z["top"])
+    head = d * DECODER_VOCAB
+    mat_b = 2.0 * (dense + n * used * 3 * d * z["expert_ffn"] + head)
+    mat_f = 2.0 * rows * (dense + n * z["top"] * 3 * d * z["expert_ffn"]) + 2.0 * seqs * head
+    depth = sum(i + 2 for i in range(n))
+    return {"attention": (attn_b, attn_f), "matmul": (mat_b, mat_f), "rope_append": (nl * rows * (hq + lat) * 4.0, 0.0),
+            "other": (rows * d * (n * (4 + 2 + 2 * z["top"] + 4 + 4 + 2 + 4.0 * z["top"]) + 4.0 * depth), 0.0)}
+
+
+def run_sotavik(args, local: int):
+    import torch
+
+    from dmlx_b200 import device as dev
+
+    torch.cuda.set_device(local)
+    torch.cuda.set_stream(torch.cuda.Stream())
+    hbm, kind = load_peaks()
+    p = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    tflops = float(json.load(open(p))["bf16_tflops"]) if os.path.exists(p) else 1590.0
+    K, W = min(args.steps, 50), max(args.warmup, 3)
+    ctxs = np.clip(np.rint(np.random.default_rng(77).lognormal(np.log(2600), 0.6, DECODER_REQS)), 256, 12000).astype(np.int64)
+    pages = int((-(-(ctxs + 4 * (K + W) + 64) // PAGE)).sum()) + 16
+    most = int(-(-(ctxs.max() + 4 * (K + W) + 64) // PAGE))
+    sampler = ClockSampler(local)
+    sampler.start()
+    out, launches = {}, 0
+    for name, z in SOTAVIK_SIZES.items():
+        for which in ("llama", *SOTAVIK_STACKS):
+            if which == "llama":
+                model = dev.LlamaModel(6, z["hidden"], z["heads"], z["kv_heads"], z["head_dim"], z["ffn"], DECODER_VOCAB, DECODER_ROWS, DECODER_REQS,
+                                       DECODER_REQS)
+                model.random_init(dev.Q_BF16, 3)
+                kv = dev.PagedKVCache(6, z["kv_heads"], z["head_dim"], pages, DECODER_REQS, most, z["heads"], max_rows=DECODER_ROWS)
+            else:
+                model = dev.DecoderModel(z["hidden"], DECODER_VOCAB, _sotavik_layers(z, SOTAVIK_STACKS[which]), 1e-5, 1.0, None, dev.DT_BF16, DECODER_ROWS,
+                                         DECODER_REQS, DECODER_REQS, flags=dev.DEC_SCALAR_NORM | dev.DEC_DEPTH_AVERAGE)
+                model.random_init(3)
+                kv = model.make_cache(pages, DECODER_REQS, most)
+            for mode in ("decode", "prefill"):
+                ms, prof, n = _time_stack(model, kv, ctxs, pages, mode, K, W)
+                launches += n
+                at = ctxs if mode == "decode" else ctxs[:2]
+                if which == "llama":
+                    work = _decoder_work(dict(z, llama_dim=z["head_dim"]), 6, 0, at, mode == "prefill", True)
+                else:
+                    work = _sotavik_work(z, SOTAVIK_STACKS[which], at, mode == "prefill")
+                entry = {"ms_per_step": ms, "tokens_per_s": (DECODER_REQS if mode == "decode" else DECODER_ROWS) / ms * 1e3}
+                for cat, (nbytes, flops) in work.items():
+                    ideal = max(nbytes / hbm / 1e6, flops / tflops / 1e9)
+                    entry[cat] = {"ms": prof[cat], "of_roofline": ideal / prof[cat] if prof[cat] > 0 else None}
+                out.setdefault(name, {}).setdefault(mode, {})[which] = entry
+            kv.close()
+            model.close()
+    clocks = sampler.stop()
+    head = out["d4096"]["decode"]["sotavik_mixed"]
+    print(json.dumps({
+        "metric": "decode tokens/sec (Sotavik stack, 6 layers)", "value": head["tokens_per_s"], "unit": "decode tokens/s", "n_gpus": 1,
+        "steps": K, "warmup": W, "ms_per_step": head["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "sotavik", "stacks": SOTAVIK_STACKS, "shapes": SOTAVIK_SIZES, "vocab": DECODER_VOCAB, "decode_requests": DECODER_REQS,
+                   "cached_tokens": int(ctxs.sum()), "prefill": f"2 prompts of {DECODER_ROWS // 2} tokens in one step", "parallelism": "dp1",
+                   "l2": "weights and caches larger than L2"},
+        "note": "of_roofline: the larger of bytes / measured copy bandwidth and FLOPs / measured burst bf16 rate, over the category's time "
+                "(eager launches with an event pair each, so small kernels carry their launch gap)",
+        "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind}, "sizes": out, "e2e": None, "gpu_launches": launches, "clocks": clocks}))
+
+
 def run_tafuvik(args, local: int):
     import torch
 
@@ -1155,64 +1324,14 @@ def run_tafuvik(args, local: int):
                                          DECODER_REQS)
                 model.random_init(3)
                 kv = model.make_cache(pages, DECODER_REQS, most)
-            kv.set_free_order(np.random.default_rng(5).permutation(pages).tolist())
             for mode in ("decode",) if which == "llama_contexts_of_1024" else ("decode", "prefill"):
-                kv.reset()
-                kv.set_free_order(np.random.default_rng(5).permutation(pages).tolist())
-                lens = ctxs.copy()
-                steps = K if mode == "decode" else max(K // 5, 4)
-                tokens = torch.randint(0, DECODER_VOCAB, (DECODER_ROWS,), dtype=torch.int32, device="cuda")
-                if mode == "decode":
-                    kv.reserve(dev.pack_desc_array([(i, int(n), 0, -1) for i, n in enumerate(ctxs)]).cuda())
-                cur = torch.zeros((DECODER_REQS if mode == "decode" else 2, 4), dtype=torch.int32, device="cuda")
-
-                def one(_=None):
-                    if mode == "decode":
-                        cur.copy_(torch.tensor([(i, 1, int(n), -1) for i, n in enumerate(lens)], dtype=torch.int32).pin_memory(), non_blocking=True)
-                        model.forward_device(kv, cur, DECODER_REQS)
-                        lens[:] += 1
-                    else:
-                        half = DECODER_ROWS // 2
-                        cur.copy_(torch.tensor([(0, half, 0, 0), (1, half, 0, half)], dtype=torch.int32).pin_memory(), non_blocking=True)
-                        model.forward_device(kv, cur, DECODER_ROWS, tokens)
-
-                def between():
-                    if mode == "prefill":  # pages back for the next prompt (on another stream: after the step has finished)
-                        torch.cuda.synchronize()
-                        kv.release([0, 1])
-
-                for _ in range(W):
-                    one()
-                    between()
-                torch.cuda.synchronize()
-                before = model.launch_count()
-                evs = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(steps if mode == "prefill" else 1)]
-                if mode == "prefill":
-                    for a, b in evs:
-                        a.record()
-                        one()
-                        b.record()
-                        between()
-                else:
-                    evs[0][0].record()
-                    for _ in range(steps):
-                        one()
-                    evs[0][1].record()
-                torch.cuda.synchronize()
-                ms = sum(a.elapsed_time(b) for a, b in evs) / steps
-                launches += model.launch_count() - before
-                model.profile_enable(True)
-                for _ in range(4):
-                    one()
-                    between()
-                prof = model.profile_collect()
-                model.profile_enable(False)
-                assert kv.error_word() == 0 and dev.qmm_error_word() == 0
+                ms, prof, n = _time_stack(model, kv, ctxs, pages, mode, K, W)
+                launches += n
                 rows = DECODER_REQS if mode == "decode" else DECODER_ROWS
                 work = _decoder_work(z, 6, window, ctxs if mode == "decode" else ctxs[:2], mode == "prefill", llama)
                 entry = {"ms_per_step": ms, "tokens_per_s": rows / ms * 1e3}
                 for cat, (nbytes, flops) in work.items():
-                    t = prof[cat][0] / 4
+                    t = prof[cat]
                     ideal = max(nbytes / hbm / 1e6, flops / tflops / 1e9)
                     entry[cat] = {"ms": t, "of_roofline": ideal / t if t > 0 else None}
                 out.setdefault(name, {}).setdefault(mode, {})[which] = entry
@@ -1283,6 +1402,10 @@ def main():
     if args.mx_persistent >= 0:
         from dmlx_b200 import _lib
         _lib.lib.b200_set_qmm_mx_persistent(args.mx_persistent)
+    if args.workload == "sotavik":
+        if rank == 0:
+            run_sotavik(args, local)
+        return
     if args.workload == "tafuvik":
         if rank == 0:
             run_tafuvik(args, local)
