@@ -1139,8 +1139,9 @@ def _time_stack(model, kv, ctxs, pages, mode, K, W):
 
     def one(_=None):
         if mode == "decode":
-            cur.copy_(torch.tensor([(i, 1, int(n), -1) for i, n in enumerate(lens)], dtype=torch.int32).pin_memory(), non_blocking=True)
-            model.forward_device(kv, cur, DECODER_REQS)
+            # (random tokens: those a random model picks itself are all alike, and would all go to the same experts)
+            cur.copy_(torch.tensor([(i, 1, int(n), i) for i, n in enumerate(lens)], dtype=torch.int32).pin_memory(), non_blocking=True)
+            model.forward_device(kv, cur, DECODER_REQS, tokens)
             lens[:] += 1
         else:
             half = DECODER_ROWS // 2

@@ -185,14 +185,15 @@ struct LatentArgs {
 // Shared memory behind the tiles, the queries and P.
 template <int NR>
 struct LatentShared {
-  uint64_t k_full[4], k_free[4], s_full[2], p_ready, pv_done, q_full;
+  uint64_t k_full[4], k_free[4], s_full[2], p_ready, pv_done, q_full, q_free;
+  long long off[NR];  // where a row's output starts
   uint32_t tmem;
   float red[4][NR], m[NR], corr[NR], l[NR];
   int ctx[NR];
 };
 
 template <int NR>
-__global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __grid_constant__ CUtensorMap kmap, LatentArgs la) {
+__global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap qmap, LatentArgs la) {
   const WinArgs& a = la.w;
   extern __shared__ unsigned char latent_dyn[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(latent_dyn) + 1023) & ~(uintptr_t)1023);
@@ -208,7 +209,8 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
     ptx::mbar_init(&sh.s_full[1], 1);
     ptx::mbar_init(&sh.p_ready, 128);
     ptx::mbar_init(&sh.pv_done, 1);
-    ptx::mbar_init(&sh.q_full, 128);
+    ptx::mbar_init(&sh.q_full, 1);
+    ptx::mbar_init(&sh.q_free, 1);
     ptx::mbar_fence_init();
   }
   if (warp == 1) {
@@ -224,9 +226,15 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
   if (warp == 0) {
     if (lane == 0) {  // ---- loads ----
       int s = 0;
-      uint32_t ph = 0, issued = 0;
-      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x) {
+      uint32_t ph = 0, issued = 0, n_item = 0;
+      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
         const WinItem it = decode_item(a, item, n_groups);
+        // the tile's rows lie one behind the other: tokens of the group, or heads of the block (what follows them is never stored)
+        ok = wait(&sh.q_free, (n_item & 1u) ^ 1u);
+        if (!ok) break;
+        ptx::mbar_expect_tx(&sh.q_full, n_kb * NR * 128);
+        for (int b = 0; b < n_kb; ++b)
+          ptx::tma_load_2d(qbuf + b * NR * 128, &qmap, b * 64, it.first_row * a.n_q_heads + it.block * a.head_block, &sh.q_full);
         const int* table = a.d.block_table + (size_t)it.seq * a.d.max_pages_per_seq;
         for (int pg = it.page_begin; pg < it.page_end; pg += kTilePages) {
           const int pages = min(kTilePages, it.page_end - pg);
@@ -243,6 +251,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
         }
       }
       if (!ok) {  // leave no copy in flight behind
+        if (n_item > 0) wait(&sh.q_full, (n_item - 1) & 1u);
         for (uint32_t i = issued > (uint32_t)stages ? issued - stages : 0; i < issued; ++i) wait(&sh.k_full[i % stages], (i / stages) & 1u);
       }
     }
@@ -253,7 +262,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
       const uint32_t q0 = ptx::smem_u32(qbuf), p0 = ptx::smem_u32(pbuf), t0 = ptx::smem_u32(smem);
       int sc = 0, sp = 0;  // stage of the next tile to score, of the next to sum
       uint32_t phc = 0, n_scored = 0, n_summed = 0, n_item = 0;
-      auto score = [&]() {  // the next tile's S^T
+      auto score = [&](bool last) {  // the next tile's S^T
         ok = wait(&sh.k_full[sc], phc);
         if (!ok) return;
         ptx::tc_fence_after_sync();
@@ -264,6 +273,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
           ptx::umma_bf16(dst, da, db, id_s, ks > 0 ? 1u : 0u);
         }
         ptx::umma_commit(&sh.s_full[n_scored & 1u]);
+        if (last) ptx::umma_commit(&sh.q_free);
         ++n_scored;
         if (++sc == stages) { sc = 0; phc ^= 1u; }
       };
@@ -272,9 +282,9 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
         const int tiles = (it.page_end - it.page_begin + kTilePages - 1) / kTilePages;
         ok = wait(&sh.q_full, n_item & 1u);
         if (!ok) break;
-        score();
+        score(tiles == 1);
         for (int j = 0; j < tiles && ok; ++j) {
-          if (stages > 1 && j + 1 < tiles) score();  // ahead of this tile's softmax
+          if (stages > 1 && j + 1 < tiles) score(j + 2 == tiles);  // ahead of this tile's softmax
           if (!ok) break;
           ok = wait(&sh.p_ready, n_summed & 1u);
           if (!ok) break;
@@ -292,7 +302,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
           ptx::umma_commit(&sh.pv_done);
           ++n_summed;
           if (++sp == stages) sp = 0;
-          if (stages == 1 && j + 1 < tiles) score();
+          if (stages == 1 && j + 1 < tiles) score(j + 2 == tiles);
         }
       }
     }
@@ -305,21 +315,13 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
     for (int item = blockIdx.x; item < n_items && !dead; item += gridDim.x) {
       const WinItem it = decode_item(a, item, n_groups);
       const int hb = a.head_block, h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0);
-      const int vecs = a.L.kd / 8;
-      for (int i = key; i < NR * vecs; i += 128) {
-        const int r = i / vecs, c = i - r * vecs, tok = r / hb, head = r - tok * hb;
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (tok < it.n_rows && head < heads_here)
-          v = *reinterpret_cast<const uint4*>(a.q + (size_t)(it.first_row + tok) * a.q_stride + (size_t)(h0 + head) * a.L.kd + c * 8);
-        *reinterpret_cast<uint4*>(qbuf + (c >> 3) * NR * 128 + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
-      }
       if (key < NR) {
         const int tok = key / hb, head = key - tok * hb;
         sh.ctx[key] = tok < it.n_rows && head < heads_here ? it.ctx0 + tok : 0;
         sh.m[key] = kAttnNone;
+        sh.off[key] = it.slot0 >= 0 ? ((long long)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd
+                                    : (long long)(it.first_row + tok) * a.out_stride + (long long)(h0 + head) * a.out_head;
       }
-      ptx::fence_proxy_async_smem();
-      ptx::mbar_arrive(&sh.q_full);
       float l[NR];
 #pragma unroll
       for (int r = 0; r < NR; ++r) l[r] = 0.f;
@@ -331,8 +333,8 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
         float v[NR];
         load_rows<NR>(tmem + lanes + (n_tile & 1u) * NR, v);
         ++n_tile;
-        const bool edge = tok0 + kTileKeys > it.ctx0 || pages < kTilePages;
-        softmax_sync_and(true);  // sh.ctx, sh.m of a new item are in place; the previous tile's sh.m has been read
+        const bool edge = tok0 + kTileKeys > it.ctx0 || pages < kTilePages, first = pg == it.page_begin;
+        if (first) softmax_sync_and(true);  // what the item's first threads wrote is in place
         {
           float w[NR];
           const bool in_tile = key < pages * 32;
@@ -354,7 +356,6 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
           sh.corr[key] = moved ? ex2(m_old - mx) : 1.f;
           if (moved) sh.m[key] = mx;
         }
-        const bool first = pg == it.page_begin;
         const bool rescale = softmax_sync_or(moved) && !first;
         if (!first) {  // P and O are the previous tile's until its product is done
           ok = wait(&sh.pv_done, n_pv & 1u) && ok;
@@ -445,11 +446,9 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
         const int dim = mc * 128 + key;
 #pragma unroll
         for (int r = 0; r < NR; ++r) {
-          const int tok = r / hb, head = r - tok * hb;
-          if (sh.ctx[r] > 0 && dim < a.L.vd) {
-            if (it.slot0 >= 0) a.part_o[((size_t)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd + dim] = o[r];
-            else if (dim < a.L.value_dim)
-              a.out[(size_t)(it.first_row + tok) * a.out_stride + (size_t)(h0 + head) * a.out_head + dim] = __float2bfloat16(o[r] * sh.l[r]);
+          if (sh.ctx[r] > 0) {
+            if (it.slot0 >= 0) { if (dim < a.L.vd) a.part_o[sh.off[r] + dim] = o[r]; }
+            else if (dim < a.L.value_dim) a.out[sh.off[r] + dim] = __float2bfloat16(o[r] * sh.l[r]);
           }
         }
         __syncwarp();
@@ -478,6 +477,11 @@ int rows_of(int heads, int total_rows) { return heads <= 16 && total_rows <= 256
 
 template <int NR>
 b200_status launch(const b200_kv* kv, LatentArgs& la, int layer, cudaStream_t s) {
+  CUtensorMap qmap;
+  const uint64_t dims[2] = {(uint64_t)la.w.L.kd, (uint64_t)la.w.total_rows * la.w.n_q_heads}, strides[1] = {(uint64_t)la.w.L.kd * 2};
+  const uint32_t box[2] = {64, (uint32_t)NR};
+  b200_status st = b200_make_tensor_map(&qmap, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, la.w.q, dims, strides, box);
+  if (st != B200_OK) return st;
   int stages = 4;
   while (stages > 1 && smem_of<NR>(la.n_kb, stages) > kSmemLimit) --stages;
   la.w.stages = stages;
@@ -488,7 +492,7 @@ b200_status launch(const b200_kv* kv, LatentArgs& la, int layer, cudaStream_t s)
     B200_CUDA_TRY(cudaFuncSetAttribute(latent_attn_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit));
     configured = true;
   }
-  latent_attn_kernel<NR><<<g_sms, kLatentThreads, smem_of<NR>(la.n_kb, stages), s>>>(kv->lay_kmap[layer], la);
+  latent_attn_kernel<NR><<<g_sms, kLatentThreads, smem_of<NR>(la.n_kb, stages), s>>>(kv->lay_kmap[layer], qmap, la);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -509,12 +513,14 @@ b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t heads, con
     B200_CUDA_TRY(cudaDeviceGetAttribute(&g_sms, cudaDevAttrMultiProcessorCount, dev));
   }
   const int rows = rows_of(heads, total_rows);
-  return b200_attn_make_plan(kv, 0, std::max(1, rows / heads), (heads + rows - 1) / rows, g_sms, d_row_seq, d_row_ctx, total_rows, stream);
+  return b200_attn_make_plan(kv, 0, std::max(1, rows / heads), (heads + rows - 1) / rows, g_sms, d_row_seq, d_row_ctx, total_rows, stream, 4.f,
+                             8.f * std::min(heads, rows) * kv->lay[layer].value_dim / (64.f * kv->lay[layer].kd));
 }
 
 b200_status b200_latent_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
                                  void* stream) {
   const KvLayerDev& L = kv->lay[c.layer];
+  if (c.q_stride != c.n_q_heads * L.kd) { b200_set_error("latent attention: query rows have to lie one behind the other"); return B200_ERR_INVALID_ARGUMENT; }
   if (c.window != 0 || c.slopes_log2) { b200_set_error("latent attention has no window and no distance bias"); return B200_ERR_UNSUPPORTED; }
   LatentArgs la;
   WinArgs& a = la.w;

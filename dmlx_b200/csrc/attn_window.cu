@@ -70,7 +70,7 @@ __device__ __forceinline__ int group_pages(int ctx_first, int ctx_last, int wind
 // and the combine pass.  It doubles until the partial slots fit the scratch (uncut groups need none), so a step always fits.
 __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict__ row_seq, const int* __restrict__ row_ctx, int total_rows,
                                                            int page_size, int window, int q_tokens, int items_per_chunk,
-                                                           int n_workers, int forced_ppc, int max_slots, int* __restrict__ group_first,
+                                                           int n_workers, int forced_ppc, int max_slots, float item_cost, float slot_cost, int* __restrict__ group_first,
                                                            int* __restrict__ chunk_start, int* __restrict__ part_base,
                                                            int* __restrict__ row_group, int* __restrict__ hdr) {
   __shared__ int warp_buf[32];
@@ -137,8 +137,8 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
       for (int k = 0; k < kCand; ++k) {
         const float length = fminf(k == kCand - 1 ? 1e9f : (float)(4 << k), (float)tot[2 * kCand + 1]);
         const float items = (float)tot[k] * per;
-        float t = fmaxf(load, length) + (items > 1.f ? 0.5f * length : 0.f) + 1.25f * items;
-        if (tot[kCand + k] > 0) t += 3.f + 0.25f * (float)tot[kCand + k] * per;
+        float t = fmaxf(load, length) + (items > 1.f ? 0.5f * length : 0.f) + item_cost * items;
+        if (tot[kCand + k] > 0) t += 3.f + slot_cost * (float)tot[kCand + k] * per;
         if (t < best) { best = t; carry_chunks = k; }
       }
     }
@@ -638,7 +638,7 @@ b200_status launch_mma_v(const b200_kv* kv, WinArgs& a, int layer, cudaStream_t 
 extern int b200_attn_pages_per_chunk;
 
 b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t items_per_chunk, int32_t n_workers, const int32_t* d_row_seq,
-                                const int32_t* d_row_ctx, int32_t total_rows, void* stream) {
+                                const int32_t* d_row_ctx, int32_t total_rows, void* stream, float item_cost, float slot_cost) {
   if (total_rows <= 0) return B200_OK;
   if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
   const int R = kv->cfg.max_rows + 2;
@@ -656,7 +656,7 @@ b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t
   }
   const int forced = b200_attn_pages_per_chunk <= 0 ? 0 : std::min(std::max(b200_attn_pages_per_chunk, 1), 1 << 20);
   window_plan_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(d_row_seq, d_row_ctx, total_rows, kv->cfg.page_size, window, qt,
-                                                          items_per_chunk, n_workers, forced, kv->max_chunks,
+                                                          items_per_chunk, n_workers, forced, kv->max_chunks, item_cost, slot_cost,
                                                           p->buf, p->buf + R, p->buf + 2 * R, p->buf + 3 * R, p->buf + 4 * R);
   B200_LAUNCH_CHECK();
   return B200_OK;
@@ -685,7 +685,7 @@ b200_status b200_window_attn_plan(b200_kv* kv, int32_t layer, int32_t window, in
   const KvLayerDev& L = kv->lay[layer];
   if (L.values_in_keys) return b200_latent_attn_plan(kv, layer, gqa, d_row_seq, d_row_ctx, total_rows, stream);
   const int per_chunk = L.heads * ((gqa + 15) / 16), warps = shape_of((L.kd + 63) / 64 + (L.vd + 63) / 64).warps;
-  return b200_attn_make_plan(kv, window, q_tokens_of(gqa), per_chunk, g_sms * warps, d_row_seq, d_row_ctx, total_rows, stream);
+  return b200_attn_make_plan(kv, window, q_tokens_of(gqa), per_chunk, g_sms * warps, d_row_seq, d_row_ctx, total_rows, stream, 1.25f, 0.25f);
 }
 
 b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,

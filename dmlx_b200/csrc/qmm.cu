@@ -2210,12 +2210,12 @@ extern "C" b200_status b200_qweight_random(int32_t mode, int32_t n_experts, int3
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
   if (mode < 0 || mode > B200_Q_BF16) { b200_set_error("unknown quantisation mode %d", mode); return B200_ERR_INVALID_QUANT_BITS; }
-  if (n_experts <= 0 || n <= 0 || k <= 0 || k % kChunkK != 0 || n % kTileN != 0) {
-    b200_set_error("random weights: N must be a multiple of 128 and K of 64");
+  if (n_experts <= 0 || n <= 0 || k <= 0 || k % kChunkK != 0 || (mode != B200_Q_BF16 && n % kTileN != 0)) {
+    b200_set_error("random weights: N must be a multiple of 128 (dense: any) and K of 64");
     return B200_ERR_INVALID_ARGUMENT;
   }
   auto* w = new b200_qweight();
-  w->mode = mode; w->n_experts = n_experts; w->n = n; w->k = k; w->nt = n / kTileN; w->kc = k / kChunkK;
+  w->mode = mode; w->n_experts = n_experts; w->n = n; w->k = k; w->nt = (n + kTileN - 1) / kTileN; w->kc = k / kChunkK;
   w->block_bytes = block_bytes(mode);
   const size_t n_blocks = (size_t)n_experts * w->nt * w->kc;
   cudaError_t e = cudaMalloc((void**)&w->d_blocks, n_blocks * w->block_bytes);

@@ -662,7 +662,7 @@ b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t whic
 b200_status b200_decoder_set_table(b200_decoder* m, int32_t layer, const int32_t* h_table, uint64_t n_elems);
 /* Fuses q/k/v and gate/up; fails, naming it, if a tensor the configuration needs was not set. */
 b200_status b200_decoder_finalize(b200_decoder* m);
-/* Synthetic weights generated on the device (benchmarks).  Matrix sizes must be multiples of 128. */
+/* Synthetic weights generated on the device (benchmarks).  Matrix sizes must be multiples of 64. */
 b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed);
 /* Cache layers the stack needs (a looped layer counts once per pass) and their shapes, for b200_kv_create_layers. */
 int32_t b200_decoder_cache_layers(const b200_decoder* m, b200_kv_layer* out, int32_t cap);
