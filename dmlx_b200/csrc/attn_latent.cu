@@ -121,7 +121,8 @@ namespace {
 
 constexpr int kTileKeys = 128, kTilePages = 4, kBoxBytes = kTileKeys * 128;  // bytes of a tile's 64-column box
 constexpr int kPBytes = kTileKeys * 128;
-constexpr int kLatentThreads = 256;    // warp 0 loads, warp 1 issues the MMAs, warps 4-7 softmax
+constexpr int kSoftmaxThreads = 256;   // two threads per key, each half of the rows
+constexpr int kLatentThreads = 128 + kSoftmaxThreads;  // warp 0 loads, warp 1 issues the MMAs, warps 4-11 softmax
 constexpr float kGrow = 8.f;           // log2 units a row's maximum may grow before its sums are rescaled
 constexpr uint32_t kPolls = 1u << 18;  // a wait inside a CTA is microseconds
 
@@ -131,25 +132,22 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// Barriers of the 128 softmax threads: true where every one (some one) of them passed true.
-__device__ __forceinline__ bool softmax_sync_and(bool x) {
+__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxThreads) : "memory"); }
+// ... and whether some thread passed true.
+__device__ __forceinline__ bool softmax_any(bool x) {
   uint32_t r;
-  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %1, 0;\n\tbar.red.and.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}" : "=r"(r) : "r"((uint32_t)x) : "memory");
-  return r != 0;
-}
-__device__ __forceinline__ bool softmax_sync_or(bool x) {
-  uint32_t r;
-  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %1, 0;\n\tbar.red.or.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}" : "=r"(r) : "r"((uint32_t)x) : "memory");
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %1, 0;\n\tbar.red.or.pred q, 1, %2, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+               : "=r"(r) : "r"((uint32_t)x), "n"(kSoftmaxThreads) : "memory");
   return r != 0;
 }
 
-// Reduces NR values over the warp's lanes: every step hands half of the columns to the partner lane.  Lane l ends up with
-// column l (NR = 32) or l / 2 (NR = 16).
-template <int NR, bool MAX>
-__device__ __forceinline__ float transpose_reduce(float (&w)[NR], int lane) {
+// Reduces N values over the warp's lanes: every step hands half of the columns to the partner lane.  Lane l ends up with
+// column l / (32 / N).
+template <int N, bool MAX>
+__device__ __forceinline__ float transpose_reduce(float (&w)[N], int lane) {
   int o = 16;
 #pragma unroll
-  for (int n = NR / 2; n >= 1; n >>= 1) {
+  for (int n = N / 2; n >= 1; n >>= 1) {
     const bool up = lane & o;
 #pragma unroll
     for (int i = 0; i < n; ++i) {
@@ -159,21 +157,23 @@ __device__ __forceinline__ float transpose_reduce(float (&w)[NR], int lane) {
     }
     o >>= 1;
   }
-  if (NR == 16) {
-    const float got = __shfl_xor_sync(0xffffffffu, w[0], 1);
+#pragma unroll
+  for (int b = 16 / N; b >= 1; b >>= 1) {
+    const float got = __shfl_xor_sync(0xffffffffu, w[0], b);
     w[0] = MAX ? fmaxf(w[0], got) : w[0] + got;
   }
   return w[0];
 }
 
-template <int NR>
-__device__ __forceinline__ void load_rows(uint32_t taddr, float (&v)[NR]) {
-  uint32_t u[NR / 16][16];
-#pragma unroll
-  for (int c = 0; c < NR / 16; ++c) ptx::tmem_ld16(taddr + c * 16, u[c]);
-  ptx::tmem_ld_wait();
-#pragma unroll
-  for (int c = 0; c < NR; ++c) v[c] = __uint_as_float(u[c / 16][c % 16]);
+template <int N>
+__device__ __forceinline__ void tmem_load(uint32_t taddr, uint32_t (&u)[N]) {
+  if constexpr (N == 8) ptx::tmem_ld8(taddr, u);
+  else ptx::tmem_ld16(taddr, u);
+}
+template <int N>
+__device__ __forceinline__ void tmem_store(uint32_t taddr, const uint32_t (&u)[N]) {
+  if constexpr (N == 8) ptx::tmem_st8(taddr, u);
+  else ptx::tmem_st16(taddr, u);
 }
 
 struct LatentArgs {
@@ -187,13 +187,16 @@ template <int NR>
 struct LatentShared {
   uint64_t k_full[4], k_free[4], s_full[2], p_ready, pv_done, q_full, q_free;
   long long off[NR];  // where a row's output starts
+  WinItem items[2];   // the loading thread looks an item up for everyone
   uint32_t tmem;
+  int dead;           // some wait ran out
   float red[4][NR], m[NR], corr[NR], l[NR];
   int ctx[NR];
 };
 
 template <int NR>
-__global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap qmap, LatentArgs la) {
+__global__ void __launch_bounds__(kLatentThreads, 1)
+    latent_attn_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap qmap, LatentArgs la) {
   const WinArgs& a = la.w;
   extern __shared__ unsigned char latent_dyn[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(latent_dyn) + 1023) & ~(uintptr_t)1023);
@@ -207,11 +210,12 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
     for (int s = 0; s < stages; ++s) { ptx::mbar_init(&sh.k_full[s], 1); ptx::mbar_init(&sh.k_free[s], 1); }
     ptx::mbar_init(&sh.s_full[0], 1);
     ptx::mbar_init(&sh.s_full[1], 1);
-    ptx::mbar_init(&sh.p_ready, 128);
+    ptx::mbar_init(&sh.p_ready, kSoftmaxThreads);
     ptx::mbar_init(&sh.pv_done, 1);
     ptx::mbar_init(&sh.q_full, 1);
     ptx::mbar_init(&sh.q_free, 1);
     ptx::mbar_fence_init();
+    sh.dead = 0;
   }
   if (warp == 1) {
     ptx::tmem_alloc(&sh.tmem, la.tmem_cols);
@@ -229,22 +233,34 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
       uint32_t ph = 0, issued = 0, n_item = 0;
       for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
         const WinItem it = decode_item(a, item, n_groups);
-        // the tile's rows lie one behind the other: tokens of the group, or heads of the block (what follows them is never stored)
+        const int* table = a.d.block_table + (size_t)it.seq * a.d.max_pages_per_seq;
+        int next[kTilePages];  // page ids of the coming tile, asked for before the wait
+#pragma unroll
+        for (int p = 0; p < kTilePages; ++p) next[p] = it.page_begin + p < it.page_end ? table[it.page_begin + p] : 0;
         ok = wait(&sh.q_free, (n_item & 1u) ^ 1u);
         if (!ok) break;
+        sh.items[n_item & 1u] = it;
+        // the tile's rows lie one behind the other: tokens of the group, or heads of the block (what follows them is never stored)
         ptx::mbar_expect_tx(&sh.q_full, n_kb * NR * 128);
         for (int b = 0; b < n_kb; ++b)
           ptx::tma_load_2d(qbuf + b * NR * 128, &qmap, b * 64, it.first_row * a.n_q_heads + it.block * a.head_block, &sh.q_full);
-        const int* table = a.d.block_table + (size_t)it.seq * a.d.max_pages_per_seq;
         for (int pg = it.page_begin; pg < it.page_end; pg += kTilePages) {
           const int pages = min(kTilePages, it.page_end - pg);
+          int id[kTilePages];
+#pragma unroll
+          for (int p = 0; p < kTilePages; ++p) {
+            id[p] = next[p];
+            const int ahead = pg + kTilePages + p;
+            next[p] = ahead < it.page_end ? table[ahead] : 0;
+          }
           ok = wait(&sh.k_free[s], ph ^ 1u);
           if (!ok) break;
           ptx::mbar_expect_tx(&sh.k_full[s], pages * n_kb * 4096);
-          for (int p = 0; p < pages; ++p) {
-            const int row0 = table[pg + p] * 32;
-            for (int b = 0; b < n_kb; ++b)
-              ptx::tma_load_2d(smem + (size_t)s * stage_bytes + b * kBoxBytes + p * 4096, &kmap, b * 64, row0, &sh.k_full[s]);
+          unsigned char* dst = smem + (size_t)s * stage_bytes;
+          for (int b = 0; b < n_kb; ++b) {
+#pragma unroll
+            for (int p = 0; p < kTilePages; ++p)
+              if (p < pages) ptx::tma_load_2d(dst + b * kBoxBytes + p * 4096, &kmap, b * 64, id[p] * 32, &sh.k_full[s]);
           }
           ++issued;
           if (++s == stages) { s = 0; ph ^= 1u; }
@@ -259,18 +275,21 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
     if (lane == 0) {  // ---- matrix products ----
       const uint32_t id_s = ptx::umma_idesc_bf16(128, NR), id_o = ptx::umma_idesc_bf16(128, 2 * NR) | ptx::kUmmaAMn | ptx::kUmmaBMn;
       const int n_ks = a.L.kd / 16;
-      const uint32_t q0 = ptx::smem_u32(qbuf), p0 = ptx::smem_u32(pbuf), t0 = ptx::smem_u32(smem);
+      // descriptors advance by adding to their address field (16-byte units)
+      const uint64_t q_desc = ptx::umma_desc_k_sw128(ptx::smem_u32(qbuf)), k_desc = ptx::umma_desc_k_sw128(ptx::smem_u32(smem));
+      const uint64_t v_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(smem), kBoxBytes), p_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(pbuf), kPBytes);
       int sc = 0, sp = 0;  // stage of the next tile to score, of the next to sum
       uint32_t phc = 0, n_scored = 0, n_summed = 0, n_item = 0;
       auto score = [&](bool last) {  // the next tile's S^T
         ok = wait(&sh.k_full[sc], phc);
         if (!ok) return;
         ptx::tc_fence_after_sync();
-        const uint32_t kt = t0 + sc * stage_bytes, dst = tmem + (n_scored & 1u) * NR;
-        for (int ks = 0; ks < n_ks; ++ks) {
-          const uint64_t da = ptx::umma_desc_k_sw128(kt + (ks >> 2) * kBoxBytes) + 2 * (ks & 3);
-          const uint64_t db = ptx::umma_desc_k_sw128(q0 + (ks >> 2) * NR * 128) + 2 * (ks & 3);
-          ptx::umma_bf16(dst, da, db, id_s, ks > 0 ? 1u : 0u);
+        const uint32_t dst = tmem + (n_scored & 1u) * NR;
+        uint64_t da = k_desc + (uint64_t)(sc * (stage_bytes >> 4)), db = q_desc;
+        for (int left = n_ks; left > 0; left -= 4, da += kBoxBytes >> 4, db += NR * 128 >> 4) {
+#pragma unroll
+          for (int k4 = 0; k4 < 4; ++k4)
+            if (k4 < left) ptx::umma_bf16(dst, da + 2 * k4, db + 2 * k4, id_s, left < n_ks || k4 > 0 ? 1u : 0u);
         }
         ptx::umma_commit(&sh.s_full[n_scored & 1u]);
         if (last) ptx::umma_commit(&sh.q_free);
@@ -278,10 +297,9 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
         if (++sc == stages) { sc = 0; phc ^= 1u; }
       };
       for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
-        const WinItem it = decode_item(a, item, n_groups);
-        const int tiles = (it.page_end - it.page_begin + kTilePages - 1) / kTilePages;
         ok = wait(&sh.q_full, n_item & 1u);
         if (!ok) break;
+        const int n_pages = sh.items[n_item & 1u].page_end - sh.items[n_item & 1u].page_begin, tiles = (n_pages + kTilePages - 1) / kTilePages;
         score(tiles == 1);
         for (int j = 0; j < tiles && ok; ++j) {
           if (stages > 1 && j + 1 < tiles) score(j + 2 == tiles);  // ahead of this tile's softmax
@@ -289,13 +307,12 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
           ok = wait(&sh.p_ready, n_summed & 1u);
           if (!ok) break;
           ptx::tc_fence_after_sync();
-          const int pages = min(kTilePages, it.page_end - it.page_begin - j * kTilePages);
-          const uint32_t kt = t0 + sp * stage_bytes;
+          const int pages = min(kTilePages, n_pages - j * kTilePages);
           for (int mc = 0; mc < n_mc; ++mc) {
-            for (int ks = 0; ks < 2 * pages; ++ks) {
-              const uint64_t da = ptx::umma_desc_mn_sw128(kt + 2 * mc * kBoxBytes + ks * 2048, kBoxBytes);
-              const uint64_t db = ptx::umma_desc_mn_sw128(p0 + ks * 2048, kPBytes);
-              ptx::umma_bf16(tmem_o + mc * 2 * NR, da, db, id_o, (j > 0 || ks > 0) ? 1u : 0u);
+            uint64_t da = v_desc + (uint64_t)(sp * (stage_bytes >> 4) + mc * (2 * kBoxBytes >> 4)), db = p_desc;
+            for (int pg = 0; pg < pages; ++pg, da += 4096 >> 4, db += 4096 >> 4) {
+              ptx::umma_bf16(tmem_o + mc * 2 * NR, da, db, id_o, j > 0 || pg > 0 ? 1u : 0u);
+              ptx::umma_bf16(tmem_o + mc * 2 * NR, da + (2048 >> 4), db + (2048 >> 4), id_o, 1u);
             }
           }
           ptx::umma_commit(&sh.k_free[sp]);
@@ -307,90 +324,110 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
       }
     }
   } else if (warp >= 4) {
-    // ---- softmax: thread = key of the tile = tensor-memory lane ----
-    const int key = tid - 128, quarter = warp - 4;
+    // ---- softmax: thread = (key of the tile = tensor-memory lane, half of the rows) ----
+    constexpr int NC = NR / 2;
+    const int quarter = warp & 3, key = quarter * 32 + lane, c0 = (warp >= 8 ? NC : 0), row = tid - 128;  // row < NR: this thread keeps it
     const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
-    uint32_t n_tile = 0, n_pv = 0;  // tiles scored / summed so far (phases of the barriers)
-    bool dead = false;              // some thread's wait ran out: decided together, so that all leave
-    for (int item = blockIdx.x; item < n_items && !dead; item += gridDim.x) {
-      const WinItem it = decode_item(a, item, n_groups);
-      const int hb = a.head_block, h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0);
-      if (key < NR) {
-        const int tok = key / hb, head = key - tok * hb;
-        sh.ctx[key] = tok < it.n_rows && head < heads_here ? it.ctx0 + tok : 0;
-        sh.m[key] = kAttnNone;
-        sh.off[key] = it.slot0 >= 0 ? ((long long)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd
+    const int hb = a.head_block;
+    uint32_t n_tile = 0, n_pv = 0, n_item = 0;  // tiles scored / summed so far, items (phases of the barriers)
+    bool dead = false;                          // some thread's wait ran out: decided together, so that all leave
+    for (int item = blockIdx.x; item < n_items && !dead; item += gridDim.x, ++n_item) {
+      ok = wait(&sh.q_full, n_item & 1u) && ok;
+      const WinItem it = sh.items[n_item & 1u];
+      const int h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0);
+      const int n_pages = ok ? it.page_end - it.page_begin : 1;  // (a thread whose wait ran out goes along to the next common decision)
+      if (row < NR) {
+        const int tok = row / hb, head = row - tok * hb;
+        sh.ctx[row] = tok < it.n_rows && head < heads_here ? it.ctx0 + tok : 0;
+        sh.m[row] = kAttnNone;
+        sh.off[row] = it.slot0 >= 0 ? ((long long)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd
                                     : (long long)(it.first_row + tok) * a.out_stride + (long long)(h0 + head) * a.out_head;
       }
-      float l[NR];
+      float l[NC], m[NC];
 #pragma unroll
-      for (int r = 0; r < NR; ++r) l[r] = 0.f;
-      for (int pg = it.page_begin; pg < it.page_end; pg += kTilePages) {
-        const int pages = min(kTilePages, it.page_end - pg), tok0 = pg * 32;
+      for (int r = 0; r < NC; ++r) { l[r] = 0.f; m[r] = kAttnNone; }
+      if (softmax_any(!ok)) { dead = true; break; }  // (and what the first threads wrote is in place)
+      for (int pg = 0; pg < n_pages; pg += kTilePages) {
+        const int pages = min(kTilePages, n_pages - pg), tok0 = (it.page_begin + pg) * 32;
         ok = wait(&sh.s_full[n_tile & 1u], (n_tile >> 1) & 1u) && ok;
         ptx::tc_fence_after_sync();
         __syncwarp();
-        float v[NR];
-        load_rows<NR>(tmem + lanes + (n_tile & 1u) * NR, v);
-        ++n_tile;
-        const bool edge = tok0 + kTileKeys > it.ctx0 || pages < kTilePages, first = pg == it.page_begin;
-        if (first) softmax_sync_and(true);  // what the item's first threads wrote is in place
+        float v[NC];
         {
-          float w[NR];
+          uint32_t u[NC];
+          tmem_load<NC>(tmem + lanes + (n_tile & 1u) * NR + c0, u);
+          ptx::tmem_ld_wait();
+#pragma unroll
+          for (int r = 0; r < NC; ++r) v[r] = __uint_as_float(u[r]) * a.scale_log2;
+        }
+        ++n_tile;
+        if (tok0 + kTileKeys > it.ctx0 || pages < kTilePages) {
           const bool in_tile = key < pages * 32;
 #pragma unroll
-          for (int r = 0; r < NR; ++r) {
-            v[r] *= a.scale_log2;
-            if (edge) v[r] = in_tile && tok0 + key < sh.ctx[r] ? v[r] : kAttnNone;
-            w[r] = v[r];
-          }
-          const float mx = transpose_reduce<NR, true>(w, lane);
-          if (NR == 32) sh.red[quarter][lane] = mx;
-          else if ((lane & 1) == 0) sh.red[quarter][lane >> 1] = mx;
+          for (int r = 0; r < NC; ++r) v[r] = in_tile && tok0 + key < sh.ctx[c0 + r] ? v[r] : kAttnNone;
         }
-        if (!softmax_sync_and(ok)) { dead = true; break; }
-        bool moved = false;
-        if (key < NR) {
-          const float m_old = sh.m[key], mx = fmaxf(fmaxf(sh.red[0][key], sh.red[1][key]), fmaxf(sh.red[2][key], sh.red[3][key]));
-          moved = mx > m_old + kGrow;
-          sh.corr[key] = moved ? ex2(m_old - mx) : 1.f;
-          if (moved) sh.m[key] = mx;
-        }
-        const bool rescale = softmax_sync_or(moved) && !first;
+        // The scale of a row stays as it is unless some key exceeds it by 2^kGrow; only then are the maxima taken.
+        bool over = false;
+#pragma unroll
+        for (int r = 0; r < NC; ++r) over = over || v[r] > m[r] + kGrow;
+        if (!ok) { sh.dead = 1; over = true; }
+        const bool move = softmax_any(over), first = pg == 0;
         if (!first) {  // P and O are the previous tile's until its product is done
           ok = wait(&sh.pv_done, n_pv & 1u) && ok;
           ++n_pv;
           ptx::tc_fence_after_sync();
           __syncwarp();
         }
-        if (rescale) {
-          float corr[NR];
+        if (move) {
+          if (!ok) sh.dead = 1;
+          {
+            float w[NC];
 #pragma unroll
-          for (int r = 0; r < NR; ++r) { corr[r] = sh.corr[r]; l[r] *= corr[r]; }
-          for (int c = 0; c < n_mc * 2; ++c) {
+            for (int r = 0; r < NC; ++r) w[r] = v[r];
+            const float mx = transpose_reduce<NC, true>(w, lane);
+            if (lane % (32 / NC) == 0) sh.red[quarter][c0 + lane / (32 / NC)] = mx;
+          }
+          softmax_sync();
+          if (*(volatile int*)&sh.dead) { dead = true; break; }
+          if (row < NR) {
+            const float m_old = sh.m[row], mx = fmaxf(fmaxf(sh.red[0][row], sh.red[1][row]), fmaxf(sh.red[2][row], sh.red[3][row]));
+            const bool moved = mx > m_old + kGrow;
+            sh.corr[row] = moved ? ex2(m_old - mx) : 1.f;
+            if (moved) sh.m[row] = mx;
+          }
+          softmax_sync();
+          float corr[NC];
 #pragma unroll
-            for (int h = 0; h < NR / 16; ++h) {
-              uint32_t o[16];
-              ptx::tmem_ld16(tmem_o + lanes + c * NR + h * 16, o);
+          for (int r = 0; r < NC; ++r) { corr[r] = sh.corr[c0 + r]; m[r] = sh.m[c0 + r]; l[r] *= corr[r]; }
+          if (!first) {
+            for (int c = 0; c < n_mc; ++c) {
+              uint32_t o[2][NC];
+              const uint32_t at = tmem_o + lanes + c * 2 * NR + c0;
+              tmem_load<NC>(at, o[0]);
+              tmem_load<NC>(at + NR, o[1]);
               ptx::tmem_ld_wait();
 #pragma unroll
-              for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * corr[h * 16 + e]);
-              ptx::tmem_st16(tmem_o + lanes + c * NR + h * 16, o);
+              for (int e = 0; e < NC; ++e) {
+                o[0][e] = __float_as_uint(__uint_as_float(o[0][e]) * corr[e]);
+                o[1][e] = __float_as_uint(__uint_as_float(o[1][e]) * corr[e]);
+              }
+              tmem_store<NC>(at, o[0]);
+              tmem_store<NC>(at + NR, o[1]);
             }
+            ptx::tmem_st_wait();
           }
-          ptx::tmem_st_wait();
         }
 #pragma unroll
-        for (int r = 0; r < NR; r += 8) {
+        for (int r = 0; r < NC; r += 8) {
           uint32_t hi[4], lo[4];
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float p[2];
 #pragma unroll
             for (int f = 0; f < 2; ++f) {
-              const float x = v[r + 2 * e + f];
-              p[f] = x > kAttnNone ? ex2(x - sh.m[r + 2 * e + f]) : 0.f;
-              l[r + 2 * e + f] += p[f];
+              const int i = r + 2 * e + f;
+              p[f] = v[i] > kAttnNone ? ex2(v[i] - m[i]) : 0.f;
+              l[i] += p[f];
             }
             const __nv_bfloat162 h2 = __floats2bfloat162_rn(p[0], p[1]);
             const float2 back = __bfloat1622float2(h2);
@@ -398,7 +435,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
             hi[e] = *reinterpret_cast<const uint32_t*>(&h2);
             lo[e] = *reinterpret_cast<const uint32_t*>(&l2);
           }
-          const int c = r / 8;
+          const int c = (c0 + r) / 8;
           *reinterpret_cast<uint4*>(pbuf + key * 128 + ((c ^ (key & 7)) << 4)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
           *reinterpret_cast<uint4*>(pbuf + key * 128 + (((c + NR / 8) ^ (key & 7)) << 4)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         }
@@ -408,53 +445,50 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_attn_kernel(const __
       }
       if (dead) break;
       {
-        const float sum = transpose_reduce<NR, false>(l, lane);
-        if (NR == 32) sh.red[quarter][lane] = sum;
-        else if ((lane & 1) == 0) sh.red[quarter][lane >> 1] = sum;
+        const float sum = transpose_reduce<NC, false>(l, lane);
+        if (lane % (32 / NC) == 0) sh.red[quarter][c0 + lane / (32 / NC)] = sum;
       }
       ok = wait(&sh.pv_done, n_pv & 1u) && ok;
       ++n_pv;
-      if (!softmax_sync_and(ok)) { dead = true; break; }
+      if (softmax_any(!ok)) { dead = true; break; }
       ptx::tc_fence_after_sync();
-      if (key < NR && sh.ctx[key] > 0) {
-        float sum = sh.red[0][key] + sh.red[1][key] + sh.red[2][key] + sh.red[3][key], f = 1.f;
-        const float m = sh.m[key];
-        const int tok = key / hb, head = key - tok * hb;
+      if (row < NR && sh.ctx[row] > 0) {
+        float sum = sh.red[0][row] + sh.red[1][row] + sh.red[2][row] + sh.red[3][row], f = 1.f;
+        const float mr = sh.m[row];
+        const int tok = row / hb, head = row - tok * hb;
         if (it.slot0 < 0) {
           if (a.sinks) {
-            const float sk = a.sinks[h0 + head], mm = fmaxf(m, sk);
-            f = exp2f(m - mm);
+            const float sk = a.sinks[h0 + head], mm = fmaxf(mr, sk);
+            f = exp2f(mr - mm);
             sum = sum * f + exp2f(sk - mm);
           }
-          sh.l[key] = sum > 0.f ? f / sum : 0.f;
+          sh.l[row] = sum > 0.f ? f / sum : 0.f;
         } else {
           const size_t pidx = (size_t)(it.slot0 + tok) * a.n_q_heads + h0 + head;
-          a.part_ml[pidx * 2] = m;
+          a.part_ml[pidx * 2] = mr;
           a.part_ml[pidx * 2 + 1] = sum;
         }
       }
-      softmax_sync_and(true);
+      softmax_sync();
       for (int mc = 0; mc < n_mc; ++mc) {
-        float o[NR];
-        {
-          float lo[NR];
-          load_rows<NR>(tmem_o + lanes + mc * 2 * NR, o);
-          load_rows<NR>(tmem_o + lanes + mc * 2 * NR + NR, lo);
-#pragma unroll
-          for (int r = 0; r < NR; ++r) o[r] += lo[r];
-        }
+        uint32_t o[NC], rest[NC];
+        const uint32_t at = tmem_o + lanes + mc * 2 * NR + c0;
+        tmem_load<NC>(at, o);
+        tmem_load<NC>(at + NR, rest);
+        ptx::tmem_ld_wait();
         const int dim = mc * 128 + key;
 #pragma unroll
-        for (int r = 0; r < NR; ++r) {
-          if (sh.ctx[r] > 0) {
-            if (it.slot0 >= 0) { if (dim < a.L.vd) a.part_o[sh.off[r] + dim] = o[r]; }
-            else if (dim < a.L.value_dim) a.out[sh.off[r] + dim] = __float2bfloat16(o[r] * sh.l[r]);
+        for (int r = 0; r < NC; ++r) {
+          const float x = __uint_as_float(o[r]) + __uint_as_float(rest[r]);
+          if (sh.ctx[c0 + r] > 0) {
+            if (it.slot0 >= 0) { if (dim < a.L.vd) a.part_o[sh.off[c0 + r] + dim] = x; }
+            else if (dim < a.L.value_dim) a.out[sh.off[c0 + r] + dim] = __float2bfloat16(x * sh.l[c0 + r]);
           }
         }
         __syncwarp();
       }
       ptx::tc_fence_before_sync();
-      softmax_sync_and(true);  // sh.ctx and sh.l have been read
+      softmax_sync();  // sh.ctx, sh.off and sh.l have been read
     }
     ok = ok && !dead;
   }
