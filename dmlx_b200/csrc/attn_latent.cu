@@ -332,7 +332,8 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
     uint32_t n_tile = 0, n_pv = 0, n_item = 0;  // tiles scored / summed so far, items (phases of the barriers)
     bool dead = false;                          // some thread's wait ran out: decided together, so that all leave
     for (int item = blockIdx.x; item < n_items && !dead; item += gridDim.x, ++n_item) {
-      ok = wait(&sh.q_full, n_item & 1u) && ok;
+      // (not q_full: that barrier may be two phases on when the item before is still being written out)
+      ok = wait(&sh.s_full[n_tile & 1u], (n_tile >> 1) & 1u) && ok;
       const WinItem it = sh.items[n_item & 1u];
       const int h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0);
       const int n_pages = ok ? it.page_end - it.page_begin : 1;  // (a thread whose wait ran out goes along to the next common decision)

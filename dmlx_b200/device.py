@@ -282,6 +282,9 @@ class LayeredKVCache(PagedKVCache):
         out = torch.empty((t, hq, vd), dtype=q.dtype, device=q.device)
         _lib.check(lib.b200_decoder_attention(self._h, layer, _ptr(q), hq, window, scale, _ptr(sl), _ptr(sk), _ptr(row_seq), _ptr(row_ctx), t,
                                               int(mma), _ptr(out), hq * vd, _stream()))
+        word = self.error_word()
+        if word:
+            raise _lib.B200Error(word)
         return out
 
 
