@@ -285,11 +285,10 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         if (!ok) return;
         ptx::tc_fence_after_sync();
         const uint32_t dst = tmem + (n_scored & 1u) * NR;
-        uint64_t da = k_desc + (uint64_t)(sc * (stage_bytes >> 4)), db = q_desc;
-        for (int left = n_ks; left > 0; left -= 4, da += kBoxBytes >> 4, db += NR * 128 >> 4) {
-#pragma unroll
-          for (int k4 = 0; k4 < 4; ++k4)
-            if (k4 < left) ptx::umma_bf16(dst, da + 2 * k4, db + 2 * k4, id_s, left < n_ks || k4 > 0 ? 1u : 0u);
+        const uint64_t k0 = k_desc + (uint64_t)(sc * (stage_bytes >> 4));
+        for (int ks = 0; ks < n_ks; ++ks) {
+          const uint64_t box = ks >> 2, in = 2 * (ks & 3);
+          ptx::umma_bf16(dst, k0 + box * (kBoxBytes >> 4) + in, q_desc + box * (NR * 128 >> 4) + in, id_s, ks > 0 ? 1u : 0u);
         }
         ptx::umma_commit(&sh.s_full[n_scored & 1u]);
         if (last) ptx::umma_commit(&sh.q_free);
