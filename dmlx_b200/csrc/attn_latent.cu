@@ -2,13 +2,15 @@
 // taken to the query side (q_head <- W_uk^T q_head) and W_uv behind the weighted sum, so the pages are read once for all heads
 // and hold kv_rank + rot_dim numbers per token.
 //
-// latent_attn_kernel (tcgen05, bf16): a tile is 128 keys (four pages, one TMA box per 64 columns of a page) against up to 32 rows, a
-// row being (token of the group, head).  The operands are swapped, so the keys fill the M = 128 side whatever the number of rows:
-//   S^T [keys][rows] = K Q^T,          A = the tile as it lies (K-major), B = the rows' queries;
-//   O^T [latent][rows] += C^T P,       A = the same tile read the other way (its latent columns are the M side), B = P.
-// The softmax warps hold one key per thread; maxima over the keys go through a shuffle transpose.  P is written as two bf16 terms
-// (value and remainder) side by side, which the second product accumulates in separate columns, so weights keep 16 bits and the
-// tile is read once for both.  The running maximum a row is scaled by moves only when it has grown by 2^8.
+// latent_attn_kernel (tcgen05, bf16): half-tiles of 64 keys (two pages, one TMA box per 64 columns of a page) against up to 32 rows,
+// a row being (token of the group, head).  The operands are swapped, so the keys fill the M side whatever the number of rows:
+//   S^T [keys][rows] = K Q^T,          A = the keys as they lie (K-major), B = the rows' queries;
+//   O^T [latent][rows] += C^T P,       A = the same keys read the other way (their latent columns are the M side), B = P.
+// Even and odd half-tiles go through two groups of softmax warps with sums of their own, so that loads, products and softmax of
+// neighbours overlap; the groups are added up at the end of a work item.  A thread holds one key and half of the rows; maxima over
+// the keys go through a shuffle transpose, but only when some key exceeds a row's scale by 2^8 (then four correction warps, which
+// reach all lanes of the sums, rescale them).  P enters the second product as two bf16 terms (value and remainder): weights keep
+// 16 bits.
 #include <cuda_bf16.h>
 
 #include <algorithm>
@@ -119,10 +121,12 @@ b200_status b200_latent_prep(b200_kv* kv, const LatentPrep& p, const int32_t* d_
 // ---- tensor-core kernel ----------------------------------------------------------------------------------------------
 namespace {
 
-constexpr int kTileKeys = 128, kTilePages = 4, kBoxBytes = kTileKeys * 128;  // bytes of a tile's 64-column box
-constexpr int kPBytes = kTileKeys * 128;
-constexpr int kSoftmaxThreads = 256;   // two threads per key, each half of the rows
-constexpr int kLatentThreads = 128 + kSoftmaxThreads;  // warp 0 loads, warp 1 issues the MMAs, warps 4-11 softmax
+// A stage of the ring holds two half-tiles of 64 keys (two pages) per 64-column box, one behind the other, so that a product with
+// M = 128 can read either: its other 64 rows are then whatever lies in the other half, in tensor-memory lanes nobody reads.
+constexpr int kHalfKeys = 64, kHalfPages = 2, kHalfBytes = kHalfKeys * 128, kBoxBytes = 2 * kHalfBytes;
+constexpr int kPBytes = kHalfKeys * 128;
+constexpr int kLatentThreads = 512;    // warp 0 loads, warp 1 issues the MMAs, warps 4-11 softmax, 12-15 correction
+constexpr int kMaxStages = 4;
 constexpr float kGrow = 8.f;           // log2 units a row's maximum may grow before its sums are rescaled
 constexpr uint32_t kPolls = 1u << 18;  // a wait inside a CTA is microseconds
 
@@ -132,12 +136,12 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxThreads) : "memory"); }
+__device__ __forceinline__ void bar_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 // ... and whether some thread passed true.
-__device__ __forceinline__ bool softmax_any(bool x) {
+__device__ __forceinline__ bool bar_any(int id, int threads, bool x) {
   uint32_t r;
-  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %1, 0;\n\tbar.red.or.pred q, 1, %2, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
-               : "=r"(r) : "r"((uint32_t)x), "n"(kSoftmaxThreads) : "memory");
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %1, 0;\n\tbar.red.or.pred q, %2, %3, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+               : "=r"(r) : "r"((uint32_t)x), "r"(id), "r"(threads) : "memory");
   return r != 0;
 }
 
@@ -182,15 +186,16 @@ struct LatentArgs {
   uint32_t tmem_cols;
 };
 
-// Shared memory behind the tiles, the queries and P.
+// Shared memory behind the tiles, the queries and P.  [2]: half-tiles with an even and an odd number, which the two groups of
+// softmax warps take.
 template <int NR>
 struct LatentShared {
-  uint64_t k_full[4], k_free[4], s_full[2], p_ready, pv_done, q_full, q_free;
+  uint64_t k_full[kMaxStages][2], k_free[kMaxStages][2], s_full[2], p_ready[2], pv_done[2], c_req[2], c_done[2], q_full, q_free;
   long long off[NR];  // where a row's output starts
   WinItem items[2];   // the loading thread looks an item up for everyone
   uint32_t tmem;
-  int dead;           // some wait ran out
-  float red[4][NR], m[NR], corr[NR], l[NR];
+  int done;
+  float red[2][2][NR], m[2][NR], corr[2][NR], w[2][NR];
   int ctx[NR];
 };
 
@@ -203,19 +208,22 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, stages = a.stages, n_kb = la.n_kb, n_mc = la.n_mc;
   const int stage_bytes = n_kb * kBoxBytes;
   unsigned char* qbuf = smem + (size_t)stages * stage_bytes;  // [box][NR rows][128 B]
-  unsigned char* pbuf = qbuf + (size_t)n_kb * NR * 128;       // [key][NR values | NR remainders]
-  LatentShared<NR>& sh = *reinterpret_cast<LatentShared<NR>*>(pbuf + kPBytes);
+  unsigned char* pbuf = qbuf + (size_t)n_kb * NR * 128;       // [group][values, remainders][key][128 B, NR of 64 columns used]
+  LatentShared<NR>& sh = *reinterpret_cast<LatentShared<NR>*>(pbuf + 4 * kPBytes);
   const int n_groups = a.hdr[0], n_items = a.chunk_start[n_groups] * a.n_blocks;
   if (tid == 0) {
-    for (int s = 0; s < stages; ++s) { ptx::mbar_init(&sh.k_full[s], 1); ptx::mbar_init(&sh.k_free[s], 1); }
-    ptx::mbar_init(&sh.s_full[0], 1);
-    ptx::mbar_init(&sh.s_full[1], 1);
-    ptx::mbar_init(&sh.p_ready, kSoftmaxThreads);
-    ptx::mbar_init(&sh.pv_done, 1);
+    for (int h = 0; h < 2; ++h) {
+      for (int s = 0; s < stages; ++s) { ptx::mbar_init(&sh.k_full[s][h], 1); ptx::mbar_init(&sh.k_free[s][h], 1); }
+      ptx::mbar_init(&sh.s_full[h], 1);
+      ptx::mbar_init(&sh.p_ready[h], 128);
+      ptx::mbar_init(&sh.pv_done[h], 1);
+      ptx::mbar_init(&sh.c_req[h], 1);
+      ptx::mbar_init(&sh.c_done[h], 128);
+    }
     ptx::mbar_init(&sh.q_full, 1);
     ptx::mbar_init(&sh.q_free, 1);
     ptx::mbar_fence_init();
-    sh.dead = 0;
+    sh.done = 0;
   }
   if (warp == 1) {
     ptx::tmem_alloc(&sh.tmem, la.tmem_cols);
@@ -224,19 +232,19 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   ptx::tc_fence_before_sync();
   __syncthreads();
   ptx::tc_fence_after_sync();
-  const uint32_t tmem = sh.tmem, tmem_o = tmem + 2 * NR;  // S twice, then O: n_mc x [NR of the values | NR of the remainders]
+  const uint32_t tmem = sh.tmem, tmem_o = tmem + 2 * NR;  // S of the two groups, then O of the two: n_mc x NR columns each
   bool ok = true;
 
   if (warp == 0) {
     if (lane == 0) {  // ---- loads ----
       int s = 0;
-      uint32_t ph = 0, issued = 0, n_item = 0;
+      uint32_t used = 0, phase = 0, n_item = 0;  // bit 2 * stage + half: loaded before; parity of its next load
       for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
         const WinItem it = decode_item(a, item, n_groups);
         const int* table = a.d.block_table + (size_t)it.seq * a.d.max_pages_per_seq;
-        int next[kTilePages];  // page ids of the coming tile, asked for before the wait
+        int next[kHalfPages];  // page ids of the coming half-tile, asked for before the wait
 #pragma unroll
-        for (int p = 0; p < kTilePages; ++p) next[p] = it.page_begin + p < it.page_end ? table[it.page_begin + p] : 0;
+        for (int p = 0; p < kHalfPages; ++p) next[p] = it.page_begin + p < it.page_end ? table[it.page_begin + p] : 0;
         ok = wait(&sh.q_free, (n_item & 1u) ^ 1u);
         if (!ok) break;
         sh.items[n_item & 1u] = it;
@@ -244,177 +252,184 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         ptx::mbar_expect_tx(&sh.q_full, n_kb * NR * 128);
         for (int b = 0; b < n_kb; ++b)
           ptx::tma_load_2d(qbuf + b * NR * 128, &qmap, b * 64, it.first_row * a.n_q_heads + it.block * a.head_block, &sh.q_full);
-        for (int pg = it.page_begin; pg < it.page_end; pg += kTilePages) {
-          const int pages = min(kTilePages, it.page_end - pg);
-          int id[kTilePages];
+        int h = 0;
+        for (int pg = it.page_begin; pg < it.page_end; pg += kHalfPages) {
+          const int pages = min(kHalfPages, it.page_end - pg), slot = 2 * s + h;
+          int id[kHalfPages];
 #pragma unroll
-          for (int p = 0; p < kTilePages; ++p) {
+          for (int p = 0; p < kHalfPages; ++p) {
             id[p] = next[p];
-            const int ahead = pg + kTilePages + p;
+            const int ahead = pg + kHalfPages + p;
             next[p] = ahead < it.page_end ? table[ahead] : 0;
           }
-          ok = wait(&sh.k_free[s], ph ^ 1u);
+          ok = wait(&sh.k_free[s][h], ((phase >> slot) & 1u) ^ 1u);
           if (!ok) break;
-          ptx::mbar_expect_tx(&sh.k_full[s], pages * n_kb * 4096);
-          unsigned char* dst = smem + (size_t)s * stage_bytes;
-          for (int b = 0; b < n_kb; ++b) {
-#pragma unroll
-            for (int p = 0; p < kTilePages; ++p)
-              if (p < pages) ptx::tma_load_2d(dst + b * kBoxBytes + p * 4096, &kmap, b * 64, id[p] * 32, &sh.k_full[s]);
-          }
-          ++issued;
-          if (++s == stages) { s = 0; ph ^= 1u; }
+          ptx::mbar_expect_tx(&sh.k_full[s][h], pages * n_kb * 4096);
+          unsigned char* dst = smem + (size_t)s * stage_bytes + h * kHalfBytes;
+          for (int b = 0; b < n_kb; ++b)
+            for (int p = 0; p < pages; ++p) ptx::tma_load_2d(dst + b * kBoxBytes + p * 4096, &kmap, b * 64, id[p] * 32, &sh.k_full[s][h]);
+          used |= 1u << slot;
+          phase ^= 1u << slot;
+          h ^= 1;
+          if (h == 0 && ++s == stages) s = 0;
         }
+        if (h == 1 && ++s == stages) s = 0;  // an item starts on an even half-tile
       }
       if (!ok) {  // leave no copy in flight behind
         if (n_item > 0) wait(&sh.q_full, (n_item - 1) & 1u);
-        for (uint32_t i = issued > (uint32_t)stages ? issued - stages : 0; i < issued; ++i) wait(&sh.k_full[i % stages], (i / stages) & 1u);
+        for (int slot = 0; slot < 2 * stages; ++slot)
+          if (used >> slot & 1u) wait(&sh.k_full[slot >> 1][slot & 1], ((phase >> slot) & 1u) ^ 1u);
       }
     }
   } else if (warp == 1) {
     if (lane == 0) {  // ---- matrix products ----
-      const uint32_t id_s = ptx::umma_idesc_bf16(128, NR), id_o = ptx::umma_idesc_bf16(128, 2 * NR) | ptx::kUmmaAMn | ptx::kUmmaBMn;
+      const uint32_t id_s = ptx::umma_idesc_bf16(128, NR), id_o = id_s | ptx::kUmmaAMn | ptx::kUmmaBMn;
       const int n_ks = a.L.kd / 16;
       // descriptors advance by adding to their address field (16-byte units)
       const uint64_t q_desc = ptx::umma_desc_k_sw128(ptx::smem_u32(qbuf)), k_desc = ptx::umma_desc_k_sw128(ptx::smem_u32(smem));
       const uint64_t v_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(smem), kBoxBytes), p_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(pbuf), kPBytes);
-      int sc = 0, sp = 0;  // stage of the next tile to score, of the next to sum
-      uint32_t phc = 0, n_scored = 0, n_summed = 0, n_item = 0;
-      auto score = [&](bool last) {  // the next tile's S^T
-        ok = wait(&sh.k_full[sc], phc);
-        if (!ok) return;
-        ptx::tc_fence_after_sync();
-        const uint32_t dst = tmem + (n_scored & 1u) * NR;
-        const uint64_t k0 = k_desc + (uint64_t)(sc * (stage_bytes >> 4));
-        for (int ks = 0; ks < n_ks; ++ks) {
-          const uint64_t box = ks >> 2, in = 2 * (ks & 3);
-          ptx::umma_bf16(dst, k0 + box * (kBoxBytes >> 4) + in, q_desc + box * (NR * 128 >> 4) + in, id_s, ks > 0 ? 1u : 0u);
-        }
-        ptx::umma_commit(&sh.s_full[n_scored & 1u]);
-        if (last) ptx::umma_commit(&sh.q_free);
-        ++n_scored;
-        if (++sc == stages) { sc = 0; phc ^= 1u; }
-      };
+      int s0 = 0;  // stage of the item's first half-tile
+      uint32_t phase = 0, n_item = 0, n_p[2] = {0, 0};
       for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
         ok = wait(&sh.q_full, n_item & 1u);
         if (!ok) break;
-        const int n_pages = sh.items[n_item & 1u].page_end - sh.items[n_item & 1u].page_begin, tiles = (n_pages + kTilePages - 1) / kTilePages;
-        score(tiles == 1);
-        for (int j = 0; j < tiles && ok; ++j) {
-          if (stages > 1 && j + 1 < tiles) score(j + 2 == tiles);  // ahead of this tile's softmax
-          if (!ok) break;
-          ok = wait(&sh.p_ready, n_summed & 1u);
-          if (!ok) break;
-          ptx::tc_fence_after_sync();
-          const int pages = min(kTilePages, n_pages - j * kTilePages);
-          for (int mc = 0; mc < n_mc; ++mc) {
-            uint64_t da = v_desc + (uint64_t)(sp * (stage_bytes >> 4) + mc * (2 * kBoxBytes >> 4)), db = p_desc;
-            for (int pg = 0; pg < pages; ++pg, da += 4096 >> 4, db += 4096 >> 4) {
-              ptx::umma_bf16(tmem_o + mc * 2 * NR, da, db, id_o, j > 0 || pg > 0 ? 1u : 0u);
-              ptx::umma_bf16(tmem_o + mc * 2 * NR, da + (2048 >> 4), db + (2048 >> 4), id_o, 1u);
+        const int n_pages = sh.items[n_item & 1u].page_end - sh.items[n_item & 1u].page_begin, halves = (n_pages + kHalfPages - 1) / kHalfPages;
+        int scored = 0, summed = 0, ss = s0, ps = s0;  // half-tiles, and the stages of the next ones
+        uint32_t idle = 0;
+        // whichever of the two next products has its operands goes first
+        while (summed < halves) {
+          const int hs = scored & 1, hp = summed & 1, slot = 2 * ss + hs;
+          if (scored < halves && scored < summed + 2 && ptx::mbar_try_wait(&sh.k_full[ss][hs], (phase >> slot) & 1u)) {
+            ptx::tc_fence_after_sync();
+            const uint64_t k0 = k_desc + (uint64_t)(ss * (stage_bytes >> 4));
+            for (int ks = 0; ks < n_ks; ++ks) {
+              const uint64_t box = ks >> 2, in = 2 * (ks & 3);
+              ptx::umma_bf16(tmem + hs * NR, k0 + box * (kBoxBytes >> 4) + in, q_desc + box * (NR * 128 >> 4) + in, id_s, ks > 0 ? 1u : 0u);
             }
+            ptx::umma_commit(&sh.s_full[hs]);
+            phase ^= 1u << slot;
+            ++scored;
+            if (scored == halves) ptx::umma_commit(&sh.q_free);
+            if (hs == 1 && ++ss == stages) ss = 0;
+            idle = 0;
+          } else if (summed < scored && ptx::mbar_try_wait(&sh.p_ready[hp], n_p[hp] & 1u)) {
+            ptx::tc_fence_after_sync();
+            const int n_steps = 2 * min(kHalfPages, n_pages - summed * kHalfPages);
+            const uint64_t v0 = v_desc + (uint64_t)(ps * (stage_bytes >> 4) + hp * (kHalfBytes >> 4)), p0 = p_desc + (uint64_t)(hp * (2 * kPBytes >> 4));
+            for (int mc = 0; mc < n_mc; ++mc) {
+              const uint32_t dst = tmem_o + (hp * n_mc + mc) * NR;
+              for (int ks = 0; ks < n_steps; ++ks) {
+                const uint64_t va = v0 + (uint64_t)(mc * (2 * kBoxBytes >> 4) + ks * (2048 >> 4)), pb = p0 + (uint64_t)(ks * (2048 >> 4));
+                ptx::umma_bf16(dst, va, pb, id_o, summed > 1 || ks > 0 ? 1u : 0u);
+                ptx::umma_bf16(dst, va, pb + (kPBytes >> 4), id_o, 1u);
+              }
+            }
+            ptx::umma_commit(&sh.k_free[ps][hp]);
+            ptx::umma_commit(&sh.pv_done[hp]);
+            ++n_p[hp];
+            ++summed;
+            if (hp == 1 && ++ps == stages) ps = 0;
+            idle = 0;
+          } else if (++idle > kPolls) {
+            ok = false;
+            break;
+          } else if (idle > 64) {
+            __nanosleep(32);
           }
-          ptx::umma_commit(&sh.k_free[sp]);
-          ptx::umma_commit(&sh.pv_done);
-          ++n_summed;
-          if (++sp == stages) sp = 0;
-          if (stages == 1 && j + 1 < tiles) score(j + 2 == tiles);
         }
+        s0 += (halves + 1) / 2 % stages;
+        if (s0 >= stages) s0 -= stages;
       }
     }
-  } else if (warp >= 4) {
-    // ---- softmax: thread = (key of the tile = tensor-memory lane, half of the rows) ----
-    constexpr int NC = NR / 2;
-    const int quarter = warp & 3, key = quarter * 32 + lane, c0 = (warp >= 8 ? NC : 0), row = tid - 128;  // row < NR: this thread keeps it
+  } else if (warp >= 4 && warp < 12) {
+    // ---- softmax: group 0 takes the even half-tiles, group 1 the odd ones; thread = (key = tensor-memory lane, half of the rows) ----
+    constexpr int NC = NR / 2, kAll = 3, kAllThreads = 256;
+    const int quarter = warp & 3, g = quarter >> 1, key = (quarter & 1) * 32 + lane, c0 = warp >= 8 ? NC : 0;
+    const int row = (warp >= 8 ? 64 : 0) + key;  // thread of the group; row < NR: it keeps that row
     const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
     const int hb = a.head_block;
-    uint32_t n_tile = 0, n_pv = 0, n_item = 0;  // tiles scored / summed so far, items (phases of the barriers)
-    bool dead = false;                          // some thread's wait ran out: decided together, so that all leave
-    for (int item = blockIdx.x; item < n_items && !dead; item += gridDim.x, ++n_item) {
+    unsigned char* p_hi = pbuf + g * 2 * kPBytes + key * 128;
+    uint32_t n_s = 0, n_pv = 0, n_c = 0, n_item = 0;  // half-tiles of the group scored / summed, rescalings, items (phases of the barriers)
+    bool dead = false;                       // some thread's wait ran out: decided together, so that all leave
+    for (int item = blockIdx.x; item < n_items; item += gridDim.x, ++n_item) {
       // (not q_full: that barrier may be two phases on when the item before is still being written out)
-      ok = wait(&sh.s_full[n_tile & 1u], (n_tile >> 1) & 1u) && ok;
+      if (g == 0) ok = wait(&sh.s_full[0], n_s & 1u) && ok;
+      if (bar_any(kAll, kAllThreads, !ok)) { dead = true; break; }
       const WinItem it = sh.items[n_item & 1u];
-      const int h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0);
-      const int n_pages = ok ? it.page_end - it.page_begin : 1;  // (a thread whose wait ran out goes along to the next common decision)
+      const int h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0), n_pages = it.page_end - it.page_begin;
+      const int halves = (n_pages + kHalfPages - 1) / kHalfPages;
       if (row < NR) {
-        const int tok = row / hb, head = row - tok * hb;
-        sh.ctx[row] = tok < it.n_rows && head < heads_here ? it.ctx0 + tok : 0;
-        sh.m[row] = kAttnNone;
-        sh.off[row] = it.slot0 >= 0 ? ((long long)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd
-                                    : (long long)(it.first_row + tok) * a.out_stride + (long long)(h0 + head) * a.out_head;
+        if (g == 0) {
+          const int tok = row / hb, head = row - tok * hb;
+          sh.ctx[row] = tok < it.n_rows && head < heads_here ? it.ctx0 + tok : 0;
+          sh.off[row] = it.slot0 >= 0 ? ((long long)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd
+                                      : (long long)(it.first_row + tok) * a.out_stride + (long long)(h0 + head) * a.out_head;
+        }
+        sh.m[g][row] = kAttnNone;
       }
       float l[NC], m[NC];
 #pragma unroll
       for (int r = 0; r < NC; ++r) { l[r] = 0.f; m[r] = kAttnNone; }
-      if (softmax_any(!ok)) { dead = true; break; }  // (and what the first threads wrote is in place)
-      for (int pg = 0; pg < n_pages; pg += kTilePages) {
-        const int pages = min(kTilePages, n_pages - pg), tok0 = (it.page_begin + pg) * 32;
-        ok = wait(&sh.s_full[n_tile & 1u], (n_tile >> 1) & 1u) && ok;
+      bar_sync(kAll, kAllThreads);
+      bool broken = false;
+      for (int j = g; j < halves; j += 2) {
+        const int pages = min(kHalfPages, n_pages - j * kHalfPages), tok0 = (it.page_begin + j * kHalfPages) * 32;
+        const bool first = j == g;
+        ok = wait(&sh.s_full[g], n_s & 1u) && ok;
+        ++n_s;
         ptx::tc_fence_after_sync();
         __syncwarp();
         float v[NC];
         {
           uint32_t u[NC];
-          tmem_load<NC>(tmem + lanes + (n_tile & 1u) * NR + c0, u);
+          tmem_load<NC>(tmem + lanes + g * NR + c0, u);
           ptx::tmem_ld_wait();
 #pragma unroll
           for (int r = 0; r < NC; ++r) v[r] = __uint_as_float(u[r]) * a.scale_log2;
         }
-        ++n_tile;
-        if (tok0 + kTileKeys > it.ctx0 || pages < kTilePages) {
+        if (tok0 + kHalfKeys > it.ctx0 || pages < kHalfPages) {
           const bool in_tile = key < pages * 32;
 #pragma unroll
           for (int r = 0; r < NC; ++r) v[r] = in_tile && tok0 + key < sh.ctx[c0 + r] ? v[r] : kAttnNone;
         }
         // The scale of a row stays as it is unless some key exceeds it by 2^kGrow; only then are the maxima taken.
-        bool over = false;
+        bool over = !ok;
 #pragma unroll
         for (int r = 0; r < NC; ++r) over = over || v[r] > m[r] + kGrow;
-        if (!ok) { sh.dead = 1; over = true; }
-        const bool move = softmax_any(over), first = pg == 0;
-        if (!first) {  // P and O are the previous tile's until its product is done
-          ok = wait(&sh.pv_done, n_pv & 1u) && ok;
+        const bool move = bar_any(1 + g, 128, over);
+        if (!first) {  // P and O are the previous half-tile's until its product is done
+          ok = wait(&sh.pv_done[g], n_pv & 1u) && ok;
           ++n_pv;
           ptx::tc_fence_after_sync();
           __syncwarp();
         }
         if (move) {
-          if (!ok) sh.dead = 1;
           {
             float w[NC];
 #pragma unroll
             for (int r = 0; r < NC; ++r) w[r] = v[r];
             const float mx = transpose_reduce<NC, true>(w, lane);
-            if (lane % (32 / NC) == 0) sh.red[quarter][c0 + lane / (32 / NC)] = mx;
+            if (lane % (32 / NC) == 0) sh.red[g][quarter & 1][c0 + lane / (32 / NC)] = mx;
           }
-          softmax_sync();
-          if (*(volatile int*)&sh.dead) { dead = true; break; }
+          if (bar_any(1 + g, 128, !ok)) { broken = true; break; }
           if (row < NR) {
-            const float m_old = sh.m[row], mx = fmaxf(fmaxf(sh.red[0][row], sh.red[1][row]), fmaxf(sh.red[2][row], sh.red[3][row]));
+            const float m_old = sh.m[g][row], mx = fmaxf(sh.red[g][0][row], sh.red[g][1][row]);
             const bool moved = mx > m_old + kGrow;
-            sh.corr[row] = moved ? ex2(m_old - mx) : 1.f;
-            if (moved) sh.m[row] = mx;
+            sh.corr[g][row] = moved ? ex2(m_old - mx) : 1.f;
+            if (moved) sh.m[g][row] = mx;
           }
-          softmax_sync();
+          bar_sync(1 + g, 128);
           float corr[NC];
 #pragma unroll
-          for (int r = 0; r < NC; ++r) { corr[r] = sh.corr[c0 + r]; m[r] = sh.m[c0 + r]; l[r] *= corr[r]; }
-          if (!first) {
-            for (int c = 0; c < n_mc; ++c) {
-              uint32_t o[2][NC];
-              const uint32_t at = tmem_o + lanes + c * 2 * NR + c0;
-              tmem_load<NC>(at, o[0]);
-              tmem_load<NC>(at + NR, o[1]);
-              ptx::tmem_ld_wait();
-#pragma unroll
-              for (int e = 0; e < NC; ++e) {
-                o[0][e] = __float_as_uint(__uint_as_float(o[0][e]) * corr[e]);
-                o[1][e] = __float_as_uint(__uint_as_float(o[1][e]) * corr[e]);
-              }
-              tmem_store<NC>(at, o[0]);
-              tmem_store<NC>(at + NR, o[1]);
-            }
-            ptx::tmem_st_wait();
+          for (int r = 0; r < NC; ++r) { corr[r] = sh.corr[g][c0 + r]; m[r] = sh.m[g][c0 + r]; l[r] *= corr[r]; }
+        }
+          if (!first) {  // the sums lie in all 128 lanes, half of which this group's warps cannot reach
+            ptx::tc_fence_before_sync();
+            if (row == 0) ptx::mbar_arrive(&sh.c_req[g]);
+            ok = wait(&sh.c_done[g], n_c & 1u) && ok;
+            ++n_c;
+            ptx::tc_fence_after_sync();
+            __syncwarp();
           }
         }
 #pragma unroll
@@ -435,62 +450,113 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
             hi[e] = *reinterpret_cast<const uint32_t*>(&h2);
             lo[e] = *reinterpret_cast<const uint32_t*>(&l2);
           }
-          const int c = (c0 + r) / 8;
-          *reinterpret_cast<uint4*>(pbuf + key * 128 + ((c ^ (key & 7)) << 4)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(pbuf + key * 128 + (((c + NR / 8) ^ (key & 7)) << 4)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          const int at = ((((c0 + r) / 8) ^ (key & 7)) << 4);
+          *reinterpret_cast<uint4*>(p_hi + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4*>(p_hi + kPBytes + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         }
         ptx::fence_proxy_async_smem();
         ptx::tc_fence_before_sync();
-        ptx::mbar_arrive(&sh.p_ready);
+        ptx::mbar_arrive(&sh.p_ready[g]);
       }
-      if (dead) break;
+      if (!broken && g < halves) {
+        ok = wait(&sh.pv_done[g], n_pv & 1u) && ok;
+        ++n_pv;
+      }
       {
         const float sum = transpose_reduce<NC, false>(l, lane);
-        if (lane % (32 / NC) == 0) sh.red[quarter][c0 + lane / (32 / NC)] = sum;
+        if (lane % (32 / NC) == 0) sh.red[g][quarter & 1][c0 + lane / (32 / NC)] = sum;
       }
-      ok = wait(&sh.pv_done, n_pv & 1u) && ok;
-      ++n_pv;
-      if (softmax_any(!ok)) { dead = true; break; }
+      if (bar_any(kAll, kAllThreads, !ok)) { dead = true; break; }
       ptx::tc_fence_after_sync();
-      if (row < NR && sh.ctx[row] > 0) {
-        float sum = sh.red[0][row] + sh.red[1][row] + sh.red[2][row] + sh.red[3][row], f = 1.f;
-        const float mr = sh.m[row];
+      if (g == 0 && row < NR && sh.ctx[row] > 0) {
+        // the two groups' sums at a common scale
+        const float m0 = sh.m[0][row], m1 = sh.m[1][row], mr = fmaxf(m0, m1);
+        float w0 = ex2(m0 - mr), w1 = ex2(m1 - mr);
+        float sum = w0 * (sh.red[0][0][row] + sh.red[0][1][row]) + w1 * (sh.red[1][0][row] + sh.red[1][1][row]);
         const int tok = row / hb, head = row - tok * hb;
         if (it.slot0 < 0) {
+          float f = 1.f;
           if (a.sinks) {
             const float sk = a.sinks[h0 + head], mm = fmaxf(mr, sk);
             f = exp2f(mr - mm);
             sum = sum * f + exp2f(sk - mm);
           }
-          sh.l[row] = sum > 0.f ? f / sum : 0.f;
+          const float inv = sum > 0.f ? f / sum : 0.f;
+          w0 *= inv;
+          w1 *= inv;
         } else {
           const size_t pidx = (size_t)(it.slot0 + tok) * a.n_q_heads + h0 + head;
           a.part_ml[pidx * 2] = mr;
           a.part_ml[pidx * 2 + 1] = sum;
         }
+        sh.w[0][row] = w0;
+        sh.w[1][row] = w1;
       }
-      softmax_sync();
+      bar_sync(kAll, kAllThreads);
       for (int mc = 0; mc < n_mc; ++mc) {
-        uint32_t o[NC], rest[NC];
-        const uint32_t at = tmem_o + lanes + mc * 2 * NR + c0;
-        tmem_load<NC>(at, o);
-        tmem_load<NC>(at + NR, rest);
+        uint32_t o[NC], odd[NC];
+        tmem_load<NC>(tmem_o + lanes + mc * NR + c0, o);
+        if (halves > 1) tmem_load<NC>(tmem_o + lanes + (n_mc + mc) * NR + c0, odd);
         ptx::tmem_ld_wait();
-        const int dim = mc * 128 + key;
+        const int dim = mc * 128 + quarter * 32 + lane;
 #pragma unroll
         for (int r = 0; r < NC; ++r) {
-          const float x = __uint_as_float(o[r]) + __uint_as_float(rest[r]);
+          float x = __uint_as_float(o[r]) * sh.w[0][c0 + r];
+          if (halves > 1) x = fmaf(__uint_as_float(odd[r]), sh.w[1][c0 + r], x);
           if (sh.ctx[c0 + r] > 0) {
             if (it.slot0 >= 0) { if (dim < a.L.vd) a.part_o[sh.off[c0 + r] + dim] = x; }
-            else if (dim < a.L.value_dim) a.out[sh.off[c0 + r] + dim] = __float2bfloat16(x * sh.l[c0 + r]);
+            else if (dim < a.L.value_dim) a.out[sh.off[c0 + r] + dim] = __float2bfloat16(x);
           }
         }
         __syncwarp();
       }
       ptx::tc_fence_before_sync();
-      softmax_sync();  // sh.ctx, sh.off and sh.l have been read
+      bar_sync(kAll, kAllThreads);  // the item's shared values have been read
     }
     ok = ok && !dead;
+    if (g == 0 && row == 0) *(volatile int*)&sh.done = 1;
+  }
+  if (warp >= 12) {
+    // ---- correction: rescales a group's sums when one of its rows' scales has moved ----
+    const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
+    uint32_t n_c[2] = {0, 0}, idle = 0;
+    bool go = true;
+    while (go) {
+      int what = -1;
+      if (lane == 0) {
+        const bool done = *(volatile int*)&sh.done != 0;  // (before the requests: none comes after it)
+        for (int g = 0; g < 2 && what < 0; ++g)
+          if (ptx::mbar_try_wait(&sh.c_req[g], n_c[g] & 1u)) what = g;
+        if (what < 0 && (done || ++idle > (1u << 24))) what = done ? 2 : 3;
+      }
+      what = __shfl_sync(0xffffffffu, what, 0);
+      if (what >= 2) {
+        ok = what == 2;
+        break;
+      }
+      if (what < 0) {
+        __nanosleep(100);
+        continue;
+      }
+      const int g = what;
+      ++n_c[g];
+      idle = 0;
+      ptx::tc_fence_after_sync();
+      for (int mc = 0; mc < n_mc; ++mc) {
+        for (int c = 0; c < NR; c += 16) {
+          uint32_t o[16];
+          const uint32_t at = tmem_o + lanes + (g * n_mc + mc) * NR + c;
+          ptx::tmem_ld16(at, o);
+          ptx::tmem_ld_wait();
+#pragma unroll
+          for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * sh.corr[g][c + e]);
+          ptx::tmem_st16(at, o);
+        }
+      }
+      ptx::tmem_st_wait();
+      ptx::tc_fence_before_sync();
+      ptx::mbar_arrive(&sh.c_done[g]);
+    }
   }
   if (!ok) atomicExch(a.d.state + ST_ATTN_ERR, B200_ERR_DEVICE_FLAGGED);
   ptx::tc_fence_before_sync();
@@ -503,11 +569,13 @@ constexpr int kSmemLimit = 227 * 1024;
 
 template <int NR>
 size_t smem_of(int n_kb, int stages) {
-  return (size_t)stages * n_kb * kBoxBytes + (size_t)n_kb * NR * 128 + kPBytes + sizeof(LatentShared<NR>) + 1024;
+  return (size_t)stages * n_kb * kBoxBytes + (size_t)n_kb * NR * 128 + 4 * kPBytes + sizeof(LatentShared<NR>) + 1024;
 }
 
-// Rows of a tile: 16 where a decode step would leave more of them empty.
-int rows_of(int heads, int total_rows) { return heads <= 16 && total_rows <= 256 ? 16 : 32; }
+// Rows of a tile: 16 where a decode step would leave more of them empty, or where the keys leave no room for 32.
+int rows_of(const KvLayerDev& L, int heads, int total_rows) {
+  return (heads <= 16 && total_rows <= 256) || smem_of<32>((L.kd + 63) / 64, 1) > kSmemLimit ? 16 : 32;
+}
 
 template <int NR>
 b200_status launch(const b200_kv* kv, LatentArgs& la, int layer, cudaStream_t s) {
@@ -516,11 +584,11 @@ b200_status launch(const b200_kv* kv, LatentArgs& la, int layer, cudaStream_t s)
   const uint32_t box[2] = {64, (uint32_t)NR};
   b200_status st = b200_make_tensor_map(&qmap, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, la.w.q, dims, strides, box);
   if (st != B200_OK) return st;
-  int stages = 4;
+  int stages = kMaxStages;
   while (stages > 1 && smem_of<NR>(la.n_kb, stages) > kSmemLimit) --stages;
   la.w.stages = stages;
   la.tmem_cols = 32;
-  while (la.tmem_cols < (uint32_t)(2 * NR + la.n_mc * 2 * NR)) la.tmem_cols <<= 1;
+  while (la.tmem_cols < (uint32_t)(2 * NR + 2 * la.n_mc * NR)) la.tmem_cols <<= 1;
   static bool configured = false;
   if (!configured) {
     B200_CUDA_TRY(cudaFuncSetAttribute(latent_attn_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit));
@@ -535,7 +603,7 @@ b200_status launch(const b200_kv* kv, LatentArgs& la, int layer, cudaStream_t s)
 
 bool b200_latent_attn_takes_mma(const b200_kv* kv, int32_t layer) {
   const KvLayerDev& L = kv->lay[layer];
-  return kv->layered && L.values_in_keys && L.heads == 1 && kv->dev.elem_bytes == 2 && smem_of<32>((L.kd + 63) / 64, 1) <= kSmemLimit &&
+  return kv->layered && L.values_in_keys && L.heads == 1 && kv->dev.elem_bytes == 2 && smem_of<16>((L.kd + 63) / 64, 1) <= kSmemLimit &&
          64 + (L.value_dim + 127) / 128 * 64 <= 512;
 }
 
@@ -546,7 +614,7 @@ b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t heads, con
     B200_CUDA_TRY(cudaGetDevice(&dev));
     B200_CUDA_TRY(cudaDeviceGetAttribute(&g_sms, cudaDevAttrMultiProcessorCount, dev));
   }
-  const int rows = rows_of(heads, total_rows);
+  const int rows = rows_of(kv->lay[layer], heads, total_rows);
   return b200_attn_make_plan(kv, 0, std::max(1, rows / heads), (heads + rows - 1) / rows, g_sms, d_row_seq, d_row_ctx, total_rows, stream, 4.f,
                              8.f * std::min(heads, rows) * kv->lay[layer].value_dim / (64.f * kv->lay[layer].kd));
 }
@@ -558,7 +626,7 @@ b200_status b200_latent_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
   if (c.window != 0 || c.slopes_log2) { b200_set_error("latent attention has no window and no distance bias"); return B200_ERR_UNSUPPORTED; }
   LatentArgs la;
   WinArgs& a = la.w;
-  const int rows = rows_of(c.n_q_heads, total_rows), hb = std::min(c.n_q_heads, rows);
+  const int rows = rows_of(L, c.n_q_heads, total_rows), hb = std::min(c.n_q_heads, rows);
   if (!b200_attn_use_plan(kv, 0, std::max(1, rows / c.n_q_heads), &a)) return B200_ERR_INVALID_ARGUMENT;
   a.d = kv->dev; a.L = L; a.L.vd = (L.value_dim + 15) / 16 * 16;
   a.q = (const __nv_bfloat16*)c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx;
