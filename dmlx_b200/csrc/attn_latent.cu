@@ -422,7 +422,6 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
           float corr[NC];
 #pragma unroll
           for (int r = 0; r < NC; ++r) { corr[r] = sh.corr[g][c0 + r]; m[r] = sh.m[g][c0 + r]; l[r] *= corr[r]; }
-        }
           if (!first) {  // the sums lie in all 128 lanes, half of which this group's warps cannot reach
             ptx::tc_fence_before_sync();
             if (row == 0) ptx::mbar_arrive(&sh.c_req[g]);
