@@ -282,9 +282,8 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {  // ---- matrix products ----
+    if (ptx::elect_one()) {  // ---- matrix products ----
       const uint32_t id_s = ptx::umma_idesc_bf16(128, NR), id_o = id_s | ptx::kUmmaAMn | ptx::kUmmaBMn;
-      const int n_ks = a.L.kd / 16;
       // descriptors advance by adding to their address field (16-byte units)
       const uint64_t q_desc = ptx::umma_desc_k_sw128(ptx::smem_u32(qbuf)), k_desc = ptx::umma_desc_k_sw128(ptx::smem_u32(smem));
       const uint64_t v_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(smem), kBoxBytes), p_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(pbuf), kPBytes);
@@ -302,9 +301,10 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
           if (scored < halves && scored < summed + 2 && ptx::mbar_try_wait(&sh.k_full[ss][hs], (phase >> slot) & 1u)) {
             ptx::tc_fence_after_sync();
             const uint64_t k0 = k_desc + (uint64_t)(ss * (stage_bytes >> 4));
-            for (int ks = 0; ks < n_ks; ++ks) {
-              const uint64_t box = ks >> 2, in = 2 * (ks & 3);
-              ptx::umma_bf16(tmem + hs * NR, k0 + box * (kBoxBytes >> 4) + in, q_desc + box * (NR * 128 >> 4) + in, id_s, ks > 0 ? 1u : 0u);
+            for (int b = 0; b < n_kb; ++b) {  // (columns behind the row's width are zeros)
+              const uint64_t da = k0 + (uint64_t)(b * (kBoxBytes >> 4)), db = q_desc + (uint64_t)(b * (NR * 128 >> 4));
+#pragma unroll
+              for (int k4 = 0; k4 < 4; ++k4) ptx::umma_bf16(tmem + hs * NR, da + 2 * k4, db + 2 * k4, id_s, b + k4 > 0 ? 1u : 0u);
             }
             ptx::umma_commit(&sh.s_full[hs]);
             phase ^= 1u << slot;
@@ -314,14 +314,17 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
             idle = 0;
           } else if (summed < scored && ptx::mbar_try_wait(&sh.p_ready[hp], n_p[hp] & 1u)) {
             ptx::tc_fence_after_sync();
-            const int n_steps = 2 * min(kHalfPages, n_pages - summed * kHalfPages);
+            const int pages = min(kHalfPages, n_pages - summed * kHalfPages);
             const uint64_t v0 = v_desc + (uint64_t)(ps * (stage_bytes >> 4) + hp * (kHalfBytes >> 4)), p0 = p_desc + (uint64_t)(hp * (2 * kPBytes >> 4));
             for (int mc = 0; mc < n_mc; ++mc) {
               const uint32_t dst = tmem_o + (hp * n_mc + mc) * NR;
-              for (int ks = 0; ks < n_steps; ++ks) {
-                const uint64_t va = v0 + (uint64_t)(mc * (2 * kBoxBytes >> 4) + ks * (2048 >> 4)), pb = p0 + (uint64_t)(ks * (2048 >> 4));
-                ptx::umma_bf16(dst, va, pb, id_o, summed > 1 || ks > 0 ? 1u : 0u);
-                ptx::umma_bf16(dst, va, pb + (kPBytes >> 4), id_o, 1u);
+              for (int pg = 0; pg < pages; ++pg) {
+                const uint64_t va = v0 + (uint64_t)(mc * (2 * kBoxBytes >> 4) + pg * (4096 >> 4)), pb = p0 + (uint64_t)(pg * (4096 >> 4));
+#pragma unroll
+                for (int ks = 0; ks < 2; ++ks) {
+                  ptx::umma_bf16(dst, va + ks * (2048 >> 4), pb + ks * (2048 >> 4), id_o, summed > 1 || pg + ks > 0 ? 1u : 0u);
+                  ptx::umma_bf16(dst, va + ks * (2048 >> 4), pb + ((kPBytes + ks * 2048) >> 4), id_o, 1u);
+                }
               }
             }
             ptx::umma_commit(&sh.k_free[ps][hp]);
