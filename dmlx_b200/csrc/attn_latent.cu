@@ -298,7 +298,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         // whichever of the two next products has its operands goes first
         while (summed < halves) {
           const int hs = scored & 1, hp = summed & 1, slot = 2 * ss + hs;
-          if (scored < halves && scored < summed + 2 && ptx::mbar_try_wait(&sh.k_full[ss][hs], (phase >> slot) & 1u)) {
+          if (scored < halves && scored < summed + 2 && ptx::mbar_test(&sh.k_full[ss][hs], (phase >> slot) & 1u)) {
             ptx::tc_fence_after_sync();
             const uint64_t k0 = k_desc + (uint64_t)(ss * (stage_bytes >> 4));
             for (int b = 0; b < n_kb; ++b) {  // (columns behind the row's width are zeros)
@@ -312,7 +312,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
             if (scored == halves) ptx::umma_commit(&sh.q_free);
             if (hs == 1 && ++ss == stages) ss = 0;
             idle = 0;
-          } else if (summed < scored && ptx::mbar_try_wait(&sh.p_ready[hp], n_p[hp] & 1u)) {
+          } else if (summed < scored && ptx::mbar_test(&sh.p_ready[hp], n_p[hp] & 1u)) {
             ptx::tc_fence_after_sync();
             const int pages = min(kHalfPages, n_pages - summed * kHalfPages);
             const uint64_t v0 = v_desc + (uint64_t)(ps * (stage_bytes >> 4) + hp * (kHalfBytes >> 4)), p0 = p_desc + (uint64_t)(hp * (2 * kPBytes >> 4));
@@ -333,11 +333,9 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
             ++summed;
             if (hp == 1 && ++ps == stages) ps = 0;
             idle = 0;
-          } else if (++idle > kPolls) {
+          } else if (++idle > (1u << 26)) {
             ok = false;
             break;
-          } else if (idle > 64) {
-            __nanosleep(32);
           }
         }
         s0 += (halves + 1) / 2 % stages;
@@ -528,7 +526,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
       if (lane == 0) {
         const bool done = *(volatile int*)&sh.done != 0;  // (before the requests: none comes after it)
         for (int g = 0; g < 2 && what < 0; ++g)
-          if (ptx::mbar_try_wait(&sh.c_req[g], n_c[g] & 1u)) what = g;
+          if (ptx::mbar_test(&sh.c_req[g], n_c[g] & 1u)) what = g;
         if (what < 0 && (done || ++idle > (1u << 24))) what = done ? 2 : 3;
       }
       what = __shfl_sync(0xffffffffu, what, 0);
@@ -618,7 +616,7 @@ b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t heads, con
   }
   const int rows = rows_of(kv->lay[layer], heads, total_rows);
   return b200_attn_make_plan(kv, 0, std::max(1, rows / heads), (heads + rows - 1) / rows, g_sms, d_row_seq, d_row_ctx, total_rows, stream, 4.f,
-                             8.f * std::min(heads, rows) * kv->lay[layer].value_dim / (64.f * kv->lay[layer].kd));
+                             4.f * std::min(heads, rows) * kv->lay[layer].value_dim / (64.f * kv->lay[layer].kd), true);
 }
 
 b200_status b200_latent_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,

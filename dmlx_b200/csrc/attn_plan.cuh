@@ -61,7 +61,7 @@ __device__ __forceinline__ WinItem decode_item(const WinArgs& a, int item, int n
 // Builds the plan of a (window, tokens per group): items_per_chunk work items per chunk, walked by n_workers.  item_cost and slot_cost:
 // what the start and end of a work item, and a row of partial results, cost in pages of one worker's stream.
 b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t q_tokens, int32_t items_per_chunk, int32_t n_workers, const int32_t* d_row_seq,
-                                const int32_t* d_row_ctx, int32_t total_rows, void* stream, float item_cost, float slot_cost);
+                                const int32_t* d_row_ctx, int32_t total_rows, void* stream, float item_cost, float slot_cost, bool fine_lengths);
 // Points the arguments at that plan; false when there is none.
 bool b200_attn_use_plan(b200_kv* kv, int32_t window, int32_t q_tokens, WinArgs* a);
 // Sums the partial results of the groups that were cut.

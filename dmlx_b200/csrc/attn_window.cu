@@ -64,10 +64,22 @@ __device__ __forceinline__ int group_pages(int ctx_first, int ctx_last, int wind
   return (max(ctx_last, 1) - 1) / page_size - first_key(ctx_first, window) / page_size + 1;
 }
 
+// Chunk lengths the plan tries: few and coarse where a grid has many workers, fine steps where a work item is a large part of a
+// worker's load and the number of waves decides.
+struct CoarseLengths {
+  static constexpr int kCand = 6;  // 4, 8, 16, 32, 64 pages, uncut
+  static __device__ __forceinline__ int at(int k) { return 4 << k; }
+};
+struct FineLengths {
+  static constexpr int kCand = 18;  // 8, 12, 16 .. 64 pages, 80, 96, uncut
+  static __device__ __forceinline__ int at(int k) { return k < 15 ? 8 + 4 * k : 80 + 16 * (k - 15); }
+};
+
 // Groups of rows and their chunks.  A group's pages are cut evenly into ceil(pages / ppc) chunks.  ppc is the candidate with
 // the smallest estimated time, in pages of one worker's stream: the average load or the longest item, half an item for
 // the uneven end of the walk, a page and a bit per item for its start and end, and, where groups are cut, the partial sums
 // and the combine pass.  It doubles until the partial slots fit the scratch (uncut groups need none), so a step always fits.
+template <typename Lengths>
 __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict__ row_seq, const int* __restrict__ row_ctx, int total_rows,
                                                            int page_size, int window, int q_tokens, int items_per_chunk,
                                                            int n_workers, int forced_ppc, int max_slots, float item_cost, float slot_cost, int* __restrict__ group_first,
@@ -101,7 +113,7 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
   if (forced_ppc > 0) {
     ppc = forced_ppc;
   } else {
-    constexpr int kCand = 6;  // 4, 8, 16, 32, 64 pages, uncut
+    constexpr int kCand = Lengths::kCand;
     long long chunks[kCand] = {}, slots[kCand] = {}, pages_sum = 0;
     int longest = 0;
     for (int g = tid; g < n_groups; g += blockDim.x) {
@@ -111,7 +123,7 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
       longest = max(longest, pages);
 #pragma unroll
       for (int k = 0; k < kCand; ++k) {
-        const int c = k == kCand - 1 ? 1 : (pages + (4 << k) - 1) >> (k + 2);
+        const int c = k == kCand - 1 ? 1 : (pages + Lengths::at(k) - 1) / Lengths::at(k);
         chunks[k] += c;
         slots[k] += c > 1 ? c * (next - first) : 0;
       }
@@ -128,22 +140,36 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
       if ((tid & 31) == 0) s_red[tid >> 5][k] = v;
     }
     __syncthreads();
+    if (tid < 2 * kCand + 2) {
+      long long sum = 0, most = 0;
+      for (int w = 0; w < (int)(blockDim.x >> 5); ++w) {
+        const long long v = s_red[w][tid];
+        sum += v;
+        most = most > v ? most : v;
+      }
+      s_red[0][tid] = tid == 2 * kCand + 1 ? most : sum;
+    }
+    __syncthreads();
     if (tid == 0) {
-      long long tot[2 * kCand + 2] = {};
-      for (int w = 0; w < (int)(blockDim.x >> 5); ++w)
-        for (int k = 0; k < 2 * kCand + 2; ++k) tot[k] = k == 2 * kCand + 1 ? (tot[k] > s_red[w][k] ? tot[k] : s_red[w][k]) : tot[k] + s_red[w][k];
+      const long long* tot = s_red[0];
       const float per = (float)items_per_chunk / (float)n_workers, load = (float)tot[2 * kCand] * per;
       float best = 3.4e38f;
       for (int k = 0; k < kCand; ++k) {
-        const float length = fminf(k == kCand - 1 ? 1e9f : (float)(4 << k), (float)tot[2 * kCand + 1]);
+        const float length = fminf(k == kCand - 1 ? 1e9f : (float)Lengths::at(k), (float)tot[2 * kCand + 1]);
         const float items = (float)tot[k] * per;
-        float t = fmaxf(load, length) + (items > 1.f ? 0.5f * length : 0.f) + item_cost * items;
+        float t;
+        if (kCand > 6) {  // whole waves of average items, the longest last
+          const float waves = ceilf(items), mean = (float)tot[2 * kCand] / (float)tot[k];
+          t = (waves - 1.f) * mean + length + item_cost * waves;
+        } else {
+          t = fmaxf(load, length) + (items > 1.f ? 0.5f * length : 0.f) + item_cost * items;
+        }
         if (tot[kCand + k] > 0) t += 3.f + slot_cost * (float)tot[kCand + k] * per;
         if (t < best) { best = t; carry_chunks = k; }
       }
     }
     __syncthreads();
-    ppc = carry_chunks == kCand - 1 ? 0x3fffffff : 4 << carry_chunks;
+    ppc = carry_chunks == kCand - 1 ? 0x3fffffff : Lengths::at(carry_chunks);
     __syncthreads();
   }
   for (int round = 0; round < 32; ++round) {
@@ -471,7 +497,7 @@ __global__ void __launch_bounds__(256) window_combine_kernel(WinArgs a) {
   if (a.sinks) l += exp2f(a.sinks[qh] - mm);
   const float inv = l > 0.f ? 1.0f / l : 0.f;
   __nv_bfloat16* dst = a.out + (size_t)row * a.out_stride + (size_t)qh * a.out_head;
-  for (int v0 = 0; v0 < a.L.vd; v0 += 128) {  // four columns per lane
+  for (int v0 = blockIdx.y * 128; v0 < a.L.vd; v0 += gridDim.y * 128) {  // four columns per lane
     const int v = v0 + 4 * lane;
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
     if (v < a.L.vd) {
@@ -638,7 +664,7 @@ b200_status launch_mma_v(const b200_kv* kv, WinArgs& a, int layer, cudaStream_t 
 extern int b200_attn_pages_per_chunk;
 
 b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t items_per_chunk, int32_t n_workers, const int32_t* d_row_seq,
-                                const int32_t* d_row_ctx, int32_t total_rows, void* stream, float item_cost, float slot_cost) {
+                                const int32_t* d_row_ctx, int32_t total_rows, void* stream, float item_cost, float slot_cost, bool fine) {
   if (total_rows <= 0) return B200_OK;
   if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
   const int R = kv->cfg.max_rows + 2;
@@ -655,7 +681,8 @@ b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t
     kv->plans.push_back(p);
   }
   const int forced = b200_attn_pages_per_chunk <= 0 ? 0 : std::min(std::max(b200_attn_pages_per_chunk, 1), 1 << 20);
-  window_plan_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(d_row_seq, d_row_ctx, total_rows, kv->cfg.page_size, window, qt,
+  auto* kernel = fine ? window_plan_kernel<FineLengths> : window_plan_kernel<CoarseLengths>;
+  kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(d_row_seq, d_row_ctx, total_rows, kv->cfg.page_size, window, qt,
                                                           items_per_chunk, n_workers, forced, kv->max_chunks, item_cost, slot_cost,
                                                           p->buf, p->buf + R, p->buf + 2 * R, p->buf + 3 * R, p->buf + 4 * R);
   B200_LAUNCH_CHECK();
@@ -672,7 +699,9 @@ bool b200_attn_use_plan(b200_kv* kv, int32_t window, int32_t q_tokens, WinArgs* 
 }
 
 b200_status b200_attn_combine(b200_kv* kv, const WinArgs& a, void* stream) {
-  window_combine_kernel<<<(unsigned)(((long long)a.total_rows * a.n_q_heads + 7) / 8), 256, 0, (cudaStream_t)stream>>>(a);
+  const long long rows = (long long)a.total_rows * a.n_q_heads;
+  // few rows (decode): their columns over several blocks
+  window_combine_kernel<<<dim3((unsigned)((rows + 7) / 8), rows <= 8192 ? (a.L.vd + 127) / 128 : 1), 256, 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -685,7 +714,7 @@ b200_status b200_window_attn_plan(b200_kv* kv, int32_t layer, int32_t window, in
   const KvLayerDev& L = kv->lay[layer];
   if (L.values_in_keys) return b200_latent_attn_plan(kv, layer, gqa, d_row_seq, d_row_ctx, total_rows, stream);
   const int per_chunk = L.heads * ((gqa + 15) / 16), warps = shape_of((L.kd + 63) / 64 + (L.vd + 63) / 64).warps;
-  return b200_attn_make_plan(kv, window, q_tokens_of(gqa), per_chunk, g_sms * warps, d_row_seq, d_row_ctx, total_rows, stream, 1.25f, 0.25f);
+  return b200_attn_make_plan(kv, window, q_tokens_of(gqa), per_chunk, g_sms * warps, d_row_seq, d_row_ctx, total_rows, stream, 1.25f, 0.25f, false);
 }
 
 b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
