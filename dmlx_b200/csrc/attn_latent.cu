@@ -239,12 +239,23 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
     if (lane == 0) {  // ---- loads ----
       int s = 0;
       uint32_t used = 0, phase = 0, n_item = 0;  // bit 2 * stage + half: loaded before; parity of its next load
-      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
-        const WinItem it = decode_item(a, item, n_groups);
-        const int* table = a.d.block_table + (size_t)it.seq * a.d.max_pages_per_seq;
-        int next[kHalfPages];  // page ids of the coming half-tile, asked for before the wait
+      // Looking an item up takes a chain of dependent loads: it is done while the item before is being worked on.
+      WinItem ahead{};
+      int next[kHalfPages], ahead_id[kHalfPages];  // page ids of the coming half-tile, and of the coming item's first
+      auto look_up = [&](int item) {
+        if (item >= n_items) return;
+        ahead = decode_item(a, item, n_groups);
+        const int* table = a.d.block_table + (size_t)ahead.seq * a.d.max_pages_per_seq;
 #pragma unroll
-        for (int p = 0; p < kHalfPages; ++p) next[p] = it.page_begin + p < it.page_end ? table[it.page_begin + p] : 0;
+        for (int p = 0; p < kHalfPages; ++p) ahead_id[p] = ahead.page_begin + p < ahead.page_end ? table[ahead.page_begin + p] : 0;
+      };
+      look_up(blockIdx.x);
+      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
+        const WinItem it = ahead;
+        const int* table = a.d.block_table + (size_t)it.seq * a.d.max_pages_per_seq;
+#pragma unroll
+        for (int p = 0; p < kHalfPages; ++p) next[p] = ahead_id[p];
+        bool looked = false;
         ok = wait(&sh.q_free, (n_item & 1u) ^ 1u);
         if (!ok) break;
         sh.items[n_item & 1u] = it;
@@ -255,12 +266,13 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         int h = 0;
         for (int pg = it.page_begin; pg < it.page_end; pg += kHalfPages) {
           const int pages = min(kHalfPages, it.page_end - pg), slot = 2 * s + h;
+          if (pg == it.page_begin + 2 * kHalfPages) { look_up(item + gridDim.x); looked = true; }
           int id[kHalfPages];
 #pragma unroll
           for (int p = 0; p < kHalfPages; ++p) {
             id[p] = next[p];
-            const int ahead = pg + kHalfPages + p;
-            next[p] = ahead < it.page_end ? table[ahead] : 0;
+            const int later = pg + kHalfPages + p;
+            next[p] = later < it.page_end ? table[later] : 0;
           }
           ok = wait(&sh.k_free[s][h], ((phase >> slot) & 1u) ^ 1u);
           if (!ok) break;
@@ -274,6 +286,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
           if (h == 0 && ++s == stages) s = 0;
         }
         if (h == 1 && ++s == stages) s = 0;  // an item starts on an even half-tile
+        if (!looked) look_up(item + gridDim.x);
       }
       if (!ok) {  // leave no copy in flight behind
         if (n_item > 0) wait(&sh.q_full, (n_item - 1) & 1u);
