@@ -56,7 +56,7 @@ __device__ __forceinline__ float silu(float g) { return g / (1.0f + expf(-g)); }
 
 // ---- token by token ------------------------------------------------------------------------------------------
 template <typename T, int VEC>
-__global__ void __launch_bounds__(512) gla_step_kernel(Gla a) {
+__global__ void __launch_bounds__(256, 3) gla_step_kernel(Gla a) {
   extern __shared__ float sh[];
   __shared__ float part[32];
   const int req = blockIdx.x, head = blockIdx.y, dk = a.dk, dv = a.dv;
@@ -207,7 +207,7 @@ __device__ __forceinline__ void ldsm4_trans(uint32_t addr, uint32_t (&r)[4]) {
 // on this route; a chunk whose decays are stronger takes the pairs one by one.
 constexpr float kMaxGrowth = 60.f;
 
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) gla_chunk_kernel(Gla a) {
   extern __shared__ __align__(16) float sh[];
   __shared__ int s_range;
@@ -222,11 +222,18 @@ __global__ void __launch_bounds__(256) gla_chunk_kernel(Gla a) {
     const int t = i / a.rank, r = i - t * a.rank;
     a1[i] = t < n ? mat_value<T, 1>(a.src, it.x + t, a.col_a() + r).v[0] : 0.f;
   }
-  for (int i = tid; i < kC * dkp; i += 256) {
-    const int t = i / dkp, c = i - t * dkp;
-    const bool on = t < n && c < dk;
-    q[t * ldr + c] = on ? mat_value<T, 1>(a.src, it.x + t, head * dk + c).v[0] * a.q_scale : 0.f;
-    k[t * ldr + c] = on ? mat_value<T, 1>(a.src, it.x + t, a.col_k() + head * dk + c).v[0] : 0.f;
+  const int groups = dkp / VEC;
+  for (int i = tid; i < kC * groups; i += 256) {
+    const int t = i / groups, c = (i - t * groups) * VEC;
+    Vec<VEC> x{}, y{};
+    if (t < n && c < dk) {
+      x = mat_value<T, VEC>(a.src, it.x + t, head * dk + c);
+      y = mat_value<T, VEC>(a.src, it.x + t, a.col_k() + head * dk + c);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x.v[e] *= a.q_scale;
+    store_vec<VEC>(q + t * ldr + c, x);
+    store_vec<VEC>(k + t * ldr + c, y);
   }
   __syncthreads();
   for (int i = tid; i < 4 * dkp; i += 256) {  // eight tokens of one key channel
@@ -271,11 +278,13 @@ __global__ void __launch_bounds__(256) gla_chunk_kernel(Gla a) {
     *reinterpret_cast<uint32_t*>(at + off_part(dkp, 2)) = hi;
     *reinterpret_cast<uint32_t*>(at + off_part(dkp, 3)) = lo;
   }
-  for (int i = tid; i < a.n_slices * kC * kScanCols; i += 256) {
-    const int s = i / (kC * kScanCols), rest = i - s * kC * kScanCols, t = rest / kScanCols, c = rest - t * kScanCols, col = s * kScanCols + c;
-    const float v = t < n && col < a.dv ? mat_value<T, 1>(a.src, it.x + t, a.col_v() + head * a.dv + col).v[0] : 0.f;
+  constexpr int kPer = kScanCols / VEC;
+  for (int i = tid; i < a.n_slices * kC * kPer; i += 256) {
+    const int s = i / (kC * kPer), rest = i - s * kC * kPer, t = rest / kPer, c = (rest - t * kPer) * VEC, col = s * kScanCols + c;
+    Vec<VEC> v{};
+    if (t < n && col < a.dv) v = mat_value<T, VEC>(a.src, it.x + t, a.col_v() + head * a.dv + col);
     unsigned char* dst = a.values + ((size_t)chunk * a.heads + head) * a.v_bytes + (size_t)s * kVSlice + (size_t)t * kVRow + c * 2;
-    *reinterpret_cast<__nv_bfloat16*>(dst) = __float2bfloat16(v);
+    store_vec<VEC>(reinterpret_cast<__nv_bfloat16*>(dst), v);
   }
   unsigned char *ahi = out + off_a(dkp, 0), *alo = out + off_a(dkp, 1);
   if (__int_as_float(s_range) >= kMaxGrowth) {
@@ -477,7 +486,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
 }
 
 // ---- chunks: norm and gate -------------------------------------------------------------------------------------------
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) gla_out_kernel(Gla a) {
   const int chunk = blockIdx.x, head = blockIdx.y, lane = threadIdx.x & 31;
   if (chunk >= a.first_chunk[a.n_req] || a.d.state[ST_ERR] != 0) return;
@@ -486,11 +495,20 @@ __global__ void __launch_bounds__(256) gla_out_kernel(Gla a) {
     const int row = it.x + i;
     const float* o = a.o + ((size_t)row * a.heads + head) * a.dv;
     float ss = 0.f;
-    for (int c = lane; c < a.dv; c += 32) ss += o[c] * o[c];
+    for (int c = lane * VEC; c < a.dv; c += 32 * VEC) {
+      const Vec<VEC> x = load_vec<VEC>(o + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += x.v[e] * x.v[e];
+    }
     const float r = 1.0f / sqrtf(warp_sum(ss) / (float)a.dv + a.eps);
     T* dst = (T*)a.out + (size_t)row * a.out_stride + (size_t)head * a.dv;
-    for (int c = lane; c < a.dv; c += 32)
-      st(dst + c, o[c] * r * a.norm[c] * silu(mat_value<T, 1>(a.src, row, a.col_g() + head * a.dv + c).v[0]));
+    for (int c = lane * VEC; c < a.dv; c += 32 * VEC) {
+      Vec<VEC> x = load_vec<VEC>(o + c);
+      const Vec<VEC> w = load_vec<VEC>(a.norm + c), g = mat_value<T, VEC>(a.src, row, a.col_g() + head * a.dv + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x.v[e] *= r * w.v[e] * silu(g.v[e]);
+      store_vec<VEC>(dst + c, x);
+    }
   }
 }
 
@@ -564,10 +582,10 @@ b200_status b200_gla_run(b200_kv* kv, const GlaScratch& g, const GlaCall& c, con
   a.stages = 0;
   // portions that are longer than the step kernel's limit exist only if some request has more than one row
   a.chunked = chunked && b200_gla_takes_chunks(c.dk, c.dv, kv->dev.elem_bytes);
+  const bool v4 = c.dk % 4 == 0 && c.dv % 4 == 0 && (c.src.ws || c.src.y_stride % 4 == 0);
   {
-    const bool v4 = c.dk % 4 == 0 && c.dv % 4 == 0 && (c.src.ws || c.src.y_stride % 4 == 0);
     a.cols = std::min(v4 ? c.dv / 4 : c.dv, 256);
-    a.groups = std::max(1, std::min(512 / a.cols, (c.dk + 7) / 8));
+    a.groups = std::max(1, std::min(256 / a.cols, (c.dk + 7) / 8));
     const size_t smem = sizeof(float) * (3 * (size_t)c.dk + c.rank + (size_t)a.groups * c.dv);
     if (smem > 200 * 1024) { b200_set_error("gla: head widths %d / %d are too large", c.dk, c.dv); return B200_ERR_UNSUPPORTED; }
     auto* kernel = f32 ? (v4 ? gla_step_kernel<float, 4> : gla_step_kernel<float, 1>) : (v4 ? gla_step_kernel<__nv_bfloat16, 4> : gla_step_kernel<__nv_bfloat16, 1>);
@@ -581,14 +599,18 @@ b200_status b200_gla_run(b200_kv* kv, const GlaScratch& g, const GlaCall& c, con
   if (smem > 220 * 1024) { b200_set_error("gla: a decay projection of inner width %d is too large", c.rank); return B200_ERR_UNSUPPORTED; }
   static bool configured = false;
   if (!configured) {
-    B200_CUDA_TRY(cudaFuncSetAttribute(gla_chunk_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+    B200_CUDA_TRY((cudaFuncSetAttribute(gla_chunk_kernel<__nv_bfloat16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
+    B200_CUDA_TRY((cudaFuncSetAttribute(gla_chunk_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
     configured = true;
   }
-  gla_chunk_kernel<__nv_bfloat16><<<dim3(chunks, c.heads), 256, smem, s>>>(a);
+  const bool wide = v4 && c.out_stride % 4 == 0;
+  auto* chunk_kernel = wide ? gla_chunk_kernel<__nv_bfloat16, 4> : gla_chunk_kernel<__nv_bfloat16, 1>;
+  chunk_kernel<<<dim3(chunks, c.heads), 256, smem, s>>>(a);
   B200_LAUNCH_CHECK();
   b200_status st = a.dkp <= 32 ? launch_scan<4>(a, n_req, s) : (a.dkp <= 64 ? launch_scan<8>(a, n_req, s) : (a.dkp <= 128 ? launch_scan<16>(a, n_req, s) : launch_scan<32>(a, n_req, s)));
   if (st != B200_OK) return st;
-  gla_out_kernel<__nv_bfloat16><<<dim3(chunks, c.heads), 256, 0, s>>>(a);
+  auto* out_kernel = wide ? gla_out_kernel<__nv_bfloat16, 4> : gla_out_kernel<__nv_bfloat16, 1>;
+  out_kernel<<<dim3(chunks, c.heads), 256, 0, s>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
