@@ -602,7 +602,9 @@ static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* la
     b200_set_error("invalid pool configuration");
     return B200_ERR_INVALID_ARGUMENT;
   }
+  static uint64_t pools = 0;
   auto* kv = new b200_kv();
+  kv->uid = ++pools;
   kv->cfg = *c;
   KvDev& d = kv->dev;
   d.n_layers = c->n_layers; d.n_kv_heads = c->n_kv_heads; d.head_dim = c->head_dim; d.page_size = c->page_size;

@@ -51,6 +51,7 @@ struct WindowPlan {
 };
 
 struct b200_kv {
+  uint64_t uid = 0;  // no two pools of a process share it (an address may be used again): captured graphs are kept by it
   b200_kv_config cfg;
   KvDev dev;
   std::vector<KvLayerDev> lay;        // host copy of dev.layer

@@ -70,7 +70,7 @@ b200_status b200_model::forward(b200_kv* kv, const b200_pack_desc* desc, int n_r
   // (the legacy default stream cannot be captured)
   if (!graphs_on || prof_on || total_rows != n_req || n_req <= 0 || !ready || stream == nullptr || !want.empty())
     return eager(kv, desc, n_req, total_rows, d_prefill_tokens, stream);
-  auto& ge = graphs[std::make_tuple((int)n_req, (const void*)desc, (const void*)kv, stream, sampling)];
+  auto& ge = graphs[std::make_tuple((int)n_req, (const void*)desc, kv->uid, stream, sampling)];
   ge.seen += 1;
   if (ge.seen == 1) return eager(kv, desc, n_req, total_rows, d_prefill_tokens, stream);
   cudaStream_t cs = (cudaStream_t)stream;

@@ -40,11 +40,11 @@ struct b200_model {
   bool sampling = false;  // the step in flight samples with d_samp instead of taking the argmax
   int last_n_req = 0;
   long long launches = 0;  // kernels launched by forward calls so far
-  // CUDA graphs of decode-only steps, keyed by (requests, device descriptor pointer, pool, stream, sampling): the
+  // CUDA graphs of decode-only steps, keyed by (requests, device descriptor pointer, the pool's uid, stream, sampling): the
   // first step of a shape runs eagerly (it may grow scratch buffers), the second is captured, later ones replay the graph.
   bool graphs_on = true;
   struct GraphEntry { int seen = 0; cudaGraphExec_t exec = nullptr; long long kernels = 0; };
-  std::map<std::tuple<int, const void*, const void*, void*, bool>, GraphEntry> graphs;
+  std::map<std::tuple<int, const void*, uint64_t, void*, bool>, GraphEntry> graphs;
   // optional CUDA-event timing per category: 0 attention, 1 matmuls, 2 cache append, 3 the rest
   bool prof_on = false;
   std::vector<cudaEvent_t> prof_events;  // pairs
