@@ -190,7 +190,7 @@ struct LatentArgs {
 // softmax warps take.
 template <int NR>
 struct LatentShared {
-  uint64_t k_full[kMaxStages][2], k_free[kMaxStages][2], s_full[2], p_ready[2], pv_done[2], c_req[2], c_done[2], q_full, q_free;
+  uint64_t k_full[kMaxStages][2], k_free[kMaxStages][2], s_full[2][2], p_ready[2], pv_done[2], c_req[2], c_done[2], q_full, q_free;
   long long off[NR];  // where a row's output starts
   WinItem items[2];   // the loading thread looks an item up for everyone
   uint32_t tmem;
@@ -214,7 +214,8 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   if (tid == 0) {
     for (int h = 0; h < 2; ++h) {
       for (int s = 0; s < stages; ++s) { ptx::mbar_init(&sh.k_full[s][h], 1); ptx::mbar_init(&sh.k_free[s][h], 1); }
-      ptx::mbar_init(&sh.s_full[h], 1);
+      ptx::mbar_init(&sh.s_full[h][0], 1);
+      ptx::mbar_init(&sh.s_full[h][1], 1);
       ptx::mbar_init(&sh.p_ready[h], 128);
       ptx::mbar_init(&sh.pv_done[h], 1);
       ptx::mbar_init(&sh.c_req[h], 1);
@@ -232,7 +233,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   ptx::tc_fence_before_sync();
   __syncthreads();
   ptx::tc_fence_after_sync();
-  const uint32_t tmem = sh.tmem, tmem_o = tmem + 2 * NR;  // S of the two groups, then O of the two: n_mc x NR columns each
+  const uint32_t tmem = sh.tmem, tmem_o = tmem + 4 * NR;  // S of the two groups, twice each, then O of the two: n_mc x NR columns each
   bool ok = true;
 
   if (warp == 0) {
@@ -301,7 +302,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
       const uint64_t q_desc = ptx::umma_desc_k_sw128(ptx::smem_u32(qbuf)), k_desc = ptx::umma_desc_k_sw128(ptx::smem_u32(smem));
       const uint64_t v_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(smem), kBoxBytes), p_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(pbuf), kPBytes);
       int s0 = 0;  // stage of the item's first half-tile
-      uint32_t phase = 0, n_item = 0, n_p[2] = {0, 0};
+      uint32_t phase = 0, n_item = 0, n_p[2] = {0, 0}, n_sc[2] = {0, 0};
       for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
         ok = wait(&sh.q_full, n_item & 1u);
         if (!ok) break;
@@ -311,15 +312,16 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         // whichever of the two next products has its operands goes first
         while (summed < halves) {
           const int hs = scored & 1, hp = summed & 1, slot = 2 * ss + hs;
-          if (scored < halves && scored < summed + 2 && ptx::mbar_test(&sh.k_full[ss][hs], (phase >> slot) & 1u)) {
+          if (scored < halves && scored < summed + 4 && ptx::mbar_test(&sh.k_full[ss][hs], (phase >> slot) & 1u)) {
             ptx::tc_fence_after_sync();
             const uint64_t k0 = k_desc + (uint64_t)(ss * (stage_bytes >> 4));
+            const uint32_t buf = n_sc[hs]++ & 1u, dst = tmem + (2 * hs + buf) * NR;
             for (int b = 0; b < n_kb; ++b) {  // (columns behind the row's width are zeros)
               const uint64_t da = k0 + (uint64_t)(b * (kBoxBytes >> 4)), db = q_desc + (uint64_t)(b * (NR * 128 >> 4));
 #pragma unroll
-              for (int k4 = 0; k4 < 4; ++k4) ptx::umma_bf16(tmem + hs * NR, da + 2 * k4, db + 2 * k4, id_s, b + k4 > 0 ? 1u : 0u);
+              for (int k4 = 0; k4 < 4; ++k4) ptx::umma_bf16(dst, da + 2 * k4, db + 2 * k4, id_s, b + k4 > 0 ? 1u : 0u);
             }
-            ptx::umma_commit(&sh.s_full[hs]);
+            ptx::umma_commit(&sh.s_full[hs][buf]);
             phase ^= 1u << slot;
             ++scored;
             if (scored == halves) ptx::umma_commit(&sh.q_free);
@@ -367,7 +369,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
     bool dead = false;                       // some thread's wait ran out: decided together, so that all leave
     for (int item = blockIdx.x; item < n_items; item += gridDim.x, ++n_item) {
       // (not q_full: that barrier may be two phases on when the item before is still being written out)
-      if (g == 0) ok = wait(&sh.s_full[0], n_s & 1u) && ok;
+      if (g == 0) ok = wait(&sh.s_full[0][n_s & 1u], (n_s >> 1) & 1u) && ok;
       if (bar_any(kAll, kAllThreads, !ok)) { dead = true; break; }
       const WinItem it = sh.items[n_item & 1u];
       const int h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0), n_pages = it.page_end - it.page_begin;
@@ -389,14 +391,15 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
       for (int j = g; j < halves; j += 2) {
         const int pages = min(kHalfPages, n_pages - j * kHalfPages), tok0 = (it.page_begin + j * kHalfPages) * 32;
         const bool first = j == g;
-        ok = wait(&sh.s_full[g], n_s & 1u) && ok;
+        ok = wait(&sh.s_full[g][n_s & 1u], (n_s >> 1) & 1u) && ok;
+        const uint32_t s_at = tmem + lanes + (2 * g + (n_s & 1u)) * NR + c0;
         ++n_s;
         ptx::tc_fence_after_sync();
         __syncwarp();
         float v[NC];
         {
           uint32_t u[NC];
-          tmem_load<NC>(tmem + lanes + g * NR + c0, u);
+          tmem_load<NC>(s_at, u);
           ptx::tmem_ld_wait();
 #pragma unroll
           for (int r = 0; r < NC; ++r) v[r] = __uint_as_float(u[r]) * a.scale_log2;
@@ -601,7 +604,7 @@ b200_status launch(const b200_kv* kv, LatentArgs& la, int layer, cudaStream_t s)
   while (stages > 1 && smem_of<NR>(la.n_kb, stages) > kSmemLimit) --stages;
   la.w.stages = stages;
   la.tmem_cols = 32;
-  while (la.tmem_cols < (uint32_t)(2 * NR + 2 * la.n_mc * NR)) la.tmem_cols <<= 1;
+  while (la.tmem_cols < (uint32_t)(4 * NR + 2 * la.n_mc * NR)) la.tmem_cols <<= 1;
   static bool configured = false;
   if (!configured) {
     B200_CUDA_TRY(cudaFuncSetAttribute(latent_attn_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit));
@@ -617,7 +620,7 @@ b200_status launch(const b200_kv* kv, LatentArgs& la, int layer, cudaStream_t s)
 bool b200_latent_attn_takes_mma(const b200_kv* kv, int32_t layer) {
   const KvLayerDev& L = kv->lay[layer];
   return kv->layered && L.values_in_keys && L.heads == 1 && kv->dev.elem_bytes == 2 && smem_of<16>((L.kd + 63) / 64, 1) <= kSmemLimit &&
-         64 + (L.value_dim + 127) / 128 * 64 <= 512;
+         128 + (L.value_dim + 127) / 128 * 64 <= 512;
 }
 
 b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t heads, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
