@@ -191,8 +191,9 @@ struct LatentArgs {
 template <int NR>
 struct LatentShared {
   uint64_t k_full[kMaxStages][2], k_free[kMaxStages][2], s_full[2][2], p_ready[2], pv_done[2], c_req[2], c_done[2], q_full, q_free;
-  long long off[NR];  // where a row's output starts
+  long long off[NR];  // where a row's output starts (-1: the row does not exist)
   WinItem items[2];   // the loading thread looks an item up for everyone
+  int3 range;         // the block's work items
   uint32_t tmem;
   int done;
   float red[2][2][NR], m[2][NR], corr[2][NR], w[2][NR];
@@ -210,7 +211,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   unsigned char* qbuf = smem + (size_t)stages * stage_bytes;  // [box][NR rows][128 B]
   unsigned char* pbuf = qbuf + (size_t)n_kb * NR * 128;       // [group][values, remainders][key][128 B, NR of 64 columns used]
   LatentShared<NR>& sh = *reinterpret_cast<LatentShared<NR>*>(pbuf + 4 * kPBytes);
-  const int n_groups = a.hdr[0], n_items = a.chunk_start[n_groups] * a.n_blocks;
+  const int n_groups = a.hdr[0];
   if (tid == 0) {
     for (int h = 0; h < 2; ++h) {
       for (int s = 0; s < stages; ++s) { ptx::mbar_init(&sh.k_full[s][h], 1); ptx::mbar_init(&sh.k_free[s][h], 1); }
@@ -225,6 +226,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
     ptx::mbar_init(&sh.q_free, 1);
     ptx::mbar_fence_init();
     sh.done = 0;
+    sh.range = worker_items(a, n_groups);
   }
   if (warp == 1) {
     ptx::tmem_alloc(&sh.tmem, la.tmem_cols);
@@ -233,6 +235,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   ptx::tc_fence_before_sync();
   __syncthreads();
   ptx::tc_fence_after_sync();
+  const int item0 = sh.range.x, n_items = sh.range.y, item_step = sh.range.z;
   const uint32_t tmem = sh.tmem, tmem_o = tmem + 4 * NR;  // S of the two groups, twice each, then O of the two: n_mc x NR columns each
   bool ok = true;
 
@@ -250,8 +253,8 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
 #pragma unroll
         for (int p = 0; p < kHalfPages; ++p) ahead_id[p] = ahead.page_begin + p < ahead.page_end ? table[ahead.page_begin + p] : 0;
       };
-      look_up(blockIdx.x);
-      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
+      look_up(item0);
+      for (int item = item0; item < n_items && ok; item += item_step, ++n_item) {
         const WinItem it = ahead;
         const int* table = a.d.block_table + (size_t)it.seq * a.d.max_pages_per_seq;
 #pragma unroll
@@ -267,7 +270,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         int h = 0;
         for (int pg = it.page_begin; pg < it.page_end; pg += kHalfPages) {
           const int pages = min(kHalfPages, it.page_end - pg), slot = 2 * s + h;
-          if (pg == it.page_begin + 2 * kHalfPages) { look_up(item + gridDim.x); looked = true; }
+          if (pg == it.page_begin + 2 * kHalfPages) { look_up(item + item_step); looked = true; }
           int id[kHalfPages];
 #pragma unroll
           for (int p = 0; p < kHalfPages; ++p) {
@@ -287,7 +290,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
           if (h == 0 && ++s == stages) s = 0;
         }
         if (h == 1 && ++s == stages) s = 0;  // an item starts on an even half-tile
-        if (!looked) look_up(item + gridDim.x);
+        if (!looked) look_up(item + item_step);
       }
       if (!ok) {  // leave no copy in flight behind
         if (n_item > 0) wait(&sh.q_full, (n_item - 1) & 1u);
@@ -303,7 +306,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
       const uint64_t v_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(smem), kBoxBytes), p_desc = ptx::umma_desc_mn_sw128(ptx::smem_u32(pbuf), kPBytes);
       int s0 = 0;  // stage of the item's first half-tile
       uint32_t phase = 0, n_item = 0, n_p[2] = {0, 0}, n_sc[2] = {0, 0};
-      for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x, ++n_item) {
+      for (int item = item0; item < n_items && ok; item += item_step, ++n_item) {
         ok = wait(&sh.q_full, n_item & 1u);
         if (!ok) break;
         const int n_pages = sh.items[n_item & 1u].page_end - sh.items[n_item & 1u].page_begin, halves = (n_pages + kHalfPages - 1) / kHalfPages;
@@ -367,7 +370,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
     unsigned char* p_hi = pbuf + g * 2 * kPBytes + key * 128;
     uint32_t n_s = 0, n_pv = 0, n_c = 0, n_item = 0;  // half-tiles of the group scored / summed, rescalings, items (phases of the barriers)
     bool dead = false;                       // some thread's wait ran out: decided together, so that all leave
-    for (int item = blockIdx.x; item < n_items; item += gridDim.x, ++n_item) {
+    for (int item = item0; item < n_items; item += item_step, ++n_item) {
       // (not q_full: that barrier may be two phases on when the item before is still being written out)
       if (g == 0) ok = wait(&sh.s_full[0][n_s & 1u], (n_s >> 1) & 1u) && ok;
       if (bar_any(kAll, kAllThreads, !ok)) { dead = true; break; }
@@ -377,8 +380,9 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
       if (row < NR) {
         if (g == 0) {
           const int tok = row / hb, head = row - tok * hb;
-          sh.ctx[row] = tok < it.n_rows && head < heads_here ? it.ctx0 + tok : 0;
-          sh.off[row] = it.slot0 >= 0 ? ((long long)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd
+          const bool on = tok < it.n_rows && head < heads_here;
+          sh.ctx[row] = on ? it.ctx0 + tok : 0;
+          sh.off[row] = !on ? -1 : it.slot0 >= 0 ? ((long long)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd
                                       : (long long)(it.first_row + tok) * a.out_stride + (long long)(h0 + head) * a.out_head;
         }
         sh.m[g][row] = kAttnNone;
@@ -515,14 +519,25 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         if (halves > 1) tmem_load<NC>(tmem_o + lanes + (n_mc + mc) * NR + c0, odd);
         ptx::tmem_ld_wait();
         const int dim = mc * 128 + quarter * 32 + lane;
+        // (shared memory is read ahead of the stores: the compiler cannot tell that they do not touch it)
+        float x[NC];
 #pragma unroll
-        for (int r = 0; r < NC; ++r) {
-          float x = __uint_as_float(o[r]) * sh.w[0][c0 + r];
-          if (halves > 1) x = fmaf(__uint_as_float(odd[r]), sh.w[1][c0 + r], x);
-          if (sh.ctx[c0 + r] > 0) {
-            if (it.slot0 >= 0) { if (dim < a.L.vd) a.part_o[sh.off[c0 + r] + dim] = x; }
-            else if (dim < a.L.value_dim) a.out[sh.off[c0 + r] + dim] = __float2bfloat16(x);
-          }
+        for (int r = 0; r < NC; ++r) x[r] = __uint_as_float(o[r]) * sh.w[0][c0 + r];
+        if (halves > 1) {
+#pragma unroll
+          for (int r = 0; r < NC; ++r) x[r] = fmaf(__uint_as_float(odd[r]), sh.w[1][c0 + r], x[r]);
+        }
+        long long off[NC];
+#pragma unroll
+        for (int r = 0; r < NC; ++r) off[r] = sh.off[c0 + r];
+        if (it.slot0 >= 0) {
+#pragma unroll
+          for (int r = 0; r < NC; ++r)
+            if (off[r] >= 0 && dim < a.L.vd) a.part_o[off[r] + dim] = x[r];
+        } else {
+#pragma unroll
+          for (int r = 0; r < NC; ++r)
+            if (off[r] >= 0 && dim < a.L.value_dim) a.out[off[r] + dim] = __float2bfloat16(x[r]);
         }
         __syncwarp();
       }

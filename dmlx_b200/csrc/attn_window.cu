@@ -84,11 +84,11 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
                                                            int page_size, int window, int q_tokens, int items_per_chunk,
                                                            int n_workers, int forced_ppc, int max_slots, float item_cost, float slot_cost, int* __restrict__ group_first,
                                                            int* __restrict__ chunk_start, int* __restrict__ part_base,
-                                                           int* __restrict__ row_group, int* __restrict__ hdr) {
+                                                           int* __restrict__ row_group, int* __restrict__ page_base, int* __restrict__ hdr) {
   __shared__ int warp_buf[32];
-  __shared__ int carry_start, carry_groups, carry_chunks, carry_slots;
+  __shared__ int carry_start, carry_groups, carry_chunks, carry_slots, carry_pages, s_share;
   const int tid = threadIdx.x;
-  if (tid == 0) { carry_start = -1; carry_groups = 0; }
+  if (tid == 0) { carry_start = -1; carry_groups = 0; s_share = 0; }
   __syncthreads();
   for (int base = 0; base < total_rows; base += blockDim.x) {
     const int i = base + tid;
@@ -167,23 +167,42 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
         if (tot[kCand + k] > 0) t += 3.f + slot_cost * (float)tot[kCand + k] * per;
         if (t < best) { best = t; carry_chunks = k; }
       }
+      // Equal shares: about one more item per worker than whole groups would make.  (Not for prompts: there the workers should walk
+      // neighbouring groups side by side, which read the same pages.)
+      if (kCand > 6 && items_per_chunk == 1 && n_groups <= 4 * n_workers) {
+        const long long pages = tot[2 * kCand];
+        const int share = max((int)((pages + n_workers - 1) / n_workers), 4);
+        const float cuts = (float)pages / (float)share, items = ((float)n_groups + cuts) / (float)n_workers;
+        const float rows_cut = fminf(2.f * cuts, (float)n_groups + cuts) * (float)total_rows / (float)n_groups;
+        if ((float)share + item_cost * fmaxf(items, 1.f) + 3.f + slot_cost * rows_cut / (float)n_workers < best) s_share = share;
+      }
     }
     __syncthreads();
     ppc = carry_chunks == kCand - 1 ? 0x3fffffff : Lengths::at(carry_chunks);
     __syncthreads();
   }
+  int share = s_share;
   for (int round = 0; round < 32; ++round) {
-    if (tid == 0) { carry_chunks = 0; carry_slots = 0; }
+    if (tid == 0) { carry_chunks = 0; carry_slots = 0; carry_pages = 0; }
     __syncthreads();
     for (int base = 0; base < n_groups; base += blockDim.x) {
       const int g = base + tid;
-      int chunks = 0, slots = 0;
+      int chunks = 0, slots = 0, pages = 0, rows = 0;
       if (g < n_groups) {
         const int first = group_first[g], next = group_first[g + 1];
-        const int pages = group_pages(row_ctx[first], row_ctx[next - 1], window, page_size);
-        chunks = pages / ppc + (pages % ppc ? 1 : 0);
-        slots = chunks > 1 ? chunks * (next - first) : 0;
+        pages = group_pages(row_ctx[first], row_ctx[next - 1], window, page_size);
+        rows = next - first;
       }
+      if (share > 0) {
+        const int base_page = carry_pages + scan_incl<false>(pages, warp_buf) - pages;
+        if (g < n_groups) {
+          page_base[g] = base_page;
+          chunks = (base_page + pages - 1) / share - base_page / share + 1;
+        }
+      } else {
+        chunks = pages / ppc + (pages % ppc ? 1 : 0);
+      }
+      slots = chunks > 1 ? chunks * rows : 0;
       const int c_incl = scan_incl<false>(chunks, warp_buf);
       const int s_incl = scan_incl<false>(slots, warp_buf);
       if (g < n_groups) {
@@ -192,16 +211,20 @@ __global__ void __launch_bounds__(1024) window_plan_kernel(const int* __restrict
       }
       __syncthreads();
       if (tid == blockDim.x - 1) { carry_chunks += c_incl; carry_slots += s_incl; }
+      const int page_sum = scan_incl<false>(pages, warp_buf);
+      if (tid == blockDim.x - 1) carry_pages += page_sum;
       __syncthreads();
     }
     if (carry_slots <= max_slots) break;
     __syncthreads();
     ppc = ppc > (1 << 28) ? ppc : ppc * 2;
+    share = share > (1 << 28) ? share : share * 2;
   }
   if (tid == 0) {
     chunk_start[n_groups] = carry_chunks;
     hdr[0] = n_groups;
     hdr[1] = ppc;
+    hdr[2] = share;
   }
 }
 
@@ -673,7 +696,7 @@ b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t
     p = new WindowPlan();
     p->window = window;
     p->q_tokens = qt;
-    if (cudaMalloc((void**)&p->buf, sizeof(int) * ((size_t)4 * R + 2)) != cudaSuccess) {
+    if (cudaMalloc((void**)&p->buf, sizeof(int) * ((size_t)5 * R + 4)) != cudaSuccess) {
       delete p;
       b200_set_error("attention plan: out of device memory");
       return B200_ERR_CUDA;
@@ -684,7 +707,7 @@ b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t
   auto* kernel = fine ? window_plan_kernel<FineLengths> : window_plan_kernel<CoarseLengths>;
   kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(d_row_seq, d_row_ctx, total_rows, kv->cfg.page_size, window, qt,
                                                           items_per_chunk, n_workers, forced, kv->max_chunks, item_cost, slot_cost,
-                                                          p->buf, p->buf + R, p->buf + 2 * R, p->buf + 3 * R, p->buf + 4 * R);
+                                                          p->buf, p->buf + R, p->buf + 2 * R, p->buf + 3 * R, p->buf + 4 * R, p->buf + 5 * R);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -693,7 +716,8 @@ bool b200_attn_use_plan(b200_kv* kv, int32_t window, int32_t q_tokens, WinArgs* 
   const WindowPlan* p = find_plan(kv, window, q_tokens);
   if (!p) { b200_set_error("attention: no plan for window %d and groups of %d", window, q_tokens); return false; }
   const int R = kv->cfg.max_rows + 2;
-  a->group_first = p->buf; a->chunk_start = p->buf + R; a->part_base = p->buf + 2 * R; a->row_group = p->buf + 3 * R; a->hdr = p->buf + 4 * R;
+  a->group_first = p->buf; a->chunk_start = p->buf + R; a->part_base = p->buf + 2 * R; a->row_group = p->buf + 3 * R; a->page_base = p->buf + 4 * R;
+  a->hdr = p->buf + 5 * R;
   a->part_o = kv->d_part_o; a->part_ml = kv->d_part_ml;
   return true;
 }
