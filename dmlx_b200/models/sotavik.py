@@ -1,8 +1,8 @@
-"""Sotavik: a decoder of gated linear attention and latent attention layers, on the configurable decoder stack.
+"""Sotavik: gated linear attention and latent attention layers on the configurable decoder stack.
 
-Every layer has one norm (its weight a single number) whose output both sublayers read; mixer and feed-forward are added to the
-residual together, and a learned average over the embedding output and all layer results so far goes on to the next layer.
-The feed-forward is a mixture of experts: a table gives each token id its experts, beside one shared expert for every token.
+A layer normalises once, with a single learned number as the weight, and feeds mixer and feed-forward from that; their sum joins
+the residual, and a learned combination of everything computed so far in depth is handed on.  The feed-forward is a mixture of
+experts looked up by token id in a table, next to an expert that serves all tokens.
 """
 from __future__ import annotations
 

@@ -680,7 +680,7 @@ b200_model* b200_decoder_model(b200_decoder* m);
  * qkv: rows of [q heads x key_dim | kv heads x key_dim | kv heads x value_dim], `stride` elements apart; adds d_bias (f32, may
  * be null), divides every q and k head by its root mean square when qk_norm, writes q as [q heads][key_dim rounded up to 16]
  * and k, v into their pages.
- * attention: d_q as written by qkv; out rows [q heads x value_dim], out_stride apart.  d_slopes_log2 / d_sinks_log2: f32 per
+ * attention (also of layers with values_in_keys): d_q as written by qkv; out rows [q heads x value_dim], out_stride apart.  d_slopes_log2 / d_sinks_log2: f32 per
  * query head, multiplied by log2(e), may be null.  `mma` as in b200_decoder_set_attn_mma. */
 b200_status b200_decoder_qkv(b200_kv* kv, int32_t layer, const void* d_qkv, int32_t stride, const float* d_bias, int32_t n_q_heads,
                              int32_t qk_norm, float eps, void* d_q, const int32_t* d_positions, const int32_t* d_row_seq,

@@ -523,6 +523,40 @@ def test_latent_attention_sink_counts_once_however_the_keys_are_cut():
         dev.set_attn_pages_per_chunk(0)
 
 
+@pytest.mark.parametrize("heads,rank,rot", [(12, 80, 16), (40, 144, 32)])
+def test_latent_attention_of_many_unequal_contexts(heads, rank, rot):
+    """A decode step whose contexts differ a hundredfold: long ones are cut between workers, short ones share one."""
+    rng = np.random.default_rng(8)
+    lens = [2900, 1700, 5, 64, 1, 333, 32, 33, 1200] + rng.integers(1, 120, 21).tolist()
+    case = LatentCase(lens, heads, rank, rot)
+    case.write()
+    rows = [(s, n - 1) for s, n in enumerate(lens)]
+    q = _bf16(rng.normal(size=(len(rows), heads, rank + rot)))
+    sink = rng.normal(size=heads)
+    want = case.want(rows, q, 0.15, sink)
+    assert _error(case.run(rows, q, 0.15, sink), want) <= 4 * _error(_bf16(want), want)
+
+
+@pytest.mark.parametrize("mma", [True, False])
+def test_latent_attention_of_scores_that_keep_growing(mma):
+    """Every page's scores exceed all before by more than the scale of a running sum tolerates, and then fall again."""
+    heads, rank, rot, n = 10, 96, 32, 640
+    case = LatentCase([n], heads, rank, rot)
+    level = np.concatenate([np.linspace(0, 80, 400), np.linspace(80, 20, 240)])
+    case.keys[0] *= 0.2
+    case.keys[0][:, rank] = level / 4
+    case.keys[0] = _bf16(case.keys[0])
+    case.write()
+    rng = np.random.default_rng(2)
+    q = _bf16(0.3 * rng.normal(size=(4, heads, rank + rot)))
+    q[:, :, rank] = 4.0
+    rows = [(0, 150), (0, 399), (0, 500), (0, 639)]
+    want = case.want(rows, q, 1.0, np.zeros(heads))
+    got = case.run(rows, q, 1.0, np.zeros(heads), mma)
+    assert np.isfinite(got).all()
+    assert _error(got, want) <= 4 * _error(_bf16(want), want)
+
+
 # ---- programs ------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_trace_replay_program(tmp_path, dtype):
