@@ -24,7 +24,7 @@
 namespace {
 
 // Angles in f64, brought into one turn before they become f32: positions far out keep their accuracy.
-__global__ void __launch_bounds__(256) rotation_table_kernel(const double* __restrict__ freq, int half, const int* __restrict__ pos, int rows,
+__global__ void __launch_bounds__(256) rotation_table_kernel(const double* __restrict__ freq, int half, float size, const int* __restrict__ pos, int rows,
                                                              float2* __restrict__ out) {
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
   if (i >= (long long)rows * half) return;
@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(256) rotation_table_kernel(const double* __res
   const double a = (double)pos[row] * freq[p];
   float s, c;
   sincosf((float)(a - rint(a / kTurn) * kTurn), &s, &c);
-  out[i] = make_float2(c, s);
+  out[i] = make_float2(c * size, s * size);
 }
 
 struct PrepArgs {
@@ -43,20 +43,37 @@ struct PrepArgs {
   const int *pos, *row_seq;
 };
 
-// One warp per (row, query head), and one for the row's latent.
+// One warp per (row, query head), one for the row's query latent, and one for the row's latent.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256) latent_prep_kernel(PrepArgs a) {
   const LatentPrep& p = a.p;
   const int row = blockIdx.x, lane = threadIdx.x & 31, u = blockIdx.y * 8 + (threadIdx.x >> 5);
-  if (u > p.heads) return;
+  if (u > p.heads + 1) return;
   const int per_head = p.dim + p.rot;
   const float2* rt = p.rotation + (size_t)row * (p.rot / 2);
   auto rotate = [&](T* dst, int col) {
     for (int i = lane; i < p.rot / 2; i += 32) {
-      const float x = mat_value<T, 1>(p.src, row, col + 2 * i).v[0], y = mat_value<T, 1>(p.src, row, col + 2 * i + 1).v[0];
+      const int at = p.halves ? i : 2 * i, to = p.halves ? i + p.rot / 2 : 2 * i + 1;
+      const float x = mat_value<T, 1>(p.src, row, col + at).v[0], y = mat_value<T, 1>(p.src, row, col + to).v[0];
       const float2 cs = rt[i];
-      st(dst + 2 * i, x * cs.x - y * cs.y);
-      st(dst + 2 * i + 1, y * cs.x + x * cs.y);
+      st(dst + at, x * cs.x - y * cs.y);
+      st(dst + to, y * cs.x + x * cs.y);
+    }
+  };
+  // columns col .. col + n - 1 divided by their root mean square, times w
+  auto normed = [&](T* dst, int col, int n, const float* w) {
+    float ss = 0.f;
+    for (int c = lane * VEC; c < n; c += 32 * VEC) {
+      const Vec<VEC> v = mat_value<T, VEC>(p.src, row, col + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += v.v[e] * v.v[e];
+    }
+    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + p.eps);
+    for (int c = lane * VEC; c < n; c += 32 * VEC) {
+      Vec<VEC> v = mat_value<T, VEC>(p.src, row, col + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v.v[e] *= r * w[c + e];
+      store_vec<VEC>(dst + c, v);
     }
   };
   if (u < p.heads) {
@@ -68,35 +85,31 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(PrepArgs a) {
     for (int c = a.L.key_dim + lane; c < a.L.kd; c += 32) st(q + c, 0.f);
     return;
   }
+  if (u == p.heads + 1) {
+    if (p.q_rank == 0) return;
+    T* dst = (T*)p.q_latent + (size_t)row * p.q_latent_stride;
+    normed(dst, 0, p.q_rank, p.q_norm);
+    for (int c = p.q_rank + lane; c < p.q_latent_stride; c += 32) st(dst + c, 0.f);
+    return;
+  }
+  if (!p.keys) return;
   const int pos = a.pos[row], seq = a.row_seq[row];
   const int page_idx = pos / a.d.page_size, slot = pos - page_idx * a.d.page_size;
   // a step whose reservation failed has no page for this row: nothing is written (the error word is set)
   if (seq < 0 || seq >= a.d.max_seqs || page_idx >= a.d.seq_pages[seq]) return;
   const int page = a.d.block_table[(size_t)seq * a.d.max_pages_per_seq + page_idx];
   T* dst = (T*)((char*)a.d.k_pool + a.L.k_off) + ((size_t)page * a.d.page_size + slot) * (size_t)a.L.kd;
-  const int col = p.heads * per_head;
-  float ss = 0.f;
-  for (int c = lane * VEC; c < p.rank; c += 32 * VEC) {
-    const Vec<VEC> v = mat_value<T, VEC>(p.src, row, col + c);
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) ss += v.v[e] * v.v[e];
-  }
-  const float r = 1.0f / sqrtf(warp_sum(ss) / (float)p.rank + p.eps);
-  for (int c = lane * VEC; c < p.rank; c += 32 * VEC) {
-    Vec<VEC> v = mat_value<T, VEC>(p.src, row, col + c);
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) v.v[e] *= r * p.norm[c + e];
-    store_vec<VEC>(dst + c, v);
-  }
+  const int col = p.q_rank + p.heads * per_head;
+  normed(dst, col, p.rank, p.norm);
   rotate(dst + p.rank, col + p.rank);
 }
 
 }  // namespace
 
-b200_status b200_rotation_table(const double* d_freq, int dims, const int32_t* d_pos, int rows, float2* d_out, void* stream) {
+b200_status b200_rotation_table(const double* d_freq, int dims, double size, const int32_t* d_pos, int rows, float2* d_out, void* stream) {
   if (rows <= 0 || dims < 2) return B200_OK;
   const long long n = (long long)rows * (dims / 2);
-  rotation_table_kernel<<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(d_freq, dims / 2, d_pos, rows, d_out);
+  rotation_table_kernel<<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(d_freq, dims / 2, (float)size, d_pos, rows, d_out);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -110,10 +123,10 @@ b200_status b200_latent_prep(b200_kv* kv, const LatentPrep& p, const int32_t* d_
   if (rows <= 0) return B200_OK;
   PrepArgs a;
   a.d = kv->dev; a.L = kv->lay[p.layer]; a.p = p; a.pos = d_pos; a.row_seq = d_row_seq;
-  const bool v4 = p.dim % 4 == 0 && p.rot % 4 == 0 && p.rank % 4 == 0 && p.plain_stride % 4 == 0 && (p.src.ws || p.src.y_stride % 4 == 0);
+  const bool v4 = p.dim % 4 == 0 && p.rot % 4 == 0 && p.rank % 4 == 0 && p.plain_stride % 4 == 0 && p.q_rank % 4 == 0 && p.q_latent_stride % 4 == 0 && (p.src.ws || p.src.y_stride % 4 == 0);
   auto* kernel = kv->dev.elem_bytes == 4 ? (v4 ? latent_prep_kernel<float, 4> : latent_prep_kernel<float, 1>)
                                          : (v4 ? latent_prep_kernel<__nv_bfloat16, 4> : latent_prep_kernel<__nv_bfloat16, 1>);
-  kernel<<<dim3(rows, (p.heads + 1 + 7) / 8), 256, 0, (cudaStream_t)stream>>>(a);
+  kernel<<<dim3(rows, (p.heads + (p.q_rank > 0 ? 2 : 1) + 7) / 8), 256, 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
@@ -197,7 +210,7 @@ struct LatentShared {
   uint32_t tmem;
   int done;
   float red[2][2][NR], m[2][NR], corr[2][NR], w[2][NR];
-  int ctx[NR];
+  int ctx[NR], lo[NR];  // a row sees keys lo .. ctx - 1
 };
 
 template <int NR>
@@ -377,11 +390,13 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
       const WinItem it = sh.items[n_item & 1u];
       const int h0 = it.block * hb, heads_here = min(hb, a.n_q_heads - h0), n_pages = it.page_end - it.page_begin;
       const int halves = (n_pages + kHalfPages - 1) / kHalfPages;
+      const int lo_last = first_key(it.ctx0 + it.n_rows - 1, a.window);  // the latest window start of the group
       if (row < NR) {
         if (g == 0) {
           const int tok = row / hb, head = row - tok * hb;
           const bool on = tok < it.n_rows && head < heads_here;
           sh.ctx[row] = on ? it.ctx0 + tok : 0;
+          sh.lo[row] = first_key(sh.ctx[row], a.window);
           sh.off[row] = !on ? -1 : it.slot0 >= 0 ? ((long long)(it.slot0 + tok) * a.n_q_heads + h0 + head) * a.L.vd
                                       : (long long)(it.first_row + tok) * a.out_stride + (long long)(h0 + head) * a.out_head;
         }
@@ -408,10 +423,10 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
 #pragma unroll
           for (int r = 0; r < NC; ++r) v[r] = __uint_as_float(u[r]) * a.scale_log2;
         }
-        if (tok0 + kHalfKeys > it.ctx0 || pages < kHalfPages) {
+        if (tok0 + kHalfKeys > it.ctx0 || pages < kHalfPages || tok0 < lo_last) {
           const bool in_tile = key < pages * 32;
 #pragma unroll
-          for (int r = 0; r < NC; ++r) v[r] = in_tile && tok0 + key < sh.ctx[c0 + r] ? v[r] : kAttnNone;
+          for (int r = 0; r < NC; ++r) v[r] = in_tile && tok0 + key < sh.ctx[c0 + r] && tok0 + key >= sh.lo[c0 + r] ? v[r] : kAttnNone;
         }
         // The scale of a row stays as it is unless some key exceeds it by 2^kGrow; only then are the maxima taken.
         bool over = !ok;
@@ -638,7 +653,7 @@ bool b200_latent_attn_takes_mma(const b200_kv* kv, int32_t layer) {
          128 + (L.value_dim + 127) / 128 * 64 <= 512;
 }
 
-b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t heads, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
+b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t window, int32_t heads, const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows,
                                   void* stream) {
   if (g_sms == 0) {
     int dev = 0;
@@ -646,7 +661,7 @@ b200_status b200_latent_attn_plan(b200_kv* kv, int32_t layer, int32_t heads, con
     B200_CUDA_TRY(cudaDeviceGetAttribute(&g_sms, cudaDevAttrMultiProcessorCount, dev));
   }
   const int rows = rows_of(kv->lay[layer], heads, total_rows);
-  return b200_attn_make_plan(kv, 0, std::max(1, rows / heads), (heads + rows - 1) / rows, g_sms, d_row_seq, d_row_ctx, total_rows, stream, 4.f,
+  return b200_attn_make_plan(kv, window, std::max(1, rows / heads), (heads + rows - 1) / rows, g_sms, d_row_seq, d_row_ctx, total_rows, stream, 4.f,
                              4.f * std::min(heads, rows) * kv->lay[layer].value_dim / (64.f * kv->lay[layer].kd), true);
 }
 
@@ -654,14 +669,14 @@ b200_status b200_latent_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
                                  void* stream) {
   const KvLayerDev& L = kv->lay[c.layer];
   if (c.q_stride != c.n_q_heads * L.kd) { b200_set_error("latent attention: query rows have to lie one behind the other"); return B200_ERR_INVALID_ARGUMENT; }
-  if (c.window != 0 || c.slopes_log2) { b200_set_error("latent attention has no window and no distance bias"); return B200_ERR_UNSUPPORTED; }
+  if (c.slopes_log2) { b200_set_error("latent attention has no distance bias"); return B200_ERR_UNSUPPORTED; }
   LatentArgs la;
   WinArgs& a = la.w;
   const int rows = rows_of(L, c.n_q_heads, total_rows), hb = std::min(c.n_q_heads, rows);
-  if (!b200_attn_use_plan(kv, 0, std::max(1, rows / c.n_q_heads), &a)) return B200_ERR_INVALID_ARGUMENT;
+  if (!b200_attn_use_plan(kv, c.window, std::max(1, rows / c.n_q_heads), true, &a)) return B200_ERR_INVALID_ARGUMENT;
   a.d = kv->dev; a.L = L; a.L.vd = (L.value_dim + 15) / 16 * 16;
   a.q = (const __nv_bfloat16*)c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx;
-  a.total_rows = total_rows; a.n_q_heads = c.n_q_heads; a.window = 0;
+  a.total_rows = total_rows; a.n_q_heads = c.n_q_heads; a.window = c.window;
   a.G = c.n_q_heads; a.head_block = hb; a.n_blocks = (c.n_q_heads + hb - 1) / hb;
   a.scale_log2 = c.scale * kAttnLog2e;
   a.slopes = nullptr; a.sinks = c.sinks_log2;

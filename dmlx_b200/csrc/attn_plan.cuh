@@ -87,6 +87,6 @@ __device__ __forceinline__ int3 worker_items(const WinArgs& a, int n_groups) {
 b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t q_tokens, int32_t items_per_chunk, int32_t n_workers, const int32_t* d_row_seq,
                                 const int32_t* d_row_ctx, int32_t total_rows, void* stream, float item_cost, float slot_cost, bool fine_lengths);
 // Points the arguments at that plan; false when there is none.
-bool b200_attn_use_plan(b200_kv* kv, int32_t window, int32_t q_tokens, WinArgs* a);
+bool b200_attn_use_plan(b200_kv* kv, int32_t window, int32_t q_tokens, bool fine, WinArgs* a);
 // Sums the partial results of the groups that were cut.
 b200_status b200_attn_combine(b200_kv* kv, const WinArgs& a, void* stream);

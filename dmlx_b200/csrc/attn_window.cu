@@ -636,9 +636,9 @@ b200_status sm_count() {
 int head_block_of(int gqa) { return std::min(gqa, 16); }
 int q_tokens_of(int gqa) { return gqa >= 16 ? 1 : 16 / gqa; }
 
-WindowPlan* find_plan(b200_kv* kv, int window, int q_tokens) {
+WindowPlan* find_plan(b200_kv* kv, int window, int q_tokens, bool fine) {
   for (WindowPlan* p : kv->plans)
-    if (p->window == window && p->q_tokens == q_tokens) return p;
+    if (p->window == window && p->q_tokens == q_tokens && p->fine == fine) return p;
   return nullptr;
 }
 
@@ -691,11 +691,12 @@ b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t
   if (total_rows <= 0) return B200_OK;
   if (total_rows > kv->cfg.max_rows) { b200_set_error("attention: %d rows > max_rows %d", total_rows, kv->cfg.max_rows); return B200_ERR_CAPACITY; }
   const int R = kv->cfg.max_rows + 2;
-  WindowPlan* p = find_plan(kv, window, qt);
+  WindowPlan* p = find_plan(kv, window, qt, fine);
   if (!p) {
     p = new WindowPlan();
     p->window = window;
     p->q_tokens = qt;
+    p->fine = fine;
     if (cudaMalloc((void**)&p->buf, sizeof(int) * ((size_t)5 * R + 4)) != cudaSuccess) {
       delete p;
       b200_set_error("attention plan: out of device memory");
@@ -712,8 +713,8 @@ b200_status b200_attn_make_plan(b200_kv* kv, int32_t window, int32_t qt, int32_t
   return B200_OK;
 }
 
-bool b200_attn_use_plan(b200_kv* kv, int32_t window, int32_t q_tokens, WinArgs* a) {
-  const WindowPlan* p = find_plan(kv, window, q_tokens);
+bool b200_attn_use_plan(b200_kv* kv, int32_t window, int32_t q_tokens, bool fine, WinArgs* a) {
+  const WindowPlan* p = find_plan(kv, window, q_tokens, fine);
   if (!p) { b200_set_error("attention: no plan for window %d and groups of %d", window, q_tokens); return false; }
   const int R = kv->cfg.max_rows + 2;
   a->group_first = p->buf; a->chunk_start = p->buf + R; a->part_base = p->buf + 2 * R; a->row_group = p->buf + 3 * R; a->page_base = p->buf + 4 * R;
@@ -736,7 +737,7 @@ b200_status b200_window_attn_plan(b200_kv* kv, int32_t layer, int32_t window, in
   b200_status st = sm_count();
   if (st != B200_OK) return st;
   const KvLayerDev& L = kv->lay[layer];
-  if (L.values_in_keys) return b200_latent_attn_plan(kv, layer, gqa, d_row_seq, d_row_ctx, total_rows, stream);
+  if (L.values_in_keys) return b200_latent_attn_plan(kv, layer, window, gqa, d_row_seq, d_row_ctx, total_rows, stream);
   const int per_chunk = L.heads * ((gqa + 15) / 16), warps = shape_of((L.kd + 63) / 64 + (L.vd + 63) / 64).warps;
   return b200_attn_make_plan(kv, window, q_tokens_of(gqa), per_chunk, g_sms * warps, d_row_seq, d_row_ctx, total_rows, stream, 1.25f, 0.25f, false);
 }
@@ -768,7 +769,7 @@ b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
   }
   if (L.values_in_keys) return b200_latent_attn_run(kv, c, d_row_seq, d_row_ctx, total_rows, stream);
   WinArgs a;
-  if (!b200_attn_use_plan(kv, c.window, q_tokens_of(G), &a)) return B200_ERR_INVALID_ARGUMENT;
+  if (!b200_attn_use_plan(kv, c.window, q_tokens_of(G), false, &a)) return B200_ERR_INVALID_ARGUMENT;
   a.d = kv->dev; a.L = L; a.q = (const __nv_bfloat16*)c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx;
   a.total_rows = total_rows; a.n_q_heads = c.n_q_heads; a.window = c.window;
   a.G = G; a.head_block = head_block_of(G); a.n_blocks = (G + 15) / 16;

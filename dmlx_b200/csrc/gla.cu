@@ -11,6 +11,11 @@
 //   gla_scan_kernel   (request, head, slice of dv): walks the chunks with S^T in registers, mma.sync;
 //   gla_out_kernel    norm and gate of the rows.
 // f32 factors enter the tensor cores as two bf16 terms (value and remainder); the state itself stays f32.
+//
+// Matrix memory runs through the same kernels: with the running maximum m taken out, S <- e^(f + m' - m) S + (e^(i - m) k) v^T has one
+// decay per head and token, both factors at most 1, and the sum of the keys is one more value column whose values are ones.
+// memory_gates_kernel makes the factors (m is a scan over (max, +)); memory_chunk_kernel and memory_out_kernel take the places of the
+// chunk and out kernels.
 #include <cuda_bf16.h>
 
 #include <algorithm>
@@ -30,6 +35,7 @@ struct Gla {
   float* state;  // the layer's [slot][heads][dk][dv]
   int rec_elems;
   int heads, dk, dv, rank, dkp;
+  int dva, dvs;  // columns of the state in use, and from row to row (matrix memory: one more than dv, padded)
   MatSrc src;
   const float *a2, *a2_bias, *norm;
   float q_scale, inv_tau, eps;
@@ -45,46 +51,71 @@ struct Gla {
   size_t chunk_bytes, v_bytes;
   int n_slices, stages;
   int cols, groups;  // step kernel: threads = columns of VEC values x groups of key channels
-  __device__ int col_k() const { return heads * dk; }
-  __device__ int col_v() const { return 2 * heads * dk; }
-  __device__ int col_g() const { return 2 * heads * dk + heads * dv; }
+  const float4* gates;
+  int col0;
+  float den_eps, out_scale;
+  __device__ int col_k() const { return col0 + heads * dk; }
+  __device__ int col_v() const { return col0 + 2 * heads * dk; }
+  __device__ int col_g() const { return col0 + 2 * heads * dk + heads * dv; }
   __device__ int col_a() const { return 2 * heads * dk + 2 * heads * dv; }
 };
 
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float silu(float g) { return g / (1.0f + expf(-g)); }
+__device__ __forceinline__ float sigmoid(float g) { return 1.0f / (1.0f + expf(-g)); }
+// Values of a matrix memory: columns dv and on are {1, 0, 0, ..}.
+template <typename T, int VEC>
+__device__ __forceinline__ Vec<VEC> memory_value(const Gla& a, int row, int head, int c) {
+  if (c < a.dv) return mat_value<T, VEC>(a.src, row, a.col_v() + head * a.dv + c);  // (VEC divides dv)
+  Vec<VEC> v{};
+  v.v[0] = c == a.dv ? 1.f : 0.f;
+  return v;
+}
 
 // ---- token by token ------------------------------------------------------------------------------------------
-template <typename T, int VEC>
+template <typename T, int VEC, bool MEM>
 __global__ void __launch_bounds__(256, 3) gla_step_kernel(Gla a) {
   extern __shared__ float sh[];
   __shared__ float part[32];
-  const int req = blockIdx.x, head = blockIdx.y, dk = a.dk, dv = a.dv;
+  const int req = blockIdx.x, head = blockIdx.y, dk = a.dk, dv = a.dv, dvs = MEM ? a.dvs : dv, dva = MEM && VEC == 1 ? a.dva : dvs;
   const int r0 = a.cu[req], count = a.cu[req + 1] - r0;
   if (count <= 0 || (a.chunked && count > kGlaStepTokens) || a.d.state[ST_ERR] != 0) return;
-  float *q = sh, *k = q + dk, *al = k + dk, *a1 = al + dk, *red = a1 + a.rank;  // red [groups][dv]
+  float *q = sh, *k = q + dk, *al = k + dk, *a1 = al + dk, *red = a1 + (MEM ? 0 : a.rank);  // red [groups][dvs]
   const int tid = threadIdx.x, nthr = blockDim.x, groups = a.groups, tx = tid % a.cols, ty = tid / a.cols;
   const int slot = a.row_seq[r0];
   if (slot < 0 || slot >= a.d.max_seqs) return;
-  float* S = a.state + (size_t)slot * a.rec_elems + (size_t)head * dk * dv;
+  float* S = a.state + (size_t)slot * a.rec_elems + (size_t)head * dk * dvs;
   for (int t = 0; t < count; ++t) {
     const int row = r0 + t;
     const bool fresh = a.pos[row] == 0;
-    for (int r = tid; r < a.rank; r += nthr) a1[r] = mat_value<T, 1>(a.src, row, a.col_a() + r).v[0];
-    __syncthreads();
+    float4 gate{};
+    if constexpr (MEM) {
+      gate = a.gates[(size_t)row * a.heads + head];
+    } else {
+      for (int r = tid; r < a.rank; r += nthr) a1[r] = mat_value<T, 1>(a.src, row, a.col_a() + r).v[0];
+      __syncthreads();
+    }
+    const float decay = MEM ? expf(gate.x) : 0.f;
     for (int c = tid; c < dk; c += nthr) {
       const int ch = head * dk + c;
-      q[c] = mat_value<T, 1>(a.src, row, ch).v[0] * a.q_scale;
+      q[c] = mat_value<T, 1>(a.src, row, a.col0 + ch).v[0] * a.q_scale;
       k[c] = mat_value<T, 1>(a.src, row, a.col_k() + ch).v[0];
+      if constexpr (MEM) {
+        k[c] *= gate.y;
+        al[c] = decay;
+        continue;
+      }
       float z = a.a2_bias[ch];
       const float* w = a.a2 + (size_t)ch * a.rank;
       for (int r = 0; r < a.rank; ++r) z = fmaf(w[r], a1[r], z);
       al[c] = expf(log_sigmoid(z) * a.inv_tau);
     }
     __syncthreads();
-    for (int c0 = ty < groups ? tx : dv; c0 * VEC < dv; c0 += a.cols) {
+    for (int c0 = ty < groups ? tx : dva; c0 * VEC < dva; c0 += a.cols) {
       const int c = c0 * VEC;
-      const Vec<VEC> v = mat_value<T, VEC>(a.src, row, a.col_v() + head * dv + c);
+      Vec<VEC> v;
+      if constexpr (MEM) v = memory_value<T, VEC>(a, row, head, c);
+      else v = mat_value<T, VEC>(a.src, row, a.col_v() + head * dv + c);
       float acc[VEC] = {};
       constexpr int U = 8;
       for (int d0 = ty; d0 < dk; d0 += groups * U) {
@@ -92,7 +123,7 @@ __global__ void __launch_bounds__(256, 3) gla_step_kernel(Gla a) {
 #pragma unroll
         for (int u = 0; u < U; ++u) {
           const int dd = d0 + u * groups;
-          if (dd < dk && !fresh) s[u] = load_vec<VEC>(S + (size_t)dd * dv + c);
+          if (dd < dk && !fresh) s[u] = load_vec<VEC>(S + (size_t)dd * dvs + c);
           else {
 #pragma unroll
             for (int e = 0; e < VEC; ++e) s[u].v[e] = 0.f;
@@ -108,18 +139,24 @@ __global__ void __launch_bounds__(256, 3) gla_step_kernel(Gla a) {
               s[u].v[e] = fmaf(s[u].v[e], aa, kk * v.v[e]);
               acc[e] = fmaf(s[u].v[e], qq, acc[e]);
             }
-            store_vec<VEC>(S + (size_t)dd * dv + c, s[u]);
+            store_vec<VEC>(S + (size_t)dd * dvs + c, s[u]);
           }
         }
       }
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) red[ty * dv + c + e] = acc[e];
+      for (int e = 0; e < VEC; ++e) red[ty * dvs + c + e] = acc[e];
     }
     __syncthreads();
-    float ss = 0.f;
+    float ss = 0.f, inv = 1.f;
+    if constexpr (MEM) {
+      float qn = 0.f;
+      for (int g = 0; g < groups; ++g) qn += red[g * dvs + dv];
+      inv = 1.0f / (fmaxf(fabsf(qn), gate.z) + a.den_eps);
+    }
     for (int c = tid; c < dv; c += nthr) {
       float o = red[c];
-      for (int g = 1; g < groups; ++g) o += red[g * dv + c];
+      for (int g = 1; g < groups; ++g) o += red[g * dvs + c];
+      if constexpr (MEM) o *= inv;
       red[c] = o;  // (column c is read and written by this thread only)
       ss += o * o;
     }
@@ -127,7 +164,8 @@ __global__ void __launch_bounds__(256, 3) gla_step_kernel(Gla a) {
     T* dst = (T*)a.out + (size_t)row * a.out_stride + (size_t)head * dv;
     for (int c = tid; c < dv; c += nthr) {
       const float g = mat_value<T, 1>(a.src, row, a.col_g() + head * dv + c).v[0];
-      st(dst + c, red[c] * r * a.norm[c] * silu(g));
+      if constexpr (MEM) st(dst + c, red[c] * r * a.norm[head * dv + c] * sigmoid(g) * a.out_scale);
+      else st(dst + c, red[c] * r * a.norm[c] * silu(g));
     }
     __syncthreads();
   }
@@ -366,7 +404,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
     for (int s = 0; s < stages && c0 + s < c1; ++s) load(c0 + s, s);
 
   const int m0 = slice * kScanCols + warp * 16;  // first value column of the warp
-  float* S = a.state + (size_t)slot * a.rec_elems + (size_t)head * a.dk * a.dv;
+  float* S = a.state + (size_t)slot * a.rec_elems + (size_t)head * a.dk * a.dvs;
   float acc[NT][4];
   const bool fresh = a.pos[r0] == 0;
 #pragma unroll
@@ -374,7 +412,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int col = m0 + g + (e >> 1) * 8, ch = j * 8 + 2 * t + (e & 1);
-      acc[j][e] = !fresh && ch < a.dk && col < a.dv ? S[(size_t)ch * a.dv + col] : 0.f;
+      acc[j][e] = !fresh && ch < a.dk && col < a.dva ? S[(size_t)ch * a.dvs + col] : 0.f;
     }
   }
   bool ok = true;
@@ -464,7 +502,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int tok = n * 8 + 2 * t + (e & 1), col = m0 + g + (e >> 1) * 8;
-        if (tok < rows && col < a.dv) a.o[((size_t)(row0 + tok) * a.heads + head) * a.dv + col] = o[n][e];
+        if (tok < rows && col < a.dva) a.o[((size_t)(row0 + tok) * a.heads + head) * a.dvs + col] = o[n][e];
       }
     }
     __syncthreads();  // every warp has read the stage
@@ -480,7 +518,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int col = m0 + g + (e >> 1) * 8, ch = j * 8 + 2 * t + (e & 1);
-      if (ch < a.dk && col < a.dv) S[(size_t)ch * a.dv + col] = acc[j][e];
+      if (ch < a.dk && col < a.dva) S[(size_t)ch * a.dvs + col] = acc[j][e];
     }
   }
 }

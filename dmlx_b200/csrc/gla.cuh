@@ -1,4 +1,4 @@
-// Gated linear attention over the recurrent state of a layered pool (gla.cu).
+// Gated linear attention and matrix memory over the recurrent state of a layered pool (gla.cu).
 #pragma once
 #include "kv_pool.cuh"
 #include "rows.cuh"
@@ -14,7 +14,29 @@ struct GlaCall {
   float q_scale = 1.f, inv_tau = 1.f, eps = 0.f;
   void* out = nullptr;
   int out_stride = 0;
+  // Matrix memory: decay and input weight are one number per head and token, made by b200_memory_gates; the keys are summed up
+  // beside the state as its column `dv` (their values are ones), and the output is divided by max(|that sum . q|, e^-m) + den_eps,
+  // normed, times norm (of every head), sigmoid(g) and out_scale.  src columns from col0: [q | k | v | g].
+  const float4* gates = nullptr;  // [rows][heads]
+  int col0 = 0;
+  float den_eps = 0.f, out_scale = 1.f;
 };
+// Elements of a matrix memory in a slot's state: S with the key sum ([heads][dk][b200_memory_width(dv)]), then m per head.
+constexpr int b200_memory_width(int dv) { return (dv + 1 + 3) / 4 * 4; }
+constexpr int b200_memory_elems(int heads, int dk, int dv) { return heads * (dk * b200_memory_width(dv) + 1); }
+
+// Gates of a matrix memory.  src columns [i | f], one per head and kind; log input gate i = cap tanh((z_i + b_i) / cap), log forget
+// gate f = log sigmoid(cap tanh((z_f + b_f) / cap)); m_t = max(f + m_(t-1), i) from m = 0, kept in the slot's state.  Written per row
+// and head: {f + m_(t-1) - m_t, e^(i - m_t), e^(-m_t), -}.
+struct MemoryGates {
+  int layer = 0, heads = 0, m_off = 0;  // m_off: where m starts in the slot's state
+  MatSrc src;
+  const float* bias = nullptr;  // [2 heads]
+  float cap = 1.f;
+  float4* out = nullptr;
+};
+b200_status b200_memory_gates(b200_kv* kv, const MemoryGates& g, const int32_t* d_cu, const int32_t* d_row_seq, const int32_t* d_pos, int n_req,
+                              int total_rows, void* stream);
 
 // Buffers of the chunk-wise path, shared by the layers of a model: made for a number of rows and requests.
 struct GlaScratch {

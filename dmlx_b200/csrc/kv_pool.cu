@@ -585,7 +585,7 @@ static b200_status kv_create(const b200_kv_config* c_in, const b200_kv_layer* la
     for (int l = 0; l < cfg.n_layers; ++l) {
       const b200_kv_layer& y = layers[l];
       const bool pages = y.n_kv_heads > 0 && y.key_dim > 0 && y.value_dim > 0 && (!y.values_in_keys || y.value_dim <= y.key_dim);
-      const bool none = y.n_kv_heads == 0 && y.key_dim == 0 && y.value_dim == 0 && y.state_elems > 0;
+      const bool none = y.n_kv_heads == 0 && y.key_dim == 0 && y.value_dim == 0;  // recurrent, or reads another layer's pages
       if ((!pages && !none) || y.state_elems < 0) {
         b200_set_error("kv_create_layers: layer %d has no shape", l);
         return B200_ERR_INVALID_ARGUMENT;

@@ -47,6 +47,7 @@ struct KvDev {
 // device once per step: groups of rows, their chunks of pages, and where partial sums go.
 struct WindowPlan {
   int window = 0, q_tokens = 1;
+  bool fine = false;  // made for the latent kernel
   // group_first [R+2] | chunk_start [R+2] | part_base [R+2] | row_group [R+2] | page_base [R+2] | {n_groups, pages per chunk, pages per
   // worker or 0, -}
   int* buf = nullptr;

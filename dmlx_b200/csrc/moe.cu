@@ -26,6 +26,7 @@ namespace {
 
 constexpr int kMaxExperts = 1024;
 constexpr int kMaxTopK = 16;
+constexpr int kMaxGroups = 64;  // of a router's experts
 
 __device__ __forceinline__ bool beats(float va, int ia, float vb, int ib) { return va > vb || (va == vb && ia > ib); }
 
@@ -243,6 +244,128 @@ __global__ void __launch_bounds__(1024) table_place_kernel(const MoeTableLayer* 
   place_assignments(L.indices, n_tokens * L.top, L.offsets, L.order, L.inv_order);
 }
 
+// ---- experts by router, over the logits as the router's matmul left them -------------------------------------------------
+// One warp per token.  Softmax scores in f32; the experts form n_groups equal groups of neighbours, of which only the `keep` with the
+// largest best score stay open; the k largest open scores are chosen and weighed by score / (their sum + 1e-20).
+template <typename T, int PER>
+__global__ void __launch_bounds__(256) route_src_kernel(MatSrc logits, int n_tokens, int n_experts, int k, int n_groups, int keep,
+                                                        uint32_t* __restrict__ out_idx, float* __restrict__ out_w) {
+  const int token = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  if (token >= n_tokens) return;
+  float sc[PER], ch[PER];
+  float mx = -INFINITY;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int e = i * 32 + lane;
+    sc[i] = e < n_experts ? mat_value<T, 1>(logits, token, e).v[0] : -INFINITY;
+    mx = fmaxf(mx, sc[i]);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    sc[i] = i * 32 + lane < n_experts ? expf(sc[i] - mx) : 0.f;
+    sum += sc[i];
+  }
+  sum = warp_sum(sum);
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    sc[i] = sc[i] / sum;
+    ch[i] = i * 32 + lane < n_experts ? sc[i] : -INFINITY;
+  }
+  if (keep < n_groups) {  // lane g holds the scores of groups g and g + 32
+    const int per = n_experts / n_groups;
+    float best[2] = {-INFINITY, -INFINITY};
+    for (int g = 0; g < n_groups; ++g) {
+      float b = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        const int e = i * 32 + lane;
+        if (e >= g * per && e < (g + 1) * per) b = fmaxf(b, ch[i]);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) b = fmaxf(b, __shfl_xor_sync(0xffffffffu, b, o));
+      if (lane == (g & 31)) best[g >> 5] = b;
+    }
+    int before[2] = {0, 0};
+    for (int g = 0; g < n_groups; ++g) {
+      const float b = __shfl_sync(0xffffffffu, best[g >> 5], g & 31);
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+        if (beats(b, -g, best[h], -(lane + 32 * h))) ++before[h];
+    }
+    const uint64_t open = (uint64_t)__ballot_sync(0xffffffffu, lane < n_groups && before[0] < keep) |
+                          (uint64_t)__ballot_sync(0xffffffffu, lane + 32 < n_groups && before[1] < keep) << 32;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int e = i * 32 + lane;
+      if (e < n_experts && !(open >> (e / per) & 1)) ch[i] = -INFINITY;
+    }
+  }
+  float total = 0.f, mine = 0.f;
+  int mine_e = 0;
+  for (int r = 0; r < k; ++r) {
+    float bv = -INFINITY, bs = 0.f;
+    int be = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int e = i * 32 + lane;
+      if (e < n_experts && beats(ch[i], -e, bv, -be)) { bv = ch[i]; be = e; bs = sc[i]; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o), os = __shfl_xor_sync(0xffffffffu, bs, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+      if (beats(ov, -oe, bv, -be)) { bv = ov; be = oe; bs = os; }
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (i * 32 + lane == be) ch[i] = -INFINITY;
+    total += bs;
+    if (lane == r) { mine = bs; mine_e = min(be, n_experts - 1); }
+  }
+  if (lane < k) {
+    out_idx[(size_t)token * k + lane] = (uint32_t)mine_e;
+    out_w[(size_t)token * k + lane] = mine / (total + 1e-20f);
+  }
+}
+
+// The plan of one layer in one launch, a CTA per expert: it counts the assignments of the experts before its own and places its
+// own; the first also lays out the work items.
+__global__ void __launch_bounds__(1024) plan_kernel(MoeTableLayer L, int n_tokens, int tile_rows) {
+  __shared__ int s_count[kMaxExperts], s_item[kMaxExperts + 1];
+  const int n = n_tokens * L.top, tid = threadIdx.x, e = blockIdx.x;
+  for (int i = tid; i < L.n_experts; i += blockDim.x) s_count[i] = 0;
+  __syncthreads();
+  for (int a = tid; a < n; a += blockDim.x) atomicAdd(&s_count[L.indices[a]], 1);
+  __syncthreads();
+  if (tid == 0) {
+    int o = 0, it = 0;
+    for (int i = 0; i < L.n_experts; ++i) {
+      const int c = s_count[i];
+      s_count[i] = o;
+      s_item[i] = it;
+      o += c;
+      it += (c + tile_rows - 1) / tile_rows;
+    }
+    s_item[L.n_experts] = it;
+    if (e == 0) {
+      L.offsets[L.n_experts] = o;
+      *L.n_items = it;
+    }
+  }
+  __syncthreads();
+  if (e == 0) {
+    for (int i = tid; i < L.n_experts; i += blockDim.x) {
+      const int first = s_count[i], end = i + 1 < L.n_experts ? s_count[i + 1] : n;
+      L.offsets[i] = first;
+      for (int t = first, at = s_item[i]; t < end; t += tile_rows, ++at) L.items[at] = make_int4(i, t, min(tile_rows, end - t), 0);
+    }
+  }
+  place_assignments(L.indices, n, s_count, L.order, L.inv_order);
+}
+
 // Rows of x in the experts' order, 16 bytes at a time.
 __global__ void __launch_bounds__(128) gather_rows_by_order_kernel(const uint4* __restrict__ x, const int* __restrict__ order, int top, int vecs,
                                                                    uint4* __restrict__ out) {
@@ -374,6 +497,7 @@ __global__ void combine_kernel(const __nv_bfloat16* __restrict__ y_sorted, const
 
 int b200_moe_max_experts() { return kMaxExperts; }
 int b200_moe_max_top() { return kMaxTopK; }
+int b200_moe_max_groups() { return kMaxGroups; }
 
 b200_status b200_moe_table_plan(const MoeTableLayer* d_layers, int n_layers, int most_experts, const uint32_t* d_tokens, int n_tokens, int vocab,
                                 int tile_rows, void* stream) {
@@ -382,6 +506,25 @@ b200_status b200_moe_table_plan(const MoeTableLayer* d_layers, int n_layers, int
   table_route_kernel<<<n_layers, 1024, 0, s>>>(d_layers, d_tokens, n_tokens, vocab, tile_rows);
   B200_LAUNCH_CHECK();
   table_place_kernel<<<dim3(most_experts, n_layers), 1024, 0, s>>>(d_layers, n_tokens);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
+b200_status b200_moe_route_plan(const MoeTableLayer& L, const MatSrc& logits, bool f32, int n_groups, int keep_groups, int n_tokens, int tile_rows,
+                                float* d_weights, void* stream) {
+  if (L.n_experts <= 0 || L.n_experts > kMaxExperts || L.top <= 0 || L.top > kMaxTopK || n_groups <= 0 || n_groups > kMaxGroups ||
+      L.n_experts % n_groups != 0 || keep_groups <= 0 || keep_groups > n_groups || L.top > keep_groups * (L.n_experts / n_groups)) {
+    b200_set_error("router: %d experts, top %d, %d of %d groups", L.n_experts, L.top, keep_groups, n_groups);
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  if (n_tokens <= 0) return B200_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  auto route = [&](auto* kernel) { kernel<<<(n_tokens + 7) / 8, 256, 0, s>>>(logits, n_tokens, L.n_experts, L.top, n_groups, keep_groups, L.indices, d_weights); };
+  const int per = (L.n_experts + 31) / 32;
+  if (f32) route(per <= 1 ? route_src_kernel<float, 1> : (per <= 4 ? route_src_kernel<float, 4> : (per <= 8 ? route_src_kernel<float, 8> : route_src_kernel<float, 32>)));
+  else route(per <= 1 ? route_src_kernel<__nv_bfloat16, 1> : (per <= 4 ? route_src_kernel<__nv_bfloat16, 4> : (per <= 8 ? route_src_kernel<__nv_bfloat16, 8> : route_src_kernel<__nv_bfloat16, 32>)));
+  B200_LAUNCH_CHECK();
+  plan_kernel<<<L.n_experts, 1024, 0, s>>>(L, n_tokens, tile_rows);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

@@ -1,11 +1,12 @@
-// Experts chosen by token id (moe.cu): the plan of a step for all layers at once.
+// Experts of a decoder layer (moe.cu): chosen by token id, the plan of a step for all layers at once, or by a router.
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>
 
 #include "dmlx_b200.h"
+#include "rows.cuh"
 
-// One layer on the device: its table [vocab][top] and where the plan goes, for up to max_rows * top assignments.
+// One layer on the device: its table [vocab][top] (null with a router) and where the plan goes, for up to max_rows * top assignments.
 struct MoeTableLayer {
   const int* table = nullptr;
   int n_experts = 0, top = 0;
@@ -15,7 +16,12 @@ struct MoeTableLayer {
 };
 int b200_moe_max_experts();
 int b200_moe_max_top();
+int b200_moe_max_groups();
 b200_status b200_moe_table_plan(const MoeTableLayer* d_layers, int n_layers, int most_experts, const uint32_t* d_tokens, int n_tokens, int vocab,
                                 int tile_rows, void* stream);
+// Routes the tokens of one layer by their router logits (softmax, best experts of the best keep_groups of n_groups groups, weights
+// renormalised over the chosen ones) and plans its matmuls.  f32: how logits that the matmul wrote itself are stored.
+b200_status b200_moe_route_plan(const MoeTableLayer& L, const MatSrc& logits, bool f32, int n_groups, int keep_groups, int n_tokens, int tile_rows,
+                                float* d_weights, void* stream);
 // out[p] = x[order[p] / top], bf16 rows of `width` elements (a multiple of 8).
 b200_status b200_moe_gather_order(const void* d_x, const int* d_order, int top, int n_assign, int width, void* d_out, void* stream);

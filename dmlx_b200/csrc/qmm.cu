@@ -93,8 +93,11 @@ __device__ __forceinline__ void row_params(const unsigned char* blk, int r, int 
   }
 }
 
+// gelu(z) = z Phi(z), the exact form.
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+
 // Epilogue of one output quad: columns n..n+3 of row `token` (residual add, SwiGLU over
-// interleaved gate/up rows, per-row scale), written as bf16.
+// interleaved gate/up rows, GELU, per-row scale), written as bf16.
 __device__ __forceinline__ void finish_store(const QmmArgs& a, int token, int n, float4 acc) {
   const float rs = a.row_scale(token);
   if (a.epilogue == B200_EPI_SWIGLU) {
@@ -111,6 +114,8 @@ __device__ __forceinline__ void finish_store(const QmmArgs& a, int token, int n,
     if (a.epilogue == B200_EPI_RESIDUAL) {
       const uint2 rv = *reinterpret_cast<const uint2*>(a.residual + o);
       acc.x += ptx::bf16_lo(rv.x); acc.y += ptx::bf16_hi(rv.x); acc.z += ptx::bf16_lo(rv.y); acc.w += ptx::bf16_hi(rv.y);
+    } else if (a.epilogue == B200_EPI_GELU) {
+      acc.x = gelu_erf(acc.x); acc.y = gelu_erf(acc.y); acc.z = gelu_erf(acc.z); acc.w = gelu_erf(acc.w);
     }
     __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x * rs, acc.y * rs), hi = __floats2bfloat162_rn(acc.z * rs, acc.w * rs);
     uint2 ov;
@@ -471,7 +476,12 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
               const int token = t0 + c0 + j;
               const size_t o = (size_t)token * a.out_stride(a.n) + y_col + n;
               float acc = __uint_as_float(v[j]);
+              if (MODE == B200_Q_BF16 && a.y_f32) {
+                reinterpret_cast<float*>(a.y)[o] = acc;
+                continue;
+              }
               if (a.epilogue == B200_EPI_RESIDUAL) acc += __bfloat162float(a.residual[o]);
+              else if (MODE == B200_Q_BF16 && a.epilogue == B200_EPI_GELU) acc = gelu_erf(acc);
               a.y[o] = __float2bfloat16(acc * a.row_scale(token));
             }
           }
@@ -518,6 +528,7 @@ __device__ __forceinline__ void tile_epilogue_store(const QmmArgs& a, const uint
         const size_t o = (size_t)token * a.out_stride(a.n) + n;
         float acc = __uint_as_float(v[j]);
         if (a.epilogue == B200_EPI_RESIDUAL) acc += __bfloat162float(a.residual[o]);
+        else if (a.epilogue == B200_EPI_GELU) acc = gelu_erf(acc);
         a.y[o] = __float2bfloat16(acc * a.row_scale(token));
       }
     }
@@ -2795,6 +2806,7 @@ static b200_status qmm_entry(const b200_qweight* w, const void* d_x, int32_t row
   if (w->n_experts != 1) { b200_set_error("qmm: stacked expert weights go through the grouped entry point"); return B200_ERR_INVALID_ARGUMENT; }
   if (epilogue == B200_EPI_RESIDUAL && !d_residual) { b200_set_error("qmm: residual epilogue without a residual"); return B200_ERR_INVALID_ARGUMENT; }
   if (epilogue == B200_EPI_SWIGLU && (w->n % 2) != 0) { b200_set_error("qmm: SwiGLU needs an even N"); return B200_ERR_INVALID_ARGUMENT; }
+  if (epilogue == B200_EPI_GELU && w->mode != B200_Q_BF16) { b200_set_error("qmm: the GELU epilogue serves dense bf16 weights"); return B200_ERR_UNSUPPORTED; }
   // Quantised weights, up to 16 rows: register-dequant mma.sync kernel (pure weight streaming).  More
   // rows: tcgen05 with the dequantised weights in tensor memory; above 128 rows the tile-pair kernel
   // where its grid is one well-filled wave without a K split (gate/up-sized matrices: 74 vs 85 us at
@@ -2879,7 +2891,7 @@ struct F32Args {
   const unsigned char* blocks;
   const float* x;
   float* y;
-  int rows, kc, x_stride, y_stride, n_valid, swiglu;
+  int rows, kc, x_stride, y_stride, n_valid, swiglu, gelu;
   size_t expert_stride;        // bytes between the matrices of a stack
   int x_group, y_group;        // block-diagonal: columns of x and y per matrix (grid z)
   const int4* items;           // grouped: {matrix, first sorted row, rows} (grid y)
@@ -2960,7 +2972,7 @@ __global__ void __launch_bounds__(256) qmm_f32_kernel(F32Args a) {
     } else {
 #pragma unroll
       for (int e = 0; e < 4; ++e)
-        if (n + e < n_valid) y[(size_t)row * y_stride + n + e] = acc[i][e];
+        if (n + e < n_valid) y[(size_t)row * y_stride + n + e] = a.gelu ? gelu_erf(acc[i][e]) : acc[i][e];
     }
   }
 }
@@ -2972,7 +2984,7 @@ extern "C" b200_status b200_qmm_f32(const b200_qweight* w, const float* d_x, int
   if (st != B200_OK) return st;
   if (w->mode != B200_Q_BF16 || w->n_experts != 1) { b200_set_error("qmm_f32: dense bf16 weights only"); return B200_ERR_UNSUPPORTED; }
   const bool swiglu = epilogue == B200_EPI_SWIGLU;
-  if ((epilogue != B200_EPI_NONE && !swiglu) || n_valid < 0 || n_valid > (swiglu ? w->n / 2 : w->n) || y_stride < n_valid) {
+  if ((epilogue != B200_EPI_NONE && epilogue != B200_EPI_GELU && !swiglu) || n_valid < 0 || n_valid > (swiglu ? w->n / 2 : w->n) || y_stride < n_valid) {
     b200_set_error("qmm_f32: bad epilogue, n_valid or stride");
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -2980,6 +2992,7 @@ extern "C" b200_status b200_qmm_f32(const b200_qweight* w, const float* d_x, int
   F32Args a{};
   a.blocks = w->d_blocks; a.x = d_x; a.y = d_y; a.rows = rows; a.kc = w->kc; a.x_stride = w->k; a.y_stride = y_stride; a.n_valid = n_valid;
   a.swiglu = swiglu ? 1 : 0;
+  a.gelu = epilogue == B200_EPI_GELU ? 1 : 0;
   qmm_f32_kernel<<<dim3(w->nt, (rows + kF32Rows - 1) / kF32Rows), 256, 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
@@ -3004,11 +3017,11 @@ b200_status b200_qmm_f32_grouped(const b200_qweight* w, const float* d_x, const 
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
   const bool swiglu = epilogue == B200_EPI_SWIGLU;
-  if (w->mode != B200_Q_BF16 || (epilogue != B200_EPI_NONE && !swiglu)) { b200_set_error("qmm_f32_grouped: dense bf16 weights, no or the SwiGLU epilogue"); return B200_ERR_UNSUPPORTED; }
+  if (w->mode != B200_Q_BF16 || (epilogue != B200_EPI_NONE && epilogue != B200_EPI_GELU && !swiglu)) { b200_set_error("qmm_f32_grouped: dense bf16 weights, no, the SwiGLU or the GELU epilogue"); return B200_ERR_UNSUPPORTED; }
   if (max_items <= 0) return B200_OK;
   F32Args a{};
   a.blocks = w->d_blocks; a.x = d_x; a.y = d_y; a.kc = w->kc; a.x_stride = w->k; a.y_stride = y_stride; a.n_valid = swiglu ? w->n / 2 : w->n;
-  a.swiglu = swiglu ? 1 : 0; a.expert_stride = (size_t)w->nt * w->kc * w->block_bytes;
+  a.swiglu = swiglu ? 1 : 0; a.gelu = epilogue == B200_EPI_GELU ? 1 : 0; a.expert_stride = (size_t)w->nt * w->kc * w->block_bytes;
   a.items = d_items; a.n_items = d_n_items; a.order = d_order; a.order_div = order_div > 0 ? order_div : 1;
   qmm_f32_kernel<<<dim3(w->nt, max_items), 256, 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
@@ -3016,7 +3029,7 @@ b200_status b200_qmm_f32_grouped(const b200_qweight* w, const float* d_x, const 
 }
 
 b200_status b200_qmm_blocks(const b200_qweight* w, const void* d_x, int32_t x_stride, int32_t x_group, int32_t rows, void* d_y, int32_t y_stride,
-                            int32_t y_group, void* stream) {
+                            int32_t y_group, void* stream, bool y_f32) {
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
   if (w->mode != B200_Q_BF16 || x_group < w->k || x_stride % 8 != 0 || x_group % 8 != 0) { b200_set_error("qmm_blocks: dense bf16 blocks, strides of 16 bytes"); return B200_ERR_INVALID_ARGUMENT; }
@@ -3025,6 +3038,7 @@ b200_status b200_qmm_blocks(const b200_qweight* w, const void* d_x, int32_t x_st
   a.blocks = w->d_blocks; a.x = (const __nv_bfloat16*)d_x; a.y = (__nv_bfloat16*)d_y;
   a.rows = rows; a.n = w->n; a.k = w->k; a.nt = w->nt; a.kc = w->kc; a.epilogue = B200_EPI_NONE;
   a.expert_stride = (size_t)w->nt * w->kc * w->block_bytes;
+  a.y_f32 = y_f32 ? 1 : 0;
   a.groups = w->n_experts; a.x_group = x_group; a.y_group = y_group; a.y_stride = y_stride;
   return launch_tc<B200_Q_BF16>(a, rows, (cudaStream_t)stream, x_stride);
 }
@@ -3038,6 +3052,7 @@ b200_status b200_qmm_grouped(const b200_qweight* w, const void* d_x, int32_t row
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
   if (rows <= 0) return B200_OK;
+  if (epilogue == B200_EPI_GELU && w->mode != B200_Q_BF16) { b200_set_error("qmm_grouped: the GELU epilogue serves dense bf16 weights"); return B200_ERR_UNSUPPORTED; }
   QmmArgs a{};
   a.blocks = w->d_blocks; a.x = (const __nv_bfloat16*)d_x; a.y = (__nv_bfloat16*)d_y; a.residual = nullptr;
   a.row_scales = d_row_scales;

@@ -54,6 +54,7 @@ struct QmmArgs {
   int y_stride;                 // elements between output rows (0: exactly the outputs of a row)
   // block-diagonal launches: matrix e of a stack multiplies columns e * x_group .. of every row and writes columns e * y_group ..
   int groups, x_group, y_group;
+  int y_f32;                    // block-diagonal launches: y holds floats
   int keep_f32;                 // the caller wants the f32 sums: no kernel writes bf16 output itself
   b200_qmm_partials* defer = nullptr;  // when set, a dense launch with epilogue NONE leaves its finish pass to the caller
 
@@ -68,9 +69,10 @@ b200_status b200_qmm_grouped(const b200_qweight* w, const void* d_x, int32_t row
 // Dense bf16 weights, rows of the output y_stride elements apart.
 b200_status b200_qmm_to(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t y_stride, int32_t epilogue, void* stream);
 // Block-diagonal matmul: the n_experts matrices [n, k] of w are the blocks (one per attention head, say).
-// y[r][e * y_group + i] = sum_j w_e[i][j] x[r][e * x_group + j]; rows of x are x_stride apart, those of y y_stride.  bf16, f32 accumulation.
+// y[r][e * y_group + i] = sum_j w_e[i][j] x[r][e * x_group + j]; rows of x are x_stride apart, those of y y_stride.  bf16, f32 accumulation;
+// y_f32: the sums are written as they are, d_y holds floats.
 b200_status b200_qmm_blocks(const b200_qweight* w, const void* d_x, int32_t x_stride, int32_t x_group, int32_t rows, void* d_y, int32_t y_stride,
-                            int32_t y_group, void* stream);
+                            int32_t y_group, void* stream, bool y_f32 = false);
 // The f32 forms (f32 activations, dense bf16 weights widened exactly, CUDA cores).  Grouped: rows of x are taken through
 // order (x row order[p] / order_div for sorted row p; null: sorted row p itself), items of at most 64 rows.
 b200_status b200_qmm_f32_blocks(const b200_qweight* w, const float* d_x, int32_t x_stride, int32_t x_group, int32_t rows, float* d_y,
