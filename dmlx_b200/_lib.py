@@ -19,7 +19,7 @@ if not os.path.exists(LIB_PATH):
 
 lib = C.CDLL(LIB_PATH)
 
-u64, u32, i32, f32 = C.c_uint64, C.c_uint32, C.c_int32, C.c_float
+u64, u32, i32, f32, f64 = C.c_uint64, C.c_uint32, C.c_int32, C.c_float, C.c_double
 vp = C.c_void_p
 P = C.POINTER
 
@@ -266,13 +266,16 @@ class ModelInfo(C.Structure):
 
 class DecoderLayer(C.Structure):
     _fields_ = [(n, i32) for n in ("n_heads", "n_kv_heads", "key_dim", "value_dim", "window", "ffn", "flags")] + [("scale", f32)] + [
-        (n, i32) for n in ("mixer", "kv_rank", "rot_dim")] + [("rot_base", f32), ("decay_rank", i32), ("decay_tau", f32)] + [
-        (n, i32) for n in ("n_experts", "top_k", "expert_ffn")]
+        (n, i32) for n in ("mixer", "kv_rank", "rot_dim")] + [("rot_base", f64), ("decay_rank", i32), ("decay_tau", f32)] + [
+        (n, i32) for n in ("n_experts", "top_k", "expert_ffn", "n_groups", "keep_groups", "q_rank", "kv_source")] + [
+        (n, f64) for n in ("yarn_factor", "yarn_original", "yarn_fast", "yarn_slow")] + [("conv_taps", i32), ("lru_decay", f32)] + [
+        (n, i32) for n in ("mem_heads", "mem_key_dim", "mem_value_dim")] + [(n, f32) for n in ("mem_gate_cap", "mix_scale", "mem_scale")]
 
 
 class DecoderConfig(C.Structure):
     _fields_ = [(n, i32) for n in ("n_layers", "hidden", "vocab", "loop_start", "loop_stop", "loop_times", "dtype", "max_rows", "max_reqs",
-                                   "max_seqs")] + [("norm_eps", f32), ("embed_scale", f32), ("logit_scale", f32), ("flags", i32)]
+                                   "max_seqs")] + [("norm_eps", f32), ("embed_scale", f32), ("logit_scale", f32), ("flags", i32),
+                                   ("residual_scale", f32)]
 
 
 class GlaShape(C.Structure):

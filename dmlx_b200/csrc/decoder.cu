@@ -30,13 +30,16 @@
 #include "common.h"
 #include "gla.cuh"
 #include "kv_pool.cuh"
+#include "lru.cuh"
 #include "model_step.cuh"
 #include "moe.cuh"
 #include "qmm.cuh"
 #include "rows.cuh"
+#include "short_conv.cuh"
 
 namespace {
 
+constexpr float kMemoryEps = 1e-6f;  // added to a matrix memory's denominator
 constexpr double kLog2e = 1.4426950408889634;
 
 int pad64(int n) { return (n + 63) / 64 * 64; }
@@ -64,6 +67,11 @@ struct RowArgs {
   const int* moe_rows = nullptr;  // [row * moe_k + j] -> row of moe_y
   int moe_k = 0, moe_stride = 0;
   float moe_w = 0.f;
+  const float* moe_wts = nullptr;  // [row * moe_k + j]: a weight of its own for each, instead of moe_w
+  // norms behind the sum: x = norm(x_scale * x + src) * norm_w is the residual and what the next matmul reads
+  float x_scale = 1.f;
+  int norm_x = 0;
+  int plain_h = 0;                // h = x without a norm
   // depth average: the result is kept as hist[n_hist], and x becomes sum_j depth[j] hist[j]
   const float* depth = nullptr;   // null for the embedding, which is kept as it is
   float* hist = nullptr;
@@ -129,8 +137,9 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
       }
       for (int m = 0; m < a.moe_k; ++m) {
         const Vec<VEC> e = load_vec<VEC>((const T*)a.moe_y + (size_t)a.moe_rows[row * a.moe_k + m] * a.moe_stride + i * VEC);
+        const float w = a.moe_wts ? a.moe_wts[row * a.moe_k + m] : a.moe_w;
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(a.moe_w, e.v[j], v.v[j]);
+        for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(w, e.v[j], v.v[j]);
       }
 #pragma unroll
       for (int j = 0; j < VEC; ++j) ys += v.v[j] * v.v[j];
@@ -149,7 +158,7 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
         if constexpr (NQ > 0) x = res[k];
         else x = load_vec<VEC>(xr + i * VEC);
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) v.v[j] += x.v[j];
+        for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(a.x_scale, x.v[j], v.v[j]);
       }
       if (a.depth) {
         float* hr = a.hist + (size_t)row * a.hidden + i * VEC;
@@ -168,8 +177,12 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
 #pragma unroll
       for (int j = 0; j < VEC; ++j) ss += v.v[j] * v.v[j];
       put(i, k, v);
-      store_vec<VEC>(xr + i * VEC, v);
+      if (!a.norm_x) store_vec<VEC>(xr + i * VEC, v);
     });
+  }
+  if (a.plain_h) {
+    T* hr = (T*)a.h + (size_t)row * a.h_stride;
+    each([&](int i, int k) { store_vec<VEC>(hr + i * VEC, get(i, k)); });
   }
   if (a.norm_w) {
     const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)a.hidden + a.eps);
@@ -180,6 +193,7 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
 #pragma unroll
       for (int j = 0; j < VEC; ++j) v.v[j] *= r * w.v[j];
       store_vec<VEC>(hr + i * VEC, v);
+      if (a.norm_x) store_vec<VEC>(xr + i * VEC, v);
     });
   }
   if (a.cat) {
@@ -225,7 +239,26 @@ struct QkvArgs {
   void* q;
   int q_stride;
   const int *pos, *row_seq;
+  // convolution, weights of the q and k norms, rotation of the first `rot` dimensions, factor on v: decoder_qkv_conv_kernel
+  const int *cu = nullptr, *row_to_req = nullptr;
+  ShortConv conv;  // channels as in the projection's columns
+  const float *q_norm = nullptr, *k_norm = nullptr;
+  const float2* rotation = nullptr;
+  int rot = 0, halves = 0;
+  float v_scale = 1.f;
 };
+
+// Where key or value head `head` of a row lives in its page; null when the step's reservation failed (nothing is written then, the
+// error word is set).
+template <typename T>
+__device__ __forceinline__ T* page_row(const QkvArgs& a, int row, int head, bool is_v) {
+  const int pos = a.pos[row], seq = a.row_seq[row];
+  const int page_idx = pos / a.d.page_size, slot = pos - page_idx * a.d.page_size;
+  if (seq < 0 || seq >= a.d.max_seqs || page_idx >= a.d.seq_pages[seq]) return nullptr;
+  const int page = a.d.block_table[(size_t)seq * a.d.max_pages_per_seq + page_idx];
+  char* pool = is_v ? (char*)a.d.v_pool + a.L.v_off : (char*)a.d.k_pool + a.L.k_off;
+  return (T*)pool + (((size_t)page * a.L.heads + head) * a.d.page_size + slot) * (size_t)(is_v ? a.L.vd : a.L.kd);
+}
 
 // One warp per (row, head); q heads, then k heads, then v heads.  Grid y covers the heads, eight at a time.
 template <typename T, int VEC>
@@ -242,13 +275,8 @@ __global__ void __launch_bounds__(256) decoder_qkv_kernel(QkvArgs a) {
   if (is_q) {
     dst = (T*)a.q + (size_t)row * a.q_stride + (size_t)head * a.L.kd;
   } else {
-    const int pos = a.pos[row], seq = a.row_seq[row];
-    const int page_idx = pos / a.d.page_size, slot = pos - page_idx * a.d.page_size;
-    // a step whose reservation failed has no page for this row: nothing is written (the error word is set)
-    if (seq < 0 || seq >= a.d.max_seqs || page_idx >= a.d.seq_pages[seq]) return;
-    const int page = a.d.block_table[(size_t)seq * a.d.max_pages_per_seq + page_idx];
-    char* pool = is_v ? (char*)a.d.v_pool + a.L.v_off : (char*)a.d.k_pool + a.L.k_off;
-    dst = (T*)pool + (((size_t)page * H + head) * a.d.page_size + slot) * (size_t)width;
+    dst = page_row<T>(a, row, head, is_v);
+    if (!dst) return;
   }
   auto value = [&](int c) {
     Vec<VEC> v = mat_value<T, VEC>(a.src, row, n0 + c);
@@ -294,7 +322,73 @@ __global__ void __launch_bounds__(256) decoder_qkv_kernel(QkvArgs a) {
   for (int c = dim + lane; c < width; c += 32) st(dst + c, 0.f);
 }
 
+// The same with everything a design may put between projection and attention: bias, convolution over the tokens before, norm with a
+// weight, rotation.  One warp per (row, head), the head's row in shared memory; the warp of a request's first row also takes the rows
+// that read the convolution's state (short_conv.cuh).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) decoder_qkv_conv_kernel(QkvArgs a) {
+  extern __shared__ float row_sh[];
+  const int first = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, H = a.L.heads, u = blockIdx.y * 8 + warp;
+  if (u >= a.hq + 2 * H || a.d.state[ST_ERR] != 0) return;
+  const bool is_q = u < a.hq, is_v = u >= a.hq + H;
+  const int head = is_q ? u : (is_v ? u - a.hq - H : u - a.hq);
+  const int dim = is_v ? a.L.value_dim : a.L.key_dim, width = is_v ? a.L.vd : a.L.kd;
+  const int n0 = is_v ? (a.hq + H) * a.L.key_dim + head * dim : u * dim;
+  float* sh = row_sh + warp * max(a.L.key_dim, a.L.value_dim);
+  const int req = a.row_to_req[first], r0 = a.cu[req], count = a.cu[req + 1] - r0, slot = a.row_seq[first];
+  if (slot < 0 || slot >= a.d.max_seqs) return;
+  auto value = [&](int row, int c) {
+    Vec<VEC> v = mat_value<T, VEC>(a.src, row, c);
+    if (a.bias) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v.v[e] += a.bias[c + e];
+    }
+    return v;
+  };
+  const int n = conv_rows(a.conv, first - r0, count);
+  const float* norm = is_q ? a.q_norm : (is_v ? nullptr : a.k_norm);
+  for (int row = first; row < first + n; ++row) {
+    T* dst = is_q ? (T*)a.q + (size_t)row * a.q_stride + (size_t)head * a.L.kd : page_row<T>(a, row, head, is_v);
+    if (!dst) return;
+    float ss = 0.f;
+    for (int c = lane * VEC; c < dim; c += 32 * VEC) {
+      const Vec<VEC> v = a.conv.taps > 0 ? conv_value<VEC>(a.conv, value, row, row - r0, a.pos[row], slot, n0 + c) : value(row, n0 + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += v.v[e] * v.v[e];
+      store_vec<VEC>(sh + c, v);
+    }
+    float r = is_v ? a.v_scale : 1.f;
+    if (a.qk_norm && !is_v) r = 1.0f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
+    __syncwarp();
+    auto at = [&](int c) { return norm ? sh[c] * r * norm[c] : sh[c] * r; };
+    const int rot = is_v ? 0 : a.rot;
+    for (int i = lane; i < rot / 2; i += 32) {
+      const int c0 = a.halves ? i : 2 * i, c1 = a.halves ? i + rot / 2 : 2 * i + 1;
+      const float2 cs = a.rotation[(size_t)row * (rot / 2) + i];
+      const float x = at(c0), y = at(c1);
+      st(dst + c0, x * cs.x - y * cs.y);
+      st(dst + c1, y * cs.x + x * cs.y);
+    }
+    for (int c = rot + lane; c < width; c += 32) st(dst + c, c < dim ? at(c) : 0.f);
+    __syncwarp();
+  }
+  if (first == r0 && a.conv.taps > 1)
+    for (int c = lane * VEC; c < dim; c += 32 * VEC) conv_update<VEC>(a.conv, value, r0, count, slot, n0 + c);
+}
+
 b200_status launch_qkv(const QkvArgs& a, int rows, cudaStream_t s) {
+  if (a.conv.taps > 0 || a.q_norm || a.rot > 0 || a.v_scale != 1.f) {
+    const bool vec = a.L.key_dim % 4 == 0 && a.L.value_dim % 4 == 0 && (a.src.ws || a.src.y_stride % 4 == 0) && a.conv.slot_elems % 4 == 0 &&
+                     a.conv.channels % 4 == 0;
+    const size_t smem = sizeof(float) * 8 * std::max(a.L.key_dim, a.L.value_dim);
+    if (smem > 200 * 1024) { b200_set_error("decoder: head widths %d / %d are too large", a.L.key_dim, a.L.value_dim); return B200_ERR_UNSUPPORTED; }
+    auto* kernel = a.d.elem_bytes == 4 ? (vec ? decoder_qkv_conv_kernel<float, 4> : decoder_qkv_conv_kernel<float, 1>)
+                                       : (vec ? decoder_qkv_conv_kernel<__nv_bfloat16, 4> : decoder_qkv_conv_kernel<__nv_bfloat16, 1>);
+    if (smem > 48 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    kernel<<<dim3(rows, (a.hq + 2 * a.L.heads + 7) / 8), 256, smem, s>>>(a);
+    B200_LAUNCH_CHECK();
+    return B200_OK;
+  }
   const bool v4 = a.L.key_dim % 4 == 0 && a.L.value_dim % 4 == 0 && a.src.y_stride % 4 == 0;
   auto* kernel = a.d.elem_bytes == 4 ? (v4 ? decoder_qkv_kernel<float, 4> : decoder_qkv_kernel<float, 1>)
                                      : (v4 ? decoder_qkv_kernel<__nv_bfloat16, 4> : decoder_qkv_kernel<__nv_bfloat16, 1>);
@@ -315,7 +409,11 @@ float bf16_to_f(uint16_t b) {
 const char* kTensorNames[] = {"q", "k", "v", "o", "gate", "up", "down", "head", "loop input", "embedding", "q bias", "k bias", "v bias",
                               "sink", "norm 1", "norm 2", "post-norm 1", "post-norm 2", "final norm", "latent", "latent norm", "key expansion",
                               "value expansion", "output gate", "decay 1", "decay 2", "decay bias", "head norm", "expert gate", "expert up",
-                              "expert down", "depth weights"};
+                              "expert down", "depth weights", "query latent", "query latent norm", "q norm", "k norm", "q convolution",
+                              "k convolution", "v convolution", "memory q", "memory k", "memory v", "memory output gate", "memory output",
+                              "memory input gate", "memory forget gate", "memory input gate bias", "memory forget gate bias", "memory norm",
+                              "lru branch", "lru branch bias", "lru input", "lru input bias", "lru convolution", "lru convolution bias",
+                              "lru decay gate", "lru decay gate bias", "lru input gate", "lru input gate bias", "lru lambda", "router"};
 
 }  // namespace
 
@@ -325,44 +423,83 @@ struct b200_decoder : b200_model {
     b200_decoder_layer s{};
     // wqkv: all projections the mixer takes from h.  wo: W_o, in parallel layers [W_o | W_down] over concatenated columns.
     b200_qweight *wqkv = nullptr, *wo = nullptr, *wgu = nullptr, *wdown = nullptr, *wuk = nullptr, *wuv = nullptr, *we_gu = nullptr, *we_down = nullptr;
+    // wuq: queries from their latent.  wgates: gates of the matrix memory, or of the LRU's blocks.
+    b200_qweight *wuq = nullptr, *wgates = nullptr, *wrouter = nullptr;
     float *bias = nullptr, *sinks = nullptr, *slopes = nullptr, *norm1 = nullptr, *norm2 = nullptr, *post1 = nullptr, *post2 = nullptr;
     float *dkv_norm = nullptr, *a2 = nullptr, *a2_bias = nullptr, *head_norm = nullptr, *depth = nullptr;
+    float *dq_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr, *conv = nullptr, *conv_bias = nullptr, *gate_bias = nullptr, *mem_norm = nullptr;
+    float *lru_bias = nullptr, *lru_rate = nullptr;  // [y | x | r | i], [width]
     int* table = nullptr;
     std::vector<int> h_table;
     int moe = -1;       // place among the layers with experts
     int rotation = -1;  // its rotation table
     int qkv_n() const {
-      if (s.mixer == B200_MIX_LATENT) return s.n_heads * (s.key_dim + s.rot_dim) + s.kv_rank + s.rot_dim;
+      if (s.mixer == B200_MIX_LATENT) return (s.q_rank > 0 ? s.q_rank : q_n()) + (s.kv_source > 0 ? 0 : s.kv_rank + s.rot_dim);
+      if (s.mixer == B200_MIX_LRU) return 2 * attn_n();
       if (s.mixer == B200_MIX_GLA) return 2 * s.n_heads * (s.key_dim + s.value_dim) + s.decay_rank;
-      return s.n_heads * s.key_dim + s.n_kv_heads * (s.key_dim + s.value_dim);
+      return attention_n() + 2 * s.mem_heads * (s.mem_key_dim + s.mem_value_dim);
     }
+    int q_n() const { return s.n_heads * (s.key_dim + s.rot_dim); }  // queries of latent attention
+    int attention_n() const { return s.n_heads * s.key_dim + s.n_kv_heads * (s.key_dim + s.value_dim); }
+    int mem_n() const { return s.mem_heads * s.mem_value_dim; }
+    int mem_col() const { return pad64(attn_n()); }
+    int router_n() const { return s.flags & B200_DEC_ROUTER ? s.n_experts : 0; }
+    // state of a slot: the matrix memory, then the convolution's inputs
+    int conv_off() const { return s.mem_heads > 0 ? (b200_memory_elems(s.mem_heads, s.mem_key_dim, s.mem_value_dim) + 3) / 4 * 4 : 0; }
+    int state_elems() const {
+      int n = 0;
+      if (s.mixer == B200_MIX_GLA) n = s.n_heads * s.key_dim * s.value_dim;
+      if (s.mixer == B200_MIX_LRU) n = (b200_lru_elems(attn_n(), s.conv_taps) + 3) / 4 * 4;
+      if (s.mixer == B200_MIX_ATTENTION) n = (conv_off() + (s.conv_taps > 1 ? s.conv_taps - 1 : 0) * attention_n() + 3) / 4 * 4;
+      return n;
+    }
+    int lru_group() const { return pad64(s.value_dim); }
     int attn_n() const { return s.n_heads * s.value_dim; }
     bool parallel() const { return (s.flags & B200_DEC_PARALLEL) != 0; }
-    int out_k() const { return pad64(attn_n()) + (parallel() && s.ffn > 0 ? pad64(s.ffn) : 0); }  // columns wo reads
+    bool gelu() const { return (s.flags & B200_DEC_FF_GELU) != 0; }
+    int epilogue() const { return gelu() ? B200_EPI_GELU : B200_EPI_SWIGLU; }
+    int ffn_col() const { return mem_col() + (s.mem_heads > 0 ? pad64(mem_n()) : 0); }
+    int out_k() const { return ffn_col() + (parallel() && s.ffn > 0 ? pad64(s.ffn) : 0); }  // columns wo reads
     int plain_stride() const { return pad64(s.key_dim); }
     int latent_width() const { return (s.kv_rank + s.rot_dim + 15) / 16 * 16; }
     std::vector<int> projections() const {
-      if (s.mixer == B200_MIX_LATENT) return {B200_DEC_W_Q, B200_DEC_W_DKV};
+      if (s.mixer == B200_MIX_LATENT) {
+        std::vector<int> w{s.q_rank > 0 ? B200_DEC_W_DQ : B200_DEC_W_Q};
+        if (s.kv_source == 0) w.push_back(B200_DEC_W_DKV);
+        return w;
+      }
+      if (s.mixer == B200_MIX_LRU) return {B200_DEC_W_LRU_Y, B200_DEC_W_LRU_X};
       if (s.mixer == B200_MIX_GLA) return {B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V, B200_DEC_W_OUT_GATE, B200_DEC_W_A1};
-      return {B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V};
+      std::vector<int> w{B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V};
+      if (s.mem_heads > 0) w.insert(w.end(), {B200_DEC_W_MEM_Q, B200_DEC_W_MEM_K, B200_DEC_W_MEM_V, B200_DEC_W_MEM_G});
+      return w;
     }
     b200_kv_layer cache() const {
-      if (s.mixer == B200_MIX_LATENT) return b200_kv_layer{1, s.kv_rank + s.rot_dim, s.kv_rank, 1, 0};
-      if (s.mixer == B200_MIX_GLA) return b200_kv_layer{0, 0, 0, 0, s.n_heads * s.key_dim * s.value_dim};
-      return b200_kv_layer{s.n_kv_heads, s.key_dim, s.value_dim, 0, 0};
+      if (s.mixer == B200_MIX_LATENT) return s.kv_source > 0 ? b200_kv_layer{0, 0, 0, 0, 0} : b200_kv_layer{1, s.kv_rank + s.rot_dim, s.kv_rank, 1, 0};
+      if (s.mixer == B200_MIX_GLA || s.mixer == B200_MIX_LRU) return b200_kv_layer{0, 0, 0, 0, state_elems()};
+      return b200_kv_layer{s.n_kv_heads, s.key_dim, s.value_dim, 0, state_elems()};
     }
   };
-  // Rotations of a step, one table per (base, width) in the stack.
-  struct Rotation { float base; int dims; double* freq; float2* rows; };
+  // Rotations of a step, one table per (base, width, scaling) in the stack.
+  struct Rotation {
+    double base, factor, original, fast, slow;
+    int dims;
+    double* freq;
+    float2* rows;
+    double size() const { return factor > 0 ? 0.1 * std::log(factor) + 1.0 : 1.0; }
+  };
   std::vector<Rotation> rotations;
   // Experts by token id: plan buffers of every layer that has them (d_moe: the same on the device), and the rows they work on.
   std::vector<MoeTableLayer> moe;
   MoeTableLayer* d_moe = nullptr;
   std::vector<int> moe_layers;
+  int n_tables = 0;  // layers whose experts come from a table
   void *moe_x = nullptr, *moe_act = nullptr, *moe_y = nullptr;
   GlaScratch gla;
-  bool has_gla = false;
-  void *q_plain = nullptr, *lat_out = nullptr;
+  bool has_gla = false;  // some layer works chunk by chunk
+  void *q_plain = nullptr, *lat_out = nullptr, *q_latent = nullptr;
+  float *lru_gates = nullptr, *moe_wts = nullptr;  // gates in front of their activation; weights of a router's experts
+  float4* mem_gates = nullptr;
   float* hist = nullptr;  // [layers + 1][max_rows][hidden]: embedding output and results of the layers
   std::vector<Layer> layers;
   struct Run { int layer; bool opens; };  // opens: the first layer of a pass of the loop
@@ -387,18 +524,23 @@ struct b200_decoder : b200_model {
   b200_status rows_step(RowArgs a, int rows, int next, cudaStream_t s);
   b200_status attention(b200_kv* kv, int run, int rows, void* stream);
   b200_status mixer(b200_kv* kv, int run, int n_req, int T, void* stream);
+  b200_status memory(b200_kv* kv, int run, const MatSrc& src, int n_req, int T, void* stream);
+  b200_status lru(b200_kv* kv, int run, const MatSrc& src, int n_req, int T, void* stream);
   b200_status experts(const Layer& l, int T, int tile_rows, void* stream);
   b200_status begin_step(b200_kv* kv, int n_req, int T, int tile_rows, void* stream);
   int moe_tile_rows(int T) const;
+  int kv_run(int run) const { return layers[runs[run].layer].s.kv_source > 0 ? layers[runs[run].layer].s.kv_source - 1 : run; }  // whose pages it reads
+  bool sum_norm() const { return (cfg.flags & B200_DEC_SUM_NORM) != 0; }
 };
 
 b200_decoder::~b200_decoder() {
-  void* dev[] = {embed, final_norm, x, x0, rec, h, cat, y, q, attn, act, last, q_plain, lat_out, hist, moe_x, moe_act, moe_y, d_moe};
+  void* dev[] = {embed, final_norm, x, x0, rec, h, cat, y, q, attn, act, last, q_plain, lat_out, hist, moe_x, moe_act, moe_y, d_moe, q_latent, lru_gates, moe_wts, mem_gates};
   for (void* p : dev) if (p) cudaFree(p);
   for (Layer& l : layers) {
-    void* lp[] = {l.bias, l.sinks, l.slopes, l.norm1, l.norm2, l.post1, l.post2, l.dkv_norm, l.a2, l.a2_bias, l.head_norm, l.depth, l.table};
+    void* lp[] = {l.bias, l.sinks, l.slopes, l.norm1, l.norm2, l.post1, l.post2, l.dkv_norm, l.a2, l.a2_bias, l.head_norm, l.depth, l.table,
+                  l.dq_norm, l.q_norm, l.k_norm, l.conv, l.conv_bias, l.gate_bias, l.mem_norm, l.lru_bias, l.lru_rate};
     for (void* p : lp) if (p) cudaFree(p);
-    for (b200_qweight* w : {l.wqkv, l.wo, l.wgu, l.wdown, l.wuk, l.wuv, l.we_gu, l.we_down}) b200_qweight_destroy(w);
+    for (b200_qweight* w : {l.wqkv, l.wo, l.wgu, l.wdown, l.wuk, l.wuv, l.we_gu, l.we_down, l.wuq, l.wgates, l.wrouter}) b200_qweight_destroy(w);
   }
   for (MoeTableLayer& t : moe) {
     void* tp[] = {t.indices, t.offsets, t.order, t.inv_order, t.n_items, t.items};
@@ -457,7 +599,11 @@ b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t 
   a.h = h;
   a.h_stride = hp;
   if (hist) { a.hist = hist; a.hist_stride = (size_t)max_rows * cfg.hidden; }
-  if (next >= 0 && next < (int)runs.size()) {
+  if (sum_norm()) {
+    if (a.tokens) a.plain_h = 1;
+    else a.norm_x = 1;
+    a.x_scale = cfg.residual_scale;
+  } else if (next >= 0 && next < (int)runs.size()) {
     if (runs[next].opens) { a.cat = cat; a.cat_stride = catp; }
     else a.norm_w = layers[runs[next].layer].norm1;
   }
@@ -474,11 +620,11 @@ b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t 
 b200_status b200_decoder::attention(b200_kv* kv, int run, int rows, void* stream) {
   const Layer& l = layers[runs[run].layer];
   WindowAttnCall c;
-  c.layer = run;
+  c.layer = kv_run(run);
   c.n_q_heads = l.s.n_heads;
   c.window = l.s.window;
   c.q = q;
-  c.q_stride = l.s.n_heads * kv->lay[run].kd;
+  c.q_stride = l.s.n_heads * kv->lay[c.layer].kd;
   c.scale = l.s.scale;
   c.slopes_log2 = l.slopes;
   c.sinks_log2 = l.sinks;
@@ -505,22 +651,24 @@ b200_status b200_decoder::begin_step(b200_kv* kv, int n_req, int T, int tile_row
   b200_decoder* m = this;
   cudaStream_t cs = (cudaStream_t)stream;
   b200_status st = B200_OK;
-  // one plan per (window, GQA group) of the stack, shared by its layers
-  std::vector<std::pair<int, int>> planned;
+  // one plan per (window, GQA group) of the stack, shared by its layers (latent layers: of the same key width)
+  std::vector<std::tuple<int, int, int>> planned;
   for (size_t r = 0; r < runs.size(); ++r) {
     const b200_decoder_layer& s = layers[runs[r].layer].s;
-    if (s.mixer == B200_MIX_GLA) continue;
-    const std::pair<int, int> key{s.window, s.mixer == B200_MIX_LATENT ? s.n_heads : s.n_heads / s.n_kv_heads};
-    if (!attn_mma || !b200_window_attn_takes_mma(kv, (int)r) || std::find(planned.begin(), planned.end(), key) != planned.end()) continue;
+    if (s.mixer == B200_MIX_GLA || s.mixer == B200_MIX_LRU) continue;
+    const bool latent = s.mixer == B200_MIX_LATENT;
+    const int pages_of = kv_run((int)r);
+    const std::tuple<int, int, int> key{s.window, latent ? s.n_heads : s.n_heads / s.n_kv_heads, latent ? kv->lay[pages_of].kd : 0};
+    if (!attn_mma || !b200_window_attn_takes_mma(kv, pages_of) || std::find(planned.begin(), planned.end(), key) != planned.end()) continue;
     planned.push_back(key);
-    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, (int)r, key.first, key.second, d_row_seq, d_row_ctx, T, stream));
+    MODEL_STEP_CAT(0, b200_window_attn_plan(kv, pages_of, std::get<0>(key), std::get<1>(key), d_row_seq, d_row_ctx, T, stream));
   }
   if (has_gla && T > n_req) MODEL_STEP_CAT(0, b200_gla_plan(gla, d_cu, n_req, T, stream));
-  for (const Rotation& t : rotations) MODEL_STEP(b200_rotation_table(t.freq, t.dims, d_pos, T, t.rows, stream));
-  if (!moe_layers.empty()) {
+  for (const Rotation& t : rotations) MODEL_STEP(b200_rotation_table(t.freq, t.dims, t.size(), d_pos, T, t.rows, stream));
+  if (n_tables > 0) {
     int most = 0;
     for (const MoeTableLayer& t : moe) most = std::max(most, t.n_experts);
-    MODEL_STEP(b200_moe_table_plan(d_moe, (int)moe.size(), most, d_tokens, T, cfg.vocab, tile_rows, stream));
+    MODEL_STEP(b200_moe_table_plan(d_moe, n_tables, most, d_tokens, T, cfg.vocab, tile_rows, stream));
   }
   return B200_OK;
 }
@@ -533,7 +681,15 @@ b200_status b200_decoder::mixer(b200_kv* kv, int run, int n_req, int T, void* st
   const b200_decoder_layer& s = l.s;
   b200_status st = B200_OK;
   MatSrc src;
+  if (s.mem_heads > 0) {  // the gates' sums stay f32, and are used up before the next product
+    MODEL_STEP_CAT(1, matmul(l.wgates, h, T, 2, &src, stream));
+    MemoryGates g;
+    g.layer = run; g.heads = s.mem_heads; g.m_off = s.mem_heads * s.mem_key_dim * b200_memory_width(s.mem_value_dim);
+    g.src = src; g.bias = l.gate_bias; g.cap = s.mem_gate_cap; g.out = mem_gates;
+    MODEL_STEP_CAT(0, b200_memory_gates(kv, g, d_cu, d_row_seq, d_pos, n_req, T, stream));
+  }
   MODEL_STEP_CAT(1, matmul(l.wqkv, h, T, 1, &src, stream));
+  if (s.mixer == B200_MIX_LRU) return lru(kv, run, src, n_req, T, stream);
   if (s.mixer == B200_MIX_GLA) {
     GlaCall c;
     c.layer = run; c.heads = s.n_heads; c.dk = s.key_dim; c.dv = s.value_dim; c.rank = s.decay_rank; c.src = src;
@@ -545,12 +701,20 @@ b200_status b200_decoder::mixer(b200_kv* kv, int run, int n_req, int T, void* st
     return B200_OK;
   }
   if (s.mixer == B200_MIX_LATENT) {
+    const int pages_of = kv_run(run);
     LatentPrep p;
-    p.layer = run; p.heads = s.n_heads; p.dim = s.key_dim; p.rot = s.rot_dim; p.rank = s.kv_rank; p.src = src; p.norm = l.dkv_norm;
+    p.layer = pages_of; p.heads = s.n_heads; p.dim = s.key_dim; p.rot = s.rot_dim; p.rank = s.kv_rank; p.src = src; p.norm = l.dkv_norm;
+    p.halves = (s.flags & B200_DEC_ROT_HALVES) != 0; p.keys = s.kv_source == 0;
     p.eps = cfg.norm_eps; p.rotation = l.rotation >= 0 ? rotations[l.rotation].rows : nullptr;
     p.q_plain = q_plain; p.plain_stride = l.plain_stride(); p.q = q;
+    if (s.q_rank > 0) {
+      p.heads = 0; p.q_rank = s.q_rank; p.q_norm = l.dq_norm; p.q_latent = q_latent; p.q_latent_stride = pad64(s.q_rank);
+      MODEL_STEP_CAT(2, b200_latent_prep(kv, p, d_pos, d_row_seq, T, stream));
+      MODEL_STEP_CAT(1, matmul(l.wuq, q_latent, T, 1, &src, stream));
+      p.heads = s.n_heads; p.q_rank = 0; p.q_latent_stride = 0; p.src = src; p.keys = false;
+    }
     MODEL_STEP_CAT(2, b200_latent_prep(kv, p, d_pos, d_row_seq, T, stream));
-    const int H = s.n_heads, kd = kv->lay[run].kd, lat = pad64(s.kv_rank);
+    const int H = s.n_heads, kd = kv->lay[pages_of].kd, lat = pad64(s.kv_rank);
     auto blocks = [&](const b200_qweight* w, const void* in, int in_group, void* out, int out_stride, int out_group) {
       return f32() ? b200_qmm_f32_blocks(w, (const float*)in, H * in_group, in_group, T, (float*)out, out_stride, out_group, stream)
                    : b200_qmm_blocks(w, in, H * in_group, in_group, T, out, out_stride, out_group, stream);
@@ -563,8 +727,50 @@ b200_status b200_decoder::mixer(b200_kv* kv, int run, int n_req, int T, void* st
   QkvArgs a;
   a.d = kv->dev; a.L = kv->lay[run]; a.src = src; a.bias = l.bias; a.hq = s.n_heads; a.qk_norm = s.flags & B200_DEC_QK_NORM ? 1 : 0;
   a.eps = cfg.norm_eps; a.q = q; a.q_stride = s.n_heads * kv->lay[run].kd; a.pos = d_pos; a.row_seq = d_row_seq;
+  a.cu = d_cu; a.row_to_req = d_row_to_req; a.q_norm = l.q_norm; a.k_norm = l.k_norm;
+  if (l.rotation >= 0) { a.rotation = rotations[l.rotation].rows; a.rot = s.rot_dim; a.halves = s.flags & B200_DEC_ROT_HALVES ? 1 : 0; }
+  if (s.conv_taps > 0) {
+    a.conv.taps = s.conv_taps; a.conv.channels = l.attention_n(); a.conv.w = l.conv;
+    a.conv.state = kv->dev.rec_pool + kv->lay[run].rec_off + l.conv_off(); a.conv.slot_elems = kv->lay[run].rec_elems;
+  }
+  if (s.mem_heads > 0) a.v_scale = s.mix_scale;  // the factor of the whole mixer
   MODEL_STEP_CAT(2, launch_qkv(a, T, cs));
+  if (s.mem_heads > 0 && (st = memory(kv, run, src, n_req, T, stream)) != B200_OK) return st;
   MODEL_STEP_CAT(0, attention(kv, run, T, stream));
+  return B200_OK;
+}
+
+// The matrix memory beside attention: its part of the projection -> its columns of the rows W_o reads.
+b200_status b200_decoder::memory(b200_kv* kv, int run, const MatSrc& src, int n_req, int T, void* stream) {
+  b200_decoder* m = this;
+  cudaStream_t cs = (cudaStream_t)stream;
+  const Layer& l = layers[runs[run].layer];
+  const b200_decoder_layer& s = l.s;
+  b200_status st = B200_OK;
+  GlaCall c;
+  c.layer = run; c.heads = s.mem_heads; c.dk = s.mem_key_dim; c.dv = s.mem_value_dim; c.src = src; c.col0 = l.attention_n();
+  c.gates = mem_gates; c.norm = l.mem_norm; c.eps = cfg.norm_eps; c.den_eps = kMemoryEps; c.out_scale = s.mem_scale;
+  c.q_scale = (float)(1.0 / std::sqrt((double)s.mem_key_dim));
+  c.out = (char*)attn + l.mem_col() * elem(); c.out_stride = l.out_k();
+  MODEL_STEP_CAT(0, b200_gla_run(kv, gla, c, d_cu, d_row_seq, d_pos, n_req, T, attn_mma, stream));
+  return B200_OK;
+}
+
+b200_status b200_decoder::lru(b200_kv* kv, int run, const MatSrc& src, int n_req, int T, void* stream) {
+  b200_decoder* m = this;
+  cudaStream_t cs = (cudaStream_t)stream;
+  const Layer& l = layers[runs[run].layer];
+  const b200_decoder_layer& s = l.s;
+  b200_status st = B200_OK;
+  const int W = l.attn_n(), ub = l.lru_group();
+  LruCall c;
+  c.layer = run; c.width = W; c.blocks = s.n_heads; c.src = src; c.y_bias = l.lru_bias; c.x_bias = l.lru_bias + W;
+  c.conv.taps = s.conv_taps; c.conv.w = l.conv; c.conv.bias = l.conv_bias; c.u = q_plain; c.u_group = ub; c.gates = lru_gates;
+  c.r_bias = l.lru_bias + 2 * W; c.i_bias = l.lru_bias + 3 * W; c.rate = l.lru_rate; c.out = attn; c.out_stride = l.out_k();
+  MODEL_STEP_CAT(2, b200_lru_prep(kv, c, d_cu, d_row_to_req, d_row_seq, d_pos, T, stream));
+  MODEL_STEP_CAT(1, f32() ? b200_qmm_f32_blocks(l.wgates, (const float*)q_plain, s.n_heads * ub, ub, T, lru_gates, 2 * W, 2 * s.value_dim, stream)
+                          : b200_qmm_blocks(l.wgates, q_plain, s.n_heads * ub, ub, T, lru_gates, 2 * W, 2 * s.value_dim, stream, true));
+  MODEL_STEP_CAT(0, b200_lru_scan(kv, c, d_cu, d_row_seq, d_pos, n_req, T, stream));
   return B200_OK;
 }
 
@@ -575,13 +781,18 @@ b200_status b200_decoder::experts(const Layer& l, int T, int tile_rows, void* st
   b200_status st = B200_OK;
   const MoeTableLayer& t = moe[l.moe];
   const int A = T * t.top, act_w = pad64(l.s.expert_ffn), items = std::min(A, t.n_experts + A / tile_rows);
+  if (l.wrouter) {
+    MatSrc z;
+    MODEL_STEP_CAT(1, matmul(l.wrouter, h, T, 2, &z, stream));
+    MODEL_STEP(b200_moe_route_plan(t, z, f32(), std::max(l.s.n_groups, 1), l.s.n_groups > 0 ? l.s.keep_groups : 1, T, tile_rows, moe_wts, stream));
+  }
   if (f32()) {
-    MODEL_STEP_CAT(1, b200_qmm_f32_grouped(l.we_gu, (const float*)h, t.order, t.top, (float*)moe_act, act_w, B200_EPI_SWIGLU, t.items, t.n_items, items, stream));
+    MODEL_STEP_CAT(1, b200_qmm_f32_grouped(l.we_gu, (const float*)h, t.order, t.top, (float*)moe_act, act_w, l.epilogue(), t.items, t.n_items, items, stream));
     MODEL_STEP_CAT(1, b200_qmm_f32_grouped(l.we_down, (const float*)moe_act, nullptr, 1, (float*)moe_y, hp, B200_EPI_NONE, t.items, t.n_items, items, stream));
     return B200_OK;
   }
   MODEL_STEP(b200_moe_gather_order(h, t.order, t.top, A, hp, moe_x, stream));
-  MODEL_STEP_CAT(1, b200_qmm_grouped(l.we_gu, moe_x, A, moe_act, B200_EPI_SWIGLU, nullptr, 0.f, t.items, t.n_items, items, tile_rows, stream));
+  MODEL_STEP_CAT(1, b200_qmm_grouped(l.we_gu, moe_x, A, moe_act, l.epilogue(), nullptr, 0.f, t.items, t.n_items, items, tile_rows, stream));
   MODEL_STEP_CAT(1, b200_qmm_grouped(l.we_down, moe_act, A, moe_y, B200_EPI_NONE, nullptr, 0.f, t.items, t.n_items, items, tile_rows, stream));
   return B200_OK;
 }
@@ -616,22 +827,24 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
     auto feed_forward = [&](void* out, int out_stride) -> b200_status {
       if (s.n_experts > 0 && (st = experts(l, T, tile_rows, stream)) != B200_OK) return st;
       if (s.ffn == 0) return B200_OK;
-      if (f32()) MODEL_STEP_CAT(1, b200_qmm_f32(l.wgu, (const float*)h, T, (float*)out, out_stride, pad64(s.ffn), B200_EPI_SWIGLU, stream));
-      else MODEL_STEP_CAT(1, b200_qmm_to(l.wgu, h, T, out, out_stride, B200_EPI_SWIGLU, stream));
+      if (f32()) MODEL_STEP_CAT(1, b200_qmm_f32(l.wgu, (const float*)h, T, (float*)out, out_stride, pad64(s.ffn), l.epilogue(), stream));
+      else MODEL_STEP_CAT(1, b200_qmm_to(l.wgu, h, T, out, out_stride, l.epilogue(), stream));
       return B200_OK;
     };
     auto last_rows = [&](const float* post) -> b200_status {  // the layer's last sublayer joins the residual
       RowArgs a{};
+      if (sum_norm()) a.norm_w = s.ffn > 0 || s.n_experts > 0 ? l.norm2 : l.norm1;
       a.src = src;
       a.post_w = post;
       if (s.n_experts > 0) {
         a.moe_y = moe_y; a.moe_rows = moe[l.moe].inv_order; a.moe_k = s.top_k; a.moe_stride = hp; a.moe_w = 1.0f / (float)s.top_k;
+        if (l.wrouter) a.moe_wts = moe_wts;
       }
       if (l.depth) { a.depth = l.depth; a.n_hist = (int)r + 1; }
       return rows_step(a, T, (int)r + 1, cs);
     };
     if (l.parallel()) {
-      if ((st = feed_forward((char*)attn + pad64(l.attn_n()) * elem(), l.out_k())) != B200_OK) return st;
+      if ((st = feed_forward((char*)attn + l.ffn_col() * elem(), l.out_k())) != B200_OK) return st;
       if ((st = mixer(kv, (int)r, n_req, T, stream)) != B200_OK) return st;
       MODEL_STEP_CAT(1, matmul(l.wo, attn, T, 1, &src, stream));
       MODEL_STEP(last_rows(nullptr));
@@ -645,7 +858,7 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
         RowArgs a{};
         a.src = src;
         a.post_w = l.post1;
-        a.norm_w = l.norm2;
+        a.norm_w = sum_norm() ? l.norm1 : l.norm2;
         MODEL_STEP(rows_step(a, T, -1, cs));
         if ((st = feed_forward(act, pad64(s.ffn))) != B200_OK) return st;
         src = MatSrc{};
@@ -692,17 +905,20 @@ uint64_t tensor_elems(const b200_decoder* m, int layer, int which) {
   }
   const b200_decoder_layer& s = m->layers[layer].s;
   const uint64_t H = s.n_heads, norm = c.flags & B200_DEC_SCALAR_NORM ? 1 : D, ef = (uint64_t)s.n_experts * s.expert_ffn;
-  const bool latent = s.mixer == B200_MIX_LATENT, gla = s.mixer == B200_MIX_GLA, soft = s.mixer == B200_MIX_ATTENTION;
+  const bool latent = s.mixer == B200_MIX_LATENT, gla = s.mixer == B200_MIX_GLA, soft = s.mixer == B200_MIX_ATTENTION, lru = s.mixer == B200_MIX_LRU;
+  const uint64_t MH = s.mem_heads, mk = MH * s.mem_key_dim, mv = MH * s.mem_value_dim, W = lru ? H * s.value_dim : 0;
+  const uint64_t gate = s.flags & B200_DEC_FF_GELU ? 0 : 1, taps = soft ? s.conv_taps : 0, weighed = soft && s.flags & B200_DEC_QK_NORM_WEIGHT ? s.key_dim : 0;
   const uint64_t qn = H * (s.key_dim + (latent ? s.rot_dim : 0)), kn = (gla ? H : s.n_kv_heads) * (uint64_t)s.key_dim,
                  vn = (gla ? H : s.n_kv_heads) * (uint64_t)s.value_dim;
   const bool bias = soft && s.flags & B200_DEC_QKV_BIAS, post = s.flags & B200_DEC_POST_NORM;
   const bool ff = s.ffn > 0 || s.n_experts > 0, second = ff && !(s.flags & B200_DEC_PARALLEL);
   switch (which) {
-    case B200_DEC_W_Q: return qn * D;
-    case B200_DEC_W_K: return latent ? 0 : kn * D;
-    case B200_DEC_W_V: return latent ? 0 : vn * D;
+    case B200_DEC_W_Q: return lru ? 0 : qn * (latent && s.q_rank > 0 ? s.q_rank : D);
+    case B200_DEC_W_K: return latent || lru ? 0 : kn * D;
+    case B200_DEC_W_V: return latent || lru ? 0 : vn * D;
     case B200_DEC_W_O: return D * H * s.value_dim;
-    case B200_DEC_W_GATE: case B200_DEC_W_UP: case B200_DEC_W_DOWN: return D * s.ffn;
+    case B200_DEC_W_GATE: return gate * D * s.ffn;
+    case B200_DEC_W_UP: case B200_DEC_W_DOWN: return D * s.ffn;
     case B200_DEC_B_Q: return bias ? qn : 0;
     case B200_DEC_B_K: return bias ? kn : 0;
     case B200_DEC_B_V: return bias ? vn : 0;
@@ -711,8 +927,10 @@ uint64_t tensor_elems(const b200_decoder* m, int layer, int which) {
     case B200_DEC_NORM2: return second ? norm : 0;
     case B200_DEC_POSTNORM1: return post ? norm : 0;
     case B200_DEC_POSTNORM2: return post && second ? norm : 0;
-    case B200_DEC_W_DKV: return latent ? (uint64_t)(s.kv_rank + s.rot_dim) * D : 0;
-    case B200_DEC_DKV_NORM: return latent ? s.kv_rank : 0;
+    case B200_DEC_W_DKV: return latent && s.kv_source == 0 ? (uint64_t)(s.kv_rank + s.rot_dim) * D : 0;
+    case B200_DEC_DKV_NORM: return latent && s.kv_source == 0 ? s.kv_rank : 0;
+    case B200_DEC_W_DQ: return latent ? s.q_rank * D : 0;
+    case B200_DEC_DQ_NORM: return latent ? s.q_rank : 0;
     case B200_DEC_W_UK: return latent ? H * s.key_dim * s.kv_rank : 0;
     case B200_DEC_W_UV: return latent ? H * s.value_dim * s.kv_rank : 0;
     case B200_DEC_W_OUT_GATE: return gla ? vn * D : 0;
@@ -720,7 +938,22 @@ uint64_t tensor_elems(const b200_decoder* m, int layer, int which) {
     case B200_DEC_W_A2: return gla ? kn * s.decay_rank : 0;
     case B200_DEC_B_A2: return gla ? kn : 0;
     case B200_DEC_HEAD_NORM: return gla ? s.value_dim : 0;
-    case B200_DEC_W_EXPERT_GATE: case B200_DEC_W_EXPERT_UP: case B200_DEC_W_EXPERT_DOWN: return ef * D;
+    case B200_DEC_W_EXPERT_GATE: return gate * ef * D;
+    case B200_DEC_W_EXPERT_UP: case B200_DEC_W_EXPERT_DOWN: return ef * D;
+    case B200_DEC_Q_NORM: case B200_DEC_K_NORM: return weighed;
+    case B200_DEC_CONV_Q: return qn * taps;
+    case B200_DEC_CONV_K: return kn * taps;
+    case B200_DEC_CONV_V: return vn * taps;
+    case B200_DEC_W_MEM_Q: case B200_DEC_W_MEM_K: return mk * D;
+    case B200_DEC_W_MEM_V: case B200_DEC_W_MEM_G: case B200_DEC_W_MEM_O: return mv * D;
+    case B200_DEC_W_MEM_I: case B200_DEC_W_MEM_F: return MH * D;
+    case B200_DEC_B_MEM_I: case B200_DEC_B_MEM_F: return MH;
+    case B200_DEC_MEM_NORM: return mv;
+    case B200_DEC_W_LRU_Y: case B200_DEC_W_LRU_X: return W * D;
+    case B200_DEC_W_LRU_R: case B200_DEC_W_LRU_I: return W * s.value_dim;
+    case B200_DEC_LRU_CONV: return W * s.conv_taps;
+    case B200_DEC_B_LRU_Y: case B200_DEC_B_LRU_X: case B200_DEC_B_LRU_CONV: case B200_DEC_B_LRU_R: case B200_DEC_B_LRU_I: case B200_DEC_LRU_LAMBDA: return W;
+    case B200_DEC_W_ROUTER: return s.flags & B200_DEC_ROUTER ? (uint64_t)s.n_experts * D : 0;
     case B200_DEC_DEPTH: return c.flags & B200_DEC_DEPTH_AVERAGE ? layer + 2 : 0;
     default: return 0;
   }
@@ -759,8 +992,58 @@ b200_status take_norm(b200_decoder* m, int layer, int which, float** out, double
   b200_status st = take(m, layer, which, &bits);
   if (st != B200_OK) return st;
   std::vector<float> v(m->cfg.hidden);
-  for (size_t i = 0; i < v.size(); ++i) v[i] = (float)(bf16_to_f(bits[bits.size() == 1 ? 0 : i]) * factor);
+  const float stored_at = m->cfg.flags & B200_DEC_NORM_OFFSET ? 1.f : 0.f;
+  for (size_t i = 0; i < v.size(); ++i) v[i] = (float)((stored_at + bf16_to_f(bits[bits.size() == 1 ? 0 : i])) * factor);
   return upload_f32(v, out);
+}
+
+// Several vectors one behind the other.
+b200_status take_vectors(b200_decoder* m, int layer, std::vector<int> which, float** out) {
+  std::vector<float> all;
+  for (int w : which) {
+    std::vector<uint16_t> bits;
+    b200_status st = take(m, layer, w, &bits);
+    if (st != B200_OK) return st;
+    for (uint16_t b : bits) all.push_back(bf16_to_f(b));
+  }
+  return upload_f32(all, out);
+}
+
+// Convolutions [channels, taps] one behind the other, as [taps][channels].
+b200_status take_conv(b200_decoder* m, int layer, std::vector<int> which, int taps, float** out) {
+  std::vector<float> all;
+  for (int w : which) {
+    std::vector<uint16_t> bits;
+    b200_status st = take(m, layer, w, &bits);
+    if (st != B200_OK) return st;
+    for (uint16_t b : bits) all.push_back(bf16_to_f(b));
+  }
+  const size_t channels = all.size() / taps;
+  std::vector<float> t(all.size());
+  for (size_t c = 0; c < channels; ++c)
+    for (int k = 0; k < taps; ++k) t[k * channels + c] = all[c * taps + k];
+  return upload_f32(t, out);
+}
+
+// The blocks' gate matrices, r rows then i rows, and exp's factor lru_decay * softplus(lam).
+b200_status take_lru(b200_decoder* m, int layer, b200_decoder::Layer& l) {
+  const int n = l.s.n_heads, w = l.s.value_dim, kp = pad64(w);
+  std::vector<uint16_t> part[2], lam;
+  b200_status st;
+  if ((st = take(m, layer, B200_DEC_W_LRU_R, &part[0])) != B200_OK || (st = take(m, layer, B200_DEC_W_LRU_I, &part[1])) != B200_OK ||
+      (st = take(m, layer, B200_DEC_LRU_LAMBDA, &lam)) != B200_OK)
+    return st;
+  std::vector<uint16_t> all((size_t)n * 2 * w * kp, 0);
+  for (int b = 0; b < n; ++b)
+    for (int g = 0; g < 2; ++g)
+      for (int r = 0; r < w; ++r) std::memcpy(&all[((size_t)b * 2 * w + g * w + r) * kp], &part[g][((size_t)b * w + r) * w], sizeof(uint16_t) * w);
+  if ((st = b200_qweight_create(B200_Q_BF16, n, 2 * w, kp, all.data(), nullptr, nullptr, &l.wgates)) != B200_OK) return st;
+  std::vector<float> rate(lam.size());
+  for (size_t i = 0; i < rate.size(); ++i) {
+    const double x = bf16_to_f(lam[i]);
+    rate[i] = (float)(l.s.lru_decay * (std::max(x, 0.0) + std::log1p(std::exp(-std::fabs(x)))));
+  }
+  return upload_f32(rate, &l.lru_rate);
 }
 
 // Matrices [n, k_i] beside one another as one weight, each padded to a multiple of 64 columns.
@@ -794,22 +1077,22 @@ b200_status take_stack(b200_decoder* m, int layer, int which, int count, int n, 
   return b200_qweight_create(B200_Q_BF16, count, n, kp, w.data(), nullptr, nullptr, out);
 }
 
-// Experts: gate and up rows interleaved, [2 pad(ff), pad(hidden)]; down [pad(hidden), pad(ff)].
+// Experts: gate and up rows interleaved, [2 pad(ff), pad(hidden)] (without a gate [pad(ff), pad(hidden)]); down [pad(hidden), pad(ff)].
 b200_status take_experts(b200_decoder* m, int layer, b200_decoder::Layer& l) {
-  const int E = l.s.n_experts, f = l.s.expert_ffn, D = m->cfg.hidden, fp = pad64(f), dp = pad64(D);
+  const int E = l.s.n_experts, f = l.s.expert_ffn, D = m->cfg.hidden, fp = pad64(f), dp = pad64(D), per = l.gelu() ? 1 : 2;
   std::vector<uint16_t> gate, up, down;
   b200_status st;
-  if ((st = take(m, layer, B200_DEC_W_EXPERT_GATE, &gate)) != B200_OK || (st = take(m, layer, B200_DEC_W_EXPERT_UP, &up)) != B200_OK ||
+  if ((per == 2 && (st = take(m, layer, B200_DEC_W_EXPERT_GATE, &gate)) != B200_OK) || (st = take(m, layer, B200_DEC_W_EXPERT_UP, &up)) != B200_OK ||
       (st = take(m, layer, B200_DEC_W_EXPERT_DOWN, &down)) != B200_OK)
     return st;
-  std::vector<uint16_t> w((size_t)E * 2 * fp * dp, 0);
+  std::vector<uint16_t> w((size_t)E * per * fp * dp, 0);
   for (int e = 0; e < E; ++e)
     for (int r = 0; r < f; ++r) {
-      uint16_t* dst = &w[((size_t)e * 2 * fp + 2 * r) * dp];
-      std::memcpy(dst, &gate[((size_t)e * f + r) * D], sizeof(uint16_t) * D);
-      std::memcpy(dst + dp, &up[((size_t)e * f + r) * D], sizeof(uint16_t) * D);
+      uint16_t* dst = &w[((size_t)e * per * fp + per * r) * dp];
+      if (per == 2) std::memcpy(dst, &gate[((size_t)e * f + r) * D], sizeof(uint16_t) * D);
+      std::memcpy(dst + (per - 1) * dp, &up[((size_t)e * f + r) * D], sizeof(uint16_t) * D);
     }
-  if ((st = b200_qweight_create(B200_Q_BF16, E, 2 * fp, dp, w.data(), nullptr, nullptr, &l.we_gu)) != B200_OK) return st;
+  if ((st = b200_qweight_create(B200_Q_BF16, E, per * fp, dp, w.data(), nullptr, nullptr, &l.we_gu)) != B200_OK) return st;
   w.assign((size_t)E * dp * fp, 0);
   for (int e = 0; e < E; ++e)
     for (int r = 0; r < D; ++r) std::memcpy(&w[((size_t)e * dp + r) * fp], &down[((size_t)e * D + r) * f], sizeof(uint16_t) * f);
@@ -826,9 +1109,12 @@ b200_status upload_table(b200_decoder* m, int layer, b200_decoder::Layer& l) {
 
 // After the last table is in place: the plan structures the kernels read.
 b200_status upload_moe(b200_decoder* m) {
-  if (m->moe.empty()) return B200_OK;
-  if (!m->d_moe) B200_CUDA_TRY(cudaMalloc((void**)&m->d_moe, sizeof(MoeTableLayer) * m->moe.size()));
-  B200_CUDA_TRY(cudaMemcpy(m->d_moe, m->moe.data(), sizeof(MoeTableLayer) * m->moe.size(), cudaMemcpyHostToDevice));
+  std::vector<MoeTableLayer> with_table;
+  for (const MoeTableLayer& t : m->moe) if (t.table) with_table.push_back(t);
+  m->n_tables = (int)with_table.size();
+  if (with_table.empty()) return B200_OK;
+  if (!m->d_moe) B200_CUDA_TRY(cudaMalloc((void**)&m->d_moe, sizeof(MoeTableLayer) * with_table.size()));
+  B200_CUDA_TRY(cudaMemcpy(m->d_moe, with_table.data(), sizeof(MoeTableLayer) * with_table.size(), cudaMemcpyHostToDevice));
   return B200_OK;
 }
 
@@ -877,7 +1163,7 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
   const bool loop = c->loop_times > 0;
   if (c->n_layers <= 0 || c->hidden <= 0 || c->vocab <= 0 || c->max_rows <= 0 || c->max_reqs <= 0 || c->max_seqs <= 0 ||
       (c->dtype != B200_DT_BF16 && c->dtype != B200_DT_F32) ||
-      (loop && (c->flags & B200_DEC_DEPTH_AVERAGE)) ||
+      (loop && (c->flags & (B200_DEC_DEPTH_AVERAGE | B200_DEC_SUM_NORM))) || ((c->flags & B200_DEC_DEPTH_AVERAGE) && (c->flags & B200_DEC_SUM_NORM)) ||
       (loop && (c->loop_start < 0 || c->loop_stop > c->n_layers || c->loop_start >= c->loop_stop))) {
     b200_set_error("decoder: invalid configuration");
     return B200_ERR_INVALID_ARGUMENT;
@@ -886,16 +1172,34 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
   auto* m = new b200_decoder();
   m->cfg = *c;
   m->layers.resize(c->n_layers);
-  size_t qw = 0, yw = pad64(c->hidden), aw = 0, fw = 0, plain_w = 0, lat_w = 0, assign = 0, moe_aw = 0;
+  size_t qw = 0, yw = pad64(c->hidden), aw = 0, fw = 0, plain_w = 0, lat_w = 0, assign = 0, moe_aw = 0, ql_w = 0, lru_w = 0, mem_w = 0;
   for (int i = 0; i < c->n_layers; ++i) {
     const b200_decoder_layer& s = layers[i];
     bool good = s.n_heads > 0 && s.key_dim > 0 && s.value_dim > 0 && s.ffn >= 0 && s.window >= 0 && s.n_experts >= 0;
-    if (s.mixer == B200_MIX_ATTENTION) good = good && s.n_kv_heads > 0 && s.n_heads % s.n_kv_heads == 0;
-    else if (s.mixer == B200_MIX_LATENT) good = good && s.kv_rank > 0 && s.rot_dim >= 0 && s.rot_dim % 2 == 0 && (s.rot_dim == 0 || s.rot_base > 0.f) && s.window == 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS));
+    if (s.mixer == B200_MIX_ATTENTION)
+      good = good && s.n_kv_heads > 0 && s.n_heads % s.n_kv_heads == 0 && s.conv_taps >= 0 && s.rot_dim >= 0 && s.rot_dim % 2 == 0 && s.rot_dim <= s.key_dim &&
+             (!(s.flags & B200_DEC_QK_NORM_WEIGHT) || (s.flags & B200_DEC_QK_NORM)) && !((s.flags & B200_DEC_SINK) && (s.flags & B200_DEC_SINK_ONE));
+    else
+      good = good && s.mem_heads == 0 && !(s.flags & (B200_DEC_SINK_ONE | B200_DEC_QK_NORM_WEIGHT));
+    if (s.mixer == B200_MIX_ATTENTION && s.mem_heads != 0) good = good && s.mem_heads > 0 && s.mem_key_dim > 0 && s.mem_value_dim > 0 && s.mem_gate_cap > 0.f;
+    if (s.rot_dim > 0)
+      good = good && s.rot_base > 1.0 && (s.yarn_factor == 0.0 || (s.yarn_factor > 0.0 && s.yarn_original > 0.0 && s.yarn_fast > 0.0 && s.yarn_slow > 0.0));
+    if (s.kv_source != 0) {
+      const int src = s.kv_source - 1;
+      good = good && !loop && s.mixer == B200_MIX_LATENT && src >= 0 && src < i && layers[src].mixer == B200_MIX_LATENT && layers[src].kv_source == 0 &&
+             layers[src].kv_rank == s.kv_rank && layers[src].rot_dim == s.rot_dim;
+    }
+    if (s.mixer == B200_MIX_ATTENTION) {}
+    else if (s.mixer == B200_MIX_LRU) good = good && s.conv_taps > 0 && s.lru_decay > 0.f && s.window == 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS | B200_DEC_SINK));
+    else if (s.mixer == B200_MIX_LATENT) good = good && s.kv_rank > 0 && s.rot_dim >= 0 && s.rot_dim % 2 == 0 && s.q_rank >= 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS));
     else if (s.mixer == B200_MIX_GLA) good = good && s.decay_rank > 0 && s.decay_tau > 0.f && s.window == 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS | B200_DEC_SINK));
     else good = false;
     if (s.n_experts > 0) good = good && s.top_k > 0 && s.top_k <= s.n_experts && s.n_experts <= b200_moe_max_experts() && s.expert_ffn > 0;
+    if (s.n_experts > 0 && s.flags & B200_DEC_ROUTER)
+      good = good && s.top_k <= b200_moe_max_top() && s.n_groups >= 0 && s.n_groups <= b200_moe_max_groups() &&
+             (s.n_groups == 0 || (s.n_experts % s.n_groups == 0 && s.keep_groups > 0 && s.keep_groups <= s.n_groups && s.top_k <= s.keep_groups * (s.n_experts / s.n_groups)));
     if (s.flags & B200_DEC_PARALLEL) good = good && !(s.flags & B200_DEC_POST_NORM);
+    if (c->flags & B200_DEC_SUM_NORM) good = good && !(s.flags & (B200_DEC_POST_NORM | B200_DEC_PARALLEL));
     if (!good) {
       b200_set_error("decoder: layer %d has an invalid shape", i);
       delete m;
@@ -904,18 +1208,33 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
     b200_decoder::Layer& l = m->layers[i];
     l.s = s;
     qw = std::max(qw, (size_t)s.n_heads * (s.mixer == B200_MIX_LATENT ? l.latent_width() : (s.key_dim + 15) / 16 * 16));
-    yw = std::max(yw, (size_t)pad64(l.qkv_n()));
+    yw = std::max({yw, (size_t)pad64(l.qkv_n()), (size_t)pad64(l.router_n()), (size_t)pad64(2 * s.mem_heads), (size_t)(s.q_rank > 0 ? pad64(l.q_n()) : 0)});
     aw = std::max(aw, (size_t)l.out_k());
     fw = std::max(fw, (size_t)pad64(s.ffn));
     if (s.mixer == B200_MIX_LATENT) {
       plain_w = std::max(plain_w, (size_t)s.n_heads * l.plain_stride());
       lat_w = std::max(lat_w, (size_t)s.n_heads * pad64(s.kv_rank));
-      for (size_t t = 0; t < m->rotations.size() && l.rotation < 0; ++t)
-        if (m->rotations[t].base == s.rot_base && m->rotations[t].dims == s.rot_dim) l.rotation = (int)t;
-      if (l.rotation < 0 && s.rot_dim > 0) {
-        l.rotation = (int)m->rotations.size();
-        m->rotations.push_back({s.rot_base, s.rot_dim, nullptr, nullptr});
+      ql_w = std::max(ql_w, (size_t)pad64(s.q_rank));
+    }
+    if (s.mixer == B200_MIX_LRU) {
+      plain_w = std::max(plain_w, (size_t)s.n_heads * l.lru_group());
+      lru_w = std::max(lru_w, (size_t)2 * l.attn_n());
+    }
+    if (s.rot_dim > 0 && (s.mixer == B200_MIX_LATENT || s.mixer == B200_MIX_ATTENTION)) {
+      for (size_t t = 0; t < m->rotations.size() && l.rotation < 0; ++t) {
+        const b200_decoder::Rotation& R = m->rotations[t];
+        if (R.base == s.rot_base && R.dims == s.rot_dim && R.factor == s.yarn_factor && R.original == s.yarn_original && R.fast == s.yarn_fast && R.slow == s.yarn_slow)
+          l.rotation = (int)t;
       }
+      if (l.rotation < 0) {
+        l.rotation = (int)m->rotations.size();
+        m->rotations.push_back({s.rot_base, s.yarn_factor, s.yarn_original, s.yarn_fast, s.yarn_slow, s.rot_dim, nullptr, nullptr});
+      }
+    }
+    if (s.mem_heads > 0) {
+      m->has_gla = true;
+      mem_w = std::max(mem_w, (size_t)s.mem_heads);
+      if (b200_gla_takes_chunks(s.mem_key_dim, s.mem_value_dim, (int)m->elem())) m->gla.need(s.mem_heads, s.mem_key_dim, b200_memory_width(s.mem_value_dim));
     }
     if (s.mixer == B200_MIX_GLA) {
       m->has_gla = true;
@@ -957,10 +1276,21 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
   alloc(&m->last, (size_t)c->max_reqs * m->hp * e);
   alloc(&m->q_plain, R * plain_w * e);
   alloc(&m->lat_out, R * lat_w * e);
+  alloc(&m->q_latent, R * ql_w * e);
+  alloc((void**)&m->lru_gates, R * lru_w * 4);
+  alloc((void**)&m->mem_gates, R * mem_w * sizeof(float4));
   if (c->flags & B200_DEC_DEPTH_AVERAGE) alloc((void**)&m->hist, (size_t)(c->n_layers + 1) * R * c->hidden * 4);
   for (b200_decoder::Rotation& t : m->rotations) {
     std::vector<double> f(t.dims / 2);
-    for (int i = 0; i < t.dims / 2; ++i) f[i] = std::pow((double)t.base, -2.0 * i / t.dims);
+    for (int i = 0; i < t.dims / 2; ++i) f[i] = std::pow(t.base, -2.0 * i / t.dims);
+    if (t.factor > 0) {
+      auto dim_of = [&](double turns) { return t.dims * std::log(t.original / (6.283185307179586476925286766559 * turns)) / (2.0 * std::log(t.base)); };
+      const double lo = std::max(std::floor(dim_of(t.fast)), 0.0), hi = std::min(std::ceil(dim_of(t.slow)), t.dims - 1.0);
+      for (int i = 0; i < t.dims / 2; ++i) {
+        const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+        f[i] = f[i] / t.factor * ramp + f[i] * (1.0 - ramp);
+      }
+    }
     alloc((void**)&t.freq, sizeof(double) * f.size());
     alloc((void**)&t.rows, sizeof(float2) * R * f.size());
     if (st == B200_OK) cudaMemcpy(t.freq, f.data(), sizeof(double) * f.size(), cudaMemcpyHostToDevice);
@@ -969,6 +1299,7 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
     if (!m->f32()) alloc(&m->moe_x, R * assign * m->hp * e);
     alloc(&m->moe_act, R * moe_aw * e);
     alloc(&m->moe_y, R * assign * m->hp * e);
+    alloc((void**)&m->moe_wts, R * assign * 4);
     for (int i : m->moe_layers) {
       const b200_decoder_layer& s = m->layers[i].s;
       const size_t A = R * s.top_k;
@@ -998,7 +1329,7 @@ void b200_decoder_destroy(b200_decoder* m) { delete m; }
 b200_model* b200_decoder_model(b200_decoder* m) { return m; }
 
 b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t which, const void* h_bf16, uint64_t n) {
-  if (which < 0 || which > B200_DEC_DEPTH || (!global_tensor(which) && (layer < 0 || layer >= m->cfg.n_layers))) {
+  if (which < 0 || which > B200_DEC_W_ROUTER || (!global_tensor(which) && (layer < 0 || layer >= m->cfg.n_layers))) {
     b200_set_error("decoder: no tensor %d in layer %d", which, layer);
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -1033,18 +1364,23 @@ b200_status b200_decoder_finalize(b200_decoder* m) {
     b200_decoder::Layer& l = m->layers[i];
     const b200_decoder_layer& s = l.s;
     if ((st = take_weight(m, i, l.projections(), c.hidden, false, &l.wqkv)) != B200_OK) return st;
-    if (l.parallel() && s.ffn > 0) st = take_beside(m, i, {{B200_DEC_W_O, l.attn_n()}, {B200_DEC_W_DOWN, s.ffn}}, c.hidden, &l.wo);
+    std::vector<std::pair<int, int>> beside{{B200_DEC_W_O, l.attn_n()}};
+    if (s.mem_heads > 0) beside.push_back({B200_DEC_W_MEM_O, l.mem_n()});
+    if (l.parallel() && s.ffn > 0) beside.push_back({B200_DEC_W_DOWN, s.ffn});
+    if (beside.size() > 1) st = take_beside(m, i, beside, c.hidden, &l.wo);
     else st = take_weight(m, i, {B200_DEC_W_O}, l.attn_n(), false, &l.wo);
     if (st != B200_OK) return st;
     if ((st = take_norm(m, i, B200_DEC_NORM1, &l.norm1)) != B200_OK) return st;
     if (s.flags & B200_DEC_POST_NORM) if ((st = take_norm(m, i, B200_DEC_POSTNORM1, &l.post1)) != B200_OK) return st;
     if (s.ffn > 0) {
-      if ((st = take_weight(m, i, {B200_DEC_W_GATE, B200_DEC_W_UP}, c.hidden, true, &l.wgu)) != B200_OK) return st;
+      st = l.gelu() ? take_weight(m, i, {B200_DEC_W_UP}, c.hidden, false, &l.wgu) : take_weight(m, i, {B200_DEC_W_GATE, B200_DEC_W_UP}, c.hidden, true, &l.wgu);
+      if (st != B200_OK) return st;
       if (!l.parallel()) if ((st = take_weight(m, i, {B200_DEC_W_DOWN}, s.ffn, false, &l.wdown)) != B200_OK) return st;
     }
     if (s.n_experts > 0) {
       if ((st = take_experts(m, i, l)) != B200_OK) return st;
-      if ((st = upload_table(m, i, l)) != B200_OK) return st;
+      st = s.flags & B200_DEC_ROUTER ? take_weight(m, i, {B200_DEC_W_ROUTER}, c.hidden, false, &l.wrouter) : upload_table(m, i, l);
+      if (st != B200_OK) return st;
     }
     if ((s.ffn > 0 || s.n_experts > 0) && !l.parallel()) {
       if ((st = take_norm(m, i, B200_DEC_NORM2, &l.norm2)) != B200_OK) return st;
@@ -1052,7 +1388,11 @@ b200_status b200_decoder_finalize(b200_decoder* m) {
     }
     if (c.flags & B200_DEC_DEPTH_AVERAGE) if ((st = take_vector(m, i, B200_DEC_DEPTH, &l.depth)) != B200_OK) return st;
     if (s.mixer == B200_MIX_LATENT) {
-      if ((st = take_vector(m, i, B200_DEC_DKV_NORM, &l.dkv_norm)) != B200_OK) return st;
+      if (s.kv_source == 0) if ((st = take_vector(m, i, B200_DEC_DKV_NORM, &l.dkv_norm)) != B200_OK) return st;
+      if (s.q_rank > 0) {
+        if ((st = take_vector(m, i, B200_DEC_DQ_NORM, &l.dq_norm)) != B200_OK) return st;
+        if ((st = take_weight(m, i, {B200_DEC_W_Q}, s.q_rank, false, &l.wuq)) != B200_OK) return st;
+      }
       if ((st = take_stack(m, i, B200_DEC_W_UK, s.n_heads, s.kv_rank, s.key_dim, true, &l.wuk)) != B200_OK) return st;
       if ((st = take_stack(m, i, B200_DEC_W_UV, s.n_heads, s.value_dim, s.kv_rank, false, &l.wuv)) != B200_OK) return st;
     }
@@ -1062,14 +1402,26 @@ b200_status b200_decoder_finalize(b200_decoder* m) {
       if ((st = take_vector(m, i, B200_DEC_HEAD_NORM, &l.head_norm)) != B200_OK) return st;
     }
     if (s.flags & B200_DEC_QKV_BIAS) {
-      std::vector<float> all;
-      for (int w : {B200_DEC_B_Q, B200_DEC_B_K, B200_DEC_B_V}) {
-        std::vector<uint16_t> bits;
-        if ((st = take(m, i, w, &bits)) != B200_OK) return st;
-        for (uint16_t b : bits) all.push_back(bf16_to_f(b));
-      }
-      if ((st = upload_f32(all, &l.bias)) != B200_OK) return st;
+      if ((st = take_vectors(m, i, {B200_DEC_B_Q, B200_DEC_B_K, B200_DEC_B_V}, &l.bias)) != B200_OK) return st;
     }
+    if (s.flags & B200_DEC_QK_NORM_WEIGHT) {
+      if ((st = take_vector(m, i, B200_DEC_Q_NORM, &l.q_norm)) != B200_OK) return st;
+      if ((st = take_vector(m, i, B200_DEC_K_NORM, &l.k_norm)) != B200_OK) return st;
+    }
+    if (s.mixer == B200_MIX_ATTENTION && s.conv_taps > 0)
+      if ((st = take_conv(m, i, {B200_DEC_CONV_Q, B200_DEC_CONV_K, B200_DEC_CONV_V}, s.conv_taps, &l.conv)) != B200_OK) return st;
+    if (s.mem_heads > 0) {
+      if ((st = take_weight(m, i, {B200_DEC_W_MEM_I, B200_DEC_W_MEM_F}, c.hidden, false, &l.wgates)) != B200_OK) return st;
+      if ((st = take_vectors(m, i, {B200_DEC_B_MEM_I, B200_DEC_B_MEM_F}, &l.gate_bias)) != B200_OK) return st;
+      if ((st = take_vector(m, i, B200_DEC_MEM_NORM, &l.mem_norm)) != B200_OK) return st;
+    }
+    if (s.mixer == B200_MIX_LRU) {
+      if ((st = take_vectors(m, i, {B200_DEC_B_LRU_Y, B200_DEC_B_LRU_X, B200_DEC_B_LRU_R, B200_DEC_B_LRU_I}, &l.lru_bias)) != B200_OK) return st;
+      if ((st = take_conv(m, i, {B200_DEC_LRU_CONV}, s.conv_taps, &l.conv)) != B200_OK) return st;
+      if ((st = take_vector(m, i, B200_DEC_B_LRU_CONV, &l.conv_bias)) != B200_OK) return st;
+      if ((st = take_lru(m, i, l)) != B200_OK) return st;
+    }
+    if (s.flags & B200_DEC_SINK_ONE) if ((st = upload_f32(std::vector<float>(s.n_heads, 0.f), &l.sinks)) != B200_OK) return st;
     if (s.flags & B200_DEC_SINK) if ((st = take_vector(m, i, B200_DEC_W_SINK, &l.sinks, kLog2e)) != B200_OK) return st;
     if ((st = make_slopes(l)) != B200_OK) return st;
   }
@@ -1102,7 +1454,7 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
     if ((st = upload_f32(ones, &l.norm1)) != B200_OK) return st;
     if (s.flags & B200_DEC_POST_NORM) if ((st = upload_f32(ones, &l.post1)) != B200_OK) return st;
     if (s.ffn > 0) {
-      if ((st = weight(2 * s.ffn, c.hidden, 16 * i + 3, &l.wgu)) != B200_OK) return st;
+      if ((st = weight((l.gelu() ? 1 : 2) * s.ffn, c.hidden, 16 * i + 3, &l.wgu)) != B200_OK) return st;
       if (!l.parallel()) if ((st = weight(c.hidden, s.ffn, 16 * i + 4, &l.wdown)) != B200_OK) return st;
     }
     if ((s.ffn > 0 || s.n_experts > 0) && !l.parallel()) {
@@ -1110,8 +1462,11 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
       if (s.flags & B200_DEC_POST_NORM) if ((st = upload_f32(ones, &l.post2)) != B200_OK) return st;
     }
     if (s.n_experts > 0) {
-      if ((st = stack(s.n_experts, 2 * s.expert_ffn, c.hidden, 16 * i + 5, &l.we_gu)) != B200_OK) return st;
+      if ((st = stack(s.n_experts, (l.gelu() ? 1 : 2) * s.expert_ffn, c.hidden, 16 * i + 5, &l.we_gu)) != B200_OK) return st;
       if ((st = stack(s.n_experts, c.hidden, s.expert_ffn, 16 * i + 6, &l.we_down)) != B200_OK) return st;
+      if (s.flags & B200_DEC_ROUTER) {
+        if ((st = weight(pad64(s.n_experts), c.hidden, 16 * i + 9, &l.wrouter)) != B200_OK) return st;
+      } else {
       l.h_table.resize((size_t)c.vocab * s.top_k);
       uint32_t x = seed * 747796405u + i;
       for (int v = 0; v < c.vocab; ++v) {  // experts an odd step apart from a random one: all different
@@ -1119,6 +1474,7 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
         for (int j = 0; j < s.top_k; ++j) l.h_table[(size_t)v * s.top_k + j] = (int)(((x >> 8) + (uint32_t)j) % (uint32_t)s.n_experts);
       }
       if ((st = upload_table(m, i, l)) != B200_OK) return st;
+      }
     }
     if (c.flags & B200_DEC_DEPTH_AVERAGE) {
       std::vector<float> d(i + 2, 0.1f);
@@ -1126,7 +1482,11 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
       if ((st = upload_f32(d, &l.depth)) != B200_OK) return st;
     }
     if (s.mixer == B200_MIX_LATENT) {
-      if ((st = upload_f32(std::vector<float>(s.kv_rank, 1.f), &l.dkv_norm)) != B200_OK) return st;
+      if (s.kv_source == 0) if ((st = upload_f32(std::vector<float>(s.kv_rank, 1.f), &l.dkv_norm)) != B200_OK) return st;
+      if (s.q_rank > 0) {
+        if ((st = upload_f32(std::vector<float>(s.q_rank, 1.f), &l.dq_norm)) != B200_OK) return st;
+        if ((st = weight(pad64(l.q_n()), s.q_rank, 16 * i + 10, &l.wuq)) != B200_OK) return st;
+      }
       if ((st = stack(s.n_heads, s.kv_rank, l.plain_stride(), 16 * i + 7, &l.wuk)) != B200_OK) return st;
       if ((st = stack(s.n_heads, s.value_dim, pad64(s.kv_rank), 16 * i + 8, &l.wuv)) != B200_OK) return st;
     }
@@ -1137,6 +1497,21 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
     }
     if (s.flags & B200_DEC_QKV_BIAS) if ((st = upload_f32(std::vector<float>(l.qkv_n(), 0.01f), &l.bias)) != B200_OK) return st;
     if (s.flags & B200_DEC_SINK) if ((st = upload_f32(std::vector<float>(s.n_heads, 0.5f), &l.sinks)) != B200_OK) return st;
+    auto fill = [&](size_t n, float v, float** out) { return upload_f32(std::vector<float>(n, v), out); };
+    if (s.flags & B200_DEC_SINK_ONE) if ((st = fill(s.n_heads, 0.f, &l.sinks)) != B200_OK) return st;
+    if (s.flags & B200_DEC_QK_NORM_WEIGHT)
+      if ((st = fill(s.key_dim, 1.f, &l.q_norm)) != B200_OK || (st = fill(s.key_dim, 1.f, &l.k_norm)) != B200_OK) return st;
+    if (s.mixer == B200_MIX_ATTENTION && s.conv_taps > 0) if ((st = fill((size_t)l.attention_n() * s.conv_taps, 0.5f, &l.conv)) != B200_OK) return st;
+    if (s.mem_heads > 0) {
+      if ((st = weight(pad64(2 * s.mem_heads), c.hidden, 16 * i + 11, &l.wgates)) != B200_OK) return st;
+      if ((st = fill(2 * s.mem_heads, 1.f, &l.gate_bias)) != B200_OK || (st = fill(l.mem_n(), 1.f, &l.mem_norm)) != B200_OK) return st;
+    }
+    if (s.mixer == B200_MIX_LRU) {
+      if ((st = stack(s.n_heads, 2 * s.value_dim, l.lru_group(), 16 * i + 12, &l.wgates)) != B200_OK) return st;
+      if ((st = fill(4 * l.attn_n(), 0.1f, &l.lru_bias)) != B200_OK || (st = fill((size_t)l.attn_n() * s.conv_taps, 0.5f, &l.conv)) != B200_OK ||
+          (st = fill(l.attn_n(), 0.f, &l.conv_bias)) != B200_OK || (st = fill(l.attn_n(), 0.5f, &l.lru_rate)) != B200_OK)
+        return st;
+    }
     if ((st = make_slopes(l)) != B200_OK) return st;
   }
   if ((st = upload_moe(m)) != B200_OK) return st;

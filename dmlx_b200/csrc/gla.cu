@@ -171,6 +171,66 @@ __global__ void __launch_bounds__(256, 3) gla_step_kernel(Gla a) {
   }
 }
 
+// ---- matrix memory: gates -----------------------------------------------------------------------------------------------
+struct GateArgs {
+  KvDev d;
+  MemoryGates g;
+  float* state;
+  int rec_elems;
+  const int *cu, *row_seq, *pos;
+};
+
+// One CTA per (request, head).  m_t = max(m_(t-1) + f_t, i_t) is a scan: the pair (F, M) stands for m -> max(m + F, M).
+template <typename T>
+__global__ void __launch_bounds__(256) memory_gates_kernel(GateArgs a) {
+  __shared__ float2 total[8];
+  __shared__ float s_m[257];
+  const int req = blockIdx.x, head = blockIdx.y, H = a.g.heads, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
+  const int r0 = a.cu[req], count = a.cu[req + 1] - r0;
+  if (count <= 0 || a.d.state[ST_ERR] != 0) return;
+  const int slot = a.row_seq[r0];
+  if (slot < 0 || slot >= a.d.max_seqs) return;
+  float* m_at = a.state + (size_t)slot * a.rec_elems + a.g.m_off + head;
+  float m_in = a.pos[r0] == 0 ? 0.f : *m_at;
+  auto capped = [&](int row, int col) {
+    const float z = mat_value<T, 1>(a.g.src, row, col).v[0] + a.g.bias[col];
+    return a.g.cap * tanhf(z / a.g.cap);
+  };
+  for (int base = 0; base < count; base += blockDim.x) {
+    const int row = r0 + base + tid;
+    const bool on = base + tid < count;
+    float in = -INFINITY, forget = 0.f;
+    if (on) {
+      in = capped(row, head);
+      forget = log_sigmoid(capped(row, H + head));
+    }
+    float F = forget, M = in;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
+      if (lane >= o) {
+        M = fmaxf(Mp + F, M);
+        F += Fp;
+      }
+    }
+    if (lane == 31) total[warp] = make_float2(F, M);
+    __syncthreads();
+    float m_warp = m_in, m_end = m_in;
+    for (int w = 0; w < n_warps; ++w) {
+      if (w == warp) m_warp = m_end;
+      m_end = fmaxf(m_end + total[w].x, total[w].y);
+    }
+    const float m = fmaxf(m_warp + F, M);
+    if (tid == 0) s_m[0] = m_in;
+    s_m[tid + 1] = m;
+    __syncthreads();
+    if (on) a.g.out[(size_t)row * H + head] = make_float4(forget + s_m[tid] - m, expf(in - m), expf(-m), 0.f);
+    m_in = m_end;
+    __syncthreads();
+  }
+  if (tid == 0) *m_at = m_in;
+}
+
 // ---- chunks: plan ------------------------------------------------------------------------------------------------
 // One CTA: the chunks of every portion that goes chunk by chunk, and where each request's start.
 __global__ void __launch_bounds__(1024) gla_plan_kernel(const int* __restrict__ cu, int n_req, int max_chunks, int4* __restrict__ plan,
@@ -550,6 +610,129 @@ __global__ void __launch_bounds__(256) gla_out_kernel(Gla a) {
   }
 }
 
+// ---- chunks of a matrix memory -----------------------------------------------------------------------------------------
+// One decay for all channels: the weights are (q_i . k_j) e^(L_i - L_j) w_j, so the exponentials stay out of the product and decays of
+// any strength take this route.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) memory_chunk_kernel(Gla a) {
+  extern __shared__ __align__(16) float sh[];
+  __shared__ float s_L[kC], s_w[kC];
+  const int chunk = blockIdx.x, head = blockIdx.y;
+  if (chunk >= a.first_chunk[a.n_req] || a.d.state[ST_ERR] != 0) return;
+  const int4 it = a.plan[chunk];
+  const int dk = a.dk, dkp = a.dkp, ldr = dkp + 8, n = it.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  float *q = sh, *k = q + kC * ldr;
+  unsigned char* out = a.chunks + ((size_t)chunk * a.heads + head) * a.chunk_bytes;
+  if (warp == 0) {
+    float4 g{};
+    if (lane < n) g = a.gates[(size_t)(it.x + lane) * a.heads + head];
+    float L = g.x;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float x = __shfl_up_sync(0xffffffffu, L, o);
+      if (lane >= o) L += x;
+    }
+    s_L[lane] = L;
+    s_w[lane] = g.y;
+  }
+  const int groups = dkp / VEC;
+  for (int i = tid; i < kC * groups; i += 256) {
+    const int t = i / groups, c = (i - t * groups) * VEC;
+    Vec<VEC> x{}, y{};
+    if (t < n && c < dk) {
+      x = mat_value<T, VEC>(a.src, it.x + t, a.col0 + head * dk + c);
+      y = mat_value<T, VEC>(a.src, it.x + t, a.col_k() + head * dk + c);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x.v[e] *= a.q_scale;
+    store_vec<VEC>(q + t * ldr + c, x);
+    store_vec<VEC>(k + t * ldr + c, y);
+  }
+  constexpr int kPer = kScanCols / VEC;
+  for (int i = tid; i < a.n_slices * kC * kPer; i += 256) {
+    const int s = i / (kC * kPer), rest = i - s * kC * kPer, t = rest / kPer, c = (rest - t * kPer) * VEC;
+    Vec<VEC> v{};
+    if (t < n) v = memory_value<T, VEC>(a, it.x + t, head, s * kScanCols + c);
+    unsigned char* dst = a.values + ((size_t)chunk * a.heads + head) * a.v_bytes + (size_t)s * kVSlice + (size_t)t * kVRow + c * 2;
+    store_vec<VEC>(reinterpret_cast<__nv_bfloat16*>(dst), v);
+  }
+  __syncthreads();
+  const float end = s_L[kC - 1];
+  for (int c = tid; c < dkp; c += 256) reinterpret_cast<float*>(out + off_decay(dkp))[c] = expf(end);
+  for (int i = tid; i < kC * (dkp / 2); i += 256) {
+    const int t = i / (dkp / 2), c = 2 * (i - t * (dkp / 2));
+    const float fq = expf(s_L[t]), fk = s_w[t] * expf(end - s_L[t]);
+    const float2 qt = *reinterpret_cast<const float2*>(&q[t * ldr + c]), kt = *reinterpret_cast<const float2*>(&k[t * ldr + c]);
+    uint32_t hi, lo;
+    split_bf16(qt.x * fq, qt.y * fq, hi, lo);
+    unsigned char* at = out + (size_t)t * qk_row(dkp) + c * 2;
+    *reinterpret_cast<uint32_t*>(at + off_part(dkp, 0)) = hi;
+    *reinterpret_cast<uint32_t*>(at + off_part(dkp, 1)) = lo;
+    split_bf16(kt.x * fk, kt.y * fk, hi, lo);
+    *reinterpret_cast<uint32_t*>(at + off_part(dkp, 2)) = hi;
+    *reinterpret_cast<uint32_t*>(at + off_part(dkp, 3)) = lo;
+  }
+  // 16 x 8 tiles, as in gla_chunk_kernel
+  unsigned char *ahi = out + off_a(dkp, 0), *alo = out + off_a(dkp, 1);
+  const int g = lane >> 2, t = lane & 3, I = warp >= 2 && warp < 6 ? 1 : 0, nt = warp < 2 ? warp : (warp < 6 ? warp - 2 : warp - 4);
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  if (warp < 6) {
+    const int i0 = 16 * I + g, i1 = i0 + 8, j = 8 * nt + g;
+    auto at2 = [&](const float* p) { return *reinterpret_cast<const float2*>(p); };
+    for (int ks = 0; ks < dkp / 16; ++ks) {
+      uint32_t qh[4], ql[4], kh[2], kl[2];
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int c = ks * 16 + h * 8 + 2 * t;
+        const float2 q0 = at2(&q[i0 * ldr + c]), q1 = at2(&q[i1 * ldr + c]), kj = at2(&k[j * ldr + c]);
+        split_bf16(q0.x, q0.y, qh[2 * h], ql[2 * h]);
+        split_bf16(q1.x, q1.y, qh[2 * h + 1], ql[2 * h + 1]);
+        split_bf16(kj.x, kj.y, kh[h], kl[h]);
+      }
+      mma16816(acc, qh, kh[0], kh[1]);
+      mma16816(acc, qh, kl[0], kl[1]);
+      mma16816(acc, ql, kh[0], kh[1]);
+    }
+  }
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int i = 16 * I + g + 8 * h, j = 8 * nt + 2 * t;
+    const float x = j <= i ? acc[2 * h] * expf(s_L[i] - s_L[j]) * s_w[j] : 0.f;
+    const float y = j + 1 <= i ? acc[2 * h + 1] * expf(s_L[i] - s_L[j + 1]) * s_w[j + 1] : 0.f;
+    uint32_t hi, lo;
+    split_bf16(x, y, hi, lo);
+    *reinterpret_cast<uint32_t*>(ahi + i * kARow + j * 2) = hi;
+    *reinterpret_cast<uint32_t*>(alo + i * kARow + j * 2) = lo;
+  }
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) memory_out_kernel(Gla a) {
+  const int chunk = blockIdx.x, head = blockIdx.y, lane = threadIdx.x & 31;
+  if (chunk >= a.first_chunk[a.n_req] || a.d.state[ST_ERR] != 0) return;
+  const int4 it = a.plan[chunk];
+  for (int i = threadIdx.x >> 5; i < it.y; i += 8) {
+    const int row = it.x + i;
+    const float* o = a.o + ((size_t)row * a.heads + head) * a.dvs;
+    const float inv = 1.0f / (fmaxf(fabsf(o[a.dv]), a.gates[(size_t)row * a.heads + head].z) + a.den_eps);
+    float ss = 0.f;
+    for (int c = lane * VEC; c < a.dv; c += 32 * VEC) {
+      const Vec<VEC> x = load_vec<VEC>(o + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += x.v[e] * inv * (x.v[e] * inv);
+    }
+    const float r = inv / sqrtf(warp_sum(ss) / (float)a.dv + a.eps) * a.out_scale;
+    T* dst = (T*)a.out + (size_t)row * a.out_stride + (size_t)head * a.dv;
+    for (int c = lane * VEC; c < a.dv; c += 32 * VEC) {
+      Vec<VEC> x = load_vec<VEC>(o + c);
+      const Vec<VEC> w = load_vec<VEC>(a.norm + head * a.dv + c), g = mat_value<T, VEC>(a.src, row, a.col_g() + head * a.dv + c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x.v[e] *= r * w.v[e] * sigmoid(g.v[e]);
+      store_vec<VEC>(dst + c, x);
+    }
+  }
+}
+
 int pad_channels(int dk) { return (dk + 31) / 32 * 32; }
 int slices_of(int dv) { return (dv + kScanCols - 1) / kScanCols; }
 
@@ -597,9 +780,27 @@ b200_status b200_gla_plan(GlaScratch& g, const int32_t* d_cu, int n_req, int tot
   return B200_OK;
 }
 
+b200_status b200_memory_gates(b200_kv* kv, const MemoryGates& g, const int32_t* d_cu, const int32_t* d_row_seq, const int32_t* d_pos, int n_req,
+                              int total_rows, void* stream) {
+  if (g.layer < 0 || g.layer >= kv->cfg.n_layers || kv->lay[g.layer].rec_elems < g.m_off + g.heads) {
+    b200_set_error("matrix memory: layer %d of the pool has no room for %d maxima", g.layer, g.heads);
+    return B200_ERR_INVALID_ARGUMENT;
+  }
+  if (n_req <= 0 || total_rows <= 0) return B200_OK;
+  GateArgs a;
+  a.d = kv->dev; a.g = g; a.state = kv->dev.rec_pool + kv->lay[g.layer].rec_off; a.rec_elems = kv->lay[g.layer].rec_elems;
+  a.cu = d_cu; a.row_seq = d_row_seq; a.pos = d_pos;
+  auto* kernel = kv->dev.elem_bytes == 4 ? memory_gates_kernel<float> : memory_gates_kernel<__nv_bfloat16>;
+  kernel<<<dim3(n_req, g.heads), total_rows > 4 * n_req ? 256 : 32, 0, (cudaStream_t)stream>>>(a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
+
 b200_status b200_gla_run(b200_kv* kv, const GlaScratch& g, const GlaCall& c, const int32_t* d_cu, const int32_t* d_row_seq,
                          const int32_t* d_pos, int n_req, int total_rows, bool chunked, void* stream) {
-  if (c.layer < 0 || c.layer >= kv->cfg.n_layers || kv->lay[c.layer].rec_elems != c.heads * c.dk * c.dv) {
+  const bool mem = c.gates != nullptr;
+  if (c.layer < 0 || c.layer >= kv->cfg.n_layers ||
+      (mem ? kv->lay[c.layer].rec_elems < b200_memory_elems(c.heads, c.dk, c.dv) : kv->lay[c.layer].rec_elems != c.heads * c.dk * c.dv)) {
     b200_set_error("gla: layer %d of the pool has no state of %d x %d x %d", c.layer, c.heads, c.dk, c.dv);
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -611,43 +812,52 @@ b200_status b200_gla_run(b200_kv* kv, const GlaScratch& g, const GlaCall& c, con
   a.state = kv->dev.rec_pool + kv->lay[c.layer].rec_off;
   a.rec_elems = kv->lay[c.layer].rec_elems;
   a.heads = c.heads; a.dk = c.dk; a.dv = c.dv; a.rank = c.rank; a.dkp = pad_channels(c.dk);
+  a.dva = mem ? c.dv + 1 : c.dv; a.dvs = mem ? b200_memory_width(c.dv) : c.dv;
+  a.gates = c.gates; a.col0 = c.col0; a.den_eps = c.den_eps; a.out_scale = c.out_scale;
   a.src = c.src; a.a2 = c.a2; a.a2_bias = c.a2_bias; a.norm = c.norm; a.q_scale = c.q_scale; a.inv_tau = c.inv_tau; a.eps = c.eps;
   a.out = c.out; a.out_stride = c.out_stride; a.cu = d_cu; a.row_seq = d_row_seq; a.pos = d_pos; a.n_req = n_req; a.total_rows = total_rows;
   a.chunks = g.chunks; a.values = g.values; a.o = g.o; a.plan = g.plan; a.first_chunk = g.first_chunk;
   a.chunk_bytes = chunk_size(a.dkp);
-  a.n_slices = slices_of(c.dv);
+  a.n_slices = slices_of(a.dva);
   a.v_bytes = a.n_slices * kVSlice;
   a.stages = 0;
   // portions that are longer than the step kernel's limit exist only if some request has more than one row
   a.chunked = chunked && b200_gla_takes_chunks(c.dk, c.dv, kv->dev.elem_bytes);
-  const bool v4 = c.dk % 4 == 0 && c.dv % 4 == 0 && (c.src.ws || c.src.y_stride % 4 == 0);
+  const bool v4 = c.dk % 4 == 0 && c.dv % 4 == 0 && c.col0 % 4 == 0 && (c.src.ws || c.src.y_stride % 4 == 0);
   {
-    a.cols = std::min(v4 ? c.dv / 4 : c.dv, 256);
+    a.cols = std::min(v4 ? a.dvs / 4 : a.dva, 256);
     a.groups = std::max(1, std::min(256 / a.cols, (c.dk + 7) / 8));
-    const size_t smem = sizeof(float) * (3 * (size_t)c.dk + c.rank + (size_t)a.groups * c.dv);
+    const size_t smem = sizeof(float) * (3 * (size_t)c.dk + (mem ? 0 : c.rank) + (size_t)a.groups * a.dvs);
     if (smem > 200 * 1024) { b200_set_error("gla: head widths %d / %d are too large", c.dk, c.dv); return B200_ERR_UNSUPPORTED; }
-    auto* kernel = f32 ? (v4 ? gla_step_kernel<float, 4> : gla_step_kernel<float, 1>) : (v4 ? gla_step_kernel<__nv_bfloat16, 4> : gla_step_kernel<__nv_bfloat16, 1>);
+    auto* kernel = f32 ? (v4 ? gla_step_kernel<float, 4, false> : gla_step_kernel<float, 1, false>)
+                       : (v4 ? gla_step_kernel<__nv_bfloat16, 4, false> : gla_step_kernel<__nv_bfloat16, 1, false>);
+    if (mem) kernel = f32 ? (v4 ? gla_step_kernel<float, 4, true> : gla_step_kernel<float, 1, true>)
+                          : (v4 ? gla_step_kernel<__nv_bfloat16, 4, true> : gla_step_kernel<__nv_bfloat16, 1, true>);
     if (smem > 48 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     kernel<<<dim3(n_req, c.heads), (a.cols * a.groups + 31) / 32 * 32, smem, s>>>(a);
     B200_LAUNCH_CHECK();
   }
   if (!a.chunked || total_rows <= n_req) return B200_OK;
   const int chunks = std::min(total_rows / kC + n_req, g.max_chunks);
-  const size_t smem = sizeof(float) * (3 * (size_t)kC * (a.dkp + 8) + (size_t)kC * c.rank);
+  const size_t smem = sizeof(float) * ((mem ? 2 : 3) * (size_t)kC * (a.dkp + 8) + (mem ? 0 : (size_t)kC * c.rank));
   if (smem > 220 * 1024) { b200_set_error("gla: a decay projection of inner width %d is too large", c.rank); return B200_ERR_UNSUPPORTED; }
   static bool configured = false;
   if (!configured) {
     B200_CUDA_TRY((cudaFuncSetAttribute(gla_chunk_kernel<__nv_bfloat16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
     B200_CUDA_TRY((cudaFuncSetAttribute(gla_chunk_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
+    B200_CUDA_TRY((cudaFuncSetAttribute(memory_chunk_kernel<__nv_bfloat16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
+    B200_CUDA_TRY((cudaFuncSetAttribute(memory_chunk_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
     configured = true;
   }
   const bool wide = v4 && c.out_stride % 4 == 0;
-  auto* chunk_kernel = wide ? gla_chunk_kernel<__nv_bfloat16, 4> : gla_chunk_kernel<__nv_bfloat16, 1>;
+  auto* chunk_kernel = mem ? (wide ? memory_chunk_kernel<__nv_bfloat16, 4> : memory_chunk_kernel<__nv_bfloat16, 1>)
+                           : (wide ? gla_chunk_kernel<__nv_bfloat16, 4> : gla_chunk_kernel<__nv_bfloat16, 1>);
   chunk_kernel<<<dim3(chunks, c.heads), 256, smem, s>>>(a);
   B200_LAUNCH_CHECK();
   b200_status st = a.dkp <= 32 ? launch_scan<4>(a, n_req, s) : (a.dkp <= 64 ? launch_scan<8>(a, n_req, s) : (a.dkp <= 128 ? launch_scan<16>(a, n_req, s) : launch_scan<32>(a, n_req, s)));
   if (st != B200_OK) return st;
-  auto* out_kernel = wide ? gla_out_kernel<__nv_bfloat16, 4> : gla_out_kernel<__nv_bfloat16, 1>;
+  auto* out_kernel = mem ? (wide ? memory_out_kernel<__nv_bfloat16, 4> : memory_out_kernel<__nv_bfloat16, 1>)
+                         : (wide ? gla_out_kernel<__nv_bfloat16, 4> : gla_out_kernel<__nv_bfloat16, 1>);
   out_kernel<<<dim3(chunks, c.heads), 256, 0, s>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;

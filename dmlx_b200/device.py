@@ -582,11 +582,14 @@ class LlamaModel(Model):
 
 DT_BF16, DT_F32 = 0, 1
 DEC_QKV_BIAS, DEC_QK_NORM, DEC_DISTANCE_BIAS, DEC_SINK, DEC_POST_NORM, DEC_PARALLEL = 1, 2, 4, 8, 16, 32
-DEC_SCALAR_NORM, DEC_DEPTH_AVERAGE = 1, 2  # of the whole stack
-MIX_ATTENTION, MIX_LATENT, MIX_GLA = 0, 1, 2
+DEC_SINK_ONE, DEC_QK_NORM_WEIGHT, DEC_ROT_HALVES, DEC_FF_GELU, DEC_ROUTER = 64, 128, 256, 512, 1024
+DEC_SCALAR_NORM, DEC_DEPTH_AVERAGE, DEC_SUM_NORM, DEC_NORM_OFFSET = 1, 2, 4, 8  # of the whole stack
+MIX_ATTENTION, MIX_LATENT, MIX_GLA, MIX_LRU = 0, 1, 2, 3
 DEC_TENSORS = ("q", "k", "v", "o", "gate", "up", "down", "head", "loop_in", "embed", "q_bias", "k_bias", "v_bias", "sink", "norm1", "norm2",
                "postnorm1", "postnorm2", "final_norm", "dkv", "dkv_norm", "uk", "uv", "out_gate", "a1", "a2", "a2_bias", "head_norm",
-               "expert_gate", "expert_up", "expert_down", "depth")
+               "expert_gate", "expert_up", "expert_down", "depth", "dq", "dq_norm", "q_norm", "k_norm", "q_conv", "k_conv", "v_conv",
+               "mem_q", "mem_k", "mem_v", "mem_g", "mem_o", "mem_i", "mem_f", "mem_i_bias", "mem_f_bias", "mem_norm", "lru_y", "lru_y_bias", "lru_x",
+               "lru_x_bias", "lru_conv", "lru_conv_bias", "lru_r", "lru_r_bias", "lru_i", "lru_i_bias", "lru_lambda", "router")
 
 
 class DecoderModel(Model):
@@ -594,10 +597,11 @@ class DecoderModel(Model):
     b200_decoder_layer; `loop` is (start, stop, times) or None."""
 
     def __init__(self, hidden: int, vocab: int, layers: Sequence[dict], norm_eps: float, embed_scale: float = 1.0, loop=None,
-                 dtype: int = DT_BF16, max_rows: int = 2048, max_reqs: int = 64, max_seqs: int = 64, logit_scale: float = 1.0, flags: int = 0):
+                 dtype: int = DT_BF16, max_rows: int = 2048, max_reqs: int = 64, max_seqs: int = 64, logit_scale: float = 1.0, flags: int = 0,
+                 residual_scale: float = 1.0):
         start, stop, times = loop if loop else (0, 0, 0)
         self.cfg = _lib.DecoderConfig(len(layers), hidden, vocab, start, stop, times, dtype, max_rows, max_reqs, max_seqs, norm_eps,
-                                      embed_scale, logit_scale, flags)
+                                      embed_scale, logit_scale, flags, residual_scale)
         arr = (_lib.DecoderLayer * max(len(layers), 1))(*[_lib.DecoderLayer(**l) for l in layers])
         h = C.c_void_p()
         _lib.check(lib.b200_decoder_create(C.byref(self.cfg), arr, C.byref(h)))

@@ -594,9 +594,13 @@ b200_status b200_model_logits(b200_model* m, int32_t first, int32_t n, float* h_
  *   x = embed[token] * embed_scale, kept in f32 between the layers;
  *   x += postnorm1(mixer(norm1(x))); x += postnorm2(ff(h)), h = norm2(x);
  *   with B200_DEC_PARALLEL instead x += mixer(h) + ff(h), h = norm1(x);
- *   mixer: grouped-query attention, latent attention or gated linear attention (B200_MIX_*);
- *   ff(h) = W_down(silu(W_gate h) * W_up h) of width ffn, plus 1 / top_k times the same of each expert the token's id has in
- *   the layer's table;
+ *   with B200_DEC_SUM_NORM instead x = norm1(residual_scale * x + mixer(x)), x = norm2(residual_scale * x + ff(x));
+ *   mixer: one of B200_MIX_*; beside attention a matrix memory may run on the same h (mem_heads > 0), the two are added with the factors
+ *   mix_scale and mem_scale;
+ *   ff(h) = W_down(silu(W_gate h) * W_up h) of width ffn (B200_DEC_FF_GELU: W_down gelu(W_up h)), plus the same of each of the top_k
+ *   experts of a token: 1 / top_k each for those the token's id has in the layer's table, or (B200_DEC_ROUTER) the best of softmax(W_router h)
+ *   with their scores, which are divided by their sum; only the keep_groups of n_groups groups of neighbouring experts with the largest
+ *   best score take part;
  *   with B200_DEC_DEPTH_AVERAGE what follows layer i is sum_j depth[j] X_j over the embedding output X_0 and the results X_1 ..
  *   X_(i+1) of the layers so far;
  *   layers loop_start .. loop_stop-1 run loop_times times with the same weights, every pass with cache layers of its own,
@@ -612,17 +616,33 @@ enum {
   B200_DEC_SINK = 8,           /* learned sink per query head in the softmax's denominator */
   B200_DEC_POST_NORM = 16,     /* RMSNorm on each sublayer's output before the residual add */
   B200_DEC_PARALLEL = 32,      /* mixer and feed-forward read the same norm and are added together */
+  B200_DEC_SINK_ONE = 64,      /* one more in the softmax's denominator: a sink of score 0 in every head */
+  B200_DEC_QK_NORM_WEIGHT = 128, /* B200_DEC_QK_NORM with a weight per dimension, shared by the heads */
+  B200_DEC_ROT_HALVES = 256,   /* rotated pairs are (i, i + rot_dim / 2) instead of (2i, 2i + 1) */
+  B200_DEC_FF_GELU = 512,      /* feed-forward and experts: exact GELU, no gate */
+  B200_DEC_ROUTER = 1024,      /* experts by a router instead of a table */
   /* of the whole stack (b200_decoder_config.flags) */
   B200_DEC_SCALAR_NORM = 1,    /* a norm's weight is one number for all coordinates */
-  B200_DEC_DEPTH_AVERAGE = 2   /* weighted average over depth after every layer */
+  B200_DEC_DEPTH_AVERAGE = 2,  /* weighted average over depth after every layer */
+  B200_DEC_SUM_NORM = 4,       /* norms behind the residual sum; the sublayers read the residual itself */
+  B200_DEC_NORM_OFFSET = 8     /* norm weights are stored around zero: 1 + w */
 };
-/* B200_MIX_ATTENTION: softmax attention, keys and values per kv head.
+/* B200_MIX_ATTENTION: softmax attention, keys and values per kv head.  With conv_taps a causal convolution per channel stands directly
+ *   behind the q, k and v projections; with rot_dim the first rot_dim dimensions of q and k are rotated, behind their norm.
  * B200_MIX_LATENT: keys and values of all heads come from one latent of kv_rank numbers per token, c = norm(W_dkv h); per head
  *   the key is W_uk c (key_dim wide) beside rot_dim rotated numbers shared by all heads, the value W_uv c (value_dim).  Cached are
- *   c and the rotated part.  Rotation: pairs (2i, 2i+1), angle position * rot_base^(-2i / rot_dim).
+ *   c and the rotated part.  Rotation: pairs (2i, 2i+1), angle position * rot_base^(-2i / rot_dim).  With q_rank the queries come from a
+ *   latent of their own, W_q norm(W_dq h).  With kv_source = 1 + j the layer has no W_dkv and reads what layer j < this one caches.
  * B200_MIX_GLA: state S [key_dim][value_dim] per head, S <- diag(alpha) S + k v^T, o = S^T q key_dim^(-1/2), alpha =
- *   sigmoid(W_a2 W_a1 h + b)^(1 / decay_tau) with decay_rank rows in W_a1; rms_norm(o) * w * silu(W_g h). */
-enum { B200_MIX_ATTENTION = 0, B200_MIX_LATENT = 1, B200_MIX_GLA = 2 };
+ *   sigmoid(W_a2 W_a1 h + b)^(1 / decay_tau) with decay_rank rows in W_a1; rms_norm(o) * w * silu(W_g h).
+ * B200_MIX_LRU: n_heads blocks of value_dim channels; y = gelu_tanh(W_y h + b), u = conv(W_x h + b) + b of conv_taps taps; per block
+ *   r = sigmoid(R u + b), i = sigmoid(I u + b); a = exp(-lru_decay r softplus(lam)), S <- a S + sqrt(1 - a^2) i u; the output is S * y.
+ * Matrix memory (mem_heads of mem_key_dim x mem_value_dim): log gates i = cap tanh((W_i h + b) / cap) and f = log sigmoid(cap tanh((W_f h + b)
+ *   / cap)), cap = mem_gate_cap; m' = max(f + m, i); S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone; o = S^T q / (max(|n . q|,
+ *   e^-m') + 1e-6), q scaled by mem_key_dim^(-1/2); rms_norm(o) * w * sigmoid(W_g h).
+ * YaRN (yarn_factor > 0): with dim(t) = rot_dim ln(yarn_original / (2 pi t)) / (2 ln rot_base), the frequencies of the pairs from
+ *   dim(yarn_fast) to dim(yarn_slow) go over to 1 / yarn_factor of themselves; cosine and sine are multiplied by 0.1 ln yarn_factor + 1. */
+enum { B200_MIX_ATTENTION = 0, B200_MIX_LATENT = 1, B200_MIX_GLA = 2, B200_MIX_LRU = 3 };
 typedef struct b200_decoder_layer {
   int32_t n_heads, n_kv_heads, key_dim, value_dim;
   int32_t window; /* position i sees j with 0 <= i - j < window; 0 = the whole context */
@@ -630,11 +650,18 @@ typedef struct b200_decoder_layer {
   int32_t flags;  /* B200_DEC_* */
   float scale;    /* score = (q . k) * scale */
   int32_t mixer;  /* B200_MIX_* */
-  int32_t kv_rank, rot_dim;                 /* latent attention */
-  float rot_base;
+  int32_t kv_rank, rot_dim;                 /* latent attention; rot_dim also of attention */
+  double rot_base;
   int32_t decay_rank;                       /* gated linear attention */
   float decay_tau;
-  int32_t n_experts, top_k, expert_ffn;     /* experts by token id (b200_decoder_set_table); n_experts 0 = none */
+  int32_t n_experts, top_k, expert_ffn;     /* experts by token id (b200_decoder_set_table) or router; n_experts 0 = none */
+  int32_t n_groups, keep_groups;            /* of a router's experts; 0 = one group */
+  int32_t q_rank, kv_source;                /* latent attention; 0 = none, its own */
+  double yarn_factor, yarn_original, yarn_fast, yarn_slow;
+  int32_t conv_taps;                        /* attention (0 = none) and LRU */
+  float lru_decay;
+  int32_t mem_heads, mem_key_dim, mem_value_dim; /* matrix memory beside attention; 0 = none */
+  float mem_gate_cap, mix_scale, mem_scale;
 } b200_decoder_layer;
 typedef struct b200_decoder_config {
   int32_t n_layers, hidden, vocab;
@@ -642,7 +669,8 @@ typedef struct b200_decoder_config {
   int32_t dtype;                             /* B200_DT_* */
   int32_t max_rows, max_reqs, max_seqs;
   float norm_eps, embed_scale, logit_scale;
-  int32_t flags; /* B200_DEC_SCALAR_NORM, B200_DEC_DEPTH_AVERAGE */
+  int32_t flags; /* those of the whole stack */
+  float residual_scale; /* B200_DEC_SUM_NORM */
 } b200_decoder_config;
 typedef struct b200_decoder b200_decoder;
 enum { B200_DEC_W_Q = 0, B200_DEC_W_K = 1, B200_DEC_W_V = 2, B200_DEC_W_O = 3, B200_DEC_W_GATE = 4, B200_DEC_W_UP = 5,
@@ -653,7 +681,14 @@ enum { B200_DEC_W_Q = 0, B200_DEC_W_K = 1, B200_DEC_W_V = 2, B200_DEC_W_O = 3, B
        B200_DEC_W_OUT_GATE = 23, B200_DEC_W_A1 = 24, B200_DEC_W_A2 = 25, B200_DEC_B_A2 = 26, B200_DEC_HEAD_NORM = 27,
        /* experts stacked: [n_experts][expert_ffn][hidden], down [n_experts][hidden][expert_ffn] */
        B200_DEC_W_EXPERT_GATE = 28, B200_DEC_W_EXPERT_UP = 29, B200_DEC_W_EXPERT_DOWN = 30,
-       B200_DEC_DEPTH = 31 /* [layer + 2] */ };
+       B200_DEC_DEPTH = 31 /* [layer + 2] */,
+       B200_DEC_W_DQ = 32, B200_DEC_DQ_NORM = 33, B200_DEC_Q_NORM = 34, B200_DEC_K_NORM = 35,
+       B200_DEC_CONV_Q = 36, B200_DEC_CONV_K = 37, B200_DEC_CONV_V = 38, /* [channels, taps] */
+       B200_DEC_W_MEM_Q = 39, B200_DEC_W_MEM_K = 40, B200_DEC_W_MEM_V = 41, B200_DEC_W_MEM_G = 42, B200_DEC_W_MEM_O = 43,
+       B200_DEC_W_MEM_I = 44, B200_DEC_W_MEM_F = 45, B200_DEC_B_MEM_I = 46, B200_DEC_B_MEM_F = 47, B200_DEC_MEM_NORM = 48 /* [heads * value] */,
+       B200_DEC_W_LRU_Y = 49, B200_DEC_B_LRU_Y = 50, B200_DEC_W_LRU_X = 51, B200_DEC_B_LRU_X = 52, B200_DEC_LRU_CONV = 53 /* [channels, taps] */,
+       B200_DEC_B_LRU_CONV = 54, B200_DEC_W_LRU_R = 55 /* [blocks, out, in] */, B200_DEC_B_LRU_R = 56, B200_DEC_W_LRU_I = 57,
+       B200_DEC_B_LRU_I = 58, B200_DEC_LRU_LAMBDA = 59, B200_DEC_W_ROUTER = 60 };
 b200_status b200_decoder_create(const b200_decoder_config* cfg, const b200_decoder_layer* layers, b200_decoder** out);
 void b200_decoder_destroy(b200_decoder* m);
 /* One tensor, bf16 on the host, matrices [out, in]; n_elems is checked against the shape the configuration gives.
