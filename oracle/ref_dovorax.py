@@ -259,3 +259,99 @@ def forward(tokens, w, cfg, rnd=ident, want_layers=False, without=NOTHING):
         trail.append(x)
     logits = linear(rnd(norm(x, "final.norm")), w["embed"])
     return (logits, np.stack(trail)) if want_layers else logits
+
+
+# ---- test models -------------------------------------------------------------------------------------
+def tensor_shapes(cfg):
+    """name -> shape of every tensor a configuration asks for."""
+    d, out = cfg["width"], {"embed": (cfg["vocab"], cfg["width"])}
+    for i, spec in enumerate(cfg["layers"]):
+        n, m = f"l{i}", spec["mixer"]
+        mix = f"{n}.mix."
+        out[f"{n}.norm1"] = (d,)
+        if spec["type"] == "latent_attention":
+            h = m["heads"]
+            out[mix + "dq"], out[mix + "dq.norm"], out[mix + "uq"] = (m["q_rank"], d), (m["q_rank"],), (h * (m["dim"] + m["rot_dim"]), m["q_rank"])
+            if m.get("kv_from") is None:
+                out[mix + "dkv"], out[mix + "dkv.norm"] = (m["kv_rank"] + m["rot_dim"], d), (m["kv_rank"],)
+            out[mix + "uk"], out[mix + "uv"], out[mix + "o"] = (h * m["dim"], m["kv_rank"]), (h * m["vdim"], m["kv_rank"]), (d, h * m["vdim"])
+        elif spec["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            for p, rows in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
+                out[f"{mix}left.{p}"] = (rows, d)
+                if a.get("conv"):
+                    out[f"{mix}left.{p}.conv"] = (rows, a["conv"])
+            out[mix + "left.q.norm"], out[mix + "left.k.norm"], out[mix + "left.o"] = (a["dim"],), (a["dim"],), (d, a["heads"] * a["vdim"])
+            for p, rows in (("q", r["dim"]), ("k", r["dim"]), ("v", r["vdim"]), ("g", r["vdim"]), ("i", 1), ("f", 1)):
+                out[f"{mix}right.{p}"] = (r["heads"] * rows, d)
+            out[mix + "right.i.b"], out[mix + "right.f.b"] = (r["heads"],), (r["heads"],)
+            out[mix + "right.norm"], out[mix + "right.o"] = (r["heads"] * r["vdim"],), (d, r["heads"] * r["vdim"])
+        else:
+            w, b = m["width"], m["blocks"]
+            for p in "xy":
+                out[mix + p], out[f"{mix}{p}.b"] = (w, d), (w,)
+            out[mix + "conv"], out[mix + "conv.b"] = (w, m["conv"]), (w,)
+            for p in ("ra", "ri"):
+                out[mix + p], out[f"{mix}{p}.b"] = (b, w // b, w // b), (b, w // b)
+            out[mix + "lam"], out[mix + "o"] = (w,), (d, w)
+        mlp = spec.get("mlp")
+        if not mlp:
+            continue
+        out[f"{n}.norm2"] = (d,)
+        if mlp["kind"] == "dense":
+            parts = [("", mlp["ff"])]
+        else:
+            parts = [(f"e{e}.", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])]
+            out[f"{n}.mlp.router"] = (mlp["router"]["experts"], d)
+            if mlp.get("shared"):
+                parts.append(("shared.", mlp["shared"]["ff"]))
+        for p, f in parts:
+            out[f"{n}.mlp.{p}up"], out[f"{n}.mlp.{p}down"] = (f, d), (d, f)
+    out["final.norm"] = (d,)
+    return out
+
+
+def random_weights(cfg, seed, decisive=True):
+    """Weights as bf16 can hold them: projections keep unit variance, norm weights scatter, gates remember some tens of tokens.
+
+    `decisive`: every token id ranks the experts of a layer by levels in a few coordinates of its own, which the sublayers
+    hardly touch, so that 16-bit rounding cannot swap two experts."""
+    from .ref_math import bf16_round
+
+    rng = np.random.default_rng(seed)
+    most = max([s["mlp"]["router"]["experts"] for s in cfg["layers"] if s.get("mlp") and s["mlp"]["kind"] == "moe"], default=0) if decisive else 0
+    out = {}
+    for name, shape in tensor_shapes(cfg).items():
+        part = name.split(".")[-1]
+        if part in ("norm1", "norm2") or name == "final.norm":
+            a = 0.3 * rng.normal(size=shape)
+            a[:most] = 0.0
+        elif part == "norm":
+            a = 1.0 + 0.3 * rng.normal(size=shape)
+        elif name.endswith(".f.b"):
+            a = 3.0 + rng.normal(size=shape)
+        elif part == "b":
+            a = rng.normal(size=shape)
+        elif part == "lam":
+            a = -3.0 + 1.5 * rng.normal(size=shape)
+        elif part == "embed":
+            a = rng.normal(size=shape)
+            if most:
+                a[:, :most] = np.stack([rng.permutation(np.linspace(-1.8, 1.8, most)) for _ in range(shape[0])])
+        elif part == "router" and most:
+            a = np.zeros(shape)
+            a[np.arange(shape[0]), rng.permutation(most)[:shape[0]]] = 1.5
+        elif part in ("i", "f"):
+            a = 2.0 * rng.normal(size=shape) / np.sqrt(shape[1])
+        else:
+            a = rng.normal(size=shape) / np.sqrt(shape[-1])
+            if part in ("o", "down") and most:
+                a[:most] *= 0.03
+        out[name] = bf16_round(np.asarray(a, np.float32)).astype(np.float64)
+    return out
+
+
+def write_model(folder, cfg, weights):
+    from .ref_sotavik import write_model as write
+
+    write(folder, cfg, weights)
