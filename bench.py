@@ -17,6 +17,8 @@ Prints ONE JSON line (rank 0).  Workloads (synthetic seeded inputs):
   tafuvik : the looped decoder stack (one GPU) beside the LLaMA stack at equal size, both bf16 — decode steps of 64
       requests and prefill steps of 4096 rows at a few layer shapes, with each kernel category against its roofline.
   sotavik : the Sotavik stack (latent attention, gated linear attention, experts by token id; one GPU) the same way.
+  dovorax : the Dovorax stack (gated linear recurrence, windowed latent attention, attention beside a matrix memory, routed experts; one
+            GPU) the same way, beside the Sotavik stacks too.
 Multi-GPU (torchrun, one rank per GPU): independent replicas of the workload, no collective in the
 step (requests never interact); `value` = tokens of all ranks / max-over-ranks time.
 """
@@ -1290,6 +1292,141 @@ def run_sotavik(args, local: int):
         "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind}, "sizes": out, "e2e": None, "gpu_launches": launches, "clocks": clocks}))
 
 
+# Layer shapes of the Dovorax bench beside LLaMA and the Sotavik stacks of equal width and feed-forward width: L latent attention with a
+# window, S the same on the latents of the layer before, P attention beside a matrix memory, R a gated linear recurrence.
+DOVORAX_SIZES = {
+    "d4096": dict(latent=dict(heads=32, dim=128, rot=64, vdim=128, rank=512, q_rank=1536, window=1024), memory=dict(heads=8, dim=256, vdim=512),
+                  attention=dict(heads=32, kv_heads=8, dim=128, rot=64), taps=4, lru=dict(width=4096, blocks=16)),
+    "d2048": dict(latent=dict(heads=16, dim=96, rot=32, vdim=64, rank=256, q_rank=768, window=1024), memory=dict(heads=4, dim=256, vdim=512),
+                  attention=dict(heads=16, kv_heads=4, dim=128, rot=64), taps=4, lru=dict(width=2560, blocks=10)),
+}
+DOVORAX_STACKS = {"dovorax_lru": "RRRRRR", "dovorax_latent": "LSLSLS", "dovorax_parallel": "PPPPPP", "dovorax_mixed": "RLPRSP"}
+
+
+def _dovorax_layers(z, order):
+    from dmlx_b200 import device as dev
+
+    ff = dict(ffn=z["shared"], n_experts=z["experts"], top_k=z["top"], expert_ffn=z["expert_ffn"], n_groups=8, keep_groups=4)
+    flags = dev.DEC_FF_GELU | dev.DEC_ROUTER
+    l, m, a, r = z["latent"], z["memory"], z["attention"], z["lru"]
+    yarn = dict(yarn_factor=4.0, yarn_original=4096.0, yarn_fast=32.0, yarn_slow=1.0, rot_base=1e4)
+    out = []
+    for i, c in enumerate(order):
+        if c in "LS":
+            source = 1 + max(j for j in range(i) if order[j] == "L") if c == "S" else 0
+            out.append(dict(mixer=dev.MIX_LATENT, n_heads=l["heads"], n_kv_heads=1, key_dim=l["dim"], value_dim=l["vdim"], kv_rank=l["rank"], rot_dim=l["rot"],
+                            q_rank=l["q_rank"], window=l["window"], scale=(l["dim"] + l["rot"]) ** -0.5, kv_source=source, flags=flags | dev.DEC_ROT_HALVES,
+                            **yarn, **ff))
+        elif c == "P":
+            out.append(dict(mixer=dev.MIX_ATTENTION, n_heads=a["heads"], n_kv_heads=a["kv_heads"], key_dim=a["dim"], value_dim=a["dim"], rot_dim=a["rot"],
+                            conv_taps=z["taps"], scale=a["dim"] ** -0.5, mem_heads=m["heads"], mem_key_dim=m["dim"], mem_value_dim=m["vdim"], mem_gate_cap=15.0,
+                            mix_scale=0.5, mem_scale=0.5, flags=flags | dev.DEC_QK_NORM | dev.DEC_QK_NORM_WEIGHT | dev.DEC_SINK_ONE | dev.DEC_ROT_HALVES,
+                            **yarn, **ff))
+        else:
+            w = r["width"] // r["blocks"]
+            out.append(dict(mixer=dev.MIX_LRU, n_heads=r["blocks"], n_kv_heads=r["blocks"], key_dim=w, value_dim=w, conv_taps=z["taps"], lru_decay=8.0,
+                            flags=flags, **ff))
+    return out
+
+
+def _dovorax_work(z, order, ctxs, prefill):
+    """As _sotavik_work."""
+    d, l, m, a, r = z["hidden"], z["latent"], z["memory"], z["attention"], z["lru"]
+    rows, seqs, n = DECODER_ROWS if prefill else len(ctxs), len(ctxs), len(order)
+
+    def seen(window):  # (query, key) pairs, cached tokens read
+        if prefill:
+            per = rows // len(ctxs)
+            return len(ctxs) * float(np.minimum(np.arange(per) + 1, window or per).sum()), float(rows)
+        return (float(np.minimum(ctxs, window or 1 << 30).sum()),) * 2
+
+    nl, ns, np_, nr = (order.count(c) for c in "LSPR")
+    state = 4.0 if prefill else 8.0  # a prompt only writes its state
+    lat, hq, hv = l["rank"] + l["rot"], l["heads"] * (l["dim"] + l["rot"]), l["heads"] * l["vdim"]
+    keys, read = seen(l["window"])
+    attn_b = (nl + ns) * (read * lat + rows * l["heads"] * (lat + l["rank"])) * 2.0
+    attn_f = (nl + ns) * 2.0 * keys * l["heads"] * (l["dim"] + l["rot"] + l["vdim"])
+    keys, read = seen(0)
+    ad, qkv = a["dim"], (a["heads"] + 2 * a["kv_heads"]) * a["dim"]
+    mk, mv, W = m["heads"] * m["dim"], m["heads"] * m["vdim"], r["width"]
+    attn_b += np_ * ((read * a["kv_heads"] + rows * a["heads"]) * 2 * ad * 2.0 + seqs * mk * m["vdim"] * state + rows * (2 * mk + 3 * mv) * 2.0)
+    attn_f += np_ * (4.0 * keys * a["heads"] * ad + 4.0 * rows * mk * m["vdim"])
+    attn_b += nr * (rows * W * 14.0 + seqs * W * state)
+    append = (nl * (l["q_rank"] + lat + hq) + ns * (l["q_rank"] + hq) + np_ * qkv + nr * 2 * W) * rows * 4.0
+    append += seqs * (z["taps"] - 1) * (np_ * qkv + nr * W) * state
+    dense = nl * d * lat + (nl + ns) * (d * l["q_rank"] + l["q_rank"] * hq + l["heads"] * (l["dim"] + l["vdim"]) * l["rank"] + d * hv)
+    dense += np_ * d * (qkv + 2 * mk + 2 * mv + 2 * m["heads"] + a["heads"] * ad + mv) + nr * (3 * d * W + 2 * W * W // r["blocks"])
+    dense += n * (2 * d * z["shared"] + d * z["experts"])
+    head = d * DECODER_VOCAB
+    mat_b = 2.0 * (dense + n * min(z["experts"], rows * z["top"]) * 2 * d * z["expert_ffn"] + head)
+    mat_f = 2.0 * rows * (dense + n * z["top"] * 2 * d * z["expert_ffn"]) + 2.0 * seqs * head
+    return {"attention": (attn_b, attn_f), "matmul": (mat_b, mat_f), "rope_append": (append, 0.0), "other": (rows * d * n * (28.0 + 6.0 * z["top"]), 0.0)}
+
+
+def run_dovorax(args, local: int):
+    import torch
+
+    from dmlx_b200 import device as dev
+
+    torch.cuda.set_device(local)
+    torch.cuda.set_stream(torch.cuda.Stream())
+    hbm, kind = load_peaks()
+    p = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    tflops = float(json.load(open(p))["bf16_tflops"]) if os.path.exists(p) else 1590.0
+    K, W = min(args.steps, 50), max(args.warmup, 3)
+    ctxs = np.clip(np.rint(np.random.default_rng(77).lognormal(np.log(2600), 0.6, DECODER_REQS)), 256, 12000).astype(np.int64)
+    pages = int((-(-(ctxs + 4 * (K + W) + 64) // PAGE)).sum()) + 16
+    most = int(-(-(ctxs.max() + 4 * (K + W) + 64) // PAGE))
+    sampler = ClockSampler(local)
+    sampler.start()
+    out, launches = {}, 0
+    for name, extra in DOVORAX_SIZES.items():
+        base = SOTAVIK_SIZES[name]
+        z = dict(base, **extra)
+        for which in ("llama", "sotavik_latent", "sotavik_gla", *DOVORAX_STACKS):
+            if which == "llama":
+                model = dev.LlamaModel(6, z["hidden"], z["heads"], z["kv_heads"], z["head_dim"], z["ffn"], DECODER_VOCAB, DECODER_ROWS, DECODER_REQS,
+                                       DECODER_REQS)
+                model.random_init(dev.Q_BF16, 3)
+                kv = dev.PagedKVCache(6, z["kv_heads"], z["head_dim"], pages, DECODER_REQS, most, z["heads"], max_rows=DECODER_ROWS)
+            else:
+                theirs = which.startswith("sotavik")
+                layers = _sotavik_layers(base, SOTAVIK_STACKS[which]) if theirs else _dovorax_layers(z, DOVORAX_STACKS[which])
+                model = dev.DecoderModel(z["hidden"], DECODER_VOCAB, layers, 1e-5, 1.0, None, dev.DT_BF16, DECODER_ROWS, DECODER_REQS, DECODER_REQS,
+                                         flags=dev.DEC_SCALAR_NORM | dev.DEC_DEPTH_AVERAGE if theirs else dev.DEC_SUM_NORM, residual_scale=2.0)
+                model.random_init(3)
+                kv = model.make_cache(pages, DECODER_REQS, most)
+            for mode in ("decode", "prefill"):
+                ms, prof, n = _time_stack(model, kv, ctxs, pages, mode, K, W)
+                launches += n
+                at = ctxs if mode == "decode" else ctxs[:2]
+                if which == "llama":
+                    work = _decoder_work(dict(z, llama_dim=z["head_dim"]), 6, 0, at, mode == "prefill", True)
+                elif which.startswith("sotavik"):
+                    work = _sotavik_work(base, SOTAVIK_STACKS[which], at, mode == "prefill")
+                else:
+                    work = _dovorax_work(z, DOVORAX_STACKS[which], at, mode == "prefill")
+                entry = {"ms_per_step": ms, "tokens_per_s": (DECODER_REQS if mode == "decode" else DECODER_ROWS) / ms * 1e3}
+                for cat, (nbytes, flops) in work.items():
+                    ideal = max(nbytes / hbm / 1e6, flops / tflops / 1e9)
+                    entry[cat] = {"ms": prof[cat], "of_roofline": ideal / prof[cat] if prof[cat] > 0 else None}
+                out.setdefault(name, {}).setdefault(mode, {})[which] = entry
+            kv.close()
+            model.close()
+    clocks = sampler.stop()
+    head = out["d4096"]["decode"]["dovorax_mixed"]
+    print(json.dumps({
+        "metric": "decode tokens/sec (Dovorax stack, 6 layers)", "value": head["tokens_per_s"], "unit": "decode tokens/s", "n_gpus": 1,
+        "steps": K, "warmup": W, "ms_per_step": head["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "dovorax", "stacks": DOVORAX_STACKS, "shapes": DOVORAX_SIZES, "feed_forward": SOTAVIK_SIZES, "vocab": DECODER_VOCAB,
+                   "decode_requests": DECODER_REQS, "cached_tokens": int(ctxs.sum()), "prefill": f"2 prompts of {DECODER_ROWS // 2} tokens in one step",
+                   "parallelism": "dp1", "l2": "weights and caches larger than L2"},
+        "note": "of_roofline: the larger of bytes / measured copy bandwidth and FLOPs / measured burst bf16 rate, over the category's time "
+                "(eager launches with an event pair each, so small kernels carry their launch gap)",
+        "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind}, "sizes": out, "e2e": None, "gpu_launches": launches, "clocks": clocks}))
+
+
 def run_tafuvik(args, local: int):
     import torch
 
@@ -1403,6 +1540,10 @@ def main():
     if args.mx_persistent >= 0:
         from dmlx_b200 import _lib
         _lib.lib.b200_set_qmm_mx_persistent(args.mx_persistent)
+    if args.workload == "dovorax":
+        if rank == 0:
+            run_dovorax(args, local)
+        return
     if args.workload == "sotavik":
         if rank == 0:
             run_sotavik(args, local)

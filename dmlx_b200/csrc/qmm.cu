@@ -3254,6 +3254,7 @@ extern "C" b200_status b200_qmm_static_scratch(const b200_qweight* w, const void
   if (rows <= 0) return B200_OK;
   if (w->n_experts != 1) { b200_set_error("qmm (static scratch): single weights only"); return B200_ERR_INVALID_ARGUMENT; }
   if (epilogue == B200_EPI_RESIDUAL && !d_residual) { b200_set_error("qmm (static scratch): residual epilogue without a residual"); return B200_ERR_INVALID_ARGUMENT; }
+  if (epilogue == B200_EPI_GELU) { b200_set_error("qmm (static scratch): no GELU epilogue"); return B200_ERR_UNSUPPORTED; }
   if (epilogue == B200_EPI_SWIGLU && (w->n % 2) != 0) { b200_set_error("qmm (static scratch): SwiGLU needs an even N"); return B200_ERR_INVALID_ARGUMENT; }
   int dev = 0;
   B200_CUDA_TRY(cudaGetDevice(&dev));
