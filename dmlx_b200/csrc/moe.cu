@@ -26,7 +26,8 @@ namespace {
 
 constexpr int kMaxExperts = 1024;
 constexpr int kMaxTopK = 16;
-constexpr int kMaxGroups = 64;  // of a router's experts
+constexpr int kMaxGroups = 64;  // of a decoder layer's router
+constexpr int kMaxRouterTop = 32;
 
 __device__ __forceinline__ bool beats(float va, int ia, float vb, int ib) { return va > vb || (va == vb && ia > ib); }
 
@@ -496,7 +497,7 @@ __global__ void combine_kernel(const __nv_bfloat16* __restrict__ y_sorted, const
 }  // namespace
 
 int b200_moe_max_experts() { return kMaxExperts; }
-int b200_moe_max_top() { return kMaxTopK; }
+int b200_moe_max_top() { return kMaxRouterTop; }
 int b200_moe_max_groups() { return kMaxGroups; }
 
 b200_status b200_moe_table_plan(const MoeTableLayer* d_layers, int n_layers, int most_experts, const uint32_t* d_tokens, int n_tokens, int vocab,
@@ -512,7 +513,7 @@ b200_status b200_moe_table_plan(const MoeTableLayer* d_layers, int n_layers, int
 
 b200_status b200_moe_route_plan(const MoeTableLayer& L, const MatSrc& logits, bool f32, int n_groups, int keep_groups, int n_tokens, int tile_rows,
                                 float* d_weights, void* stream) {
-  if (L.n_experts <= 0 || L.n_experts > kMaxExperts || L.top <= 0 || L.top > kMaxTopK || n_groups <= 0 || n_groups > kMaxGroups ||
+  if (L.n_experts <= 0 || L.n_experts > kMaxExperts || L.top <= 0 || L.top > kMaxRouterTop || n_groups <= 0 || n_groups > kMaxGroups ||
       L.n_experts % n_groups != 0 || keep_groups <= 0 || keep_groups > n_groups || L.top > keep_groups * (L.n_experts / n_groups)) {
     b200_set_error("router: %d experts, top %d, %d of %d groups", L.n_experts, L.top, keep_groups, n_groups);
     return B200_ERR_INVALID_ARGUMENT;

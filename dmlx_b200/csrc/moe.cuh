@@ -15,6 +15,7 @@ struct MoeTableLayer {
   int4* items = nullptr;        // {expert, first sorted row, rows}
 };
 int b200_moe_max_experts();
+// Limits of a layer's router.
 int b200_moe_max_top();
 int b200_moe_max_groups();
 b200_status b200_moe_table_plan(const MoeTableLayer* d_layers, int n_layers, int most_experts, const uint32_t* d_tokens, int n_tokens, int vocab,
