@@ -43,16 +43,18 @@ struct PrepArgs {
   const int *pos, *row_seq;
 };
 
-// One warp per (row, query head), one for the row's query latent, and one for the row's latent.
+// One warp per (row, query head); blocks of their own for the row's latent and its query latent.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256) latent_prep_kernel(PrepArgs a) {
   const LatentPrep& p = a.p;
-  const int row = blockIdx.x, lane = threadIdx.x & 31, u = blockIdx.y * 8 + (threadIdx.x >> 5);
-  if (u > p.heads + 1) return;
+  __shared__ float part[32];
+  const int row = blockIdx.x, lane = threadIdx.x & 31, head_blocks = (p.heads + 7) / 8, u = blockIdx.y * 8 + (threadIdx.x >> 5);
+  const bool of_heads = (int)blockIdx.y < head_blocks;
+  if (of_heads && u >= p.heads) return;
   const int per_head = p.dim + p.rot;
   const float2* rt = p.rotation + (size_t)row * (p.rot / 2);
-  auto rotate = [&](T* dst, int col) {
-    for (int i = lane; i < p.rot / 2; i += 32) {
+  auto rotate = [&](T* dst, int col, int first, int step) {
+    for (int i = first; i < p.rot / 2; i += step) {
       const int at = p.halves ? i : 2 * i, to = p.halves ? i + p.rot / 2 : 2 * i + 1;
       const float x = mat_value<T, 1>(p.src, row, col + at).v[0], y = mat_value<T, 1>(p.src, row, col + to).v[0];
       const float2 cs = rt[i];
@@ -60,39 +62,49 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(PrepArgs a) {
       st(dst + to, y * cs.x + x * cs.y);
     }
   };
-  // columns col .. col + n - 1 divided by their root mean square, times w
+  // by the whole block: columns col .. col + n - 1 divided by their root mean square, times w (the first ones stay in registers)
   auto normed = [&](T* dst, int col, int n, const float* w) {
+    constexpr int KEEP = 2;
+    Vec<VEC> keep[KEEP];
     float ss = 0.f;
-    for (int c = lane * VEC; c < n; c += 32 * VEC) {
+    auto each = [&](auto f) {
+#pragma unroll
+      for (int k = 0; k < KEEP; ++k) {
+        const int c = (k * 256 + (int)threadIdx.x) * VEC;
+        if (c < n) f(c, k);
+      }
+      for (int c = (KEEP * 256 + (int)threadIdx.x) * VEC; c < n; c += 256 * VEC) f(c, -1);
+    };
+    each([&](int c, int k) {
       const Vec<VEC> v = mat_value<T, VEC>(p.src, row, col + c);
+      if (k >= 0) keep[k] = v;
 #pragma unroll
       for (int e = 0; e < VEC; ++e) ss += v.v[e] * v.v[e];
-    }
-    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + p.eps);
-    for (int c = lane * VEC; c < n; c += 32 * VEC) {
-      Vec<VEC> v = mat_value<T, VEC>(p.src, row, col + c);
+    });
+    const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)n + p.eps);
+    each([&](int c, int k) {
+      Vec<VEC> v = k >= 0 ? keep[k >= 0 ? k : 0] : mat_value<T, VEC>(p.src, row, col + c);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) v.v[e] *= r * w[c + e];
       store_vec<VEC>(dst + c, v);
-    }
+    });
   };
-  if (u < p.heads) {
+  if (of_heads) {
     T* plain = (T*)p.q_plain + ((size_t)row * p.heads + u) * p.plain_stride;
     for (int c = lane * VEC; c < p.dim; c += 32 * VEC) store_vec<VEC>(plain + c, mat_value<T, VEC>(p.src, row, u * per_head + c));
     for (int c = p.dim + lane; c < p.plain_stride; c += 32) st(plain + c, 0.f);
     T* q = (T*)p.q + ((size_t)row * p.heads + u) * a.L.kd;
-    rotate(q + p.rank, u * per_head + p.dim);
+    rotate(q + p.rank, u * per_head + p.dim, lane, 32);
     for (int c = a.L.key_dim + lane; c < a.L.kd; c += 32) st(q + c, 0.f);
     return;
   }
-  if (u == p.heads + 1) {
+  if ((int)blockIdx.y > head_blocks || !p.keys) {
     if (p.q_rank == 0) return;
     T* dst = (T*)p.q_latent + (size_t)row * p.q_latent_stride;
     normed(dst, 0, p.q_rank, p.q_norm);
-    for (int c = p.q_rank + lane; c < p.q_latent_stride; c += 32) st(dst + c, 0.f);
+    for (int c = p.q_rank + (int)threadIdx.x; c < p.q_latent_stride; c += 256) st(dst + c, 0.f);
     return;
   }
-  if (!p.keys) return;
   const int pos = a.pos[row], seq = a.row_seq[row];
   const int page_idx = pos / a.d.page_size, slot = pos - page_idx * a.d.page_size;
   // a step whose reservation failed has no page for this row: nothing is written (the error word is set)
@@ -101,7 +113,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(PrepArgs a) {
   T* dst = (T*)((char*)a.d.k_pool + a.L.k_off) + ((size_t)page * a.d.page_size + slot) * (size_t)a.L.kd;
   const int col = p.q_rank + p.heads * per_head;
   normed(dst, col, p.rank, p.norm);
-  rotate(dst + p.rank, col + p.rank);
+  rotate(dst + p.rank, col + p.rank, threadIdx.x, 256);
 }
 
 }  // namespace
@@ -126,7 +138,7 @@ b200_status b200_latent_prep(b200_kv* kv, const LatentPrep& p, const int32_t* d_
   const bool v4 = p.dim % 4 == 0 && p.rot % 4 == 0 && p.rank % 4 == 0 && p.plain_stride % 4 == 0 && p.q_rank % 4 == 0 && p.q_latent_stride % 4 == 0 && (p.src.ws || p.src.y_stride % 4 == 0);
   auto* kernel = kv->dev.elem_bytes == 4 ? (v4 ? latent_prep_kernel<float, 4> : latent_prep_kernel<float, 1>)
                                          : (v4 ? latent_prep_kernel<__nv_bfloat16, 4> : latent_prep_kernel<__nv_bfloat16, 1>);
-  kernel<<<dim3(rows, (p.heads + (p.q_rank > 0 ? 2 : 1) + 7) / 8), 256, 0, (cudaStream_t)stream>>>(a);
+  kernel<<<dim3(rows, (p.heads + 7) / 8 + (p.keys ? 1 : 0) + (p.q_rank > 0 ? 1 : 0)), 256, 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

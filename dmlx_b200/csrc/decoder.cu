@@ -376,10 +376,133 @@ __global__ void __launch_bounds__(256) decoder_qkv_conv_kernel(QkvArgs a) {
     for (int c = lane * VEC; c < dim; c += 32 * VEC) conv_update<VEC>(a.conv, value, r0, count, slot, n0 + c);
 }
 
+// The same for four taps and heads up to KEEP * 128 wide, R rows per warp: a head's row stays in registers but for the columns that are
+// rotated, and rows of one request that lie next to each other share the loads of their inputs and of the weights.
+template <typename T, int KEEP, int R>
+__global__ void __launch_bounds__(256) decoder_qkv_conv4_kernel(QkvArgs a, int rows) {
+  extern __shared__ float row_sh[];  // [warp][rot]
+  const int begin = blockIdx.x * R, end = min(begin + R, rows);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, H = a.L.heads, u = blockIdx.y * 8 + warp;
+  if (u >= a.hq + 2 * H || a.d.state[ST_ERR] != 0) return;
+  const bool is_q = u < a.hq, is_v = u >= a.hq + H;
+  const int head = is_q ? u : (is_v ? u - a.hq - H : u - a.hq);
+  const int dim = is_v ? a.L.value_dim : a.L.key_dim, width = is_v ? a.L.vd : a.L.kd;
+  const int n0 = is_v ? (a.hq + H) * a.L.key_dim + head * dim : u * dim;
+  const int rot = is_v ? 0 : a.rot, half = rot / 2;
+  float* sh = row_sh + warp * a.rot;
+  const float* norm = is_q ? a.q_norm : (is_v ? nullptr : a.k_norm);
+  auto value = [&](int row, int c) {
+    Vec<4> v = mat_value<T, 4>(a.src, row, c);
+    if (a.bias) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v.v[e] += a.bias[c + e];
+    }
+    return v;
+  };
+  auto finish = [&](int row, Vec<4> (&x)[KEEP]) {  // norm, rotation, store
+    T* dst = is_q ? (T*)a.q + (size_t)row * a.q_stride + (size_t)head * a.L.kd : page_row<T>(a, row, head, is_v);
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      if ((k * 32 + lane) * 4 < dim) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss += x[k].v[e] * x[k].v[e];
+      }
+    }
+    float r = is_v ? a.v_scale : 1.f;
+    if (a.qk_norm && !is_v) r = 1.0f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int c = (k * 32 + lane) * 4;
+      if (c < dim) {
+        Vec<4> f{{1.f, 1.f, 1.f, 1.f}};
+        if (norm) f = load_vec<4>(norm + c);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          x[k].v[e] *= r * f.v[e];
+          if (c + e < rot) sh[c + e] = x[k].v[e];
+        }
+      }
+    }
+    __syncwarp();
+    if (dst) {
+#pragma unroll
+      for (int k = 0; k < KEEP; ++k) {
+        const int c = (k * 32 + lane) * 4;
+        if (c < dim) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int i = c + e;
+            if (i < rot) {
+              const bool up = a.halves ? i >= half : (i & 1);
+              const int other = a.halves ? (up ? i - half : i + half) : i ^ 1;
+              const float2 cs = a.rotation[(size_t)row * half + (a.halves ? (up ? i - half : i) : i >> 1)];
+              x[k].v[e] = fmaf(up ? cs.y : -cs.y, sh[other], x[k].v[e] * cs.x);
+            }
+          }
+          store_vec<4>(dst + c, x[k]);
+        }
+      }
+      for (int c = dim + lane; c < width; c += 32) st(dst + c, 0.f);
+    }
+    __syncwarp();
+  };
+  if constexpr (R > 1) {
+    if (begin + R <= rows && a.row_to_req[begin] == a.row_to_req[begin + R - 1] && begin - a.cu[a.row_to_req[begin]] >= 3) {
+      Vec<4> x[KEEP][R];
+#pragma unroll
+      for (int k = 0; k < KEEP; ++k) {
+        const int c = (k * 32 + lane) * 4;
+        if (c < dim) conv_values_inside<4, R, 4>(a.conv, value, begin, n0 + c, x[k]);
+      }
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        Vec<4> row[KEEP];
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) row[k] = x[k][r];
+        finish(begin + r, row);
+      }
+      return;
+    }
+  }
+  for (int first = begin; first < end; ++first) {
+    const int req = a.row_to_req[first], r0 = a.cu[req], count = a.cu[req + 1] - r0, slot = a.row_seq[first];
+    if (slot < 0 || slot >= a.d.max_seqs) continue;
+    const int n = conv_rows(a.conv, first - r0, count);
+    for (int row = first; row < first + n; ++row) {
+      const int pos = a.pos[row];
+      Vec<4> x[KEEP];
+#pragma unroll
+      for (int k = 0; k < KEEP; ++k) {
+        const int c = (k * 32 + lane) * 4;
+        if (c < dim) x[k] = conv_value<4>(a.conv, value, row, row - r0, pos, slot, n0 + c);
+      }
+      finish(row, x);
+    }
+    if (first == r0)
+      for (int c = lane * 4; c < dim; c += 128) conv_update<4>(a.conv, value, r0, count, slot, n0 + c);
+  }
+}
+
 b200_status launch_qkv(const QkvArgs& a, int rows, cudaStream_t s) {
   if (a.conv.taps > 0 || a.q_norm || a.rot > 0 || a.v_scale != 1.f) {
     const bool vec = a.L.key_dim % 4 == 0 && a.L.value_dim % 4 == 0 && (a.src.ws || a.src.y_stride % 4 == 0) && a.conv.slot_elems % 4 == 0 &&
                      a.conv.channels % 4 == 0;
+    if (vec && a.conv.taps == 4 && !a.conv.bias && a.L.key_dim <= 256 && a.L.value_dim <= 256) {
+      const bool narrow = a.L.key_dim <= 128 && a.L.value_dim <= 128, many = rows >= 1024;
+      auto run = [&](auto* kernel, int per) {
+        kernel<<<dim3((rows + per - 1) / per, (a.hq + 2 * a.L.heads + 7) / 8), 256, sizeof(float) * 8 * std::max(a.rot, 1), s>>>(a, rows);
+      };
+      auto pick = [&](auto tag) {
+        using T = decltype(tag);
+        if (many) narrow ? run(decoder_qkv_conv4_kernel<T, 1, 4>, 4) : run(decoder_qkv_conv4_kernel<T, 2, 4>, 4);
+        else narrow ? run(decoder_qkv_conv4_kernel<T, 1, 1>, 1) : run(decoder_qkv_conv4_kernel<T, 2, 1>, 1);
+      };
+      if (a.d.elem_bytes == 4) pick(float{});
+      else pick(__nv_bfloat16{});
+      B200_LAUNCH_CHECK();
+      return B200_OK;
+    }
     const size_t smem = sizeof(float) * 8 * std::max(a.L.key_dim, a.L.value_dim);
     if (smem > 200 * 1024) { b200_set_error("decoder: head widths %d / %d are too large", a.L.key_dim, a.L.value_dim); return B200_ERR_UNSUPPORTED; }
     auto* kernel = a.d.elem_bytes == 4 ? (vec ? decoder_qkv_conv_kernel<float, 4> : decoder_qkv_conv_kernel<float, 1>)
@@ -427,8 +550,9 @@ struct b200_decoder : b200_model {
     b200_qweight *wuq = nullptr, *wgates = nullptr, *wrouter = nullptr;
     float *bias = nullptr, *sinks = nullptr, *slopes = nullptr, *norm1 = nullptr, *norm2 = nullptr, *post1 = nullptr, *post2 = nullptr;
     float *dkv_norm = nullptr, *a2 = nullptr, *a2_bias = nullptr, *head_norm = nullptr, *depth = nullptr;
-    float *dq_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr, *conv = nullptr, *conv_bias = nullptr, *gate_bias = nullptr, *mem_norm = nullptr;
+    float *dq_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr, *conv_bias = nullptr, *gate_bias = nullptr, *mem_norm = nullptr;
     float *lru_bias = nullptr, *lru_rate = nullptr;  // [y | x | r | i], [width]
+    __nv_bfloat16* conv = nullptr;                   // [taps][channels]
     int* table = nullptr;
     std::vector<int> h_table;
     int moe = -1;       // place among the layers with experts
@@ -1009,20 +1133,26 @@ b200_status take_vectors(b200_decoder* m, int layer, std::vector<int> which, flo
   return upload_f32(all, out);
 }
 
+b200_status upload_bf16(const std::vector<uint16_t>& v, __nv_bfloat16** out) {
+  B200_CUDA_TRY(cudaMalloc((void**)out, 2 * std::max<size_t>(v.size(), 1)));
+  B200_CUDA_TRY(cudaMemcpy(*out, v.data(), 2 * v.size(), cudaMemcpyHostToDevice));
+  return B200_OK;
+}
+
 // Convolutions [channels, taps] one behind the other, as [taps][channels].
-b200_status take_conv(b200_decoder* m, int layer, std::vector<int> which, int taps, float** out) {
-  std::vector<float> all;
+b200_status take_conv(b200_decoder* m, int layer, std::vector<int> which, int taps, __nv_bfloat16** out) {
+  std::vector<uint16_t> all;
   for (int w : which) {
     std::vector<uint16_t> bits;
     b200_status st = take(m, layer, w, &bits);
     if (st != B200_OK) return st;
-    for (uint16_t b : bits) all.push_back(bf16_to_f(b));
+    all.insert(all.end(), bits.begin(), bits.end());
   }
   const size_t channels = all.size() / taps;
-  std::vector<float> t(all.size());
+  std::vector<uint16_t> t(all.size());
   for (size_t c = 0; c < channels; ++c)
     for (int k = 0; k < taps; ++k) t[k * channels + c] = all[c * taps + k];
-  return upload_f32(t, out);
+  return upload_bf16(t, out);
 }
 
 // The blocks' gate matrices, r rows then i rows, and exp's factor lru_decay * softplus(lam).
@@ -1501,14 +1631,14 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
     if (s.flags & B200_DEC_SINK_ONE) if ((st = fill(s.n_heads, 0.f, &l.sinks)) != B200_OK) return st;
     if (s.flags & B200_DEC_QK_NORM_WEIGHT)
       if ((st = fill(s.key_dim, 1.f, &l.q_norm)) != B200_OK || (st = fill(s.key_dim, 1.f, &l.k_norm)) != B200_OK) return st;
-    if (s.mixer == B200_MIX_ATTENTION && s.conv_taps > 0) if ((st = fill((size_t)l.attention_n() * s.conv_taps, 0.5f, &l.conv)) != B200_OK) return st;
+    if (s.mixer == B200_MIX_ATTENTION && s.conv_taps > 0) if ((st = upload_bf16(std::vector<uint16_t>((size_t)l.attention_n() * s.conv_taps, 0x3F00), &l.conv)) != B200_OK) return st;
     if (s.mem_heads > 0) {
       if ((st = weight(pad64(2 * s.mem_heads), c.hidden, 16 * i + 11, &l.wgates)) != B200_OK) return st;
       if ((st = fill(2 * s.mem_heads, 1.f, &l.gate_bias)) != B200_OK || (st = fill(l.mem_n(), 1.f, &l.mem_norm)) != B200_OK) return st;
     }
     if (s.mixer == B200_MIX_LRU) {
       if ((st = stack(s.n_heads, 2 * s.value_dim, l.lru_group(), 16 * i + 12, &l.wgates)) != B200_OK) return st;
-      if ((st = fill(4 * l.attn_n(), 0.1f, &l.lru_bias)) != B200_OK || (st = fill((size_t)l.attn_n() * s.conv_taps, 0.5f, &l.conv)) != B200_OK ||
+      if ((st = fill(4 * l.attn_n(), 0.1f, &l.lru_bias)) != B200_OK || (st = upload_bf16(std::vector<uint16_t>((size_t)l.attn_n() * s.conv_taps, 0x3F00), &l.conv)) != B200_OK ||
           (st = fill(l.attn_n(), 0.f, &l.conv_bias)) != B200_OK || (st = fill(l.attn_n(), 0.5f, &l.lru_rate)) != B200_OK)
         return st;
     }

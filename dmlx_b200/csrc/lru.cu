@@ -26,36 +26,52 @@ __device__ __forceinline__ float gelu_tanh(float z) {
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
-// One thread per (row, VEC channels).
-template <typename T, int VEC>
-__global__ void __launch_bounds__(256) lru_prep_kernel(LruArgs a) {
+// One thread per (R rows, VEC channels).
+template <typename T, int VEC, int R>
+__global__ void __launch_bounds__(256) lru_prep_kernel(LruArgs a, int rows) {
   const LruCall& c = a.c;
-  const int first = blockIdx.x, ch = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+  const int begin = blockIdx.x * R, end = min(begin + R, rows), ch = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
   if (ch >= c.width) return;
-  {
-    Vec<VEC> y = mat_value<T, VEC>(c.src, first, ch);
-    const Vec<VEC> b = load_vec<VEC>(c.y_bias + ch);
+  const Vec<VEC> yb = load_vec<VEC>(c.y_bias + ch), xb = load_vec<VEC>(c.x_bias + ch);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) y.v[e] = gelu_tanh(y.v[e] + b.v[e]);
-    store_vec<VEC>((T*)c.out + (size_t)first * c.out_stride + ch, y);
+  for (int r = 0; r < R; ++r) {
+    if (begin + r < end) {
+      Vec<VEC> y = mat_value<T, VEC>(c.src, begin + r, ch);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y.v[e] = gelu_tanh(y.v[e] + yb.v[e]);
+      store_vec<VEC>((T*)c.out + (size_t)(begin + r) * c.out_stride + ch, y);
+    }
   }
-  const int req = a.row_to_req[first], r0 = a.cu[req], count = a.cu[req + 1] - r0, slot = a.row_seq[first];
-  if (slot < 0 || slot >= a.max_seqs || a.pool_state[ST_ERR] != 0) return;
-  const Vec<VEC> xb = load_vec<VEC>(c.x_bias + ch);
+  if (a.pool_state[ST_ERR] != 0) return;
   auto value = [&](int row, int col) {
     Vec<VEC> v = mat_value<T, VEC>(c.src, row, c.width + col);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) v.v[e] += xb.v[e];
     return v;
   };
-  const int b = ch / a.block, o = ch - b * a.block, n = conv_rows(c.conv, first - r0, count);
-  for (int row = first; row < first + n; ++row) {
+  const int b = ch / a.block, o = ch - b * a.block;
+  auto put = [&](int row, const Vec<VEC>& v) {
     T* u = (T*)c.u + ((size_t)row * c.blocks + b) * c.u_group;
-    store_vec<VEC>(u + o, conv_value<VEC>(c.conv, value, row, row - r0, a.pos[row], slot, ch));
+    store_vec<VEC>(u + o, v);
     if (o + VEC == a.block)
       for (int z = a.block; z < c.u_group; ++z) st(u + z, 0.f);
+  };
+  if constexpr (R > 1) {
+    if (c.conv.taps == 4 && begin + R <= rows && a.row_to_req[begin] == a.row_to_req[begin + R - 1] && begin - a.cu[a.row_to_req[begin]] >= 3) {
+      Vec<VEC> v[R];
+      conv_values_inside<4, R, VEC>(c.conv, value, begin, ch, v);
+#pragma unroll
+      for (int r = 0; r < R; ++r) put(begin + r, v[r]);
+      return;
+    }
   }
-  if (first == r0) conv_update<VEC>(c.conv, value, r0, count, slot, ch);
+  for (int first = begin; first < end; ++first) {
+    const int req = a.row_to_req[first], r0 = a.cu[req], count = a.cu[req + 1] - r0, slot = a.row_seq[first];
+    if (slot < 0 || slot >= a.max_seqs) continue;
+    const int n = conv_rows(c.conv, first - r0, count);
+    for (int row = first; row < first + n; ++row) put(row, conv_value<VEC>(c.conv, value, row, row - r0, a.pos[row], slot, ch));
+    if (first == r0) conv_update<VEC>(c.conv, value, r0, count, slot, ch);
+  }
 }
 
 // SEG = 1: a thread walks all tokens of a request for one channel; otherwise a warp's lanes are 32 channels, and the block's SEG
@@ -144,9 +160,10 @@ b200_status b200_lru_prep(b200_kv* kv, LruCall c, const int32_t* d_cu, const int
   a.cu = d_cu; a.row_to_req = d_row_to_req; a.row_seq = d_row_seq; a.pos = d_pos;
   const bool v4 = a.block % 4 == 0 && c.u_group % 4 == 0 && c.out_stride % 4 == 0 && a.rec_elems % 4 == 0 && (c.src.ws || c.src.y_stride % 4 == 0);
   const int groups = v4 ? c.width / 4 : c.width, threads = std::min(256, (groups + 31) / 32 * 32);
-  auto* kernel = kv->dev.elem_bytes == 4 ? (v4 ? lru_prep_kernel<float, 4> : lru_prep_kernel<float, 1>)
-                                         : (v4 ? lru_prep_kernel<__nv_bfloat16, 4> : lru_prep_kernel<__nv_bfloat16, 1>);
-  kernel<<<dim3(total_rows, (groups + threads - 1) / threads), threads, 0, (cudaStream_t)stream>>>(a);
+  const bool many = total_rows >= 1024, f32 = kv->dev.elem_bytes == 4;
+  auto* kernel = f32 ? (v4 ? lru_prep_kernel<float, 4, 1> : lru_prep_kernel<float, 1, 1>) : (v4 ? lru_prep_kernel<__nv_bfloat16, 4, 1> : lru_prep_kernel<__nv_bfloat16, 1, 1>);
+  if (many) kernel = f32 ? (v4 ? lru_prep_kernel<float, 4, 4> : lru_prep_kernel<float, 1, 4>) : (v4 ? lru_prep_kernel<__nv_bfloat16, 4, 4> : lru_prep_kernel<__nv_bfloat16, 1, 4>);
+  kernel<<<dim3(many ? (total_rows + 3) / 4 : total_rows, (groups + threads - 1) / threads), threads, 0, (cudaStream_t)stream>>>(a, total_rows);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }

@@ -9,7 +9,7 @@
 
 struct ShortConv {
   int taps = 0, channels = 0;   // taps 0: no convolution
-  const float* w = nullptr;     // [taps][channels], the current token's last
+  const __nv_bfloat16* w = nullptr;  // [taps][channels], the current token's last
   const float* bias = nullptr;  // [channels] on the result, may be null
   float* state = nullptr;       // of slot 0
   size_t slot_elems = 0;
@@ -34,6 +34,27 @@ __device__ __forceinline__ Vec<VEC> conv_value(const ShortConv& s, F value, int 
     for (int e = 0; e < VEC; ++e) acc.v[e] = fmaf(w.v[e], u.v[e], acc.v[e]);
   }
   return acc;
+}
+
+// Results at R consecutive rows of one request that do not read the state (the first has TAPS - 1 rows before it in the step).  The
+// weights and the inputs between the rows are read once.
+template <int TAPS, int R, int VEC, typename F>
+__device__ __forceinline__ void conv_values_inside(const ShortConv& s, F value, int row, int c, Vec<VEC> (&out)[R]) {
+  Vec<VEC> u[TAPS - 1 + R], w[TAPS], bias{};
+#pragma unroll
+  for (int i = 0; i < TAPS - 1 + R; ++i) u[i] = value(row - (TAPS - 1) + i, c);
+#pragma unroll
+  for (int t = 0; t < TAPS; ++t) w[t] = load_vec<VEC>(s.w + (size_t)t * s.channels + c);
+  if (s.bias) bias = load_vec<VEC>(s.bias + c);
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    out[r] = bias;
+#pragma unroll
+    for (int t = 0; t < TAPS; ++t) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) out[r].v[e] = fmaf(w[t].v[e], u[r + t].v[e], out[r].v[e]);
+    }
+  }
 }
 
 // State behind a request whose first row in the step is r0 (entries move up, so the far ones are written first).

@@ -248,6 +248,27 @@ def test_convolutions_whose_oldest_tap_is_the_heaviest(tmp_path, taps, dtype):
         assert _close(_step(loaded, toks, portions), want, tol), portions
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_a_large_step_of_unequal_portions(tmp_path, dtype):
+    """More than a thousand rows in one step, portions that start and end anywhere among them, and a second step behind it."""
+    from dmlx_b200.serving import TokenFeeder
+
+    cfg = config(64, 90, [parallel(4, 2, 24, 40, 4, rotation(12), (2, 20, 24)), rglru(48, 2, 4),
+                          parallel(2, 1, 136, 144, 4, rotation(136), (1, 16, 16), dense(24))], alpha=1.0)
+    loaded, w = _load(tmp_path, cfg, 23, dtype, max_rows=1400, slots=8)
+    lens = (610, 1, 2, 3, 37, 500, 4)
+    prompts = {i: _tokens(cfg, n + 9, 500 + i) for i, n in enumerate(lens)}
+    feeder = TokenFeeder(loaded, 60)
+    first = feeder.step([(i, p[:-9], range(len(p) - 9)) for i, p in prompts.items()])
+    second = feeder.step([(i, p[-9:], range(9)) for i, p in prompts.items()])
+    at = 0
+    for i, n in enumerate(lens):
+        want = R.forward(prompts[i], w, cfg)
+        got = np.concatenate([first[at:at + n], second[9 * i:9 * i + 9]])
+        assert _close(got, want, _tol(dtype, w, cfg, prompts[i])), n
+        at += n
+
+
 def _special_token(cfg, w, token, coordinate=0, size=6.0):
     """One token id lights up a coordinate that is dark for all others and that no sublayer writes."""
     w["embed"][:, coordinate] = 0.0
