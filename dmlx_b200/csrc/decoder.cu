@@ -39,6 +39,7 @@
 
 namespace {
 
+constexpr int kPageTokens = 32;     // of every pool
 constexpr float kMemoryEps = 1e-6f;  // added to a matrix memory's denominator
 constexpr double kLog2e = 1.4426950408889634;
 
@@ -253,11 +254,11 @@ struct QkvArgs {
 template <typename T>
 __device__ __forceinline__ T* page_row(const QkvArgs& a, int row, int head, bool is_v) {
   const int pos = a.pos[row], seq = a.row_seq[row];
-  const int page_idx = pos / a.d.page_size, slot = pos - page_idx * a.d.page_size;
-  if (seq < 0 || seq >= a.d.max_seqs || page_idx >= a.d.seq_pages[seq]) return nullptr;
+  const int page_idx = pos / kPageTokens, slot = pos % kPageTokens;
+  if (seq < 0 || seq >= a.d.max_seqs || page_idx >= min(a.d.seq_pages[seq], a.d.max_pages_per_seq)) return nullptr;
   const int page = a.d.block_table[(size_t)seq * a.d.max_pages_per_seq + page_idx];
   char* pool = is_v ? (char*)a.d.v_pool + a.L.v_off : (char*)a.d.k_pool + a.L.k_off;
-  return (T*)pool + (((size_t)page * a.L.heads + head) * a.d.page_size + slot) * (size_t)(is_v ? a.L.vd : a.L.kd);
+  return (T*)pool + (((size_t)page * a.L.heads + head) * kPageTokens + slot) * (size_t)(is_v ? a.L.vd : a.L.kd);
 }
 
 // One warp per (row, head); q heads, then k heads, then v heads.  Grid y covers the heads, eight at a time.
@@ -399,8 +400,9 @@ __global__ void __launch_bounds__(256) decoder_qkv_conv4_kernel(QkvArgs a, int r
     }
     return v;
   };
-  auto finish = [&](int row, Vec<4> (&x)[KEEP]) {  // norm, rotation, store
-    T* dst = is_q ? (T*)a.q + (size_t)row * a.q_stride + (size_t)head * a.L.kd : page_row<T>(a, row, head, is_v);
+  auto place = [&](int row) { return is_q ? (T*)a.q + (size_t)row * a.q_stride + (size_t)head * a.L.kd : page_row<T>(a, row, head, is_v); };
+  const bool by_four = a.halves && half % 4 == 0;
+  auto finish = [&](int row, Vec<4> (&x)[KEEP], T* dst) {  // norm, rotation, store
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
@@ -430,6 +432,23 @@ __global__ void __launch_bounds__(256) decoder_qkv_conv4_kernel(QkvArgs a, int r
       for (int k = 0; k < KEEP; ++k) {
         const int c = (k * 32 + lane) * 4;
         if (c < dim) {
+          if (by_four) {
+            if (c < rot) {
+              const bool up = c >= half;
+              const int i = up ? c - half : c;
+              const Vec<4> other = load_vec<4>(sh + (up ? i : c + half));
+              const float* cs = reinterpret_cast<const float*>(a.rotation + (size_t)row * half + i);
+              const Vec<4> lo = load_vec<4>(cs), hi = load_vec<4>(cs + 4);  // cosine, sine, cosine, ..
+              const float sign = up ? 1.f : -1.f;
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const Vec<4>& v = e < 2 ? lo : hi;
+                x[k].v[e] = fmaf(sign * v.v[(2 * e + 1) & 3], other.v[e], x[k].v[e] * v.v[(2 * e) & 3]);
+              }
+            }
+            store_vec<4>(dst + c, x[k]);
+            continue;
+          }
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int i = c + e;
@@ -450,6 +469,9 @@ __global__ void __launch_bounds__(256) decoder_qkv_conv4_kernel(QkvArgs a, int r
   if constexpr (R > 1) {
     if (begin + R <= rows && a.row_to_req[begin] == a.row_to_req[begin + R - 1] && begin - a.cu[a.row_to_req[begin]] >= 3) {
       Vec<4> x[KEEP][R];
+      T* dst[R];
+#pragma unroll
+      for (int r = 0; r < R; ++r) dst[r] = place(begin + r);
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         const int c = (k * 32 + lane) * 4;
@@ -460,7 +482,7 @@ __global__ void __launch_bounds__(256) decoder_qkv_conv4_kernel(QkvArgs a, int r
         Vec<4> row[KEEP];
 #pragma unroll
         for (int k = 0; k < KEEP; ++k) row[k] = x[k][r];
-        finish(begin + r, row);
+        finish(begin + r, row, dst[r]);
       }
       return;
     }
@@ -477,7 +499,7 @@ __global__ void __launch_bounds__(256) decoder_qkv_conv4_kernel(QkvArgs a, int r
         const int c = (k * 32 + lane) * 4;
         if (c < dim) x[k] = conv_value<4>(a.conv, value, row, row - r0, pos, slot, n0 + c);
       }
-      finish(row, x);
+      finish(row, x, place(row));
     }
     if (first == r0)
       for (int c = lane * 4; c < dim; c += 128) conv_update<4>(a.conv, value, r0, count, slot, n0 + c);
