@@ -380,7 +380,7 @@ __global__ void __launch_bounds__(256) decoder_qkv_conv_kernel(QkvArgs a) {
 // The same for four taps and heads up to KEEP * 128 wide, R rows per warp: a head's row stays in registers but for the columns that are
 // rotated, and rows of one request that lie next to each other share the loads of their inputs and of the weights.
 template <typename T, int KEEP, int R>
-__global__ void __launch_bounds__(256) decoder_qkv_conv4_kernel(QkvArgs a, int rows) {
+__global__ void __launch_bounds__(256, KEEP == 1 ? 3 : 2) decoder_qkv_conv4_kernel(QkvArgs a, int rows) {
   extern __shared__ float row_sh[];  // [warp][rot]
   const int begin = blockIdx.x * R, end = min(begin + R, rows);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, H = a.L.heads, u = blockIdx.y * 8 + warp;
@@ -475,7 +475,14 @@ __global__ void __launch_bounds__(256) decoder_qkv_conv4_kernel(QkvArgs a, int r
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         const int c = (k * 32 + lane) * 4;
-        if (c < dim) conv_values_inside<4, R, 4>(a.conv, value, begin, n0 + c, x[k]);
+        if (c < dim) {
+          if (a.src.ws || a.bias) {
+            conv_values_inside<4, R, 4>(a.conv, value, begin, n0 + c, x[k]);
+          } else {  // rows the matmul wrote itself
+            const T* y = (const T*)a.src.y + (size_t)begin * a.src.y_stride;
+            conv_values_inside<4, R, 4>(a.conv, [&](int row, int col) { return load_vec<4>(y + (row - begin) * a.src.y_stride + col); }, begin, n0 + c, x[k]);
+          }
+        }
       }
 #pragma unroll
       for (int r = 0; r < R; ++r) {

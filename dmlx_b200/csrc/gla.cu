@@ -182,9 +182,9 @@ struct GateArgs {
 
 // One CTA per (request, head).  m_t = max(m_(t-1) + f_t, i_t) is a scan: the pair (F, M) stands for m -> max(m + F, M).
 template <typename T>
-__global__ void __launch_bounds__(256) memory_gates_kernel(GateArgs a) {
-  __shared__ float2 total[8];
-  __shared__ float s_m[257];
+__global__ void __launch_bounds__(1024) memory_gates_kernel(GateArgs a) {
+  __shared__ float2 total[32];
+  __shared__ float s_m[1025];
   const int req = blockIdx.x, head = blockIdx.y, H = a.g.heads, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
   const int r0 = a.cu[req], count = a.cu[req + 1] - r0;
   if (count <= 0 || a.d.state[ST_ERR] != 0) return;
@@ -791,7 +791,7 @@ b200_status b200_memory_gates(b200_kv* kv, const MemoryGates& g, const int32_t* 
   a.d = kv->dev; a.g = g; a.state = kv->dev.rec_pool + kv->lay[g.layer].rec_off; a.rec_elems = kv->lay[g.layer].rec_elems;
   a.cu = d_cu; a.row_seq = d_row_seq; a.pos = d_pos;
   auto* kernel = kv->dev.elem_bytes == 4 ? memory_gates_kernel<float> : memory_gates_kernel<__nv_bfloat16>;
-  kernel<<<dim3(n_req, g.heads), total_rows > 4 * n_req ? 256 : 32, 0, (cudaStream_t)stream>>>(a);
+  kernel<<<dim3(n_req, g.heads), total_rows > 256 * n_req ? 1024 : (total_rows > 4 * n_req ? 256 : 32), 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
