@@ -13,6 +13,15 @@
 // single decoder_rows_kernel adds it, gathers the experts' rows, averages over depth and norms for the next layer.  Experts by
 // token id are planned for all layers at the start of the step (moe.cu).
 //
+// A matrix memory beside attention shares its projection and W_o: gate matmul (f32 sums) and memory_gates_kernel, projection of both
+// branches, decoder_qkv_conv(4)_kernel (convolution, norms, rotation, pages), attention, the kernels of gla.cu.  The branches' factors ride on
+// the values and on the memory's output, so the product needs none.  Gated linear recurrence: projection, lru_prep_kernel, the blocks' gate
+// matmuls with f32 sums, lru_scan_kernel (lru.cu).  Latent queries may take a detour over a latent of their own (one more norm and matmul), and
+// a latent layer may read the pages of an earlier one.  A router's logits stay f32 sums, which route_src_kernel reads in place (moe.cu).
+//
+// With norms behind the sum decoder_rows_kernel scales the residual, adds, norms, and writes the result twice: as the residual and as the
+// operand of the next matmul.
+//
 // The residual, every norm, the biases and the logits are f32; matrix operands are bf16, or f32 with B200_DT_F32 (the same
 // kernels instantiated for float, matmuls through b200_qmm_f32, attention on CUDA cores).
 //

@@ -507,6 +507,26 @@ def test_prefix_sharing_of_layers_that_share_their_latents(tmp_path):
     assert generate(loaded, prompts, 10, prefill_chunk=32, prefix_sharing=True) == [_greedy(w, cfg, p, 10) for p in prompts]
 
 
+def test_prefix_pages_of_shared_latents_saved_and_restored(tmp_path):
+    from dmlx_b200.prefix_store import PrefixDiskStore
+
+    cfg = CASES["latent_only"]
+    loaded, _ = _load(tmp_path / "m", cfg, 96, "bfloat16")
+    toks = _tokens(cfg, 100, 8)
+    kv = loaded.new_cache(8, 4)
+    loaded.model.step(kv, [(0, 96, 0, 0)], toks[:96])
+    store = PrefixDiskStore(str(tmp_path / "pages"))
+    assert store.save_prefix(kv, 0, toks[:96]) == 3
+    fresh = loaded.new_cache(8, 4)
+    fresh.set_free_order([5, 2, 7, 0, 1, 3, 4, 6])
+    assert store.restore_prefix(fresh, 0, toks[:97]) == 96
+    out = []
+    for pool in (kv, fresh):
+        loaded.model.step(pool, [(0, 4, 96, 0)], toks[96:], [0, 1, 2, 3])
+        out.append(loaded.model.logits(1, 4))
+    np.testing.assert_array_equal(out[0], out[1])
+
+
 def test_stop_tokens_and_sampling(tmp_path):
     from dmlx_b200.serving import generate
 
