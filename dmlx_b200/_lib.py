@@ -261,7 +261,7 @@ class KvLayer(C.Structure):
 
 
 class ModelInfo(C.Structure):
-    _fields_ = [(n, i32) for n in ("vocab", "max_rows", "max_reqs", "max_seqs", "logits_f32")]
+    _fields_ = [(n, i32) for n in ("vocab", "max_rows", "max_reqs", "max_seqs", "logits_f32", "max_positions")]
 
 
 class DecoderLayer(C.Structure):
@@ -269,13 +269,15 @@ class DecoderLayer(C.Structure):
         (n, i32) for n in ("mixer", "kv_rank", "rot_dim")] + [("rot_base", f64), ("decay_rank", i32), ("decay_tau", f32)] + [
         (n, i32) for n in ("n_experts", "top_k", "expert_ffn", "n_groups", "keep_groups", "q_rank", "kv_source")] + [
         (n, f64) for n in ("yarn_factor", "yarn_original", "yarn_fast", "yarn_slow")] + [("conv_taps", i32), ("lru_decay", f32)] + [
-        (n, i32) for n in ("mem_heads", "mem_key_dim", "mem_value_dim")] + [(n, f32) for n in ("mem_gate_cap", "mix_scale", "mem_scale")]
+        (n, i32) for n in ("mem_heads", "mem_key_dim", "mem_value_dim")] + [(n, f32) for n in ("mem_gate_cap", "mix_scale", "mem_scale")] + [
+        (n, i32) for n in ("input_taps", "rel_buckets", "rel_reach")] + [("q_temp_coef", f32), ("q_temp_every", i32)] + [
+        (n, f32) for n in ("router_scale", "ff_limit", "ff_alpha", "ff_shift")]
 
 
 class DecoderConfig(C.Structure):
     _fields_ = [(n, i32) for n in ("n_layers", "hidden", "vocab", "loop_start", "loop_stop", "loop_times", "dtype", "max_rows", "max_reqs",
                                    "max_seqs")] + [("norm_eps", f32), ("embed_scale", f32), ("logit_scale", f32), ("flags", i32),
-                                   ("residual_scale", f32)]
+                                   ("residual_scale", f32), ("max_positions", i32)]
 
 
 class GlaShape(C.Structure):
@@ -283,6 +285,11 @@ class GlaShape(C.Structure):
 
 
 _sig("b200_decoder_gla", i32, vp, i32, P(GlaShape), vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, vp, i32, vp)
+class DeltaShape(C.Structure):
+    _fields_ = [(n, i32) for n in ("heads", "kv_heads", "key_dim", "value_dim", "taps")] + [("eps", f32)]
+
+
+_sig("b200_decoder_delta", i32, vp, i32, P(DeltaShape), vp, i32, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, vp, i32, vp)
 _sig("b200_kv_create_layers", i32, P(KvConfig), P(KvLayer), P(vp))
 _sig("b200_argmax_f32", i32, vp, i32, i32, vp, vp)
 _sig("b200_qmm_f32", i32, vp, vp, i32, vp, i32, i32, i32, vp)
@@ -312,7 +319,7 @@ _sig("b200_decoder_recorded_layers", i32, vp, i32, P(f32))
 _sig("b200_decoder_set_attn_mma", None, vp, i32)
 _sig("b200_decoder_model", vp, vp)
 _sig("b200_decoder_qkv", i32, vp, i32, vp, i32, vp, i32, i32, f32, vp, vp, vp, i32, vp)
-_sig("b200_decoder_attention", i32, vp, i32, vp, i32, i32, f32, vp, vp, vp, vp, i32, i32, vp, i32, vp)
+_sig("b200_decoder_attention", i32, vp, i32, vp, i32, i32, f32, vp, vp, vp, i32, vp, vp, i32, i32, vp, i32, vp)
 _sig("b200_engine_create_model", vp, vp, vp, u64)
 
 _sig("b200_request_prompt", u64, vp, P(u32), u64)

@@ -22,6 +22,8 @@ struct WinArgs {
   float* part_ml;  // [slot][q head][2]
   float scale_log2;
   const float *slopes, *sinks;
+  const float* dist = nullptr;  // [q head][dist_len]: bias by distance, times log2(e); the last one for everything further away
+  int dist_len = 0;
   __nv_bfloat16* out;
   int out_stride, out_head;  // elements between rows, between heads of a row
   int stages;                // ring slots: pages per warp, or tiles per CTA

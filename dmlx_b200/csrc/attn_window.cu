@@ -1,4 +1,4 @@
-// Paged attention for layers with a sliding window, a distance bias and a learned sink, keys and values of different
+// Paged attention for layers with a sliding window, a distance bias (linear, or by a table) and a learned sink, keys and values of different
 // widths, and any GQA group; decode rows and prefill chunks through one path.
 //
 // Rows are grouped: consecutive rows of one sequence (a prefill chunk) share a pass over the pages, a decoded token is a
@@ -340,6 +340,10 @@ __global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
     const int lo_last = first_key(it.ctx0 + it.n_rows - 1, a.window);  // the latest window start of the group
     const bool any_b = it.n_rows * hb > 8;                            // rows 8..15 of the tile carry something
     const float slA = a.slopes ? a.slopes[qhA] : 0.f, slB = a.slopes ? a.slopes[qhB] : 0.f;
+    const float *tabA = a.dist + (size_t)qhA * a.dist_len, *tabB = a.dist + (size_t)qhB * a.dist_len;  // (used with a table only)
+    const float farA = a.dist ? tabA[a.dist_len - 1] : 0.f, farB = a.dist ? tabB[a.dist_len - 1] : 0.f;
+    // the first key that some row of the group sees at a distance of its own
+    const int near_from = a.dist ? it.ctx0 - (a.dist_len - 1) : 0x7fffffff;
     uint32_t qa0[KS], qa1[KS], qa2[KS], qa3[KS];
     {
       const uint32_t* qA = reinterpret_cast<const uint32_t*>(a.q + (size_t)(it.first_row + (onA ? tokA : 0)) * a.q_stride + (size_t)qhA * a.L.kd);
@@ -382,22 +386,22 @@ __global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
       // ---- online softmax on rows g (A) and, where the tile has any, g+8 (B), each with its own window and bias ----
       const int tok0 = pg * 32;
       uint32_t ph[2][4], pl[2][4];
-      // a page every row of the group sees whole needs no masks
-      const bool edge = tok0 + 32 > it.ctx0 || tok0 < lo_last;
-      auto row_softmax = [&](auto edge_tag, auto half_tag, float& m, float& l, int ctx, int lo, float slope) -> float {
-        constexpr bool EDGE = decltype(edge_tag)::value;
+      // a page every row of the group sees whole needs no masks; beyond the reach of a distance table all keys have the same bias
+      const int kind = tok0 + 31 >= near_from ? 2 : (tok0 + 32 > it.ctx0 || tok0 < lo_last ? 1 : 0);
+      auto row_softmax = [&](auto kind_tag, auto half_tag, float& m, float& l, int ctx, int lo, float slope, float far, const float* tab) -> float {
+        constexpr bool EDGE = decltype(kind_tag)::value > 0, TABLE = decltype(kind_tag)::value == 2;
         constexpr int E0 = decltype(half_tag)::value;  // 0: row g, 1: row g + 8
         float mx = kNone;
-        const float b0 = slope * (float)(tok0 + 2 * t - (ctx - 1));  // exact integers; the bias of the lane's first key
+        const float b0 = fmaf(slope, (float)(tok0 + 2 * t - (ctx - 1)), far);  // (exact integers) the bias of the lane's first key
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) {
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            float v = sc[nt][2 * E0 + e] * a.scale_log2 + fmaf(slope, (float)(nt * 8 + e), b0);
-            if (EDGE) {
-              const int tok = tok0 + nt * 8 + 2 * t + e;
-              v = tok < ctx && tok >= lo ? v : kNone;
-            }
+            const int tok = tok0 + nt * 8 + 2 * t + e;
+            float v;
+            if constexpr (TABLE) v = fmaf(sc[nt][2 * E0 + e], a.scale_log2, tab[min(max(ctx - 1 - tok, 0), a.dist_len - 1)]);
+            else v = sc[nt][2 * E0 + e] * a.scale_log2 + fmaf(slope, (float)(nt * 8 + e), b0);
+            if (EDGE) v = tok < ctx && tok >= lo ? v : kNone;
             sc[nt][2 * E0 + e] = v;
             mx = fmaxf(mx, v);
           }
@@ -425,10 +429,15 @@ __global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
       };
       using T0 = std::integral_constant<int, 0>;
       using T1 = std::integral_constant<int, 1>;
-      float corrA, corrB = 1.f;
-      corrA = edge ? row_softmax(std::true_type{}, T0{}, mA, lA, ctxA, loA, slA) : row_softmax(std::false_type{}, T0{}, mA, lA, ctxA, loA, slA);
+      using T2 = std::integral_constant<int, 2>;
+      auto softmax = [&](auto half_tag, float& m, float& l, int ctx, int lo, float slope, float far, const float* tab) -> float {
+        if (kind == 0) return row_softmax(T0{}, half_tag, m, l, ctx, lo, slope, far, tab);
+        return kind == 1 ? row_softmax(T1{}, half_tag, m, l, ctx, lo, slope, far, tab) : row_softmax(T2{}, half_tag, m, l, ctx, lo, slope, far, tab);
+      };
+      const float corrA = softmax(T0{}, mA, lA, ctxA, loA, slA, farA, tabA);
+      float corrB = 1.f;
       if (any_b) {
-        corrB = edge ? row_softmax(std::true_type{}, T1{}, mB, lB, ctxB, loB, slB) : row_softmax(std::false_type{}, T1{}, mB, lB, ctxB, loB, slB);
+        corrB = softmax(T1{}, mB, lB, ctxB, loB, slB, farB, tabB);
       } else {
 #pragma unroll
         for (int kt = 0; kt < 2; ++kt) { ph[kt][1] = ph[kt][3] = pl[kt][1] = pl[kt][3] = 0u; }
@@ -553,7 +562,8 @@ struct SimtArgs {
   const int* row_ctx;
   int total_rows, n_q_heads, window;
   float scale;
-  const float *slopes_log2, *sinks_log2;
+  const float *slopes_log2, *sinks_log2, *dist_log2;
+  int dist_len;
   void* out;
   int out_stride, out_head_stride;
 };
@@ -580,6 +590,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(SimtArgs a) {
   const T* vp = a.L.values_in_keys ? kp : (const T*)((const char*)a.d.v_pool + a.L.v_off);
   const int v_row = a.L.values_in_keys ? a.L.kd : a.L.vd;
   const float slope = a.slopes_log2 ? a.slopes_log2[qh] : 0.f, scale = a.scale * kLog2e;
+  const float* tab = a.dist_log2 ? a.dist_log2 + (size_t)qh * a.dist_len : nullptr;
   float m = kNone, l = 0.f;
   for (int pg = lo / 32; pg * 32 < ctx; ++pg) {
     const int tok = pg * 32 + lane;
@@ -591,6 +602,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(SimtArgs a) {
       float acc = 0.f;
       for (int c = 0; c < kd; ++c) acc = fmaf(q[c], to_f(kr[c]), acc);
       s = acc * scale - slope * (float)(ctx - 1 - tok);
+      if (tab) s += tab[min(ctx - 1 - tok, a.dist_len - 1)];
     }
     float mx = s;
 #pragma unroll
@@ -757,6 +769,7 @@ b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
     SimtArgs a;
     a.d = kv->dev; a.L = L; a.q = c.q; a.q_stride = c.q_stride; a.row_seq = d_row_seq; a.row_ctx = d_row_ctx; a.total_rows = total_rows;
     a.n_q_heads = c.n_q_heads; a.window = c.window; a.scale = c.scale; a.slopes_log2 = c.slopes_log2; a.sinks_log2 = c.sinks_log2;
+    a.dist_log2 = c.dist_log2; a.dist_len = c.dist_len;
     a.out = c.out; a.out_stride = c.out_stride; a.out_head_stride = c.out_head_stride > 0 ? c.out_head_stride : L.value_dim;
     const size_t smem = sizeof(float) * 4 * (L.key_dim + L.value_dim);
     if (smem > 200 * 1024) { b200_set_error("window attention: head widths %d / %d are too large", L.key_dim, L.value_dim); return B200_ERR_UNSUPPORTED; }
@@ -774,7 +787,7 @@ b200_status b200_window_attn_run(b200_kv* kv, const WindowAttnCall& c, const int
   a.total_rows = total_rows; a.n_q_heads = c.n_q_heads; a.window = c.window;
   a.G = G; a.head_block = head_block_of(G); a.n_blocks = (G + 15) / 16;
   a.scale_log2 = c.scale * kLog2e;
-  a.slopes = c.slopes_log2; a.sinks = c.sinks_log2;
+  a.slopes = c.slopes_log2; a.sinks = c.sinks_log2; a.dist = c.dist_log2; a.dist_len = c.dist_len;
   a.out = (__nv_bfloat16*)c.out; a.out_stride = c.out_stride; a.out_head = c.out_head_stride > 0 ? c.out_head_stride : L.value_dim;
   if (L.kd <= 64) st = launch_mma_v<1>(kv, a, c.layer, s);
   else if (L.kd <= 128) st = launch_mma_v<2>(kv, a, c.layer, s);

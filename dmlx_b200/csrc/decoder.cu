@@ -22,6 +22,10 @@
 // With norms behind the sum decoder_rows_kernel scales the residual, adds, norms, and writes the result twice: as the residual and as the
 // operand of the next matmul.
 //
+// Gated delta rule: projection; delta_prep_kernel; the kernels of delta.cu and gla.cu.  Where a sublayer reads h + conv(h), decoder_rows_kernel
+// writes both in steps of single tokens; otherwise input_conv_kernel stands behind it.  A gate on a sublayer's result is a matmul from h whose
+// partial sums wait aside (b200_qmm_deferred_aside) until decoder_rows_kernel multiplies its sigmoid in, ahead of the post-norm.
+//
 // The residual, every norm, the biases and the logits are f32; matrix operands are bf16, or f32 with B200_DT_F32 (the same
 // kernels instantiated for float, matmuls through b200_qmm_f32, attention on CUDA cores).
 //
@@ -33,10 +37,12 @@
 #include <cmath>
 #include <cstring>
 #include <map>
+#include <type_traits>
 #include <vector>
 
 #include "attn_latent.cuh"
 #include "common.h"
+#include "delta.cuh"
 #include "gla.cuh"
 #include "kv_pool.cuh"
 #include "lru.cuh"
@@ -62,7 +68,12 @@ struct RowArgs {
   const __nv_bfloat16* embed = nullptr;
   int vocab = 0;
   float embed_scale = 1.f;
+  const __nv_bfloat16* pos_embed = nullptr;  // [max_positions][hidden], added to the embedding
+  int max_positions = 0;
   MatSrc src;
+  const float* src_scale = nullptr;  // factor per row on src (not on the experts)
+  MatSrc gate;                    // with a bias: src and experts are multiplied by sigmoid(gate + gate_bias), ahead of the post-norm
+  const float* gate_bias = nullptr;
   const float* post_w = nullptr;  // post-norm of the sublayer's output
   int replace = 0;                // x = src instead of x += src
   float* x = nullptr;
@@ -87,7 +98,20 @@ struct RowArgs {
   float* hist = nullptr;
   size_t hist_stride = 0;
   int n_hist = 0;
+  // rows of single tokens: hc = h + conv(h), and the convolution's state moves on
+  ShortConv conv;
+  void* hc = nullptr;
+  const int *pos = nullptr, *row_seq = nullptr, *pool_state = nullptr;
+  int max_seqs = 0;
 };
+
+// x as a later kernel finds it in an operand of this type.
+template <typename T>
+__device__ __forceinline__ float as_stored(float x) {
+  if constexpr (std::is_same_v<T, float>) return x;
+  else return __bfloat162float(__float2bfloat16(x));
+}
+__device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // One CTA per row: sublayer output -> residual stream -> what the next matmul reads.  NQ > 0: a thread keeps its NQ
 // groups of VEC columns in registers and asks for the residual before the first reduction; NQ = 0: any width, the row
@@ -127,7 +151,14 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
     each([&](int i, int k) {
       Vec<VEC> v = load_vec<VEC>(e + i * VEC);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) { v.v[j] *= a.embed_scale; ss += v.v[j] * v.v[j]; }
+      for (int j = 0; j < VEC; ++j) v.v[j] *= a.embed_scale;
+      if (a.pos_embed) {
+        const Vec<VEC> p = load_vec<VEC>(a.pos_embed + (size_t)min(a.pos[row], a.max_positions - 1) * a.hidden + i * VEC);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v.v[j] += p.v[j];
+      }
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) ss += v.v[j] * v.v[j];
       put(i, k, v);
       store_vec<VEC>(xr + i * VEC, v);
       if (x0r) store_vec<VEC>(x0r + i * VEC, v);
@@ -135,12 +166,15 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
     });
   } else {
     float ys = 0.f;
+    const float src_scale = a.src_scale ? a.src_scale[row] : 1.f;
     Vec<VEC> res[NQ > 0 ? NQ : 1];
     each([&](int i, int k) {
       if constexpr (NQ > 0) { if (!a.replace) res[k] = load_vec<VEC>(xr + i * VEC); }
       Vec<VEC> v;
       if (a.src.ws || a.src.y) {
         v = mat_value<T, VEC>(a.src, row, i * VEC);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v.v[j] *= src_scale;
       } else {
 #pragma unroll
         for (int j = 0; j < VEC; ++j) v.v[j] = 0.f;
@@ -150,6 +184,11 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
         const float w = a.moe_wts ? a.moe_wts[row * a.moe_k + m] : a.moe_w;
 #pragma unroll
         for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(w, e.v[j], v.v[j]);
+      }
+      if (a.gate_bias) {
+        const Vec<VEC> z = mat_value<T, VEC>(a.gate, row, i * VEC), b = load_vec<VEC>(a.gate_bias + i * VEC);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v.v[j] *= sigmoid(z.v[j] + b.v[j]);
       }
 #pragma unroll
       for (int j = 0; j < VEC; ++j) ys += v.v[j] * v.v[j];
@@ -197,12 +236,36 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
   if (a.norm_w) {
     const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)a.hidden + a.eps);
     T* hr = (T*)a.h + (size_t)row * a.h_stride;
+    const int slot = a.hc ? a.row_seq[row] : 0;
+    const bool conv = a.hc && slot >= 0 && slot < a.max_seqs && a.pool_state[ST_ERR] == 0;
+    const int back = conv ? min(a.conv.taps - 1, a.pos[row]) : 0;
     each([&](int i, int k) {
       Vec<VEC> v = get(i, k);
       const Vec<VEC> w = load_vec<VEC>(a.norm_w + i * VEC);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) v.v[j] *= r * w.v[j];
       store_vec<VEC>(hr + i * VEC, v);
+      if (conv) {
+        float* state = a.conv.state + (size_t)slot * a.conv.slot_elems + i * VEC;
+        Vec<VEC> own, acc{};
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) own.v[j] = as_stored<T>(v.v[j]);
+        Vec<VEC> carried = own;  // entries move up by one
+        for (int d = 1; d < a.conv.taps; ++d) {
+          const Vec<VEC> u = load_vec<VEC>(state + (size_t)(d - 1) * a.conv.channels);
+          store_vec<VEC>(state + (size_t)(d - 1) * a.conv.channels, carried);
+          carried = u;
+          if (d <= back) {
+            const Vec<VEC> tap = load_vec<VEC>(a.conv.w + (size_t)(a.conv.taps - 1 - d) * a.conv.channels + i * VEC);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) acc.v[j] = fmaf(tap.v[j], u.v[j], acc.v[j]);
+          }
+        }
+        const Vec<VEC> tap = load_vec<VEC>(a.conv.w + (size_t)(a.conv.taps - 1) * a.conv.channels + i * VEC);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) acc.v[j] = own.v[j] + fmaf(tap.v[j], own.v[j], acc.v[j]);
+        store_vec<VEC>((T*)a.hc + (size_t)row * a.h_stride + i * VEC, acc);
+      }
       if (a.norm_x) store_vec<VEC>(xr + i * VEC, v);
     });
   }
@@ -219,6 +282,60 @@ template <typename T>
 void (*rows_kernel(int vec, int nq))(RowArgs) {
   if (vec == 1) return decoder_rows_kernel<T, 1, 0>;
   return nq <= 1 ? decoder_rows_kernel<T, 4, 1> : (nq <= 2 ? decoder_rows_kernel<T, 4, 2> : (nq <= 4 ? decoder_rows_kernel<T, 4, 4> : decoder_rows_kernel<T, 4, 0>));
+}
+
+// hc = h + conv(h) over the rows of a step, portions of any length.  One thread per (R rows, VEC channels).
+struct InputConvArgs {
+  ShortConv conv;
+  const void* h;
+  void* hc;
+  int hidden, stride, max_seqs;
+  const int *pool_state, *cu, *row_to_req, *row_seq, *pos;
+};
+
+template <typename T, int VEC, int TAPS, int R>
+__global__ void __launch_bounds__(256) input_conv_kernel(InputConvArgs a, int rows) {
+  const int begin = blockIdx.x * R, end = min(begin + R, rows), ch = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+  if (ch >= a.hidden || a.pool_state[ST_ERR] != 0) return;
+  auto value = [&](int row, int col) { return load_vec<VEC>((const T*)a.h + (size_t)row * a.stride + col); };
+  auto put = [&](int row, Vec<VEC> y) {
+    const Vec<VEC> x = value(row, ch);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) y.v[e] += x.v[e];
+    store_vec<VEC>((T*)a.hc + (size_t)row * a.stride + ch, y);
+  };
+  if constexpr (R > 1 && TAPS > 0) {
+    if (begin + R <= rows && a.row_to_req[begin] == a.row_to_req[begin + R - 1] && begin - a.cu[a.row_to_req[begin]] >= TAPS - 1) {
+      Vec<VEC> y[R];
+      conv_values_inside<TAPS, R, VEC>(a.conv, value, begin, ch, y);
+#pragma unroll
+      for (int r = 0; r < R; ++r) put(begin + r, y[r]);
+      return;
+    }
+  }
+  for (int first = begin; first < end; ++first) {
+    const int req = a.row_to_req[first], r0 = a.cu[req], count = a.cu[req + 1] - r0, slot = a.row_seq[first];
+    if (slot < 0 || slot >= a.max_seqs) continue;
+    const int n = conv_rows(a.conv, first - r0, count);
+    for (int row = first; row < first + n; ++row) put(row, conv_value<VEC>(a.conv, value, row, row - r0, a.pos[row], slot, ch));
+    if (first == r0) conv_update<VEC>(a.conv, value, r0, count, slot, ch);
+  }
+}
+
+b200_status launch_input_conv(const InputConvArgs& a, int rows, bool f32, cudaStream_t s) {
+  const bool v4 = a.hidden % 4 == 0 && a.stride % 4 == 0 && a.conv.slot_elems % 4 == 0, many = rows >= 256 && v4 && !f32;
+  const int groups = v4 ? a.hidden / 4 : a.hidden, threads = std::min(256, (groups + 31) / 32 * 32);
+  auto run = [&](auto* kernel, int per) -> b200_status {
+    kernel<<<dim3((rows + per - 1) / per, (groups + threads - 1) / threads), threads, 0, s>>>(a, rows);
+    B200_LAUNCH_CHECK();
+    return B200_OK;
+  };
+  using B = __nv_bfloat16;
+  if (many && a.conv.taps == 2) return run(input_conv_kernel<B, 4, 2, 4>, 4);
+  if (many && a.conv.taps == 3) return run(input_conv_kernel<B, 4, 3, 4>, 4);
+  if (many && a.conv.taps == 4) return run(input_conv_kernel<B, 4, 4, 4>, 4);
+  if (f32) return v4 ? run(input_conv_kernel<float, 4, 0, 1>, 1) : run(input_conv_kernel<float, 1, 0, 1>, 1);
+  return v4 ? run(input_conv_kernel<B, 4, 0, 1>, 1) : run(input_conv_kernel<B, 1, 0, 1>, 1);
 }
 
 // Rows idx[r] of x, normalised, as the head's operand.
@@ -256,6 +373,10 @@ struct QkvArgs {
   const float2* rotation = nullptr;
   int rot = 0, halves = 0;
   float v_scale = 1.f;
+  // norms over the whole projection, query temperature, queries alone: decoder_qkv_row_kernel
+  bool norm_row = false, keys = true;
+  float temp_coef = 0.f;
+  int temp_every = 0;  // 0: none
 };
 
 // Where key or value head `head` of a row lives in its page; null when the step's reservation failed (nothing is written then, the
@@ -522,7 +643,78 @@ __global__ void __launch_bounds__(256, KEEP == 1 ? 3 : 2) decoder_qkv_conv4_kern
   }
 }
 
+// The same where a row's norms span all heads of q and of k: one CTA per row, which waits in shared memory for its sums of squares.  The queries are
+// also scaled by a temperature that grows with the position; without keys there are queries only.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) decoder_qkv_row_kernel(QkvArgs a) {
+  extern __shared__ __align__(16) float row_sh[];
+  __shared__ float part[32];
+  const int row = blockIdx.x, H = a.keys ? a.L.heads : 0, dim = a.L.key_dim, nq = a.hq * dim, nqk = nq + H * dim, all = nqk + H * a.L.value_dim;
+  const int pos = a.pos[row];
+  T *q = (T*)a.q + (size_t)row * a.q_stride, *kr = nullptr, *vr = nullptr;
+  if (a.keys) {
+    kr = page_row<T>(a, row, 0, false);
+    if (!kr) return;
+    vr = page_row<T>(a, row, 0, true);
+  }
+  const size_t k_head = (size_t)kPageTokens * a.L.kd, v_head = (size_t)kPageTokens * a.L.vd;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * VEC; c < all; c += 256 * VEC) {
+    Vec<VEC> v = mat_value<T, VEC>(a.src, row, c);
+    if (a.bias) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v.v[e] += a.bias[c + e];
+    }
+    if (c >= nqk) {
+      const int head = (c - nqk) / a.L.value_dim;
+      store_vec<VEC>(vr + head * v_head + (c - nqk - head * a.L.value_dim), v);
+      continue;
+    }
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) s += v.v[e] * v.v[e];
+    if (c < nq) sq += s;
+    else sk += s;
+    store_vec<VEC>(row_sh + c, v);
+  }
+  float rq = 1.f, rk = 1.f;
+  if (a.norm_row) {
+    rq = 1.0f / sqrtf(block_sum(sq, part) / (float)nq + a.eps);
+    __syncthreads();
+    if (a.keys) rk = 1.0f / sqrtf(block_sum(sk, part) / (float)(nqk - nq) + a.eps);
+  }
+  if (a.temp_every > 0) rq *= 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1));
+  for (int c = threadIdx.x * VEC; c < nqk; c += 256 * VEC) {  // (a thread reads what it wrote)
+    const bool is_q = c < nq;
+    const int k = is_q ? c : c - nq, head = k / dim;
+    Vec<VEC> v = load_vec<VEC>(row_sh + c);
+    const float* w = is_q ? a.q_norm : a.k_norm;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v.v[e] *= (is_q ? rq : rk) * (w ? w[k + e] : 1.f);
+    store_vec<VEC>((is_q ? q + (size_t)head * a.L.kd : kr + head * k_head) + (k - head * dim), v);
+  }
+  for (int i = threadIdx.x; i < (a.hq + H) * (a.L.kd - dim); i += 256) {  // padding behind a head
+    const int u = i / (a.L.kd - dim), c = dim + i - u * (a.L.kd - dim);
+    st((u < a.hq ? q + (size_t)u * a.L.kd : kr + (u - a.hq) * k_head) + c, 0.f);
+  }
+  for (int i = threadIdx.x; i < H * (a.L.vd - a.L.value_dim); i += 256) {
+    const int u = i / (a.L.vd - a.L.value_dim);
+    st(vr + u * v_head + a.L.value_dim + i - u * (a.L.vd - a.L.value_dim), 0.f);
+  }
+}
+
 b200_status launch_qkv(const QkvArgs& a, int rows, cudaStream_t s) {
+  if (a.norm_row || a.temp_every > 0 || !a.keys) {
+    const bool vec = a.L.key_dim % 4 == 0 && a.L.value_dim % 4 == 0 && (a.src.ws || a.src.y_stride % 4 == 0);
+    const size_t smem = sizeof(float) * (a.hq + (a.keys ? a.L.heads : 0)) * (size_t)a.L.key_dim;
+    if (smem > 200 * 1024) { b200_set_error("decoder: %d heads of %d are too wide for a row's norm", a.hq, a.L.key_dim); return B200_ERR_UNSUPPORTED; }
+    auto* kernel = a.d.elem_bytes == 4 ? (vec ? decoder_qkv_row_kernel<float, 4> : decoder_qkv_row_kernel<float, 1>)
+                                       : (vec ? decoder_qkv_row_kernel<__nv_bfloat16, 4> : decoder_qkv_row_kernel<__nv_bfloat16, 1>);
+    if (smem > 48 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    kernel<<<rows, 256, smem, s>>>(a);
+    B200_LAUNCH_CHECK();
+    return B200_OK;
+  }
   if (a.conv.taps > 0 || a.q_norm || a.rot > 0 || a.v_scale != 1.f) {
     const bool vec = a.L.key_dim % 4 == 0 && a.L.value_dim % 4 == 0 && (a.src.ws || a.src.y_stride % 4 == 0) && a.conv.slot_elems % 4 == 0 &&
                      a.conv.channels % 4 == 0;
@@ -574,7 +766,10 @@ const char* kTensorNames[] = {"q", "k", "v", "o", "gate", "up", "down", "head", 
                               "k convolution", "v convolution", "memory q", "memory k", "memory v", "memory output gate", "memory output",
                               "memory input gate", "memory forget gate", "memory input gate bias", "memory forget gate bias", "memory norm",
                               "lru branch", "lru branch bias", "lru input", "lru input bias", "lru convolution", "lru convolution bias",
-                              "lru decay gate", "lru decay gate bias", "lru input gate", "lru input gate bias", "lru lambda", "router"};
+                              "lru decay gate", "lru decay gate bias", "lru input gate", "lru input gate bias", "lru lambda", "router",
+                              "positions", "distance table", "input convolution 1", "input convolution 2", "result gate 1", "result gate 2",
+                              "result gate bias 1", "result gate bias 2", "beta", "decay", "decay rate", "decay bias", "shared expert gate"};
+static_assert(sizeof(kTensorNames) / sizeof(kTensorNames[0]) == B200_DEC_LAST_TENSOR + 1, "a name per tensor");
 
 }  // namespace
 
@@ -591,6 +786,12 @@ struct b200_decoder : b200_model {
     float *dq_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr, *conv_bias = nullptr, *gate_bias = nullptr, *mem_norm = nullptr;
     float *lru_bias = nullptr, *lru_rate = nullptr;  // [y | x | r | i], [width]
     __nv_bfloat16* conv = nullptr;                   // [taps][channels]
+    // of the two sublayers: convolution of what they read, gate on their result
+    __nv_bfloat16* in_conv[2] = {};
+    b200_qweight* wgate[2] = {};
+    float* out_gate_bias[2] = {};
+    float *dist = nullptr, *rate = nullptr, *dt_bias = nullptr;  // bias by distance, [heads][dist_len]; of the delta rule, [heads]
+    int dist_len = 0, hidden = 0;
     int* table = nullptr;
     std::vector<int> h_table;
     int moe = -1;       // place among the layers with experts
@@ -598,28 +799,41 @@ struct b200_decoder : b200_model {
     int qkv_n() const {
       if (s.mixer == B200_MIX_LATENT) return (s.q_rank > 0 ? s.q_rank : q_n()) + (s.kv_source > 0 ? 0 : s.kv_rank + s.rot_dim);
       if (s.mixer == B200_MIX_LRU) return 2 * attn_n();
+      if (delta()) return b200_delta_channels(s.n_heads, s.n_kv_heads, s.key_dim, s.value_dim) + s.n_heads * (s.value_dim + 2);
       if (s.mixer == B200_MIX_GLA) return 2 * s.n_heads * (s.key_dim + s.value_dim) + s.decay_rank;
       return attention_n() + 2 * s.mem_heads * (s.mem_key_dim + s.mem_value_dim);
     }
     int q_n() const { return s.n_heads * (s.key_dim + s.rot_dim); }  // queries of latent attention
-    int attention_n() const { return s.n_heads * s.key_dim + s.n_kv_heads * (s.key_dim + s.value_dim); }
+    bool delta() const { return s.mixer == B200_MIX_DELTA; }
+    int attention_n() const { return s.n_heads * s.key_dim + (s.kv_source > 0 ? 0 : s.n_kv_heads * (s.key_dim + s.value_dim)); }
     int mem_n() const { return s.mem_heads * s.mem_value_dim; }
     int mem_col() const { return pad64(attn_n()); }
     int router_n() const { return s.flags & B200_DEC_ROUTER ? s.n_experts : 0; }
     // state of a slot: the matrix memory, then the convolution's inputs
     int conv_off() const { return s.mem_heads > 0 ? (b200_memory_elems(s.mem_heads, s.mem_key_dim, s.mem_value_dim) + 3) / 4 * 4 : 0; }
-    int state_elems() const {
+    int mixer_elems() const {
       int n = 0;
+      if (delta()) n = (b200_delta_elems(s.n_heads, s.n_kv_heads, s.key_dim, s.value_dim, s.conv_taps) + 3) / 4 * 4;
       if (s.mixer == B200_MIX_GLA) n = s.n_heads * s.key_dim * s.value_dim;
       if (s.mixer == B200_MIX_LRU) n = (b200_lru_elems(attn_n(), s.conv_taps) + 3) / 4 * 4;
       if (s.mixer == B200_MIX_ATTENTION) n = (conv_off() + (s.conv_taps > 1 ? s.conv_taps - 1 : 0) * attention_n() + 3) / 4 * 4;
       return n;
     }
+    // behind the mixer's part: inputs of the convolutions in front of the sublayers
+    bool second() const { return (s.ffn > 0 || s.n_experts > 0) && !parallel(); }
+    int in_conv_off(int which) const { return (mixer_elems() + 3) / 4 * 4 + which * (s.input_taps - 1) * hidden; }
+    int state_elems() const {
+      if (s.input_taps < 2) return mixer_elems();
+      return (in_conv_off(second() ? 2 : 1) + 3) / 4 * 4;
+    }
     int lru_group() const { return pad64(s.value_dim); }
     int attn_n() const { return s.n_heads * s.value_dim; }
     bool parallel() const { return (s.flags & B200_DEC_PARALLEL) != 0; }
     bool gelu() const { return (s.flags & B200_DEC_FF_GELU) != 0; }
-    int epilogue() const { return gelu() ? B200_EPI_GELU : B200_EPI_SWIGLU; }
+    bool plain_ff() const { return (s.flags & (B200_DEC_FF_GELU | B200_DEC_FF_RELU2)) != 0; }  // without a gate
+    int epilogue() const { return gelu() ? B200_EPI_GELU : (plain_ff() ? B200_EPI_RELU2 : B200_EPI_SWIGLU); }
+    SwigluShape swiglu() const { return SwigluShape{s.ff_limit, s.ff_alpha > 0.f ? s.ff_alpha : 1.f, s.ff_shift}; }
+    bool shared_gate() const { return (s.flags & B200_DEC_SHARED_GATE) != 0; }
     int ffn_col() const { return mem_col() + (s.mem_heads > 0 ? pad64(mem_n()) : 0); }
     int out_k() const { return ffn_col() + (parallel() && s.ffn > 0 ? pad64(s.ffn) : 0); }  // columns wo reads
     int plain_stride() const { return pad64(s.key_dim); }
@@ -632,13 +846,15 @@ struct b200_decoder : b200_model {
       }
       if (s.mixer == B200_MIX_LRU) return {B200_DEC_W_LRU_Y, B200_DEC_W_LRU_X};
       if (s.mixer == B200_MIX_GLA) return {B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V, B200_DEC_W_OUT_GATE, B200_DEC_W_A1};
+      if (delta()) return {B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V, B200_DEC_W_OUT_GATE, B200_DEC_W_BETA, B200_DEC_W_DECAY};
+      if (s.kv_source > 0) return {B200_DEC_W_Q};
       std::vector<int> w{B200_DEC_W_Q, B200_DEC_W_K, B200_DEC_W_V};
       if (s.mem_heads > 0) w.insert(w.end(), {B200_DEC_W_MEM_Q, B200_DEC_W_MEM_K, B200_DEC_W_MEM_V, B200_DEC_W_MEM_G});
       return w;
     }
     b200_kv_layer cache() const {
-      if (s.mixer == B200_MIX_LATENT) return s.kv_source > 0 ? b200_kv_layer{0, 0, 0, 0, 0} : b200_kv_layer{1, s.kv_rank + s.rot_dim, s.kv_rank, 1, 0};
-      if (s.mixer == B200_MIX_GLA || s.mixer == B200_MIX_LRU) return b200_kv_layer{0, 0, 0, 0, state_elems()};
+      if (s.mixer == B200_MIX_LATENT && s.kv_source == 0) return b200_kv_layer{1, s.kv_rank + s.rot_dim, s.kv_rank, 1, state_elems()};
+      if (s.mixer == B200_MIX_GLA || s.mixer == B200_MIX_LRU || delta() || s.kv_source > 0) return b200_kv_layer{0, 0, 0, 0, state_elems()};
       return b200_kv_layer{s.n_kv_heads, s.key_dim, s.value_dim, 0, state_elems()};
     }
   };
@@ -667,12 +883,16 @@ struct b200_decoder : b200_model {
   struct Run { int layer; bool opens; };  // opens: the first layer of a pass of the loop
   std::vector<Run> runs;
   std::map<std::pair<int, int>, HostTensor> staged;
-  __nv_bfloat16* embed = nullptr;
+  __nv_bfloat16 *embed = nullptr, *pos_embed = nullptr;
   float* final_norm = nullptr;
   b200_qweight *head = nullptr, *loop_in = nullptr;
   // activations: residual and embedding output in f32, operands in the model's type
   float *x = nullptr, *x0 = nullptr, *rec = nullptr;
   void *h = nullptr, *cat = nullptr, *y = nullptr, *q = nullptr, *attn = nullptr, *act = nullptr, *last = nullptr;
+  void *hc = nullptr, *gate_y = nullptr;  // h + conv(h); rows of a result's gate where the matmul writes them itself
+  float* shared_w = nullptr;              // weight of a token's shared expert
+  b200_kv* step_kv = nullptr;             // of the step in flight
+  int step_reqs = 0;
   int hp = 0, catp = 0;  // padded widths of h and [x ; x0]
   bool attn_mma = true, recording = false;
 
@@ -683,7 +903,9 @@ struct b200_decoder : b200_model {
   b200_status run_layers(b200_kv* kv, int n_req, int T, int n_logits, void* stream) override;
   b200_status reserve_logit_rows(int rows) override;
   b200_status matmul(const b200_qweight* w, const void* in, int rows, int defer, MatSrc* src, void* stream);
-  b200_status rows_step(RowArgs a, int rows, int next, cudaStream_t s);
+  b200_status rows_step(RowArgs a, int rows, int next, cudaStream_t s, int run = -1, int which = 0);
+  b200_status result_gate(const Layer& l, int which, int rows, MatSrc* src, void* stream);
+  const void* in_of(const Layer& l) const { return l.s.input_taps > 0 ? hc : h; }  // what a sublayer's matmuls read
   b200_status attention(b200_kv* kv, int run, int rows, void* stream);
   b200_status mixer(b200_kv* kv, int run, int n_req, int T, void* stream);
   b200_status memory(b200_kv* kv, int run, const MatSrc& src, int n_req, int T, void* stream);
@@ -696,13 +918,15 @@ struct b200_decoder : b200_model {
 };
 
 b200_decoder::~b200_decoder() {
-  void* dev[] = {embed, final_norm, x, x0, rec, h, cat, y, q, attn, act, last, q_plain, lat_out, hist, moe_x, moe_act, moe_y, d_moe, q_latent, lru_gates, moe_wts, mem_gates};
+  void* dev[] = {embed, final_norm, x, x0, rec, h, cat, y, q, attn, act, last, q_plain, lat_out, hist, moe_x, moe_act, moe_y, d_moe, q_latent, lru_gates, moe_wts, mem_gates,
+                 pos_embed, hc, gate_y, shared_w};
   for (void* p : dev) if (p) cudaFree(p);
   for (Layer& l : layers) {
     void* lp[] = {l.bias, l.sinks, l.slopes, l.norm1, l.norm2, l.post1, l.post2, l.dkv_norm, l.a2, l.a2_bias, l.head_norm, l.depth, l.table,
-                  l.dq_norm, l.q_norm, l.k_norm, l.conv, l.conv_bias, l.gate_bias, l.mem_norm, l.lru_bias, l.lru_rate};
+                  l.dq_norm, l.q_norm, l.k_norm, l.conv, l.conv_bias, l.gate_bias, l.mem_norm, l.lru_bias, l.lru_rate,
+                  l.in_conv[0], l.in_conv[1], l.out_gate_bias[0], l.out_gate_bias[1], l.dist, l.rate, l.dt_bias};
     for (void* p : lp) if (p) cudaFree(p);
-    for (b200_qweight* w : {l.wqkv, l.wo, l.wgu, l.wdown, l.wuk, l.wuv, l.we_gu, l.we_down, l.wuq, l.wgates, l.wrouter}) b200_qweight_destroy(w);
+    for (b200_qweight* w : {l.wqkv, l.wo, l.wgu, l.wdown, l.wuk, l.wuv, l.we_gu, l.we_down, l.wuq, l.wgates, l.wrouter, l.wgate[0], l.wgate[1]}) b200_qweight_destroy(w);
   }
   for (MoeTableLayer& t : moe) {
     void* tp[] = {t.indices, t.offsets, t.order, t.inv_order, t.n_items, t.items};
@@ -751,9 +975,22 @@ b200_status b200_decoder::matmul(const b200_qweight* w, const void* in, int rows
   return st;
 }
 
+// Gate on the result of a sublayer, from the h it is given.
+b200_status b200_decoder::result_gate(const Layer& l, int which, int rows, MatSrc* src, void* stream) {
+  const b200_qweight* w = l.wgate[which];
+  *src = MatSrc{};
+  src->y = gate_y;
+  src->y_stride = w->n;
+  if (f32()) return b200_qmm_f32(w, (const float*)h, rows, (float*)gate_y, w->n, w->n, B200_EPI_NONE, stream);
+  b200_qmm_partials p;
+  const b200_status st = b200_qmm_deferred_aside(w, h, rows, gate_y, 1, stream, &p);
+  if (st == B200_OK && p.pending) { src->ws = p.d_ws; src->splits = p.splits; src->tn = p.tn; src->tts = p.tts; }
+  return st;
+}
+
 // decoder_rows_kernel with what run `next` reads (its first norm, or [x ; x0] when it opens a pass; nothing past the end).
-// next < 0: a.norm_w is already set.
-b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t s) {
+// next < 0: a.norm_w is already set, for sublayer `which` of run `run`.  The convolution of what a sublayer reads is done here as well.
+b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t s, int run, int which) {
   a.hidden = cfg.hidden;
   a.eps = cfg.norm_eps;
   a.x = x;
@@ -767,7 +1004,25 @@ b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t 
     a.x_scale = cfg.residual_scale;
   } else if (next >= 0 && next < (int)runs.size()) {
     if (runs[next].opens) { a.cat = cat; a.cat_stride = catp; }
-    else a.norm_w = layers[runs[next].layer].norm1;
+    else {
+      a.norm_w = layers[runs[next].layer].norm1;
+      run = next;
+      which = 0;
+    }
+  }
+  a.pos = d_pos;
+  InputConvArgs ic{};
+  if (run >= 0 && layers[runs[run].layer].s.input_taps > 0) {
+    const Layer& l = layers[runs[run].layer];
+    const KvLayerDev& L = step_kv->lay[run];
+    ic.conv.taps = l.s.input_taps; ic.conv.channels = cfg.hidden; ic.conv.w = l.in_conv[which];
+    ic.conv.state = step_kv->dev.rec_pool + L.rec_off + l.in_conv_off(which); ic.conv.slot_elems = L.rec_elems;
+    if (rows == step_reqs) {  // a token per request
+      a.conv = ic.conv; a.hc = hc; a.row_seq = d_row_seq; a.pool_state = step_kv->dev.state; a.max_seqs = step_kv->dev.max_seqs;
+    } else {
+      ic.h = h; ic.hc = hc; ic.hidden = cfg.hidden; ic.stride = hp; ic.max_seqs = step_kv->dev.max_seqs; ic.pool_state = step_kv->dev.state;
+      ic.cu = d_cu; ic.row_to_req = d_row_to_req; ic.row_seq = d_row_seq; ic.pos = d_pos;
+    }
   }
   const int vec = cfg.hidden % 4 == 0 ? 4 : 1;
   const int threads = std::min(rows >= 512 ? 256 : 512, (cfg.hidden / vec + 31) / 32 * 32), nq = (cfg.hidden / vec + threads - 1) / threads;
@@ -776,7 +1031,7 @@ b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t 
   if (smem > 47 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   kernel<<<rows, threads, smem, s>>>(a);
   B200_LAUNCH_CHECK();
-  return B200_OK;
+  return ic.hc ? launch_input_conv(ic, rows, f32(), s) : B200_OK;
 }
 
 b200_status b200_decoder::attention(b200_kv* kv, int run, int rows, void* stream) {
@@ -790,6 +1045,8 @@ b200_status b200_decoder::attention(b200_kv* kv, int run, int rows, void* stream
   c.scale = l.s.scale;
   c.slopes_log2 = l.slopes;
   c.sinks_log2 = l.sinks;
+  c.dist_log2 = l.dist;
+  c.dist_len = l.dist_len;
   c.out = attn;
   c.out_stride = l.out_k();
   if (l.s.mixer == B200_MIX_LATENT) {
@@ -813,11 +1070,13 @@ b200_status b200_decoder::begin_step(b200_kv* kv, int n_req, int T, int tile_row
   b200_decoder* m = this;
   cudaStream_t cs = (cudaStream_t)stream;
   b200_status st = B200_OK;
+  step_kv = kv;
+  step_reqs = n_req;
   // one plan per (window, GQA group) of the stack, shared by its layers (latent layers: of the same key width)
   std::vector<std::tuple<int, int, int>> planned;
   for (size_t r = 0; r < runs.size(); ++r) {
     const b200_decoder_layer& s = layers[runs[r].layer].s;
-    if (s.mixer == B200_MIX_GLA || s.mixer == B200_MIX_LRU) continue;
+    if (s.mixer == B200_MIX_GLA || s.mixer == B200_MIX_LRU || s.mixer == B200_MIX_DELTA) continue;
     const bool latent = s.mixer == B200_MIX_LATENT;
     const int pages_of = kv_run((int)r);
     const std::tuple<int, int, int> key{s.window, latent ? s.n_heads : s.n_heads / s.n_kv_heads, latent ? kv->lay[pages_of].kd : 0};
@@ -844,13 +1103,22 @@ b200_status b200_decoder::mixer(b200_kv* kv, int run, int n_req, int T, void* st
   b200_status st = B200_OK;
   MatSrc src;
   if (s.mem_heads > 0) {  // the gates' sums stay f32, and are used up before the next product
-    MODEL_STEP_CAT(1, matmul(l.wgates, h, T, 2, &src, stream));
+    MODEL_STEP_CAT(1, matmul(l.wgates, in_of(l), T, 2, &src, stream));
     MemoryGates g;
     g.layer = run; g.heads = s.mem_heads; g.m_off = s.mem_heads * s.mem_key_dim * b200_memory_width(s.mem_value_dim);
     g.src = src; g.bias = l.gate_bias; g.cap = s.mem_gate_cap; g.out = mem_gates;
     MODEL_STEP_CAT(0, b200_memory_gates(kv, g, d_cu, d_row_seq, d_pos, n_req, T, stream));
   }
-  MODEL_STEP_CAT(1, matmul(l.wqkv, h, T, 1, &src, stream));
+  MODEL_STEP_CAT(1, matmul(l.wqkv, in_of(l), T, 1, &src, stream));
+  if (l.delta()) {
+    DeltaCall c;
+    c.layer = run; c.heads = s.n_heads; c.kv_heads = s.n_kv_heads; c.dk = s.key_dim; c.dv = s.value_dim; c.src = src;
+    c.conv.taps = s.conv_taps; c.conv.w = l.conv; c.rate = l.rate; c.dt_bias = l.dt_bias; c.norm = l.head_norm; c.eps = cfg.norm_eps;
+    c.out = attn; c.out_stride = l.out_k();
+    MODEL_STEP_CAT(2, b200_delta_prep(kv, gla, c, d_cu, d_row_to_req, d_row_seq, d_pos, T, stream));
+    MODEL_STEP_CAT(0, b200_delta_run(kv, gla, c, d_cu, d_row_seq, d_pos, n_req, T, attn_mma, stream));
+    return B200_OK;
+  }
   if (s.mixer == B200_MIX_LRU) return lru(kv, run, src, n_req, T, stream);
   if (s.mixer == B200_MIX_GLA) {
     GlaCall c;
@@ -887,8 +1155,9 @@ b200_status b200_decoder::mixer(b200_kv* kv, int run, int n_req, int T, void* st
     return B200_OK;
   }
   QkvArgs a;
-  a.d = kv->dev; a.L = kv->lay[run]; a.src = src; a.bias = l.bias; a.hq = s.n_heads; a.qk_norm = s.flags & B200_DEC_QK_NORM ? 1 : 0;
-  a.eps = cfg.norm_eps; a.q = q; a.q_stride = s.n_heads * kv->lay[run].kd; a.pos = d_pos; a.row_seq = d_row_seq;
+  a.d = kv->dev; a.L = kv->lay[kv_run(run)]; a.src = src; a.bias = l.bias; a.hq = s.n_heads; a.qk_norm = s.flags & B200_DEC_QK_NORM ? 1 : 0;
+  a.norm_row = (s.flags & B200_DEC_QK_NORM_ROW) != 0; a.keys = s.kv_source == 0; a.temp_coef = s.q_temp_coef; a.temp_every = s.q_temp_every;
+  a.eps = cfg.norm_eps; a.q = q; a.q_stride = s.n_heads * a.L.kd; a.pos = d_pos; a.row_seq = d_row_seq;
   a.cu = d_cu; a.row_to_req = d_row_to_req; a.q_norm = l.q_norm; a.k_norm = l.k_norm;
   if (l.rotation >= 0) { a.rotation = rotations[l.rotation].rows; a.rot = s.rot_dim; a.halves = s.flags & B200_DEC_ROT_HALVES ? 1 : 0; }
   if (s.conv_taps > 0) {
@@ -942,18 +1211,22 @@ b200_status b200_decoder::experts(const Layer& l, int T, int tile_rows, void* st
   cudaStream_t cs = (cudaStream_t)stream;
   b200_status st = B200_OK;
   const MoeTableLayer& t = moe[l.moe];
+  const void* in = in_of(l);
   const int A = T * t.top, act_w = pad64(l.s.expert_ffn), items = std::min(A, t.n_experts + A / tile_rows);
   if (l.wrouter) {
     MatSrc z;
-    MODEL_STEP_CAT(1, matmul(l.wrouter, h, T, 2, &z, stream));
-    MODEL_STEP(b200_moe_route_plan(t, z, f32(), std::max(l.s.n_groups, 1), l.s.n_groups > 0 ? l.s.keep_groups : 1, T, tile_rows, moe_wts, stream));
+    MODEL_STEP_CAT(1, matmul(l.wrouter, in, T, 2, &z, stream));
+    RouterScores scores;
+    if (l.s.flags & B200_DEC_ROUTER_PLAIN) { scores.renormalise = false; scores.scale = l.s.router_scale; }
+    if (l.shared_gate()) scores.shared = shared_w;
+    MODEL_STEP(b200_moe_route_plan(t, z, f32(), std::max(l.s.n_groups, 1), l.s.n_groups > 0 ? l.s.keep_groups : 1, T, tile_rows, moe_wts, stream, scores));
   }
   if (f32()) {
-    MODEL_STEP_CAT(1, b200_qmm_f32_grouped(l.we_gu, (const float*)h, t.order, t.top, (float*)moe_act, act_w, l.epilogue(), t.items, t.n_items, items, stream));
+    MODEL_STEP_CAT(1, b200_qmm_f32_grouped(l.we_gu, (const float*)in, t.order, t.top, (float*)moe_act, act_w, l.epilogue(), t.items, t.n_items, items, stream));
     MODEL_STEP_CAT(1, b200_qmm_f32_grouped(l.we_down, (const float*)moe_act, nullptr, 1, (float*)moe_y, hp, B200_EPI_NONE, t.items, t.n_items, items, stream));
     return B200_OK;
   }
-  MODEL_STEP(b200_moe_gather_order(h, t.order, t.top, A, hp, moe_x, stream));
+  MODEL_STEP(b200_moe_gather_order(in, t.order, t.top, A, hp, moe_x, stream));
   MODEL_STEP_CAT(1, b200_qmm_grouped(l.we_gu, moe_x, A, moe_act, l.epilogue(), nullptr, 0.f, t.items, t.n_items, items, tile_rows, stream));
   MODEL_STEP_CAT(1, b200_qmm_grouped(l.we_down, moe_act, A, moe_y, B200_EPI_NONE, nullptr, 0.f, t.items, t.n_items, items, tile_rows, stream));
   return B200_OK;
@@ -972,6 +1245,8 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
     a.embed = embed;
     a.vocab = cfg.vocab;
     a.embed_scale = cfg.embed_scale;
+    a.pos_embed = pos_embed;
+    a.max_positions = max_positions;
     MODEL_STEP(rows_step(a, T, 0, cs));
   }
   for (size_t r = 0; r < runs.size(); ++r) {
@@ -983,14 +1258,16 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
       a.src = src;
       a.replace = 1;
       a.norm_w = l.norm1;
-      MODEL_STEP(rows_step(a, T, -1, cs));
+      MODEL_STEP(rows_step(a, T, -1, cs, (int)r, 0));
     }
+    MatSrc gate;
+    const bool gated = (s.flags & B200_DEC_RESULT_GATE) != 0;
     // SwiGLU of the dense feed-forward, experts: both from h
     auto feed_forward = [&](void* out, int out_stride) -> b200_status {
       if (s.n_experts > 0 && (st = experts(l, T, tile_rows, stream)) != B200_OK) return st;
       if (s.ffn == 0) return B200_OK;
-      if (f32()) MODEL_STEP_CAT(1, b200_qmm_f32(l.wgu, (const float*)h, T, (float*)out, out_stride, pad64(s.ffn), l.epilogue(), stream));
-      else MODEL_STEP_CAT(1, b200_qmm_to(l.wgu, h, T, out, out_stride, l.epilogue(), stream));
+      if (f32()) MODEL_STEP_CAT(1, b200_qmm_f32_shaped(l.wgu, (const float*)in_of(l), T, (float*)out, out_stride, pad64(s.ffn), l.epilogue(), stream, l.swiglu()));
+      else MODEL_STEP_CAT(1, b200_qmm_to(l.wgu, in_of(l), T, out, out_stride, l.epilogue(), stream, l.swiglu()));
       return B200_OK;
     };
     auto last_rows = [&](const float* post) -> b200_status {  // the layer's last sublayer joins the residual
@@ -1001,7 +1278,9 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
       if (s.n_experts > 0) {
         a.moe_y = moe_y; a.moe_rows = moe[l.moe].inv_order; a.moe_k = s.top_k; a.moe_stride = hp; a.moe_w = 1.0f / (float)s.top_k;
         if (l.wrouter) a.moe_wts = moe_wts;
+        if (l.shared_gate()) a.src_scale = shared_w;
       }
+      if (gated) { a.gate = gate; a.gate_bias = l.out_gate_bias[l.second() ? 1 : 0]; }
       if (l.depth) { a.depth = l.depth; a.n_hist = (int)r + 1; }
       return rows_step(a, T, (int)r + 1, cs);
     };
@@ -1012,6 +1291,7 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
       MODEL_STEP(last_rows(nullptr));
     } else {
       const bool ff = s.ffn > 0 || s.n_experts > 0;
+      if (gated) MODEL_STEP_CAT(1, result_gate(l, 0, T, &gate, stream));
       if ((st = mixer(kv, (int)r, n_req, T, stream)) != B200_OK) return st;
       MODEL_STEP_CAT(1, matmul(l.wo, attn, T, 1, &src, stream));
       if (!ff) {
@@ -1021,7 +1301,9 @@ b200_status b200_decoder::run_layers(b200_kv* kv, int n_req, int T, int n_logits
         a.src = src;
         a.post_w = l.post1;
         a.norm_w = sum_norm() ? l.norm1 : l.norm2;
-        MODEL_STEP(rows_step(a, T, -1, cs));
+        if (gated) { a.gate = gate; a.gate_bias = l.out_gate_bias[0]; }
+        MODEL_STEP(rows_step(a, T, -1, cs, (int)r, 1));
+        if (gated) MODEL_STEP_CAT(1, result_gate(l, 1, T, &gate, stream));
         if ((st = feed_forward(act, pad64(s.ffn))) != B200_OK) return st;
         src = MatSrc{};
         if (s.ffn > 0) MODEL_STEP_CAT(1, matmul(l.wdown, act, T, 1, &src, stream));
@@ -1061,17 +1343,20 @@ uint64_t tensor_elems(const b200_decoder* m, int layer, int which) {
   const uint64_t D = c.hidden;
   switch (which) {
     case B200_DEC_W_HEAD: case B200_DEC_W_EMBED: return (uint64_t)c.vocab * D;
+    case B200_DEC_W_POS: return (uint64_t)c.max_positions * D;
     case B200_DEC_W_LOOP_IN: return c.loop_times > 0 ? 2 * D * D : 0;
     case B200_DEC_FINAL_NORM: return c.flags & B200_DEC_SCALAR_NORM ? 1 : D;
     default: break;
   }
   const b200_decoder_layer& s = m->layers[layer].s;
   const uint64_t H = s.n_heads, norm = c.flags & B200_DEC_SCALAR_NORM ? 1 : D, ef = (uint64_t)s.n_experts * s.expert_ffn;
-  const bool latent = s.mixer == B200_MIX_LATENT, gla = s.mixer == B200_MIX_GLA, soft = s.mixer == B200_MIX_ATTENTION, lru = s.mixer == B200_MIX_LRU;
+  const bool latent = s.mixer == B200_MIX_LATENT, gla = s.mixer == B200_MIX_GLA, soft = s.mixer == B200_MIX_ATTENTION, lru = s.mixer == B200_MIX_LRU,
+             delta = s.mixer == B200_MIX_DELTA, own = !soft || s.kv_source == 0;
   const uint64_t MH = s.mem_heads, mk = MH * s.mem_key_dim, mv = MH * s.mem_value_dim, W = lru ? H * s.value_dim : 0;
-  const uint64_t gate = s.flags & B200_DEC_FF_GELU ? 0 : 1, taps = soft ? s.conv_taps : 0, weighed = soft && s.flags & B200_DEC_QK_NORM_WEIGHT ? s.key_dim : 0;
-  const uint64_t qn = H * (s.key_dim + (latent ? s.rot_dim : 0)), kn = (gla ? H : s.n_kv_heads) * (uint64_t)s.key_dim,
-                 vn = (gla ? H : s.n_kv_heads) * (uint64_t)s.value_dim;
+  const uint64_t gate = m->layers[layer].plain_ff() ? 0 : 1, taps = soft || delta ? s.conv_taps : 0, weighed = soft && s.flags & B200_DEC_QK_NORM_WEIGHT ? s.key_dim : 0;
+  const uint64_t qn = (delta ? s.n_kv_heads : H) * (s.key_dim + (latent ? s.rot_dim : 0)), kn = own ? (gla ? H : s.n_kv_heads) * (uint64_t)s.key_dim : 0,
+                 vn = own ? (gla || delta ? H : s.n_kv_heads) * (uint64_t)s.value_dim : 0;
+  const bool norm_row = soft && s.flags & B200_DEC_QK_NORM_ROW, result_gate = s.flags & B200_DEC_RESULT_GATE;
   const bool bias = soft && s.flags & B200_DEC_QKV_BIAS, post = s.flags & B200_DEC_POST_NORM;
   const bool ff = s.ffn > 0 || s.n_experts > 0, second = ff && !(s.flags & B200_DEC_PARALLEL);
   switch (which) {
@@ -1095,14 +1380,15 @@ uint64_t tensor_elems(const b200_decoder* m, int layer, int which) {
     case B200_DEC_DQ_NORM: return latent ? s.q_rank : 0;
     case B200_DEC_W_UK: return latent ? H * s.key_dim * s.kv_rank : 0;
     case B200_DEC_W_UV: return latent ? H * s.value_dim * s.kv_rank : 0;
-    case B200_DEC_W_OUT_GATE: return gla ? vn * D : 0;
+    case B200_DEC_W_OUT_GATE: return gla || delta ? vn * D : 0;
     case B200_DEC_W_A1: return gla ? s.decay_rank * D : 0;
     case B200_DEC_W_A2: return gla ? kn * s.decay_rank : 0;
     case B200_DEC_B_A2: return gla ? kn : 0;
-    case B200_DEC_HEAD_NORM: return gla ? s.value_dim : 0;
+    case B200_DEC_HEAD_NORM: return gla || delta ? s.value_dim : 0;
     case B200_DEC_W_EXPERT_GATE: return gate * ef * D;
     case B200_DEC_W_EXPERT_UP: case B200_DEC_W_EXPERT_DOWN: return ef * D;
-    case B200_DEC_Q_NORM: case B200_DEC_K_NORM: return weighed;
+    case B200_DEC_Q_NORM: return norm_row ? qn : weighed;
+    case B200_DEC_K_NORM: return norm_row ? kn : weighed;
     case B200_DEC_CONV_Q: return qn * taps;
     case B200_DEC_CONV_K: return kn * taps;
     case B200_DEC_CONV_V: return vn * taps;
@@ -1116,13 +1402,23 @@ uint64_t tensor_elems(const b200_decoder* m, int layer, int which) {
     case B200_DEC_LRU_CONV: return W * s.conv_taps;
     case B200_DEC_B_LRU_Y: case B200_DEC_B_LRU_X: case B200_DEC_B_LRU_CONV: case B200_DEC_B_LRU_R: case B200_DEC_B_LRU_I: case B200_DEC_LRU_LAMBDA: return W;
     case B200_DEC_W_ROUTER: return s.flags & B200_DEC_ROUTER ? (uint64_t)s.n_experts * D : 0;
+    case B200_DEC_W_REL: return soft ? (uint64_t)s.rel_buckets * H : 0;
+    case B200_DEC_IN_CONV1: return D * s.input_taps;
+    case B200_DEC_IN_CONV2: return second ? D * s.input_taps : 0;
+    case B200_DEC_W_RESULT_GATE1: return result_gate ? D * D : 0;
+    case B200_DEC_W_RESULT_GATE2: return result_gate && second ? D * D : 0;
+    case B200_DEC_B_RESULT_GATE1: return result_gate ? D : 0;
+    case B200_DEC_B_RESULT_GATE2: return result_gate && second ? D : 0;
+    case B200_DEC_W_BETA: case B200_DEC_W_DECAY: return delta ? H * D : 0;
+    case B200_DEC_A_LOG: case B200_DEC_DT_BIAS: return delta ? H : 0;
+    case B200_DEC_W_SHARED_GATE: return s.flags & B200_DEC_SHARED_GATE ? D : 0;
     case B200_DEC_DEPTH: return c.flags & B200_DEC_DEPTH_AVERAGE ? layer + 2 : 0;
     default: return 0;
   }
 }
 
 bool global_tensor(int which) {
-  return which == B200_DEC_W_HEAD || which == B200_DEC_W_EMBED || which == B200_DEC_W_LOOP_IN || which == B200_DEC_FINAL_NORM;
+  return which == B200_DEC_W_HEAD || which == B200_DEC_W_EMBED || which == B200_DEC_W_POS || which == B200_DEC_W_LOOP_IN || which == B200_DEC_FINAL_NORM;
 }
 
 b200_status take(b200_decoder* m, int layer, int which, std::vector<uint16_t>* out) {
@@ -1247,7 +1543,7 @@ b200_status take_stack(b200_decoder* m, int layer, int which, int count, int n, 
 
 // Experts: gate and up rows interleaved, [2 pad(ff), pad(hidden)] (without a gate [pad(ff), pad(hidden)]); down [pad(hidden), pad(ff)].
 b200_status take_experts(b200_decoder* m, int layer, b200_decoder::Layer& l) {
-  const int E = l.s.n_experts, f = l.s.expert_ffn, D = m->cfg.hidden, fp = pad64(f), dp = pad64(D), per = l.gelu() ? 1 : 2;
+  const int E = l.s.n_experts, f = l.s.expert_ffn, D = m->cfg.hidden, fp = pad64(f), dp = pad64(D), per = l.plain_ff() ? 1 : 2;
   std::vector<uint16_t> gate, up, down;
   b200_status st;
   if ((per == 2 && (st = take(m, layer, B200_DEC_W_EXPERT_GATE, &gate)) != B200_OK) || (st = take(m, layer, B200_DEC_W_EXPERT_UP, &up)) != B200_OK ||
@@ -1320,6 +1616,28 @@ b200_status make_slopes(b200_decoder::Layer& l) {
   return upload_f32(v, &l.slopes);
 }
 
+// The rows of a distance table [buckets][heads] spread out over distances: one row each for the near half, the far half by the logarithm, up
+// to the first distance of the last row.
+b200_status make_distances(b200_decoder::Layer& l, const std::vector<float>& table) {
+  const int B = l.s.rel_buckets, H = l.s.n_heads, near = B / 2;
+  std::vector<int> row;
+  for (int n = 0; row.empty() || row.back() < B - 1; ++n)
+    row.push_back(n < near ? n : std::min(B - 1, near + (int)std::floor(std::log((double)n / near) / std::log((double)l.s.rel_reach / near) * (B - near))));
+  l.dist_len = (int)row.size();
+  std::vector<float> v((size_t)H * l.dist_len);
+  for (int h = 0; h < H; ++h)
+    for (int n = 0; n < l.dist_len; ++n) v[(size_t)h * l.dist_len + n] = (float)(table[(size_t)row[n] * H + h] * kLog2e);
+  return upload_f32(v, &l.dist);
+}
+
+b200_status take_floats(b200_decoder* m, int layer, int which, std::vector<float>* out) {
+  std::vector<uint16_t> bits;
+  b200_status st = take(m, layer, which, &bits);
+  out->clear();
+  for (uint16_t b : bits) out->push_back(bf16_to_f(b));
+  return st;
+}
+
 }  // namespace
 
 extern "C" {
@@ -1341,26 +1659,41 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
   m->cfg = *c;
   m->layers.resize(c->n_layers);
   size_t qw = 0, yw = pad64(c->hidden), aw = 0, fw = 0, plain_w = 0, lat_w = 0, assign = 0, moe_aw = 0, ql_w = 0, lru_w = 0, mem_w = 0;
+  int taps = 0;
+  bool gated = false;
   for (int i = 0; i < c->n_layers; ++i) {
     const b200_decoder_layer& s = layers[i];
     bool good = s.n_heads > 0 && s.key_dim > 0 && s.value_dim > 0 && s.ffn >= 0 && s.window >= 0 && s.n_experts >= 0;
     if (s.mixer == B200_MIX_ATTENTION)
       good = good && s.n_kv_heads > 0 && s.n_heads % s.n_kv_heads == 0 && s.conv_taps >= 0 && s.rot_dim >= 0 && s.rot_dim % 2 == 0 && s.rot_dim <= s.key_dim &&
+             s.q_temp_every >= 0 &&
              (!(s.flags & B200_DEC_QK_NORM_WEIGHT) || (s.flags & B200_DEC_QK_NORM)) && !((s.flags & B200_DEC_SINK) && (s.flags & B200_DEC_SINK_ONE));
     else
-      good = good && s.mem_heads == 0 && !(s.flags & (B200_DEC_SINK_ONE | B200_DEC_QK_NORM_WEIGHT));
+      good = good && s.mem_heads == 0 && !(s.flags & (B200_DEC_SINK_ONE | B200_DEC_QK_NORM_WEIGHT | B200_DEC_QK_NORM_ROW)) && s.rel_buckets == 0 && s.q_temp_every == 0;
+    if (s.rel_buckets != 0) good = good && s.rel_buckets >= 2 && s.rel_reach > s.rel_buckets / 2 && !(s.flags & B200_DEC_DISTANCE_BIAS);
+    if (s.mixer == B200_MIX_ATTENTION && ((s.flags & B200_DEC_QK_NORM_ROW) || s.q_temp_every > 0 || s.kv_source != 0))  // (decoder_qkv_row_kernel)
+      good = good && s.conv_taps == 0 && s.rot_dim == 0 && s.mem_heads == 0 && !(s.flags & B200_DEC_QK_NORM);
+    good = good && s.input_taps >= 0 && s.ff_limit >= 0.f && !((s.flags & B200_DEC_FF_GELU) && (s.flags & B200_DEC_FF_RELU2));
+    if (s.input_taps > 0 || (s.flags & B200_DEC_RESULT_GATE)) good = good && !(c->flags & B200_DEC_SUM_NORM);
+    if (s.flags & B200_DEC_RESULT_GATE) good = good && !(s.flags & B200_DEC_PARALLEL);
+    if (s.flags & B200_DEC_ROUTER_PLAIN) good = good && (s.flags & B200_DEC_ROUTER);
+    if (s.flags & B200_DEC_SHARED_GATE) good = good && (s.flags & B200_DEC_ROUTER) && s.n_experts > 0 && s.ffn > 0;
     if (s.mixer == B200_MIX_ATTENTION && s.mem_heads != 0) good = good && s.mem_heads > 0 && s.mem_key_dim > 0 && s.mem_value_dim > 0 && s.mem_gate_cap > 0.f;
     if (s.rot_dim > 0)
       good = good && s.rot_base > 1.0 && (s.yarn_factor == 0.0 || (s.yarn_factor > 0.0 && s.yarn_original > 0.0 && s.yarn_fast > 0.0 && s.yarn_slow > 0.0));
     if (s.kv_source != 0) {
       const int src = s.kv_source - 1;
-      good = good && !loop && s.mixer == B200_MIX_LATENT && src >= 0 && src < i && layers[src].mixer == B200_MIX_LATENT && layers[src].kv_source == 0 &&
-             layers[src].kv_rank == s.kv_rank && layers[src].rot_dim == s.rot_dim;
+      good = good && !loop && src >= 0 && src < i && layers[src].mixer == s.mixer && layers[src].kv_source == 0;
+      if (s.mixer == B200_MIX_ATTENTION)
+        good = good && layers[src].n_kv_heads == s.n_kv_heads && layers[src].key_dim == s.key_dim && layers[src].value_dim == s.value_dim;
+      else
+        good = good && s.mixer == B200_MIX_LATENT && layers[src].kv_rank == s.kv_rank && layers[src].rot_dim == s.rot_dim;
     }
     if (s.mixer == B200_MIX_ATTENTION) {}
     else if (s.mixer == B200_MIX_LRU) good = good && s.conv_taps > 0 && s.lru_decay > 0.f && s.window == 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS | B200_DEC_SINK));
     else if (s.mixer == B200_MIX_LATENT) good = good && s.kv_rank > 0 && s.rot_dim >= 0 && s.rot_dim % 2 == 0 && s.q_rank >= 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS));
     else if (s.mixer == B200_MIX_GLA) good = good && s.decay_rank > 0 && s.decay_tau > 0.f && s.window == 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS | B200_DEC_SINK));
+    else if (s.mixer == B200_MIX_DELTA) good = good && s.n_kv_heads > 0 && s.n_heads % s.n_kv_heads == 0 && s.conv_taps > 0 && s.window == 0 && !(s.flags & (B200_DEC_QKV_BIAS | B200_DEC_QK_NORM | B200_DEC_DISTANCE_BIAS | B200_DEC_SINK));
     else good = false;
     if (s.n_experts > 0) good = good && s.top_k > 0 && s.top_k <= s.n_experts && s.n_experts <= b200_moe_max_experts() && s.expert_ffn > 0;
     if (s.n_experts > 0 && s.flags & B200_DEC_ROUTER)
@@ -1375,8 +1708,11 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
     }
     b200_decoder::Layer& l = m->layers[i];
     l.s = s;
+    l.hidden = c->hidden;
+    taps = std::max(taps, s.input_taps);
+    gated = gated || (s.flags & B200_DEC_RESULT_GATE);
     qw = std::max(qw, (size_t)s.n_heads * (s.mixer == B200_MIX_LATENT ? l.latent_width() : (s.key_dim + 15) / 16 * 16));
-    yw = std::max({yw, (size_t)pad64(l.qkv_n()), (size_t)pad64(l.router_n()), (size_t)pad64(2 * s.mem_heads), (size_t)(s.q_rank > 0 ? pad64(l.q_n()) : 0)});
+    yw = std::max({yw, (size_t)pad64(l.qkv_n()), (size_t)pad64(l.router_n() + 1), (size_t)pad64(2 * s.mem_heads), (size_t)(s.q_rank > 0 ? pad64(l.q_n()) : 0)});
     aw = std::max(aw, (size_t)l.out_k());
     fw = std::max(fw, (size_t)pad64(s.ffn));
     if (s.mixer == B200_MIX_LATENT) {
@@ -1408,6 +1744,10 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
       m->has_gla = true;
       if (b200_gla_takes_chunks(s.key_dim, s.value_dim, (int)m->elem())) m->gla.need(s.n_heads, s.key_dim, s.value_dim);
     }
+    if (l.delta()) {
+      m->has_gla = true;
+      m->gla.need_delta(s.n_heads, s.n_kv_heads, s.key_dim, s.value_dim, b200_gla_takes_chunks(s.key_dim, s.value_dim, (int)m->elem()));
+    }
     if (s.n_experts > 0) {
       l.moe = (int)m->moe_layers.size();
       m->moe_layers.push_back(i);
@@ -1436,7 +1776,13 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
     alloc((void**)&m->x0, R * c->hidden * 4);
     alloc(&m->cat, R * m->catp * e);
   }
+  if (c->max_positions > 0) {
+    alloc((void**)&m->pos_embed, (size_t)c->max_positions * c->hidden * 2);
+    m->max_positions = c->max_positions;
+  }
   alloc(&m->h, R * m->hp * e);
+  if (taps > 0) alloc(&m->hc, R * m->hp * e);
+  if (gated) alloc(&m->gate_y, R * m->hp * e);
   alloc(&m->y, std::max(R * yw, (size_t)c->max_reqs * 64) * e);
   alloc(&m->q, R * qw * e);
   alloc(&m->attn, R * aw * e);
@@ -1468,6 +1814,7 @@ b200_status b200_decoder_create(const b200_decoder_config* c, const b200_decoder
     alloc(&m->moe_act, R * moe_aw * e);
     alloc(&m->moe_y, R * assign * m->hp * e);
     alloc((void**)&m->moe_wts, R * assign * 4);
+    alloc((void**)&m->shared_w, R * 4);
     for (int i : m->moe_layers) {
       const b200_decoder_layer& s = m->layers[i].s;
       const size_t A = R * s.top_k;
@@ -1497,7 +1844,7 @@ void b200_decoder_destroy(b200_decoder* m) { delete m; }
 b200_model* b200_decoder_model(b200_decoder* m) { return m; }
 
 b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t which, const void* h_bf16, uint64_t n) {
-  if (which < 0 || which > B200_DEC_W_ROUTER || (!global_tensor(which) && (layer < 0 || layer >= m->cfg.n_layers))) {
+  if (which < 0 || which > B200_DEC_LAST_TENSOR || (!global_tensor(which) && (layer < 0 || layer >= m->cfg.n_layers))) {
     b200_set_error("decoder: no tensor %d in layer %d", which, layer);
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -1541,13 +1888,15 @@ b200_status b200_decoder_finalize(b200_decoder* m) {
     if ((st = take_norm(m, i, B200_DEC_NORM1, &l.norm1)) != B200_OK) return st;
     if (s.flags & B200_DEC_POST_NORM) if ((st = take_norm(m, i, B200_DEC_POSTNORM1, &l.post1)) != B200_OK) return st;
     if (s.ffn > 0) {
-      st = l.gelu() ? take_weight(m, i, {B200_DEC_W_UP}, c.hidden, false, &l.wgu) : take_weight(m, i, {B200_DEC_W_GATE, B200_DEC_W_UP}, c.hidden, true, &l.wgu);
+      st = l.plain_ff() ? take_weight(m, i, {B200_DEC_W_UP}, c.hidden, false, &l.wgu) : take_weight(m, i, {B200_DEC_W_GATE, B200_DEC_W_UP}, c.hidden, true, &l.wgu);
       if (st != B200_OK) return st;
       if (!l.parallel()) if ((st = take_weight(m, i, {B200_DEC_W_DOWN}, s.ffn, false, &l.wdown)) != B200_OK) return st;
     }
     if (s.n_experts > 0) {
       if ((st = take_experts(m, i, l)) != B200_OK) return st;
-      st = s.flags & B200_DEC_ROUTER ? take_weight(m, i, {B200_DEC_W_ROUTER}, c.hidden, false, &l.wrouter) : upload_table(m, i, l);
+      std::vector<int> rows{B200_DEC_W_ROUTER};
+      if (l.shared_gate()) rows.push_back(B200_DEC_W_SHARED_GATE);
+      st = s.flags & B200_DEC_ROUTER ? take_weight(m, i, rows, c.hidden, false, &l.wrouter) : upload_table(m, i, l);
       if (st != B200_OK) return st;
     }
     if ((s.ffn > 0 || s.n_experts > 0) && !l.parallel()) {
@@ -1576,7 +1925,28 @@ b200_status b200_decoder_finalize(b200_decoder* m) {
       if ((st = take_vector(m, i, B200_DEC_Q_NORM, &l.q_norm)) != B200_OK) return st;
       if ((st = take_vector(m, i, B200_DEC_K_NORM, &l.k_norm)) != B200_OK) return st;
     }
-    if (s.mixer == B200_MIX_ATTENTION && s.conv_taps > 0)
+    if (s.flags & B200_DEC_QK_NORM_ROW) {
+      if ((st = take_vector(m, i, B200_DEC_Q_NORM, &l.q_norm)) != B200_OK) return st;
+      if (s.kv_source == 0) if ((st = take_vector(m, i, B200_DEC_K_NORM, &l.k_norm)) != B200_OK) return st;
+    }
+    std::vector<float> v;
+    if (s.rel_buckets > 0)
+      if ((st = take_floats(m, i, B200_DEC_W_REL, &v)) != B200_OK || (st = make_distances(l, v)) != B200_OK) return st;
+    const int subs = l.second() ? 2 : 1;
+    for (int w = 0; w < subs && s.input_taps > 0; ++w)
+      if ((st = take_conv(m, i, {w ? B200_DEC_IN_CONV2 : B200_DEC_IN_CONV1}, s.input_taps, &l.in_conv[w])) != B200_OK) return st;
+    for (int w = 0; w < subs && s.flags & B200_DEC_RESULT_GATE; ++w) {
+      if ((st = take_weight(m, i, {w ? B200_DEC_W_RESULT_GATE2 : B200_DEC_W_RESULT_GATE1}, c.hidden, false, &l.wgate[w])) != B200_OK) return st;
+      if ((st = take_vector(m, i, w ? B200_DEC_B_RESULT_GATE2 : B200_DEC_B_RESULT_GATE1, &l.out_gate_bias[w])) != B200_OK) return st;
+    }
+    if (l.delta()) {
+      if ((st = take_vector(m, i, B200_DEC_DT_BIAS, &l.dt_bias)) != B200_OK || (st = take_vector(m, i, B200_DEC_HEAD_NORM, &l.head_norm)) != B200_OK ||
+          (st = take_floats(m, i, B200_DEC_A_LOG, &v)) != B200_OK)
+        return st;
+      for (float& x : v) x = (float)std::exp((double)x);
+      if ((st = upload_f32(v, &l.rate)) != B200_OK) return st;
+    }
+    if ((s.mixer == B200_MIX_ATTENTION || l.delta()) && s.conv_taps > 0)
       if ((st = take_conv(m, i, {B200_DEC_CONV_Q, B200_DEC_CONV_K, B200_DEC_CONV_V}, s.conv_taps, &l.conv)) != B200_OK) return st;
     if (s.mem_heads > 0) {
       if ((st = take_weight(m, i, {B200_DEC_W_MEM_I, B200_DEC_W_MEM_F}, c.hidden, false, &l.wgates)) != B200_OK) return st;
@@ -1599,6 +1969,10 @@ b200_status b200_decoder_finalize(b200_decoder* m) {
   if ((st = take_norm(m, -1, B200_DEC_FINAL_NORM, &m->final_norm, c.logit_scale)) != B200_OK) return st;
   if ((st = upload_moe(m)) != B200_OK) return st;
   std::vector<uint16_t> table;
+  if (c.max_positions > 0) {
+    if ((st = take(m, -1, B200_DEC_W_POS, &table)) != B200_OK) return st;
+    B200_CUDA_TRY(cudaMemcpy(m->pos_embed, table.data(), table.size() * 2, cudaMemcpyHostToDevice));
+  }
   if ((st = take(m, -1, B200_DEC_W_EMBED, &table)) != B200_OK) return st;
   B200_CUDA_TRY(cudaMemcpy(m->embed, table.data(), table.size() * 2, cudaMemcpyHostToDevice));
   m->ready = true;
@@ -1622,7 +1996,7 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
     if ((st = upload_f32(ones, &l.norm1)) != B200_OK) return st;
     if (s.flags & B200_DEC_POST_NORM) if ((st = upload_f32(ones, &l.post1)) != B200_OK) return st;
     if (s.ffn > 0) {
-      if ((st = weight((l.gelu() ? 1 : 2) * s.ffn, c.hidden, 16 * i + 3, &l.wgu)) != B200_OK) return st;
+      if ((st = weight((l.plain_ff() ? 1 : 2) * s.ffn, c.hidden, 16 * i + 3, &l.wgu)) != B200_OK) return st;
       if (!l.parallel()) if ((st = weight(c.hidden, s.ffn, 16 * i + 4, &l.wdown)) != B200_OK) return st;
     }
     if ((s.ffn > 0 || s.n_experts > 0) && !l.parallel()) {
@@ -1630,10 +2004,10 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
       if (s.flags & B200_DEC_POST_NORM) if ((st = upload_f32(ones, &l.post2)) != B200_OK) return st;
     }
     if (s.n_experts > 0) {
-      if ((st = stack(s.n_experts, (l.gelu() ? 1 : 2) * s.expert_ffn, c.hidden, 16 * i + 5, &l.we_gu)) != B200_OK) return st;
+      if ((st = stack(s.n_experts, (l.plain_ff() ? 1 : 2) * s.expert_ffn, c.hidden, 16 * i + 5, &l.we_gu)) != B200_OK) return st;
       if ((st = stack(s.n_experts, c.hidden, s.expert_ffn, 16 * i + 6, &l.we_down)) != B200_OK) return st;
       if (s.flags & B200_DEC_ROUTER) {
-        if ((st = weight(pad64(s.n_experts), c.hidden, 16 * i + 9, &l.wrouter)) != B200_OK) return st;
+        if ((st = weight(pad64(s.n_experts + (l.shared_gate() ? 1 : 0)), c.hidden, 16 * i + 9, &l.wrouter)) != B200_OK) return st;
       } else {
       l.h_table.resize((size_t)c.vocab * s.top_k);
       uint32_t x = seed * 747796405u + i;
@@ -1670,6 +2044,20 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
     if (s.flags & B200_DEC_QK_NORM_WEIGHT)
       if ((st = fill(s.key_dim, 1.f, &l.q_norm)) != B200_OK || (st = fill(s.key_dim, 1.f, &l.k_norm)) != B200_OK) return st;
     if (s.mixer == B200_MIX_ATTENTION && s.conv_taps > 0) if ((st = upload_bf16(std::vector<uint16_t>((size_t)l.attention_n() * s.conv_taps, 0x3F00), &l.conv)) != B200_OK) return st;
+    if (s.flags & B200_DEC_QK_NORM_ROW)
+      if ((st = fill((size_t)s.n_heads * s.key_dim, 1.f, &l.q_norm)) != B200_OK || (st = fill((size_t)s.n_kv_heads * s.key_dim, 1.f, &l.k_norm)) != B200_OK) return st;
+    if (s.rel_buckets > 0) if ((st = make_distances(l, std::vector<float>((size_t)s.rel_buckets * s.n_heads, 0.25f))) != B200_OK) return st;
+    for (int w = 0; w < (l.second() ? 2 : 1); ++w) {
+      if (s.input_taps > 0) if ((st = upload_bf16(std::vector<uint16_t>((size_t)c.hidden * s.input_taps, 0x3E80), &l.in_conv[w])) != B200_OK) return st;
+      if (s.flags & B200_DEC_RESULT_GATE)
+        if ((st = weight(c.hidden, c.hidden, 16 * i + 13 + w, &l.wgate[w])) != B200_OK || (st = fill(c.hidden, 0.1f, &l.out_gate_bias[w])) != B200_OK) return st;
+    }
+    if (l.delta()) {
+      const size_t channels = b200_delta_channels(s.n_heads, s.n_kv_heads, s.key_dim, s.value_dim);
+      if ((st = upload_bf16(std::vector<uint16_t>(channels * s.conv_taps, 0x3F00), &l.conv)) != B200_OK || (st = fill(s.n_heads, 0.5f, &l.rate)) != B200_OK ||
+          (st = fill(s.n_heads, -2.f, &l.dt_bias)) != B200_OK || (st = fill(s.value_dim, 1.f, &l.head_norm)) != B200_OK)
+        return st;
+    }
     if (s.mem_heads > 0) {
       if ((st = weight(pad64(2 * s.mem_heads), c.hidden, 16 * i + 11, &l.wgates)) != B200_OK) return st;
       if ((st = fill(2 * s.mem_heads, 1.f, &l.gate_bias)) != B200_OK || (st = fill(l.mem_n(), 1.f, &l.mem_norm)) != B200_OK) return st;
@@ -1690,6 +2078,7 @@ b200_status b200_decoder_random_init(b200_decoder* m, uint32_t seed) {
   uint32_t s = seed * 2654435761u + 12345u;
   for (auto& e : emb) { s = s * 1664525u + 1013904223u; e = (uint16_t)(((s >> 16) & 0x807F) | 0x3C80); }
   B200_CUDA_TRY(cudaMemcpy(m->embed, emb.data(), emb.size() * 2, cudaMemcpyHostToDevice));
+  if (c.max_positions > 0) B200_CUDA_TRY(cudaMemset(m->pos_embed, 0, (size_t)c.max_positions * c.hidden * 2));
   m->ready = true;
   return B200_OK;
 }
@@ -1740,11 +2129,11 @@ b200_status b200_decoder_qkv(b200_kv* kv, int32_t layer, const void* d_qkv, int3
 }
 
 b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, int32_t n_q_heads, int32_t window, float scale,
-                                   const float* d_slopes_log2, const float* d_sinks_log2, const int32_t* d_row_seq,
-                                   const int32_t* d_row_ctx, int32_t total_rows, int32_t mma, void* d_out,
+                                   const float* d_slopes_log2, const float* d_sinks_log2, const float* d_dist_log2, int32_t dist_len,
+                                   const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows, int32_t mma, void* d_out,
                                    int32_t out_stride, void* stream) {
   if (!kv->layered || layer < 0 || layer >= kv->cfg.n_layers || n_q_heads <= 0 || n_q_heads > kv->cfg.n_q_heads || kv->lay[layer].heads <= 0 ||
-      n_q_heads % kv->lay[layer].heads != 0 || window < 0) {
+      n_q_heads % kv->lay[layer].heads != 0 || window < 0 || (d_dist_log2 && (dist_len <= 0 || kv->lay[layer].values_in_keys))) {
     b200_set_error("decoder_attention: layer %d with %d query heads, window %d", layer, n_q_heads, window);
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -1754,7 +2143,7 @@ b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, 
   if (st != B200_OK) return st;
   WindowAttnCall c;
   c.layer = layer; c.n_q_heads = n_q_heads; c.window = window; c.q = d_q; c.q_stride = n_q_heads * kv->lay[layer].kd; c.scale = scale;
-  c.slopes_log2 = d_slopes_log2; c.sinks_log2 = d_sinks_log2; c.out = d_out; c.out_stride = out_stride;
+  c.slopes_log2 = d_slopes_log2; c.sinks_log2 = d_sinks_log2; c.dist_log2 = d_dist_log2; c.dist_len = dist_len; c.out = d_out; c.out_stride = out_stride;
   return b200_window_attn_run(kv, c, d_row_seq, d_row_ctx, total_rows, mma != 0, stream);
 }
 
@@ -1778,6 +2167,30 @@ b200_status b200_decoder_gla(b200_kv* kv, int32_t layer, const b200_gla_shape* z
   const cudaError_t e = cudaStreamSynchronize((cudaStream_t)stream);
   g.free();
   if (st == B200_OK && e != cudaSuccess) { b200_set_error("decoder_gla: %s", cudaGetErrorString(e)); return B200_ERR_CUDA; }
+  return st;
+}
+
+b200_status b200_decoder_delta(b200_kv* kv, int32_t layer, const b200_delta_shape* z, const void* d_rows, int32_t stride, const void* d_conv,
+                               const float* d_rate, const float* d_dt_bias, const float* d_norm, const int32_t* d_cu, const int32_t* d_row_to_req,
+                               const int32_t* d_row_seq, const int32_t* d_positions, int32_t n_req, int32_t total_rows, int32_t chunked,
+                               void* d_out, int32_t out_stride, void* stream) {
+  if (n_req <= 0 || total_rows <= 0) return B200_OK;
+  GlaScratch g;
+  g.max_rows = total_rows;
+  g.max_reqs = n_req;
+  g.need_delta(z->heads, z->kv_heads, z->key_dim, z->value_dim, b200_gla_takes_chunks(z->key_dim, z->value_dim, kv->dev.elem_bytes));
+  if (!g.alloc()) { g.free(); b200_set_error("decoder_delta: no memory for %d rows", total_rows); return B200_ERR_CUDA; }
+  DeltaCall c;
+  c.layer = layer; c.heads = z->heads; c.kv_heads = z->kv_heads; c.dk = z->key_dim; c.dv = z->value_dim;
+  c.src.y = d_rows; c.src.y_stride = stride;
+  c.conv.taps = z->taps; c.conv.w = (const __nv_bfloat16*)d_conv;
+  c.rate = d_rate; c.dt_bias = d_dt_bias; c.norm = d_norm; c.eps = z->eps; c.out = d_out; c.out_stride = out_stride;
+  b200_status st = b200_gla_plan(g, d_cu, n_req, total_rows, stream);
+  if (st == B200_OK) st = b200_delta_prep(kv, g, c, d_cu, d_row_to_req, d_row_seq, d_positions, total_rows, stream);
+  if (st == B200_OK) st = b200_delta_run(kv, g, c, d_cu, d_row_seq, d_positions, n_req, total_rows, chunked != 0, stream);
+  const cudaError_t e = cudaStreamSynchronize((cudaStream_t)stream);
+  g.free();
+  if (st == B200_OK && e != cudaSuccess) { b200_set_error("decoder_delta: %s", cudaGetErrorString(e)); return B200_ERR_CUDA; }
   return st;
 }
 

@@ -44,6 +44,7 @@ struct b200_engine {
   uint64_t n_deferred = 0, n_preempted = 0, n_failed = 0;
   bool pressure = false;  // the previous step left a running request out or preempted one: admit nobody new
   int32_t max_pages_per_seq = 0, pool_pages = 0;
+  uint64_t max_seq_tokens = 0;  // what a page table holds, or the model's positions
   std::vector<b200_request*> running_tmp;
 };
 
@@ -125,6 +126,10 @@ b200_engine* b200_engine_create_model(b200_model* model, b200_kv* kv, uint64_t m
   int32_t max_seqs = 0, page_size = 0;
   b200_kv_dims(kv, &e->pool_pages, &max_seqs);
   b200_kv_limits(kv, &e->max_pages_per_seq, &page_size);
+  b200_model_info info;
+  b200_model_get_info(model, &info);
+  e->max_seq_tokens = (uint64_t)e->max_pages_per_seq * kPageTokens;
+  if (info.max_positions > 0) e->max_seq_tokens = std::min<uint64_t>(e->max_seq_tokens, (uint64_t)info.max_positions);
   e->sched = b200_scheduler_create(e->bm, e->max_prefill);
   return e;
 }
@@ -142,7 +147,7 @@ b200_status b200_engine_submit(b200_engine* e, uint64_t id, const uint32_t* prom
   if (e->requests.count(id)) { b200_set_error("engine: request id %llu already exists", (unsigned long long)id); return B200_ERR_INVALID_ARGUMENT; }
   if (n_prompt == 0 || max_tokens == 0) { b200_set_error("engine: empty prompt or max_tokens 0"); return B200_ERR_INVALID_ARGUMENT; }
   // A request whose prompt alone can never fit is refused here instead of blocking the queue for ever.
-  const uint64_t most = std::min<uint64_t>((uint64_t)e->max_pages_per_seq, (uint64_t)e->pool_pages) * kPageTokens;
+  const uint64_t most = std::min<uint64_t>(e->max_seq_tokens, (uint64_t)e->pool_pages * kPageTokens);
   if (n_prompt + 1 > most) {
     b200_set_error("engine: a prompt of %llu tokens exceeds what one sequence can hold (%llu tokens)", (unsigned long long)n_prompt,
                    (unsigned long long)most);
@@ -209,10 +214,10 @@ b200_status b200_engine_step(b200_engine* e, b200_token_output* out, uint64_t ca
     b200_scheduler_hold_admission(e->sched, 0);
     if (st != B200_OK) return st;
     if (np + nd == 0) { e->pressure = false; return B200_OK; }
-    // A sequence that has reached the length its page table can hold ends here, alone (CacheOverflow,
+    // A sequence that has reached the length its page table can hold, or the model has positions for, ends here, alone (CacheOverflow,
     // src/kvcache/quantized.zig:135); the others go on.
     {
-      const uint64_t most = (uint64_t)e->max_pages_per_seq * kPageTokens;
+      const uint64_t most = e->max_seq_tokens;
       uint64_t kept = 0;
       for (uint64_t i = 0; i < nd; ++i) {
         b200_request* r = e->decode[i];

@@ -14,6 +14,7 @@
 //
 // Matrix memory runs through the same kernels: with the running maximum m taken out, S <- e^(f + m' - m) S + (e^(i - m) k) v^T has one
 // decay per head and token, both factors at most 1, and the sum of the keys is one more value column whose values are ones.
+// The delta rule (delta.cu) goes through the scan and out kernels, with more to do per chunk.
 // memory_gates_kernel makes the factors (m is a scan over (max, +)); memory_chunk_kernel and memory_out_kernel take the places of the
 // chunk and out kernels.
 #include <cuda_bf16.h>
@@ -21,44 +22,9 @@
 #include <algorithm>
 
 #include "common.h"
-#include "gla.cuh"
-#include "ptx.cuh"
+#include "gla_chunks.cuh"
 
 namespace {
-
-constexpr int kC = 32;        // tokens of a chunk
-constexpr int kScanWarps = 4;  // 16 value columns each
-constexpr int kScanCols = kScanWarps * 16;
-
-struct Gla {
-  KvDev d;
-  float* state;  // the layer's [slot][heads][dk][dv]
-  int rec_elems;
-  int heads, dk, dv, rank, dkp;
-  int dva, dvs;  // columns of the state in use, and from row to row (matrix memory: one more than dv, padded)
-  MatSrc src;
-  const float *a2, *a2_bias, *norm;
-  float q_scale, inv_tau, eps;
-  void* out;
-  int out_stride;
-  const int *cu, *row_seq, *pos;
-  int n_req, total_rows;
-  bool chunked;  // longer portions are left to the chunk kernels
-  unsigned char *chunks, *values;
-  float* o;
-  const int4* plan;
-  const int* first_chunk;
-  size_t chunk_bytes, v_bytes;
-  int n_slices, stages;
-  int cols, groups;  // step kernel: threads = columns of VEC values x groups of key channels
-  const float4* gates;
-  int col0;
-  float den_eps, out_scale;
-  __device__ int col_k() const { return col0 + heads * dk; }
-  __device__ int col_v() const { return col0 + 2 * heads * dk; }
-  __device__ int col_g() const { return col0 + 2 * heads * dk + heads * dv; }
-  __device__ int col_a() const { return 2 * heads * dk + 2 * heads * dv; }
-};
 
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float silu(float g) { return g / (1.0f + expf(-g)); }
@@ -163,7 +129,7 @@ __global__ void __launch_bounds__(256, 3) gla_step_kernel(Gla a) {
     const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)dv + a.eps);
     T* dst = (T*)a.out + (size_t)row * a.out_stride + (size_t)head * dv;
     for (int c = tid; c < dv; c += nthr) {
-      const float g = mat_value<T, 1>(a.src, row, a.col_g() + head * dv + c).v[0];
+      const float g = mat_value<T, 1>(a.src, row, a.col_g + head * dv + c).v[0];
       if constexpr (MEM) st(dst + c, red[c] * r * a.norm[head * dv + c] * sigmoid(g) * a.out_scale);
       else st(dst + c, red[c] * r * a.norm[c] * silu(g));
     }
@@ -267,36 +233,6 @@ __global__ void __launch_bounds__(1024) gla_plan_kernel(const int* __restrict__ 
     __syncthreads();
   }
   if (tid == 0) first_chunk[n_req] = min(base, max_chunks);
-}
-
-// ---- chunks: layout of what gla_chunk_kernel hands to gla_scan_kernel ----------------------------------------------
-// Rows are padded by 16 bytes so that the 8 rows of an ldmatrix lie in different banks; a chunk and a slice of its values are
-// contiguous, one bulk copy each.
-__host__ __device__ constexpr int qk_row(int dkp) { return dkp * 2 + 16; }
-constexpr int kARow = kC * 2 + 16;
-constexpr int kVRow = kScanCols * 2 + 16;
-__host__ __device__ constexpr size_t off_part(int dkp, int i) { return (size_t)i * kC * qk_row(dkp); }  // 0 q, 1 q rest, 2 k, 3 k rest
-__host__ __device__ constexpr size_t off_a(int dkp, int i) { return off_part(dkp, 4) + (size_t)i * kC * kARow; }
-__host__ __device__ constexpr size_t off_decay(int dkp) { return off_a(dkp, 2); }
-__host__ __device__ constexpr size_t chunk_size(int dkp) { return (off_decay(dkp) + sizeof(float) * dkp + 127) / 128 * 128; }
-constexpr size_t kVSlice = kC * kVRow;
-
-__device__ __forceinline__ void split_bf16(float p0, float p1, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
-  const float2 f = __bfloat1622float2(h);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(p0 - f.x, p1 - f.y);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = *reinterpret_cast<const uint32_t*>(&l);
-}
-__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4_trans(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 
 // ---- chunks: decays, scaled q and k, weights of the sum -------------------------------------------------------------
@@ -435,7 +371,9 @@ __global__ void __launch_bounds__(256) gla_chunk_kernel(Gla a) {
 // ---- chunks: the walk ------------------------------------------------------------------------------------------------
 // One warp holds 16 value columns of S^T [dv][dk] as MMA accumulators, which are at the same time the A operand of
 // o^T = S^T q^T.  A ring of stages, each a chunk's block and its slice of values (two bulk copies).
-template <int NT>  // 8-channel tiles of the state a warp holds
+// DELTA: the values that enter the state are u = U - W S with the state at the chunk's start, W [tokens][dk] and U [tokens][dv] made by
+// delta_chunk_kernel (delta.cu); u is f32 and enters the tensor cores as two terms.
+template <int NT, bool DELTA>  // NT: 8-channel tiles of the state a warp holds
 __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
   extern __shared__ unsigned char scan_dyn[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(scan_dyn) + 127) & ~(uintptr_t)127);
@@ -444,7 +382,8 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
   if (c0 >= c1 || a.d.state[ST_ERR] != 0) return;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int dkp = a.dkp, n_t = dkp / 8, stages = a.stages;
-  const uint32_t cbytes = (uint32_t)chunk_size(dkp), stage_bytes = cbytes + (uint32_t)kVSlice;
+  constexpr uint32_t vbytes = (uint32_t)(DELTA ? kUSlice : kVSlice);
+  const uint32_t cbytes = (uint32_t)(DELTA ? delta_chunk_size(dkp) : chunk_size(dkp)), stage_bytes = cbytes + vbytes;
   uint64_t* full = reinterpret_cast<uint64_t*>(smem + (size_t)stages * stage_bytes);
   const int r0 = a.cu[req], slot = a.row_seq[r0];
   if (slot < 0 || slot >= a.d.max_seqs) return;
@@ -458,7 +397,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
     const size_t ch = (size_t)c * a.heads + head;
     ptx::mbar_expect_tx(&full[s], stage_bytes);
     ptx::bulk_g2s(dst, a.chunks + ch * a.chunk_bytes, cbytes, &full[s]);
-    ptx::bulk_g2s(dst + cbytes, a.values + ch * a.v_bytes + (size_t)slice * kVSlice, (uint32_t)kVSlice, &full[s]);
+    ptx::bulk_g2s(dst + cbytes, a.values + ch * a.v_bytes + (size_t)slice * vbytes, vbytes, &full[s]);
   };
   if (tid == 0)
     for (int s = 0; s < stages && c0 + s < c1; ++s) load(c0 + s, s);
@@ -484,9 +423,12 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
     const unsigned char* st_ = smem + (size_t)s * stage_bytes;
     const uint32_t base = ptx::smem_u32(st_), vbase = base + cbytes;
     const int lr = lane & 7, lm = lane >> 3;
-    float o[4][4];
+    float o[4][4], w[4][4];  // w: W S
 #pragma unroll
-    for (int n = 0; n < 4; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
+    for (int n = 0; n < 4; ++n) {
+      o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+      w[n][0] = w[n][1] = w[n][2] = w[n][3] = 0.f;
+    }
     // from the state: k = channels.  One ldmatrix.x4 covers 8 tokens x 32 channels (two k steps).
 #pragma unroll
     for (int kk = 0; kk < NT / 4; ++kk) {
@@ -512,16 +454,36 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
             mma16816(o[n], sh_[u], bl[2 * u], bl[2 * u + 1]);
             mma16816(o[n], sl_[u], bh[2 * u], bh[2 * u + 1]);
           }
+          if constexpr (DELTA) {
+            ldsm4(at + (uint32_t)off_w(dkp, 0), bh);
+            ldsm4(at + (uint32_t)off_w(dkp, 1), bl);
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+              mma16816(w[n], sh_[u], bh[2 * u], bh[2 * u + 1]);
+              mma16816(w[n], sh_[u], bl[2 * u], bl[2 * u + 1]);
+              mma16816(w[n], sl_[u], bh[2 * u], bh[2 * u + 1]);
+            }
+          }
         }
       }
     }
     // v^T as A operand: rows = value columns, k = tokens (two steps of 16)
-    uint32_t va[2][4];
+    uint32_t va[2][4], vr[2][4];  // vr: the remainders
+    if constexpr (DELTA) {
+      const float* U = reinterpret_cast<const float*>(st_ + cbytes) + (warp * 16 + g) * kUStride + 2 * t;
 #pragma unroll
-    for (int u = 0; u < 2; ++u) {
-      // the four 8 x 8 blocks of v [tokens][columns], transposed: (cols 0-7, tok 0-7), (cols 8-15, tok 0-7), (cols 0-7, tok 8-15), ...
-      const int row = u * 16 + (lm >> 1) * 8 + lr, col = warp * 16 + (lm & 1) * 8;
-      ldsm4_trans(vbase + (uint32_t)(row * kVRow + col * 2), va[u]);
+      for (int n = 0; n < 4; ++n) {
+        const float2 x = *reinterpret_cast<const float2*>(U + n * 8), y = *reinterpret_cast<const float2*>(U + 8 * kUStride + n * 8);
+        split_bf16(x.x - w[n][0], x.y - w[n][1], va[n >> 1][(n & 1) * 2], vr[n >> 1][(n & 1) * 2]);
+        split_bf16(y.x - w[n][2], y.y - w[n][3], va[n >> 1][(n & 1) * 2 + 1], vr[n >> 1][(n & 1) * 2 + 1]);
+      }
+    } else {
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        // the four 8 x 8 blocks of v [tokens][columns], transposed: (cols 0-7, tok 0-7), (cols 8-15, tok 0-7), (cols 0-7, tok 8-15), ...
+        const int row = u * 16 + (lm >> 1) * 8 + lr, col = warp * 16 + (lm & 1) * 8;
+        ldsm4_trans(vbase + (uint32_t)(row * kVRow + col * 2), va[u]);
+      }
     }
 #pragma unroll
     for (int n = 0; n < 4; ++n) {
@@ -533,6 +495,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
       for (int u = 0; u < 2; ++u) {
         mma16816(o[n], va[u], bh[2 * u], bh[2 * u + 1]);
         mma16816(o[n], va[u], bl[2 * u], bl[2 * u + 1]);
+        if constexpr (DELTA) mma16816(o[n], vr[u], bh[2 * u], bh[2 * u + 1]);
       }
     }
     // the state moves on: decay its columns, add v^T k
@@ -552,6 +515,10 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
             ldsm4_trans(base + (uint32_t)(off_part(dkp, p) + row * qk_row(dkp) + col * 2), b);
             mma16816(acc[j], va[u], b[0], b[1]);
             mma16816(acc[j + 1], va[u], b[2], b[3]);
+            if (DELTA && p == 2) {
+              mma16816(acc[j], vr[u], b[0], b[1]);
+              mma16816(acc[j + 1], vr[u], b[2], b[3]);
+            }
           }
         }
       }
@@ -602,7 +569,7 @@ __global__ void __launch_bounds__(256) gla_out_kernel(Gla a) {
     T* dst = (T*)a.out + (size_t)row * a.out_stride + (size_t)head * a.dv;
     for (int c = lane * VEC; c < a.dv; c += 32 * VEC) {
       Vec<VEC> x = load_vec<VEC>(o + c);
-      const Vec<VEC> w = load_vec<VEC>(a.norm + c), g = mat_value<T, VEC>(a.src, row, a.col_g() + head * a.dv + c);
+      const Vec<VEC> w = load_vec<VEC>(a.norm + c), g = mat_value<T, VEC>(a.src, row, a.col_g + head * a.dv + c);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) x.v[e] *= r * w.v[e] * silu(g.v[e]);
       store_vec<VEC>(dst + c, x);
@@ -725,7 +692,7 @@ __global__ void __launch_bounds__(256) memory_out_kernel(Gla a) {
     T* dst = (T*)a.out + (size_t)row * a.out_stride + (size_t)head * a.dv;
     for (int c = lane * VEC; c < a.dv; c += 32 * VEC) {
       Vec<VEC> x = load_vec<VEC>(o + c);
-      const Vec<VEC> w = load_vec<VEC>(a.norm + head * a.dv + c), g = mat_value<T, VEC>(a.src, row, a.col_g() + head * a.dv + c);
+      const Vec<VEC> w = load_vec<VEC>(a.norm + head * a.dv + c), g = mat_value<T, VEC>(a.src, row, a.col_g + head * a.dv + c);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) x.v[e] *= r * w.v[e] * sigmoid(g.v[e]);
       store_vec<VEC>(dst + c, x);
@@ -733,43 +700,63 @@ __global__ void __launch_bounds__(256) memory_out_kernel(Gla a) {
   }
 }
 
-int pad_channels(int dk) { return (dk + 31) / 32 * 32; }
-int slices_of(int dv) { return (dv + kScanCols - 1) / kScanCols; }
-
-template <int NT>
+template <int NT, bool DELTA>
 b200_status launch_scan(Gla& a, int n_req, cudaStream_t s) {
-  const size_t stage = chunk_size(a.dkp) + kVSlice;
+  const size_t stage = DELTA ? delta_chunk_size(a.dkp) + kUSlice : chunk_size(a.dkp) + kVSlice;
   a.stages = (int)std::min<size_t>(4, (220 * 1024) / stage);
   const size_t smem = a.stages * (stage + sizeof(uint64_t)) + 128;
   static bool configured = false;
   if (!configured) {
-    B200_CUDA_TRY(cudaFuncSetAttribute(gla_scan_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
+    B200_CUDA_TRY((cudaFuncSetAttribute(gla_scan_kernel<NT, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024)));
     configured = true;
   }
-  gla_scan_kernel<NT><<<dim3(n_req, a.heads, a.n_slices), kScanWarps * 32, smem, s>>>(a);
+  gla_scan_kernel<NT, DELTA><<<dim3(n_req, a.heads, a.n_slices), kScanWarps * 32, smem, s>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
 
+template <bool DELTA>
+b200_status launch_scan_of(Gla& a, int n_req, cudaStream_t s) {
+  if (a.dkp <= 32) return launch_scan<4, DELTA>(a, n_req, s);
+  if (a.dkp <= 64) return launch_scan<8, DELTA>(a, n_req, s);
+  return a.dkp <= 128 ? launch_scan<16, DELTA>(a, n_req, s) : launch_scan<32, DELTA>(a, n_req, s);
+}
+
 }  // namespace
+
+b200_status b200_gla_scan(Gla& a, int n_req, bool delta, cudaStream_t s) { return delta ? launch_scan_of<true>(a, n_req, s) : launch_scan_of<false>(a, n_req, s); }
+
+b200_status b200_gla_out(const Gla& a, int chunks, bool wide, cudaStream_t s) {
+  auto* kernel = wide ? gla_out_kernel<__nv_bfloat16, 4> : gla_out_kernel<__nv_bfloat16, 1>;
+  kernel<<<dim3(chunks, a.heads), 256, 0, s>>>(a);
+  B200_LAUNCH_CHECK();
+  return B200_OK;
+}
 
 bool b200_gla_takes_chunks(int dk, int dv, int elem_bytes) { return elem_bytes == 2 && dk <= 256; }
 
-void GlaScratch::need(int heads, int dk, int dv) {
-  chunk_bytes = std::max(chunk_bytes, heads * chunk_size(pad_channels(dk)));
-  v_bytes = std::max(v_bytes, heads * slices_of(dv) * kVSlice);
+void GlaScratch::need(int heads, int dk, int dv, bool delta) {
+  chunk_bytes = std::max(chunk_bytes, heads * (delta ? delta_chunk_size(pad_channels(dk)) : chunk_size(pad_channels(dk))));
+  v_bytes = std::max(v_bytes, heads * slices_of(dv) * (delta ? kUSlice : kVSlice));
   o_elems = std::max(o_elems, (size_t)heads * dv);
+}
+
+void GlaScratch::need_delta(int heads, int kv_heads, int dk, int dv, bool chunks) {
+  if (chunks) need(heads, dk, dv, true);
+  row_elems = std::max(row_elems, ((size_t)2 * kv_heads * dk + (size_t)heads * dv + 3) / 4 * 4);
+  gate_heads = std::max(gate_heads, heads);
 }
 
 bool GlaScratch::alloc() {
   max_chunks = max_rows / kC + max_reqs;
   auto get = [](auto** p, size_t bytes) { return cudaMalloc((void**)p, std::max<size_t>(bytes, 16)) == cudaSuccess; };
   return get(&chunks, max_chunks * chunk_bytes) && get(&values, max_chunks * v_bytes) && get(&o, sizeof(float) * o_elems * max_rows) &&
-         get(&plan, sizeof(int4) * max_chunks) && get(&first_chunk, sizeof(int) * (max_reqs + 1));
+         get(&plan, sizeof(int4) * max_chunks) && get(&first_chunk, sizeof(int) * (max_reqs + 1)) &&
+         get(&rows, sizeof(float) * row_elems * max_rows) && get(&gates, sizeof(float2) * gate_heads * max_rows);
 }
 
 void GlaScratch::free() {
-  void* ptrs[] = {chunks, values, o, plan, first_chunk};
+  void* ptrs[] = {chunks, values, o, plan, first_chunk, rows, gates};
   for (void* p : ptrs) if (p) cudaFree(p);
 }
 
@@ -800,7 +787,7 @@ b200_status b200_gla_run(b200_kv* kv, const GlaScratch& g, const GlaCall& c, con
                          const int32_t* d_pos, int n_req, int total_rows, bool chunked, void* stream) {
   const bool mem = c.gates != nullptr;
   if (c.layer < 0 || c.layer >= kv->cfg.n_layers ||
-      (mem ? kv->lay[c.layer].rec_elems < b200_memory_elems(c.heads, c.dk, c.dv) : kv->lay[c.layer].rec_elems != c.heads * c.dk * c.dv)) {
+      (mem ? kv->lay[c.layer].rec_elems < b200_memory_elems(c.heads, c.dk, c.dv) : kv->lay[c.layer].rec_elems < c.heads * c.dk * c.dv)) {
     b200_set_error("gla: layer %d of the pool has no state of %d x %d x %d", c.layer, c.heads, c.dk, c.dv);
     return B200_ERR_INVALID_ARGUMENT;
   }
@@ -813,6 +800,7 @@ b200_status b200_gla_run(b200_kv* kv, const GlaScratch& g, const GlaCall& c, con
   a.rec_elems = kv->lay[c.layer].rec_elems;
   a.heads = c.heads; a.dk = c.dk; a.dv = c.dv; a.rank = c.rank; a.dkp = pad_channels(c.dk);
   a.dva = mem ? c.dv + 1 : c.dv; a.dvs = mem ? b200_memory_width(c.dv) : c.dv;
+  a.col_g = c.col0 + 2 * c.heads * c.dk + c.heads * c.dv;
   a.gates = c.gates; a.col0 = c.col0; a.den_eps = c.den_eps; a.out_scale = c.out_scale;
   a.src = c.src; a.a2 = c.a2; a.a2_bias = c.a2_bias; a.norm = c.norm; a.q_scale = c.q_scale; a.inv_tau = c.inv_tau; a.eps = c.eps;
   a.out = c.out; a.out_stride = c.out_stride; a.cu = d_cu; a.row_seq = d_row_seq; a.pos = d_pos; a.n_req = n_req; a.total_rows = total_rows;
@@ -854,10 +842,10 @@ b200_status b200_gla_run(b200_kv* kv, const GlaScratch& g, const GlaCall& c, con
                            : (wide ? gla_chunk_kernel<__nv_bfloat16, 4> : gla_chunk_kernel<__nv_bfloat16, 1>);
   chunk_kernel<<<dim3(chunks, c.heads), 256, smem, s>>>(a);
   B200_LAUNCH_CHECK();
-  b200_status st = a.dkp <= 32 ? launch_scan<4>(a, n_req, s) : (a.dkp <= 64 ? launch_scan<8>(a, n_req, s) : (a.dkp <= 128 ? launch_scan<16>(a, n_req, s) : launch_scan<32>(a, n_req, s)));
+  b200_status st = b200_gla_scan(a, n_req, false, s);
   if (st != B200_OK) return st;
-  auto* out_kernel = mem ? (wide ? memory_out_kernel<__nv_bfloat16, 4> : memory_out_kernel<__nv_bfloat16, 1>)
-                         : (wide ? gla_out_kernel<__nv_bfloat16, 4> : gla_out_kernel<__nv_bfloat16, 1>);
+  if (!mem) return b200_gla_out(a, chunks, wide, s);
+  auto* out_kernel = wide ? memory_out_kernel<__nv_bfloat16, 4> : memory_out_kernel<__nv_bfloat16, 1>;
   out_kernel<<<dim3(chunks, c.heads), 256, 0, s>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;

@@ -46,8 +46,14 @@ struct GlaScratch {
   float* o = nullptr;
   int4* plan = nullptr;      // [max_chunks] {first row, rows, request, -}
   int* first_chunk = nullptr;  // [max_reqs + 1]
+  // delta rule (delta.cuh): q, k and v of a row behind their convolutions, and {log decay, beta} per head
+  size_t row_elems = 0;
+  int gate_heads = 0;
+  float* rows = nullptr;
+  float2* gates = nullptr;
   bool alloc();              // false: out of memory
-  void need(int heads, int dk, int dv);  // before alloc: a layer of this shape will use it
+  void need(int heads, int dk, int dv, bool delta = false);  // before alloc: a layer of this shape will use it
+  void need_delta(int heads, int kv_heads, int dk, int dv, bool chunks);
   void free();
 };
 

@@ -97,6 +97,8 @@ struct WindowAttnCall {
   float scale = 1.f;
   const float* slopes_log2 = nullptr;
   const float* sinks_log2 = nullptr;
+  const float* dist_log2 = nullptr;  // [n_q_heads][dist_len], bias by distance (the last one for all beyond)
+  int dist_len = 0;
   void* out = nullptr;
   int out_stride = 0;
   int out_head_stride = 0;  // elements between heads of an output row (0: value_dim)

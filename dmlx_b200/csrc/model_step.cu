@@ -150,10 +150,11 @@ b200_status b200_model::step(b200_kv* kv, const b200_pack_desc* descs, int n_req
   }
   if (total > max_rows) { b200_set_error("model step: %lld rows > max_rows %d", total, max_rows); return B200_ERR_CAPACITY; }
   // positions beyond a page table would be read from the next sequence's
-  const long long most = (long long)kv->cfg.max_pages_per_seq * kv->cfg.page_size;
+  long long most = (long long)kv->cfg.max_pages_per_seq * kv->cfg.page_size;
+  if (max_positions > 0) most = std::min<long long>(most, max_positions);
   for (int i = 0; i < n_req; ++i)
     if (descs[i].base_pos < 0 || (long long)descs[i].base_pos + std::max(descs[i].count, 0) > most) {
-      b200_set_error("model step: positions %d + %d exceed the %lld a page table holds", descs[i].base_pos, descs[i].count, most);
+      b200_set_error("model step: positions %d + %d exceed the %lld a sequence may have", descs[i].base_pos, descs[i].count, most);
       return B200_ERR_INVALID_BATCH_INDEX;
     }
   for (int32_t r : want)
@@ -200,7 +201,7 @@ b200_status b200_model::step(b200_kv* kv, const b200_pack_desc* descs, int n_req
 extern "C" {
 
 void b200_model_get_info(const b200_model* m, b200_model_info* out) {
-  *out = b200_model_info{m->vocab, m->max_rows, m->max_reqs, m->max_seqs, m->logits_f32 ? 1 : 0};
+  *out = b200_model_info{m->vocab, m->max_rows, m->max_reqs, m->max_seqs, m->logits_f32 ? 1 : 0, m->max_positions};
 }
 
 b200_status b200_model_step(b200_model* m, b200_kv* kv, const b200_pack_desc* h_desc, int32_t n_req, const uint32_t* h_prefill_tokens,

@@ -18,6 +18,7 @@ b200_status b200_scatter_tokens(const uint32_t* d_next, const b200_pack_desc* d_
 
 struct b200_model {
   int vocab = 0, max_rows = 0, max_reqs = 0, max_seqs = 0;
+  int max_positions = 0;  // positions a sequence may have, 0: as many as its page table holds
   bool logits_f32 = false;
   bool ready = false;  // every weight is in place
   void* logits = nullptr;  // [max_reqs + extra_rows, vocab], bf16 or f32

@@ -249,7 +249,7 @@ __global__ void __launch_bounds__(1024) table_place_kernel(const MoeTableLayer* 
 // One warp per token.  Softmax scores in f32; the experts form n_groups equal groups of neighbours, of which only the `keep` with the
 // largest best score stay open; the k largest open scores are chosen and weighed by score / (their sum + 1e-20).
 template <typename T, int PER>
-__global__ void __launch_bounds__(256) route_src_kernel(MatSrc logits, int n_tokens, int n_experts, int k, int n_groups, int keep,
+__global__ void __launch_bounds__(256) route_src_kernel(MatSrc logits, int n_tokens, int n_experts, int k, int n_groups, int keep, RouterScores scores,
                                                         uint32_t* __restrict__ out_idx, float* __restrict__ out_w) {
   const int token = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (token >= n_tokens) return;
@@ -328,8 +328,9 @@ __global__ void __launch_bounds__(256) route_src_kernel(MatSrc logits, int n_tok
   }
   if (lane < k) {
     out_idx[(size_t)token * k + lane] = (uint32_t)mine_e;
-    out_w[(size_t)token * k + lane] = mine / (total + 1e-20f);
+    out_w[(size_t)token * k + lane] = (scores.renormalise ? mine / (total + 1e-20f) : mine) * scores.scale;
   }
+  if (scores.shared && lane == 0) scores.shared[token] = 1.0f / (1.0f + expf(-mat_value<T, 1>(logits, token, n_experts).v[0]));
 }
 
 // The plan of one layer in one launch, a CTA per expert: it counts the assignments of the experts before its own and places its
@@ -512,7 +513,7 @@ b200_status b200_moe_table_plan(const MoeTableLayer* d_layers, int n_layers, int
 }
 
 b200_status b200_moe_route_plan(const MoeTableLayer& L, const MatSrc& logits, bool f32, int n_groups, int keep_groups, int n_tokens, int tile_rows,
-                                float* d_weights, void* stream) {
+                                float* d_weights, void* stream, const RouterScores& scores) {
   if (L.n_experts <= 0 || L.n_experts > kMaxExperts || L.top <= 0 || L.top > kMaxRouterTop || n_groups <= 0 || n_groups > kMaxGroups ||
       L.n_experts % n_groups != 0 || keep_groups <= 0 || keep_groups > n_groups || L.top > keep_groups * (L.n_experts / n_groups)) {
     b200_set_error("router: %d experts, top %d, %d of %d groups", L.n_experts, L.top, keep_groups, n_groups);
@@ -520,7 +521,7 @@ b200_status b200_moe_route_plan(const MoeTableLayer& L, const MatSrc& logits, bo
   }
   if (n_tokens <= 0) return B200_OK;
   cudaStream_t s = (cudaStream_t)stream;
-  auto route = [&](auto* kernel) { kernel<<<(n_tokens + 7) / 8, 256, 0, s>>>(logits, n_tokens, L.n_experts, L.top, n_groups, keep_groups, L.indices, d_weights); };
+  auto route = [&](auto* kernel) { kernel<<<(n_tokens + 7) / 8, 256, 0, s>>>(logits, n_tokens, L.n_experts, L.top, n_groups, keep_groups, scores, L.indices, d_weights); };
   const int per = (L.n_experts + 31) / 32;
   if (f32) route(per <= 1 ? route_src_kernel<float, 1> : (per <= 4 ? route_src_kernel<float, 4> : (per <= 8 ? route_src_kernel<float, 8> : route_src_kernel<float, 32>)));
   else route(per <= 1 ? route_src_kernel<__nv_bfloat16, 1> : (per <= 4 ? route_src_kernel<__nv_bfloat16, 4> : (per <= 8 ? route_src_kernel<__nv_bfloat16, 8> : route_src_kernel<__nv_bfloat16, 32>)));

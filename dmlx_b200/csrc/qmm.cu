@@ -96,26 +96,37 @@ __device__ __forceinline__ void row_params(const unsigned char* blk, int r, int 
 // gelu(z) = z Phi(z), the exact form.
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 
+// The epilogues of dense bf16 weights that act on every output by itself.
+__host__ __device__ __forceinline__ bool elementwise(int epilogue) { return epilogue == B200_EPI_GELU || epilogue == B200_EPI_RELU2; }
+__device__ __forceinline__ float activate(int epilogue, float z) {
+  if (epilogue == B200_EPI_GELU) return gelu_erf(z);
+  if (epilogue == B200_EPI_RELU2) { z = fmaxf(z, 0.f); return z * z; }
+  return z;
+}
+// Gate and up of the SwiGLU epilogue: both clamped where there is a limit, then g sigmoid(alpha g) (u + shift).
+__device__ __forceinline__ float gated(const QmmArgs& a, float g, float u) {
+  if (a.swiglu_limit > 0.f) {
+    const float L = a.swiglu_limit;
+    g = fminf(g, L);
+    u = fminf(fmaxf(u, -L), L);
+  }
+  return g / (1.0f + __expf(-a.swiglu_alpha * g)) * (u + a.swiglu_shift);
+}
+
 // Epilogue of one output quad: columns n..n+3 of row `token` (residual add, SwiGLU over
 // interleaved gate/up rows, GELU, per-row scale), written as bf16.
 __device__ __forceinline__ void finish_store(const QmmArgs& a, int token, int n, float4 acc) {
   const float rs = a.row_scale(token);
   if (a.epilogue == B200_EPI_SWIGLU) {
-    float g0 = acc.x, u0 = acc.y, g1 = acc.z, u1 = acc.w;
-    if (a.swiglu_limit > 0.f) {
-      const float L = a.swiglu_limit;
-      g0 = fminf(g0, L); g1 = fminf(g1, L);
-      u0 = fminf(fmaxf(u0, -L), L); u1 = fminf(fmaxf(u1, -L), L);
-    }
-    const float y0 = g0 / (1.0f + __expf(-g0)) * u0 * rs, y1 = g1 / (1.0f + __expf(-g1)) * u1 * rs;
+    const float y0 = gated(a, acc.x, acc.y) * rs, y1 = gated(a, acc.z, acc.w) * rs;
     *reinterpret_cast<__nv_bfloat162*>(a.y + (size_t)a.row_base_out(token) * a.out_stride(a.n / 2) + n / 2) = __floats2bfloat162_rn(y0, y1);
   } else {
     const size_t o = (size_t)a.row_base_out(token) * a.out_stride(a.n) + n;
     if (a.epilogue == B200_EPI_RESIDUAL) {
       const uint2 rv = *reinterpret_cast<const uint2*>(a.residual + o);
       acc.x += ptx::bf16_lo(rv.x); acc.y += ptx::bf16_hi(rv.x); acc.z += ptx::bf16_lo(rv.y); acc.w += ptx::bf16_hi(rv.y);
-    } else if (a.epilogue == B200_EPI_GELU) {
-      acc.x = gelu_erf(acc.x); acc.y = gelu_erf(acc.y); acc.z = gelu_erf(acc.z); acc.w = gelu_erf(acc.w);
+    } else if (elementwise(a.epilogue)) {
+      acc.x = activate(a.epilogue, acc.x); acc.y = activate(a.epilogue, acc.y); acc.z = activate(a.epilogue, acc.z); acc.w = activate(a.epilogue, acc.w);
     }
     __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x * rs, acc.y * rs), hi = __floats2bfloat162_rn(acc.z * rs, acc.w * rs);
     uint2 ov;
@@ -463,10 +474,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
             const float mine = __uint_as_float(v[j]);
             const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
             if ((lane & 1) == 0 && c0 + j < rows_here && n < a.n) {
-              float g = mine, u = other;
-              if (a.swiglu_limit > 0.f) { g = fminf(g, a.swiglu_limit); u = fminf(fmaxf(u, -a.swiglu_limit), a.swiglu_limit); }
               const int token = t0 + c0 + j;
-              a.y[(size_t)token * a.out_stride(a.n / 2) + n / 2] = __float2bfloat16(g / (1.0f + __expf(-g)) * u * a.row_scale(token));
+              a.y[(size_t)token * a.out_stride(a.n / 2) + n / 2] = __float2bfloat16(gated(a, mine, other) * a.row_scale(token));
             }
           }
         } else {
@@ -481,7 +490,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) qmm_tc_kernel(const __grid_cons
                 continue;
               }
               if (a.epilogue == B200_EPI_RESIDUAL) acc += __bfloat162float(a.residual[o]);
-              else if (MODE == B200_Q_BF16 && a.epilogue == B200_EPI_GELU) acc = gelu_erf(acc);
+              else if (MODE == B200_Q_BF16) acc = activate(a.epilogue, acc);
               a.y[o] = __float2bfloat16(acc * a.row_scale(token));
             }
           }
@@ -506,7 +515,6 @@ __device__ __forceinline__ void tile_epilogue_store(const QmmArgs& a, const uint
   } else if (a.epilogue == B200_EPI_SWIGLU) {
     // rows 2i / 2i+1 of the tile are gate_i / up_i: neighbouring lanes.  The even lane takes token j,
     // the odd lane token j+1 (one exchange per token pair, no lane idles in the arithmetic).
-    const float L = a.swiglu_limit;
     const bool odd = lane & 1;
 #pragma unroll
     for (int j = 0; j < 32; j += 2) {
@@ -514,10 +522,8 @@ __device__ __forceinline__ void tile_epilogue_store(const QmmArgs& a, const uint
       const float got = __shfl_xor_sync(0xffffffffu, odd ? a0 : a1, 1);
       const int tok = c0 + j + (int)odd;
       if (tok < rows_here && n < a.n) {
-        float g = odd ? got : a0, u = odd ? a1 : got;
-        if (L > 0.f) { g = fminf(g, L); u = fminf(fmaxf(u, -L), L); }
         const int token = t0 + tok;
-        a.y[(size_t)token * a.out_stride(a.n / 2) + n / 2] = __float2bfloat16(g / (1.0f + __expf(-g)) * u * a.row_scale(token));
+        a.y[(size_t)token * a.out_stride(a.n / 2) + n / 2] = __float2bfloat16(gated(a, odd ? got : a0, odd ? a1 : got) * a.row_scale(token));
       }
     }
   } else {
@@ -528,7 +534,7 @@ __device__ __forceinline__ void tile_epilogue_store(const QmmArgs& a, const uint
         const size_t o = (size_t)token * a.out_stride(a.n) + n;
         float acc = __uint_as_float(v[j]);
         if (a.epilogue == B200_EPI_RESIDUAL) acc += __bfloat162float(a.residual[o]);
-        else if (a.epilogue == B200_EPI_GELU) acc = gelu_erf(acc);
+        else acc = activate(a.epilogue, acc);
         a.y[o] = __float2bfloat16(acc * a.row_scale(token));
       }
     }
@@ -943,7 +949,6 @@ __global__ void __launch_bounds__(kTc2Threads, 1) qmm_tc2_kernel(const __grid_co
       if (all_ok) {
         ptx::tc_fence_after_sync();
         __nv_bfloat16* stage_h = reinterpret_cast<__nv_bfloat16*>(smem);
-        const float L = a.swiglu_limit;
         if (etile < n_tiles) {
           const int lq = warp & 3;
           const int ch = ((tn / 2 + 31) / 32) * 32;
@@ -960,11 +965,9 @@ __global__ void __launch_bounds__(kTc2Threads, 1) qmm_tc2_kernel(const __grid_co
             for (int j = 0; j < 32; j += 2) {
               const float a0 = __uint_as_float(v[j]), a1 = __uint_as_float(v[j + 1]);
               const float got = __shfl_xor_sync(0xffffffffu, odd ? a0 : a1, 1);
-              float g = odd ? got : a0, u = odd ? a1 : got;
               const float rs = __shfl_sync(0xffffffffu, rs_mine, j + (int)odd);
-              if (L > 0.f) { g = fminf(g, L); u = fminf(fmaxf(u, -L), L); }
               stage_h[((size_t)(c0 + j + (int)odd) * 2 + etile) * 64 + lq * 16 + (lane >> 1)] =
-                  __float2bfloat16(g / (1.0f + __expf(-g)) * u * rs);
+                  __float2bfloat16(gated(a, odd ? got : a0, odd ? a1 : got) * rs);
             }
           }
         }
@@ -1757,7 +1760,6 @@ __global__ void __launch_bounds__(kMxThreads, 1)
       const bool swiglu = a.epilogue == B200_EPI_SWIGLU;
       const int out_per_tile = swiglu ? kTileN / 2 : kTileN, chunks = out_per_tile / 8;
       const int n_out = swiglu ? a.n / 2 : a.n;
-      const float L = a.swiglu_limit;
       for (int tile = 0; tile < n_tiles; ++tile) {
         for (int idx = tid; idx < rows_here * chunks; idx += 128) {
           const int tok = idx / chunks, ch = idx - tok * chunks;
@@ -1770,10 +1772,8 @@ __global__ void __launch_bounds__(kMxThreads, 1)
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
               const float4 f = reinterpret_cast<const float4*>(src)[q];  // gate, up, gate, up
-              float g0 = f.x, u0 = f.y, g1 = f.z, u1 = f.w;
-              if (L > 0.f) { g0 = fminf(g0, L); u0 = fminf(fmaxf(u0, -L), L); g1 = fminf(g1, L); u1 = fminf(fmaxf(u1, -L), L); }
-              o[2 * q] = g0 / (1.0f + __expf(-g0)) * u0 * rs;
-              o[2 * q + 1] = g1 / (1.0f + __expf(-g1)) * u1 * rs;
+              o[2 * q] = gated(a, f.x, f.y) * rs;
+              o[2 * q + 1] = gated(a, f.z, f.w) * rs;
             }
           } else {
             const float4 f0 = reinterpret_cast<const float4*>(src)[0], f1 = reinterpret_cast<const float4*>(src)[1];
@@ -1970,7 +1970,6 @@ __global__ void __launch_bounds__(kMxpThreads, 1)
     const bool swiglu = a.epilogue == B200_EPI_SWIGLU;
     const int out_per_tile = swiglu ? kTileN / 2 : kTileN, chunks = out_per_tile / 8;
     const int n_out = swiglu ? a.n / 2 : a.n;
-    const float L = a.swiglu_limit;
     uint32_t n_done = 0;
     for (int w = blockIdx.x; w < n_work; w += gridDim.x, ++n_done) {
       const Work k = decode(w);
@@ -2026,10 +2025,8 @@ __global__ void __launch_bounds__(kMxpThreads, 1)
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
               const float4 f = reinterpret_cast<const float4*>(src)[q];  // gate, up, gate, up
-              float g0 = f.x, u0 = f.y, g1 = f.z, u1 = f.w;
-              if (L > 0.f) { g0 = fminf(g0, L); u0 = fminf(fmaxf(u0, -L), L); g1 = fminf(g1, L); u1 = fminf(fmaxf(u1, -L), L); }
-              o[2 * q] = g0 / (1.0f + __expf(-g0)) * u0 * rs;
-              o[2 * q + 1] = g1 / (1.0f + __expf(-g1)) * u1 * rs;
+              o[2 * q] = gated(a, f.x, f.y) * rs;
+              o[2 * q + 1] = gated(a, f.z, f.w) * rs;
             }
           } else {
             const float4 f0 = reinterpret_cast<const float4*>(src)[0], f1 = reinterpret_cast<const float4*>(src)[1];
@@ -2068,8 +2065,10 @@ __global__ void __launch_bounds__(kMxpThreads, 1)
 // address in their kernel arguments and keep writing their partial sums there.  An outgrown buffer is
 // retired (kept until the process exits) and new launches use the larger one; no device-wide
 // synchronisation is needed for that.
-float* g_ws = nullptr;
-size_t g_ws_bytes = 0;
+// (two of them: the partial sums of one deferred matmul may wait while another one runs)
+float* g_ws[2] = {nullptr, nullptr};
+size_t g_ws_bytes[2] = {0, 0};
+int g_place = 0;
 int* g_err = nullptr;
 int g_sms = 0;
 std::vector<void*> g_retired;  // outgrown scratch buffers, still referenced by captured graphs
@@ -2082,13 +2081,13 @@ b200_status ensure_state(size_t ws_bytes) {
     B200_CUDA_TRY(cudaGetDevice(&dev));
     B200_CUDA_TRY(cudaDeviceGetAttribute(&g_sms, cudaDevAttrMultiProcessorCount, dev));
   }
-  if (ws_bytes > g_ws_bytes) {
+  if (ws_bytes > g_ws_bytes[g_place]) {
     const size_t want = std::max(ws_bytes + ws_bytes / 4, (size_t)64 << 20);
     float* grown = nullptr;
     B200_CUDA_TRY(cudaMalloc((void**)&grown, want));
-    if (g_ws) g_retired.push_back(g_ws);
-    g_ws = grown;
-    g_ws_bytes = want;
+    if (g_ws[g_place]) g_retired.push_back(g_ws[g_place]);
+    g_ws[g_place] = grown;
+    g_ws_bytes[g_place] = want;
   }
   return B200_OK;
 }
@@ -2329,7 +2328,7 @@ static b200_status launch_simt(QmmArgs& a, int rows, cudaStream_t s) {
   const int splits = (a.kc + a.chunks_per_split - 1) / a.chunks_per_split;
   st = ensure_state((size_t)splits * (size_t)tts * TT * a.nt * kTileN * sizeof(float));
   if (st != B200_OK) return st;
-  a.ws = g_ws; a.err = g_err;
+  a.ws = g_ws[g_place]; a.err = g_err;
   qmm_simt_kernel<MODE, TT><<<dim3(a.nt, splits, tts), kTileN, 0, s>>>(a);
   B200_LAUNCH_CHECK();
   return launch_finish(a, splits, s);
@@ -2376,7 +2375,7 @@ static b200_status launch_tc(QmmArgs& a, int rows, cudaStream_t s, int x_stride 
   const int splits = (a.kc + a.chunks_per_split - 1) / a.chunks_per_split;
   st = ensure_state(grouped_bf16 ? 0 : (size_t)splits * (a.items ? (size_t)rows : (size_t)tts * tn) * a.nt * kTileN * sizeof(float));
   if (st != B200_OK) return st;
-  a.ws = g_ws; a.err = g_err;
+  a.ws = g_ws[g_place]; a.err = g_err;
   CUtensorMap xmap;
   st = make_x_map(&xmap, a.x, rows, x_stride > 0 ? x_stride : a.k, tn);
   if (st != B200_OK) return st;
@@ -2436,7 +2435,7 @@ static b200_status launch_tca(QmmArgs& a, int rows, cudaStream_t s) {
   const bool direct = splits == 1 && (tn <= 64 || a.direct_large) && !a.keep_f32;
   st = ensure_state(direct ? 0 : (size_t)splits * (a.items ? (size_t)rows : (size_t)tts * tn) * a.nt * kTileN * sizeof(float));
   if (st != B200_OK) return st;
-  a.ws = g_ws; a.err = g_err;
+  a.ws = g_ws[g_place]; a.err = g_err;
   CUtensorMap xmap;
   st = make_x_map(&xmap, a.x, rows, a.k, tn);
   if (st != B200_OK) return st;
@@ -2569,7 +2568,7 @@ static b200_status launch_mx(const b200_qweight* w, QmmArgs& a, int rows, cudaSt
     if (real_splits > 1) {
       st = ensure_state((size_t)real_splits * (size_t)tts * tn * a.nt * kTileN * sizeof(float));
       if (st != B200_OK) return st;
-      a.ws = g_ws;
+      a.ws = g_ws[g_place];
     }
     const long long n_work = a.items ? (long long)pairs * a.max_items : (long long)pairs * tts * real_splits;
     const int grid = (int)std::max<long long>(1, std::min<long long>(g_sms, n_work));
@@ -2628,7 +2627,7 @@ static b200_status launch_tc2(QmmArgs& a, int rows, cudaStream_t s) {
   const int splits = (a.kc + a.chunks_per_split - 1) / a.chunks_per_split;
   st = ensure_state(splits > 1 || a.keep_f32 ? (size_t)splits * (size_t)tts * tn * a.nt * kTileN * sizeof(float) : 0);
   if (st != B200_OK) return st;
-  a.ws = g_ws; a.err = g_err;
+  a.ws = g_ws[g_place]; a.err = g_err;
   CUtensorMap xmap;
   st = make_x_map(&xmap, a.x, rows, a.k, tn);
   if (st != B200_OK) return st;
@@ -2669,7 +2668,7 @@ static b200_status launch_mma_nt(QmmArgs& a, int rows, cudaStream_t s) {
   a.chunks_per_split = (a.kc + splits - 1) / splits;
   st = ensure_state((size_t)splits * (size_t)tts * tile * a.nt * kTileN * sizeof(float));
   if (st != B200_OK) return st;
-  a.ws = g_ws; a.err = g_err;
+  a.ws = g_ws[g_place]; a.err = g_err;
   a.x_slab = 1;
   const size_t smem = base_smem + slab_bytes(a.chunks_per_split);
   static bool configured = false;
@@ -2714,7 +2713,7 @@ static b200_status launch_mma8_nt(QmmArgs& a, int rows, cudaStream_t s) {
   a.chunks_per_split = (a.kc + splits - 1) / splits;
   st = ensure_state((size_t)splits * (size_t)tts * tile * a.nt * kTileN * sizeof(float));
   if (st != B200_OK) return st;
-  a.ws = g_ws; a.err = g_err;
+  a.ws = g_ws[g_place]; a.err = g_err;
   a.x_slab = 1;
   const size_t smem = base_smem + slab_bytes(a.chunks_per_split);
   static bool configured = false;
@@ -2758,6 +2757,7 @@ extern "C" b200_status b200_qmm(const b200_qweight* w, const void* d_x, int32_t 
 // Set by b200_qmm_deferred around its call of qmm_entry (one calling thread per process uses the matmul entry points).
 static b200_qmm_partials* g_defer_target = nullptr;
 static int g_y_stride = 0;         // set by b200_qmm_to around its call
+static SwigluShape g_shape;        // likewise
 static bool g_defer_always = false;  // defer = 2: also when K is not split
 
 extern "C" b200_status b200_qmm_deferred(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t defer, void* stream,
@@ -2772,10 +2772,19 @@ extern "C" b200_status b200_qmm_deferred(const b200_qweight* w, const void* d_x,
   return st;
 }
 
-b200_status b200_qmm_to(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t y_stride, int32_t epilogue, void* stream) {
+b200_status b200_qmm_deferred_aside(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t defer, void* stream, b200_qmm_partials* out) {
+  g_place = 1;
+  const b200_status st = b200_qmm_deferred(w, d_x, rows, d_y, defer, stream, out);
+  g_place = 0;
+  return st;
+}
+
+b200_status b200_qmm_to(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t y_stride, int32_t epilogue, void* stream, const SwigluShape& shape) {
   if (w->mode != B200_Q_BF16 || epilogue == B200_EPI_RESIDUAL || y_stride % 8 != 0) { b200_set_error("qmm_to: dense bf16 weights, no residual, output rows of 16-byte multiples"); return B200_ERR_INVALID_ARGUMENT; }
   g_y_stride = y_stride;
-  const b200_status st = qmm_entry(w, d_x, rows, d_y, epilogue, nullptr, 0.f, B200_QMM_AUTO, stream, nullptr, 0.f, nullptr, nullptr);
+  g_shape = shape;
+  const b200_status st = qmm_entry(w, d_x, rows, d_y, epilogue, nullptr, shape.limit, B200_QMM_AUTO, stream, nullptr, 0.f, nullptr, nullptr);
+  g_shape = SwigluShape{};
   g_y_stride = 0;
   return st;
 }
@@ -2806,7 +2815,7 @@ static b200_status qmm_entry(const b200_qweight* w, const void* d_x, int32_t row
   if (w->n_experts != 1) { b200_set_error("qmm: stacked expert weights go through the grouped entry point"); return B200_ERR_INVALID_ARGUMENT; }
   if (epilogue == B200_EPI_RESIDUAL && !d_residual) { b200_set_error("qmm: residual epilogue without a residual"); return B200_ERR_INVALID_ARGUMENT; }
   if (epilogue == B200_EPI_SWIGLU && (w->n % 2) != 0) { b200_set_error("qmm: SwiGLU needs an even N"); return B200_ERR_INVALID_ARGUMENT; }
-  if (epilogue == B200_EPI_GELU && w->mode != B200_Q_BF16) { b200_set_error("qmm: the GELU epilogue serves dense bf16 weights"); return B200_ERR_UNSUPPORTED; }
+  if (elementwise(epilogue) && w->mode != B200_Q_BF16) { b200_set_error("qmm: the elementwise epilogues serve dense bf16 weights"); return B200_ERR_UNSUPPORTED; }
   // Quantised weights, up to 16 rows: register-dequant mma.sync kernel (pure weight streaming).  More
   // rows: tcgen05 with the dequantised weights in tensor memory; above 128 rows the tile-pair kernel
   // where its grid is one well-filled wave without a K split (gate/up-sized matrices: 74 vs 85 us at
@@ -2850,6 +2859,7 @@ static b200_status qmm_entry(const b200_qweight* w, const void* d_x, int32_t row
   a.norm_w = (const __nv_bfloat16*)d_norm_w; a.norm_out = (__nv_bfloat16*)d_norm_out; a.norm_eps = norm_eps;
   a.defer = g_defer_target;
   a.y_stride = g_y_stride;
+  a.swiglu_alpha = g_shape.alpha; a.swiglu_shift = g_shape.shift;
   a.keep_f32 = g_defer_always ? 1 : 0;
   cudaStream_t s = (cudaStream_t)stream;
   auto dispatch = [&]() -> b200_status {
@@ -2891,7 +2901,8 @@ struct F32Args {
   const unsigned char* blocks;
   const float* x;
   float* y;
-  int rows, kc, x_stride, y_stride, n_valid, swiglu, gelu;
+  int rows, kc, x_stride, y_stride, n_valid, epilogue;
+  SwigluShape shape;
   size_t expert_stride;        // bytes between the matrices of a stack
   int x_group, y_group;        // block-diagonal: columns of x and y per matrix (grid z)
   const int4* items;           // grouped: {matrix, first sorted row, rows} (grid y)
@@ -2902,7 +2913,7 @@ struct F32Args {
 __global__ void __launch_bounds__(256) qmm_f32_kernel(F32Args a) {
   __shared__ float xs[kF32K][kF32Rows + 4];
   __shared__ float ws[kF32K][kTileN + 4];
-  const int nt = blockIdx.x, tid = threadIdx.x, kc = a.kc, n_valid = a.n_valid, y_stride = a.y_stride, swiglu = a.swiglu;
+  const int nt = blockIdx.x, tid = threadIdx.x, kc = a.kc, n_valid = a.n_valid, y_stride = a.y_stride;
   int r0 = blockIdx.y * kF32Rows, rows = a.rows;
   const unsigned char* blocks = a.blocks + (size_t)blockIdx.z * a.expert_stride;
   const float* x = a.x + (size_t)blockIdx.z * a.x_group;
@@ -2962,40 +2973,45 @@ __global__ void __launch_bounds__(256) qmm_f32_kernel(F32Args a) {
   for (int i = 0; i < 8; ++i) {
     const int row = r0 + tr + i;
     if (row >= rows) continue;
-    if (swiglu) {  // columns alternate gate, up
+    if (a.epilogue == B200_EPI_SWIGLU) {  // columns alternate gate, up
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int col = n / 2 + e;
-        const float gt = acc[i][2 * e], up = acc[i][2 * e + 1];
-        if (col < n_valid) y[(size_t)row * y_stride + col] = gt / (1.0f + expf(-gt)) * up;
+        const float L = a.shape.limit > 0.f ? a.shape.limit : INFINITY, gt = fminf(acc[i][2 * e], L), up = fminf(fmaxf(acc[i][2 * e + 1], -L), L);
+        if (col < n_valid) y[(size_t)row * y_stride + col] = gt / (1.0f + expf(-a.shape.alpha * gt)) * (up + a.shape.shift);
       }
     } else {
 #pragma unroll
       for (int e = 0; e < 4; ++e)
-        if (n + e < n_valid) y[(size_t)row * y_stride + n + e] = a.gelu ? gelu_erf(acc[i][e]) : acc[i][e];
+        if (n + e < n_valid) y[(size_t)row * y_stride + n + e] = activate(a.epilogue, acc[i][e]);
     }
   }
 }
 }  // namespace
 
-extern "C" b200_status b200_qmm_f32(const b200_qweight* w, const float* d_x, int32_t rows, float* d_y, int32_t y_stride, int32_t n_valid,
-                                    int32_t epilogue, void* stream) {
+b200_status b200_qmm_f32_shaped(const b200_qweight* w, const float* d_x, int32_t rows, float* d_y, int32_t y_stride, int32_t n_valid,
+                                int32_t epilogue, void* stream, const SwigluShape& shape) {
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
   if (w->mode != B200_Q_BF16 || w->n_experts != 1) { b200_set_error("qmm_f32: dense bf16 weights only"); return B200_ERR_UNSUPPORTED; }
   const bool swiglu = epilogue == B200_EPI_SWIGLU;
-  if ((epilogue != B200_EPI_NONE && epilogue != B200_EPI_GELU && !swiglu) || n_valid < 0 || n_valid > (swiglu ? w->n / 2 : w->n) || y_stride < n_valid) {
+  if ((epilogue != B200_EPI_NONE && !elementwise(epilogue) && !swiglu) || n_valid < 0 || n_valid > (swiglu ? w->n / 2 : w->n) || y_stride < n_valid) {
     b200_set_error("qmm_f32: bad epilogue, n_valid or stride");
     return B200_ERR_INVALID_ARGUMENT;
   }
   if (rows <= 0) return B200_OK;
   F32Args a{};
   a.blocks = w->d_blocks; a.x = d_x; a.y = d_y; a.rows = rows; a.kc = w->kc; a.x_stride = w->k; a.y_stride = y_stride; a.n_valid = n_valid;
-  a.swiglu = swiglu ? 1 : 0;
-  a.gelu = epilogue == B200_EPI_GELU ? 1 : 0;
+  a.epilogue = epilogue;
+  a.shape = shape;
   qmm_f32_kernel<<<dim3(w->nt, (rows + kF32Rows - 1) / kF32Rows), 256, 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
   return B200_OK;
+}
+
+extern "C" b200_status b200_qmm_f32(const b200_qweight* w, const float* d_x, int32_t rows, float* d_y, int32_t y_stride, int32_t n_valid,
+                                    int32_t epilogue, void* stream) {
+  return b200_qmm_f32_shaped(w, d_x, rows, d_y, y_stride, n_valid, epilogue, stream, SwigluShape{});
 }
 
 b200_status b200_qmm_f32_blocks(const b200_qweight* w, const float* d_x, int32_t x_stride, int32_t x_group, int32_t rows, float* d_y,
@@ -3017,11 +3033,11 @@ b200_status b200_qmm_f32_grouped(const b200_qweight* w, const float* d_x, const 
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
   const bool swiglu = epilogue == B200_EPI_SWIGLU;
-  if (w->mode != B200_Q_BF16 || (epilogue != B200_EPI_NONE && epilogue != B200_EPI_GELU && !swiglu)) { b200_set_error("qmm_f32_grouped: dense bf16 weights, no, the SwiGLU or the GELU epilogue"); return B200_ERR_UNSUPPORTED; }
+  if (w->mode != B200_Q_BF16 || (epilogue != B200_EPI_NONE && !elementwise(epilogue) && !swiglu)) { b200_set_error("qmm_f32_grouped: dense bf16 weights, no, the SwiGLU or an elementwise epilogue"); return B200_ERR_UNSUPPORTED; }
   if (max_items <= 0) return B200_OK;
   F32Args a{};
   a.blocks = w->d_blocks; a.x = d_x; a.y = d_y; a.kc = w->kc; a.x_stride = w->k; a.y_stride = y_stride; a.n_valid = swiglu ? w->n / 2 : w->n;
-  a.swiglu = swiglu ? 1 : 0; a.gelu = epilogue == B200_EPI_GELU ? 1 : 0; a.expert_stride = (size_t)w->nt * w->kc * w->block_bytes;
+  a.epilogue = epilogue; a.expert_stride = (size_t)w->nt * w->kc * w->block_bytes;
   a.items = d_items; a.n_items = d_n_items; a.order = d_order; a.order_div = order_div > 0 ? order_div : 1;
   qmm_f32_kernel<<<dim3(w->nt, max_items), 256, 0, (cudaStream_t)stream>>>(a);
   B200_LAUNCH_CHECK();
@@ -3052,7 +3068,7 @@ b200_status b200_qmm_grouped(const b200_qweight* w, const void* d_x, int32_t row
   b200_status st = b200_require_device();
   if (st != B200_OK) return st;
   if (rows <= 0) return B200_OK;
-  if (epilogue == B200_EPI_GELU && w->mode != B200_Q_BF16) { b200_set_error("qmm_grouped: the GELU epilogue serves dense bf16 weights"); return B200_ERR_UNSUPPORTED; }
+  if (elementwise(epilogue) && w->mode != B200_Q_BF16) { b200_set_error("qmm_grouped: the elementwise epilogues serve dense bf16 weights"); return B200_ERR_UNSUPPORTED; }
   QmmArgs a{};
   a.blocks = w->d_blocks; a.x = (const __nv_bfloat16*)d_x; a.y = (__nv_bfloat16*)d_y; a.residual = nullptr;
   a.row_scales = d_row_scales;
@@ -3254,7 +3270,7 @@ extern "C" b200_status b200_qmm_static_scratch(const b200_qweight* w, const void
   if (rows <= 0) return B200_OK;
   if (w->n_experts != 1) { b200_set_error("qmm (static scratch): single weights only"); return B200_ERR_INVALID_ARGUMENT; }
   if (epilogue == B200_EPI_RESIDUAL && !d_residual) { b200_set_error("qmm (static scratch): residual epilogue without a residual"); return B200_ERR_INVALID_ARGUMENT; }
-  if (epilogue == B200_EPI_GELU) { b200_set_error("qmm (static scratch): no GELU epilogue"); return B200_ERR_UNSUPPORTED; }
+  if (elementwise(epilogue)) { b200_set_error("qmm (static scratch): no GELU or squared ReLU epilogue"); return B200_ERR_UNSUPPORTED; }
   if (epilogue == B200_EPI_SWIGLU && (w->n % 2) != 0) { b200_set_error("qmm (static scratch): SwiGLU needs an even N"); return B200_ERR_INVALID_ARGUMENT; }
   int dev = 0;
   B200_CUDA_TRY(cudaGetDevice(&dev));

@@ -16,6 +16,9 @@ struct b200_qweight {
   alignas(64) unsigned char mx_map[128] = {};  // CUtensorMap over d_mx_codes
 };
 
+// The SwiGLU epilogue: g = min(gate, limit), u = clamp(up, -limit, limit) (limit 0: as they are), g sigmoid(alpha g) (u + shift).
+struct SwigluShape { float limit = 0.f, alpha = 1.f, shift = 0.f; };
+
 struct QmmArgs {
   const unsigned char* blocks;  // first block of the weight (expert) this launch/tile uses
   const __nv_bfloat16* x;       // [rows, k]
@@ -37,7 +40,7 @@ struct QmmArgs {
   int epilogue;
   int x_slab;                   // small-batch kernel: activations staged in shared memory
   int x_row0;                   // first row of this launch within the tensor map
-  float swiglu_limit;
+  float swiglu_limit, swiglu_alpha = 1.f, swiglu_shift = 0.f;
   // split-K finish fused with the RMSNorm that reads the result next (residual epilogue only)
   const __nv_bfloat16* norm_w;  // non-null: the finish pass also writes norm_out = rmsnorm(y) * norm_w
   __nv_bfloat16* norm_out;
@@ -67,7 +70,12 @@ b200_status b200_qmm_grouped(const b200_qweight* w, const void* d_x, int32_t row
                              const float* d_row_scales, float swiglu_limit, const int4* d_items, const int* d_n_items,
                              int32_t max_items, int32_t tile_rows, void* stream);
 // Dense bf16 weights, rows of the output y_stride elements apart.
-b200_status b200_qmm_to(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t y_stride, int32_t epilogue, void* stream);
+b200_status b200_qmm_to(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t y_stride, int32_t epilogue, void* stream,
+                        const SwigluShape& shape = SwigluShape{});
+// b200_qmm_deferred with partial sums that outlive the next matmuls, up to the next call of this kind.
+b200_status b200_qmm_deferred_aside(const b200_qweight* w, const void* d_x, int32_t rows, void* d_y, int32_t defer, void* stream, b200_qmm_partials* out);
+b200_status b200_qmm_f32_shaped(const b200_qweight* w, const float* d_x, int32_t rows, float* d_y, int32_t y_stride, int32_t n_valid,
+                                int32_t epilogue, void* stream, const SwigluShape& shape);
 // Block-diagonal matmul: the n_experts matrices [n, k] of w are the blocks (one per attention head, say).
 // y[r][e * y_group + i] = sum_j w_e[i][j] x[r][e * x_group + j]; rows of x are x_stride apart, those of y y_stride.  bf16, f32 accumulation;
 // y_f32: the sums are written as they are, d_y holds floats.

@@ -273,14 +273,14 @@ class LayeredKVCache(PagedKVCache):
 
     def window_attention(self, layer: int, q: torch.Tensor, row_seq: torch.Tensor, row_ctx: torch.Tensor, scale: float, window: int = 0,
                          slopes: Optional[np.ndarray] = None, sinks: Optional[np.ndarray] = None,
-                         mma: bool = True) -> torch.Tensor:
-        """b200_decoder_attention on q as qkv() returns it -> [T, heads, value width]."""
+                         mma: bool = True, distances: Optional[np.ndarray] = None) -> torch.Tensor:
+        """b200_decoder_attention on q as qkv() returns it -> [T, heads, value width].  distances: [heads, n], a bias by distance."""
         t, hq, _ = q.shape
         vd = self.layers[layer][2]
         log2 = lambda a: None if a is None else torch.tensor(np.asarray(a, np.float64) * 1.4426950408889634, dtype=torch.float32, device=q.device)
-        sl, sk = log2(slopes), log2(sinks)
+        sl, sk, ds = log2(slopes), log2(sinks), log2(distances)
         out = torch.empty((t, hq, vd), dtype=q.dtype, device=q.device)
-        _lib.check(lib.b200_decoder_attention(self._h, layer, _ptr(q), hq, window, scale, _ptr(sl), _ptr(sk), _ptr(row_seq), _ptr(row_ctx), t,
+        _lib.check(lib.b200_decoder_attention(self._h, layer, _ptr(q), hq, window, scale, _ptr(sl), _ptr(sk), _ptr(ds), 0 if distances is None else ds.shape[1], _ptr(row_seq), _ptr(row_ctx), t,
                                               int(mma), _ptr(out), hq * vd, _stream()))
         word = self.error_word()
         if word:
@@ -583,13 +583,16 @@ class LlamaModel(Model):
 DT_BF16, DT_F32 = 0, 1
 DEC_QKV_BIAS, DEC_QK_NORM, DEC_DISTANCE_BIAS, DEC_SINK, DEC_POST_NORM, DEC_PARALLEL = 1, 2, 4, 8, 16, 32
 DEC_SINK_ONE, DEC_QK_NORM_WEIGHT, DEC_ROT_HALVES, DEC_FF_GELU, DEC_ROUTER = 64, 128, 256, 512, 1024
+DEC_RESULT_GATE, DEC_QK_NORM_ROW, DEC_FF_RELU2, DEC_ROUTER_PLAIN, DEC_SHARED_GATE = 2048, 4096, 8192, 16384, 32768
 DEC_SCALAR_NORM, DEC_DEPTH_AVERAGE, DEC_SUM_NORM, DEC_NORM_OFFSET = 1, 2, 4, 8  # of the whole stack
-MIX_ATTENTION, MIX_LATENT, MIX_GLA, MIX_LRU = 0, 1, 2, 3
+MIX_ATTENTION, MIX_LATENT, MIX_GLA, MIX_LRU, MIX_DELTA = 0, 1, 2, 3, 4
 DEC_TENSORS = ("q", "k", "v", "o", "gate", "up", "down", "head", "loop_in", "embed", "q_bias", "k_bias", "v_bias", "sink", "norm1", "norm2",
                "postnorm1", "postnorm2", "final_norm", "dkv", "dkv_norm", "uk", "uv", "out_gate", "a1", "a2", "a2_bias", "head_norm",
                "expert_gate", "expert_up", "expert_down", "depth", "dq", "dq_norm", "q_norm", "k_norm", "q_conv", "k_conv", "v_conv",
                "mem_q", "mem_k", "mem_v", "mem_g", "mem_o", "mem_i", "mem_f", "mem_i_bias", "mem_f_bias", "mem_norm", "lru_y", "lru_y_bias", "lru_x",
-               "lru_x_bias", "lru_conv", "lru_conv_bias", "lru_r", "lru_r_bias", "lru_i", "lru_i_bias", "lru_lambda", "router")
+               "lru_x_bias", "lru_conv", "lru_conv_bias", "lru_r", "lru_r_bias", "lru_i", "lru_i_bias", "lru_lambda", "router",
+               "positions", "distances", "in_conv1", "in_conv2", "result_gate1", "result_gate2", "result_gate1_bias", "result_gate2_bias", "beta",
+               "decay", "a_log", "dt_bias", "shared_gate")
 
 
 class DecoderModel(Model):
@@ -598,10 +601,10 @@ class DecoderModel(Model):
 
     def __init__(self, hidden: int, vocab: int, layers: Sequence[dict], norm_eps: float, embed_scale: float = 1.0, loop=None,
                  dtype: int = DT_BF16, max_rows: int = 2048, max_reqs: int = 64, max_seqs: int = 64, logit_scale: float = 1.0, flags: int = 0,
-                 residual_scale: float = 1.0):
+                 residual_scale: float = 1.0, max_positions: int = 0):
         start, stop, times = loop if loop else (0, 0, 0)
         self.cfg = _lib.DecoderConfig(len(layers), hidden, vocab, start, stop, times, dtype, max_rows, max_reqs, max_seqs, norm_eps,
-                                      embed_scale, logit_scale, flags, residual_scale)
+                                      embed_scale, logit_scale, flags, residual_scale, max_positions)
         arr = (_lib.DecoderLayer * max(len(layers), 1))(*[_lib.DecoderLayer(**l) for l in layers])
         h = C.c_void_p()
         _lib.check(lib.b200_decoder_create(C.byref(self.cfg), arr, C.byref(h)))

@@ -76,4 +76,4 @@ def load_model(folder: str, dtype: str = "bfloat16", limits: Optional[Limits] = 
     return _REGISTRY[name](config, folder, dtype, limits or Limits())
 
 
-from . import dovorax, llama, sotavik, tafuvik  # noqa: E402,F401  (each registers itself)
+from . import dovorax, llama, lorulix, sotavik, tafuvik  # noqa: E402,F401  (each registers itself)

@@ -430,7 +430,7 @@ b200_status b200_qweight_random(int32_t mode, int32_t n_experts, int32_t n, int3
 b200_status b200_qweight_export(const b200_qweight* w, int32_t expert, void* h_packed, void* h_scales,
                                 void* h_biases);
 void b200_qweight_destroy(b200_qweight* w);
-enum { B200_EPI_NONE = 0, B200_EPI_RESIDUAL = 1, B200_EPI_SWIGLU = 2, B200_EPI_GELU = 3 };
+enum { B200_EPI_NONE = 0, B200_EPI_RESIDUAL = 1, B200_EPI_SWIGLU = 2, B200_EPI_GELU = 3, B200_EPI_RELU2 = 4 };
 enum { B200_QMM_AUTO = 0, B200_QMM_SIMT = 1, B200_QMM_TCGEN05 = 2, B200_QMM_MMA = 3, B200_QMM_TCGEN05_X2 = 4,
        B200_QMM_TCGEN05_TMEM_A = 5, B200_QMM_MXFP4_BLOCK_SCALED = 6, B200_QMM_MMA_I8 = 7 };
 /* Tuning hook (no reference counterpart): 1 sends the grouped (MoE) matmuls through the kernel that
@@ -567,6 +567,7 @@ b200_model* b200_llama_model(b200_llama* m);
 typedef struct b200_model_info {
   int32_t vocab, max_rows, max_reqs, max_seqs;
   int32_t logits_f32;  /* element type of the logits on the device: 1 = f32, 0 = bf16 */
+  int32_t max_positions; /* tokens a sequence may have; 0 = as many as its page table holds */
 } b200_model_info;
 void b200_model_get_info(const b200_model* m, b200_model_info* out);
 /* The b200_llama_* calls of the same names, for any model. */
@@ -591,16 +592,21 @@ b200_status b200_model_logits(b200_model* m, int32_t first, int32_t n, float* h_
 /* ---- configurable decoder stack ------------------------------------------------------------------- */
 /* A decoder-only stack whose layers are described one by one (no reference counterpart; the reference has one file per
  * model family).  Every mechanism is a parameter of its layer, and a layer that does not set it does not have it:
- *   x = embed[token] * embed_scale, kept in f32 between the layers;
+ *   x = embed[token] * embed_scale (+ a learned vector per position, max_positions), kept in f32 between the layers;
  *   x += postnorm1(mixer(norm1(x))); x += postnorm2(ff(h)), h = norm2(x);
  *   with B200_DEC_PARALLEL instead x += mixer(h) + ff(h), h = norm1(x);
  *   with B200_DEC_SUM_NORM instead x = norm1(residual_scale * x + mixer(x)), x = norm2(residual_scale * x + ff(x));
  *   mixer: one of B200_MIX_*; beside attention a matrix memory may run on the same h (mem_heads > 0), the two are added with the factors
  *   mix_scale and mem_scale;
- *   ff(h) = W_down(silu(W_gate h) * W_up h) of width ffn (B200_DEC_FF_GELU: W_down gelu(W_up h)), plus the same of each of the top_k
- *   experts of a token: 1 / top_k each for those the token's id has in the layer's table, or (B200_DEC_ROUTER) the best of softmax(W_router h)
- *   with their scores, which are divided by their sum; only the keep_groups of n_groups groups of neighbouring experts with the largest
- *   best score take part;
+ *   ff(h) = W_down(silu(W_gate h) * W_up h) of width ffn (B200_DEC_FF_GELU: W_down gelu(W_up h); B200_DEC_FF_RELU2: W_down relu(W_up h)^2),
+ *   plus the same of each of the top_k experts of a token: 1 / top_k each for those the token's id has in the layer's table, or
+ *   (B200_DEC_ROUTER) the best of softmax(W_router h) with their scores, which are divided by their sum (B200_DEC_ROUTER_PLAIN: multiplied by
+ *   router_scale instead); only the keep_groups of n_groups groups of neighbouring experts with the largest best score take part;
+ *   B200_DEC_SHARED_GATE multiplies the feed-forward beside the experts by sigmoid(W_sg h), one number per token;
+ *   the gated form with a limit or other constants: g = min(W_gate h, ff_limit), u = clamp(W_up h, -ff_limit, ff_limit),
+ *   W_down(g sigmoid(ff_alpha g) (u + ff_shift)), ff_limit 0 = none, ff_alpha 0 = 1;
+ *   with input_taps a sublayer reads h + conv(h) instead of h, conv causal per channel; with B200_DEC_RESULT_GATE its result is multiplied by
+ *   sigmoid(W h + b) of the h in front of that convolution, ahead of the post-norm;
  *   with B200_DEC_DEPTH_AVERAGE what follows layer i is sum_j depth[j] X_j over the embedding output X_0 and the results X_1 ..
  *   X_(i+1) of the layers so far;
  *   layers loop_start .. loop_stop-1 run loop_times times with the same weights, every pass with cache layers of its own,
@@ -621,6 +627,11 @@ enum {
   B200_DEC_ROT_HALVES = 256,   /* rotated pairs are (i, i + rot_dim / 2) instead of (2i, 2i + 1) */
   B200_DEC_FF_GELU = 512,      /* feed-forward and experts: exact GELU, no gate */
   B200_DEC_ROUTER = 1024,      /* experts by a router instead of a table */
+  B200_DEC_RESULT_GATE = 2048, /* a gate per element on each sublayer's result */
+  B200_DEC_QK_NORM_ROW = 4096, /* RMSNorm of q, and of k, over all heads at once, with a weight per row of the projection */
+  B200_DEC_FF_RELU2 = 8192,    /* feed-forward and experts: square of relu, no gate */
+  B200_DEC_ROUTER_PLAIN = 16384, /* the chosen experts' scores as they are, times router_scale */
+  B200_DEC_SHARED_GATE = 32768, /* the feed-forward beside the experts is weighted by a gate per token */
   /* of the whole stack (b200_decoder_config.flags) */
   B200_DEC_SCALAR_NORM = 1,    /* a norm's weight is one number for all coordinates */
   B200_DEC_DEPTH_AVERAGE = 2,  /* weighted average over depth after every layer */
@@ -628,7 +639,10 @@ enum {
   B200_DEC_NORM_OFFSET = 8     /* norm weights are stored around zero: 1 + w */
 };
 /* B200_MIX_ATTENTION: softmax attention, keys and values per kv head.  With conv_taps a causal convolution per channel stands directly
- *   behind the q, k and v projections; with rot_dim the first rot_dim dimensions of q and k are rotated, behind their norm.
+ *   behind the q, k and v projections; with rot_dim the first rot_dim dimensions of q and k are rotated, behind their norm.  With q_temp_every
+ *   q is multiplied by 1 + q_temp_coef ln(floor((p + 1) / q_temp_every) + 1) at position p.  With rel_buckets the score gets table[bucket(i - j)]
+ *   of its head: bucket(n) = n below half = rel_buckets / 2, min(rel_buckets - 1, half + floor(ln(n / half) / ln(rel_reach / half) *
+ *   (rel_buckets - half))) from there on.  With kv_source = 1 + j the layer has queries only and reads the pages of layer j < this one.
  * B200_MIX_LATENT: keys and values of all heads come from one latent of kv_rank numbers per token, c = norm(W_dkv h); per head
  *   the key is W_uk c (key_dim wide) beside rot_dim rotated numbers shared by all heads, the value W_uv c (value_dim).  Cached are
  *   c and the rotated part.  Rotation: pairs (2i, 2i+1), angle position * rot_base^(-2i / rot_dim).  With q_rank the queries come from a
@@ -637,12 +651,15 @@ enum {
  *   sigmoid(W_a2 W_a1 h + b)^(1 / decay_tau) with decay_rank rows in W_a1; rms_norm(o) * w * silu(W_g h).
  * B200_MIX_LRU: n_heads blocks of value_dim channels; y = gelu_tanh(W_y h + b), u = conv(W_x h + b) + b of conv_taps taps; per block
  *   r = sigmoid(R u + b), i = sigmoid(I u + b); a = exp(-lru_decay r softplus(lam)), S <- a S + sqrt(1 - a^2) i u; the output is S * y.
+ * B200_MIX_DELTA: q and k of n_kv_heads heads, v of n_heads; each passes a causal convolution of conv_taps taps and silu, q and k of a head
+ *   become unit vectors (1e-6 inside the root), q also times key_dim^(-1/2); per head g = exp(-exp(A_log) softplus(W_a h + dt_bias)), beta =
+ *   sigmoid(W_b h); S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q; rms_norm(o) * w * silu(W_g h).
  * Matrix memory (mem_heads of mem_key_dim x mem_value_dim): log gates i = cap tanh((W_i h + b) / cap) and f = log sigmoid(cap tanh((W_f h + b)
  *   / cap)), cap = mem_gate_cap; m' = max(f + m, i); S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone; o = S^T q / (max(|n . q|,
  *   e^-m') + 1e-6), q scaled by mem_key_dim^(-1/2); rms_norm(o) * w * sigmoid(W_g h).
  * YaRN (yarn_factor > 0): with dim(t) = rot_dim ln(yarn_original / (2 pi t)) / (2 ln rot_base), the frequencies of the pairs from
  *   dim(yarn_fast) to dim(yarn_slow) go over to 1 / yarn_factor of themselves; cosine and sine are multiplied by 0.1 ln yarn_factor + 1. */
-enum { B200_MIX_ATTENTION = 0, B200_MIX_LATENT = 1, B200_MIX_GLA = 2, B200_MIX_LRU = 3 };
+enum { B200_MIX_ATTENTION = 0, B200_MIX_LATENT = 1, B200_MIX_GLA = 2, B200_MIX_LRU = 3, B200_MIX_DELTA = 4 };
 typedef struct b200_decoder_layer {
   int32_t n_heads, n_kv_heads, key_dim, value_dim;
   int32_t window; /* position i sees j with 0 <= i - j < window; 0 = the whole context */
@@ -656,12 +673,18 @@ typedef struct b200_decoder_layer {
   float decay_tau;
   int32_t n_experts, top_k, expert_ffn;     /* experts by token id (b200_decoder_set_table) or router; n_experts 0 = none */
   int32_t n_groups, keep_groups;            /* of a router's experts; 0 = one group */
-  int32_t q_rank, kv_source;                /* latent attention; 0 = none, its own */
+  int32_t q_rank, kv_source;                /* latent attention; kv_source also of attention; 0 = none, its own */
   double yarn_factor, yarn_original, yarn_fast, yarn_slow;
-  int32_t conv_taps;                        /* attention (0 = none) and LRU */
+  int32_t conv_taps;                        /* attention (0 = none), LRU and the delta rule */
   float lru_decay;
   int32_t mem_heads, mem_key_dim, mem_value_dim; /* matrix memory beside attention; 0 = none */
   float mem_gate_cap, mix_scale, mem_scale;
+  int32_t input_taps;                       /* convolution of what each sublayer reads; 0 = none */
+  int32_t rel_buckets, rel_reach;           /* attention: table of biases by distance; 0 = none */
+  float q_temp_coef;
+  int32_t q_temp_every;                     /* attention; 0 = none */
+  float router_scale;                       /* B200_DEC_ROUTER_PLAIN */
+  float ff_limit, ff_alpha, ff_shift;       /* of the gated feed-forward */
 } b200_decoder_layer;
 typedef struct b200_decoder_config {
   int32_t n_layers, hidden, vocab;
@@ -671,6 +694,7 @@ typedef struct b200_decoder_config {
   float norm_eps, embed_scale, logit_scale;
   int32_t flags; /* those of the whole stack */
   float residual_scale; /* B200_DEC_SUM_NORM */
+  int32_t max_positions; /* rows of the table of position vectors; 0 = none */
 } b200_decoder_config;
 typedef struct b200_decoder b200_decoder;
 enum { B200_DEC_W_Q = 0, B200_DEC_W_K = 1, B200_DEC_W_V = 2, B200_DEC_W_O = 3, B200_DEC_W_GATE = 4, B200_DEC_W_UP = 5,
@@ -688,11 +712,15 @@ enum { B200_DEC_W_Q = 0, B200_DEC_W_K = 1, B200_DEC_W_V = 2, B200_DEC_W_O = 3, B
        B200_DEC_W_MEM_I = 44, B200_DEC_W_MEM_F = 45, B200_DEC_B_MEM_I = 46, B200_DEC_B_MEM_F = 47, B200_DEC_MEM_NORM = 48 /* [heads * value] */,
        B200_DEC_W_LRU_Y = 49, B200_DEC_B_LRU_Y = 50, B200_DEC_W_LRU_X = 51, B200_DEC_B_LRU_X = 52, B200_DEC_LRU_CONV = 53 /* [channels, taps] */,
        B200_DEC_B_LRU_CONV = 54, B200_DEC_W_LRU_R = 55 /* [blocks, out, in] */, B200_DEC_B_LRU_R = 56, B200_DEC_W_LRU_I = 57,
-       B200_DEC_B_LRU_I = 58, B200_DEC_LRU_LAMBDA = 59, B200_DEC_W_ROUTER = 60 };
+       B200_DEC_B_LRU_I = 58, B200_DEC_LRU_LAMBDA = 59, B200_DEC_W_ROUTER = 60,
+       B200_DEC_W_POS = 61 /* [max_positions, hidden] */, B200_DEC_W_REL = 62 /* [rel_buckets, heads] */, B200_DEC_IN_CONV1 = 63 /* [hidden, taps] */,
+       B200_DEC_IN_CONV2 = 64, B200_DEC_W_RESULT_GATE1 = 65, B200_DEC_W_RESULT_GATE2 = 66, B200_DEC_B_RESULT_GATE1 = 67,
+       B200_DEC_B_RESULT_GATE2 = 68, B200_DEC_W_BETA = 69, B200_DEC_W_DECAY = 70, B200_DEC_A_LOG = 71, B200_DEC_DT_BIAS = 72,
+       B200_DEC_W_SHARED_GATE = 73, B200_DEC_LAST_TENSOR = 73 };
 b200_status b200_decoder_create(const b200_decoder_config* cfg, const b200_decoder_layer* layers, b200_decoder** out);
 void b200_decoder_destroy(b200_decoder* m);
 /* One tensor, bf16 on the host, matrices [out, in]; n_elems is checked against the shape the configuration gives.
- * `layer` is ignored for embed, head, loop_in and final_norm. */
+ * `layer` is ignored for embed, positions, head, loop_in and final_norm. */
 b200_status b200_decoder_set_tensor(b200_decoder* m, int32_t layer, int32_t which, const void* h_bf16, uint64_t n_elems);
 /* Experts of every token id in one layer: [vocab][top_k] expert numbers, all different within a row. */
 b200_status b200_decoder_set_table(b200_decoder* m, int32_t layer, const int32_t* h_table, uint64_t n_elems);
@@ -717,13 +745,14 @@ b200_model* b200_decoder_model(b200_decoder* m);
  * be null), divides every q and k head by its root mean square when qk_norm, writes q as [q heads][key_dim rounded up to 16]
  * and k, v into their pages.
  * attention (also of layers with values_in_keys): d_q as written by qkv; out rows [q heads x value_dim], out_stride apart.  d_slopes_log2 / d_sinks_log2: f32 per
- * query head, multiplied by log2(e), may be null.  `mma` as in b200_decoder_set_attn_mma. */
+ * query head, multiplied by log2(e), may be null.  d_dist_log2 (may be null): [q heads][dist_len], a bias by distance, likewise, its last
+ * number for all distances beyond.  `mma` as in b200_decoder_set_attn_mma. */
 b200_status b200_decoder_qkv(b200_kv* kv, int32_t layer, const void* d_qkv, int32_t stride, const float* d_bias, int32_t n_q_heads,
                              int32_t qk_norm, float eps, void* d_q, const int32_t* d_positions, const int32_t* d_row_seq,
                              int32_t total_rows, void* stream);
 b200_status b200_decoder_attention(b200_kv* kv, int32_t layer, const void* d_q, int32_t n_q_heads, int32_t window, float scale,
-                                   const float* d_slopes_log2, const float* d_sinks_log2, const int32_t* d_row_seq,
-                                   const int32_t* d_row_ctx, int32_t total_rows, int32_t mma, void* d_out,
+                                   const float* d_slopes_log2, const float* d_sinks_log2, const float* d_dist_log2, int32_t dist_len,
+                                   const int32_t* d_row_seq, const int32_t* d_row_ctx, int32_t total_rows, int32_t mma, void* d_out,
                                    int32_t out_stride, void* stream);
 /* Gated linear attention of one layer over the rows of a batch, for hosts that drive the layers themselves: d_rows [rows][q | k | v |
  * g | a1] in the pool's element type, `stride` elements apart; d_cu [n_req + 1] the requests' first rows, d_row_seq and d_positions
@@ -736,6 +765,17 @@ b200_status b200_decoder_gla(b200_kv* kv, int32_t layer, const b200_gla_shape* s
                              const float* d_a2_bias, const float* d_norm, const int32_t* d_cu, const int32_t* d_row_seq,
                              const int32_t* d_positions, int32_t n_req, int32_t total_rows, int32_t chunked, void* d_out, int32_t out_stride,
                              void* stream);
+
+/* The gated delta rule of one layer, likewise: d_rows [rows][q | k | v | g | b | a], d_conv the taps of the convolutions in bf16, [taps][q | k | v
+ * channels], the current token's last; d_rate (exp(A_log)) and d_dt_bias f32 per head. */
+typedef struct b200_delta_shape {
+  int32_t heads, kv_heads, key_dim, value_dim, taps;
+  float eps;
+} b200_delta_shape;
+b200_status b200_decoder_delta(b200_kv* kv, int32_t layer, const b200_delta_shape* shape, const void* d_rows, int32_t stride, const void* d_conv,
+                               const float* d_rate, const float* d_dt_bias, const float* d_norm, const int32_t* d_cu, const int32_t* d_row_to_req,
+                               const int32_t* d_row_seq, const int32_t* d_positions, int32_t n_req, int32_t total_rows, int32_t chunked,
+                               void* d_out, int32_t out_stride, void* stream);
 
 /* ---- engine step: schedule -> pack -> model step -> postprocess ------------------------------- */
 /* The Engine_Step loop of src/scheduler.zig:7-10 wired to a forward pass (the reference leaves
