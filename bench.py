@@ -19,6 +19,8 @@ Prints ONE JSON line (rank 0).  Workloads (synthetic seeded inputs):
   sotavik : the Sotavik stack (latent attention, gated linear attention, experts by token id; one GPU) the same way.
   dovorax : the Dovorax stack (gated linear recurrence, windowed latent attention, attention beside a matrix memory, routed experts; one
             GPU) the same way, beside the Sotavik stacks too.
+  lorulix : the Lorulix stack (gated delta rule, attention with distance tables, gated sublayers, routed experts; one GPU) the same way,
+            beside the gated linear attention of Sotavik and the routed experts of Dovorax.
 Multi-GPU (torchrun, one rank per GPU): independent replicas of the workload, no collective in the
 step (requests never interact); `value` = tokens of all ranks / max-over-ranks time.
 """
@@ -1427,6 +1429,132 @@ def run_dovorax(args, local: int):
         "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind}, "sizes": out, "e2e": None, "gpu_launches": launches, "clocks": clocks}))
 
 
+# Dense feed-forwards as wide as LLaMA's; the experts of the mixed stacks are Dovorax's.  The delta rule's state is as large as GLA's.
+LORULIX_SIZES = {
+    "d4096": dict(delta=dict(heads=32, kv_heads=16, dim=128, vdim=128), taps=4, input_taps=4, buckets=32, reach=128),
+    "d2048": dict(delta=dict(heads=16, kv_heads=8, dim=128, vdim=128), taps=4, input_taps=4, buckets=32, reach=128),
+}
+# D delta rule, A attention, S attention on the pages of the last A; lower case: with experts
+LORULIX_STACKS = {"lorulix_attention": "AAAAAA", "lorulix_shared": "ASASAS", "lorulix_delta": "DDDDDD", "lorulix_experts": "dadsda"}
+
+
+def _lorulix_layers(z, order):
+    from dmlx_b200 import device as dev
+
+    t, out = z["delta"], []
+    for i, c in enumerate(order):
+        flags = dev.DEC_POST_NORM | dev.DEC_RESULT_GATE
+        if c.islower():
+            flags |= dev.DEC_ROUTER | dev.DEC_ROUTER_PLAIN | dev.DEC_FF_RELU2 | dev.DEC_SHARED_GATE
+            ff = dict(ffn=z["shared"], n_experts=z["experts"], top_k=z["top"], expert_ffn=z["expert_ffn"], router_scale=2.0)
+        else:
+            ff = dict(ffn=z["ffn"], ff_limit=7.0, ff_alpha=1.702, ff_shift=1.0)
+        if c in "Dd":
+            mix = dict(mixer=dev.MIX_DELTA, n_heads=t["heads"], n_kv_heads=t["kv_heads"], key_dim=t["dim"], value_dim=t["vdim"], conv_taps=z["taps"])
+        else:
+            source = 1 + max(j for j in range(i) if order[j] in "Aa") if c in "Ss" else 0
+            mix = dict(mixer=dev.MIX_ATTENTION, n_heads=z["heads"], n_kv_heads=z["kv_heads"], key_dim=z["head_dim"], value_dim=z["head_dim"],
+                       scale=z["head_dim"] ** -0.5, kv_source=source, rel_buckets=z["buckets"], rel_reach=z["reach"], q_temp_coef=0.1, q_temp_every=1024)
+            flags |= dev.DEC_QK_NORM_ROW
+        out.append(dict(mix, flags=flags, input_taps=z["input_taps"], **ff))
+    return out
+
+
+def _lorulix_work(z, order, ctxs, prefill):
+    """As _sotavik_work."""
+    d, t = z["hidden"], z["delta"]
+    rows, seqs, n = DECODER_ROWS if prefill else len(ctxs), len(ctxs), len(order)
+    if prefill:
+        per = rows // len(ctxs)
+        keys, read = len(ctxs) * per * (per + 1) / 2.0, float(rows)
+    else:
+        keys = read = float(ctxs.sum())
+    na, ns, nd, nx = (sum(c in k for c in order) for k in ("Aa", "Ss", "Dd", "ads"))
+    hq, hk = z["heads"] * z["head_dim"], z["kv_heads"] * z["head_dim"]
+    qk, v = t["kv_heads"] * t["dim"], t["heads"] * t["vdim"]
+    state = 4.0 if prefill else 8.0  # a prompt only writes its state
+    attn_b = (na + ns) * (read * 2 * hk + rows * 2 * hq) * 2.0 + nd * (seqs * t["heads"] * t["dim"] * t["vdim"] * state + rows * (2 * qk + 3 * v) * 2.0)
+    attn_f = (na + ns) * 4.0 * keys * hq + nd * 6.0 * rows * t["heads"] * t["dim"] * t["vdim"]
+    append = (na * (hq + 2 * hk) + ns * hq + nd * (2 * qk + v)) * rows * 4.0 + nd * seqs * (z["taps"] - 1) * (2 * qk + v) * state
+    dense = (na + ns) * 2 * d * hq + na * 2 * d * hk + nd * d * (2 * qk + 3 * v + 2 * t["heads"]) + n * 2 * d * d
+    dense += (n - nx) * 3 * d * z["ffn"] + nx * (2 * d * z["shared"] + d * (z["experts"] + 1))
+    head = d * DECODER_VOCAB
+    mat_b = 2.0 * (dense + nx * min(z["experts"], rows * z["top"]) * 2 * d * z["expert_ffn"] + head)
+    mat_f = 2.0 * rows * (dense + nx * z["top"] * 2 * d * z["expert_ffn"]) + 2.0 * seqs * head
+    return {"attention": (attn_b, attn_f), "matmul": (mat_b, mat_f), "rope_append": (append, 0.0),
+            "other": (rows * d * (n * 36.0 + nx * 6.0 * z["top"]), 0.0)}
+
+
+def run_lorulix(args, local: int):
+    import torch
+
+    from dmlx_b200 import device as dev
+
+    torch.cuda.set_device(local)
+    torch.cuda.set_stream(torch.cuda.Stream())
+    hbm, kind = load_peaks()
+    p = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    tflops = float(json.load(open(p))["bf16_tflops"]) if os.path.exists(p) else 1590.0
+    K, W = min(args.steps, 50), max(args.warmup, 3)
+    ctxs = np.clip(np.rint(np.random.default_rng(77).lognormal(np.log(2600), 0.6, DECODER_REQS)), 256, 12000).astype(np.int64)
+    pages = int((-(-(ctxs + 4 * (K + W) + 64) // PAGE)).sum()) + 16
+    most = int(-(-(ctxs.max() + 4 * (K + W) + 64) // PAGE))
+    sampler = ClockSampler(local)
+    sampler.start()
+    out, launches = {}, 0
+    for name, extra in LORULIX_SIZES.items():
+        base = SOTAVIK_SIZES[name]
+        z = dict(base, **extra)
+
+        def stack(layers, **kw):
+            model = dev.DecoderModel(z["hidden"], DECODER_VOCAB, layers, 1e-5, 1.0, None, dev.DT_BF16, DECODER_ROWS, DECODER_REQS, DECODER_REQS, **kw)
+            model.random_init(3)
+            return model, model.make_cache(pages, DECODER_REQS, most)
+
+        def llama():
+            model = dev.LlamaModel(6, z["hidden"], z["heads"], z["kv_heads"], z["head_dim"], z["ffn"], DECODER_VOCAB, DECODER_ROWS, DECODER_REQS, DECODER_REQS)
+            model.random_init(dev.Q_BF16, 3)
+            return model, dev.PagedKVCache(6, z["kv_heads"], z["head_dim"], pages, DECODER_REQS, most, z["heads"], max_rows=DECODER_ROWS)
+
+        dov = dict(base, **DOVORAX_SIZES[name])
+        cases = {
+            "llama": (llama, lambda at, pre: _decoder_work(dict(z, llama_dim=z["head_dim"]), 6, 0, at, pre, True)),
+            "sotavik_gla": (lambda: stack(_sotavik_layers(base, "GGGGGG"), flags=dev.DEC_SCALAR_NORM | dev.DEC_DEPTH_AVERAGE),
+                            lambda at, pre: _sotavik_work(base, "GGGGGG", at, pre)),
+            "dovorax_mixed": (lambda: stack(_dovorax_layers(dov, DOVORAX_STACKS["dovorax_mixed"]), flags=dev.DEC_SUM_NORM, residual_scale=2.0),
+                              lambda at, pre: _dovorax_work(dov, DOVORAX_STACKS["dovorax_mixed"], at, pre)),
+        }
+        for which, order in LORULIX_STACKS.items():
+            cases[which] = (lambda order=order: stack(_lorulix_layers(z, order), flags=dev.DEC_NORM_OFFSET, max_positions=16384),
+                            lambda at, pre, order=order: _lorulix_work(z, order, at, pre))
+        for which, (make, work_of) in cases.items():
+            if args.stacks and which not in args.stacks.split(","):
+                continue
+            model, kv = make()
+            for mode in ("decode", "prefill"):
+                ms, prof, n = _time_stack(model, kv, ctxs, pages, mode, K, W)
+                launches += n
+                entry = {"ms_per_step": ms, "tokens_per_s": (DECODER_REQS if mode == "decode" else DECODER_ROWS) / ms * 1e3}
+                for cat, (nbytes, flops) in work_of(ctxs if mode == "decode" else ctxs[:2], mode == "prefill").items():
+                    ideal = max(nbytes / hbm / 1e6, flops / tflops / 1e9)
+                    entry[cat] = {"ms": prof[cat], "of_roofline": ideal / prof[cat] if prof[cat] > 0 else None}
+                out.setdefault(name, {}).setdefault(mode, {})[which] = entry
+            kv.close()
+            model.close()
+    clocks = sampler.stop()
+    head = out["d4096"]["decode"].get("lorulix_experts", {"tokens_per_s": None, "ms_per_step": None})
+    print(json.dumps({
+        "metric": "decode tokens/sec (Lorulix stack, 6 layers)", "value": head["tokens_per_s"], "unit": "decode tokens/s", "n_gpus": 1,
+        "steps": K, "warmup": W, "ms_per_step": head["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "lorulix", "stacks": LORULIX_STACKS, "shapes": LORULIX_SIZES, "feed_forward": SOTAVIK_SIZES, "vocab": DECODER_VOCAB,
+                   "decode_requests": DECODER_REQS, "cached_tokens": int(ctxs.sum()), "prefill": f"2 prompts of {DECODER_ROWS // 2} tokens in one step",
+                   "parallelism": "dp1", "l2": "weights and caches larger than L2"},
+        "note": "of_roofline: the larger of bytes / measured copy bandwidth and FLOPs / measured burst bf16 rate, over the category's time "
+                "(eager launches with an event pair each, so small kernels carry their launch gap)",
+        "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind}, "sizes": out, "e2e": None, "gpu_launches": launches, "clocks": clocks}))
+
+
 def run_tafuvik(args, local: int):
     import torch
 
@@ -1507,6 +1635,7 @@ def main():
     ap.add_argument("--path", type=int, default=0, help="qmm_* only: kernel path (0 = automatic)")
     ap.add_argument("--seqs", type=int, default=64, help="sequences per GPU (64 = the configuration; fewer for profiling)")
     ap.add_argument("--mx-persistent", type=int, default=-1, help="block-scaled MXFP4 path: 1 persistent CTAs over work items, 0 one CTA per item (default: library choice)")
+    ap.add_argument("--stacks", default="", help="lorulix only: the stacks to time, separated by commas (default: all)")
     ap.add_argument("--no-arrivals", action="store_true", help="llama8b_int4 only: skip the arrival-process scenarios")
     ap.add_argument("--attn-pages-per-chunk", type=int, default=0,
                     help="tuning: pages per split-K chunk of the decode attention (0 = the library's default)")
@@ -1540,6 +1669,10 @@ def main():
     if args.mx_persistent >= 0:
         from dmlx_b200 import _lib
         _lib.lib.b200_set_qmm_mx_persistent(args.mx_persistent)
+    if args.workload == "lorulix":
+        if rank == 0:
+            run_lorulix(args, local)
+        return
     if args.workload == "dovorax":
         if rank == 0:
             run_dovorax(args, local)

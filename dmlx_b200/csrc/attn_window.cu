@@ -256,9 +256,9 @@ __device__ __forceinline__ void split_bf16(float p0, float p1, uint32_t& hi, uin
 }
 
 // KB, VB: 64-column boxes a key / value row may take (1, 2 or 4); the steps beyond the layer's own widths are skipped.
-// A block is as many independent warps as its shared memory and registers feed.
+// A block is as many independent warps as its shared memory and registers feed.  TABLE: the layer has a bias by distance.
 constexpr int most_warps(int kb, int vb) { return kb + vb == 2 ? 12 : (kb + vb == 3 ? 9 : 8); }
-template <int KB, int VB>
+template <int KB, int VB, bool TABLE>
 __global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
     window_attn_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap, WinArgs a) {
   constexpr int KS = KB * 4;  // 16-column steps of Q K^T
@@ -340,10 +340,8 @@ __global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
     const int lo_last = first_key(it.ctx0 + it.n_rows - 1, a.window);  // the latest window start of the group
     const bool any_b = it.n_rows * hb > 8;                            // rows 8..15 of the tile carry something
     const float slA = a.slopes ? a.slopes[qhA] : 0.f, slB = a.slopes ? a.slopes[qhB] : 0.f;
-    const float *tabA = a.dist + (size_t)qhA * a.dist_len, *tabB = a.dist + (size_t)qhB * a.dist_len;  // (used with a table only)
-    const float farA = a.dist ? tabA[a.dist_len - 1] : 0.f, farB = a.dist ? tabB[a.dist_len - 1] : 0.f;
     // the first key that some row of the group sees at a distance of its own
-    const int near_from = a.dist ? it.ctx0 - (a.dist_len - 1) : 0x7fffffff;
+    const int near_from = TABLE ? it.ctx0 - (a.dist_len - 1) : 0;
     uint32_t qa0[KS], qa1[KS], qa2[KS], qa3[KS];
     {
       const uint32_t* qA = reinterpret_cast<const uint32_t*>(a.q + (size_t)(it.first_row + (onA ? tokA : 0)) * a.q_stride + (size_t)qhA * a.L.kd);
@@ -387,19 +385,21 @@ __global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
       const int tok0 = pg * 32;
       uint32_t ph[2][4], pl[2][4];
       // a page every row of the group sees whole needs no masks; beyond the reach of a distance table all keys have the same bias
-      const int kind = tok0 + 31 >= near_from ? 2 : (tok0 + 32 > it.ctx0 || tok0 < lo_last ? 1 : 0);
-      auto row_softmax = [&](auto kind_tag, auto half_tag, float& m, float& l, int ctx, int lo, float slope, float far, const float* tab) -> float {
-        constexpr bool EDGE = decltype(kind_tag)::value > 0, TABLE = decltype(kind_tag)::value == 2;
+      const int kind = TABLE && tok0 + 31 >= near_from ? 2 : (tok0 + 32 > it.ctx0 || tok0 < lo_last ? 1 : 0);
+      auto row_softmax = [&](auto kind_tag, auto half_tag, float& m, float& l, int ctx, int lo, float slope, int qh) -> float {
+        constexpr bool EDGE = decltype(kind_tag)::value > 0, NEAR = decltype(kind_tag)::value == 2;
         constexpr int E0 = decltype(half_tag)::value;  // 0: row g, 1: row g + 8
         float mx = kNone;
-        const float b0 = fmaf(slope, (float)(tok0 + 2 * t - (ctx - 1)), far);  // (exact integers) the bias of the lane's first key
+        const float* tab = TABLE ? a.dist + (size_t)qh * a.dist_len : nullptr;
+        float b0 = slope * (float)(tok0 + 2 * t - (ctx - 1));  // exact integers; the bias of the lane's first key
+        if constexpr (TABLE && !NEAR) b0 += tab[a.dist_len - 1];
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) {
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             const int tok = tok0 + nt * 8 + 2 * t + e;
             float v;
-            if constexpr (TABLE) v = fmaf(sc[nt][2 * E0 + e], a.scale_log2, tab[min(max(ctx - 1 - tok, 0), a.dist_len - 1)]);
+            if constexpr (NEAR) v = fmaf(sc[nt][2 * E0 + e], a.scale_log2, tab[min(max(ctx - 1 - tok, 0), a.dist_len - 1)]);
             else v = sc[nt][2 * E0 + e] * a.scale_log2 + fmaf(slope, (float)(nt * 8 + e), b0);
             if (EDGE) v = tok < ctx && tok >= lo ? v : kNone;
             sc[nt][2 * E0 + e] = v;
@@ -430,14 +430,16 @@ __global__ void __launch_bounds__(most_warps(KB, VB) * 32, 1)
       using T0 = std::integral_constant<int, 0>;
       using T1 = std::integral_constant<int, 1>;
       using T2 = std::integral_constant<int, 2>;
-      auto softmax = [&](auto half_tag, float& m, float& l, int ctx, int lo, float slope, float far, const float* tab) -> float {
-        if (kind == 0) return row_softmax(T0{}, half_tag, m, l, ctx, lo, slope, far, tab);
-        return kind == 1 ? row_softmax(T1{}, half_tag, m, l, ctx, lo, slope, far, tab) : row_softmax(T2{}, half_tag, m, l, ctx, lo, slope, far, tab);
+      auto softmax = [&](auto half_tag, float& m, float& l, int ctx, int lo, float slope, int qh) -> float {
+        if constexpr (TABLE) {
+          if (kind == 2) return row_softmax(T2{}, half_tag, m, l, ctx, lo, slope, qh);
+        }
+        return kind == 0 ? row_softmax(T0{}, half_tag, m, l, ctx, lo, slope, qh) : row_softmax(T1{}, half_tag, m, l, ctx, lo, slope, qh);
       };
-      const float corrA = softmax(T0{}, mA, lA, ctxA, loA, slA, farA, tabA);
+      const float corrA = softmax(T0{}, mA, lA, ctxA, loA, slA, qhA);
       float corrB = 1.f;
       if (any_b) {
-        corrB = softmax(T1{}, mB, lB, ctxB, loB, slB, farB, tabB);
+        corrB = softmax(T1{}, mB, lB, ctxB, loB, slB, qhB);
       } else {
 #pragma unroll
         for (int kt = 0; kt < 2; ++kt) { ph[kt][1] = ph[kt][3] = pl[kt][1] = pl[kt][3] = 0u; }
@@ -670,7 +672,7 @@ Shape shape_of(int boxes) {
   }
 }
 
-template <int KB, int VB>
+template <int KB, int VB, bool TABLE>
 b200_status launch_mma(const b200_kv* kv, WinArgs& a, int layer, cudaStream_t s) {
   const int boxes = (a.L.kd + 63) / 64 + (a.L.vd + 63) / 64;
   const Shape sh = shape_of(boxes);
@@ -679,19 +681,19 @@ b200_status launch_mma(const b200_kv* kv, WinArgs& a, int layer, cudaStream_t s)
   const size_t smem = (size_t)sh.warps * sh.stages * (boxes * 4096 + sizeof(uint64_t)) + 1024;
   static bool configured = false;
   if (!configured) {
-    B200_CUDA_TRY((cudaFuncSetAttribute(window_attn_mma_kernel<KB, VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024)));
+    B200_CUDA_TRY((cudaFuncSetAttribute(window_attn_mma_kernel<KB, VB, TABLE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024)));
     configured = true;
   }
-  window_attn_mma_kernel<KB, VB><<<g_sms, sh.warps * 32, smem, s>>>(kv->lay_kmap[layer], kv->lay_vmap[layer], a);
+  window_attn_mma_kernel<KB, VB, TABLE><<<g_sms, sh.warps * 32, smem, s>>>(kv->lay_kmap[layer], kv->lay_vmap[layer], a);
   B200_LAUNCH_CHECK();
   return B200_OK;
 }
 
 template <int KB>
 b200_status launch_mma_v(const b200_kv* kv, WinArgs& a, int layer, cudaStream_t s) {
-  if (a.L.vd <= 64) return launch_mma<KB, 1>(kv, a, layer, s);
-  if (a.L.vd <= 128) return launch_mma<KB, 2>(kv, a, layer, s);
-  return launch_mma<KB, 4>(kv, a, layer, s);
+  if (a.L.vd <= 64) return a.dist ? launch_mma<KB, 1, true>(kv, a, layer, s) : launch_mma<KB, 1, false>(kv, a, layer, s);
+  if (a.L.vd <= 128) return a.dist ? launch_mma<KB, 2, true>(kv, a, layer, s) : launch_mma<KB, 2, false>(kv, a, layer, s);
+  return a.dist ? launch_mma<KB, 4, true>(kv, a, layer, s) : launch_mma<KB, 4, false>(kv, a, layer, s);
 }
 
 }  // namespace

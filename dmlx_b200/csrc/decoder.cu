@@ -115,9 +115,11 @@ __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-
 
 // One CTA per row: sublayer output -> residual stream -> what the next matmul reads.  NQ > 0: a thread keeps its NQ
 // groups of VEC columns in registers and asks for the residual before the first reduction; NQ = 0: any width, the row
-// waits in shared memory.
-template <typename T, int VEC, int NQ>
-__global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
+// waits in shared memory.  FEW: steps of few rows, bound by the latency of their loads, so more of them are in flight; only they may do the
+// convolution of the coming sublayer.
+constexpr int kStateAhead = 3;  // entries of its state that are asked for before the row's sums are known
+template <typename T, int VEC, int NQ, bool FEW>
+__global__ void __launch_bounds__(512, FEW ? 1 : 2) decoder_rows_kernel(RowArgs a) {
   extern __shared__ float row_sh[];
   __shared__ float part[32];
   const int row = blockIdx.x, n = a.hidden / VEC;
@@ -144,6 +146,23 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
     if constexpr (NQ > 0) keep[k] = v;
     else store_vec<VEC>(row_sh + i * VEC, v);
   };
+  auto value = [&](const MatSrc& src, int c) {
+    if constexpr (FEW) return mat_value_ahead<T, VEC, 8>(src, row, c);
+    else return mat_value<T, VEC>(src, row, c);
+  };
+  const int slot = FEW && a.hc ? a.row_seq[row] : 0;
+  const bool conv = FEW && a.hc && slot >= 0 && slot < a.max_seqs && a.pool_state[ST_ERR] == 0;
+  const int back = conv ? min(a.conv.taps - 1, a.pos[row]) : 0;
+  float* state = conv ? a.conv.state + (size_t)slot * a.conv.slot_elems : nullptr;
+  constexpr int kAhead = FEW && NQ > 0 ? kStateAhead : 0;
+  Vec<VEC> old[kAhead > 0 ? NQ * kAhead : 1];
+  if (kAhead > 0 && conv) {
+    each([&](int i, int k) {
+#pragma unroll
+      for (int d = 0; d < kAhead; ++d)
+        if (d + 1 < a.conv.taps) old[k * kAhead + d] = load_vec<VEC>(state + (size_t)d * a.conv.channels + i * VEC);
+    });
+  }
   float ss = 0.f;
   if (a.tokens) {
     const uint32_t tok = min(a.tokens[row], (uint32_t)(a.vocab - 1));
@@ -172,7 +191,7 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
       if constexpr (NQ > 0) { if (!a.replace) res[k] = load_vec<VEC>(xr + i * VEC); }
       Vec<VEC> v;
       if (a.src.ws || a.src.y) {
-        v = mat_value<T, VEC>(a.src, row, i * VEC);
+        v = value(a.src, i * VEC);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) v.v[j] *= src_scale;
       } else {
@@ -186,7 +205,7 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
         for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(w, e.v[j], v.v[j]);
       }
       if (a.gate_bias) {
-        const Vec<VEC> z = mat_value<T, VEC>(a.gate, row, i * VEC), b = load_vec<VEC>(a.gate_bias + i * VEC);
+        const Vec<VEC> z = value(a.gate, i * VEC), b = load_vec<VEC>(a.gate_bias + i * VEC);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) v.v[j] *= sigmoid(z.v[j] + b.v[j]);
       }
@@ -236,9 +255,6 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
   if (a.norm_w) {
     const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)a.hidden + a.eps);
     T* hr = (T*)a.h + (size_t)row * a.h_stride;
-    const int slot = a.hc ? a.row_seq[row] : 0;
-    const bool conv = a.hc && slot >= 0 && slot < a.max_seqs && a.pool_state[ST_ERR] == 0;
-    const int back = conv ? min(a.conv.taps - 1, a.pos[row]) : 0;
     each([&](int i, int k) {
       Vec<VEC> v = get(i, k);
       const Vec<VEC> w = load_vec<VEC>(a.norm_w + i * VEC);
@@ -246,21 +262,24 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
       for (int j = 0; j < VEC; ++j) v.v[j] *= r * w.v[j];
       store_vec<VEC>(hr + i * VEC, v);
       if (conv) {
-        float* state = a.conv.state + (size_t)slot * a.conv.slot_elems + i * VEC;
+        float* entry = state + i * VEC;
         Vec<VEC> own, acc{};
 #pragma unroll
         for (int j = 0; j < VEC; ++j) own.v[j] = as_stored<T>(v.v[j]);
         Vec<VEC> carried = own;  // entries move up by one
-        for (int d = 1; d < a.conv.taps; ++d) {
-          const Vec<VEC> u = load_vec<VEC>(state + (size_t)(d - 1) * a.conv.channels);
-          store_vec<VEC>(state + (size_t)(d - 1) * a.conv.channels, carried);
+        auto step = [&](int d, const Vec<VEC>& u) {
+          store_vec<VEC>(entry + (size_t)(d - 1) * a.conv.channels, carried);
           carried = u;
           if (d <= back) {
             const Vec<VEC> tap = load_vec<VEC>(a.conv.w + (size_t)(a.conv.taps - 1 - d) * a.conv.channels + i * VEC);
 #pragma unroll
             for (int j = 0; j < VEC; ++j) acc.v[j] = fmaf(tap.v[j], u.v[j], acc.v[j]);
           }
-        }
+        };
+#pragma unroll
+        for (int d = 1; d <= kAhead; ++d)
+          if (d < a.conv.taps) step(d, old[k * kAhead + d - 1]);
+        for (int d = kAhead + 1; d < a.conv.taps; ++d) step(d, load_vec<VEC>(entry + (size_t)(d - 1) * a.conv.channels));
         const Vec<VEC> tap = load_vec<VEC>(a.conv.w + (size_t)(a.conv.taps - 1) * a.conv.channels + i * VEC);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) acc.v[j] = own.v[j] + fmaf(tap.v[j], own.v[j], acc.v[j]);
@@ -278,10 +297,10 @@ __global__ void __launch_bounds__(512) decoder_rows_kernel(RowArgs a) {
   }
 }
 
-template <typename T>
+template <typename T, bool FEW>
 void (*rows_kernel(int vec, int nq))(RowArgs) {
-  if (vec == 1) return decoder_rows_kernel<T, 1, 0>;
-  return nq <= 1 ? decoder_rows_kernel<T, 4, 1> : (nq <= 2 ? decoder_rows_kernel<T, 4, 2> : (nq <= 4 ? decoder_rows_kernel<T, 4, 4> : decoder_rows_kernel<T, 4, 0>));
+  if (vec == 1) return decoder_rows_kernel<T, 1, 0, FEW>;
+  return nq <= 1 ? decoder_rows_kernel<T, 4, 1, FEW> : (nq <= 2 ? decoder_rows_kernel<T, 4, 2, FEW> : (nq <= 4 ? decoder_rows_kernel<T, 4, 4, FEW> : decoder_rows_kernel<T, 4, 0, FEW>));
 }
 
 // hc = h + conv(h) over the rows of a step, portions of any length.  One thread per (R rows, VEC channels).
@@ -645,8 +664,8 @@ __global__ void __launch_bounds__(256, KEEP == 1 ? 3 : 2) decoder_qkv_conv4_kern
 
 // The same where a row's norms span all heads of q and of k: one CTA per row, which waits in shared memory for its sums of squares.  The queries are
 // also scaled by a temperature that grows with the position; without keys there are queries only.
-template <typename T, int VEC>
-__global__ void __launch_bounds__(256) decoder_qkv_row_kernel(QkvArgs a) {
+template <typename T, int VEC, int THREADS>
+__global__ void __launch_bounds__(THREADS, 1024 / THREADS) decoder_qkv_row_kernel(QkvArgs a) {
   extern __shared__ __align__(16) float row_sh[];
   __shared__ float part[32];
   const int row = blockIdx.x, H = a.keys ? a.L.heads : 0, dim = a.L.key_dim, nq = a.hq * dim, nqk = nq + H * dim, all = nqk + H * a.L.value_dim;
@@ -659,8 +678,10 @@ __global__ void __launch_bounds__(256) decoder_qkv_row_kernel(QkvArgs a) {
   }
   const size_t k_head = (size_t)kPageTokens * a.L.kd, v_head = (size_t)kPageTokens * a.L.vd;
   float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x * VEC; c < all; c += 256 * VEC) {
-    Vec<VEC> v = mat_value<T, VEC>(a.src, row, c);
+  for (int c = threadIdx.x * VEC; c < all; c += THREADS * VEC) {
+    Vec<VEC> v;
+    if constexpr (THREADS > 256) v = mat_value_ahead<T, VEC, 8>(a.src, row, c);
+    else v = mat_value<T, VEC>(a.src, row, c);
     if (a.bias) {
 #pragma unroll
       for (int e = 0; e < VEC; ++e) v.v[e] += a.bias[c + e];
@@ -684,7 +705,7 @@ __global__ void __launch_bounds__(256) decoder_qkv_row_kernel(QkvArgs a) {
     if (a.keys) rk = 1.0f / sqrtf(block_sum(sk, part) / (float)(nqk - nq) + a.eps);
   }
   if (a.temp_every > 0) rq *= 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1));
-  for (int c = threadIdx.x * VEC; c < nqk; c += 256 * VEC) {  // (a thread reads what it wrote)
+  for (int c = threadIdx.x * VEC; c < nqk; c += THREADS * VEC) {  // (a thread reads what it wrote)
     const bool is_q = c < nq;
     const int k = is_q ? c : c - nq, head = k / dim;
     Vec<VEC> v = load_vec<VEC>(row_sh + c);
@@ -693,11 +714,11 @@ __global__ void __launch_bounds__(256) decoder_qkv_row_kernel(QkvArgs a) {
     for (int e = 0; e < VEC; ++e) v.v[e] *= (is_q ? rq : rk) * (w ? w[k + e] : 1.f);
     store_vec<VEC>((is_q ? q + (size_t)head * a.L.kd : kr + head * k_head) + (k - head * dim), v);
   }
-  for (int i = threadIdx.x; i < (a.hq + H) * (a.L.kd - dim); i += 256) {  // padding behind a head
+  for (int i = threadIdx.x; i < (a.hq + H) * (a.L.kd - dim); i += THREADS) {  // padding behind a head
     const int u = i / (a.L.kd - dim), c = dim + i - u * (a.L.kd - dim);
     st((u < a.hq ? q + (size_t)u * a.L.kd : kr + (u - a.hq) * k_head) + c, 0.f);
   }
-  for (int i = threadIdx.x; i < H * (a.L.vd - a.L.value_dim); i += 256) {
+  for (int i = threadIdx.x; i < H * (a.L.vd - a.L.value_dim); i += THREADS) {
     const int u = i / (a.L.vd - a.L.value_dim);
     st(vr + u * v_head + a.L.value_dim + i - u * (a.L.vd - a.L.value_dim), 0.f);
   }
@@ -708,10 +729,13 @@ b200_status launch_qkv(const QkvArgs& a, int rows, cudaStream_t s) {
     const bool vec = a.L.key_dim % 4 == 0 && a.L.value_dim % 4 == 0 && (a.src.ws || a.src.y_stride % 4 == 0);
     const size_t smem = sizeof(float) * (a.hq + (a.keys ? a.L.heads : 0)) * (size_t)a.L.key_dim;
     if (smem > 200 * 1024) { b200_set_error("decoder: %d heads of %d are too wide for a row's norm", a.hq, a.L.key_dim); return B200_ERR_UNSUPPORTED; }
-    auto* kernel = a.d.elem_bytes == 4 ? (vec ? decoder_qkv_row_kernel<float, 4> : decoder_qkv_row_kernel<float, 1>)
-                                       : (vec ? decoder_qkv_row_kernel<__nv_bfloat16, 4> : decoder_qkv_row_kernel<__nv_bfloat16, 1>);
+    const bool few = rows < 512;  // (one block per SM at most: more threads per row)
+    auto* kernel = a.d.elem_bytes == 4 ? (vec ? decoder_qkv_row_kernel<float, 4, 256> : decoder_qkv_row_kernel<float, 1, 256>)
+                                       : (vec ? decoder_qkv_row_kernel<__nv_bfloat16, 4, 256> : decoder_qkv_row_kernel<__nv_bfloat16, 1, 256>);
+    if (few) kernel = a.d.elem_bytes == 4 ? (vec ? decoder_qkv_row_kernel<float, 4, 1024> : decoder_qkv_row_kernel<float, 1, 1024>)
+                                          : (vec ? decoder_qkv_row_kernel<__nv_bfloat16, 4, 1024> : decoder_qkv_row_kernel<__nv_bfloat16, 1, 1024>);
     if (smem > 48 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    kernel<<<rows, 256, smem, s>>>(a);
+    kernel<<<rows, few ? 1024 : 256, smem, s>>>(a);
     B200_LAUNCH_CHECK();
     return B200_OK;
   }
@@ -1025,9 +1049,11 @@ b200_status b200_decoder::rows_step(RowArgs a, int rows, int next, cudaStream_t 
     }
   }
   const int vec = cfg.hidden % 4 == 0 ? 4 : 1;
-  const int threads = std::min(rows >= 512 ? 256 : 512, (cfg.hidden / vec + 31) / 32 * 32), nq = (cfg.hidden / vec + threads - 1) / threads;
+  const bool few = rows < 512 || a.hc;
+  const int threads = std::min(few ? 512 : 256, (cfg.hidden / vec + 31) / 32 * 32), nq = (cfg.hidden / vec + threads - 1) / threads;
   const size_t smem = vec == 4 && nq <= 4 ? 0 : sizeof(float) * cfg.hidden;
-  auto* kernel = f32() ? rows_kernel<float>(vec, nq) : rows_kernel<__nv_bfloat16>(vec, nq);
+  auto* kernel = f32() ? (few ? rows_kernel<float, true>(vec, nq) : rows_kernel<float, false>(vec, nq))
+                       : (few ? rows_kernel<__nv_bfloat16, true>(vec, nq) : rows_kernel<__nv_bfloat16, false>(vec, nq));
   if (smem > 47 * 1024) B200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   kernel<<<rows, threads, smem, s>>>(a);
   B200_LAUNCH_CHECK();

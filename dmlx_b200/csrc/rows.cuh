@@ -74,6 +74,29 @@ __device__ __forceinline__ Vec<VEC> mat_value(const MatSrc& s, int row, int c) {
   return acc;
 }
 
+// The same with the loads of up to AHEAD splits in flight, for kernels of few rows.
+template <typename T, int VEC, int AHEAD>
+__device__ __forceinline__ Vec<VEC> mat_value_ahead(const MatSrc& s, int row, int c) {
+  if (!s.ws) return load_vec<VEC>((const T*)s.y + (size_t)row * s.y_stride + c);
+  const int nt = c >> 7, r = c & 127, tt = row / s.tn, tr = row - tt * s.tn;
+  const float* p = s.ws + (((size_t)(nt * s.tts + tt) * s.splits) * s.tn + tr) * 128 + r;
+  Vec<VEC> acc{};
+  for (int i = 0; i < s.splits; i += AHEAD) {
+    Vec<VEC> b[AHEAD];
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      b[u] = Vec<VEC>{};
+      if (i + u < s.splits) b[u] = load_vec<VEC>(p + (size_t)(i + u) * s.tn * 128);
+    }
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc.v[e] += b[u].v[e];
+    }
+  }
+  return acc;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

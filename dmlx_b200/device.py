@@ -271,6 +271,19 @@ class LayeredKVCache(PagedKVCache):
                                         _ptr(row_seq), _ptr(positions), cu.shape[0] - 1, rows.shape[0], int(chunked), _ptr(out), heads * vd, _stream()))
         return out
 
+    def delta(self, layer: int, rows: torch.Tensor, conv: torch.Tensor, rate: torch.Tensor, dt_bias: torch.Tensor, norm: torch.Tensor, kv_heads: int,
+              key_dim: int, eps: float, cu: torch.Tensor, row_to_req: torch.Tensor, row_seq: torch.Tensor, positions: torch.Tensor,
+              chunked: bool = True) -> torch.Tensor:
+        """b200_decoder_delta on projection rows [q | k | v | g | b | a], conv bf16 [taps, channels] -> [T, heads, value width]; the
+        layer's state moves on."""
+        heads, vd = rate.shape[0], norm.shape[0]
+        shape = _lib.DeltaShape(heads, kv_heads, key_dim, vd, conv.shape[0], eps)
+        out = torch.zeros((rows.shape[0], heads, vd), dtype=rows.dtype, device=rows.device)
+        _lib.check(lib.b200_decoder_delta(self._h, layer, C.byref(shape), _ptr(rows), rows.shape[1], _ptr(conv), _ptr(rate), _ptr(dt_bias), _ptr(norm),
+                                          _ptr(cu), _ptr(row_to_req), _ptr(row_seq), _ptr(positions), cu.shape[0] - 1, rows.shape[0], int(chunked),
+                                          _ptr(out), heads * vd, _stream()))
+        return out
+
     def window_attention(self, layer: int, q: torch.Tensor, row_seq: torch.Tensor, row_ctx: torch.Tensor, scale: float, window: int = 0,
                          slopes: Optional[np.ndarray] = None, sinks: Optional[np.ndarray] = None,
                          mma: bool = True, distances: Optional[np.ndarray] = None) -> torch.Tensor:
@@ -280,8 +293,8 @@ class LayeredKVCache(PagedKVCache):
         log2 = lambda a: None if a is None else torch.tensor(np.asarray(a, np.float64) * 1.4426950408889634, dtype=torch.float32, device=q.device)
         sl, sk, ds = log2(slopes), log2(sinks), log2(distances)
         out = torch.empty((t, hq, vd), dtype=q.dtype, device=q.device)
-        _lib.check(lib.b200_decoder_attention(self._h, layer, _ptr(q), hq, window, scale, _ptr(sl), _ptr(sk), _ptr(ds), 0 if distances is None else ds.shape[1], _ptr(row_seq), _ptr(row_ctx), t,
-                                              int(mma), _ptr(out), hq * vd, _stream()))
+        _lib.check(lib.b200_decoder_attention(self._h, layer, _ptr(q), hq, window, scale, _ptr(sl), _ptr(sk), _ptr(ds),
+                                              0 if distances is None else ds.shape[1], _ptr(row_seq), _ptr(row_ctx), t, int(mma), _ptr(out), hq * vd, _stream()))
         word = self.error_word()
         if word:
             raise _lib.B200Error(word)

@@ -32,7 +32,7 @@ def softplus(z):
 def causal_convolution(u, taps):
     """u [T, C], taps [C, K], the last one the current token's; zeros before the first token."""
     y = np.zeros_like(u)
-    for back in range(taps.shape[1]):
+    for back in range(min(taps.shape[1], u.shape[0])):
         y[back:] += taps[:, -1 - back] * u[:u.shape[0] - back]
     return y
 
@@ -196,3 +196,95 @@ def forward(tokens, w, cfg, rnd=ident, want_layers=False, without=NOTHING):
     one = 0.0 if "unit_offset" in without else 1.0
     logits = linear(rnd(root_mean_square_norm(x, eps, one + w["final.norm"])), w["head"])
     return (logits, np.stack(trail)) if want_layers else logits
+
+
+# ---- test models -------------------------------------------------------------------------------------
+def tensor_shapes(cfg, buckets=8):
+    """name -> shape of every tensor a configuration asks for; `buckets`: rows of the distance tables, one number or a function of the layer."""
+    d = cfg["width"]
+    out = {"embed": (cfg["vocab"], d), "pos": (cfg["max_positions"], d), "final.norm": (d,), "head": (cfg["vocab"], d)}
+    for i, spec in enumerate(cfg["layers"]):
+        n, m, mlp = f"l{i}", spec["mixer"], spec.get("mlp")
+        mix = f"{n}.mix."
+        for s in "12" if mlp else "1":
+            out[f"{n}.norm{s}"], out[f"{n}.norm{s}b"], out[f"{n}.canon{s}"] = (d,), (d,), (d, cfg["canon"]["taps"])
+            out[f"{n}.rg{s}"], out[f"{n}.rg{s}.b"] = (d, d), (d,)
+        if spec["type"] == "delta":
+            for p, rows in (("q", m["kv_heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["heads"] * m["vdim"])):
+                out[mix + p], out[f"{mix}{p}.conv"] = (rows, d), (rows, m["conv"])
+            out[mix + "b"], out[mix + "a"], out[mix + "g"] = (m["heads"], d), (m["heads"], d), (m["heads"] * m["vdim"], d)
+            out[mix + "A_log"], out[mix + "dt_bias"], out[mix + "norm"] = (m["heads"],), (m["heads"],), (m["vdim"],)
+        else:
+            h, g = m["heads"], m["kv_heads"]
+            out[mix + "q"], out[mix + "q.norm"] = (h * m["dim"], d), (h * m["dim"],)
+            out[mix + "rel"] = (buckets(i) if callable(buckets) else buckets, h)
+            if m.get("kv_from") is None:
+                out[mix + "k"], out[mix + "k.norm"], out[mix + "v"] = (g * m["dim"], d), (g * m["dim"],), (g * m["vdim"], d)
+        out[mix + "o"] = (d, m["heads"] * m["vdim"])
+        if not mlp:
+            continue
+        if mlp["kind"] == "dense":
+            out[f"{n}.mlp.gate"], out[f"{n}.mlp.up"], out[f"{n}.mlp.down"] = (mlp["ff"], d), (mlp["ff"], d), (d, mlp["ff"])
+            continue
+        parts = [(f"e{e}.", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])]
+        out[f"{n}.mlp.router"] = (mlp["router"]["experts"], d)
+        if mlp.get("shared"):
+            parts.append(("shared.", mlp["shared"]["ff"]))
+            out[f"{n}.mlp.shared.sg"] = (1, d)
+        for p, f in parts:
+            out[f"{n}.mlp.{p}up"], out[f"{n}.mlp.{p}down"] = (f, d), (d, f)
+    return out
+
+
+def random_weights(cfg, seed, decisive=True, buckets=8):
+    """Weights as bf16 can hold them: projections keep unit variance, norm weights scatter, states remember some tens of tokens.
+
+    `decisive`: every token id ranks the experts of a layer by levels in a few coordinates of its own, which the sublayers hardly touch,
+    so that 16-bit rounding cannot swap two experts."""
+    from .ref_math import bf16_round
+
+    rng = np.random.default_rng(seed)
+    most = max([s["mlp"]["router"]["experts"] for s in cfg["layers"] if s.get("mlp") and s["mlp"]["kind"] == "moe"], default=0) if decisive else 0
+    out = {}
+    for name, shape in tensor_shapes(cfg, buckets).items():
+        part = name.split(".")[-1]
+        if part in ("norm1", "norm2", "norm1b", "norm2b") or name == "final.norm":
+            a = 0.3 * rng.normal(size=shape)
+            a[:most] = 0.0
+        elif part == "norm":
+            a = 1.0 + 0.3 * rng.normal(size=shape)
+        elif part in ("canon1", "canon2"):
+            a = 0.5 * rng.normal(size=shape)
+            a[:most] = 0.0
+        elif name.endswith(("rg1.b", "rg2.b")):
+            a = rng.normal(size=shape)
+        elif part == "A_log":
+            a = -1.5 + rng.normal(size=shape)
+        elif part == "dt_bias":
+            a = -1.0 + rng.normal(size=shape)
+        elif part == "rel":
+            a = 1.5 * rng.normal(size=shape)
+        elif part == "pos":
+            a = 0.7 * rng.normal(size=shape)
+            a[:, :most] = 0.0
+        elif part == "embed":
+            a = rng.normal(size=shape)
+            if most:
+                a[:, :most] = np.stack([rng.permutation(np.linspace(-1.8, 1.8, most)) for _ in range(shape[0])])
+        elif part == "router" and most:
+            a = np.zeros(shape)
+            a[np.arange(shape[0]), rng.permutation(most)[:shape[0]]] = 1.5
+        elif part in ("a", "b", "sg"):
+            a = 2.0 * rng.normal(size=shape) / np.sqrt(shape[1])
+        else:
+            a = rng.normal(size=shape) / np.sqrt(shape[-1])
+            if part in ("o", "down") and most:
+                a[:most] *= 0.03
+        out[name] = bf16_round(np.asarray(a, np.float32)).astype(np.float64)
+    return out
+
+
+def write_model(folder, cfg, weights):
+    from .ref_sotavik import write_model as write
+
+    write(folder, cfg, weights)
