@@ -111,7 +111,6 @@ __device__ __forceinline__ float as_stored(float x) {
   if constexpr (std::is_same_v<T, float>) return x;
   else return __bfloat162float(__float2bfloat16(x));
 }
-__device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // One CTA per row: sublayer output -> residual stream -> what the next matmul reads.  NQ > 0: a thread keeps its NQ
 // groups of VEC columns in registers and asks for the residual before the first reduction; NQ = 0: any width, the row
@@ -122,6 +121,7 @@ template <typename T, int VEC, int NQ, bool FEW>
 __global__ void __launch_bounds__(512, FEW ? 1 : 2) decoder_rows_kernel(RowArgs a) {
   extern __shared__ float row_sh[];
   __shared__ float part[32];
+  __shared__ float4 part4[32];
   const int row = blockIdx.x, n = a.hidden / VEC;
   float* xr = a.x + (size_t)row * a.hidden;
   float* x0r = a.x0 ? a.x0 + (size_t)row * a.hidden : nullptr;
@@ -163,7 +163,10 @@ __global__ void __launch_bounds__(512, FEW ? 1 : 2) decoder_rows_kernel(RowArgs 
         if (d + 1 < a.conv.taps) old[k * kAhead + d] = load_vec<VEC>(state + (size_t)d * a.conv.channels + i * VEC);
     });
   }
-  float ss = 0.f;
+  float ss = 0.f, r_h = 0.f;
+  // With a post-norm both norms come out of one round of sums: |x + r p|^2 = |x|^2 + 2 r x.p + r^2 |p|^2 for p = w y.
+  const bool one_round = NQ > 0 && sizeof(T) == 2 && !a.tokens && a.post_w && a.norm_w && !a.replace && !a.depth && !a.norm_x && !a.plain_h && !a.cat;
+  float4 sums = make_float4(0.f, 0.f, 0.f, 0.f);
   if (a.tokens) {
     const uint32_t tok = min(a.tokens[row], (uint32_t)(a.vocab - 1));
     const __nv_bfloat16* e = a.embed + (size_t)tok * a.hidden;
@@ -187,11 +190,18 @@ __global__ void __launch_bounds__(512, FEW ? 1 : 2) decoder_rows_kernel(RowArgs 
     float ys = 0.f;
     const float src_scale = a.src_scale ? a.src_scale[row] : 1.f;
     Vec<VEC> res[NQ > 0 ? NQ : 1];
+    if (NQ > 0 && !a.replace) each([&](int i, int k) { res[k] = load_vec<VEC>(xr + i * VEC); });
+    // rows that the matmuls wrote themselves are asked for at once
+    constexpr bool kRowsAhead = NQ > 0 && !FEW;
+    Raw<T, VEC> y_raw[kRowsAhead ? NQ : 1], z_raw[kRowsAhead ? NQ : 1];
+    const T* y_row = kRowsAhead && !a.src.ws && a.src.y ? (const T*)a.src.y + (size_t)row * a.src.y_stride : nullptr;
+    const T* z_row = kRowsAhead && !a.gate.ws && a.gate_bias ? (const T*)a.gate.y + (size_t)row * a.gate.y_stride : nullptr;
+    if (y_row) each([&](int i, int k) { y_raw[k] = load_raw<T, VEC>(y_row + i * VEC); });
+    if (z_row) each([&](int i, int k) { z_raw[k] = load_raw<T, VEC>(z_row + i * VEC); });
     each([&](int i, int k) {
-      if constexpr (NQ > 0) { if (!a.replace) res[k] = load_vec<VEC>(xr + i * VEC); }
       Vec<VEC> v;
       if (a.src.ws || a.src.y) {
-        v = value(a.src, i * VEC);
+        v = y_row ? widen<T, VEC>(y_raw[kRowsAhead ? k : 0]) : value(a.src, i * VEC);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) v.v[j] *= src_scale;
       } else {
@@ -205,55 +215,80 @@ __global__ void __launch_bounds__(512, FEW ? 1 : 2) decoder_rows_kernel(RowArgs 
         for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(w, e.v[j], v.v[j]);
       }
       if (a.gate_bias) {
-        const Vec<VEC> z = value(a.gate, i * VEC), b = load_vec<VEC>(a.gate_bias + i * VEC);
+        const Vec<VEC> z = z_row ? widen<T, VEC>(z_raw[kRowsAhead ? k : 0]) : value(a.gate, i * VEC), b = load_vec<VEC>(a.gate_bias + i * VEC);
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) v.v[j] *= sigmoid(z.v[j] + b.v[j]);
+        for (int j = 0; j < VEC; ++j) v.v[j] *= sigmoid_for<T>(z.v[j] + b.v[j]);
       }
+      if (one_round) {
+        const Vec<VEC> w = load_vec<VEC>(a.post_w + i * VEC), x = res[NQ > 0 ? k : 0];
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) ys += v.v[j] * v.v[j];
-      put(i, k, v);
-    });
-    const float r = a.post_w ? 1.0f / sqrtf(block_sum(ys, part) / (float)a.hidden + a.eps) : 1.f;
-    each([&](int i, int k) {
-      Vec<VEC> v = get(i, k);
-      if (a.post_w) {
-        const Vec<VEC> w = load_vec<VEC>(a.post_w + i * VEC);
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) v.v[j] *= r * w.v[j];
-      }
-      if (!a.replace) {
-        Vec<VEC> x;
-        if constexpr (NQ > 0) x = res[k];
-        else x = load_vec<VEC>(xr + i * VEC);
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(a.x_scale, x.v[j], v.v[j]);
-      }
-      if (a.depth) {
-        float* hr = a.hist + (size_t)row * a.hidden + i * VEC;
-        store_vec<VEC>(hr + a.n_hist * a.hist_stride, v);
-        const float own = a.depth[a.n_hist];
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) v.v[j] *= own;
-#pragma unroll 4
-        for (int d = 0; d < a.n_hist; ++d) {
-          const Vec<VEC> x = load_vec<VEC>(hr + d * a.hist_stride);
-          const float w = a.depth[d];
-#pragma unroll
-          for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(w, x.v[j], v.v[j]);
+        for (int j = 0; j < VEC; ++j) {
+          sums.x = fmaf(v.v[j], v.v[j], sums.x);
+          v.v[j] *= w.v[j];
+          sums.y = fmaf(x.v[j], x.v[j], sums.y);
+          sums.z = fmaf(x.v[j], v.v[j], sums.z);
+          sums.w = fmaf(v.v[j], v.v[j], sums.w);
         }
-      }
+      } else {
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) ss += v.v[j] * v.v[j];
+        for (int j = 0; j < VEC; ++j) ys += v.v[j] * v.v[j];
+      }
       put(i, k, v);
-      if (!a.norm_x) store_vec<VEC>(xr + i * VEC, v);
     });
+    if (one_round) {
+      sums = block_sum4(sums, part4);
+      const float r = 1.0f / sqrtf(sums.x / (float)a.hidden + a.eps);
+      r_h = 1.0f / sqrtf(fmaxf(fmaf(r, fmaf(r, sums.w, 2.f * sums.z), sums.y), 0.f) / (float)a.hidden + a.eps);
+      each([&](int i, int k) {
+        Vec<VEC> v = get(i, k), x = res[NQ > 0 ? k : 0];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(r, v.v[j], x.v[j]);
+        put(i, k, v);
+        store_vec<VEC>(xr + i * VEC, v);
+      });
+    } else {
+      const float r = a.post_w ? 1.0f / sqrtf(block_sum(ys, part) / (float)a.hidden + a.eps) : 1.f;
+      each([&](int i, int k) {
+        Vec<VEC> v = get(i, k);
+        if (a.post_w) {
+          const Vec<VEC> w = load_vec<VEC>(a.post_w + i * VEC);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) v.v[j] *= r * w.v[j];
+        }
+        if (!a.replace) {
+          Vec<VEC> x;
+          if constexpr (NQ > 0) x = res[k];
+          else x = load_vec<VEC>(xr + i * VEC);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(a.x_scale, x.v[j], v.v[j]);
+        }
+        if (a.depth) {
+          float* hr = a.hist + (size_t)row * a.hidden + i * VEC;
+          store_vec<VEC>(hr + a.n_hist * a.hist_stride, v);
+          const float own = a.depth[a.n_hist];
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) v.v[j] *= own;
+#pragma unroll 4
+          for (int d = 0; d < a.n_hist; ++d) {
+            const Vec<VEC> x = load_vec<VEC>(hr + d * a.hist_stride);
+            const float w = a.depth[d];
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v.v[j] = fmaf(w, x.v[j], v.v[j]);
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) ss += v.v[j] * v.v[j];
+        put(i, k, v);
+        if (!a.norm_x) store_vec<VEC>(xr + i * VEC, v);
+      });
+    }
   }
   if (a.plain_h) {
     T* hr = (T*)a.h + (size_t)row * a.h_stride;
     each([&](int i, int k) { store_vec<VEC>(hr + i * VEC, get(i, k)); });
   }
   if (a.norm_w) {
-    const float r = 1.0f / sqrtf(block_sum(ss, part) / (float)a.hidden + a.eps);
+    const float r = one_round ? r_h : 1.0f / sqrtf(block_sum(ss, part) / (float)a.hidden + a.eps);
     T* hr = (T*)a.h + (size_t)row * a.h_stride;
     each([&](int i, int k) {
       Vec<VEC> v = get(i, k);

@@ -64,7 +64,7 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(PrepArgs a, int n_rows)
   auto activate = [&](Vec<VEC>& x, float& ss) {
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
-      x.v[e] = silu(x.v[e]);
+      x.v[e] *= sigmoid_for<T>(x.v[e]);
       ss += x.v[e] * x.v[e];
     }
   };
@@ -294,24 +294,25 @@ __global__ void __launch_bounds__(256, 3) delta_chunk_kernel(Delta a) {
     s_beta[lane] = gate.y;
   }
   const bool v4 = dk % 4 == 0;
-  if (v4) {
-    const int groups = dkp / 4;
-    for (int i = tid; i < kC * groups; i += 256) {
-      const int t = i / groups, c = (i - t * groups) * 4;
-      Vec<4> x{}, y{};
-      if (t < n && c < dk) {
-        x = load_vec<4>(a.q(it.x + t, head) + c);
-        y = load_vec<4>(a.k(it.x + t, head) + c);
+#pragma unroll
+  for (int t = warp; t < kC; t += 8) {
+    const float *qg = a.q(it.x + min(t, n - 1), head), *kg = a.k(it.x + min(t, n - 1), head);
+    if (v4) {
+      for (int c = lane * 4; c < dkp; c += 128) {
+        Vec<4> x{}, y{};
+        if (t < n && c < dk) {
+          x = load_vec<4>(qg + c);
+          y = load_vec<4>(kg + c);
+        }
+        store_vec<4>(q + t * ldr + c, x);
+        store_vec<4>(k + t * ldr + c, y);
       }
-      store_vec<4>(q + t * ldr + c, x);
-      store_vec<4>(k + t * ldr + c, y);
-    }
-  } else {
-    for (int i = tid; i < kC * dkp; i += 256) {
-      const int t = i / dkp, c = i - t * dkp;
-      const bool in = t < n && c < dk;
-      q[t * ldr + c] = in ? a.q(it.x + t, head)[c] : 0.f;
-      k[t * ldr + c] = in ? a.k(it.x + t, head)[c] : 0.f;
+    } else {
+      for (int c = lane; c < dkp; c += 32) {
+        const bool in = t < n && c < dk;
+        q[t * ldr + c] = in ? qg[c] : 0.f;
+        k[t * ldr + c] = in ? kg[c] : 0.f;
+      }
     }
   }
   __syncthreads();
@@ -375,18 +376,21 @@ __global__ void __launch_bounds__(256, 3) delta_chunk_kernel(Delta a) {
     }
   } else {
     for (int c = tid - 32; c < dkp; c += 224) reinterpret_cast<float*>(out + off_decay(dkp))[c] = expf(end);
-    for (int i = tid - 32; i < kC * (dkp / 2); i += 224) {
-      const int tok = i / (dkp / 2), c = 2 * (i - tok * (dkp / 2));
+    for (int tok = warp - 1; tok < kC; tok += 7) {
       const float fq = expf(s_L[tok]), fk = expf(end - s_L[tok]);
-      const float2 qt = *reinterpret_cast<const float2*>(&q[tok * ldr + c]), kt = *reinterpret_cast<const float2*>(&k[tok * ldr + c]);
-      uint32_t hi, lo;
-      split_bf16(qt.x * fq, qt.y * fq, hi, lo);
-      unsigned char* at = out + (size_t)tok * qk_row(dkp) + c * 2;
-      *reinterpret_cast<uint32_t*>(at + off_part(dkp, 0)) = hi;
-      *reinterpret_cast<uint32_t*>(at + off_part(dkp, 1)) = lo;
-      split_bf16(kt.x * fk, kt.y * fk, hi, lo);
-      *reinterpret_cast<uint32_t*>(at + off_part(dkp, 2)) = hi;
-      *reinterpret_cast<uint32_t*>(at + off_part(dkp, 3)) = lo;
+      for (int c = lane * 4; c < dkp; c += 128) {
+        const Vec<4> qt = load_vec<4>(&q[tok * ldr + c]), kt = load_vec<4>(&k[tok * ldr + c]);
+        uint2 hi, lo;
+        unsigned char* at = out + (size_t)tok * qk_row(dkp) + c * 2;
+        split_bf16(qt.v[0] * fq, qt.v[1] * fq, hi.x, lo.x);
+        split_bf16(qt.v[2] * fq, qt.v[3] * fq, hi.y, lo.y);
+        *reinterpret_cast<uint2*>(at + off_part(dkp, 0)) = hi;
+        *reinterpret_cast<uint2*>(at + off_part(dkp, 1)) = lo;
+        split_bf16(kt.v[0] * fk, kt.v[1] * fk, hi.x, lo.x);
+        split_bf16(kt.v[2] * fk, kt.v[3] * fk, hi.y, lo.y);
+        *reinterpret_cast<uint2*>(at + off_part(dkp, 2)) = hi;
+        *reinterpret_cast<uint2*>(at + off_part(dkp, 3)) = lo;
+      }
     }
   }
   __syncthreads();

@@ -571,7 +571,7 @@ __global__ void __launch_bounds__(256) gla_out_kernel(Gla a) {
       Vec<VEC> x = load_vec<VEC>(o + c);
       const Vec<VEC> w = load_vec<VEC>(a.norm + c), g = mat_value<T, VEC>(a.src, row, a.col_g + head * a.dv + c);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) x.v[e] *= r * w.v[e] * silu(g.v[e]);
+      for (int e = 0; e < VEC; ++e) x.v[e] *= r * w.v[e] * g.v[e] * sigmoid_for<T>(g.v[e]);
       store_vec<VEC>(dst + c, x);
     }
   }

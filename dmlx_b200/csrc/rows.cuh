@@ -59,6 +59,22 @@ __device__ __forceinline__ void store_vec(__nv_bfloat16* p, const Vec<VEC>& x) {
   }
 }
 
+// A vector as it lies in memory, for loads that are to be in flight while something else happens.
+template <typename T, int VEC>
+struct Raw;
+template <>
+struct Raw<float, 4> { float4 r; };
+template <>
+struct Raw<float, 1> { float r; };
+template <>
+struct Raw<__nv_bfloat16, 4> { uint2 r; };
+template <>
+struct Raw<__nv_bfloat16, 1> { __nv_bfloat16 r; };
+template <typename T, int VEC>
+__device__ __forceinline__ Raw<T, VEC> load_raw(const T* p) { return *reinterpret_cast<const Raw<T, VEC>*>(p); }
+template <typename T, int VEC>
+__device__ __forceinline__ Vec<VEC> widen(const Raw<T, VEC>& raw) { return load_vec<VEC>(reinterpret_cast<const T*>(&raw)); }
+
 // Columns c .. c + VEC - 1 of one row; the splits are summed in split order.
 template <typename T, int VEC>
 __device__ __forceinline__ Vec<VEC> mat_value(const MatSrc& s, int row, int c) {
@@ -97,10 +113,27 @@ __device__ __forceinline__ Vec<VEC> mat_value_ahead(const MatSrc& s, int row, in
   return acc;
 }
 
+// Sigmoid for results that are kept as T: bf16 ones take the hardware's exponential and reciprocal.
+template <typename T>
+__device__ __forceinline__ float sigmoid_for(float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.0f, 1.0f + __expf(-z));
+  else return 1.0f / (1.0f + expf(-z));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
   return v;
+}
+
+// Four sums at once; part holds a number of the block's warps.
+__device__ __forceinline__ float4 block_sum4(float4 v, float4* part) {
+  v = make_float4(warp_sum(v.x), warp_sum(v.y), warp_sum(v.z), warp_sum(v.w));
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
+  __syncthreads();
+  const int lane = threadIdx.x & 31;
+  v = lane < (int)(blockDim.x >> 5) ? part[lane] : make_float4(0.f, 0.f, 0.f, 0.f);  // (every warp for itself)
+  return make_float4(warp_sum(v.x), warp_sum(v.y), warp_sum(v.z), warp_sum(v.w));
 }
 
 __device__ __forceinline__ float block_sum(float v, float* part) {
