@@ -442,26 +442,33 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
           split_bf16(acc[j + 1][0], acc[j + 1][1], sh_[u][2], sl_[u][2]);
           split_bf16(acc[j + 1][2], acc[j + 1][3], sh_[u][3], sl_[u][3]);
         }
+        // two tiles of tokens side by side (and o beside w), so that an MMA does not wait for the one before it
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
-          uint32_t bh[4], bl[4];
-          const uint32_t at = base + (uint32_t)((n * 8 + lr) * qk_row(dkp) + kk * 64 + lm * 16);
-          ldsm4(at + (uint32_t)off_part(dkp, 0), bh);
-          ldsm4(at + (uint32_t)off_part(dkp, 1), bl);
+        for (int n = 0; n < 4; n += 2) {
+          uint32_t qh[2][4], ql[2][4], wh[2][4], wl[2][4];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const uint32_t at = base + (uint32_t)(((n + e) * 8 + lr) * qk_row(dkp) + kk * 64 + lm * 16);
+            ldsm4(at + (uint32_t)off_part(dkp, 0), qh[e]);
+            ldsm4(at + (uint32_t)off_part(dkp, 1), ql[e]);
+            if constexpr (DELTA) {
+              ldsm4(at + (uint32_t)off_w(dkp, 0), wh[e]);
+              ldsm4(at + (uint32_t)off_w(dkp, 1), wl[e]);
+            }
+          }
 #pragma unroll
           for (int u = 0; u < 2; ++u) {
-            mma16816(o[n], sh_[u], bh[2 * u], bh[2 * u + 1]);
-            mma16816(o[n], sh_[u], bl[2 * u], bl[2 * u + 1]);
-            mma16816(o[n], sl_[u], bh[2 * u], bh[2 * u + 1]);
-          }
-          if constexpr (DELTA) {
-            ldsm4(at + (uint32_t)off_w(dkp, 0), bh);
-            ldsm4(at + (uint32_t)off_w(dkp, 1), bl);
 #pragma unroll
-            for (int u = 0; u < 2; ++u) {
-              mma16816(w[n], sh_[u], bh[2 * u], bh[2 * u + 1]);
-              mma16816(w[n], sh_[u], bl[2 * u], bl[2 * u + 1]);
-              mma16816(w[n], sl_[u], bh[2 * u], bh[2 * u + 1]);
+            for (int term = 0; term < 3; ++term) {  // value x value, value x remainder, remainder x value
+#pragma unroll
+              for (int e = 0; e < 2; ++e) {
+                const uint32_t* q = term == 1 ? ql[e] : qh[e];
+                mma16816(o[n + e], term == 2 ? sl_[u] : sh_[u], q[2 * u], q[2 * u + 1]);
+                if constexpr (DELTA) {
+                  const uint32_t* x = term == 1 ? wl[e] : wh[e];
+                  mma16816(w[n + e], term == 2 ? sl_[u] : sh_[u], x[2 * u], x[2 * u + 1]);
+                }
+              }
             }
           }
         }
@@ -501,23 +508,30 @@ __global__ void __launch_bounds__(kScanWarps * 32) gla_scan_kernel(Gla a) {
     // the state moves on: decay its columns, add v^T k
     const float* dec = reinterpret_cast<const float*>(st_ + off_decay(dkp));
 #pragma unroll
-    for (int j = 0; j < NT; j += 2) {
+    for (int j = 0; j < NT; j += 4) {
       if (j < n_t) {
-        const float2 d0 = *reinterpret_cast<const float2*>(dec + j * 8 + 2 * t), d1 = *reinterpret_cast<const float2*>(dec + j * 8 + 8 + 2 * t);
-        acc[j][0] *= d0.x; acc[j][1] *= d0.y; acc[j][2] *= d0.x; acc[j][3] *= d0.y;
-        acc[j + 1][0] *= d1.x; acc[j + 1][1] *= d1.y; acc[j + 1][2] *= d1.x; acc[j + 1][3] *= d1.y;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 d = *reinterpret_cast<const float2*>(dec + (j + e) * 8 + 2 * t);
+          acc[j + e][0] *= d.x; acc[j + e][1] *= d.y; acc[j + e][2] *= d.x; acc[j + e][3] *= d.y;
+        }
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
+          uint32_t b[2][2][4];  // [value, remainder][pair of tiles]: k [tokens][channels], transposed: tokens 0-7 / 8-15 of the step x channels 0-7 / 8-15
 #pragma unroll
-          for (int p = 2; p < 4; ++p) {  // value and remainder
-            uint32_t b[4];  // k [tokens][channels], transposed: tokens 0-7 / 8-15 of the step x channels 0-7 / 8-15
-            const int row = u * 16 + (lm & 1) * 8 + lr, col = j * 8 + (lm >> 1) * 8;
-            ldsm4_trans(base + (uint32_t)(off_part(dkp, p) + row * qk_row(dkp) + col * 2), b);
-            mma16816(acc[j], va[u], b[0], b[1]);
-            mma16816(acc[j + 1], va[u], b[2], b[3]);
-            if (DELTA && p == 2) {
-              mma16816(acc[j], vr[u], b[0], b[1]);
-              mma16816(acc[j + 1], vr[u], b[2], b[3]);
+          for (int p = 0; p < 2; ++p) {
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const int row = u * 16 + (lm & 1) * 8 + lr, col = (j + 2 * e) * 8 + (lm >> 1) * 8;
+              ldsm4_trans(base + (uint32_t)(off_part(dkp, 2 + p) + row * qk_row(dkp) + col * 2), b[p][e]);
+            }
+          }
+#pragma unroll
+          for (int term = 0; term < (DELTA ? 3 : 2); ++term) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const uint32_t* k = b[term == 1 ? 1 : 0][e >> 1] + 2 * (e & 1);
+              mma16816(acc[j + e], term == 2 ? vr[u] : va[u], k[0], k[1]);
             }
           }
         }
